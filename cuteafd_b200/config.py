@@ -15,6 +15,67 @@ from typing import Any
 
 
 @dataclass(frozen=True)
+class LatentSpec:
+    """Latent attention of one layer: all heads' keys and values come out of a normed latent of ``kv_rank`` values plus one
+    shared rotated key part of ``rot_dim``; a query at position i sees the last ``window`` positions (0 = all of them)."""
+    heads: int
+    dim: int                             # unrotated query / key dims per head
+    rot_dim: int
+    vdim: int
+    kv_rank: int
+    window: int
+    scale: float
+    rope_base: float
+
+    @property
+    def record(self) -> int:
+        return self.kv_rank + self.rot_dim
+
+
+@dataclass(frozen=True)
+class DeltaSpec:
+    """Gated delta rule of one layer: per head a [dim, vdim] state; q / k heads are shared by ``heads // kv_heads`` heads;
+    q, k and v pass a causal convolution of ``conv`` taps."""
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    conv: int
+
+    @property
+    def conv_channels(self) -> int:
+        return 2 * self.kv_heads * self.dim + self.heads * self.vdim
+
+
+@dataclass(frozen=True)
+class RouterSpec:
+    """Routed feed-forward of one layer: ``experts`` SwiGLU experts of width ``ffn`` and ``identity`` outputs that hand the
+    input through; ``top`` of them per token out of the best ``groups_kept`` of ``groups``."""
+    experts: int
+    ffn: int
+    top: int
+    identity: int = 0
+    groups: int = 1
+    groups_kept: int = 1
+
+    @property
+    def outputs(self) -> int:
+        return self.experts + self.identity
+
+
+@dataclass(frozen=True)
+class LayerSpec:
+    mixer: Any                           # LatentSpec | DeltaSpec
+    router: RouterSpec | None = None     # None = the layer has no feed-forward
+
+    @staticmethod
+    def from_dict(d: dict[str, Any]) -> "LayerSpec":
+        m = d["mixer"]
+        mixer = LatentSpec(**m) if "kv_rank" in m else DeltaSpec(**m)
+        return LayerSpec(mixer, RouterSpec(**d["router"]) if d.get("router") else None)
+
+
+@dataclass(frozen=True)
 class ModelConfig:
     name: str = "tiny-moe"
     family: str = "deepseek_v3"          # deepseek_v3 | deepseek_v32 | qwen3_moe | glm4_moe | qwen2 | llama | tiny_moe
@@ -71,6 +132,11 @@ class ModelConfig:
     weight_format: str = "bf16"          # bf16 | fp8_block128 | nvfp4 | mxfp4 | exl3
     tie_embeddings: bool = False
     kv_format: str = "bf16"              # MLA cache record: bf16 (1152 bytes) | fp8_ds_mla (656 bytes; sparse attention only)
+    # per-layer designs (attention == "hybrid"): one LayerSpec per layer; the flat fields above then only summarise it
+    layer_specs: tuple = ()
+    canon_taps: int = 0                  # taps of the convolution every sublayer's input passes (0 = none)
+    norm_groups: int = 1                 # channel groups of the RMS norms
+    compute_dtype: str = "bf16"          # bf16 | f32 (every product and activation in 32-bit; hybrid engine only)
 
     # ---- derived -----------------------------------------------------------------
     @property
@@ -82,8 +148,31 @@ class ModelConfig:
         return self.qk_nope_dim + self.qk_rope_dim if self.is_mla else self.head_dim
 
     @property
+    def is_hybrid(self) -> bool:
+        return self.attention == "hybrid"
+
+    @property
+    def state_bytes(self) -> int:
+        """Recurrent state of one sequence (fp32): delta-rule states and the last inputs of every causal convolution."""
+        n = 0
+        for s in self.layer_specs:
+            n += (self.canon_taps - 1) * self.hidden * (2 if s.router is not None else 1)
+            if isinstance(s.mixer, DeltaSpec):
+                n += s.mixer.heads * s.mixer.dim * s.mixer.vdim + (s.mixer.conv - 1) * s.mixer.conv_channels
+        return 4 * n
+
+    def kv_elems_of(self, layer: int) -> int:
+        """Elements ``layer`` caches per token."""
+        if self.is_hybrid:
+            m = self.layer_specs[layer].mixer
+            return m.record if isinstance(m, LatentSpec) else 0
+        return self.kv_record_elems
+
+    @property
     def kv_record_elems(self) -> int:
-        """Elements cached per token per layer (latent+rope for MLA, K and V for GQA)."""
+        """Elements cached per token per layer (latent+rope for MLA, K and V for GQA; the average over a hybrid's layers)."""
+        if self.is_hybrid:
+            return -(-sum(self.kv_elems_of(i) for i in range(self.num_layers)) // max(1, self.num_layers))
         if self.is_mla:
             return self.kv_lora_rank + self.qk_rope_dim
         return 2 * self.num_kv_heads * self.head_dim
@@ -97,6 +186,8 @@ class ModelConfig:
 
     def window_of(self, layer: int) -> int:
         """Sliding window of ``layer`` in tokens; 0 = full causal attention."""
+        if self.is_hybrid:
+            return getattr(self.layer_specs[layer].mixer, "window", 0)
         if not self.sliding_window or self.is_mla:
             return 0
         if self.window_layers:
@@ -104,10 +195,21 @@ class ModelConfig:
         return self.sliding_window
 
     def is_moe_layer(self, layer: int) -> bool:
+        if self.is_hybrid:
+            return self.layer_specs[layer].router is not None
         return self.num_experts > 0 and layer >= self.first_dense_layers
+
+    def mixer_params(self, layer: int) -> int:
+        h, m = self.hidden, self.layer_specs[layer].mixer
+        if isinstance(m, LatentSpec):
+            return (h * (m.heads * (m.dim + m.rot_dim) + m.record + 2 * m.heads * m.vdim)
+                    + m.kv_rank * (1 + m.heads * (m.dim + m.vdim)))
+        return h * (m.conv_channels + 2 * m.heads + 2 * m.heads * m.vdim) + m.conv * m.conv_channels + 2 * m.heads + m.vdim
 
     def attention_params(self) -> int:
         h = self.hidden
+        if self.is_hybrid:
+            return sum(self.mixer_params(i) for i in range(self.num_layers)) // max(1, self.num_layers)
         if self.is_mla:
             q = (h * self.q_lora_rank + self.q_lora_rank * self.num_heads * self.qk_head_dim
                  if self.q_lora_rank else h * self.num_heads * self.qk_head_dim)
@@ -121,6 +223,12 @@ class ModelConfig:
         return 3 * self.hidden * self.expert_ffn
 
     def layer_params(self, layer: int) -> int:
+        if self.is_hybrid:
+            r = self.layer_specs[layer].router
+            p = self.mixer_params(layer) + (2 + self.canon_taps) * self.hidden
+            if r is not None:
+                p += (2 + self.canon_taps) * self.hidden + r.outputs * (self.hidden + 1) + 3 * r.experts * self.hidden * r.ffn
+            return p
         p = self.attention_params() + 2 * self.hidden
         if self.is_moe_layer(layer):
             p += self.num_experts * self.expert_params() + self.hidden * self.num_experts
@@ -139,7 +247,10 @@ class ModelConfig:
     @staticmethod
     def from_dict(d: dict[str, Any]) -> "ModelConfig":
         names = {f.name for f in dataclasses.fields(ModelConfig)}
-        return ModelConfig(**{k: v for k, v in d.items() if k in names})
+        d = {k: v for k, v in d.items() if k in names}
+        if d.get("layer_specs"):
+            d["layer_specs"] = tuple(v if isinstance(v, LayerSpec) else LayerSpec.from_dict(v) for v in d["layer_specs"])
+        return ModelConfig(**d)
 
     def replace(self, **kw: Any) -> "ModelConfig":
         return dataclasses.replace(self, **kw)
@@ -219,7 +330,39 @@ def kimi_k2() -> ModelConfig:
                                  rope_factor=32.0, rope_beta_fast=1.0, rope_beta_slow=1.0)
 
 
+def hybrid_config(name: str, vocab: int, hidden: int, specs, canon_taps: int, norm_groups: int, eps: float,
+                  family: str = "karusun") -> ModelConfig:
+    """ModelConfig of a per-layer design.  The flat fields carry the widest layer's values for code that only sizes
+    things (planner, reports); the engine reads the specs."""
+    specs = tuple(specs)
+    lat = [s.mixer for s in specs if isinstance(s.mixer, LatentSpec)]
+    routers = [s.router for s in specs if s.router is not None]
+    big = max(lat, key=lambda m: m.heads * (m.dim + m.rot_dim), default=None)
+    wide = max(routers, key=lambda r: r.experts * r.ffn, default=None)
+    return ModelConfig(
+        name=name, family=family, vocab_size=vocab, num_layers=len(specs), hidden=hidden, attention="hybrid", layer_specs=specs,
+        canon_taps=canon_taps, norm_groups=norm_groups, rms_eps=eps, rope_interleaved=False,
+        num_heads=max(s.mixer.heads for s in specs), num_kv_heads=1, head_dim=(big.dim + big.rot_dim) if big else specs[0].mixer.dim,
+        q_lora_rank=0, kv_lora_rank=big.kv_rank if big else 0, qk_nope_dim=big.dim if big else 0, qk_rope_dim=big.rot_dim if big else 0,
+        v_head_dim=big.vdim if big else specs[0].mixer.vdim, rope_theta=big.rope_base if big else 10000.0,
+        sliding_window=max((m.window for m in lat), default=0), dense_ffn=0, first_dense_layers=0,
+        num_experts=wide.experts if wide else 0, expert_ffn=wide.ffn if wide else 0, top_k=wide.top if wide else 0,
+        num_groups=wide.groups if wide else 1, topk_groups=wide.groups_kept if wide else 1, num_shared_experts=0,
+        norm_topk_prob=False, router_bias=bool(routers))
+
+
+def karusun_bench() -> ModelConfig:
+    """A Karusun-shaped stack at the sizes of a real model's layers (latent 512 + 64, heads of 128, 64 experts top-6 of which
+    the last eight hand their input through): three delta-rule layers to one latent attention layer."""
+    r = RouterSpec(experts=56, ffn=1024, top=6, identity=8, groups=8, groups_kept=4)
+    lat = LatentSpec(heads=32, dim=128, rot_dim=64, vdim=128, kv_rank=512, window=2048, scale=192 ** -0.5, rope_base=1.0e6)
+    delta = DeltaSpec(heads=32, kv_heads=16, dim=128, vdim=128, conv=4)
+    specs = [LayerSpec(lat if i % 4 == 3 else delta, r) for i in range(24)]
+    return hybrid_config("karusun-bench", 65536, 2048, specs, canon_taps=4, norm_groups=4, eps=1e-5)
+
+
 PRESETS = {
+    "karusun-bench": karusun_bench,
     "tiny-moe": tiny_moe,
     "mixtral-8x7b": mixtral_8x7b,
     "mistral-7b": mistral_7b,
@@ -233,6 +376,9 @@ PRESETS = {
 
 def scaled_down(cfg: ModelConfig, layers: int = 2, vocab: int = 2048) -> ModelConfig:
     """Same per-layer geometry with fewer layers and a small vocabulary (tests, smoke)."""
+    if cfg.is_hybrid:
+        return hybrid_config(cfg.name + "-mini", vocab, cfg.hidden, cfg.layer_specs[:layers], cfg.canon_taps, cfg.norm_groups,
+                             cfg.rms_eps, cfg.family)
     first_dense = min(cfg.first_dense_layers, max(layers - 1, 0)) if cfg.first_dense_layers else 0
     return cfg.replace(name=cfg.name + "-mini", num_layers=layers, vocab_size=vocab,
                        first_dense_layers=first_dense)

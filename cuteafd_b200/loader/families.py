@@ -144,6 +144,38 @@ class Qwen2(Family):
     id, model_types, attention = "qwen2", ("qwen2",), "gqa"
 
 
+class KarusunModel(FamilyModel):
+    """Tensor roles of the per-layer designs: ``l<i>.mix.*``, ``l<i>.mlp.*``, norms and input convolutions beside them."""
+    _LAYER = re.compile(r"l(\d+)\.(.*)")
+
+    def classify(self, name: str) -> tuple[str, int | None, int | None]:
+        if name in ("embed", "head", "final.norm"):
+            return {"embed": "embedding", "head": "head", "final.norm": "final_norm"}[name], None, None
+        m = self._LAYER.match(name)
+        if not m:
+            return "other", None, None
+        layer, rest = int(m.group(1)), m.group(2)
+        if rest.startswith("mix."):
+            return "attention", layer, None
+        e = re.match(r"mlp\.e(\d+)\.", rest)
+        if e:
+            return "routed_expert", layer, int(e.group(1))
+        if rest.startswith("mlp."):
+            return "router", layer, None
+        return ("norm" if rest.startswith(("norm", "canon")) else "other"), layer, None
+
+
+class Karusun(Family):
+    """Per-layer hybrids (windowed latent attention and gated delta-rule layers): served by the hybrid engine."""
+    id, model_types, attention = "karusun", ("karusun",), "hybrid"
+
+    def detect(self, hf_config: dict) -> bool:
+        return hf_config.get("architecture") == "Karusun"
+
+    def open(self, cfg: ModelConfig, hf_config: dict) -> FamilyModel:
+        return KarusunModel(self, cfg, ExpertContract(formats=("bf16",)))
+
+
 class TinyMoe(Family):
     id, model_types = "tiny_moe", ("tiny_moe",)
 
@@ -163,7 +195,7 @@ def canonical_name(name: str) -> str:
     return _MIXTRAL_RE.sub(lambda m: m.group(1) + _MIXTRAL_PROJ[m.group(2)] + m.group(3), name)
 
 
-REGISTRY: tuple[Family, ...] = (DeepseekV32(), DeepseekV3(), Qwen3Moe(), Glm4Moe(), Qwen2(), Llama(), TinyMoe())
+REGISTRY: tuple[Family, ...] = (DeepseekV32(), DeepseekV3(), Qwen3Moe(), Glm4Moe(), Qwen2(), Llama(), TinyMoe(), Karusun())
 
 
 def detect(hf_config: dict) -> Family | None:

@@ -12,7 +12,7 @@ import os
 
 import torch
 
-from ..config import ModelConfig
+from ..config import DeltaSpec, LatentSpec, LayerSpec, ModelConfig, RouterSpec, hybrid_config
 from ..ref.model import init_weights
 from . import formats
 from .safetensors_io import write_sharded
@@ -22,7 +22,60 @@ ARCH = {"llama": "LlamaForCausalLM", "qwen3_moe": "Qwen3MoeForCausalLM", "deepse
         "qwen2": "Qwen2ForCausalLM"}
 
 
+def _layer_list_to_json(cfg: ModelConfig) -> dict:
+    """config.json of a per-layer design (the ``layers`` list form)."""
+    layers = []
+    for s in cfg.layer_specs:
+        m, r = s.mixer, s.router
+        if isinstance(m, LatentSpec):
+            e = {"type": "latent_attention", "mixer": {
+                "heads": m.heads, "dim": m.dim, "rot_dim": m.rot_dim, "vdim": m.vdim, "kv_rank": m.kv_rank, "scale": m.scale,
+                "mask": {"size": m.window}, "rot": {"base": m.rope_base, "dims": m.rot_dim}}}
+        else:
+            e = {"type": "delta", "mixer": {"heads": m.heads, "kv_heads": m.kv_heads, "dim": m.dim, "vdim": m.vdim, "conv": m.conv}}
+        e["mlp"] = None if r is None else {"kind": "moe", "expert": {"ff": r.ffn}, "router": {
+            "experts": r.experts, "identity": r.identity, "top": r.top, "groups": {"count": r.groups, "keep": r.groups_kept}}}
+        layers.append(e)
+    return {"architecture": "Karusun", "name": cfg.name, "vocab": cfg.vocab_size, "width": cfg.hidden, "layers": layers,
+            "canon": {"taps": cfg.canon_taps}, "norm": {"eps": cfg.rms_eps, "groups": cfg.norm_groups}}
+
+
+def _layer_list_from_json(d: dict) -> ModelConfig:
+    """The ``layers`` list form of config.json.  Every layer carries its own sizes; a type or kind that is not built is
+    refused by name."""
+    specs = []
+    for i, e in enumerate(d["layers"]):
+        m, mlp = e["mixer"], e.get("mlp")
+        if e["type"] == "latent_attention":
+            rot = m["rot"]
+            if rot.get("dims", m["rot_dim"]) != m["rot_dim"]:
+                raise ValueError(f"layer {i}: {rot['dims']} rotated dims of a rotated part of {m['rot_dim']} are not supported")
+            mixer = LatentSpec(heads=m["heads"], dim=m["dim"], rot_dim=m["rot_dim"], vdim=m["vdim"], kv_rank=m["kv_rank"],
+                               window=m["mask"]["size"], scale=float(m["scale"]), rope_base=float(rot["base"]))
+        elif e["type"] == "delta":
+            mixer = DeltaSpec(heads=m["heads"], kv_heads=m.get("kv_heads", m["heads"]), dim=m["dim"], vdim=m["vdim"], conv=m["conv"])
+            if mixer.heads % mixer.kv_heads:
+                raise ValueError(f"layer {i}: {mixer.heads} heads over {mixer.kv_heads} key heads")
+        else:
+            raise ValueError(f"layer {i}: unsupported mixer {e['type']!r}")
+        router = None
+        if mlp is not None:
+            if mlp.get("kind") != "moe":
+                raise ValueError(f"layer {i}: unsupported feed-forward {mlp.get('kind')!r}")
+            r = mlp["router"]
+            g = r.get("groups") or {"count": 1, "keep": 1}
+            router = RouterSpec(experts=r["experts"], ffn=mlp["expert"]["ff"], top=r["top"], identity=r.get("identity", 0) or 0,
+                                groups=g["count"], groups_kept=g["keep"])
+            if router.outputs % router.groups:
+                raise ValueError(f"layer {i}: {router.outputs} router outputs in {router.groups} groups")
+        specs.append(LayerSpec(mixer, router))
+    return hybrid_config(d.get("name", d["architecture"].lower()), d["vocab"], d["width"], specs, d["canon"]["taps"],
+                         d["norm"].get("groups", 1), float(d["norm"]["eps"]))
+
+
 def to_hf_config(cfg: ModelConfig) -> dict:
+    if cfg.is_hybrid:
+        return _layer_list_to_json(cfg)
     d = {"architectures": [ARCH.get(cfg.family, "DeepseekV3ForCausalLM")], "model_type": cfg.family,
          "vocab_size": cfg.vocab_size, "hidden_size": cfg.hidden, "num_hidden_layers": cfg.num_layers,
          "num_attention_heads": cfg.num_heads, "rms_norm_eps": cfg.rms_eps, "rope_theta": cfg.rope_theta,
@@ -116,6 +169,8 @@ def _rope_scaling(d: dict) -> dict:
 
 def from_hf_config(d: dict) -> ModelConfig:
     """Map a config.json onto the engine's geometry.  Unknown architectures raise ValueError."""
+    if d.get("architecture") == "Karusun":
+        return _layer_list_from_json(d)
     mt = d.get("model_type", "")
     extra = d.get("cuteafd", {})
     q = d.get("quantization_config") or {}
@@ -241,6 +296,15 @@ def write_random_snapshot(cfg: ModelConfig, directory: str, fmt: str | None = No
     ``scope`` = "experts": only routed experts carry the quantised format (the usual shipped
     mix); "linear": every projection does (DeepSeek FP8 style)."""
     fmt = fmt or cfg.weight_format
+    if cfg.is_hybrid:
+        if fmt != "bf16":
+            raise ValueError(f"per-layer designs are stored in bf16, not {fmt}")
+        from ..ref.hybrid import init_hybrid_weights
+        os.makedirs(directory, exist_ok=True)
+        with open(os.path.join(directory, "config.json"), "w") as f:
+            json.dump(to_hf_config(cfg), f, indent=1, sort_keys=True)
+        write_sharded(directory, {k: v.to(torch.bfloat16) for k, v in init_hybrid_weights(cfg, seed).items()}, shard_bytes)
+        return directory
     cfg = cfg.replace(weight_format=fmt if not fmt.startswith("exl3") else "exl3")
     params = init_weights(cfg, seed=seed)
     gen = torch.Generator().manual_seed(seed + 17)

@@ -1,0 +1,291 @@
+"""CPU oracle of the per-layer hybrid decoders (``ModelConfig.layer_specs``): windowed latent attention layers and gated
+delta-rule layers in any order, each behind grouped RMS norms, input convolutions and a routed feed-forward.
+
+One function per mechanism, written as the equations read: no chunking, no absorbed products, one token at a time where a
+recurrence runs.  ``HybridRefDecoder`` strings them together over a parameter dictionary in the checkpoint's own tensor
+names and plugs into the same places as ``RefDecoder``.  All arithmetic is in the dtype the parameters are given in
+(fp32 or fp64); nothing here is shared with the CUDA path.
+"""
+from __future__ import annotations
+
+import torch
+
+from ..config import DeltaSpec, LatentSpec, ModelConfig, RouterSpec
+
+Params = dict[str, torch.Tensor]
+
+
+# ---- mechanisms -----------------------------------------------------------------------------------------------------
+def rms(x: torch.Tensor, eps: float) -> torch.Tensor:
+    """x / sqrt(mean(x^2) + eps) over the last dimension."""
+    return x / torch.sqrt((x * x).mean(-1, keepdim=True) + eps)
+
+
+def group_rms(x: torch.Tensor, w: torch.Tensor, groups: int, eps: float) -> torch.Tensor:
+    """RMS norm in ``groups`` equal runs of channels, each with its own root mean square; one weight per channel."""
+    parts = x.reshape(*x.shape[:-1], groups, x.shape[-1] // groups)
+    return rms(parts, eps).reshape(x.shape) * w
+
+
+def causal_conv(x: torch.Tensor, w: torch.Tensor, past: torch.Tensor) -> tuple[torch.Tensor, torch.Tensor]:
+    """Per-channel causal convolution over time.  x [T, C], w [C, taps] (last column = the current token), ``past``
+    [taps - 1, C] the inputs just before x.  Returns (y [T, C], the new past)."""
+    taps, T = w.shape[1], x.shape[0]
+    full = torch.cat([past, x])
+    y = torch.zeros_like(x)
+    for j in range(taps):
+        y = y + w[:, j] * full[j:j + T]
+    return y, full[T:]
+
+
+def rotate_half(x: torch.Tensor, positions: torch.Tensor, base: float) -> torch.Tensor:
+    """x [T, ..., d]: dimension i is paired with i + d/2 and turned by position * base^(-2i/d)."""
+    d = x.shape[-1]
+    f = torch.tensor([base ** (-2.0 * i / d) for i in range(d // 2)], dtype=x.dtype)
+    a = positions.to(x.dtype)[:, None] * f
+    a = a.reshape(a.shape[0], *([1] * (x.dim() - 2)), d // 2)
+    u, v = x[..., :d // 2], x[..., d // 2:]
+    return torch.cat([u * a.cos() - v * a.sin(), v * a.cos() + u * a.sin()], -1)
+
+
+def window_attention(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, start: int, window: int, scale: float) -> torch.Tensor:
+    """Softmax attention; q [T, H, Dk] at positions start.., k [L, H, Dk], v [L, H, Dv] at positions 0..; a query at
+    position i sees j with 0 <= i - j < window."""
+    out = []
+    for t in range(q.shape[0]):
+        i = start + t
+        lo = max(0, i - window + 1)
+        s = torch.einsum("hd,jhd->hj", q[t], k[lo:i + 1]) * scale
+        out.append(torch.einsum("hj,jhd->hd", torch.softmax(s, -1), v[lo:i + 1]))
+    return torch.stack(out)
+
+
+def delta_recurrence(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, beta: torch.Tensor, g: torch.Tensor,
+                     S: torch.Tensor) -> tuple[torch.Tensor, torch.Tensor]:
+    """Gated delta rule.  q, k [T, H, D], v [T, H, Dv], beta, g [T, H], S [H, D, Dv].  Per token: decay the state, move
+    what it holds under k towards v by beta, read with q (the read sees this token's write)."""
+    out = []
+    for t in range(q.shape[0]):
+        S = g[t][:, None, None] * S
+        u = beta[t][:, None] * (v[t] - torch.einsum("hdv,hd->hv", S, k[t]))
+        S = S + torch.einsum("hd,hv->hdv", k[t], u)
+        out.append(torch.einsum("hdv,hd->hv", S, q[t]))
+    return torch.stack(out), S
+
+
+def unit(x: torch.Tensor) -> torch.Tensor:
+    return x / torch.sqrt((x * x).sum(-1, keepdim=True) + 1e-6)
+
+
+def silu(x: torch.Tensor) -> torch.Tensor:
+    return x * torch.sigmoid(x)
+
+
+def route(h: torch.Tensor, w: torch.Tensor, correction: torch.Tensor, r: RouterSpec) -> tuple[torch.Tensor, torch.Tensor]:
+    """Softmax scores over experts and identity experts; the choice goes by score + correction inside the best groups
+    (a group counts by its best member); the weights are the plain scores.  Returns (ids [T, top], weights [T, top])."""
+    s = torch.softmax(h @ w.T, -1)
+    ids, wts = [], []
+    n = s.shape[1]
+    for t in range(s.shape[0]):
+        choice = s[t] + correction
+        per = n // r.groups
+        best = [(max(choice[g * per:(g + 1) * per].tolist()), -g) for g in range(r.groups)]
+        kept = {-g for _, g in sorted(best, reverse=True)[:r.groups_kept]}
+        order = sorted((e for e in range(n) if e // per in kept), key=lambda e: (-float(choice[e]), e))[:r.top]
+        ids.append(order)
+        wts.append(s[t][order])
+    return torch.tensor(ids), torch.stack(wts)
+
+
+def routed_ffn(h: torch.Tensor, p: Params, pre: str, r: RouterSpec) -> torch.Tensor:
+    ids, wts = route(h, p[pre + "router"], p[pre + "correction"], r)
+    y = torch.zeros_like(h)
+    for e in ids.unique().tolist():
+        t, slot = (ids == e).nonzero(as_tuple=True)
+        x = h[t]
+        if e < r.experts:
+            x = (silu(x @ p[f"{pre}e{e}.gate"].T) * (x @ p[f"{pre}e{e}.up"].T)) @ p[f"{pre}e{e}.down"].T
+        y[t] += wts[t, slot][:, None] * x
+    return y
+
+
+# ---- mixers ---------------------------------------------------------------------------------------------------------
+def latent_mixer(h: torch.Tensor, p: Params, pre: str, m: LatentSpec, eps: float, start: int, st: dict) -> torch.Tensor:
+    """Latent attention: keys and values of every head come out of one normed latent per token; a shared rotated key part."""
+    T = h.shape[0]
+    pos = torch.arange(start, start + T)
+    q = (h @ p[pre + "q"].T).view(T, m.heads, m.dim + m.rot_dim)
+    q = torch.cat([q[..., :m.dim], rotate_half(q[..., m.dim:], pos, m.rope_base)], -1)
+    d = h @ p[pre + "dkv"].T
+    c = rms(d[:, :m.kv_rank], eps) * p[pre + "dkv.norm"]
+    kr = rotate_half(d[:, m.kv_rank:], pos, m.rope_base)
+    st["c"] = torch.cat([st["c"], c])
+    st["kr"] = torch.cat([st["kr"], kr])
+    L = st["c"].shape[0]
+    k = (st["c"] @ p[pre + "uk"].T).view(L, m.heads, m.dim)
+    k = torch.cat([k, st["kr"][:, None].expand(L, m.heads, m.rot_dim)], -1)
+    v = (st["c"] @ p[pre + "uv"].T).view(L, m.heads, m.vdim)
+    o = window_attention(q, k, v, start, m.window, m.scale).reshape(T, m.heads * m.vdim)
+    return (o * torch.sigmoid(h @ p[pre + "g"].T)) @ p[pre + "o"].T
+
+
+def delta_mixer(h: torch.Tensor, p: Params, pre: str, m: DeltaSpec, eps: float, st: dict) -> torch.Tensor:
+    T = h.shape[0]
+    x = {}
+    for n in ("q", "k", "v"):
+        y, st["conv." + n] = causal_conv(h @ p[pre + n].T, p[pre + n + ".conv"], st["conv." + n])
+        x[n] = silu(y)
+    rep = m.heads // m.kv_heads
+    q = unit(x["q"].view(T, m.kv_heads, m.dim)).repeat_interleave(rep, 1) * m.dim ** -0.5
+    k = unit(x["k"].view(T, m.kv_heads, m.dim)).repeat_interleave(rep, 1)
+    v = x["v"].view(T, m.heads, m.vdim)
+    beta = torch.sigmoid(h @ p[pre + "b"].T)
+    a = h @ p[pre + "a"].T + p[pre + "dt_bias"]
+    g = torch.exp(-torch.exp(p[pre + "A_log"]) * torch.log1p(torch.exp(-a.abs())).add(a.clamp_min(0)))
+    o, st["S"] = delta_recurrence(q, k, v, beta, g, st["S"])
+    o = rms(o, eps) * p[pre + "norm"]
+    o = o.reshape(T, m.heads * m.vdim) * silu(h @ p[pre + "g"].T)
+    return o @ p[pre + "o"].T
+
+
+# ---- state ----------------------------------------------------------------------------------------------------------
+class HybridState:
+    """What one sequence carries: latent records per position, and the recurrent parts.  The recurrent parts cannot be
+    cut back, so the state keeps a copy per token of the last call; ``truncate`` returns to one of them."""
+
+    def __init__(self, cfg: ModelConfig, dtype: torch.dtype = torch.float32):
+        self.length_ = 0
+        self.layers: list[dict] = []
+        self.marks: dict[int, list[dict]] = {}
+        for spec in cfg.layer_specs:
+            z = lambda *s: torch.zeros(*s, dtype=dtype)               # noqa: E731
+            st = {"canon1": z(cfg.canon_taps - 1, cfg.hidden), "canon2": z(cfg.canon_taps - 1, cfg.hidden)}
+            m = spec.mixer
+            if isinstance(m, LatentSpec):
+                st.update(c=z(0, m.kv_rank), kr=z(0, m.rot_dim))
+            else:
+                st.update(S=z(m.heads, m.dim, m.vdim))
+                for n, c in (("q", m.kv_heads * m.dim), ("k", m.kv_heads * m.dim), ("v", m.heads * m.vdim)):
+                    st["conv." + n] = z(m.conv - 1, c)
+            self.layers.append(st)
+
+    def length(self, layer: int = 0) -> int:
+        return self.length_
+
+    @property
+    def rows(self) -> list[list[torch.Tensor]]:
+        """Every tensor of the state, per layer (state hashes)."""
+        return [[st[k] for k in sorted(st)] for st in self.layers]
+
+    def truncate(self, length: int) -> None:
+        if length == self.length_:
+            return
+        if length not in self.marks:
+            raise ValueError(f"recurrent state at {self.length_} tokens cannot return to {length}")
+        self.layers = [dict(st) for st in self.marks[length]]
+        self.length_ = length
+
+
+# ---- whole model ----------------------------------------------------------------------------------------------------
+class HybridRefDecoder:
+    def __init__(self, cfg: ModelConfig, params: Params, mark_rows: int = 16):
+        self.cfg, self.p = cfg, params
+        self.usage = None
+        self.moe_fn = None
+        self.mark_rows = mark_rows        # calls of at most this many tokens keep a state per token (``truncate``)
+        self.trace: list | None = None    # residual after every layer, when set to a list
+
+    def new_state(self) -> HybridState:
+        return HybridState(self.cfg, self.p["embed"].dtype)
+
+    def _layer(self, i: int, x: torch.Tensor, start: int, st: dict) -> torch.Tensor:
+        cfg, p, spec, pre = self.cfg, self.p, self.cfg.layer_specs[i], f"l{i}."
+
+        def sublayer(x, n, fn):
+            h = group_rms(x, p[f"{pre}norm{n}"], cfg.norm_groups, cfg.rms_eps)
+            y, st[f"canon{n}"] = causal_conv(h, p[f"{pre}canon{n}"], st[f"canon{n}"])
+            return x + group_rms(fn(h + y), p[f"{pre}norm{n}b"], cfg.norm_groups, cfg.rms_eps)
+
+        m = spec.mixer
+        if isinstance(m, LatentSpec):
+            x = sublayer(x, 1, lambda h: latent_mixer(h, p, pre + "mix.", m, cfg.rms_eps, start, st))
+        else:
+            x = sublayer(x, 1, lambda h: delta_mixer(h, p, pre + "mix.", m, cfg.rms_eps, st))
+        if spec.router is not None:
+            x = sublayer(x, 2, lambda h: routed_ffn(h, p, pre + "mlp.", spec.router))
+        return x
+
+    def _run(self, tokens: torch.Tensor, kv: HybridState) -> torch.Tensor:
+        x, start = self.p["embed"][tokens], kv.length_
+        for i in range(len(self.cfg.layer_specs)):
+            x = self._layer(i, x, start, kv.layers[i])
+            if self.trace is not None:
+                self.trace.append(x)
+        kv.length_ = start + tokens.shape[0]
+        return x
+
+    def hidden_states(self, tokens: torch.Tensor, kv: HybridState, embeds: tuple | None = None) -> torch.Tensor:
+        if embeds is not None:
+            raise ValueError("media rows are not part of this family")
+        kv.marks = {kv.length_: [dict(st) for st in kv.layers]}
+        if tokens.shape[0] > self.mark_rows:
+            return self._run(tokens, kv)
+        out = []
+        for t in range(tokens.shape[0]):
+            out.append(self._run(tokens[t:t + 1], kv))
+            kv.marks[kv.length_] = [dict(st) for st in kv.layers]
+        return torch.cat(out)
+
+    def head(self, x: torch.Tensor) -> torch.Tensor:
+        return group_rms(x, self.p["final.norm"], self.cfg.norm_groups, self.cfg.rms_eps) @ self.p["head"].T
+
+    def forward(self, tokens: torch.Tensor, kv: HybridState, embeds: tuple | None = None) -> torch.Tensor:
+        return self.head(self.hidden_states(tokens, kv, embeds))
+
+
+def init_hybrid_weights(cfg: ModelConfig, seed: int = 0, dtype: torch.dtype = torch.float32, std: float | None = None) -> Params:
+    """Random parameters under the checkpoint's tensor names, scaled so that every branch matters."""
+    g = torch.Generator().manual_seed(seed)
+
+    def w(*shape: int, s: float | None = None) -> torch.Tensor:
+        return (torch.randn(*shape, generator=g) * (s if s is not None else std if std is not None else shape[-1] ** -0.5)).to(dtype)
+
+    def near_one(n: int) -> torch.Tensor:
+        return (1 + 0.2 * torch.randn(n, generator=g)).to(dtype)
+
+    H = cfg.hidden
+    p: Params = {"embed": w(cfg.vocab_size, H, s=1.0), "final.norm": near_one(H), "head": w(cfg.vocab_size, H)}
+    for i, spec in enumerate(cfg.layer_specs):
+        pre, m, r = f"l{i}.", spec.mixer, spec.router
+        for n in ("norm1", "norm1b") + (("norm2", "norm2b") if r is not None else ()):
+            p[pre + n] = near_one(H)
+        for n in ("canon1",) + (("canon2",) if r is not None else ()):
+            p[pre + n] = w(H, cfg.canon_taps, s=0.3)
+        x = pre + "mix."
+        if isinstance(m, LatentSpec):
+            p.update({x + "q": w(m.heads * (m.dim + m.rot_dim), H), x + "dkv": w(m.kv_rank + m.rot_dim, H),
+                      x + "dkv.norm": near_one(m.kv_rank), x + "uk": w(m.heads * m.dim, m.kv_rank),
+                      x + "uv": w(m.heads * m.vdim, m.kv_rank), x + "g": w(m.heads * m.vdim, H)})
+        else:
+            kd, vd = m.kv_heads * m.dim, m.heads * m.vdim
+            p.update({x + "q": w(kd, H), x + "k": w(kd, H), x + "v": w(vd, H), x + "g": w(vd, H), x + "b": w(m.heads, H),
+                      x + "a": w(m.heads, H), x + "A_log": w(m.heads, s=0.5), x + "dt_bias": w(m.heads, s=1.0) - 2,
+                      x + "norm": near_one(m.vdim), x + "q.conv": w(kd, m.conv), x + "k.conv": w(kd, m.conv), x + "v.conv": w(vd, m.conv)})
+        p[x + "o"] = w(H, m.heads * m.vdim)
+        if r is not None:
+            x = pre + "mlp."
+            p[x + "router"] = w(r.experts + r.identity, H)
+            p[x + "correction"] = w(r.experts + r.identity, s=0.1)
+            for e in range(r.experts):
+                p[f"{x}e{e}.gate"], p[f"{x}e{e}.up"], p[f"{x}e{e}.down"] = w(r.ffn, H), w(r.ffn, H), w(H, r.ffn)
+    return p
+
+
+def bf16_params(p: Params, dtype: torch.dtype = torch.float32) -> Params:
+    """The parameters as a bfloat16 checkpoint holds them."""
+    return {k: v.to(torch.bfloat16).to(dtype) for k, v in p.items()}
+
+
+__all__ = ["HybridRefDecoder", "HybridState", "init_hybrid_weights", "bf16_params", "group_rms", "causal_conv", "rotate_half",
+           "window_attention", "delta_recurrence", "route", "routed_ffn", "latent_mixer", "delta_mixer", "rms", "unit"]
