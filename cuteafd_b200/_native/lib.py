@@ -76,6 +76,39 @@ class MoeLayout(C.Structure):
     ]
 
 
+class NormArgs(C.Structure):
+    """cafd_norm_conv (csrc/hybrid_norm.cu)."""
+    _fields_ = [(n, C.c_void_p) for n in ("tokens", "embed", "x_in", "y", "slot_w", "slot_idx", "ident", "w_b", "w", "conv", "x_out",
+                                          "h_out", "row_idx", "state", "state_in", "state_out", "q_start")]
+    _fields_ += [("slot_stride", C.c_longlong), ("state_off", C.c_longlong)]
+    _fields_ += [(n, C.c_int) for n in ("T", "H", "S", "ldy", "groups", "taps", "top_k", "n_experts", "vocab", "run")] + [("eps", C.c_float)]
+
+
+class LatentPrep(C.Structure):
+    """cafd_latent_prep (csrc/latent.cu)."""
+    _fields_ = [(n, C.c_void_p) for n in ("a", "norm_w", "inv_freq", "positions", "slots", "cache", "slab", "q_abs", "lat_out")]
+    _fields_ += [(n, C.c_int) for n in ("lda", "q_off", "kv_off", "heads", "dim", "rot", "rank", "rec", "dim_pad", "t_pad", "T")]
+    _fields_ += [("eps", C.c_float)]
+
+
+class LatentAttn(C.Structure):
+    """cafd_latent_attn (csrc/latent.cu)."""
+    _fields_ = [(n, C.c_void_p) for n in ("q_abs", "cache", "page_table", "positions", "q_start", "out")]
+    _fields_ += [(n, C.c_int) for n in ("T", "S", "heads", "rank", "rot", "rec", "max_pages", "window", "t_pad", "out_ld",
+                                        "heads_per_block")]
+    _fields_ += [("scale", C.c_float)]
+
+
+class DeltaArgs(C.Structure):
+    """cafd_delta_step (csrc/delta.cu)."""
+    _fields_ = [(n, C.c_void_p) for n in ("proj", "conv_w", "A_log", "dt_bias", "norm_w", "state", "state_in", "state_out", "q_start",
+                                          "out", "raw")]
+    _fields_ += [(n, C.c_longlong) for n in ("slot_stride", "s_off", "c_off")]
+    _fields_ += [(n, C.c_int) for n in ("ld", "q_off", "k_off", "v_off", "g_off", "b_off", "a_off", "T", "S", "heads", "kv_heads", "dim",
+                                        "vdim", "taps", "out_vd")]
+    _fields_ += [("eps", C.c_float)]
+
+
 class TpReduceArgs(C.Structure):
     _fields_ = [
         ("partials", C.c_void_p), ("residual", C.c_void_p), ("norm_w", C.c_void_p), ("x_out", C.c_void_p * 8),
@@ -126,7 +159,7 @@ def cuda_lib():
         _sig(lib, "cafd_argmax_slices", [])
         _sig(lib, "cafd_bump_epoch", [P, P])
         _sig(lib, "cafd_decode_advance", [P, P, P, P, P, P, I, I, I, P])
-        _sig(lib, "cafd_route_topk", [P, P, P, P, I, I, I, I, I, I, I, F, P])
+        _sig(lib, "cafd_route_topk", [P, P, P, P, I, I, I, I, I, I, I, F, I, P])
         _sig(lib, "cafd_moe_meta_ints", [I, I])
         _sig(lib, "cafd_wait_flag", [P, P, P, P])
         _sig(lib, "cafd_tp_reduce_norm_gather", [C.POINTER(TpReduceArgs), P])
@@ -140,7 +173,7 @@ def cuda_lib():
         _sig(lib, "cafd_moe_plan_wide", [P, I, I, I, I, C.POINTER(MoeLayout), P, P, P, P, P])
         _sig(lib, "cafd_moe_plan_wide_ints", [I, I])
         _sig(lib, "cafd_moe_plan_dispatch", [P, I, I, I, I, C.POINTER(MoeLayout), P, P, P, P, I, P, P])
-        _sig(lib, "cafd_norm_route", [P, P, F, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, F, P])
+        _sig(lib, "cafd_norm_route", [P, P, F, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, F, I, P])
         _sig(lib, "cafd_moe_combine_norm", [P, P, P, P, P, I, I, I, P, I, P, P, P, F, P, P])
         _sig(lib, "cafd_moe_dispatch", [P, P, P, I, I, I, C.POINTER(MoeLayout), P, P, P])
         _sig(lib, "cafd_moe_combine", [P, P, P, P, P, I, I, I, P, I, P, P, P])
@@ -152,7 +185,7 @@ def cuda_lib():
         _sig(lib, "cafd_fixed_kv_split", [])
         _sig(lib, "cafd_attn_prefill", [P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, F, I, P])
         _sig(lib, "cafd_mla_scratch_floats", [I, I], C.c_longlong)
-        _sig(lib, "cafd_mla_attention", [P, P, P, P, P, P, P, P, P, P, C.c_longlong, I, I, I, I, I, I, F, P, I, P])
+        _sig(lib, "cafd_mla_attention", [P, P, P, P, P, P, P, P, P, P, C.c_longlong, I, I, I, I, I, I, F, P, I, I, P])
         _sig(lib, "cafd_indexer_scores", [P, P, P, I, F, P, P, P, P, P, P, P, C.c_longlong, I, I, I, I, I, I, P])
         _sig(lib, "cafd_index_topk", [P, I, P, P, P, I, I, I, P, P])
         _sig(lib, "cafd_index_k_store", [P, I, P, P, I, P])
@@ -162,13 +195,20 @@ def cuda_lib():
         _sig(lib, "cafd_mla_attention_partial", [P, P, P, P, P, P, P, P, P, I, I, P, C.c_longlong, I, I, I, I, I, F, P])
         _sig(lib, "cafd_mla_merge", [P, P, P, P, P, I, I, I, I, P])
         _sig(lib, "cafd_mla_attention_gathered", [P, P, P, P, P, P, P, P, P, P, C.c_longlong, I, I, I, I, I, F, P, I, P])
-        _sig(lib, "cafd_attn_prefill_mla", [P, I, P, I, I, P, P, C.c_longlong, P, P, P, P, P, P, P, I, I, I, I, I, I, F, P])
+        _sig(lib, "cafd_attn_prefill_mla", [P, I, I, P, I, I, P, P, C.c_longlong, P, P, P, P, P, P, P, I, I, I, I, I, I, F, I, P])
         _sig(lib, "cafd_gemm_w4", [C.POINTER(GemmArgs), I, P, P, P])
         _sig(lib, "cafd_w4_dequant", [P, P, P, P, C.c_longlong, I, I, I, P])
         _sig(lib, "cafd_fp8_dequant_block128", [P, P, P, C.c_longlong, I, P])
         _sig(lib, "cafd_gemm_exl3", [P, I, P, P, P, P, P, I, P, P, P, I, I, I, I, I, I, P])
         _sig(lib, "cafd_sample_rows", [P, I, I, P, P, I, P, P, P])
         _sig(lib, "cafd_accept_prefix", [P, P, P, I, P, P, P])
+        _sig(lib, "cafd_norm_conv", [C.POINTER(NormArgs), I, P])
+        _sig(lib, "cafd_swap_ids", [P, P, I, P])
+        _sig(lib, "cafd_gemm_f32", [P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, P])
+        _sig(lib, "cafd_latent_prep", [C.POINTER(LatentPrep), I, P])
+        _sig(lib, "cafd_latent_attn", [C.POINTER(LatentAttn), I, P])
+        _sig(lib, "cafd_latent_gate", [P, P, I, I, I, I, I, I, I, P])
+        _sig(lib, "cafd_delta_step", [C.POINTER(DeltaArgs), I, P])
         _sig(lib, "cafd_mla_q_split", [P, I, P, P, P, P, I, I, I, I, P])
         _sig(lib, "cafd_mla_small_rows", [])
         _sig(lib, "cafd_mla_absorb_small", [P, I, P, P, P, P, I, I, I, P])

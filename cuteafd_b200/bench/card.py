@@ -70,9 +70,19 @@ def device_decode_loop(gen: Generator, seqs, last_tokens: list[int], steps: int,
         b.seq_lens[0][i] = s.kv_len + 1
         b.q_start[0][i] = i
     b.q_start[0][S] = S
+    outs, extra = [], {}
+    if gen.states is not None:               # the loop alternates two private slots per stream; forks share their base's slot
+        for s in seqs:
+            own = gen.states.alloc()
+            eng.kv.state[own].copy_(eng.kv.state[s.state])
+            gen.states.release(s.state)
+            s.state = own
+        ins, outs = gen.states.begin(seqs)
+        b.set_states(ins, outs)
+        extra = b.states(S)
     b.upload()
     batch = Batch(b.tokens[1][:S], b.positions[1][:S], b.slots[1][:S], b.page_table[1].view(S, gen.max_pages),
-                  b.seq_lens[1][:S], b.q_start[1][:S + 1], 1, False, None)
+                  b.seq_lens[1][:S], b.q_start[1][:S + 1], 1, False, None, **extra)
 
     def step():
         if hasattr(eng, "decode_step"):          # forward + selection + device-side advance, one launch where the engine fuses it
@@ -109,6 +119,9 @@ def device_decode_loop(gen: Generator, seqs, last_tokens: list[int], steps: int,
     assert K.read_status() == 0, "a bounded wait ran out during the timed region"
     for s in seqs:                           # account for the tokens the device loop appended
         s.kv_len += warmup + steps
+        s.state_len = s.kv_len
+    if outs:
+        gen.states.abort(outs)
     return ms, launches
 
 

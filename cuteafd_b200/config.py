@@ -248,6 +248,8 @@ class ModelConfig:
     def from_dict(d: dict[str, Any]) -> "ModelConfig":
         names = {f.name for f in dataclasses.fields(ModelConfig)}
         d = {k: v for k, v in d.items() if k in names}
+        if "window_layers" in d:
+            d["window_layers"] = tuple(d["window_layers"])
         if d.get("layer_specs"):
             d["layer_specs"] = tuple(v if isinstance(v, LayerSpec) else LayerSpec.from_dict(v) for v in d["layer_specs"])
         return ModelConfig(**d)

@@ -434,22 +434,24 @@ extern "C" int cafd_attn_prefill(const void* q, const void* k_cache, const void*
   return static_cast<int>(cudaGetLastError());
 }
 
-// MLA prefill in expanded form.  q_nope [total_q, heads * q_head_stride] bf16 (the first 128 columns of every head);
+// MLA prefill in expanded form.  q_nope [total_q, heads * q_head_stride] bf16, q_pitch elements from row to row (the first
+// 128 columns of every head);
 // q_rope [total_q, heads * qr_head_stride] bf16 with the rotated 64 rope dims of head h at column
 // h * qr_head_stride + qr_col0; k_exp / v_exp [tmp_rows, heads * 128] bf16 = per-head K_nope / V of every cached
 // token of the sequences, sequence s starting at row kv_tmp_start[s] (a multiple of 64); latent cache
 // [num_pages, 64, 576] supplies the shared rope keys (columns 512..575) through the page table.
 // out [total_q, heads, 128].
-extern "C" int cafd_attn_prefill_mla(const void* q_nope, int q_head_stride, const void* q_rope, int qr_head_stride, int qr_col0,
+extern "C" int cafd_attn_prefill_mla(const void* q_nope, int q_pitch, int q_head_stride, const void* q_rope, int qr_head_stride, int qr_col0,
                                      const void* k_exp, const void* v_exp, long long tmp_rows, const int* kv_tmp_start,
                                      const void* latent_cache, const int* page_table, const int* seq_lens, const int* q_start,
                                      void* out, uint32_t* status, int total_q, int num_seqs, int max_q_len, int num_pages,
-                                     int max_pages, int heads, float scale, cafd_stream_t s) {
+                                     int max_pages, int heads, float scale, int window, cafd_stream_t s) {
   if (num_seqs <= 0 || total_q <= 0) return 0;
+  if (window < 0 || q_pitch < heads * q_head_stride || (q_pitch % 8)) return -10;
   if (tmp_rows % kPageTok || (q_head_stride % 8) || (qr_head_stride % 8) || (qr_col0 % 8)) return -10;
   CUtensorMap tq, tqr, tk, tv, tkr;
   int rc = cached_tmap_2d(&tq, q_nope, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, total_q, static_cast<uint64_t>(heads) * q_head_stride,
-                          static_cast<uint64_t>(heads) * q_head_stride * 2, kBQ, 64);
+                          static_cast<uint64_t>(q_pitch) * 2, kBQ, 64);
   if (rc) return rc;
   rc = cached_tmap_2d(&tqr, q_rope, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, total_q, static_cast<uint64_t>(heads) * qr_head_stride,
                       static_cast<uint64_t>(heads) * qr_head_stride * 2, kBQ, 64);
@@ -473,7 +475,7 @@ extern "C" int cafd_attn_prefill_mla(const void* q_nope, int q_head_stride, cons
   p.status = status;
   p.max_pages = max_pages; p.Hq = heads; p.Hkv = heads;
   p.scale_log2 = scale * 1.4426950408889634f;
-  p.window = 0;
+  p.window = window;
   p.kv_tmp_start = kv_tmp_start; p.q_head_stride = q_head_stride; p.qr_head_stride = qr_head_stride; p.qr_col0 = qr_col0;
   static bool attr = false;
   if (!attr) {

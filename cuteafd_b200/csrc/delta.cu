@@ -1,0 +1,241 @@
+// Gated delta rule layers (one decay per head): short causal convolutions with silu on q, k and v, unit norms, the
+// recurrence
+//     S <- g S;  u = beta (v - S^T k);  S <- S + k u^T;  o = S^T q
+// and the output norm under a silu gate.
+//
+// delta_step runs any mix of portions token by token with the state in registers: decode rows, speculative-verify rows,
+// short portions, any sizes, bf16 or fp32 activations.  The state, the convolutions' inputs, the norms, the step size and
+// the decay are fp32 throughout.  The state is read from one slot and written to another, so a step can be repeated
+// (graph capture, rejected drafts) and a sequence may start from a slot that a cached prefix owns.
+#include "cafd_api.h"
+#include "common.cuh"
+
+namespace cafd {
+
+template <typename E> __device__ __forceinline__ float de_f(E v);
+template <> __device__ __forceinline__ float de_f<float>(float v) { return v; }
+template <> __device__ __forceinline__ float de_f<__nv_bfloat16>(__nv_bfloat16 v) { return __bfloat162float(v); }
+template <typename E> __device__ __forceinline__ E de_e(float v);
+template <> __device__ __forceinline__ float de_e<float>(float v) { return v; }
+template <> __device__ __forceinline__ __nv_bfloat16 de_e<__nv_bfloat16>(float v) { return __float2bfloat16(v); }
+
+struct DeltaArgs {
+  const void* proj;           // [T, ld] E: q | k | v | gate | b | a sections at the offsets below
+  const float* conv_w;        // [channels, taps] (q heads, k heads, v heads)
+  const float* A_log;         // [heads]
+  const float* dt_bias;       // [heads]
+  const float* norm_w;        // [vdim]
+  float* state;               // pool, slot_stride floats per slot
+  const int* state_in;        // [S]
+  const int* state_out;       // [S]
+  const int* q_start;         // [S + 1]
+  void* out;                  // [T, heads * out_vd] E: normed and gated rows (head h at h * out_vd)
+  float* raw;                 // [T, heads * vdim] fp32: o before the norm, when a head's columns span several blocks
+  long long slot_stride, s_off, c_off;   // the layer's state and convolution inputs inside a slot
+  int ld, q_off, k_off, v_off, g_off, b_off, a_off;
+  int T, S, heads, kv_heads, dim, vdim, taps, out_vd;
+  float eps;
+};
+
+constexpr int kDeltaRows = 32;      // state rows per thread
+constexpr int kDeltaCols = 128;     // state columns per block at most
+
+__device__ __forceinline__ float softplus(float a) { return fmaxf(a, 0.f) + log1pf(expf(-fabsf(a))); }
+__device__ __forceinline__ float sigmoid_f(float x) { return 1.0f / (1.0f + expf(-x)); }
+
+template <typename E, int MAXT, int NT>
+__global__ void __launch_bounds__(NT) delta_step_kernel(const DeltaArgs p) {
+  extern __shared__ float sm[];
+  const int h = blockIdx.x, seq = blockIdx.y, v0 = blockIdx.z * kDeltaCols;
+  const int tid = threadIdx.x, lane = tid & 31;
+  const int vt = min(kDeltaCols, p.vdim - v0);
+  const int n_slice = (p.dim + kDeltaRows - 1) / kDeltaRows;
+  const int slice = tid / vt, col = tid - slice * vt;
+  const bool worker = slice < n_slice;
+  const int r0 = slice * kDeltaRows;
+  const int n_ch = 2 * p.dim + vt;
+  float* ch = sm;                                // [2][n_ch]
+  float* red = ch + 2 * n_ch;                    // [2][n_slice][vt]
+  float* so = red + 2 * n_slice * vt;            // [vt]
+  float* sgb = so + vt;                          // [2][2]: decay, beta
+
+  // The state of this step was written a whole step ago: its loads need not wait for the projection.
+  float S[kDeltaRows];
+  const float* st_in = p.state + static_cast<size_t>(p.state_in[seq]) * p.slot_stride;
+  float* st_out = p.state + static_cast<size_t>(p.state_out[seq]) * p.slot_stride;
+  const size_t s_base = p.s_off + (static_cast<size_t>(h) * p.dim) * p.vdim + v0 + col;
+#pragma unroll
+  for (int r = 0; r < kDeltaRows; ++r)
+    S[r] = (worker && r0 + r < p.dim) ? st_in[s_base + static_cast<size_t>(r0 + r) * p.vdim] : 0.f;
+
+  // this thread's convolution channel
+  const int rep = p.heads / p.kv_heads, kh = h / rep;
+  const int kd = p.kv_heads * p.dim, channels = 2 * kd + p.heads * p.vdim;
+  int chan = -1, src = 0;
+  bool keeper = false;                           // writes the channel's inputs to the new state
+  if (tid < p.dim) { chan = kh * p.dim + tid; src = p.q_off + chan; keeper = h == kh * rep && blockIdx.z == 0; }
+  else if (tid < 2 * p.dim) { const int c = kh * p.dim + tid - p.dim; chan = kd + c; src = p.k_off + c; keeper = h == kh * rep && blockIdx.z == 0; }
+  else if (tid < n_ch) { const int c = h * p.vdim + v0 + tid - 2 * p.dim; chan = 2 * kd + c; src = p.v_off + c; keeper = true; }
+  const int halo = p.taps - 1;
+  float win[MAXT - 1], cw[MAXT];
+#pragma unroll
+  for (int j = 0; j < MAXT; ++j) {
+    const int tap = j - (MAXT - p.taps);
+    cw[j] = (chan >= 0 && tap >= 0) ? p.conv_w[static_cast<size_t>(chan) * p.taps + tap] : 0.f;
+  }
+#pragma unroll
+  for (int j = 0; j < MAXT - 1; ++j) {
+    const int i = j - (MAXT - 1 - halo);
+    win[j] = (chan >= 0 && i >= 0) ? st_in[p.c_off + static_cast<size_t>(i) * channels + chan] : 0.f;
+  }
+  const float a_scale = tid == 0 ? -expf(p.A_log[h]) : 0.f, dt = tid == 0 ? p.dt_bias[h] : 0.f;
+  const float nw = (slice == 0 && p.out) ? p.norm_w[v0 + col] : 0.f;
+
+  pdl_wait();
+  pdl_trigger();
+  const int t0 = p.q_start[seq], t1 = p.q_start[seq + 1];
+  const E* proj = static_cast<const E*>(p.proj);
+  float x = (chan >= 0 && t0 < t1) ? de_f<E>(proj[static_cast<size_t>(t0) * p.ld + src]) : 0.f;
+  for (int t = t0; t < t1; ++t) {
+    const int buf = (t - t0) & 1;
+    const E* row = proj + static_cast<size_t>(t) * p.ld;
+    float* c = ch + buf * n_ch;
+    if (chan >= 0) {
+      float y = cw[MAXT - 1] * x;
+#pragma unroll
+      for (int j = 0; j < MAXT - 1; ++j) y = fmaf(cw[j], win[j], y);
+#pragma unroll
+      for (int j = 0; j + 1 < MAXT - 1; ++j) win[j] = win[j + 1];
+      win[MAXT - 2] = x;
+      c[tid] = y * sigmoid_f(y);
+    }
+    if (tid == 0) {
+      sgb[2 * buf] = expf(a_scale * softplus(de_f<E>(row[p.a_off + h]) + dt));
+      sgb[2 * buf + 1] = sigmoid_f(de_f<E>(row[p.b_off + h]));
+    }
+    __syncthreads();
+    if (chan >= 0 && t + 1 < t1) x = de_f<E>(row[p.ld + src]);
+    const float gate = (slice == 0 && p.out) ? de_f<E>(row[p.g_off + h * p.vdim + v0 + col]) : 0.f;
+    float qq = 0.f, kk = 0.f, qk = 0.f;
+    for (int i = lane; i < p.dim; i += 32) {
+      const float a = c[i], b = c[p.dim + i];
+      qq = fmaf(a, a, qq); kk = fmaf(b, b, kk); qk = fmaf(a, b, qk);
+    }
+    qq = warp_sum(qq); kk = warp_sum(kk); qk = warp_sum(qk);
+    const float ik = 1.0f / sqrtf(kk + 1e-6f), iq = 1.0f / (sqrtf(qq + 1e-6f) * sqrtf(static_cast<float>(p.dim)));
+    float sk = 0.f, sq = 0.f;
+    if (worker) {
+#pragma unroll
+      for (int r = 0; r < kDeltaRows; ++r) {
+        if (r0 + r < p.dim) {
+          sq = fmaf(S[r], c[r0 + r], sq);
+          sk = fmaf(S[r], c[p.dim + r0 + r], sk);
+        }
+      }
+      red[slice * vt + col] = sk;
+      red[(n_slice + slice) * vt + col] = sq;
+    }
+    __syncthreads();
+    if (worker) {
+      sk = 0.f; sq = 0.f;
+      for (int i = 0; i < n_slice; ++i) { sk += red[i * vt + col]; sq += red[(n_slice + i) * vt + col]; }
+      const float g = sgb[2 * buf], beta = sgb[2 * buf + 1];
+      const float u = beta * (c[2 * p.dim + col] - g * (ik * sk));
+      const float uk = u * ik;
+#pragma unroll
+      for (int r = 0; r < kDeltaRows; ++r)
+        if (r0 + r < p.dim) S[r] = fmaf(c[p.dim + r0 + r], uk, g * S[r]);
+      if (slice == 0) {
+        const float o = g * (iq * sq) + (qk * ik * iq) * u;
+        if (p.out) so[col] = o;
+        else p.raw[static_cast<size_t>(t) * p.heads * p.vdim + h * p.vdim + v0 + col] = o;
+      }
+    }
+    if (p.out) {
+      __syncthreads();
+      if ((tid & ~31) < vt) {
+        float ss = 0.f;
+        for (int i = lane; i < vt; i += 32) ss = fmaf(so[i], so[i], ss);
+        ss = warp_sum(ss);
+        if (tid < vt) {
+          const float inv = 1.0f / sqrtf(ss / static_cast<float>(vt) + p.eps);
+          static_cast<E*>(p.out)[(static_cast<size_t>(t) * p.heads + h) * p.out_vd + tid] =
+              de_e<E>(so[tid] * inv * nw * gate * sigmoid_f(gate));
+        }
+      }
+    }
+  }
+  if (t1 > t0) {
+    if (worker) {
+#pragma unroll
+      for (int r = 0; r < kDeltaRows; ++r)
+        if (r0 + r < p.dim) st_out[s_base + static_cast<size_t>(r0 + r) * p.vdim] = S[r];
+    }
+    if (chan >= 0 && keeper) {
+#pragma unroll
+      for (int j = 0; j < MAXT - 1; ++j) {
+        const int i = j - (MAXT - 1 - halo);
+        if (i >= 0) st_out[p.c_off + static_cast<size_t>(i) * channels + chan] = win[j];
+      }
+    }
+  }
+}
+
+// out[t, h] = raw[t, h] / rms(raw[t, h]) * norm_w * silu(gate): one warp per (token, head)
+template <typename E>
+__global__ void __launch_bounds__(256) delta_out_kernel(const DeltaArgs p) {
+  pdl_wait();
+  pdl_trigger();
+  const long long n = static_cast<long long>(p.T) * p.heads;
+  const int lane = threadIdx.x & 31;
+  for (long long i = static_cast<long long>(blockIdx.x) * 8 + (threadIdx.x >> 5); i < n; i += static_cast<long long>(gridDim.x) * 8) {
+    const long long t = i / p.heads;
+    const int h = static_cast<int>(i - t * p.heads);
+    const float* o = p.raw + i * p.vdim;
+    const E* gate = static_cast<const E*>(p.proj) + t * p.ld + p.g_off + h * p.vdim;
+    float ss = 0.f;
+    for (int v = lane; v < p.vdim; v += 32) ss = fmaf(o[v], o[v], ss);
+    const float inv = 1.0f / sqrtf(warp_sum(ss) / static_cast<float>(p.vdim) + p.eps);
+    E* dst = static_cast<E*>(p.out) + i * p.out_vd;
+    for (int v = lane; v < p.vdim; v += 32) {
+      const float g = de_f<E>(gate[v]);
+      dst[v] = de_e<E>(o[v] * inv * p.norm_w[v] * g * sigmoid_f(g));
+    }
+  }
+}
+
+template <typename E, int MAXT>
+static int launch_delta(const DeltaArgs& p, cudaStream_t st) {
+  const int vt = p.vdim < kDeltaCols ? p.vdim : kDeltaCols;
+  const int n_slice = (p.dim + kDeltaRows - 1) / kDeltaRows;
+  int threads = vt * n_slice;
+  if (threads < 2 * p.dim + vt) threads = 2 * p.dim + vt;
+  threads = (threads + 31) / 32 * 32;
+  if (threads > 1024) return -12;
+  const size_t smem = static_cast<size_t>(2 * (2 * p.dim + vt) + 2 * n_slice * vt + vt + 4) * 4;
+  const int tiles = (p.vdim + kDeltaCols - 1) / kDeltaCols;
+  DeltaArgs q = p;
+  if (tiles > 1) { if (!p.raw) return -13; q.out = nullptr; }
+  const dim3 grid(p.heads, p.S, tiles);
+  if (threads <= 512) launch_pdl(delta_step_kernel<E, MAXT, 512>, grid, dim3(threads), smem, st, q);
+  else launch_pdl(delta_step_kernel<E, MAXT, 1024>, grid, dim3(threads), smem, st, q);
+  if (tiles > 1) {
+    const long long rows = static_cast<long long>(p.T) * p.heads;
+    const int blocks = static_cast<int>(rows < 8 * 148 * 8 ? (rows + 7) / 8 : 148 * 8);
+    launch_pdl(delta_out_kernel<E>, dim3(blocks), dim3(256), 0, st, p);
+  }
+  return static_cast<int>(cudaGetLastError());
+}
+
+}  // namespace cafd
+
+using namespace cafd;
+
+extern "C" int cafd_delta_step(const DeltaArgs* p, int is_f32, cafd_stream_t s) {
+  if (p->T <= 0) return 0;
+  if (p->S < 1 || p->kv_heads < 1 || p->heads % p->kv_heads || p->dim < 1 || p->dim > 256 || p->taps < 1 || p->taps > 16) return -10;
+  if (!p->state || !p->state_in || !p->state_out || !p->out || p->out_vd < p->vdim) return -10;
+  cudaStream_t st = static_cast<cudaStream_t>(s);
+  if (p->taps <= 4) return is_f32 ? launch_delta<float, 4>(*p, st) : launch_delta<__nv_bfloat16, 4>(*p, st);
+  return is_f32 ? launch_delta<float, 16>(*p, st) : launch_delta<__nv_bfloat16, 16>(*p, st);
+}

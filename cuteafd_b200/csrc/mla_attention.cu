@@ -47,6 +47,7 @@ struct MlaDev {
   uint32_t* status;
   uint32_t* trace;         // optional progress words, 4 per CTA (producer, MMA, softmax, exit); host-mapped memory works
   int max_pages, heads, splits;
+  int window;              // sliding window: a query at position t sees positions (t - window, t]; 0 = all earlier ones
   int split_tiles;         // > 0: split s owns kv tiles [s * split_tiles, (s + 1) * split_tiles) of every block (batch-invariant form)
   int out_tpad;            // 0: out rows are (token, head); > 0: head-major rows head * out_tpad + token
   float scale_log2;
@@ -106,9 +107,11 @@ mla_attn_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant_
   const int base_vis = p.kv_base ? p.kv_base[seq] : kv_len - q_len;
   const int max_limit = sparse ? min(kv_len - q_len + last_tok + 1, p.sparse_k) : min(kv_len, base_vis + last_tok + 1);
   const int total_tiles = (tok0 < q_len && max_limit > 0) ? (max_limit + kKvTile - 1) / kKvTile : 0;   // block past the new tokens: idle
-  const int per_split = p.split_tiles > 0 ? p.split_tiles : (total_tiles + p.splits - 1) / p.splits;
-  const int t_begin = split * per_split;
-  const int t_end = min(total_tiles, t_begin + per_split);
+  // with a window the tiles wholly before the first token's window are skipped (the splits divide what remains)
+  const int tile0 = p.window > 0 ? max(0, base_vis + tok0 + 1 - p.window) / kKvTile : 0;
+  const int per_split = p.split_tiles > 0 ? p.split_tiles : (max(0, total_tiles - tile0) + p.splits - 1) / p.splits;
+  const int t_begin = p.split_tiles > 0 ? max(tile0, split * per_split) : tile0 + split * per_split;
+  const int t_end = min(total_tiles, p.split_tiles > 0 ? (split + 1) * per_split : t_begin + per_split);
   const int n_tiles = max(0, t_end - t_begin);
   const int seq_pages = (kv_len + 63) / 64;
   uint32_t* tr = p.trace ? p.trace + 4 * ((blockIdx.z * gridDim.y + blockIdx.y) * gridDim.x + blockIdx.x) : nullptr;
@@ -267,6 +270,7 @@ mla_attn_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant_
     const int ti = row / p.heads;
     const bool row_valid = (tok0 + ti) < q_len && ti < tok_per_blk;
     const int limit = !row_valid ? 0 : sparse ? max_limit : min(kv_len, base_vis + tok0 + ti + 1);
+    const int low = p.window > 0 ? base_vis + tok0 + ti + 1 - p.window : 0;      // first position inside this row's window
     const uint32_t lane_off = static_cast<uint32_t>(quad * 32) << 16;
     float m_run = -INFINITY, l_run = 0.f;
     bool ok = true;
@@ -286,7 +290,7 @@ mla_attn_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant_
       float s[32];
 #pragma unroll
       for (int i = 0; i < 32; ++i) {
-        s[i] = (col0 + i < limit) ? __uint_as_float(r[i]) * p.scale_log2 : -INFINITY;
+        s[i] = (col0 + i < limit && col0 + i >= low) ? __uint_as_float(r[i]) * p.scale_log2 : -INFINITY;
         mx = fmaxf(mx, s[i]);
       }
       // The running reference m_run only moves when the tile maximum exceeds it by more than 8 (in log2
@@ -494,8 +498,10 @@ static int mla_attention_impl(const void* q, const void* cache, const int* page_
                               float* scratch, uint32_t* status, long long total_rows, int n_blocks, int num_pages,
                               int max_pages, int heads, int splits, int out_tpad, float scale,
                               const int* sparse_idx, int sparse_k, int gathered, cafd_stream_t s,
-                              const int* kv_base = nullptr, void* const* peer_scratch = nullptr, int n_peers = 0, int my_rank = 0) {
+                              const int* kv_base = nullptr, void* const* peer_scratch = nullptr, int n_peers = 0, int my_rank = 0,
+                              int window = 0) {
   if (n_blocks <= 0) return 0;
+  if (window < 0 || (window && sparse_idx)) return -16;
   if (heads <= 0 || kMlaRows % heads) return -10;
   if (splits < 1) splits = 1;
   if (splits > kMaxSplits) return -13;
@@ -510,6 +516,7 @@ static int mla_attention_impl(const void* q, const void* cache, const int* page_
   rc = make_tmap_nd(&tc, cache, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 3, dims, strides, box, true);
   if (rc) return rc;
   MlaDev p;
+  p.window = window;
   p.page_table = page_table; p.seq_lens = seq_lens; p.q_start = q_start; p.block_seq = block_seq; p.block_tok0 = block_tok0;
   p.out = static_cast<__nv_bfloat16*>(out);
   p.partial = scratch;
@@ -551,9 +558,10 @@ extern "C" int cafd_mla_attention(const void* q, const void* cache, const int* p
                                   const int* q_start, const int* block_seq, const int* block_tok0, void* out,
                                   float* scratch, uint32_t* status, long long total_rows, int n_blocks, int num_pages,
                                   int max_pages, int heads, int splits, int out_tpad, float scale,
-                                  const int* sparse_idx, int sparse_k, cafd_stream_t s) {
+                                  const int* sparse_idx, int sparse_k, int window, cafd_stream_t s) {
   return mla_attention_impl(q, cache, page_table, seq_lens, q_start, block_seq, block_tok0, out, scratch, status, total_rows,
-                            n_blocks, num_pages, max_pages, heads, splits, out_tpad, scale, sparse_idx, sparse_k, 0, s);
+                            n_blocks, num_pages, max_pages, heads, splits, out_tpad, scale, sparse_idx, sparse_k, 0, s, nullptr,
+                            nullptr, 0, 0, window);
 }
 
 // Sparse attention over records that mla_fp8_gather expanded: gathered [n_blocks, sparse_k, 576] bf16.

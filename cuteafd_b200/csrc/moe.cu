@@ -70,13 +70,13 @@ template <int kPerLane>
 __global__ void __launch_bounds__(128) route_topk_kernel(const float* __restrict__ logits, const float* __restrict__ bias,
                                                          int* __restrict__ out_idx, float* __restrict__ out_w, int T,
                                                          int E, int top_k, int sigmoid, int num_groups,
-                                                         int topk_groups, int normalize, float routed_scale) {
+                                                         int topk_groups, int normalize, float routed_scale, int group_max) {
   pdl_wait();
   pdl_trigger();
   const int t = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
   if (t >= T) return;
   route_row<kPerLane>(logits + static_cast<size_t>(t) * E, bias, out_idx, out_w, t, E, top_k, sigmoid, num_groups, topk_groups,
-                      normalize, routed_scale);
+                      normalize, routed_scale, group_max);
 }
 
 // Decode-sized batches: RMSNorm of the residual row, the router scores and the top-k selection in one
@@ -94,7 +94,7 @@ __global__ void __launch_bounds__(256) norm_route_kernel(const __nv_bfloat16* __
                                                          int* __restrict__ out_idx, float* __restrict__ out_w,
                                                          float* __restrict__ logits_buf, uint32_t* __restrict__ tickets, int H,
                                                          int E, int top_k, int sigmoid, int num_groups, int topk_groups,
-                                                         int normalize, float routed_scale) {
+                                                         int normalize, float routed_scale, int group_max) {
   pdl_wait();
   pdl_trigger();
   __shared__ __align__(16) __nv_bfloat16 sx[kNormRouteMaxH];
@@ -115,6 +115,13 @@ __global__ void __launch_bounds__(256) norm_route_kernel(const __nv_bfloat16* __
 #pragma unroll
     for (int e = 0; e < 4; ++e) ss += bf16_lo(q[e]) * bf16_lo(q[e]) + bf16_hi(q[e]) * bf16_hi(q[e]);
   }
+  if (!ln_w) {                               // the rows are normalised already: scores and selection only
+#pragma unroll
+    for (int i = 0; i < kRowVec; ++i) {
+      const int c = tid + i * 256;
+      if (c < nvec) reinterpret_cast<uint4*>(sx)[c] = hv[i];
+    }
+  } else {
   ss = warp_sum(ss);
   if (lane == 0) red[warp] = ss;
   __syncthreads();
@@ -135,6 +142,7 @@ __global__ void __launch_bounds__(256) norm_route_kernel(const __nv_bfloat16* __
       reinterpret_cast<uint4*>(sx)[c] = ov;
       if (g == 0) reinterpret_cast<uint4*>(x_out + static_cast<size_t>(t) * H)[c] = ov;
     }
+  }
   }
   __syncthreads();
   const int per = (E + static_cast<int>(gridDim.y) - 1) / static_cast<int>(gridDim.y);
@@ -175,7 +183,7 @@ __global__ void __launch_bounds__(256) norm_route_kernel(const __nv_bfloat16* __
   if (s_last && warp == 0) {
     __threadfence();
     route_row<kPerLane>(logits_buf + static_cast<size_t>(t) * E, bias, out_idx, out_w, t, E, top_k, sigmoid, num_groups,
-                        topk_groups, normalize, routed_scale);
+                        topk_groups, normalize, routed_scale, group_max);
   }
 }
 
@@ -718,7 +726,7 @@ static bool wire_ok(const cafd_moe_layout* l, int H) {
 }
 
 int cafd_route_topk(const float* logits, const float* bias, int* out_idx, float* out_w, int T, int E, int top_k,
-                    int sigmoid, int num_groups, int topk_groups, int normalize, float routed_scale,
+                    int sigmoid, int num_groups, int topk_groups, int normalize, float routed_scale, int group_max,
                     cafd_stream_t s) {
   if (T <= 0) return 0;
   if (E > kMaxExperts || top_k > 32 || num_groups > 32 || (num_groups > 1 && E % num_groups)) return -10;
@@ -726,7 +734,7 @@ int cafd_route_topk(const float* logits, const float* bias, int* out_idx, float*
   const int blocks = (T + 3) / 4;
 #define CAFD_ROUTE(N)                                                                                          \
   launch_pdl(route_topk_kernel<N>, dim3(blocks), dim3(128), 0, st, logits, bias, out_idx, out_w, T, E, top_k, sigmoid, num_groups, \
-                                               topk_groups, normalize, routed_scale)
+                                               topk_groups, normalize, routed_scale, group_max)
   if (E <= 32) CAFD_ROUTE(1);
   else if (E <= 64) CAFD_ROUTE(2);
   else if (E <= 128) CAFD_ROUTE(4);
@@ -782,10 +790,10 @@ int cafd_moe_plan_dispatch(const int* idx, int T, int top_k, int E, int tile_row
 }
 
 // RMSNorm + router scores + top-k for decode-sized batches.  logits_buf [T, E] fp32 receives the scores;
-// tickets [T] uint32 must be zero (the kernel leaves them zero).
+// tickets [T] uint32 must be zero (the kernel leaves them zero).  ln_w null: h holds normalised rows (no norm, x_out unused).
 int cafd_norm_route(const void* h, const void* ln_w, float eps, const void* router_w, const float* bias, void* x_out,
                     int* out_idx, float* out_w, float* logits_buf, uint32_t* tickets, int T, int H, int E, int top_k, int sigmoid,
-                    int num_groups, int topk_groups, int normalize, float routed_scale, cafd_stream_t s) {
+                    int num_groups, int topk_groups, int normalize, float routed_scale, int group_max, cafd_stream_t s) {
   if (T <= 0) return 0;
   if (E > kMaxExperts || top_k > 32 || num_groups > 32 || (num_groups > 1 && E % num_groups) || H % 8 || H > kNormRouteMaxH ||
       !logits_buf || !tickets)
@@ -800,7 +808,7 @@ int cafd_norm_route(const void* h, const void* ln_w, float eps, const void* rout
   launch_pdl(norm_route_kernel<N>, dim3(T, groups), dim3(256), 0, st, static_cast<const __nv_bfloat16*>(h),                    \
              static_cast<const __nv_bfloat16*>(ln_w), eps, static_cast<const __nv_bfloat16*>(router_w), bias,                 \
              static_cast<__nv_bfloat16*>(x_out), out_idx, out_w, logits_buf, tickets, H, E, top_k, sigmoid, num_groups,        \
-             topk_groups, normalize, routed_scale)
+             topk_groups, normalize, routed_scale, group_max)
   if (E <= 32) CAFD_NROUTE(1);
   else if (E <= 64) CAFD_NROUTE(2);
   else if (E <= 128) CAFD_NROUTE(4);

@@ -14,7 +14,7 @@ namespace cafd {
 template <int kPerLane>
 __device__ __forceinline__ void route_row(const float* row, const float* __restrict__ bias, int* __restrict__ out_idx,
                                           float* __restrict__ out_w, int t, int E, int top_k, int sigmoid, int num_groups,
-                                          int topk_groups, int normalize, float routed_scale) {
+                                          int topk_groups, int normalize, float routed_scale, int group_max = 0) {
   const int lane = threadIdx.x & 31;
   float score[kPerLane], sel[kPerLane];
   float mx = -INFINITY;
@@ -63,7 +63,7 @@ __device__ __forceinline__ void route_row(const float* row, const float* __restr
     unsigned keep = 0;   // bit g set = group g kept
     float gscore_mine = -INFINITY;   // lane g holds the score of group g
     for (int g = 0; g < num_groups; ++g) {
-      // the group's two best selection scores: per-lane best and runner-up first, then one warp reduction of pairs
+      // the group's two best selection scores (group_max: a group counts by its best alone): per-lane best and runner-up first, then one warp reduction of pairs
       float top1 = -INFINITY, top2 = -INFINITY;
       int i1 = 0x7fffffff;
 #pragma unroll
@@ -82,7 +82,7 @@ __device__ __forceinline__ void route_row(const float* row, const float* __restr
         if (o1 > top1 || (o1 == top1 && oi < i1)) { top2 = fmaxf(top1, o2); top1 = o1; i1 = oi; }
         else top2 = fmaxf(top2, o1);
       }
-      if (lane == g) gscore_mine = top1 + top2;
+      if (lane == g) gscore_mine = group_max ? top1 : top1 + top2;
     }
     for (int it = 0; it < topk_groups; ++it) {
       float v = (lane < num_groups && !((keep >> lane) & 1u)) ? gscore_mine : -INFINITY;

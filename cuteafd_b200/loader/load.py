@@ -305,6 +305,18 @@ def load_gqa_engine_weights(path: str, device: torch.device, with_experts: bool 
     return cfg, W
 
 
+def load_hybrid_weights(snap: OpenedSnapshot, cfg: ModelConfig, device: torch.device):
+    """Device weights of a per-layer hybrid, read from the catalog tensor by tensor."""
+    from ..models.hybrid import HybridWeights
+    missing = object()
+
+    def get(name: str) -> torch.Tensor:
+        if snap.catalog.entries.get(name, missing) is missing:
+            raise ValueError(f"{snap.path}: the checkpoint has no tensor {name}")
+        return snap.catalog.read(name)
+    return HybridWeights.build(cfg, get, torch.device(device))
+
+
 def host_embedding_table(path: str, **kw):
     """The snapshot's token embedding as a memory-mapped host table (``--embedding-placement host``): rows are gathered
     per step instead of the table living in GPU memory.  bf16 / f16 / f32 tables only (a quantised embedding is
@@ -319,12 +331,29 @@ def host_embedding_table(path: str, **kw):
     return MappedTable.from_safetensors(snap.catalog, name, **kw)
 
 
-def load_engine(path: str, device: torch.device, num_pages: int, max_tokens: int, max_seqs: int, kv_format: str = "auto"):
+def hybrid_state_slots(rows: int) -> int:
+    """Slots for decode steps of ``rows`` rows (8 per sequence): per sequence its state, the state before an unsettled
+    step and the one being written, and as many again for cached prefixes."""
+    return 2 + 6 * max(1, -(-rows // 8))
+
+
+def load_engine(path: str, device: torch.device, num_pages: int, max_tokens: int, max_seqs: int, kv_format: str = "auto",
+                compute_dtype: str = "bf16", state_slots: int = 0):
     """(cfg, engine) for a snapshot: the GQA engine streams its weights tensor by tensor; MLA checkpoints (and any
     checkpoint with MTP depths) go through the dense parameter dictionary, decoded to bf16.  ``kv_format`` "auto"
-    picks the 656-byte FP8 latent record for sparse-attention (indexer) checkpoints and bf16 records otherwise."""
+    picks the 656-byte FP8 latent record for sparse-attention (indexer) checkpoints and bf16 records otherwise.
+    Per-layer hybrids: ``compute_dtype`` "f32" runs everything in 32-bit, ``state_slots`` is the number of recurrent state
+    slots (0: enough for ``max_seqs`` rows' sequences in flight and as many cached prefixes)."""
     snap = open_snapshot(path)
     cfg = snap.cfg
+    if cfg.is_hybrid:
+        from ..models.hybrid import HybridCache, HybridEngine
+        cfg = cfg.replace(compute_dtype=compute_dtype)
+        W = load_hybrid_weights(snap, cfg, device)
+        kv = HybridCache(cfg, num_pages, device, state_slots or hybrid_state_slots(max_seqs))
+        return cfg, HybridEngine(cfg, W, kv, max_tokens=max_tokens, max_seqs=max_seqs)
+    if compute_dtype != "bf16":
+        raise ValueError(f"{cfg.family}: only the per-layer hybrids run in {compute_dtype}")
     if cfg.is_mla:
         want = ("fp8_ds_mla" if cfg.indexer_heads else "bf16") if kv_format == "auto" else kv_format
         if want == "fp8_ds_mla" and not cfg.indexer_heads:

@@ -37,6 +37,9 @@ class Batch:
     # media rows: (row indices int64 [m], embeddings [m, hidden] bf16), both on the device; those rows of the input
     # take the tower's output instead of the embedding table's row (eager prefill only)
     embeds: tuple | None = None
+    # recurrent layers: per sequence the state slot read and the slot written (never the same)
+    state_in: torch.Tensor | None = None    # [S]
+    state_out: torch.Tensor | None = None   # [S]
 
 
 class LayerWeights:

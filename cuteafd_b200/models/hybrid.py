@@ -1,0 +1,473 @@
+"""Per-layer hybrid decoders (``ModelConfig.layer_specs``): windowed latent attention and gated delta-rule layers in any
+order, grouped RMS norms before and after every sublayer, a causal convolution on every sublayer's input, routed
+feed-forwards with identity outputs.
+
+A layer is a fixed launch sequence over preallocated workspaces:
+
+    norm_conv -> fused projection -> mixer kernels -> o projection -> norm_conv -> routes -> plan / dispatch -> fc1 -> fc2
+
+``norm_conv`` is everything between two sublayers (the routed rows' weighted sum, the norm after the sublayer, the fp32
+residual, the norm before the next one, its convolution).  What a sequence carries besides latent records lives in slots
+of one fp32 pool; a step reads one slot per sequence and writes another (``Batch.state_in`` / ``state_out``), so a step
+can be repeated and a slot can be shared with a cached prefix.  ``compute_dtype`` "f32" runs the same sequence with every
+product and activation in 32-bit.
+"""
+from __future__ import annotations
+
+import torch
+
+from ..config import DeltaSpec, LatentSpec, ModelConfig
+from ..ops import kernels as K
+from ..parallel.moe_exchange import ExchangeGeometry, LocalExchange
+from .gqa_moe import PAGE, Batch
+from .mla_moe import _HeadTiles
+
+
+def pad8(n: int) -> int:
+    return -(-n // 8) * 8
+
+
+def engine_dtype(cfg: ModelConfig) -> torch.dtype:
+    return torch.float32 if cfg.compute_dtype == "f32" else torch.bfloat16
+
+
+def record_pitch(m: LatentSpec) -> int:
+    """Elements of one cached record: latent, rotated key part, padding to whole 16-byte pieces."""
+    return pad8(m.record)
+
+
+class HybridLayer:
+    """One layer's weights in the layout the kernels stream: the projections that read the same input are one matrix
+    (``offs`` names its sections, each padded to a multiple of 8 rows), experts are stacked."""
+    __slots__ = ("norm1", "norm1b", "norm2", "norm2b", "canon1", "canon2", "w_in", "offs", "w_o",
+                 "kv_norm", "w_uk", "w_uv", "w_kb", "conv_w", "A_log", "dt_bias", "out_norm",
+                 "router", "correction", "w_gate", "w_up", "w_down")
+
+    def __init__(self) -> None:
+        for s in self.__slots__:
+            setattr(self, s, None)
+
+
+class HybridWeights:
+    def __init__(self, cfg: ModelConfig):
+        self.cfg = cfg
+        self.embed = self.final_norm = self.lm_head = None
+        self.layers: list[HybridLayer] = []
+
+    @staticmethod
+    def build(cfg: ModelConfig, get, device: torch.device) -> "HybridWeights":
+        """``get(name) -> tensor`` under the checkpoint's names (any float dtype, any device)."""
+        dt = engine_dtype(cfg)
+
+        def t(name: str, shape: tuple | None = None) -> torch.Tensor:
+            x = get(name).to(device=device, dtype=dt)
+            if shape is not None and tuple(x.shape) != shape:
+                raise ValueError(f"{name}: shape {tuple(x.shape)}, the configuration says {shape}")
+            return x.contiguous()
+
+        def f(name: str) -> torch.Tensor:
+            return get(name).to(device=device, dtype=torch.float32).contiguous()
+
+        def fuse(parts: list[tuple[str, torch.Tensor]]) -> tuple[torch.Tensor, dict]:
+            rows = sum(pad8(x.shape[0]) for _, x in parts)
+            out = torch.zeros(rows, cfg.hidden, dtype=dt, device=device)
+            offs, o = {}, 0
+            for n, x in parts:
+                out[o:o + x.shape[0]] = x
+                offs[n] = o
+                o += pad8(x.shape[0])
+            return out, offs
+
+        def heads_o(name: str, heads: int, vdim: int) -> torch.Tensor:
+            """o projection with every head's columns padded to the row layout the mixers write."""
+            w = t(name, (cfg.hidden, heads * vdim)).view(cfg.hidden, heads, vdim)
+            out = torch.zeros(cfg.hidden, heads, pad8(vdim), dtype=dt, device=device)
+            out[..., :vdim] = w
+            return out.view(cfg.hidden, heads * pad8(vdim))
+
+        H = cfg.hidden
+        W = HybridWeights(cfg)
+        W.embed, W.final_norm, W.lm_head = t("embed", (cfg.vocab_size, H)), f("final.norm"), t("head", (cfg.vocab_size, H))
+        for i, spec in enumerate(cfg.layer_specs):
+            pre, m, r, L = f"l{i}.", spec.mixer, spec.router, HybridLayer()
+            x = pre + "mix."
+            L.norm1, L.norm1b = f(pre + "norm1"), f(pre + "norm1b")
+            L.canon1 = f(pre + "canon1").T.contiguous()
+            if isinstance(m, LatentSpec):
+                L.w_in, L.offs = fuse([("q", t(x + "q", (m.heads * (m.dim + m.rot_dim), H))), ("kv", t(x + "dkv", (m.record, H))),
+                                       ("g", t(x + "g", (m.heads * m.vdim, H)))])
+                L.kv_norm = f(x + "dkv.norm")
+                uk = t(x + "uk", (m.heads * m.dim, m.kv_rank)).view(m.heads, m.dim, m.kv_rank)
+                L.w_uk = torch.zeros(m.heads, m.kv_rank, pad8(m.dim), dtype=dt, device=device)
+                L.w_uk[..., :m.dim] = uk.transpose(1, 2)
+                L.w_uv = torch.zeros(m.heads, m.vdim, pad8(m.kv_rank), dtype=dt, device=device)
+                L.w_uv[..., :m.kv_rank] = t(x + "uv", (m.heads * m.vdim, m.kv_rank)).view(m.heads, m.vdim, m.kv_rank)
+                if tensor_core_latent(cfg, m):
+                    L.w_kb = uk.reshape(m.heads * m.dim, m.kv_rank).contiguous()
+            else:
+                kd, vd = m.kv_heads * m.dim, m.heads * m.vdim
+                L.w_in, L.offs = fuse([(n, t(x + n, (rows, H))) for n, rows in
+                                       (("q", kd), ("k", kd), ("v", vd), ("g", vd), ("b", m.heads), ("a", m.heads))])
+                L.conv_w = torch.cat([f(x + n + ".conv") for n in ("q", "k", "v")]).contiguous()
+                if tuple(L.conv_w.shape) != (m.conv_channels, m.conv):
+                    raise ValueError(f"{x}*.conv: {tuple(L.conv_w.shape)}, the configuration says {(m.conv_channels, m.conv)}")
+                L.A_log, L.dt_bias, L.out_norm = f(x + "A_log"), f(x + "dt_bias"), f(x + "norm")
+            L.w_o = heads_o(x + "o", m.heads, m.vdim)
+            if r is not None:
+                y = pre + "mlp."
+                L.norm2, L.norm2b = f(pre + "norm2"), f(pre + "norm2b")
+                L.canon2 = f(pre + "canon2").T.contiguous()
+                L.router, L.correction = t(y + "router", (r.outputs, H)), f(y + "correction")
+                F = pad8(r.ffn)
+                L.w_gate, L.w_up = (torch.zeros(r.experts, F, H, dtype=dt, device=device) for _ in range(2))
+                L.w_down = torch.zeros(r.experts, H, F, dtype=dt, device=device)
+                for e in range(r.experts):
+                    L.w_gate[e, :r.ffn] = t(f"{y}e{e}.gate", (r.ffn, H))
+                    L.w_up[e, :r.ffn] = t(f"{y}e{e}.up", (r.ffn, H))
+                    L.w_down[e, :, :r.ffn] = t(f"{y}e{e}.down", (H, r.ffn))
+            W.layers.append(L)
+        return W
+
+    @staticmethod
+    def from_params(cfg: ModelConfig, p: dict[str, torch.Tensor], device: torch.device) -> "HybridWeights":
+        return HybridWeights.build(cfg, p.__getitem__, device)
+
+    @staticmethod
+    def random_init(cfg: ModelConfig, device: torch.device, seed: int = 0, std: float = 0.02) -> "HybridWeights":
+        """Random weights made on the device tensor by tensor: N(0, std) matrices, norm weights one, mild decays."""
+        g = torch.Generator(device=device).manual_seed(seed)
+        shapes = tensor_shapes(cfg)
+
+        def get(name: str) -> torch.Tensor:
+            shape = shapes[name]
+            if name.rsplit(".", 1)[-1].startswith("norm"):
+                return torch.ones(shape, device=device)
+            s = 0.3 if "conv" in name or "canon" in name else std
+            x = torch.empty(shape, dtype=torch.float32, device=device).normal_(0.0, s, generator=g)
+            return x - 3.0 if name.endswith("dt_bias") else x
+        return HybridWeights.build(cfg, get, device)
+
+
+def tensor_shapes(cfg: ModelConfig) -> dict[str, tuple]:
+    """Every tensor of the checkpoint and its shape."""
+    H = cfg.hidden
+    out: dict[str, tuple] = {"embed": (cfg.vocab_size, H), "final.norm": (H,), "head": (cfg.vocab_size, H)}
+    for i, spec in enumerate(cfg.layer_specs):
+        pre, m, r = f"l{i}.", spec.mixer, spec.router
+        x = pre + "mix."
+        out.update({pre + "norm1": (H,), pre + "norm1b": (H,), pre + "canon1": (H, cfg.canon_taps), x + "o": (H, m.heads * m.vdim),
+                    x + "g": (m.heads * m.vdim, H)})
+        if isinstance(m, LatentSpec):
+            out.update({x + "q": (m.heads * (m.dim + m.rot_dim), H), x + "dkv": (m.record, H), x + "dkv.norm": (m.kv_rank,),
+                        x + "uk": (m.heads * m.dim, m.kv_rank), x + "uv": (m.heads * m.vdim, m.kv_rank)})
+        else:
+            kd, vd = m.kv_heads * m.dim, m.heads * m.vdim
+            for n, c in (("q", kd), ("k", kd), ("v", vd)):
+                out[x + n], out[x + n + ".conv"] = (c, H), (c, m.conv)
+            out.update({x + "b": (m.heads, H), x + "a": (m.heads, H), x + "A_log": (m.heads,), x + "dt_bias": (m.heads,), x + "norm": (m.vdim,)})
+        if r is not None:
+            y = pre + "mlp."
+            out.update({pre + "norm2": (H,), pre + "norm2b": (H,), pre + "canon2": (H, cfg.canon_taps), y + "router": (r.outputs, H),
+                        y + "correction": (r.outputs,)})
+            for e in range(r.experts):
+                out.update({f"{y}e{e}.gate": (r.ffn, H), f"{y}e{e}.up": (r.ffn, H), f"{y}e{e}.down": (H, r.ffn)})
+    return out
+
+
+def tensor_core_latent(cfg: ModelConfig, m: LatentSpec) -> bool:
+    """Whether the tcgen05 latent attention kernels take this layer (their record and head sizes are fixed)."""
+    return (engine_dtype(cfg) == torch.bfloat16 and (m.kv_rank, m.rot_dim, m.dim, m.vdim) == (512, 64, 128, 128)
+            and 128 % m.heads == 0)
+
+
+class HybridCache:
+    """Paged latent records of the latent attention layers and the slot pool of everything recurrent.
+
+    ``c``: one pool [pages, 64, record] per latent layer (page 0 stays zero).  ``state`` [slots, floats] fp32: slot 0 is
+    the zero state every sequence starts from, slot 1 takes the writes of dummy steps."""
+
+    def __init__(self, cfg: ModelConfig, num_pages: int, device: torch.device, state_slots: int = 34):
+        dt = engine_dtype(cfg)
+        self.num_pages = num_pages
+        self.c: list[torch.Tensor] = []
+        self.of_layer: dict[int, torch.Tensor] = {}
+        self.offsets: list[dict[str, int]] = []
+        n = 0
+        for i, spec in enumerate(cfg.layer_specs):
+            m, off = spec.mixer, {}
+            parts = [("canon1", (cfg.canon_taps - 1) * cfg.hidden)]
+            if spec.router is not None:
+                parts.append(("canon2", (cfg.canon_taps - 1) * cfg.hidden))
+            if isinstance(m, DeltaSpec):
+                parts += [("S", m.heads * m.dim * m.vdim), ("conv", (m.conv - 1) * m.conv_channels)]
+            else:
+                self.of_layer[i] = torch.zeros(num_pages, PAGE, record_pitch(m), dtype=dt, device=device)
+                self.c.append(self.of_layer[i])
+            for name, size in parts:
+                off[name] = n
+                n += -(-size // 32) * 32
+            self.offsets.append(off)
+        self.state = torch.zeros(max(3, state_slots), max(n, 32), dtype=torch.float32, device=device)
+
+    @property
+    def state_slots(self) -> int:
+        return self.state.shape[0]
+
+    def bytes_per_page(self) -> int:
+        return sum(t[0].numel() * t.element_size() for t in self.c)
+
+    def copy_page(self, src: int, dst: int) -> None:
+        for c in self.c:
+            c[dst].copy_(c[src])
+
+
+class _LatentWs:
+    """Workspaces shared by the latent layers of one shape."""
+
+    def __init__(self, cfg: ModelConfig, m: LatentSpec, max_tokens: int, device: torch.device):
+        kw = dict(dtype=engine_dtype(cfg), device=device)
+        rows = -(-max_tokens // 128) * 128
+        self.q_slab = torch.zeros(m.heads * rows * pad8(m.dim), **kw)
+        self.o_slab = torch.zeros(m.heads * rows * pad8(m.kv_rank), **kw)
+        self.q_abs = torch.zeros(max_tokens, m.heads, record_pitch(m), **kw)
+        self.attn = torch.zeros(max_tokens, m.heads, pad8(m.vdim), **kw)
+        i = torch.arange(0, m.rot_dim, 2, dtype=torch.float64)
+        self.inv_freq = (m.rope_base ** (-i / max(1, m.rot_dim))).float().to(device)
+        self.lat = self.k_exp = self.v_exp = None      # expanded-form prompts: made on first use
+
+
+class HybridEngine:
+    """Single-GPU engine of the per-layer hybrids behind the same calls as the other engines (``forward`` on a ``Batch``)."""
+    embed_rows = None
+    EXPANDED_PREFILL_TOKENS = 64     # fresh prompt chunks of at least this many tokens use the expanded-form attention
+    FUSED_ROUTE_TOKENS = 64          # steps up to this many tokens run router scores + selection as one launch
+
+    def __init__(self, cfg: ModelConfig, weights: HybridWeights, kv: HybridCache, max_tokens: int, max_seqs: int = 64):
+        assert cfg.is_hybrid
+        if cfg.hidden % 8:
+            raise ValueError(f"width {cfg.hidden} is not a multiple of 8")
+        self.cfg, self.W, self.kv = cfg, weights, kv
+        self.device = dev = weights.embed.device
+        self.dtype = dt = engine_dtype(cfg)
+        # a decode step may carry as many rows again: accepted rows the recurrent state has yet to see
+        max_seqs *= 2
+        self.max_tokens = max_tokens = max(max_tokens, max_seqs)
+        H = cfg.hidden
+
+        class _Ws:
+            pass
+        ws = self.ws = _Ws()
+        ws.x = [torch.empty(max_tokens, H, dtype=torch.float32, device=dev) for _ in range(2)]
+        ws.h = [torch.empty(max_tokens, H, dtype=dt, device=dev) for _ in range(2)]
+        ws.y = torch.empty(max_tokens, H, dtype=dt, device=dev)
+        ws.proj = torch.empty(max_tokens * max(L.w_in.shape[0] for L in weights.layers), dtype=dt, device=dev)
+        outs = max((s.router.outputs for s in cfg.layer_specs if s.router), default=1)
+        ws.router = torch.empty(max_tokens * outs, dtype=torch.float32, device=dev)
+        self._lat: dict[LatentSpec, _LatentWs] = {}
+        self._delta: dict[DeltaSpec, torch.Tensor] = {}
+        self._moe: dict = {}
+        raw = 0
+        for spec in cfg.layer_specs:
+            m, r = spec.mixer, spec.router
+            if isinstance(m, LatentSpec):
+                if m not in self._lat:
+                    self._lat[m] = _LatentWs(cfg, m, max_tokens, dev)
+            else:
+                if m not in self._delta:
+                    self._delta[m] = torch.zeros(max_tokens, m.heads, pad8(m.vdim), dtype=dt, device=dev)
+                if m.vdim > 128:
+                    raw = max(raw, m.heads * m.vdim)
+            if r is not None and r not in self._moe:
+                self._moe[r] = LocalExchange(ExchangeGeometry(H, pad8(r.ffn), r.experts, r.top, max_tokens, 1), dev, dtype=dt)
+        ws.raw = torch.empty(max_tokens, raw, dtype=torch.float32, device=dev) if raw else None
+        self.moe = None
+        rows = max_seqs
+        self._logits = torch.empty(rows, pad8(cfg.vocab_size), dtype=torch.float32, device=dev)
+        self.logits = self._logits[:, :cfg.vocab_size]
+        self.next_tokens = torch.empty(rows, dtype=torch.int32, device=dev)
+        self._tiles: dict[tuple[int, int], _HeadTiles] = {}
+        self._blocks: dict = {}
+        self._zero1 = torch.zeros(1, dtype=torch.int32, device=dev)
+        self._scratch: torch.Tensor | None = None
+        self.fixed_kv_split = K.batch_invariant_from_env()
+        self.layer_hook = None           # callable(layer, residual [T, H]) for tests and traces (eager mode only)
+        self.launches = 0
+        self._pending: dict = {}
+
+    # ---- between sublayers ------------------------------------------------------------------------------------------
+    def _between(self, b: Batch, T: int, w: torch.Tensor, conv: torch.Tensor, off: int) -> torch.Tensor:
+        """Residual, norms and input convolution up to the next sublayer; returns its input rows."""
+        ws, p = self.ws, self._pending
+        h = ws.h[self._hi][:T]
+        src = dict(tokens=b.tokens, embed=self.W.embed) if self._x is None else dict(x_in=self._x)
+        xo = ws.x[0 if self._x is None or self._x.data_ptr() != ws.x[0].data_ptr() else 1][:T]
+        K.norm_conv(h, w, self.cfg.norm_groups, self.cfg.rms_eps, conv=conv, x_out=xo, state=self.kv.state, state_off=off,
+                    state_in=b.state_in, state_out=b.state_out, q_start=b.q_start, **src, **p)
+        self._x, self._hi = xo, self._hi ^ 1
+        self.launches += 1
+        return h
+
+    def residual(self, T: int) -> torch.Tensor:
+        """The residual stream [T, H] after everything launched so far (tests and traces)."""
+        x = self._x.clone()
+        p = self._pending
+        if p:
+            y, G = p["y"].float(), self.cfg.norm_groups
+            if "slots" in p:
+                w, idx, n, ident = p["slots"]
+                rows = torch.where((idx >= n)[..., None], ident.float()[:, None], y.view(T, w.shape[1], -1))
+                y = (w[..., None] * rows).sum(1)
+            g = y.view(T, G, -1)
+            x = x + (g / torch.sqrt((g * g).mean(-1, keepdim=True) + self.cfg.rms_eps)).view(T, -1) * p["w_b"]
+        return x
+
+    # ---- mixers -----------------------------------------------------------------------------------------------------
+    def _project(self, i: int, h: torch.Tensor, T: int) -> torch.Tensor:
+        w = self.W.layers[i].w_in
+        a = self.ws.proj[:T * w.shape[0]].view(T, w.shape[0])
+        self.launches += 1
+        return K.linear(h, w, out=a)
+
+    def _block_table(self, S: int, max_q_len: int, per: int):
+        key = (S, max_q_len, per)
+        if key not in self._blocks:
+            nb = (max_q_len + per - 1) // per
+            i32 = dict(dtype=torch.int32, device=self.device)
+            self._blocks[key] = (torch.arange(S, **i32).repeat_interleave(nb).contiguous(), (torch.arange(nb, **i32) * per).repeat(S).contiguous())
+        return self._blocks[key]
+
+    def _latent(self, i: int, m: LatentSpec, h: torch.Tensor, T: int, b: Batch) -> None:
+        L, ws, lw = self.W.layers[i], self.ws, self._lat[m]
+        a = self._project(i, h, T)
+        cache = self.kv.of_layer[i]
+        key = (T, m.heads)
+        if key not in self._tiles:
+            self._tiles[key] = _HeadTiles(T, m.heads, self.device)
+        ht = self._tiles[key]
+        dp, rp, vp, rec = pad8(m.dim), pad8(m.kv_rank), pad8(m.vdim), record_pitch(m)
+        fast = L.w_kb is not None
+        attn = lw.attn[:T]
+        expanded = fast and b.prefill and b.fresh and T >= self.EXPANDED_PREFILL_TOKENS
+        if expanded and lw.lat is None:
+            rows, kw = -(-self.max_tokens // 64) * 64, dict(dtype=self.dtype, device=self.device)
+            lw.lat = torch.zeros(self.max_tokens, m.kv_rank, **kw)
+            lw.k_exp, lw.v_exp = torch.zeros(rows, m.heads * 128, **kw), torch.zeros(rows, m.heads * 128, **kw)
+        slab = lw.q_slab[:m.heads * ht.t_pad * dp].view(m.heads, ht.t_pad, dp)
+        o_slab = lw.o_slab[:m.heads * ht.t_pad * rp].view(m.heads, ht.t_pad, rp)
+        K.latent_prep(a, L.offs["q"], L.offs["kv"], m.heads, m.dim, m.rot_dim, L.kv_norm, lw.inv_freq, b.positions, b.slots, cache,
+                      None if expanded else slab, lw.q_abs[:T], self.cfg.rms_eps, lat_out=lw.lat[:T] if expanded else None)
+        self.launches += 1
+        if expanded:
+            rows = -(-T // 64) * 64
+            K.linear(lw.lat[:T], L.w_kb, out=lw.k_exp[:T])
+            K.linear(lw.lat[:T], L.w_uv.view(m.heads * m.vdim, m.kv_rank), out=lw.v_exp[:T])
+            K.attn_prefill_mla(a[:, L.offs["q"]:L.offs["q"] + m.heads * (m.dim + m.rot_dim)], lw.q_abs[:T], lw.k_exp[:rows], lw.v_exp[:rows],
+                               self._zero1, cache, b.page_table, b.seq_lens, b.q_start, attn, b.max_q_len, m.heads, m.scale,
+                               window=m.window)
+            self.launches += 3
+        else:
+            K.grouped_linear(slab.view(-1, dp), L.w_uk, lw.q_abs, ht.tile_expert, ht.tile_row0, ht.num_tiles, ht.max_tiles, ht.tile_rows,
+                             row_dst=ht.row_dst, ldo=rec, split_k=False)
+            if fast:
+                self._attend_tensor_core(m, lw, T, b, cache, o_slab, ht.t_pad)
+            else:
+                K.latent_attn(lw.q_abs[:T], cache, m.kv_rank, m.rot_dim, b.page_table, b.positions, b.q_start, o_slab, m.scale, m.window)
+            K.grouped_linear(o_slab.view(-1, rp), L.w_uv, attn, ht.tile_expert, ht.tile_row0, ht.num_tiles, ht.max_tiles, ht.tile_rows,
+                             row_dst=ht.row_dst, ldo=vp, split_k=False)
+            self.launches += 3
+        K.latent_gate(attn, a, L.offs["g"], m.heads, m.vdim)
+        K.linear(attn.view(T, -1), L.w_o, out=ws.y[:T])
+        self.launches += 2
+
+    def _attend_tensor_core(self, m: LatentSpec, lw: _LatentWs, T: int, b: Batch, cache: torch.Tensor, o_slab: torch.Tensor, t_pad: int) -> None:
+        S, max_pages = b.page_table.shape
+        bseq, btok = self._block_table(S, b.max_q_len, 128 // m.heads)
+        nb = bseq.numel()
+        tiles = max_pages * 2
+        if m.window > 0:
+            tiles = min(tiles, (m.window + b.max_q_len + 31) // 32 + 1)
+        splits = 1 if b.prefill else max(1, min(K.num_sms() // max(1, nb * 2), max(1, tiles // 8), 32))
+        if self.fixed_kv_split and not b.prefill:
+            splits = K.kv_splits_fixed(max_pages, cap=64)
+        if splits > 1:
+            need = K.mla_scratch_floats(nb, splits)
+            if self._scratch is None or self._scratch.numel() < need:
+                self._scratch = torch.empty(need, dtype=torch.float32, device=self.device)
+        K.mla_attention(lw.q_abs[:T], cache, b.page_table, b.seq_lens, b.q_start, bseq, btok, o_slab, m.scale, splits,
+                        self._scratch if splits > 1 else None, out_tpad=t_pad, window=m.window)
+        self.launches += 1 if splits > 1 else 0
+
+    def _delta_mixer(self, i: int, m: DeltaSpec, h: torch.Tensor, T: int, b: Batch) -> None:
+        L, ws = self.W.layers[i], self.ws
+        a = self._project(i, h, T)
+        off, out = self.kv.offsets[i], self._delta[m][:T]
+        K.delta_step(a, L.offs, m, L, self.kv.state, off["S"], off["conv"], b.state_in, b.state_out, b.q_start, out,
+                     ws.raw if m.vdim > 128 else None, self.cfg.rms_eps)
+        K.linear(out.view(T, -1), L.w_o, out=ws.y[:T])
+        self.launches += 2
+
+    # ---- routed feed-forward ----------------------------------------------------------------------------------------
+    def _experts(self, i: int, r, h: torch.Tensor, T: int) -> tuple:
+        L, moe = self.W.layers[i], self._moe[r]
+        kw = dict(scoring="softmax", bias=L.correction, num_groups=r.groups, topk_groups=r.groups_kept, normalize=False, routed_scale=1.0,
+                  group_score="max")
+        logits = None
+        idx, w = moe.att.idx[:T], moe.att.w[:T]
+        if self.dtype == torch.bfloat16 and T <= self.FUSED_ROUTE_TOKENS and self.cfg.hidden <= 8192:
+            K.norm_route(h, None, 0.0, L.router, None, idx, w, r.top, **kw)
+            self.launches += 1
+        else:
+            logits = K.linear(h, L.router, out=self.ws.router[:T * r.outputs].view(T, r.outputs), out_f32=True,
+                              swap=True if r.outputs % 4 else None)
+            self.launches += 2
+        moe.experts(h, logits, kw, L.w_gate, L.w_up, L.w_down)
+        self.launches += 4
+        return w, idx, r.experts, h
+
+    # ---- whole step -------------------------------------------------------------------------------------------------
+    def layers(self, b: Batch) -> int:
+        T = b.tokens.shape[0]
+        assert T <= self.max_tokens
+        if b.embeds is not None:
+            raise ValueError("media rows are not part of this family")
+        self._x, self._hi, self._pending = None, 0, {}
+        for i, spec in enumerate(self.cfg.layer_specs):
+            L, off, m, r = self.W.layers[i], self.kv.offsets[i], spec.mixer, spec.router
+            h = self._between(b, T, L.norm1, L.canon1, off["canon1"])
+            if isinstance(m, LatentSpec):
+                self._latent(i, m, h, T, b)
+            else:
+                self._delta_mixer(i, m, h, T, b)
+            self._pending = dict(y=self.ws.y[:T], w_b=L.norm1b)
+            if r is not None:
+                h = self._between(b, T, L.norm2, L.canon2, off["canon2"])
+                slots = self._experts(i, r, h, T)
+                self._pending = dict(y=self._moe[r].att.combine, w_b=L.norm2b, slots=slots)
+            if self.layer_hook is not None:
+                self.layer_hook(i, self.residual(T))
+        return T
+
+    def head(self, T: int, rows: torch.Tensor | None = None) -> torch.Tensor:
+        """fp32 logits of ``rows`` (None = all) of the step ``layers`` just ran."""
+        n = T if rows is None else rows.shape[0]
+        xn = self.ws.h[self._hi][:n]
+        if rows is not None and rows.dtype != torch.int32:
+            rows = rows.to(torch.int32)
+        K.norm_conv(xn, self.W.final_norm, self.cfg.norm_groups, self.cfg.rms_eps, x_in=self._x, rows=rows, **self._pending)
+        self.launches += 2
+        return K.linear(xn, self.W.lm_head, out=self.logits[:n], out_f32=True)
+
+    def forward(self, b: Batch) -> torch.Tensor:
+        return self.head(self.layers(b), b.last_rows)
+
+    def greedy(self, logits: torch.Tensor) -> torch.Tensor:
+        self.launches += 1
+        return K.argmax(logits, out=self.next_tokens[:logits.shape[0]])
+
+    def decode_step(self, b: Batch, advance: bool = False) -> torch.Tensor:
+        out = self.greedy(self.forward(b))
+        if advance:
+            K.decode_advance(b.tokens, out, b.positions, b.seq_lens, b.slots, b.page_table)
+            K.swap_ids(b.state_in, b.state_out)
+            self.launches += 2
+        return out

@@ -99,6 +99,9 @@ def linear(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor | None = None, *,
     """
     T, K = x.shape
     N = w.shape[0]
+    if x.dtype == torch.float32:
+        assert residual is None
+        return linear_f32(x, w, out, w_up=w_up)
     assert x.dtype == torch.bfloat16 and w.dtype == torch.bfloat16 and x.is_contiguous() and w.is_contiguous()
     assert w.shape[1] == K
     if out is None:
@@ -124,6 +127,19 @@ def linear(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor | None = None, *,
     return out
 
 
+def linear_f32(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor | None = None, *, w_up: torch.Tensor | None = None) -> torch.Tensor:
+    """``linear`` with fp32 operands and fp32 products (no reduced-precision mode)."""
+    T, K = x.shape
+    N = w.shape[0]
+    assert x.dtype == torch.float32 and w.dtype == torch.float32 and x.stride(1) == 1 and w.is_contiguous() and w.shape[1] == K
+    if out is None:
+        out = torch.empty(T, N, dtype=torch.float32, device=x.device)
+    assert out.dtype == torch.float32
+    _n.check(_n.cuda_lib().cafd_gemm_f32(w.data_ptr(), _ptr(w_up), x.data_ptr(), out.data_ptr(), None, None, None, None, K, N, T,
+                                         x.stride(0), out.stride(0), 0, 0, 0, _stream()), "gemm_f32")
+    return out
+
+
 def grouped_linear(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, tile_expert: torch.Tensor,
                    tile_row0: torch.Tensor, num_tiles: torch.Tensor, max_tiles: int, tile_rows: int, *,
                    w_up: torch.Tensor | None = None, row_dst: torch.Tensor | None = None,
@@ -137,6 +153,13 @@ def grouped_linear(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, tile_exp
     ``out_ptr`` overrides the destination address (a peer GPU's buffer).
     """
     E, N, K = w.shape
+    if x.dtype == torch.float32:
+        assert w.dtype == torch.float32 and wait_flag is None and signal_flag is None
+        _n.check(_n.cuda_lib().cafd_gemm_f32(w.data_ptr(), _ptr(w_up), x.data_ptr(), out_ptr if out_ptr is not None else out.data_ptr(),
+                                             _ptr(row_dst), tile_expert.data_ptr(), tile_row0.data_ptr(), num_tiles.data_ptr(), K, N,
+                                             x.shape[0], x.stride(0), ldo if ldo is not None else out.stride(0), N, max_tiles, tile_rows,
+                                             _stream()), "gemm_f32(grouped)")
+        return
     a = _n.GemmArgs()
     a.w0, a.w1, a.x = w.data_ptr(), _ptr(w_up), x.data_ptr()
     a.out = out_ptr if out_ptr is not None else out.data_ptr()
@@ -233,7 +256,8 @@ def bump_epoch(epoch: torch.Tensor) -> None:
 # ---- MoE -------------------------------------------------------------------------------------------
 def route_topk(logits: torch.Tensor, top_k: int, scoring: str = "softmax", bias: torch.Tensor | None = None,
                num_groups: int = 1, topk_groups: int = 1, normalize: bool = True, routed_scale: float = 1.0,
-               out_idx: torch.Tensor | None = None, out_w: torch.Tensor | None = None):
+               out_idx: torch.Tensor | None = None, out_w: torch.Tensor | None = None, group_score: str = "top2"):
+    """``group_score``: what a group counts by in group-limited routing, the sum of its two best ("top2") or its best ("max")."""
     T, E = logits.shape
     assert logits.dtype == torch.float32 and logits.is_contiguous()
     if out_idx is None:
@@ -242,7 +266,7 @@ def route_topk(logits: torch.Tensor, top_k: int, scoring: str = "softmax", bias:
         out_w = torch.empty(T, top_k, dtype=torch.float32, device=logits.device)
     _n.check(_n.cuda_lib().cafd_route_topk(logits.data_ptr(), _ptr(bias), out_idx.data_ptr(), out_w.data_ptr(), T, E,
                                            top_k, int(scoring == "sigmoid"), num_groups, topk_groups, int(normalize),
-                                           routed_scale, _stream()), "route_topk")
+                                           routed_scale, int(group_score == "max"), _stream()), "route_topk")
     return out_idx, out_w
 
 
@@ -287,13 +311,13 @@ _plan_scratch: dict = {}
 _route_scratch: dict = {}
 
 
-def norm_route(h: torch.Tensor, ln_w: torch.Tensor, eps: float, router_w: torch.Tensor, x_out: torch.Tensor, out_idx: torch.Tensor,
+def norm_route(h: torch.Tensor, ln_w: torch.Tensor | None, eps: float, router_w: torch.Tensor, x_out: torch.Tensor | None, out_idx: torch.Tensor,
                out_w: torch.Tensor, top_k: int, *, scoring: str = "softmax", bias: torch.Tensor | None = None, num_groups: int = 1,
                topk_groups: int = 1, normalize: bool = True, routed_scale: float = 1.0,
-               logits_out: torch.Tensor | None = None) -> None:
+               logits_out: torch.Tensor | None = None, group_score: str = "top2") -> None:
     """x_out = RMSNorm(h) * ln_w, router scores x_out @ router_w.T and the top-k routing of every row in one launch
     (grid token x 8 expert groups; meant for decode-sized batches).  ``logits_out`` [T, E] fp32 receives the scores
-    (a per-device scratch is used when it is not given)."""
+    (a per-device scratch is used when it is not given).  ``ln_w`` None: the rows are normalised already."""
     T, H = h.shape
     E = router_w.shape[0]
     key = h.device.index
@@ -304,10 +328,10 @@ def norm_route(h: torch.Tensor, ln_w: torch.Tensor, eps: float, router_w: torch.
         _route_scratch[key] = sc
     buf = logits_out if logits_out is not None else sc[0].view(-1)[:T * E].view(T, E)
     assert buf.is_contiguous()
-    _n.check(_n.cuda_lib().cafd_norm_route(h.data_ptr(), ln_w.data_ptr(), eps, router_w.data_ptr(), _ptr(bias), x_out.data_ptr(),
+    _n.check(_n.cuda_lib().cafd_norm_route(h.data_ptr(), _ptr(ln_w), eps, router_w.data_ptr(), _ptr(bias), _ptr(x_out),
                                            out_idx.data_ptr(), out_w.data_ptr(), buf.data_ptr(), sc[1].data_ptr(), T, H, E, top_k,
                                            int(scoring == "sigmoid"), num_groups, topk_groups, int(normalize), routed_scale,
-                                           _stream()), "norm_route")
+                                           int(group_score == "max"), _stream()), "norm_route")
 
 
 def moe_dispatch(x: torch.Tensor, idx: torch.Tensor, dest_row: torch.Tensor, layout: "_n.MoeLayout",
@@ -466,14 +490,16 @@ def mla_scratch_floats(n_blocks: int, splits: int) -> int:
 def mla_attention(q_abs: torch.Tensor, cache: torch.Tensor, page_table: torch.Tensor, seq_lens: torch.Tensor,
                   q_start: torch.Tensor, block_seq: torch.Tensor, block_tok0: torch.Tensor, out: torch.Tensor,
                   scale: float, splits: int = 1, scratch: torch.Tensor | None = None, out_tpad: int = 0,
-                  sparse_idx: torch.Tensor | None = None, gathered: torch.Tensor | None = None) -> torch.Tensor:
+                  sparse_idx: torch.Tensor | None = None, gathered: torch.Tensor | None = None, window: int = 0) -> torch.Tensor:
     """Absorbed MLA: q_abs [tokens, heads, 576] (512 latent-projected + 64 rope), cache [pages, 64, 576]
     (page 0 zero), out [tokens, heads, 512] = softmax(q c^T * scale) c[:, :512] with the causal rule
     that query token i of a sequence sees kv positions <= seq_len - q_len + i.  With ``out_tpad`` > 0
     the output is head-major: out [heads, out_tpad, 512].  With ``sparse_idx`` [tokens, k] (ascending positions,
     -1 padded; from ``index_topk``) each block must be a single token (``mla_blocks(q_lens, 128)``) and the
     token attends to its listed positions only.  With ``gathered`` [blocks, k, 576] (from ``mla_fp8_gather``) the
-    listed records are read from that buffer instead of the cache, which may then be None."""
+    listed records are read from that buffer instead of the cache, which may then be None.  ``window`` > 0: a query at
+    position t sees positions (t - window, t] only; tiles wholly before a block's windows are not read."""
+    assert not (window and sparse_idx is not None)
     T, heads, rec = q_abs.shape
     assert rec == 576 and 128 % heads == 0 and q_abs.is_contiguous() and out.is_contiguous()
     _, max_pages = page_table.shape
@@ -492,7 +518,7 @@ def mla_attention(q_abs: torch.Tensor, cache: torch.Tensor, page_table: torch.Te
                                               q_start.data_ptr(), block_seq.data_ptr(), block_tok0.data_ptr(), out.data_ptr(),
                                               _ptr(scratch), status_word(q_abs.device).data_ptr(), T * heads,
                                               block_seq.numel(), num_pages, max_pages, heads, splits, out_tpad, scale,
-                                              _ptr(sparse_idx), sparse_idx.shape[1] if sparse_idx is not None else 0, _stream()),
+                                              _ptr(sparse_idx), sparse_idx.shape[1] if sparse_idx is not None else 0, window, _stream()),
              "mla_attention")
     return out
 
@@ -590,20 +616,21 @@ def mla_prep_a(a: torch.Tensor, q_lora: int, q_norm_w: torch.Tensor | None, kv_n
 
 def attn_prefill_mla(q_nope: torch.Tensor, q_rope: torch.Tensor, k_exp: torch.Tensor, v_exp: torch.Tensor, kv_tmp_start: torch.Tensor,
                      latent_cache: torch.Tensor, page_table: torch.Tensor, seq_lens: torch.Tensor, q_start: torch.Tensor,
-                     out: torch.Tensor, max_q_len: int, heads: int, scale: float, qr_col0: int = 512) -> torch.Tensor:
+                     out: torch.Tensor, max_q_len: int, heads: int, scale: float, qr_col0: int = 512, window: int = 0) -> torch.Tensor:
     """MLA prefill in expanded form.  q_nope [T, heads * 192] (first 128 columns of each head are used), q_rope
     [T, heads, 576]-like buffer holding the rotated rope dims at ``qr_col0`` of every head, k_exp / v_exp
     [rows, heads * 128] (kv_b applied to the cached latents in order; rows a multiple of 64), the latent cache for
     the shared rope keys.  out [T, heads, 128]."""
     T = q_nope.shape[0]
     S, max_pages = page_table.shape
+    assert q_nope.stride(1) == 1
     qs, qrs = q_nope.shape[1] // heads, q_rope.numel() // (q_rope.shape[0] * heads)
     assert k_exp.shape[0] % 64 == 0 and k_exp.shape[1] == heads * 128 and k_exp.is_contiguous() and v_exp.is_contiguous()
-    _n.check(_n.cuda_lib().cafd_attn_prefill_mla(q_nope.data_ptr(), qs, q_rope.data_ptr(), qrs, qr_col0, k_exp.data_ptr(),
+    _n.check(_n.cuda_lib().cafd_attn_prefill_mla(q_nope.data_ptr(), q_nope.stride(0), qs, q_rope.data_ptr(), qrs, qr_col0, k_exp.data_ptr(),
                                                  v_exp.data_ptr(), k_exp.shape[0], kv_tmp_start.data_ptr(), latent_cache.data_ptr(),
                                                  page_table.data_ptr(), seq_lens.data_ptr(), q_start.data_ptr(), out.data_ptr(),
                                                  status_word(q_nope.device).data_ptr(), T, S, max_q_len, latent_cache.shape[0],
-                                                 max_pages, heads, scale, _stream()), "attn_prefill_mla")
+                                                 max_pages, heads, scale, window, _stream()), "attn_prefill_mla")
     return out
 
 
@@ -638,6 +665,100 @@ def mla_unabsorb_small(o_lat: torch.Tensor, w_uv: torch.Tensor, attn: torch.Tens
     assert T <= MLA_SMALL_ROWS and w_uv.shape == (heads, 128, 512) and w_uv.is_contiguous() and attn.is_contiguous()
     _n.check(_n.cuda_lib().cafd_mla_unabsorb_small(o_lat.data_ptr(), t_pad, w_uv.data_ptr(), attn.data_ptr(), T, heads, _stream()),
              "mla_unabsorb_small")
+
+
+# ---- per-layer hybrids (csrc/hybrid_norm.cu, latent.cu, delta.cu) --------------------------------------------
+def norm_conv(h_out: torch.Tensor, w: torch.Tensor, groups: int, eps: float, *, tokens: torch.Tensor | None = None,
+              embed: torch.Tensor | None = None, x_in: torch.Tensor | None = None, y: torch.Tensor | None = None,
+              w_b: torch.Tensor | None = None, slots: tuple | None = None, conv: torch.Tensor | None = None,
+              x_out: torch.Tensor | None = None, rows: torch.Tensor | None = None, state: torch.Tensor | None = None, state_off: int = 0,
+              state_in: torch.Tensor | None = None, state_out: torch.Tensor | None = None, q_start: torch.Tensor | None = None,
+              run: int = 0) -> None:
+    """x = embed[tokens] or ``x_in`` (fp32); x += groupnorm(y) * w_b; h = groupnorm(x) * w; h_out = h + causal_conv(h).
+
+    ``slots`` = (weights [T, k], ids [T, k], number of experts, identity rows [T, H]): ``y`` then holds the routed experts'
+    rows [T * k, H] and is their weighted sum.  ``conv`` [taps, H] fp32 (last row = current token) with the sequences'
+    earlier inputs in ``state`` [slots, floats] at ``state_off``.  ``rows``: compute only these rows (no convolution)."""
+    a = _n.NormArgs()
+    H = w.shape[0]
+    a.tokens, a.embed, a.x_in, a.y = _ptr(tokens), _ptr(embed), _ptr(x_in), _ptr(y)
+    a.w_b, a.w, a.conv, a.x_out, a.h_out, a.row_idx = _ptr(w_b), w.data_ptr(), _ptr(conv), _ptr(x_out), h_out.data_ptr(), _ptr(rows)
+    a.vocab = embed.shape[0] if embed is not None else 0
+    a.T, a.H, a.groups, a.eps, a.run = h_out.shape[0], H, groups, eps, run
+    a.ldy = y.stride(0) if y is not None else 0
+    assert h_out.is_contiguous() and h_out.shape[1] == H and w.dtype == torch.float32
+    if slots is not None:
+        sw, si, n, ident = slots
+        a.slot_w, a.slot_idx, a.n_experts, a.ident, a.top_k = sw.data_ptr(), si.data_ptr(), n, ident.data_ptr(), sw.shape[1]
+        assert y.stride(0) == H and ident.stride(0) == H and sw.is_contiguous() and si.is_contiguous()
+    if conv is not None:
+        a.taps, a.S = conv.shape[0], q_start.shape[0] - 1
+        a.state, a.state_in, a.state_out, a.q_start = state.data_ptr(), state_in.data_ptr(), state_out.data_ptr(), q_start.data_ptr()
+        a.slot_stride, a.state_off = state.stride(0), state_off
+        assert conv.is_contiguous() and conv.dtype == torch.float32 and state.dtype == torch.float32
+    _n.check(_n.cuda_lib().cafd_norm_conv(C.byref(a), int(h_out.dtype == torch.float32), _stream()), "norm_conv")
+
+
+def swap_ids(a: torch.Tensor, b: torch.Tensor) -> None:
+    _n.check(_n.cuda_lib().cafd_swap_ids(a.data_ptr(), b.data_ptr(), a.numel(), _stream()), "swap_ids")
+
+
+def latent_prep(a: torch.Tensor, q_off: int, kv_off: int, heads: int, dim: int, rot: int, norm_w: torch.Tensor, inv_freq: torch.Tensor,
+                positions: torch.Tensor, slots: torch.Tensor, cache: torch.Tensor, slab: torch.Tensor | None, q_abs: torch.Tensor,
+                eps: float, lat_out: torch.Tensor | None = None) -> None:
+    """One launch per step and layer: latent norm, rotations, the cache record at ``slots`` and the query parts (unrotated
+    into ``slab`` [heads, t_pad, dim_pad], rotated into ``q_abs`` [T, heads, rec])."""
+    p = _n.LatentPrep()
+    p.a, p.norm_w, p.inv_freq, p.positions, p.slots = a.data_ptr(), norm_w.data_ptr(), inv_freq.data_ptr(), positions.data_ptr(), slots.data_ptr()
+    p.cache, p.slab, p.q_abs, p.lat_out = cache.data_ptr(), _ptr(slab), q_abs.data_ptr(), _ptr(lat_out)
+    p.lda, p.q_off, p.kv_off, p.heads, p.dim, p.rot, p.rank = a.stride(0), q_off, kv_off, heads, dim, rot, norm_w.shape[0]
+    p.rec, p.T, p.eps = cache.shape[-1], a.shape[0], eps
+    p.dim_pad, p.t_pad = (slab.shape[2], slab.shape[1]) if slab is not None else (0, 0)
+    assert cache.is_contiguous() and q_abs.is_contiguous() and q_abs.shape[-1] == p.rec and a.dtype == cache.dtype == q_abs.dtype
+    _n.check(_n.cuda_lib().cafd_latent_prep(C.byref(p), int(a.dtype == torch.float32), _stream()), "latent_prep")
+
+
+def latent_attn(q_abs: torch.Tensor, cache: torch.Tensor, rank: int, rot: int, page_table: torch.Tensor, positions: torch.Tensor,
+                q_start: torch.Tensor, out: torch.Tensor, scale: float, window: int) -> None:
+    """Absorbed latent attention at any sizes: q_abs [T, heads, rec], out [heads, t_pad, ld] head-major."""
+    p = _n.LatentAttn()
+    p.q_abs, p.cache, p.page_table, p.positions = q_abs.data_ptr(), cache.data_ptr(), page_table.data_ptr(), positions.data_ptr()
+    p.q_start, p.out = q_start.data_ptr(), out.data_ptr()
+    p.T, p.heads, p.rec = q_abs.shape
+    p.S, p.max_pages = page_table.shape
+    p.rank, p.rot, p.window, p.t_pad, p.out_ld, p.scale = rank, rot, window, out.shape[1], out.shape[2], scale
+    assert q_abs.is_contiguous() and out.is_contiguous() and page_table.is_contiguous() and q_start.shape[0] == p.S + 1
+    _n.check(_n.cuda_lib().cafd_latent_attn(C.byref(p), int(q_abs.dtype == torch.float32), _stream()), "latent_attn")
+
+
+def latent_gate(attn: torch.Tensor, gate: torch.Tensor, g_off: int, heads: int, vdim: int) -> None:
+    """attn [T, heads, ld] *= sigmoid(gate row's head sections), in place."""
+    T, _, ld = attn.shape
+    _n.check(_n.cuda_lib().cafd_latent_gate(attn.data_ptr(), gate.data_ptr(), T, heads, vdim, ld, gate.stride(0), g_off,
+                                            int(attn.dtype == torch.float32), _stream()), "latent_gate")
+
+
+def delta_args(proj: torch.Tensor, offs: dict, m, w, state: torch.Tensor, s_off: int, c_off: int, state_in: torch.Tensor,
+               state_out: torch.Tensor, q_start: torch.Tensor, out: torch.Tensor, raw: torch.Tensor | None, eps: float) -> "_n.DeltaArgs":
+    """Arguments shared by the delta-rule kernels.  ``m`` carries heads / kv_heads / dim / vdim / conv, ``w`` the layer's
+    conv_w [channels, taps], A_log, dt_bias and out_norm (fp32), ``out`` [T, heads, vdim padded]."""
+    p = _n.DeltaArgs()
+    p.proj, p.conv_w, p.A_log, p.dt_bias, p.norm_w = proj.data_ptr(), w.conv_w.data_ptr(), w.A_log.data_ptr(), w.dt_bias.data_ptr(), w.out_norm.data_ptr()
+    p.state, p.state_in, p.state_out, p.q_start = state.data_ptr(), state_in.data_ptr(), state_out.data_ptr(), q_start.data_ptr()
+    p.out, p.raw = out.data_ptr(), _ptr(raw)
+    p.slot_stride, p.s_off, p.c_off, p.ld = state.stride(0), s_off, c_off, proj.stride(0)
+    for n in ("q", "k", "v", "g", "b", "a"):
+        setattr(p, n + "_off", offs[n])
+    p.T, p.S, p.heads, p.kv_heads, p.dim, p.vdim, p.taps = proj.shape[0], q_start.shape[0] - 1, m.heads, m.kv_heads, m.dim, m.vdim, m.conv
+    p.out_vd, p.eps = out.shape[2], eps
+    assert out.is_contiguous() and out.dtype == proj.dtype and state.dtype == torch.float32
+    return p
+
+
+def delta_step(proj: torch.Tensor, *args, **kw) -> None:
+    """Gated delta rule over any mix of portions, token by token (see ``delta_args``)."""
+    p = delta_args(proj, *args, **kw)
+    _n.check(_n.cuda_lib().cafd_delta_step(C.byref(p), int(proj.dtype == torch.float32), _stream()), "delta_step")
 
 
 # ---- sampling ---------------------------------------------------------------------------------------------

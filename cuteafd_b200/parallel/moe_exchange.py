@@ -109,12 +109,13 @@ class ExpertSide:
     _dq_scratch: dict = {}           # per device: one layer's experts expanded to bf16 (shared by all regions)
 
     def __init__(self, geo: ExchangeGeometry, device: torch.device, slab: torch.Tensor | None = None,
-                 meta: torch.Tensor | None = None, flags: torch.Tensor | None = None, num_layers: int = 1):
+                 meta: torch.Tensor | None = None, flags: torch.Tensor | None = None, num_layers: int = 1,
+                 dtype: torch.dtype = torch.bfloat16):
         self.geo = geo
-        self.slab = slab if slab is not None else torch.zeros(geo.max_rows, geo.hidden, dtype=torch.bfloat16, device=device)
+        self.slab = slab if slab is not None else torch.zeros(geo.max_rows, geo.hidden, dtype=dtype, device=device)
         self.meta = meta if meta is not None else torch.zeros(geo.meta_ints, dtype=torch.int32, device=device)
         self.flags = flags if flags is not None else torch.zeros(num_layers, dtype=torch.int32, device=device)
-        self.hbuf = torch.zeros(geo.max_rows, geo.expert_ffn, dtype=torch.bfloat16, device=device)
+        self.hbuf = torch.zeros(geo.max_rows, geo.expert_ffn, dtype=dtype, device=device)
         self.done = torch.zeros(4, dtype=torch.int32, device=device)
         mt = geo.max_tiles
         self.num_tiles = self.meta[0:1]
@@ -123,7 +124,7 @@ class ExpertSide:
         self.row_dst = self.meta[16 + 2 * mt:]
         # E4M3 wire format: the same receive slab read as [max_rows, H] bytes followed by [max_rows, H / 128] fp32 scales
         # (fits: H + H / 32 bytes per row against 2 H for bf16), so a step may arrive in either form.
-        if geo.hidden % 128 == 0:
+        if geo.hidden % 128 == 0 and dtype == torch.bfloat16:
             raw = self.slab.view(-1).view(torch.uint8)
             nq = geo.max_rows * geo.hidden
             self.wire_q = raw[:nq].view(torch.float8_e4m3fn).view(geo.max_rows, geo.hidden)
@@ -221,13 +222,13 @@ class AttentionSide:
     """Buffers the attention rank owns: routes, plan output, the combine buffer and its flags."""
 
     def __init__(self, geo: ExchangeGeometry, device: torch.device, combine: torch.Tensor | None = None,
-                 flags: torch.Tensor | None = None, num_layers: int = 1):
+                 flags: torch.Tensor | None = None, num_layers: int = 1, dtype: torch.dtype = torch.bfloat16):
         self.geo = geo
         T, k = geo.max_tokens, geo.top_k
         self.idx = torch.zeros(T, k, dtype=torch.int32, device=device)
         self.w = torch.zeros(T, k, dtype=torch.float32, device=device)
         self.dest_row = torch.zeros(T * k, dtype=torch.int32, device=device)
-        self.combine = combine if combine is not None else torch.zeros(T * k, geo.hidden, dtype=torch.bfloat16, device=device)
+        self.combine = combine if combine is not None else torch.zeros(T * k, geo.hidden, dtype=dtype, device=device)
         # one word per (layer, expert rank), written by that rank's fc2 kernel
         self.flags = flags if flags is not None else torch.zeros(num_layers * _n.MAX_RANKS, dtype=torch.int32, device=device)
         self.done = torch.zeros(4, dtype=torch.int32, device=device)
@@ -270,7 +271,9 @@ class AttentionSide:
             K.route_topk(logits, g.top_k, out_idx=idx, out_w=w, **route_kw)
         for r in range(g.n_expert_ranks):
             self.layout.flag[r] = self._rank_ptrs[r][2] + 4 * layer
-        if (T * g.top_k <= self.FUSED_DISPATCH_ROWS and T * g.top_k * g.hidden * 2 <= self.FUSED_DISPATCH_BYTES
+        if x.dtype == torch.float32:              # rows travel as bytes: a 32-bit row is a bf16 row of twice the length
+            x = x.view(torch.bfloat16)
+        if (T * g.top_k <= self.FUSED_DISPATCH_ROWS and T * g.top_k * x.shape[1] * 2 <= self.FUSED_DISPATCH_BYTES
                 and not wire_fp8):
             K.moe_plan(idx, g.num_experts, tile_rows, self.layout, self.dest_row, self.expert_count, x=x, epoch=epoch)
         else:
@@ -289,13 +292,23 @@ class AttentionSide:
 class LocalExchange:
     """Single-GPU MoE: attention side and expert side in one process, stream-ordered."""
 
-    def __init__(self, geo: ExchangeGeometry, device: torch.device):
+    def __init__(self, geo: ExchangeGeometry, device: torch.device, dtype: torch.dtype = torch.bfloat16):
         assert geo.n_expert_ranks == 1
         self.geo = geo
-        self.att = AttentionSide(geo, device)
-        self.exp = ExpertSide(geo, device)
+        self.att = AttentionSide(geo, device, dtype=dtype)
+        self.exp = ExpertSide(geo, device, dtype=dtype)
         self.att.bind_rank(0, self.exp.slab.data_ptr(), self.exp.meta.data_ptr(), self.exp.flags.data_ptr())
         self.epoch = torch.zeros(1, dtype=torch.int32, device=device)
+
+    def experts(self, x: torch.Tensor, logits: torch.Tensor | None, route_kw: dict, w_gate: torch.Tensor, w_up: torch.Tensor,
+                w_down: torch.Tensor) -> None:
+        """Everything but the combine: the unweighted rows are left in ``att.combine`` [(token, slot), hidden], the routes in
+        ``att.idx`` / ``att.w``.  Routes to ids at or above the number of experts (identity outputs) take no expert row."""
+        T = x.shape[0]
+        g = self.geo
+        tile_rows = pick_tile_rows(T, g.top_k, g.num_experts)
+        self.att.dispatch(x, logits, route_kw, tile_rows, 0, self.epoch)
+        self.exp.run(w_gate, w_up, w_down, tile_rows, 0, self.epoch, self.att.combine.data_ptr(), None, wait=False)
 
     def forward(self, x: torch.Tensor, logits: torch.Tensor, route_kw: dict, w_gate: torch.Tensor, w_up: torch.Tensor,
                 w_down: torch.Tensor, out: torch.Tensor, *, shared: torch.Tensor | None = None,

@@ -22,6 +22,9 @@ MoeFn = Callable[[int, torch.Tensor, torch.Tensor, torch.Tensor], torch.Tensor]
 def init_weights(cfg: ModelConfig, seed: int = 0, dtype: torch.dtype = torch.float32, std: float = 0.02,
                  device: str = "cpu") -> dict[str, torch.Tensor]:
     """Random-init parameters N(0, std), norm weights one, router bias zero."""
+    if cfg.is_hybrid:
+        from .hybrid import init_hybrid_weights
+        return init_hybrid_weights(cfg, seed, dtype)
     g = torch.Generator(device="cpu").manual_seed(seed)
 
     def w(*shape: int) -> torch.Tensor:
@@ -143,6 +146,9 @@ class RefDecoder:
         xf = x.float()
         act = torch.nn.functional.silu(xf @ p[prefix + "gate_proj.weight"].float().T) * (xf @ p[prefix + "up_proj.weight"].float().T)
         self.observe(prefix + "down_proj", act.to(x.dtype))
+
+    def new_state(self) -> KvState:
+        return KvState(self.cfg)
 
     # ---- pieces ---------------------------------------------------------------------------
     def expert_stack(self, layer: int, lo: int = 0, hi: int | None = None):
@@ -328,3 +334,11 @@ class RefDecoder:
             out_t.append(torch.cat(toks))
             out_l.append(torch.stack(ls))
         return torch.stack(out_t), torch.stack(out_l)
+
+
+def decoder_for(cfg: ModelConfig, params: dict[str, torch.Tensor]):
+    """The oracle decoder of a configuration."""
+    if cfg.is_hybrid:
+        from .hybrid import HybridRefDecoder
+        return HybridRefDecoder(cfg, params)
+    return RefDecoder(cfg, params)

@@ -9,6 +9,7 @@ rust/crates/cuteafd-bench/examples/fake_server.rs:1-50).
 """
 from __future__ import annotations
 
+import contextlib
 from dataclasses import dataclass
 
 import torch
@@ -32,14 +33,17 @@ class OracleBackend:
 
     def __init__(self, cfg: ModelConfig, params: dict[str, torch.Tensor], total_pages: int = 512, prefill_chunk: int = 64,
                  max_decode_rows: int = 64, fail_on_step: int | None = None, host_slots: int = 0):
-        from ..ref.model import RefDecoder
-        self.cfg, self.model = cfg, RefDecoder(cfg, params)
+        from ..ref.model import decoder_for
+        self.cfg, self.model = cfg, decoder_for(cfg, params)
         self.vocab_size, self.prefill_chunk, self.max_decode_rows = cfg.vocab_size, prefill_chunk, max_decode_rows
         self.total_pages = total_pages
         self.pool = make_pool(total_pages)
         self.table = SequenceTable(self.pool)
         self.prefix = PrefixCache(self.pool, self.table, max_pages=total_pages // 2)
+        self.prefix.whole_snapshots = cfg.is_hybrid      # recurrent layers resume only where a snapshot kept their state
         self.tier = None
+        if host_slots and cfg.is_hybrid:
+            raise ValueError("the host cache tier does not hold recurrent state")
         if host_slots:                            # host tier on a virtual clock: the oracle's KV rides in the snapshot marks
             from .host_tier import HostTier
             from .hostcache import HostCache, StubCopyEngine
@@ -88,11 +92,13 @@ class OracleBackend:
         return toks, status
 
     def open(self, tokens: list[int], cold: bool = False) -> tuple[_Handle, int]:
-        from ..ref.model import KvState
         if cold:                                   # probe: compute the whole prompt, whatever the cache holds
-            return _Handle(self.table.new(), KvState(self.cfg)), 0
+            return _Handle(self.table.new(), self.model.new_state()), 0
         seq, m = self.prefix.admit(tokens)
-        kv = KvState(self.cfg)
+        if self.cfg.is_hybrid:
+            import copy
+            return _Handle(seq, copy.deepcopy(m.snapshot.mark) if m.length else self.model.new_state()), m.length
+        kv = self.model.new_state()
         got = self.tier.try_restore(tokens, m.length) if self.tier is not None else None
         if got is not None and got[2].mark is not None:
             self.table.free(seq)
@@ -197,7 +203,16 @@ class EngineBackend:
         self.gen = Generator(engine, self.pool, max_pages_per_seq, max_decode_rows, prefill_chunk, use_graphs)
         self.table = self.gen.table
         self.prefix = PrefixCache(self.pool, self.table, max_pages=num_pages // 2)
+        # Recurrent layers: a snapshot holds a reference to the slot of the state at its end, and only whole snapshots are
+        # resumed from; a slot that a step needs is taken from the least recently used snapshot.
+        self.states = self.gen.states
+        if self.states is not None:
+            self.prefix.whole_snapshots = True
+            self.prefix.on_release = lambda s: self.states.release(s.mark) if s.mark is not None else None
+            self.states.on_exhausted = self._evict_state
         self.tier = None
+        if host_cache_bytes > 0 and self.states is not None:
+            raise ValueError("the pinned-host cache tier does not hold recurrent state: run without a host cache")
         if host_cache_bytes > 0 and engine.device.type == "cuda":
             # pinned-host tier behind the device cache: evicted snapshots are copied out on a side stream and come
             # back through the same engine when a later request asks for their prefix
@@ -221,7 +236,8 @@ class EngineBackend:
         self.max_pages = max_pages_per_seq
         # longest sequence one page-table row can describe (speculative rows of the last step included)
         self.max_context_tokens = max(PAGE, (max_pages_per_seq - 1) * PAGE)
-        self.bufs = StepBuffers(max_decode_rows * 8, max_decode_rows, max_pages_per_seq, engine.device)
+        # (recurrent layers run up to 7 accepted rows of a partly rejected step again in front of the next one)
+        self.bufs = StepBuffers(max_decode_rows * (16 if self.states is not None else 8), max_decode_rows, max_pages_per_seq, engine.device)
         self.quarantined: list[_Handle] = []
         self._sel = None
         self._last_batch = None
@@ -294,10 +310,31 @@ class EngineBackend:
         if got is not None:
             self.table.free(seq)
             return _Handle(got[0]), got[1]
+        if self.states is not None and m.length:
+            self.states.retain(m.snapshot.mark)
+            seq.state, seq.state_len = m.snapshot.mark, m.length
         return _Handle(seq), m.length
+
+    def _evict_state(self) -> bool:
+        """Release the least recently used snapshot that holds a state slot."""
+        held = [s for s in self.prefix.snapshots.values() if s.mark is not None]
+        if not held:
+            return False
+        self.prefix.release(min(held, key=lambda s: s.last_use).sid)
+        return True
+
+    def _states_for(self, b, seqs: list) -> list[int] | None:
+        """Stage the state slots of a step over ``seqs``; returns the slots it writes."""
+        if self.states is None:
+            return None
+        ins, outs = self.states.begin(seqs)
+        b.set_states(ins, outs)
+        return outs
 
     def prefill(self, h: _Handle, tokens: list[int], last: bool):
         from ..models.gqa_moe import Batch
+        if self.states is not None:
+            return self.prefill_packed([(h, tokens, last)])[0]
         seq = h.seq
         start, n = seq.kv_len, len(tokens)
         self.table.reserve(seq, start + n, copy_page=self._copy_page)
@@ -340,10 +377,55 @@ class EngineBackend:
     def prefill_packed(self, items: list) -> list:
         """Chunks of several prompts in one forward step: [(handle, tokens, last)] -> per item the fp32 logits of its
         last row when ``last`` (on the host), else None.  Media rows and the MTP fill work as in ``prefill``."""
+        S = len(items)
+        batch, nxt, done = self._ragged([(h, toks) for h, toks, _ in items])
+        with done:
+            logits = self.engine.forward(batch)
+            if self.has_mtp:
+                self.engine.mtp_forward(0, batch, torch.tensor([t if t < self.vocab_size else 0 for t in nxt], dtype=torch.int32).to(self.engine.device))
+            host = logits[:S].float().cpu() if any(last for _, _, last in items) else None
+        return [host[i:i + 1] if last else None for i, (_, _, last) in enumerate(items)]
+
+    def step(self, items: list) -> list[torch.Tensor]:
+        """One engine step over portions of any lengths, prompt portions beside single decoded tokens: [(handle, tokens,
+        wanted places)] -> per item the fp32 logits [wanted, vocab] on the host.  A step of more tokens than the engine
+        takes at once is cut; every item's tokens keep their order."""
+        out = [[] for _ in items]
+        pos = [0] * len(items)
+        while any(p < len(t) for p, (_, t, _) in zip(pos, items)):
+            part, room = [], self.prefill_chunk
+            for i, (h, toks, want) in enumerate(items):
+                n = min(room, len(toks) - pos[i])
+                if n > 0 and len(part) < 16:
+                    part.append((i, h, toks[pos[i]:pos[i] + n]))
+                    room -= n
+            batch, _, done = self._ragged([(h, t) for _, h, t in part])
+            rows, owner, o = [], [], 0
+            for i, _, t in part:
+                for w in items[i][2]:
+                    if pos[i] <= w < pos[i] + len(t):
+                        rows.append(o + w - pos[i])
+                        owner.append(i)
+                o += len(t)
+            dev, cap = self.engine.device, self.engine.logits.shape[0]
+            with done:
+                T = self.engine.layers(batch)
+                for c in range(0, len(rows), cap):
+                    got = self.engine.head(T, torch.tensor(rows[c:c + cap], dtype=torch.int32).to(dev)).float().cpu()
+                    for i, row in zip(owner[c:c + cap], got):
+                        out[i].append(row)
+            for i, _, t in part:
+                pos[i] += len(t)
+        return [torch.stack(r) if r else torch.empty(0, self.vocab_size) for r in out]
+
+    def _ragged(self, items: list, replay: bool = False):
+        """Stage one multi-sequence step of portions [(handle, tokens)]: (batch, each row's next token, context that books
+        the tokens when the step it encloses went through).  ``replay``: the tokens are the ones each recurrent state has
+        yet to see; their K/V counts already."""
         from ..models.gqa_moe import Batch
         from ..media.processor import overrides_for
         from .generate import StepBuffers
-        S, T = len(items), sum(len(t) for _, t, _ in items)
+        S, T = len(items), sum(len(t) for _, t in items)
         if getattr(self, "_pack_bufs", None) is None:
             self._pack_bufs = StepBuffers(self.prefill_chunk, 16, self.max_pages, self.engine.device)
         b = self._pack_bufs
@@ -351,9 +433,9 @@ class EngineBackend:
         V = self.vocab_size
         pt = b.page_table[0].view(b.max_seqs, self.max_pages)
         o, rows, vals, nxt = 0, [], [], []
-        for i, (h, toks, _) in enumerate(items):
+        for i, (h, toks) in enumerate(items):
             seq = h.seq
-            start, n = seq.kv_len, len(toks)
+            start, n = seq.state_len if replay else seq.kv_len, len(toks)
             self.table.reserve(seq, start + n, copy_page=self._copy_page)
             if any(t >= V for t in toks):
                 ov = overrides_for(getattr(h, "media", None), start, n)
@@ -372,23 +454,45 @@ class EngineBackend:
             nxt += toks[1:] + toks[-1:]
             o += n
         b.q_start[0][S] = T
+        seqs = [h.seq for h, _ in items]
+        outs = self._states_for(b, seqs)
         b.upload()
         self._stage_embeddings(b.tokens[0][:T])
         batch = Batch(b.tokens[1][:T], b.positions[1][:T], b.slots[1][:T], pt_dev(b, self.max_pages)[:S], b.seq_lens[1][:S],
-                      b.q_start[1][:S + 1], max(len(t) for _, t, _ in items), True, b.last_rows[1][:S], fresh=False)
+                      b.q_start[1][:S + 1], max(len(t) for _, t in items), True, b.last_rows[1][:S],
+                      fresh=outs is not None and S == 1 and seqs[0].kv_len == 0, **(b.states(S) if outs is not None else {}))
         if rows:
             dev = self.engine.device
             batch.embeds = (torch.tensor(rows, dtype=torch.long).to(dev), torch.cat(vals).to(dev, torch.bfloat16))
-        logits = self.engine.forward(batch)
-        if self.has_mtp:
-            self.engine.mtp_forward(0, batch, torch.tensor([t if t < V else 0 for t in nxt], dtype=torch.int32).to(self.engine.device))
-        host = logits[:S].float().cpu() if any(last for _, _, last in items) else None
-        out = []
-        for i, (h, toks, last) in enumerate(items):
-            h.seq.tokens.extend(toks)
-            h.seq.kv_len += len(toks)
-            out.append(host[i:i + 1] if last else None)
-        return out
+
+        @contextlib.contextmanager
+        def booked():
+            with self._state_step(seqs, outs):
+                yield
+                if not replay:
+                    for h, toks in items:
+                        h.seq.tokens.extend(toks)
+                        h.seq.kv_len += len(toks)
+        return batch, nxt, booked()
+
+    @contextlib.contextmanager
+    def _state_step(self, seqs: list, outs: list[int] | None, keep_old: bool = False):
+        """Encloses a step: the state slots it wrote replace the sequences' when it went through, and go back when not."""
+        try:
+            yield
+        except BaseException:
+            if outs is not None:
+                self.states.abort(outs)
+            raise
+        if outs is not None:
+            self.states.commit(seqs, outs, keep_old)
+
+    def _catch_up(self, handles: list[_Handle]) -> None:
+        """Run the tokens the recurrent states have yet to see as a step of their own (a long run of rejected drafts)."""
+        for i in range(0, len(handles), 16):
+            batch, _, done = self._ragged([(h, h.seq.tokens[h.seq.state_len:h.seq.kv_len]) for h in handles[i:i + 16]], replay=True)
+            with done:
+                self.engine.layers(batch)
 
     # ---- decode graph bank ------------------------------------------------------------------------------
     def _step_batch(self, key: tuple[int, int, int]):
@@ -396,7 +500,7 @@ class EngineBackend:
         S, T, mq = key
         b = self.bufs
         return Batch(b.tokens[1][:T], b.positions[1][:T], b.slots[1][:T], b.page_table[1].view(b.max_seqs, self.max_pages)[:S],
-                     b.seq_lens[1][:S], b.q_start[1][:S + 1], mq, False, None)
+                     b.seq_lens[1][:S], b.q_start[1][:S + 1], mq, False, None, **(b.states(S) if self.states is not None else {}))
 
     def _capture(self, key: tuple[int, int, int], batch) -> None:
         """The step's inputs are already in the static buffers.  Kernels run during the warm-up write the same K/V the
@@ -478,6 +582,9 @@ class EngineBackend:
             for i in range(S):
                 starts.append(starts[-1] + per + (1 if i < extra else 0))
             b.q_start[0][:S + 1] = torch.tensor(starts, dtype=torch.int32)
+            if self.states is not None:
+                from .state import SCRATCH_SLOT, ZERO_SLOT
+                b.set_states([ZERO_SLOT] * S, [SCRATCH_SLOT] * S)
             b.upload()
             self._stage_embeddings(b.tokens[0][:T])
             self._capture((S, T, mq), self._step_batch((S, T, mq)))
@@ -494,35 +601,47 @@ class EngineBackend:
         return keys
 
     def _verify_device(self, handles: list[_Handle], rows: list[list[int]]) -> torch.Tensor:
-        from ..models.gqa_moe import Batch
+        # Recurrent layers after a partly rejected draft: the accepted tokens the state has not seen lead the rows again
+        # (same positions, same K/V); their logits are dropped.
+        new = rows
+        behind = [h for h in handles if self.states is not None and h.seq.lag > 7]
+        if behind:
+            self._catch_up(behind)
+        rows = [h.seq.tokens[h.seq.state_len:h.seq.kv_len] + r if self.states is not None else r for h, r in zip(handles, rows)]
         S = len(handles)
         T = sum(len(r) for r in rows)
         b = self.bufs
         pt = b.page_table[0].view(b.max_seqs, self.max_pages)
-        o = 0
+        o, keep = 0, []
         for i, (h, r) in enumerate(zip(handles, rows)):
             seq = h.seq
-            self.table.reserve(seq, seq.kv_len + len(r), copy_page=self._copy_page)
             n = len(r)
+            start = seq.kv_len + len(new[i]) - n
+            self.table.reserve(seq, start + n, copy_page=self._copy_page)
             b.tokens[0][o:o + n] = torch.tensor(r, dtype=torch.int32)
-            b.positions[0][o:o + n] = torch.arange(seq.kv_len, seq.kv_len + n, dtype=torch.int32)
-            b.slots[0][o:o + n] = torch.tensor(self.table.slots(seq, seq.kv_len, n), dtype=torch.int32)
+            b.positions[0][o:o + n] = torch.arange(start, start + n, dtype=torch.int32)
+            b.slots[0][o:o + n] = torch.tensor(self.table.slots(seq, start, n), dtype=torch.int32)
             pt[i].zero_()
             pt[i, :len(seq.pages)] = torch.tensor(seq.pages, dtype=torch.int32)
-            b.seq_lens[0][i] = seq.kv_len + n
+            b.seq_lens[0][i] = start + n
             b.q_start[0][i] = o
+            keep += range(o + n - len(new[i]), o + n)
             o += n
         b.q_start[0][S] = T
+        seqs = [h.seq for h in handles]
+        outs = self._states_for(b, seqs)
         b.upload()
         self._stage_embeddings(b.tokens[0][:T])
         key = (S, T, max(len(r) for r in rows))
         batch = self._step_batch(key)
-        logits = self._run_step(key, batch)
-        for h, r in zip(handles, rows):
-            h.seq.tokens.extend(r)
-            h.seq.kv_len += len(r)
+        with self._state_step(seqs, outs, keep_old=any(len(r) > 1 for r in new)):
+            logits = self._run_step(key, batch)
+            for h, r in zip(handles, new):
+                h.seq.tokens.extend(r)
+                h.seq.kv_len += len(r)
         self._last_batch = batch
-        return logits[:T]
+        logits = logits[:T]
+        return logits if len(keep) == T else logits.index_select(0, torch.tensor(keep).to(logits.device))
 
     def verify(self, handles: list[_Handle], rows: list[list[int]]) -> torch.Tensor:
         from ..ops import kernels as K
@@ -572,9 +691,18 @@ class EngineBackend:
     def commit(self, h: _Handle, keep_tokens: int) -> None:
         if keep_tokens < h.seq.kv_len:
             self.table.truncate(h.seq, keep_tokens)
+        if self.states is not None:
+            self.states.settle(h.seq, keep_tokens)
 
     def capture(self, h: _Handle, kind: str) -> None:
-        self.prefix.capture(h.seq, PROMPT if kind == "prompt" else TURN)
+        mark = None
+        if self.states is not None:
+            if h.seq.lag:
+                return                            # the state has yet to see the last tokens: nothing to resume from here
+            mark = h.seq.state
+            self.states.retain(mark)
+        if self.prefix.capture(h.seq, PROMPT if kind == "prompt" else TURN, mark=mark) is None and mark is not None:
+            self.states.release(mark)
 
     def release(self, h: _Handle) -> None:
         if not h.dead:
@@ -606,6 +734,8 @@ class EngineBackend:
                 for part in (got[:-1], last):
                     if part.numel():
                         d.update(part.contiguous().view(torch.uint8).cpu().numpy().tobytes())
+        if self.states is not None:
+            d.update(kv.state[seq.state].cpu().numpy().tobytes())
         return d.hexdigest()
 
     def pages_of(self, h: _Handle) -> int:

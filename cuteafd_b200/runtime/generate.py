@@ -25,7 +25,7 @@ class StepBuffers:
 
     def __init__(self, max_tokens: int, max_seqs: int, max_pages: int, device: torch.device):
         self.max_tokens, self.max_seqs, self.max_pages = max_tokens, max_seqs, max_pages
-        n = 3 * max_tokens + max_seqs * max_pages + max_seqs + (max_seqs + 1) + max_seqs
+        n = 3 * max_tokens + max_seqs * max_pages + max_seqs + (max_seqs + 1) + max_seqs + 2 * max_seqs
         self.host = torch.zeros(n, dtype=torch.int32).pin_memory() if device.type == "cuda" else torch.zeros(n, dtype=torch.int32)
         self.dev = torch.zeros(n, dtype=torch.int32, device=device)
         self._inflight = [torch.zeros(n, dtype=torch.int32).pin_memory() for _ in range(2)] if device.type == "cuda" else []
@@ -43,7 +43,16 @@ class StepBuffers:
         self.tokens, self.positions, self.slots = take(max_tokens), take(max_tokens), take(max_tokens)
         self.page_table = take(max_seqs * max_pages)
         self.seq_lens, self.q_start, self.last_rows = take(max_seqs), take(max_seqs + 1), take(max_seqs)
+        self.state_in, self.state_out = take(max_seqs), take(max_seqs)
         self.bytes = n * 4
+
+    def set_states(self, ins: list[int], outs: list[int]) -> None:
+        self.state_in[0][:len(ins)] = torch.tensor(ins, dtype=torch.int32)
+        self.state_out[0][:len(outs)] = torch.tensor(outs, dtype=torch.int32)
+
+    def states(self, S: int) -> dict:
+        """Batch fields of the staged state slots."""
+        return dict(state_in=self.state_in[1][:S], state_out=self.state_out[1][:S])
 
     def upload(self) -> int:
         if not self._inflight:
@@ -60,12 +69,22 @@ class StepBuffers:
         return self.bytes
 
 
+def make_states(engine):
+    """The slot pool of an engine whose cache holds recurrent state (one per engine), None for the others."""
+    slots = getattr(getattr(engine, "kv", None), "state_slots", 0)
+    if not slots:
+        return None
+    from .state import StatePool
+    return StatePool(slots)
+
+
 class Generator:
     def __init__(self, engine, pool: PagePool, max_pages_per_seq: int, max_seqs: int, prefill_chunk: int = 8192,
                  use_graphs: bool = True, max_graphs: int = 16):
         self.engine, self.pool = engine, pool
         self.max_graphs = max_graphs          # decode graphs kept (exact batch size is the key); least recently used goes first
-        self.table = SequenceTable(pool)
+        self.states = make_states(engine)     # slots of recurrent state, None for models without recurrent layers
+        self.table = SequenceTable(pool, self.states)
         self.device = engine.device
         self.max_pages, self.max_seqs, self.chunk = max_pages_per_seq, max_seqs, prefill_chunk
         self.use_graphs = use_graphs and self.device.type == "cuda"
@@ -93,12 +112,19 @@ class Generator:
             b.seq_lens[0][0] = start + n
             b.q_start[0][0], b.q_start[0][1] = 0, n
             b.last_rows[0][0] = n - 1
+            outs, extra = None, {}
+            if self.states is not None:
+                ins, outs = self.states.begin([seq])
+                b.set_states(ins, outs)
+                extra = b.states(1)
             self.h2d_bytes += b.upload()
             batch = Batch(b.tokens[1][:n], b.positions[1][:n], b.slots[1][:n], b.page_table[1].view(1, self.max_pages),
-                          b.seq_lens[1][:1], b.q_start[1][:2], n, True, b.last_rows[1][:1], fresh=start == 0)
+                          b.seq_lens[1][:1], b.q_start[1][:2], n, True, b.last_rows[1][:1], fresh=start == 0, **extra)
             logits = self.engine.forward(batch)
             seq.tokens.extend(part)
             seq.kv_len = start + n
+            if outs is not None:
+                self.states.commit([seq], outs)
             if c0 + self.chunk >= len(tokens):
                 nxt = int(self.engine.greedy(logits)[0].item())
                 self.d2h_bytes += 4
@@ -107,7 +133,7 @@ class Generator:
     # ---- decode -------------------------------------------------------------------------------------
     def _decode_batch(self, b: StepBuffers, S: int) -> Batch:
         return Batch(b.tokens[1][:S], b.positions[1][:S], b.slots[1][:S], b.page_table[1].view(self.max_seqs_of(b), self.max_pages)[:S],
-                     b.seq_lens[1][:S], b.q_start[1][:S + 1], 1, False, None)
+                     b.seq_lens[1][:S], b.q_start[1][:S + 1], 1, False, None, **(b.states(S) if self.states is not None else {}))
 
     @staticmethod
     def max_seqs_of(b: StepBuffers) -> int:
@@ -131,6 +157,10 @@ class Generator:
             b.seq_lens[0][i] = s.kv_len + 1
             b.q_start[0][i] = i
         b.q_start[0][S] = S
+        outs = None
+        if self.states is not None:
+            ins, outs = self.states.begin(seqs)
+            b.set_states(ins, outs)
         self.h2d_bytes += b.upload()
         if self.use_graphs:
             if S not in self.graphs:
@@ -162,4 +192,6 @@ class Generator:
         for s, tok, nt in zip(seqs, last_tokens, new):
             s.tokens.append(tok)
             s.kv_len += 1
+        if outs is not None:
+            self.states.commit(seqs, outs)
         return new

@@ -100,6 +100,14 @@ class Sequence:
     tokens: list[int] = field(default_factory=list)     # every token whose KV is (or will be) cached
     pages: list[int] = field(default_factory=list)
     kv_len: int = 0                                     # tokens whose KV is written
+    state: int = 0                                      # recurrent state slot (``runtime.state``; 0 = the zero state)
+    state_len: int = 0                                  # tokens the state has seen
+    old_state: tuple | None = None                      # (slot, tokens) before the last speculative step, until it is settled
+
+    @property
+    def lag(self) -> int:
+        """Tokens whose KV counts but which the recurrent state has yet to see (rejected drafts took it back)."""
+        return self.kv_len - self.state_len
 
     def pages_needed(self, new_len: int) -> int:
         return max(0, (new_len + PAGE - 1) // PAGE - len(self.pages))
@@ -108,8 +116,9 @@ class Sequence:
 class SequenceTable:
     """Owns sequences and their pages; produces slot mappings for KV writes."""
 
-    def __init__(self, pool: PagePool):
+    def __init__(self, pool: PagePool, states=None):
         self.pool = pool
+        self.states = states                            # runtime.state.StatePool of a model with recurrent layers
         self.seqs: dict[int, Sequence] = {}
         self._next = 0
 
@@ -137,7 +146,12 @@ class SequenceTable:
     def fork(self, src: Sequence, length: int | None = None) -> Sequence:
         """New sequence sharing the first ``length`` tokens of ``src`` by reference."""
         length = src.kv_len if length is None else length
+        if self.states is not None and length != src.state_len:
+            raise ValueError(f"a sequence with recurrent state at {src.state_len} tokens cannot fork at {length}")
         s = self.new()
+        if self.states is not None:
+            self.states.retain(src.state)
+            s.state, s.state_len = src.state, length
         n_pages = (length + PAGE - 1) // PAGE
         s.pages = list(src.pages[:n_pages])
         for p in s.pages:
@@ -155,6 +169,8 @@ class SequenceTable:
         del s.tokens[length:]
 
     def free(self, s: Sequence) -> None:
+        if self.states is not None:
+            self.states.close(s)
         for p in s.pages:
             self.pool.release(p)
         s.pages.clear()

@@ -99,6 +99,10 @@ class PrefixCache:
         self.stats = PrefixStats()
         self.spill = spill
         self.salt = salt
+        # A model with recurrent layers resumes only where a snapshot kept its state: lookups then match whole snapshots
+        # that carry a mark, nothing between.  ``on_release(snapshot)``: the snapshot's extras are given back.
+        self.whole_snapshots = False
+        self.on_release: Callable[[Snapshot], None] | None = None
         self._next = 1
         pool.on_exhausted = self.reclaim          # snapshots give pages back before an allocation fails
 
@@ -106,6 +110,8 @@ class PrefixCache:
     def lookup(self, tokens: list[int], media_key: bytes = b"") -> Match:
         self.stats.lookups += 1
         self.stats.lookup_tokens += len(tokens)
+        if self.whole_snapshots:
+            return self._lookup_snapshot(tokens, media_key)
         node, pages = self.root, []
         for h in chain_hashes(tokens, self.salt + media_key):
             nxt = node.children.get(h)
@@ -146,6 +152,28 @@ class PrefixCache:
             self.stats.hit_tokens += length
             self._touch(node if not whole else snap.node, snap)
         return Match(length, pages, tail_shared, snap, whole)
+
+    @staticmethod
+    def _pages_of(s: Snapshot) -> list[int]:
+        pages, n = [], s.node
+        while n is not None and n.parent is not None:
+            pages.append(n.page)
+            n = n.parent
+        pages.reverse()
+        return pages + ([s.tail_page] if s.tail_page is not None else [])
+
+    def _lookup_snapshot(self, tokens: list[int], media_key: bytes) -> Match:
+        best = None
+        for s in self.snapshots.values():
+            if (s.mark is not None and s.media_key == media_key and s.length < len(tokens) and (best is None or s.length > best.length)
+                    and s.tokens == tuple(tokens[:s.length])):
+                best = s
+        if best is None:
+            return Match(0, [], False, None)
+        self.stats.hits += 1
+        self.stats.hit_tokens += best.length
+        self._touch(None, best)
+        return Match(best.length, self._pages_of(best), best.tail_page is not None, best)
 
     def _ending_at(self, node: Node, tokens: list[int]):
         for s in self.snapshots.values():
@@ -226,6 +254,8 @@ class PrefixCache:
         s = self.snapshots.pop(sid, None)
         if s is None:
             return
+        if self.on_release is not None:
+            self.on_release(s)
         if spill and self.spill is not None:
             pages = []
             n = s.node

@@ -535,7 +535,13 @@ def build_state(args) -> ServerState:
             kvf = getattr(args, "kv_format", "auto")
             if cfg.is_mla and (kvf == "fp8_ds_mla" or (kvf == "auto" and cfg.indexer_heads)):
                 cfg = cfg.replace(kv_format="fp8_ds_mla")
-            if cfg.is_mla:
+            if cfg.is_hybrid:
+                from ..loader.load import hybrid_state_slots
+                from ..models.hybrid import HybridCache, HybridEngine as Engine, HybridWeights as Weights
+
+                def Cache(c, n, d):
+                    return HybridCache(c, n, d, hybrid_state_slots(rows))
+            elif cfg.is_mla:
                 from ..models.mla_moe import LatentCache as Cache, MlaMoeEngine as Engine, MlaMoeWeights as Weights
             else:
                 from ..models.gqa_moe import GqaMoeEngine as Engine, GqaMoeWeights as Weights, KvCache as Cache
@@ -549,6 +555,9 @@ def build_state(args) -> ServerState:
             if not cfg.tie_embeddings:
                 getattr(eng, "inner", eng).W.embed = None          # the device copy is not needed: free it
                 torch.cuda.empty_cache()
+        if cfg.is_hybrid and float(getattr(args, "host_cache_gib", 0.0)) > 0:
+            print("[serve] the pinned-host cache tier does not hold recurrent state: off for this model", flush=True)
+            args.host_cache_gib = 0.0
         be = EngineBackend(eng, num_pages, pages_per_seq, prefill_chunk=2048, max_decode_rows=args.concurrency,
                            use_graphs=getattr(args, "decode_graphs", "on") != "off",
                            host_cache_bytes=int(float(getattr(args, "host_cache_gib", 0.0)) * (1 << 30)), host_embedding=table)
