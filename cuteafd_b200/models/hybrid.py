@@ -315,7 +315,7 @@ class HybridEngine:
             y, G = p["y"].float(), self.cfg.norm_groups
             if "slots" in p:
                 w, idx, n, ident = p["slots"]
-                rows = torch.where((idx >= n)[..., None], ident.float()[:, None], y.view(T, w.shape[1], -1))
+                rows = torch.where((idx >= n)[..., None], ident.float()[:, None], y[:T * w.shape[1]].view(T, w.shape[1], -1))
                 y = (w[..., None] * rows).sum(1)
             g = y.view(T, G, -1)
             x = x + (g / torch.sqrt((g * g).mean(-1, keepdim=True) + self.cfg.rms_eps)).view(T, -1) * p["w_b"]
