@@ -96,6 +96,12 @@ def detect_operands(cat: Catalog) -> dict[str, QuantOperand]:
     return ops
 
 
+def plain_operands(cat: Catalog) -> dict[str, QuantOperand]:
+    """Every tensor as an operand of its own, for checkpoints that store unquantised tensors under bare names."""
+    return {n: QuantOperand(n, _plain(e), (e.shape[0], e.shape[1] if len(e.shape) > 1 else 1), n, bits=8.0 * e.nbytes / max(e.numel, 1))
+            for n, e in cat.entries.items()}
+
+
 def _plain(e: TensorEntry) -> str:
     return {"BF16": "bf16", "F16": "f16", "F32": "f32", "F8_E4M3": "e4m3", "F8_E5M2": "e5m2", "U8": "int8",
             "I8": "int8"}.get(e.dtype, e.dtype.lower())

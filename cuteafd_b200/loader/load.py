@@ -50,7 +50,7 @@ def open_snapshot(path: str, core_view: str | None = None) -> OpenedSnapshot:
     sel = select_view(path, core_view)
     cfg, hf = read_config(path, core_view)
     cat = Catalog(path, rename=families.canonical_name, weight_map=view_weight_map(path, core_view))
-    ops = formats.detect_operands(cat)
+    ops = formats.plain_operands(cat) if cfg.is_hybrid else formats.detect_operands(cat)
     fam = families.detect(hf)
     model = fam.open(cfg, hf) if fam else None
     return OpenedSnapshot(path, cfg, hf, cat, ops, fam, model, sel)
@@ -65,6 +65,11 @@ def load_params(path: str, dtype: torch.dtype = torch.float32, device: str = "cp
     snap = open_snapshot(path)
     out: dict[str, torch.Tensor] = {}
     covered = set()
+    if snap.cfg.is_hybrid:                  # plain tensors under the checkpoint's own names
+        for name in snap.catalog.names():
+            if not (only and only not in name) and not (exclude and exclude in name) and (keep is None or keep(name)):
+                out[name] = snap.catalog.read(name).to(device=device, dtype=dtype)
+        return snap.cfg, out
     for pre, op in snap.operands.items():
         if (exclude and exclude in pre) or (keep is not None and not keep(pre)):
             covered.update(n for n in (op.weight, op.scale_tensor, op.global_scale, op.input_scale, *op.companions.values()) if n)

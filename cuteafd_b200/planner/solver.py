@@ -117,6 +117,8 @@ def weight_bytes(params: int, fmt: str) -> int:
 
 
 def kv_bytes_per_token_per_layer(cfg: ModelConfig, kv_format: str) -> int:
+    if cfg.is_hybrid:
+        return 2 * cfg.kv_record_elems           # averaged over the layers: recurrent ones cache nothing per token
     if cfg.is_mla:
         if kv_format in ("auto", "fp8_ds_mla") and cfg.weight_format != "bf16":
             return cfg.kv_lora_rank + 4 * (cfg.kv_lora_rank // 128) + 2 * cfg.qk_rope_dim      # 656 B for 512 + 64
@@ -177,7 +179,7 @@ def _place(req: PlacementRequest, att: int, exp: int, pp: int) -> Placement:
     kv_tok_layer = kv_bytes_per_token_per_layer(cfg, req.kv_format)
     layers_per_stage = math.ceil(cfg.num_layers / pp)
     # MLA latent KV is replicated across attention TP ranks; GQA KV heads are split when they divide.
-    kv_shard = 1 if cfg.is_mla else min(att, cfg.num_kv_heads)
+    kv_shard = 1 if cfg.is_mla or cfg.is_hybrid else min(att, cfg.num_kv_heads)
     kv_per_token_dev = kv_tok_layer * layers_per_stage // kv_shard
     act_rows = max(req.prefill_rows, req.decode_rows)
     ranges = _expert_ranges(cfg.num_experts, exp if exp else att * pp) if cfg.num_experts else []
@@ -210,6 +212,10 @@ def _place(req: PlacementRequest, att: int, exp: int, pp: int) -> Placement:
             qkv = (cfg.num_heads * cfg.qk_head_dim * 3 if cfg.is_mla else (cfg.num_heads + 2 * cfg.num_kv_heads) * cfg.head_dim) * 2
             g.add("workspace", "activations", act_rows * (4 * width + 2 * qkv // att + cfg.dense_ffn * 2 // att))
             g.add("workspace", "logits", req.decode_rows * cfg.vocab_size * 4)
+            if cfg.is_hybrid:
+                # per sequence in flight its slot, the one before an unsettled step and the one being written, and as many
+                # again for cached prefixes
+                g.add("recurrent state", "slots", (2 + 6 * req.concurrency) * cfg.state_bytes)
             if cfg.num_experts:
                 g.add("exchange", "combine+routes", act_rows * cfg.top_k * (cfg.hidden * 2 + 12))
                 if colocated:
@@ -267,6 +273,8 @@ def _place(req: PlacementRequest, att: int, exp: int, pp: int) -> Placement:
 def kernel_geometry(cfg: ModelConfig) -> str:
     """Why the CUDA engines cannot run this geometry ("" = they can): their attention kernels are written for one head
     shape per family."""
+    if cfg.is_hybrid:
+        return "the hybrid engine takes a width that is a multiple of 8" if cfg.hidden % 8 else ""
     if cfg.is_mla:
         if (cfg.kv_lora_rank, cfg.qk_rope_dim, cfg.qk_nope_dim, cfg.v_head_dim) != (512, 64, 128, 128):
             return "the MLA kernels take the DeepSeek shape (latent 512, rope 64, nope 128, value 128)"
@@ -287,6 +295,10 @@ def engine_for(cfg: ModelConfig, att: int, exp: int, pp: int) -> tuple[str, str]
     why = kernel_geometry(cfg)
     if why:
         return "", why + "; the CPU oracle serves this checkpoint (serve --fake-engine)"
+    if cfg.is_hybrid:
+        if (att, exp, pp) == (1, 0, 1):
+            return "single", "per-layer hybrid stack on one GPU (models/hybrid.py)"
+        return "", "per-layer hybrids are not split over GPUs"
     if pp > 1:
         if att == 1 and exp == 0 and not cfg.is_mla:
             return "pp", "layer ranges as pipeline stages with ring hops (models/pp_gqa.py)"
@@ -313,6 +325,8 @@ HTTP_ENGINES = ("single", "afd", "tp")
 def candidates(req: PlacementRequest) -> list[tuple[int, int, int]]:
     cfg = req.cfg
     out = []
+    if cfg.is_hybrid and not req.attention_ranks and not req.expert_ranks and req.pipeline_stages == 1:
+        return [(1, 0, 1)]
     att_opts = [req.attention_ranks] if req.attention_ranks else [a for a in (1, 2, 4, 8) if a <= req.gpus and cfg.num_heads % a == 0]
     for a in att_opts:
         pp = req.pipeline_stages

@@ -1,0 +1,70 @@
+"""Small per-layer hybrid configurations and helpers shared by the hybrid tests."""
+import torch
+
+from cuteafd_b200.config import DeltaSpec, LatentSpec, LayerSpec, RouterSpec, hybrid_config
+from cuteafd_b200.ref import hybrid as R
+
+
+def latent(heads=3, dim=24, rot_dim=8, vdim=20, kv_rank=40, window=37, scale=None, base=5000.0):
+    return LatentSpec(heads, dim, rot_dim, vdim, kv_rank, window, scale if scale is not None else 1.7 * (dim + rot_dim) ** -0.5, base)
+
+
+def delta(heads=6, kv_heads=2, dim=20, vdim=36, conv=3):
+    return DeltaSpec(heads, kv_heads, dim, vdim, conv)
+
+
+def odd_config():
+    """Nothing is a power of two, every layer differs: layers without a feed-forward, routers with and without identity
+    outputs and groups, a value size above one block's columns."""
+    return hybrid_config("odd", 203, 96, [
+        LayerSpec(latent(), RouterSpec(6, 28, 3, 2, 4, 2)),
+        LayerSpec(delta()),
+        LayerSpec(delta(2, 2, 40, 136, 5), RouterSpec(5, 24, 2)),
+        LayerSpec(latent(5, 16, 12, 24, 64, 130, base=300.0), RouterSpec(7, 16, 4, 5, 3, 1)),
+        LayerSpec(latent(1, 8, 4, 8, 12, 1))], canon_taps=3, norm_groups=3, eps=2e-5)
+
+
+def plain_config():
+    """Values that make a mechanism vanish: one norm group, one-tap convolutions, one head, one group of experts."""
+    return hybrid_config("plain", 130, 64, [
+        LayerSpec(delta(1, 1, 16, 16, 1), RouterSpec(4, 8, 1, 1, 5, 5)),
+        LayerSpec(latent(1, 16, 2, 16, 24, 500), RouterSpec(2, 40, 2)),
+        LayerSpec(delta(4, 1, 64, 24, 4))], canon_taps=1, norm_groups=1, eps=1e-3)
+
+
+def wide_config(window=100):
+    """The sizes the tensor-core kernels take."""
+    return hybrid_config("wide", 500, 256, [
+        LayerSpec(latent(8, 128, 64, 128, 512, window, base=1e5), RouterSpec(8, 128, 2, 2, 5, 3)),
+        LayerSpec(delta(4, 2, 128, 128, 4), RouterSpec(6, 64, 3, 3, 3, 2)),
+        LayerSpec(latent(16, 128, 64, 128, 512, 2 * window + 3, base=1e4))], canon_taps=4, norm_groups=4, eps=1e-5)
+
+
+def params(cfg, seed=0, spread=0.4):
+    """Random bf16-representable weights.  The selection correction is spread out by ``spread``: above 1 the choice is the
+    correction's alone, so that 16-bit rounding cannot flip a close one."""
+    p = R.init_hybrid_weights(cfg, seed)
+    g = torch.Generator().manual_seed(seed + 99)
+    for k in p:
+        if k.endswith(".correction"):
+            p[k] = (torch.randperm(p[k].numel(), generator=g).float() - p[k].numel() / 2) * spread
+        elif k.endswith(".A_log"):
+            p[k] = p[k] - 1.0
+    return R.bf16_params(p)
+
+
+def tokens(n, vocab, seed=0):
+    return torch.randint(0, vocab, (n,), generator=torch.Generator().manual_seed(seed)).tolist()
+
+
+def oracle_logits(cfg, p, toks, dtype=torch.float32):
+    m = R.HybridRefDecoder(cfg, {k: v.to(dtype) for k, v in p.items()}, mark_rows=0)
+    with torch.no_grad():
+        return m.forward(torch.tensor(toks), m.new_state()).float()
+
+
+def err(got, want):
+    """Per row: rms of the difference over the rms of the wanted logits, means taken off."""
+    d = got.float() - want.float()
+    d, w = d - d.mean(-1, keepdim=True), want - want.mean(-1, keepdim=True)
+    return d.pow(2).mean(-1).sqrt() / w.pow(2).mean().sqrt()
