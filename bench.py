@@ -52,8 +52,9 @@ def main() -> None:
     ap.add_argument("--levels", default="1,8,32")
     ap.add_argument("--layers", type=int, default=0, help="debug only: fewer layers (marks the run invalid)")
     ap.add_argument("--no-graphs", action="store_true")
-    ap.add_argument("--config", default="qwen3", choices=["qwen3", "dsv3"],
-                    help="qwen3 = the headline Qwen3-30B-A3B bf16 card (with 8 GPUs the DeepSeek-V3 card follows it); dsv3 = only "
+    ap.add_argument("--config", default="qwen3", choices=["qwen3", "dsv3", "karusun"],
+                    help="karusun = the per-layer hybrid (latent attention + delta-rule layers) at the sizes of a real model's layers, and the "
+                         "MLA engine at equal size beside it (one GPU); qwen3 = the headline Qwen3-30B-A3B bf16 card (with 8 GPUs the DeepSeek-V3 card follows it); dsv3 = only "
                          "the DeepSeek-V3 shape: MLA attention replicas, E4M3 block-scaled experts on the other GPUs (needs 8 GPUs)")
     ap.add_argument("--attention-ranks", type=int, default=0,
                     help="data-parallel attention replicas of the disaggregated layout (0 = 1 on two GPUs, 2 on four or more)")
@@ -98,11 +99,18 @@ def main() -> None:
         """Build the deployment of one model configuration, run the card on it, tear it down.  Returns (cfg, card result
         or None on ranks that do not drive a card, parallelism string, clocks summary)."""
         cfg = qwen3_30b_a3b()
+        if name in ("karusun", "karusun-mla"):
+            from cuteafd_b200.config import karusun_bench, karusun_bench_mla
+            assert world == 1, "per-layer hybrids run on one GPU"
+            cfg = karusun_bench() if name == "karusun" else karusun_bench_mla()
         if name == "dsv3":
             from cuteafd_b200 import deepseek_v3
             cfg = deepseek_v3().replace(mtp_layers=0)
             assert world > 2, "the DeepSeek-V3 shape needs expert ranks"
-        if args.layers:
+        if args.layers and cfg.is_hybrid:
+            from cuteafd_b200.config import scaled_down
+            cfg = scaled_down(cfg, args.layers, cfg.vocab_size)
+        elif args.layers:
             cfg = cfg.replace(num_layers=args.layers)
         handle, gen, sync, replica, replicas = None, None, None, 0, 1
         mode = "afd" if args.parallelism == "auto" else args.parallelism
@@ -136,12 +144,19 @@ def main() -> None:
             if handle.worker is not None:
                 handle.worker.serve()            # returns when attention rank 0 sends STOP
         else:
-            from cuteafd_b200.models.gqa_moe import GqaMoeEngine, GqaMoeWeights, KvCache
+            from cuteafd_b200.models.gqa_moe import GqaMoeEngine as Engine, GqaMoeWeights as Weights, KvCache as Cache
             from cuteafd_b200.runtime.generate import Generator
             from cuteafd_b200.runtime.native import make_pool
-            W = GqaMoeWeights.random_init(cfg, dev, seed=0)
-            kv = KvCache(cfg, num_pages, dev)
-            eng = GqaMoeEngine(cfg, W, kv, max_tokens=args.prompt_len, max_seqs=max(levels))
+            if cfg.is_hybrid:
+                from cuteafd_b200.models.hybrid import HybridCache, HybridEngine as Engine, HybridWeights as Weights
+
+                def Cache(c, n, d):
+                    return HybridCache(c, n, d, state_slots=2 + 4 * max(levels))
+            elif cfg.is_mla:
+                from cuteafd_b200.models.mla_moe import LatentCache as Cache, MlaMoeEngine as Engine, MlaMoeWeights as Weights
+            W = Weights.random_init(cfg, dev, seed=0)
+            kv = Cache(cfg, num_pages, dev)
+            eng = Engine(cfg, W, kv, max_tokens=args.prompt_len, max_seqs=max(levels))
             gen = Generator(eng, make_pool(num_pages), pages_per_seq, max(levels), prefill_chunk=args.prompt_len,
                             use_graphs=not args.no_graphs)
             torch.cuda.synchronize()
@@ -188,7 +203,7 @@ def main() -> None:
             "value": round(r.tok_s, 2), "unit": "tok/s", "n_gpus": args.gpus, "steps": args.steps, "warmup": warmup,
             "ms_per_step": round(r.ms_per_step, 4), "higher_is_better": True, "scaling": "strong",
             "vs_baseline": round(r.tok_s / PUBLISHED["c8"], 3) if headline == 8 and args.config == "qwen3" else None,
-            "dtype": "bf16" if args.config == "qwen3" else "fp8 experts and, at decode, fp8 q_b / o / shared-expert projections (E4M3, 128x128 weight / 1x128 activation scales); MLA attention math, q_a / kv_a and prompt chunks in bf16", "data": "synthetic (uniform random token ids, N(0,0.02) random-init weights)",
+            "dtype": "bf16" if args.config != "dsv3" else "fp8 experts and, at decode, fp8 q_b / o / shared-expert projections (E4M3, 128x128 weight / 1x128 activation scales); MLA attention math, q_a / kv_a and prompt chunks in bf16", "data": "synthetic (uniform random token ids, N(0,0.02) random-init weights)",
             "config": {"model": cfg.name + ("" if valid else f"-{cfg.num_layers}layers-INVALID"),
                        "global_batch": headline, "seq_len": args.prompt_len, "parallelism": parallelism,
                        "l2": "inputs larger than L2 (each step streams GBs of weights and KV)",
@@ -216,6 +231,11 @@ def main() -> None:
         except Exception as e:                   # the headline line is still printed
             if rank == 0 and out is not None:
                 out["extra"]["dsv3_error"] = f"{type(e).__name__}: {e}"
+    if args.config == "karusun" and out is not None:
+        mcfg, mres, _, mclk = run_config("karusun-mla")
+        out["extra"].update(card_extra(mres, "mla_equal_size_"))
+        out["extra"]["mla_equal_size_config"] = {"model": mcfg.name, "clocks": mclk, "parameters": mcfg.total_params(),
+                                                 "hybrid_parameters": cfg.total_params()}
     if world > 1:
         dist.barrier()
         dist.destroy_process_group()

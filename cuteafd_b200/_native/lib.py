@@ -203,6 +203,8 @@ def cuda_lib():
         _sig(lib, "cafd_sample_rows", [P, I, I, P, P, I, P, P, P])
         _sig(lib, "cafd_accept_prefix", [P, P, P, I, P, P, P])
         _sig(lib, "cafd_norm_conv", [C.POINTER(NormArgs), I, P])
+        _sig(lib, "cafd_delta_chunked", [C.POINTER(DeltaArgs), P, C.c_longlong, P])
+        _sig(lib, "cafd_delta_chunk_bytes", [I, I, I], C.c_longlong)
         _sig(lib, "cafd_swap_ids", [P, P, I, P])
         _sig(lib, "cafd_gemm_f32", [P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, P])
         _sig(lib, "cafd_latent_prep", [C.POINTER(LatentPrep), I, P])

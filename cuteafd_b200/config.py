@@ -363,6 +363,14 @@ def karusun_bench() -> ModelConfig:
     return hybrid_config("karusun-bench", 65536, 2048, specs, canon_taps=4, norm_groups=4, eps=1e-5)
 
 
+def karusun_bench_mla() -> ModelConfig:
+    """The MLA decoder at the size of ``karusun_bench``: same width, depth, heads, latent, experts and vocabulary."""
+    return ModelConfig(name="karusun-bench-mla", family="deepseek_v3", vocab_size=65536, num_layers=24, hidden=2048, attention="mla",
+                       num_heads=32, q_lora_rank=0, kv_lora_rank=512, qk_nope_dim=128, qk_rope_dim=64, v_head_dim=128, rope_theta=1.0e6,
+                       rope_interleaved=False, rms_eps=1e-5, dense_ffn=0, first_dense_layers=0, num_experts=56, expert_ffn=1024, top_k=6,
+                       scoring="softmax", num_groups=8, topk_groups=4, num_shared_experts=0, norm_topk_prob=False, router_bias=True)
+
+
 PRESETS = {
     "karusun-bench": karusun_bench,
     "tiny-moe": tiny_moe,

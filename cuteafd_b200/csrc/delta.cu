@@ -9,39 +9,12 @@
 // (graph capture, rejected drafts) and a sequence may start from a slot that a cached prefix owns.
 #include "cafd_api.h"
 #include "common.cuh"
+#include "delta.cuh"
 
 namespace cafd {
 
-template <typename E> __device__ __forceinline__ float de_f(E v);
-template <> __device__ __forceinline__ float de_f<float>(float v) { return v; }
-template <> __device__ __forceinline__ float de_f<__nv_bfloat16>(__nv_bfloat16 v) { return __bfloat162float(v); }
-template <typename E> __device__ __forceinline__ E de_e(float v);
-template <> __device__ __forceinline__ float de_e<float>(float v) { return v; }
-template <> __device__ __forceinline__ __nv_bfloat16 de_e<__nv_bfloat16>(float v) { return __float2bfloat16(v); }
-
-struct DeltaArgs {
-  const void* proj;           // [T, ld] E: q | k | v | gate | b | a sections at the offsets below
-  const float* conv_w;        // [channels, taps] (q heads, k heads, v heads)
-  const float* A_log;         // [heads]
-  const float* dt_bias;       // [heads]
-  const float* norm_w;        // [vdim]
-  float* state;               // pool, slot_stride floats per slot
-  const int* state_in;        // [S]
-  const int* state_out;       // [S]
-  const int* q_start;         // [S + 1]
-  void* out;                  // [T, heads * out_vd] E: normed and gated rows (head h at h * out_vd)
-  float* raw;                 // [T, heads * vdim] fp32: o before the norm, when a head's columns span several blocks
-  long long slot_stride, s_off, c_off;   // the layer's state and convolution inputs inside a slot
-  int ld, q_off, k_off, v_off, g_off, b_off, a_off;
-  int T, S, heads, kv_heads, dim, vdim, taps, out_vd;
-  float eps;
-};
-
 constexpr int kDeltaRows = 32;      // state rows per thread
 constexpr int kDeltaCols = 128;     // state columns per block at most
-
-__device__ __forceinline__ float softplus(float a) { return fmaxf(a, 0.f) + log1pf(expf(-fabsf(a))); }
-__device__ __forceinline__ float sigmoid_f(float x) { return 1.0f / (1.0f + expf(-x)); }
 
 template <typename E, int MAXT, int NT>
 __global__ void __launch_bounds__(NT) delta_step_kernel(const DeltaArgs p) {
@@ -177,29 +150,6 @@ __global__ void __launch_bounds__(NT) delta_step_kernel(const DeltaArgs p) {
         const int i = j - (MAXT - 1 - halo);
         if (i >= 0) st_out[p.c_off + static_cast<size_t>(i) * channels + chan] = win[j];
       }
-    }
-  }
-}
-
-// out[t, h] = raw[t, h] / rms(raw[t, h]) * norm_w * silu(gate): one warp per (token, head)
-template <typename E>
-__global__ void __launch_bounds__(256) delta_out_kernel(const DeltaArgs p) {
-  pdl_wait();
-  pdl_trigger();
-  const long long n = static_cast<long long>(p.T) * p.heads;
-  const int lane = threadIdx.x & 31;
-  for (long long i = static_cast<long long>(blockIdx.x) * 8 + (threadIdx.x >> 5); i < n; i += static_cast<long long>(gridDim.x) * 8) {
-    const long long t = i / p.heads;
-    const int h = static_cast<int>(i - t * p.heads);
-    const float* o = p.raw + i * p.vdim;
-    const E* gate = static_cast<const E*>(p.proj) + t * p.ld + p.g_off + h * p.vdim;
-    float ss = 0.f;
-    for (int v = lane; v < p.vdim; v += 32) ss = fmaf(o[v], o[v], ss);
-    const float inv = 1.0f / sqrtf(warp_sum(ss) / static_cast<float>(p.vdim) + p.eps);
-    E* dst = static_cast<E*>(p.out) + i * p.out_vd;
-    for (int v = lane; v < p.vdim; v += 32) {
-      const float g = de_f<E>(gate[v]);
-      dst[v] = de_e<E>(o[v] * inv * p.norm_w[v] * g * sigmoid_f(g));
     }
   }
 }

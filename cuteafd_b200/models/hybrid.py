@@ -240,6 +240,8 @@ class HybridEngine:
     """Single-GPU engine of the per-layer hybrids behind the same calls as the other engines (``forward`` on a ``Batch``)."""
     embed_rows = None
     EXPANDED_PREFILL_TOKENS = 64     # fresh prompt chunks of at least this many tokens use the expanded-form attention
+    CHUNKED_DELTA_TOKENS = 32        # steps with a portion of at least this many tokens take the chunked delta rule
+    CHUNK_SCRATCH_BYTES = 128 << 20  # its operands of one slab of chunks (about an L2's worth)
     FUSED_ROUTE_TOKENS = 64          # steps up to this many tokens run router scores + selection as one launch
 
     def __init__(self, cfg: ModelConfig, weights: HybridWeights, kv: HybridCache, max_tokens: int, max_seqs: int = 64):
@@ -266,7 +268,7 @@ class HybridEngine:
         self._lat: dict[LatentSpec, _LatentWs] = {}
         self._delta: dict[DeltaSpec, torch.Tensor] = {}
         self._moe: dict = {}
-        raw = 0
+        raw = scratch = 0
         for spec in cfg.layer_specs:
             m, r = spec.mixer, spec.router
             if isinstance(m, LatentSpec):
@@ -275,11 +277,17 @@ class HybridEngine:
             else:
                 if m not in self._delta:
                     self._delta[m] = torch.zeros(max_tokens, m.heads, pad8(m.vdim), dtype=dt, device=dev)
-                if m.vdim > 128:
+                chunked = K.delta_chunk_ok(m, dt)
+                if m.vdim > 128 or chunked:
                     raw = max(raw, m.heads * m.vdim)
+                if chunked:
+                    per = K.delta_chunk_bytes(m)
+                    chunks = max(max(1, self.CHUNK_SCRATCH_BYTES // per), 1)
+                    scratch = max(scratch, per * min(chunks, max_tokens // 64 + max_seqs))
             if r is not None and r not in self._moe:
                 self._moe[r] = LocalExchange(ExchangeGeometry(H, pad8(r.ffn), r.experts, r.top, max_tokens, 1), dev, dtype=dt)
-        ws.raw = torch.empty(max_tokens, raw, dtype=torch.float32, device=dev) if raw else None
+        ws.raw = torch.empty(max_tokens * raw, dtype=torch.float32, device=dev) if raw else None
+        ws.chunk = torch.empty(scratch, dtype=torch.uint8, device=dev) if scratch else None
         self.moe = None
         rows = max_seqs
         self._logits = torch.empty(rows, pad8(cfg.vocab_size), dtype=torch.float32, device=dev)
@@ -401,10 +409,16 @@ class HybridEngine:
         L, ws = self.W.layers[i], self.ws
         a = self._project(i, h, T)
         off, out = self.kv.offsets[i], self._delta[m][:T]
-        K.delta_step(a, L.offs, m, L, self.kv.state, off["S"], off["conv"], b.state_in, b.state_out, b.q_start, out,
-                     ws.raw if m.vdim > 128 else None, self.cfg.rms_eps)
+        args = (a, L.offs, m, L, self.kv.state, off["S"], off["conv"], b.state_in, b.state_out, b.q_start, out, ws.raw, self.cfg.rms_eps)
+        if b.prefill and b.max_q_len >= self.CHUNKED_DELTA_TOKENS and K.delta_chunk_ok(m, self.dtype):
+            K.delta_chunked(ws.chunk, *args)
+            slabs = -(-(T // 64 + b.q_start.shape[0] - 1) * K.delta_chunk_bytes(m) // ws.chunk.numel())
+            self.launches += 2 * slabs + 1
+        else:
+            K.delta_step(*args)
+            self.launches += 1 if m.vdim <= 128 else 2
         K.linear(out.view(T, -1), L.w_o, out=ws.y[:T])
-        self.launches += 2
+        self.launches += 1
 
     # ---- routed feed-forward ----------------------------------------------------------------------------------------
     def _experts(self, i: int, r, h: torch.Tensor, T: int) -> tuple:

@@ -761,6 +761,22 @@ def delta_step(proj: torch.Tensor, *args, **kw) -> None:
     _n.check(_n.cuda_lib().cafd_delta_step(C.byref(p), int(proj.dtype == torch.float32), _stream()), "delta_step")
 
 
+def delta_chunk_ok(m, dtype: torch.dtype) -> bool:
+    """Whether the chunked form takes a delta-rule layer of this shape."""
+    return dtype == torch.bfloat16 and m.dim in (64, 128) and m.vdim % 32 == 0 and m.conv <= 4
+
+
+def delta_chunk_bytes(m) -> int:
+    """Scratch bytes per 64-token chunk."""
+    return int(_n.cuda_lib().cafd_delta_chunk_bytes(m.heads, m.dim, m.vdim))
+
+
+def delta_chunked(scratch: torch.Tensor, proj: torch.Tensor, *args, **kw) -> None:
+    """``delta_step`` for prompt portions, 64 tokens at a time on the tensor cores; ``scratch`` [bytes] uint8."""
+    p = delta_args(proj, *args, **kw)
+    _n.check(_n.cuda_lib().cafd_delta_chunked(C.byref(p), scratch.data_ptr(), scratch.numel(), _stream()), "delta_chunked")
+
+
 # ---- sampling ---------------------------------------------------------------------------------------------
 _SAMPLE_ROW = None
 

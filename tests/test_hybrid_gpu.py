@@ -275,6 +275,56 @@ def test_delta_rule(dtype, m):
         ins, outs = outs, [5, 6, 7] if step == 0 else [2, 8, 9]
 
 
+@pytest.mark.parametrize("slab", [1, 3, 64])
+@pytest.mark.parametrize("m", [delta(4, 2, 128, 128, 4), delta(3, 3, 64, 32, 2), delta(2, 1, 64, 96, 4), delta(2, 2, 128, 32, 1)], ids=str)
+def test_delta_rule_in_chunks(m, slab):
+    """The chunked form over ragged portions (whole chunks, parts of one, single tokens), three steps in a row, in slabs of
+    one, three and all chunks: rows and states against the token-by-token equations.  Decays from almost none to almost
+    everything, and keys that repeat."""
+    from cuteafd_b200.ops import kernels as K
+    eps, w = 1e-5, _delta_layer(m)
+    w.A_log = w.A_log + torch.linspace(-4, 5, m.heads)
+    kd, vd = m.kv_heads * m.dim, m.heads * m.vdim
+    widths = dict(q=kd, k=kd, v=vd, g=vd, b=m.heads, a=m.heads)
+    offs, o = {}, 0
+    for n, c in widths.items():
+        offs[n] = o
+        o += -(-c // 8) * 8
+    s_sz, c_sz = m.heads * m.dim * m.vdim, (m.conv - 1) * m.conv_channels
+    state = torch.full((12, s_sz + c_sz + 32), 3.0, device=dev())
+    state[0] = 0
+    st = [dict(S=torch.zeros(m.heads, m.dim, m.vdim), q=torch.zeros(m.conv - 1, kd), k=torch.zeros(m.conv - 1, kd), v=torch.zeros(m.conv - 1, vd))
+          for _ in range(3)]
+
+    class D:
+        pass
+    wd = D()
+    for n in ("conv_w", "A_log", "dt_bias", "out_norm"):
+        setattr(wd, n, getattr(w, n).to(dev()))
+    scratch = torch.empty(slab * K.delta_chunk_bytes(m), dtype=torch.uint8, device=dev())
+    ins, outs = [0, 0, 0], [2, 3, 4]
+    for step, lens in enumerate([[130, 1, 64], [2, 65, 63], [1, 200, 3]]):
+        T, qs = sum(lens), [0]
+        for n in lens:
+            qs.append(qs[-1] + n)
+        a = rnd(T, o, seed=20 + step, dtype=torch.bfloat16)
+        if step == 1:
+            a[10:50, offs["k"]:offs["k"] + kd] = a[10, offs["k"]:offs["k"] + kd]
+        out = torch.zeros(T, m.heads, m.vdim, dtype=torch.bfloat16, device=dev())
+        raw = torch.empty(T * vd, device=dev())
+        K.delta_chunked(scratch, a.to(dev(), torch.bfloat16), offs, m, wd, state, 0, s_sz, i32(ins), i32(outs), i32(qs), out, raw, eps)
+        for s in range(3):
+            x = {n: a[qs[s]:qs[s + 1], offs[n]:offs[n] + c] for n, c in widths.items()}
+            want = _delta_oracle(m, w, x, st[s], eps)
+            close(out[qs[s]:qs[s + 1]], want, torch.bfloat16)
+            got = state[outs[s], :s_sz].view(m.heads, m.dim, m.vdim).cpu()
+            for hh in range(m.heads):
+                close(got[hh], st[s]["S"][hh], torch.float32, 10)
+            if m.conv > 1:
+                close(state[outs[s], s_sz:s_sz + c_sz].view(m.conv - 1, -1), torch.cat([st[s][n] for n in "qkv"], 1), torch.float32)
+        ins, outs = outs, [5, 6, 7] if step == 0 else [2, 8, 9]
+
+
 @pytest.mark.parametrize("r", [RouterSpec(6, 1, 3, 2, 4, 2), RouterSpec(5, 1, 2), RouterSpec(40, 1, 6, 8, 6, 2), RouterSpec(100, 1, 8, 20, 8, 8)], ids=str)
 def test_routes(r):
     from cuteafd_b200.ops import kernels as K
