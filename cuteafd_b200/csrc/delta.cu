@@ -17,7 +17,7 @@ constexpr int kDeltaRows = 32;      // state rows per thread
 constexpr int kDeltaCols = 128;     // state columns per block at most
 
 template <typename E, int MAXT, int NT>
-__global__ void __launch_bounds__(NT) delta_step_kernel(const DeltaArgs p) {
+__global__ void __launch_bounds__(NT, MAXT <= 4 && NT <= 512 ? 2 : 1) delta_step_kernel(const DeltaArgs p) {
   extern __shared__ float sm[];
   const int h = blockIdx.x, seq = blockIdx.y, v0 = blockIdx.z * kDeltaCols;
   const int tid = threadIdx.x, lane = tid & 31;

@@ -33,14 +33,60 @@ struct DeltaArgs {
 __device__ __forceinline__ float softplus(float a) { return fmaxf(a, 0.f) + log1pf(expf(-fabsf(a))); }
 __device__ __forceinline__ float sigmoid_f(float x) { return 1.0f / (1.0f + expf(-x)); }
 
-// out[t, h] = raw[t, h] / rms(raw[t, h]) * norm_w * silu(gate): one warp per (token, head)
+__device__ __forceinline__ void de_load4(const float* p, float (&v)[4]) {
+  const float4 q = *reinterpret_cast<const float4*>(p);
+  v[0] = q.x; v[1] = q.y; v[2] = q.z; v[3] = q.w;
+}
+__device__ __forceinline__ void de_load4(const __nv_bfloat16* p, float (&v)[4]) {
+  const uint2 q = *reinterpret_cast<const uint2*>(p);
+  v[0] = bf16_lo(q.x); v[1] = bf16_hi(q.x); v[2] = bf16_lo(q.y); v[3] = bf16_hi(q.y);
+}
+__device__ __forceinline__ void de_store4(float* p, const float (&v)[4]) { *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]); }
+__device__ __forceinline__ void de_store4(__nv_bfloat16* p, const float (&v)[4]) {
+  *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16(v[0], v[1]), pack_bf16(v[2], v[3]));
+}
+
+// out[t, h] = raw[t, h] / rms(raw[t, h]) * norm_w * silu(gate): one warp per (token, head), two in flight where a head
+// is at most 128 columns of whole 16-byte pieces
 template <typename E>
 __global__ void __launch_bounds__(256) delta_out_kernel(const DeltaArgs p) {
   pdl_wait();
   pdl_trigger();
-  const long long n = static_cast<long long>(p.T) * p.heads;
+  const long long n = static_cast<long long>(p.T) * p.heads, stride = static_cast<long long>(gridDim.x) * 8;
   const int lane = threadIdx.x & 31;
-  for (long long i = static_cast<long long>(blockIdx.x) * 8 + (threadIdx.x >> 5); i < n; i += static_cast<long long>(gridDim.x) * 8) {
+  long long i = static_cast<long long>(blockIdx.x) * 8 + (threadIdx.x >> 5);
+  if (p.vdim <= 128 && p.vdim % 4 == 0 && p.out_vd % 4 == 0 && p.ld % 4 == 0 && p.g_off % 4 == 0) {
+    const bool on = 4 * lane < p.vdim;
+    float nw[4] = {};
+    if (on) de_load4(p.norm_w + 4 * lane, nw);
+    for (; i < n; i += 2 * stride) {
+      float o[2][4] = {}, g[2][4] = {};
+#pragma unroll
+      for (int j = 0; j < 2; ++j) {
+        const long long r = i + j * stride;
+        if (r < n && on) {
+          const long long t = r / p.heads;
+          const int h = static_cast<int>(r - t * p.heads);
+          de_load4(p.raw + r * p.vdim + 4 * lane, o[j]);
+          de_load4(static_cast<const E*>(p.proj) + t * p.ld + p.g_off + h * p.vdim + 4 * lane, g[j]);
+        }
+      }
+#pragma unroll
+      for (int j = 0; j < 2; ++j) {
+        const long long r = i + j * stride;
+        const float ss = warp_sum(o[j][0] * o[j][0] + o[j][1] * o[j][1] + o[j][2] * o[j][2] + o[j][3] * o[j][3]);
+        const float inv = 1.0f / sqrtf(ss / static_cast<float>(p.vdim) + p.eps);
+        if (r < n && on) {
+          float v[4];
+#pragma unroll
+          for (int e = 0; e < 4; ++e) v[e] = o[j][e] * inv * nw[e] * g[j][e] * sigmoid_f(g[j][e]);
+          de_store4(static_cast<E*>(p.out) + r * p.out_vd + 4 * lane, v);
+        }
+      }
+    }
+    return;
+  }
+  for (; i < n; i += stride) {
     const long long t = i / p.heads;
     const int h = static_cast<int>(i - t * p.heads);
     const float* o = p.raw + i * p.vdim;

@@ -17,6 +17,8 @@
 // two bf16 halves (16 significant bits together) and multiplied as hi hi + hi lo + lo hi with fp32 accumulation; the
 // triangular inverse, decays and norms are fp32.  delta_prepare leaves its results in the order of the mma fragments, so
 // delta_scan loads operands straight into registers, 16 bytes per lane.
+#include <type_traits>
+
 #include "cafd_api.h"
 #include "common.cuh"
 #include "delta.cuh"
@@ -82,7 +84,7 @@ __global__ void __launch_bounds__(kChunkThreads, 2) delta_prepare_kernel(const D
   __nv_bfloat16* yl = yh + kChunk * kP;
   float* Lm = reinterpret_cast<float*>(yl + kChunk * kP); // [64][kTPitch]
   float* Tm = Lm + kChunk * kTPitch;
-  __shared__ float sG[kChunk], sB[kChunk], sIq[kChunk], sIk[kChunk];
+  __shared__ float sG[kChunk], sB[kChunk], sIq[kChunk], sIk[kChunk], sW[kChunk], sE[kChunk];
 
   pdl_wait();
   pdl_trigger();
@@ -97,12 +99,19 @@ __global__ void __launch_bounds__(kChunkThreads, 2) delta_prepare_kernel(const D
   const int rep = p.heads / p.kv_heads, kvh = h / rep;
   const int kd = p.kv_heads * p.dim, channels = 2 * kd + p.heads * p.vdim;
 
-  // convolution + silu of `cols` channels from channel `chan0` (column src0 of the projection) into hi / lo tiles
-  auto conv = [&](__nv_bfloat16* dh, __nv_bfloat16* dl, int src0, int chan0, int cols) {
-    const int pairs = cols >> 1, groups = kChunkThreads / pairs, per = kChunk / groups;
-    const int pr = tid % pairs, grp = tid / pairs;
-    if (grp >= groups) return;
-    const int c = chan0 + 2 * pr;
+  // convolution + silu of kCols channels from channel `chan0` (column src0 of the projection) into hi / lo tiles: a thread
+  // takes two channels of kPer consecutive tokens, all their loads in flight at once
+  auto conv = [&](auto cols_c, __nv_bfloat16* dh, __nv_bfloat16* dl, int src0, int chan0) {
+    constexpr int kCols = decltype(cols_c)::value, kPairs = kCols / 2, kGroups = kChunkThreads / kPairs, kPer = kChunk / kGroups;
+    const int pr = tid % kPairs, grp = tid / kPairs;
+    const int c = chan0 + 2 * pr, i0 = off + grp * kPer;
+    const __nv_bfloat16* src = proj + static_cast<size_t>(t0) * p.ld + src0 + 2 * pr;
+    uint32_t raw[kPer + 3];
+#pragma unroll
+    for (int j = 0; j < kPer + 3; ++j) {
+      const int i = min(max(i0 - 3 + j, 0), len - 1);
+      raw[j] = *reinterpret_cast<const uint32_t*>(src + static_cast<size_t>(i) * p.ld);
+    }
     float w0[4], w1[4];
 #pragma unroll
     for (int j = 0; j < 4; ++j) {
@@ -110,38 +119,31 @@ __global__ void __launch_bounds__(kChunkThreads, 2) delta_prepare_kernel(const D
       w0[j] = tap >= 0 ? p.conv_w[static_cast<size_t>(c) * p.taps + tap] : 0.f;
       w1[j] = tap >= 0 ? p.conv_w[static_cast<size_t>(c + 1) * p.taps + tap] : 0.f;
     }
-    auto fetch = [&](int i, float& a, float& bb) {          // input of token i of the portion (negative: before it)
-      a = bb = 0.f;
-      if (i >= 0) {
-        if (i < len) {
-          const uint32_t v = *reinterpret_cast<const uint32_t*>(proj + static_cast<size_t>(t0 + i) * p.ld + src0 + 2 * pr);
-          a = bf16_lo(v); bb = bf16_hi(v);
-        }
-      } else if (i + p.taps - 1 >= 0) {
-        const float* s = st_in + static_cast<size_t>(i + p.taps - 1) * channels + c;
-        a = s[0]; bb = s[1];
-      }
-    };
     float x0[4], x1[4];
-    const int i0 = off + grp * per;
 #pragma unroll
-    for (int j = 0; j < 3; ++j) fetch(i0 - 3 + j, x0[j + 1], x1[j + 1]);
-#pragma unroll 8
-    for (int r = 0; r < per; ++r) {
-      float a, bb;
-      fetch(i0 + r, a, bb);
+    for (int j = 0; j < 3; ++j) {
+      const int i = i0 - 3 + j;
+      x0[j + 1] = bf16_lo(raw[j]); x1[j + 1] = bf16_hi(raw[j]);
+      if (i < 0) {                                          // before the portion: the state's inputs
+        const bool have = i + p.taps - 1 >= 0;
+        const float* s = st_in + static_cast<size_t>(have ? i + p.taps - 1 : 0) * channels + c;
+        x0[j + 1] = have ? s[0] : 0.f; x1[j + 1] = have ? s[1] : 0.f;
+      }
+    }
+#pragma unroll
+    for (int r = 0; r < kPer; ++r) {
 #pragma unroll
       for (int j = 0; j < 3; ++j) { x0[j] = x0[j + 1]; x1[j] = x1[j + 1]; }
-      x0[3] = a; x1[3] = bb;
+      x0[3] = bf16_lo(raw[r + 3]); x1[3] = bf16_hi(raw[r + 3]);
       float y0 = 0.f, y1 = 0.f;
 #pragma unroll
       for (int j = 0; j < 4; ++j) { y0 = fmaf(w0[j], x0[j], y0); y1 = fmaf(w1[j], x1[j], y1); }
       const bool live = i0 + r < len;
-      y0 = live ? silu(y0) : 0.f;
-      y1 = live ? silu(y1) : 0.f;
+      y0 = live ? y0 / (1.0f + __expf(-y0)) : 0.f;
+      y1 = live ? y1 / (1.0f + __expf(-y1)) : 0.f;
       uint32_t hi, lo;
       split2(y0, y1, hi, lo);
-      const int at = (grp * per + r) * kP + 2 * pr;
+      const int at = (grp * kPer + r) * kP + 2 * pr;
       *reinterpret_cast<uint32_t*>(dh + at) = hi;
       *reinterpret_cast<uint32_t*>(dl + at) = lo;
     }
@@ -171,8 +173,8 @@ __global__ void __launch_bounds__(kChunkThreads, 2) delta_prepare_kernel(const D
     sG[2 * lane] = run - lg[1];
     sG[2 * lane + 1] = run;
   }
-  conv(kh, kl, p.k_off + kvh * D, kd + kvh * D, D);
-  conv(yh, yl, p.q_off + kvh * D, kvh * D, D);
+  conv(std::integral_constant<int, D>{}, kh, kl, p.k_off + kvh * D, kd + kvh * D);
+  conv(std::integral_constant<int, D>{}, yh, yl, p.q_off + kvh * D, kvh * D);
   __syncthreads();
   // inverse norms of q (with 1 / sqrt(dim)) and k
   for (int r = warp; r < 2 * kChunk; r += 8) {
@@ -188,7 +190,12 @@ __global__ void __launch_bounds__(kChunkThreads, 2) delta_prepare_kernel(const D
     s = warp_sum(s);
     if (lane == 0) {
       if (is_q) sIq[r & 63] = 1.0f / (sqrtf(s + 1e-6f) * sqrtf(static_cast<float>(D)));
-      else sIk[r] = 1.0f / sqrtf(s + 1e-6f);
+      else {
+        const float ik = 1.0f / sqrtf(s + 1e-6f), G = sG[r];
+        sIk[r] = ik;
+        sW[r] = sB[r] * ik * expf(G);                       // beta e^G / |k|
+        sE[r] = ik * expf(sG[kChunk - 1] - G);              // e^(G_63 - G) / |k|
+      }
     }
   }
   __syncthreads();
@@ -279,7 +286,7 @@ __global__ void __launch_bounds__(kChunkThreads, 2) delta_prepare_kernel(const D
 #pragma unroll
     for (int e = 0; e < 4; ++e) {
       const int t = ks * 16 + (e >> 1) * 8 + tc + (e & 1);
-      s[e] = sIk[t] * expf(G_end - sG[t]);
+      s[e] = sE[t];
     }
 #pragma unroll
     for (int e = 0; e < 4; ++e)
@@ -331,8 +338,7 @@ __global__ void __launch_bounds__(kChunkThreads, 2) delta_prepare_kernel(const D
     for (int e = 0; e < 4; ++e) {
       const int row = (e & 1) ? r_hi : r_lo, col = ks * 16 + (e >> 1) * 8 + tc;
       const float2 v = *reinterpret_cast<const float2*>(Tm + row * kTPitch + col);
-      float s0 = sB[col], s1 = sB[col + 1];
-      if (with_k) { s0 *= sIk[col] * expf(sG[col]); s1 *= sIk[col + 1] * expf(sG[col + 1]); }
+      const float s0 = with_k ? sW[col] : sB[col], s1 = with_k ? sW[col + 1] : sB[col + 1];
       split2(v.x * s0, v.y * s1, hi[e], lo[e]);
     }
   };
@@ -372,7 +378,9 @@ __global__ void __launch_bounds__(kChunkThreads, 2) delta_prepare_kernel(const D
   for (int v0 = 0; v0 < p.vdim; v0 += 64) {
     const int cols = min(64, p.vdim - v0);
     if (v0) __syncthreads();
-    conv(yh, yl, p.v_off + h * p.vdim + v0, 2 * kd + h * p.vdim + v0, cols);
+    const int v_src = p.v_off + h * p.vdim + v0, v_chan = 2 * kd + h * p.vdim + v0;
+    if (cols == 64) conv(std::integral_constant<int, 64>{}, yh, yl, v_src, v_chan);
+    else conv(std::integral_constant<int, 32>{}, yh, yl, v_src, v_chan);
     __syncthreads();
     if (nh * 32 < cols) {
       float c[4][4] = {};

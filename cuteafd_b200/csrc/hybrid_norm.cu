@@ -68,7 +68,23 @@ __device__ __forceinline__ void store_vec(E* p, const float (&v)[V]) {
   }
 }
 
+// V elements as they sit in memory: loads of rows to come stay packed in registers until their turn
+template <typename E, int V> struct Packed;
+template <> struct Packed<float, 4> { float4 q; };
+template <> struct Packed<__nv_bfloat16, 4> { uint2 q; };
+template <> struct Packed<float, 1> { float q; };
+template <> struct Packed<__nv_bfloat16, 1> { __nv_bfloat16 q; };
+template <typename E, int V>
+__device__ __forceinline__ Packed<E, V> load_packed(const E* p) { return *reinterpret_cast<const Packed<E, V>*>(p); }
+__device__ __forceinline__ void unpack(const Packed<float, 4>& a, float (&v)[4]) { v[0] = a.q.x; v[1] = a.q.y; v[2] = a.q.z; v[3] = a.q.w; }
+__device__ __forceinline__ void unpack(const Packed<__nv_bfloat16, 4>& a, float (&v)[4]) {
+  v[0] = bf16_lo(a.q.x); v[1] = bf16_hi(a.q.x); v[2] = bf16_lo(a.q.y); v[3] = bf16_hi(a.q.y);
+}
+__device__ __forceinline__ void unpack(const Packed<float, 1>& a, float (&v)[1]) { v[0] = a.q; }
+__device__ __forceinline__ void unpack(const Packed<__nv_bfloat16, 1>& a, float (&v)[1]) { v[0] = __bfloat162float(a.q); }
+
 constexpr int kNormThreads = 512;
+constexpr int kSlotBatch = 8;       // routed rows of a token whose loads are in flight together
 
 // 1 / sqrt(mean of squares + eps) of the group each of this thread's vectors lies in.  `part` holds one number per 32
 // vectors when groups are whole multiples of that (fast), else one per vector; `gsum` one per group (slow form only).
@@ -125,8 +141,8 @@ __device__ __forceinline__ void group_inv(const float (&v)[KV][V], float (&inv)[
   }
 }
 
-template <typename E, int V, int KV, int MAXT>
-__global__ void __launch_bounds__(kNormThreads) norm_conv_kernel(const NormArgs a) {
+template <typename E, int V, int KV, int MAXT, bool kSlots, int kMaxThreads, int kMinBlocks>
+__global__ void __launch_bounds__(kMaxThreads, kMinBlocks) norm_conv_kernel(const NormArgs a) {
   extern __shared__ float sm[];
   pdl_wait();
   pdl_trigger();
@@ -139,12 +155,6 @@ __global__ void __launch_bounds__(kNormThreads) norm_conv_kernel(const NormArgs 
   if (r0 >= a.T) return;
   const int halo = a.conv ? a.taps - 1 : 0;
 
-  float wn[KV][V];
-#pragma unroll
-  for (int k = 0; k < KV; ++k) {
-    const int i = tid + k * nt;
-    if (i < nvec) load_vec<float, V>(a.w + i * V, wn[k]);
-  }
   float win[MAXT > 1 ? MAXT - 1 : 1][KV][V];   // the last taps - 1 convolution inputs, oldest first, at the array's end
 #pragma unroll
   for (int j = 0; j < MAXT - 1; ++j)
@@ -181,6 +191,29 @@ __global__ void __launch_bounds__(kNormThreads) norm_conv_kernel(const NormArgs 
   };
   if (a.conv && t == s_lo && halo > 0) load_state();
   int flip = 0;
+  // The residual and the sublayer's output of the next token are loaded while this one is normalised.
+  Packed<float, V> nx[KV];
+  Packed<E, V> ny[KV];
+  auto fetch = [&](int tt) {
+    const int row = a.row_idx ? a.row_idx[tt] : tt;
+    if (!a.embed) {
+      const float* src = a.x_in + static_cast<size_t>(row) * a.H;
+#pragma unroll
+      for (int k = 0; k < KV; ++k) {
+        const int i = tid + k * nt;
+        if (i < nvec) nx[k] = load_packed<float, V>(src + i * V);
+      }
+    }
+    if (!kSlots && a.y) {
+      const E* src = static_cast<const E*>(a.y) + static_cast<size_t>(row) * a.ldy;
+#pragma unroll
+      for (int k = 0; k < KV; ++k) {
+        const int i = tid + k * nt;
+        if (i < nvec) ny[k] = load_packed<E, V>(src + i * V);
+      }
+    }
+  };
+  fetch(t);
   for (; t < r1; ++t) {
     if (a.conv && t == s_hi) {                  // next sequence (empty ones are skipped)
       do { ++seq; s_lo = s_hi; s_hi = a.q_start[seq + 1]; } while (s_hi == s_lo && seq + 1 < a.S);
@@ -188,7 +221,11 @@ __global__ void __launch_bounds__(kNormThreads) norm_conv_kernel(const NormArgs 
     }
     const int row = a.row_idx ? a.row_idx[t] : t;
     const bool own = t >= r0;
-    float x[KV][V];
+    float x[KV][V], y[KV][V];
+#pragma unroll
+    for (int k = 0; k < KV; ++k)
+#pragma unroll
+      for (int e = 0; e < V; ++e) { x[k][e] = 0.f; y[k][e] = 0.f; }
     if (a.embed) {
       int tok = a.tokens[row];
       tok = tok < 0 ? 0 : tok >= a.vocab ? a.vocab - 1 : tok;
@@ -197,48 +234,55 @@ __global__ void __launch_bounds__(kNormThreads) norm_conv_kernel(const NormArgs 
       for (int k = 0; k < KV; ++k) {
         const int i = tid + k * nt;
         if (i < nvec) load_vec<E, V>(src + i * V, x[k]);
-        else for (int e = 0; e < V; ++e) x[k][e] = 0.f;
       }
     } else {
-      const float* src = a.x_in + static_cast<size_t>(row) * a.H;
-#pragma unroll
-      for (int k = 0; k < KV; ++k) {
-        const int i = tid + k * nt;
-        if (i < nvec) load_vec<float, V>(src + i * V, x[k]);
-        else for (int e = 0; e < V; ++e) x[k][e] = 0.f;
-      }
-    }
-    if (a.y) {
-      float y[KV][V], inv[KV];
 #pragma unroll
       for (int k = 0; k < KV; ++k)
+        if (tid + k * nt < nvec) unpack(nx[k], x[k]);
+    }
+    if (!kSlots && a.y) {
 #pragma unroll
-        for (int e = 0; e < V; ++e) y[k][e] = 0.f;
-      if (a.slot_w) {
-        for (int s = 0; s < a.top_k; ++s) {
-          const float g = a.slot_w[static_cast<size_t>(row) * a.top_k + s];
-          const bool pass = a.slot_idx[static_cast<size_t>(row) * a.top_k + s] >= a.n_experts;
-          const E* src = pass ? static_cast<const E*>(a.ident) + static_cast<size_t>(row) * a.H
-                              : static_cast<const E*>(a.y) + (static_cast<size_t>(row) * a.top_k + s) * a.H;
+      for (int k = 0; k < KV; ++k)
+        if (tid + k * nt < nvec) unpack(ny[k], y[k]);
+    }
+    if constexpr (kSlots) {
+      const float* sw = a.slot_w + static_cast<size_t>(row) * a.top_k;
+      const int* si = a.slot_idx + static_cast<size_t>(row) * a.top_k;
+      for (int s0 = 0; s0 < a.top_k; s0 += kSlotBatch) {
+        int src[kSlotBatch];                    // row offsets; identity slots: the input row, marked by a negative number
+        float g[kSlotBatch];
 #pragma unroll
-          for (int k = 0; k < KV; ++k) {
-            const int i = tid + k * nt;
-            if (i < nvec) {
-              float v[V];
-              load_vec<E, V>(src + i * V, v);
-#pragma unroll
-              for (int e = 0; e < V; ++e) y[k][e] += g * v[e];
-            }
-          }
+        for (int j = 0; j < kSlotBatch; ++j) {
+          const int s = min(s0 + j, a.top_k - 1);
+          g[j] = s0 + j < a.top_k ? sw[s] : 0.f;
+          src[j] = si[s] >= a.n_experts ? -1 : row * a.top_k + s;
         }
-      } else {
-        const E* src = static_cast<const E*>(a.y) + static_cast<size_t>(row) * a.ldy;
 #pragma unroll
         for (int k = 0; k < KV; ++k) {
           const int i = tid + k * nt;
-          if (i < nvec) load_vec<E, V>(src + i * V, y[k]);
+          if (i < nvec) {
+            Packed<E, V> raw[kSlotBatch];
+#pragma unroll
+            for (int j = 0; j < kSlotBatch; ++j)
+              if (s0 + j < a.top_k)
+                raw[j] = load_packed<E, V>((src[j] < 0 ? static_cast<const E*>(a.ident) + static_cast<size_t>(row) * a.H
+                                                       : static_cast<const E*>(a.y) + static_cast<size_t>(src[j]) * a.H) + i * V);
+#pragma unroll
+            for (int j = 0; j < kSlotBatch; ++j) {
+              if (s0 + j < a.top_k) {
+                float v[V];
+                unpack(raw[j], v);
+#pragma unroll
+                for (int e = 0; e < V; ++e) y[k][e] += g[j] * v[e];
+              }
+            }
+          }
         }
       }
+    }
+    if (t + 1 < r1) fetch(t + 1);
+    if (a.y) {
+      float inv[KV];
       group_inv<V, KV>(y, inv, sm + flip * stride, sm + flip * stride + nvec, nvec, gvec, fast, a.eps);
       flip ^= 1;
 #pragma unroll
@@ -263,9 +307,15 @@ __global__ void __launch_bounds__(kNormThreads) norm_conv_kernel(const NormArgs 
     group_inv<V, KV>(x, inv, sm + flip * stride, sm + flip * stride + nvec, nvec, gvec, fast, a.eps);
     flip ^= 1;
 #pragma unroll
-    for (int k = 0; k < KV; ++k)
+    for (int k = 0; k < KV; ++k) {                                           // x now holds h
+      const int i = tid + k * nt;
+      if (i < nvec) {
+        float wn[V];
+        load_vec<float, V>(a.w + i * V, wn);
 #pragma unroll
-      for (int e = 0; e < V; ++e) x[k][e] = x[k][e] * inv[k] * wn[k][e];     // x now holds h
+        for (int e = 0; e < V; ++e) x[k][e] = x[k][e] * inv[k] * wn[e];
+      }
+    }
     if (own) {
 #pragma unroll
       for (int k = 0; k < KV; ++k) {
@@ -325,15 +375,20 @@ __global__ void __launch_bounds__(kNormThreads) norm_conv_kernel(const NormArgs 
   }
 }
 
-template <typename E, int V, int KV>
+template <typename E, int V, int KV, int kMaxThreads = kNormThreads, int kMinBlocks = 1>
 static int launch_norm(const NormArgs& a, int threads, cudaStream_t st) {
   const int nvec = a.H / V, gvec = nvec / a.groups;
   const int stride = (gvec % 32 == 0) ? nvec / 32 : nvec + a.groups;
   const size_t smem = static_cast<size_t>(2 * stride) * 4;
   if (smem > 48 * 1024) return -12;
   const dim3 grid((a.T + a.run - 1) / a.run);
-  if (!a.conv || a.taps <= 4) launch_pdl(norm_conv_kernel<E, V, KV, 4>, grid, dim3(threads), smem, st, a);
-  else launch_pdl(norm_conv_kernel<E, V, KV, 16>, grid, dim3(threads), smem, st, a);
+  if (!a.conv || a.taps <= 4) {
+    if (a.slot_w) launch_pdl(norm_conv_kernel<E, V, KV, 4, true, kMaxThreads, kMinBlocks>, grid, dim3(threads), smem, st, a);
+    else launch_pdl(norm_conv_kernel<E, V, KV, 4, false, kMaxThreads, kMinBlocks>, grid, dim3(threads), smem, st, a);
+  } else {
+    if (a.slot_w) launch_pdl(norm_conv_kernel<E, V, KV, 16, true, kMaxThreads, 1>, grid, dim3(threads), smem, st, a);
+    else launch_pdl(norm_conv_kernel<E, V, KV, 16, false, kMaxThreads, 1>, grid, dim3(threads), smem, st, a);
+  }
   return static_cast<int>(cudaGetLastError());
 }
 
@@ -342,6 +397,8 @@ static int dispatch_norm(NormArgs a, cudaStream_t st) {
   if ((a.H / a.groups) % 4 == 0) {
     const int nvec = a.H / 4;
     auto threads = [&](int kv) { return ((nvec + kv - 1) / kv + 31) / 32 * 32; };
+    // prompts: small blocks (several per SM, each at its own token) hide the loads and barriers better than wide ones
+    if (a.T >= 512 && nvec >= 256 && nvec <= kNormThreads) return launch_norm<E, 4, 2, 256, 3>(a, threads(2), st);
     if (nvec <= kNormThreads) return launch_norm<E, 4, 1>(a, threads(1), st);
     if (nvec <= 2 * kNormThreads) return launch_norm<E, 4, 2>(a, threads(2), st);
     if (nvec <= 4 * kNormThreads) return launch_norm<E, 4, 4>(a, threads(4), st);
@@ -378,7 +435,7 @@ extern "C" int cafd_norm_conv(const NormArgs* args, int is_f32, cafd_stream_t s)
   if (a.x_out && a.x_out == a.x_in) return -11;
   if (a.run <= 0) {
     // decode: one token per block; prompts: runs long enough that the recomputed inputs stay a small share
-    int run = (a.T + 2 * 148 - 1) / (2 * 148);
+    int run = (a.T + 4 * 148 - 1) / (4 * 148);
     a.run = run <= 2 ? 1 : run > 32 ? 32 : run;
   }
   cudaStream_t st = static_cast<cudaStream_t>(s);

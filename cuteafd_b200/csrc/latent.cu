@@ -200,6 +200,24 @@ __global__ void __launch_bounds__(256) latent_gate_kernel(E* __restrict__ attn, 
   pdl_wait();
   pdl_trigger();
   const int n = heads * vdim;
+  if (sizeof(E) == 2 && ld_head == vdim && n % 8 == 0 && ldg % 8 == 0 && g_off % 8 == 0) {   // 16-byte pieces
+    const int nv = n / 8;
+    for (int t = blockIdx.x; t < T; t += gridDim.x) {
+      uint4* o = reinterpret_cast<uint4*>(attn + static_cast<size_t>(t) * n);
+      const uint4* gr = reinterpret_cast<const uint4*>(gate + static_cast<size_t>(t) * ldg + g_off);
+#pragma unroll 2
+      for (int i = threadIdx.x; i < nv; i += blockDim.x) {
+        const uint4 a = o[i], g = gr[i];
+        const uint32_t av[4] = {a.x, a.y, a.z, a.w}, gv[4] = {g.x, g.y, g.z, g.w};
+        uint32_t r[4];
+#pragma unroll
+        for (int e = 0; e < 4; ++e)
+          r[e] = pack_bf16(bf16_lo(av[e]) / (1.0f + expf(-bf16_lo(gv[e]))), bf16_hi(av[e]) / (1.0f + expf(-bf16_hi(gv[e]))));
+        o[i] = make_uint4(r[0], r[1], r[2], r[3]);
+      }
+    }
+    return;
+  }
   for (int t = blockIdx.x; t < T; t += gridDim.x)
     for (int i = threadIdx.x; i < n; i += blockDim.x) {
       const int h = i / vdim, d = i - h * vdim;

@@ -251,11 +251,12 @@ __global__ void __launch_bounds__(128) mla_absorb_small_kernel(const __nv_bfloat
 }
 
 // o_lat [heads, t_pad, 512] (head-major attention output) -> attn [T, heads * 128]: attn[t, h] = o_lat[h, t] @ W_uv[h]^T
-// (W_uv [heads, 128, 512]).  grid (heads, 2): CTA (h, s) computes output rows [64 s, 64 s + 64); each of its eight
+// (W_uv [heads, 128, 512]), times sigmoid(gate[t, h * 128 ..]) where a gate is given.  grid (heads, 2): CTA (h, s) computes output rows [64 s, 64 s + 64); each of its eight
 // warps takes eight weight rows, lanes along K (a warp load is 512 contiguous bytes), all sixteen loads in flight.
 __global__ void __launch_bounds__(256) mla_unabsorb_small_kernel(const __nv_bfloat16* __restrict__ o_lat, int t_pad,
                                                                  const __nv_bfloat16* __restrict__ w_uv,
-                                                                 __nv_bfloat16* __restrict__ attn, int T, int heads) {
+                                                                 __nv_bfloat16* __restrict__ attn, int T, int heads,
+                                                                 const __nv_bfloat16* __restrict__ gate, int ldg) {
   pdl_wait();
   pdl_trigger();
   __shared__ __align__(16) __nv_bfloat16 sx[kSmallT][kLatent];
@@ -289,6 +290,7 @@ __global__ void __launch_bounds__(256) mla_unabsorb_small_kernel(const __nv_bflo
       float v = acc[0];
 #pragma unroll
       for (int r = 1; r < 8; ++r) v = lane == r ? acc[r] : v;
+      if (gate) v /= 1.0f + expf(-__bfloat162float(gate[static_cast<size_t>(t) * ldg + h * 128 + row0 + lane]));
       attn[static_cast<size_t>(t) * heads * 128 + h * 128 + row0 + lane] = __float2bfloat16(v);
     }
   }
@@ -364,12 +366,12 @@ extern "C" int cafd_mla_absorb_small(const void* q, int ldq, const void* w_uk, c
              static_cast<__nv_bfloat16*>(q_abs), T, heads, interleaved);
   return static_cast<int>(cudaGetLastError());
 }
-extern "C" int cafd_mla_unabsorb_small(const void* o_lat, int t_pad, const void* w_uv, void* attn, int T, int heads,
+extern "C" int cafd_mla_unabsorb_small(const void* o_lat, int t_pad, const void* w_uv, void* attn, int T, int heads, const void* gate, int ldg,
                                        cafd_stream_t s) {
   if (T <= 0) return 0;
   if (T > cafd::kSmallT) return -10;
   launch_pdl(mla_unabsorb_small_kernel, dim3(heads, 2), dim3(256), 0, static_cast<cudaStream_t>(s),
              static_cast<const __nv_bfloat16*>(o_lat), t_pad, static_cast<const __nv_bfloat16*>(w_uv),
-             static_cast<__nv_bfloat16*>(attn), T, heads);
+             static_cast<__nv_bfloat16*>(attn), T, heads, static_cast<const __nv_bfloat16*>(gate), ldg);
   return static_cast<int>(cudaGetLastError());
 }

@@ -362,16 +362,27 @@ class HybridEngine:
             lw.k_exp, lw.v_exp = torch.zeros(rows, m.heads * 128, **kw), torch.zeros(rows, m.heads * 128, **kw)
         slab = lw.q_slab[:m.heads * ht.t_pad * dp].view(m.heads, ht.t_pad, dp)
         o_slab = lw.o_slab[:m.heads * ht.t_pad * rp].view(m.heads, ht.t_pad, rp)
+        qg = (a[:, L.offs["q"]:L.offs["q"] + m.heads * (m.dim + m.rot_dim)], a[:, L.offs["g"]:L.offs["g"] + m.heads * m.vdim])
+        # (the batch-invariant form keeps one absorb / un-absorb route for every decode width: the grouped GEMMs)
+        small = fast and T <= K.MLA_SMALL_ROWS and not self.fixed_kv_split
         K.latent_prep(a, L.offs["q"], L.offs["kv"], m.heads, m.dim, m.rot_dim, L.kv_norm, lw.inv_freq, b.positions, b.slots, cache,
-                      None if expanded else slab, lw.q_abs[:T], self.cfg.rms_eps, lat_out=lw.lat[:T] if expanded else None)
+                      None if expanded or small else slab, None if small else lw.q_abs[:T], self.cfg.rms_eps,
+                      lat_out=lw.lat[:T] if expanded else None)
         self.launches += 1
+        if small:
+            # decode-sized step: rotation and absorb in one launch, un-absorb and output gate in another
+            K.mla_absorb_small(qg[0], L.w_uk, lw.inv_freq, b.positions, lw.q_abs[:T], m.heads, False)
+            self._attend_tensor_core(m, lw, T, b, cache, o_slab, ht.t_pad)
+            K.mla_unabsorb_small(o_slab, L.w_uv, attn, T, gate=qg[1])
+            K.linear(attn.view(T, -1), L.w_o, out=ws.y[:T])
+            self.launches += 4
+            return
         if expanded:
             rows = -(-T // 64) * 64
             K.linear(lw.lat[:T], L.w_kb, out=lw.k_exp[:T])
             K.linear(lw.lat[:T], L.w_uv.view(m.heads * m.vdim, m.kv_rank), out=lw.v_exp[:T])
-            K.attn_prefill_mla(a[:, L.offs["q"]:L.offs["q"] + m.heads * (m.dim + m.rot_dim)], lw.q_abs[:T], lw.k_exp[:rows], lw.v_exp[:rows],
-                               self._zero1, cache, b.page_table, b.seq_lens, b.q_start, attn, b.max_q_len, m.heads, m.scale,
-                               window=m.window)
+            K.attn_prefill_mla(qg[0], lw.q_abs[:T], lw.k_exp[:rows], lw.v_exp[:rows], self._zero1, cache, b.page_table, b.seq_lens, b.q_start,
+                               attn, b.max_q_len, m.heads, m.scale, window=m.window)
             self.launches += 3
         else:
             K.grouped_linear(slab.view(-1, dp), L.w_uk, lw.q_abs, ht.tile_expert, ht.tile_row0, ht.num_tiles, ht.max_tiles, ht.tile_rows,

@@ -658,12 +658,13 @@ def mla_absorb_small(q: torch.Tensor, w_uk: torch.Tensor, inv_freq: torch.Tensor
              "mla_absorb_small")
 
 
-def mla_unabsorb_small(o_lat: torch.Tensor, w_uv: torch.Tensor, attn: torch.Tensor, T: int) -> None:
+def mla_unabsorb_small(o_lat: torch.Tensor, w_uv: torch.Tensor, attn: torch.Tensor, T: int, gate: torch.Tensor | None = None) -> None:
     """Decode-sized steps: o_lat [heads, t_pad, 512] (head-major attention output) -> attn [T, heads*128] through
-    W_uv[h] [128, 512]."""
+    W_uv[h] [128, 512]; ``gate`` [T, heads*128] (any row stride): times sigmoid(gate)."""
     heads, t_pad, _ = o_lat.shape
     assert T <= MLA_SMALL_ROWS and w_uv.shape == (heads, 128, 512) and w_uv.is_contiguous() and attn.is_contiguous()
-    _n.check(_n.cuda_lib().cafd_mla_unabsorb_small(o_lat.data_ptr(), t_pad, w_uv.data_ptr(), attn.data_ptr(), T, heads, _stream()),
+    _n.check(_n.cuda_lib().cafd_mla_unabsorb_small(o_lat.data_ptr(), t_pad, w_uv.data_ptr(), attn.data_ptr(), T, heads, _ptr(gate),
+                                                   gate.stride(0) if gate is not None else 0, _stream()),
              "mla_unabsorb_small")
 
 
@@ -704,17 +705,20 @@ def swap_ids(a: torch.Tensor, b: torch.Tensor) -> None:
 
 
 def latent_prep(a: torch.Tensor, q_off: int, kv_off: int, heads: int, dim: int, rot: int, norm_w: torch.Tensor, inv_freq: torch.Tensor,
-                positions: torch.Tensor, slots: torch.Tensor, cache: torch.Tensor, slab: torch.Tensor | None, q_abs: torch.Tensor,
+                positions: torch.Tensor, slots: torch.Tensor, cache: torch.Tensor, slab: torch.Tensor | None, q_abs: torch.Tensor | None,
                 eps: float, lat_out: torch.Tensor | None = None) -> None:
     """One launch per step and layer: latent norm, rotations, the cache record at ``slots`` and the query parts (unrotated
-    into ``slab`` [heads, t_pad, dim_pad], rotated into ``q_abs`` [T, heads, rec])."""
+    into ``slab`` [heads, t_pad, dim_pad], rotated into ``q_abs`` [T, heads, rec]); ``q_abs`` None: the record alone."""
     p = _n.LatentPrep()
     p.a, p.norm_w, p.inv_freq, p.positions, p.slots = a.data_ptr(), norm_w.data_ptr(), inv_freq.data_ptr(), positions.data_ptr(), slots.data_ptr()
-    p.cache, p.slab, p.q_abs, p.lat_out = cache.data_ptr(), _ptr(slab), q_abs.data_ptr(), _ptr(lat_out)
+    p.cache, p.slab, p.q_abs, p.lat_out = cache.data_ptr(), _ptr(slab), _ptr(q_abs), _ptr(lat_out)
+    if q_abs is None:
+        heads = 0
     p.lda, p.q_off, p.kv_off, p.heads, p.dim, p.rot, p.rank = a.stride(0), q_off, kv_off, heads, dim, rot, norm_w.shape[0]
     p.rec, p.T, p.eps = cache.shape[-1], a.shape[0], eps
     p.dim_pad, p.t_pad = (slab.shape[2], slab.shape[1]) if slab is not None else (0, 0)
-    assert cache.is_contiguous() and q_abs.is_contiguous() and q_abs.shape[-1] == p.rec and a.dtype == cache.dtype == q_abs.dtype
+    assert cache.is_contiguous() and a.dtype == cache.dtype
+    assert q_abs is None or (q_abs.is_contiguous() and q_abs.shape[-1] == p.rec and q_abs.dtype == a.dtype)
     _n.check(_n.cuda_lib().cafd_latent_prep(C.byref(p), int(a.dtype == torch.float32), _stream()), "latent_prep")
 
 
