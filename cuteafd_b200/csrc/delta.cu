@@ -17,7 +17,7 @@ constexpr int kDeltaRows = 32;      // state rows per thread
 constexpr int kDeltaCols = 128;     // state columns per block at most
 
 template <typename E, int MAXT, int NT>
-__global__ void __launch_bounds__(NT, MAXT <= 4 && NT <= 512 ? 2 : 1) delta_step_kernel(const DeltaArgs p) {
+__global__ void __launch_bounds__(NT) delta_step_kernel(const DeltaArgs p) {
   extern __shared__ float sm[];
   const int h = blockIdx.x, seq = blockIdx.y, v0 = blockIdx.z * kDeltaCols;
   const int tid = threadIdx.x, lane = tid & 31;
@@ -154,8 +154,158 @@ __global__ void __launch_bounds__(NT, MAXT <= 4 && NT <= 512 ? 2 : 1) delta_step
   }
 }
 
+// The same recurrence for heads of 128 columns and D = 64 or 128 rows, as decode steps want it: 256 threads, a warp holds
+// D / 8 state rows with four columns per lane (16-byte loads and stores), the output norm stays inside one warp.
+template <typename E, int D>
+__global__ void __launch_bounds__(256, 2) delta_step128_kernel(const DeltaArgs p) {
+  constexpr int kR = D / 8, kCh = 2 * D + 128, kTaps = 4;
+  __shared__ __align__(16) float ch[2][kCh];
+  __shared__ __align__(16) float red[2][8][128];
+  __shared__ float sgb[2][2];
+  const int h = blockIdx.x, seq = blockIdx.y, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  // the state of this step was written a whole step ago: its loads need not wait for the projection
+  const float* st_in = p.state + static_cast<size_t>(p.state_in[seq]) * p.slot_stride;
+  float* st_out = p.state + static_cast<size_t>(p.state_out[seq]) * p.slot_stride;
+  const size_t s_at = p.s_off + (static_cast<size_t>(h) * D + warp * kR) * 128 + 4 * lane;
+  float4 S[kR];
+#pragma unroll
+  for (int r = 0; r < kR; ++r) S[r] = __ldcg(reinterpret_cast<const float4*>(st_in + s_at + r * 128));
+  const int rep = p.heads / p.kv_heads, kh = h / rep;
+  const int kd = p.kv_heads * D, channels = 2 * kd + p.heads * 128, halo = p.taps - 1;
+  constexpr int kN = (kCh + 255) / 256;          // channels per thread
+  int chan[kN], src[kN];
+  float win[kN][kTaps - 1], cw[kN][kTaps], x[kN];
+#pragma unroll
+  for (int n = 0; n < kN; ++n) {
+    const int c = tid + n * 256;
+    chan[n] = -1; src[n] = 0;
+    if (c < D) { chan[n] = kh * D + c; src[n] = p.q_off + chan[n]; }
+    else if (c < 2 * D) { chan[n] = kd + kh * D + c - D; src[n] = p.k_off + kh * D + c - D; }
+    else if (c < kCh) { chan[n] = 2 * kd + h * 128 + c - 2 * D; src[n] = p.v_off + h * 128 + c - 2 * D; }
+#pragma unroll
+    for (int j = 0; j < kTaps; ++j) {
+      const int tap = j - (kTaps - p.taps);
+      cw[n][j] = (chan[n] >= 0 && tap >= 0) ? p.conv_w[static_cast<size_t>(chan[n]) * p.taps + tap] : 0.f;
+    }
+#pragma unroll
+    for (int j = 0; j < kTaps - 1; ++j) {
+      const int i = j - (kTaps - 1 - halo);
+      win[n][j] = (chan[n] >= 0 && i >= 0) ? st_in[p.c_off + static_cast<size_t>(i) * channels + chan[n]] : 0.f;
+    }
+  }
+  const float a_scale = tid == 0 ? -expf(p.A_log[h]) : 0.f, dt = tid == 0 ? p.dt_bias[h] : 0.f;
+  float nw[4] = {};
+  if (warp == 0) de_load4(p.norm_w + 4 * lane, nw);
+
+  pdl_wait();
+  pdl_trigger();
+  const int t0 = p.q_start[seq], t1 = p.q_start[seq + 1];
+  const E* proj = static_cast<const E*>(p.proj);
+#pragma unroll
+  for (int n = 0; n < kN; ++n) x[n] = (chan[n] >= 0 && t0 < t1) ? de_f<E>(proj[static_cast<size_t>(t0) * p.ld + src[n]]) : 0.f;
+  for (int t = t0; t < t1; ++t) {
+    const int buf = (t - t0) & 1;
+    const E* row = proj + static_cast<size_t>(t) * p.ld;
+    float* c = ch[buf];
+    float gate[4] = {};
+    if (warp == 0) {
+      if (p.g_off % 4 == 0 && p.ld % 4 == 0) de_load4(row + p.g_off + h * 128 + 4 * lane, gate);
+      else
+        for (int e = 0; e < 4; ++e) gate[e] = de_f<E>(row[p.g_off + h * 128 + 4 * lane + e]);
+    }
+    if (tid == 0) {
+      sgb[buf][0] = expf(a_scale * softplus(de_f<E>(row[p.a_off + h]) + dt));
+      sgb[buf][1] = sigmoid_f(de_f<E>(row[p.b_off + h]));
+    }
+#pragma unroll
+    for (int n = 0; n < kN; ++n) {
+      if (chan[n] >= 0) {
+        float y = cw[n][kTaps - 1] * x[n];
+#pragma unroll
+        for (int j = 0; j < kTaps - 1; ++j) y = fmaf(cw[n][j], win[n][j], y);
+        win[n][0] = win[n][1]; win[n][1] = win[n][2]; win[n][2] = x[n];
+        c[tid + n * 256] = y * sigmoid_f(y);
+      }
+    }
+    __syncthreads();
+#pragma unroll
+    for (int n = 0; n < kN; ++n)
+      if (chan[n] >= 0 && t + 1 < t1) x[n] = de_f<E>(row[p.ld + src[n]]);
+    float qq = 0.f, kk = 0.f, qk = 0.f;
+#pragma unroll
+    for (int i = 0; i < D / 32; ++i) {
+      const float a = c[lane + 32 * i], b = c[D + lane + 32 * i];
+      qq = fmaf(a, a, qq); kk = fmaf(b, b, kk); qk = fmaf(a, b, qk);
+    }
+    float4 sk = make_float4(0.f, 0.f, 0.f, 0.f), sq = sk;
+#pragma unroll
+    for (int r = 0; r < kR; ++r) {
+      const float qv = c[warp * kR + r], kv = c[D + warp * kR + r];
+      sq.x = fmaf(S[r].x, qv, sq.x); sq.y = fmaf(S[r].y, qv, sq.y); sq.z = fmaf(S[r].z, qv, sq.z); sq.w = fmaf(S[r].w, qv, sq.w);
+      sk.x = fmaf(S[r].x, kv, sk.x); sk.y = fmaf(S[r].y, kv, sk.y); sk.z = fmaf(S[r].z, kv, sk.z); sk.w = fmaf(S[r].w, kv, sk.w);
+    }
+    *reinterpret_cast<float4*>(&red[0][warp][4 * lane]) = sk;
+    *reinterpret_cast<float4*>(&red[1][warp][4 * lane]) = sq;
+    qq = warp_sum(qq); kk = warp_sum(kk); qk = warp_sum(qk);
+    const float ik = 1.0f / sqrtf(kk + 1e-6f), iq = 1.0f / (sqrtf(qq + 1e-6f) * sqrtf(static_cast<float>(D)));
+    __syncthreads();
+    sk = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+    for (int w = 0; w < 8; ++w) {
+      const float4 v = *reinterpret_cast<const float4*>(&red[0][w][4 * lane]);
+      sk.x += v.x; sk.y += v.y; sk.z += v.z; sk.w += v.w;
+    }
+    const float g = sgb[buf][0], beta = sgb[buf][1], gk = g * ik;
+    const float4 v = *reinterpret_cast<const float4*>(c + 2 * D + 4 * lane);
+    float u[4] = {beta * (v.x - gk * sk.x), beta * (v.y - gk * sk.y), beta * (v.z - gk * sk.z), beta * (v.w - gk * sk.w)};
+    if (warp == 0) {
+      sq = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+      for (int w = 0; w < 8; ++w) {
+        const float4 z = *reinterpret_cast<const float4*>(&red[1][w][4 * lane]);
+        sq.x += z.x; sq.y += z.y; sq.z += z.z; sq.w += z.w;
+      }
+      const float gq = g * iq, qki = qk * ik * iq;
+      float o[4] = {gq * sq.x + qki * u[0], gq * sq.y + qki * u[1], gq * sq.z + qki * u[2], gq * sq.w + qki * u[3]};
+      const float ss = warp_sum(o[0] * o[0] + o[1] * o[1] + o[2] * o[2] + o[3] * o[3]);
+      const float inv = 1.0f / sqrtf(ss * (1.0f / 128.0f) + p.eps);
+#pragma unroll
+      for (int e = 0; e < 4; ++e) o[e] *= inv * nw[e] * gate[e] * sigmoid_f(gate[e]);
+      de_store4(static_cast<E*>(p.out) + (static_cast<size_t>(t) * p.heads + h) * p.out_vd + 4 * lane, o);
+    }
+#pragma unroll
+    for (int e = 0; e < 4; ++e) u[e] *= ik;
+#pragma unroll
+    for (int r = 0; r < kR; ++r) {
+      const float kv = c[D + warp * kR + r];
+      S[r].x = fmaf(kv, u[0], g * S[r].x); S[r].y = fmaf(kv, u[1], g * S[r].y);
+      S[r].z = fmaf(kv, u[2], g * S[r].z); S[r].w = fmaf(kv, u[3], g * S[r].w);
+    }
+  }
+  if (t1 > t0) {
+#pragma unroll
+    for (int r = 0; r < kR; ++r) __stcg(reinterpret_cast<float4*>(st_out + s_at + r * 128), S[r]);
+#pragma unroll
+    for (int n = 0; n < kN; ++n) {
+      const int c = tid + n * 256;
+      if (chan[n] >= 0 && (c >= 2 * D || h == kh * rep)) {
+#pragma unroll
+        for (int j = 0; j < kTaps - 1; ++j) {
+          const int i = j - (kTaps - 1 - halo);
+          if (i >= 0) st_out[p.c_off + static_cast<size_t>(i) * channels + chan[n]] = win[n][j];
+        }
+      }
+    }
+  }
+}
+
 template <typename E, int MAXT>
 static int launch_delta(const DeltaArgs& p, cudaStream_t st) {
+  if (MAXT <= 4 && p.vdim == 128 && (p.dim == 64 || p.dim == 128) && p.out_vd % 4 == 0 && p.s_off % 4 == 0 && p.slot_stride % 4 == 0) {
+    if (p.dim == 64) launch_pdl(delta_step128_kernel<E, 64>, dim3(p.heads, p.S), dim3(256), 0, st, p);
+    else launch_pdl(delta_step128_kernel<E, 128>, dim3(p.heads, p.S), dim3(256), 0, st, p);
+    return static_cast<int>(cudaGetLastError());
+  }
   const int vt = p.vdim < kDeltaCols ? p.vdim : kDeltaCols;
   const int n_slice = (p.dim + kDeltaRows - 1) / kDeltaRows;
   int threads = vt * n_slice;

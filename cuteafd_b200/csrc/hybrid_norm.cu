@@ -45,7 +45,16 @@ template <> __device__ __forceinline__ float ld_e<__nv_bfloat16>(const __nv_bflo
 
 template <typename E, int V>
 __device__ __forceinline__ void load_vec(const E* p, float (&v)[V]) {
-  if constexpr (V == 4 && sizeof(E) == 4) {
+  if constexpr (V == 8 && sizeof(E) == 4) {
+    const float4 q = *reinterpret_cast<const float4*>(p), r = *reinterpret_cast<const float4*>(p + 4);
+    v[0] = q.x; v[1] = q.y; v[2] = q.z; v[3] = q.w;
+    v[4] = r.x; v[5] = r.y; v[6] = r.z; v[7] = r.w;
+  } else if constexpr (V == 8) {
+    const uint4 q = *reinterpret_cast<const uint4*>(p);
+    const uint32_t w[4] = {q.x, q.y, q.z, q.w};
+#pragma unroll
+    for (int e = 0; e < 4; ++e) { v[2 * e] = bf16_lo(w[e]); v[2 * e + 1] = bf16_hi(w[e]); }
+  } else if constexpr (V == 4 && sizeof(E) == 4) {
     const float4 q = *reinterpret_cast<const float4*>(p);
     v[0] = q.x; v[1] = q.y; v[2] = q.z; v[3] = q.w;
   } else if constexpr (V == 4) {
@@ -57,7 +66,12 @@ __device__ __forceinline__ void load_vec(const E* p, float (&v)[V]) {
 }
 template <typename E, int V>
 __device__ __forceinline__ void store_vec(E* p, const float (&v)[V]) {
-  if constexpr (V == 4 && sizeof(E) == 4) {
+  if constexpr (V == 8 && sizeof(E) == 4) {
+    *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]);
+    *reinterpret_cast<float4*>(p + 4) = make_float4(v[4], v[5], v[6], v[7]);
+  } else if constexpr (V == 8) {
+    *reinterpret_cast<uint4*>(p) = make_uint4(pack_bf16(v[0], v[1]), pack_bf16(v[2], v[3]), pack_bf16(v[4], v[5]), pack_bf16(v[6], v[7]));
+  } else if constexpr (V == 4 && sizeof(E) == 4) {
     *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]);
   } else if constexpr (V == 4) {
     *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16(v[0], v[1]), pack_bf16(v[2], v[3]));
@@ -70,6 +84,8 @@ __device__ __forceinline__ void store_vec(E* p, const float (&v)[V]) {
 
 // V elements as they sit in memory: loads of rows to come stay packed in registers until their turn
 template <typename E, int V> struct Packed;
+template <> struct __align__(16) Packed<float, 8> { float4 q, r; };
+template <> struct Packed<__nv_bfloat16, 8> { uint4 q; };
 template <> struct Packed<float, 4> { float4 q; };
 template <> struct Packed<__nv_bfloat16, 4> { uint2 q; };
 template <> struct Packed<float, 1> { float q; };
@@ -80,6 +96,15 @@ __device__ __forceinline__ void unpack(const Packed<float, 4>& a, float (&v)[4])
 __device__ __forceinline__ void unpack(const Packed<__nv_bfloat16, 4>& a, float (&v)[4]) {
   v[0] = bf16_lo(a.q.x); v[1] = bf16_hi(a.q.x); v[2] = bf16_lo(a.q.y); v[3] = bf16_hi(a.q.y);
 }
+__device__ __forceinline__ void unpack(const Packed<float, 8>& a, float (&v)[8]) {
+  v[0] = a.q.x; v[1] = a.q.y; v[2] = a.q.z; v[3] = a.q.w;
+  v[4] = a.r.x; v[5] = a.r.y; v[6] = a.r.z; v[7] = a.r.w;
+}
+__device__ __forceinline__ void unpack(const Packed<__nv_bfloat16, 8>& a, float (&v)[8]) {
+  const uint32_t w[4] = {a.q.x, a.q.y, a.q.z, a.q.w};
+#pragma unroll
+  for (int e = 0; e < 4; ++e) { v[2 * e] = bf16_lo(w[e]); v[2 * e + 1] = bf16_hi(w[e]); }
+}
 __device__ __forceinline__ void unpack(const Packed<float, 1>& a, float (&v)[1]) { v[0] = a.q; }
 __device__ __forceinline__ void unpack(const Packed<__nv_bfloat16, 1>& a, float (&v)[1]) { v[0] = __bfloat162float(a.q); }
 
@@ -88,11 +113,11 @@ constexpr int kSlotBatch = 8;       // routed rows of a token whose loads are in
 
 // 1 / sqrt(mean of squares + eps) of the group each of this thread's vectors lies in.  `part` holds one number per 32
 // vectors when groups are whole multiples of that (fast), else one per vector; `gsum` one per group (slow form only).
-template <int V, int KV>
+template <int V, int KV, bool kExact>
 __device__ __forceinline__ void group_inv(const float (&v)[KV][V], float (&inv)[KV], float* part, float* gsum, int nvec, int gvec,
-                                          bool fast, float eps) {
+                                          const int (&grp)[KV], float inv_n, bool fast, float eps) {
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, nt = blockDim.x;
-  const float inv_n = 1.0f / static_cast<float>(gvec * V);
+  auto root = [&](float s) { return kExact ? 1.0f / sqrtf(s * inv_n + eps) : rsqrtf(s * inv_n + eps); };
   if (fast) {
 #pragma unroll
     for (int k = 0; k < KV; ++k) {
@@ -110,10 +135,10 @@ __device__ __forceinline__ void group_inv(const float (&v)[KV][V], float (&inv)[
       const int i = tid + k * nt;
       float s = 0.f;
       if (i < nvec) {
-        const int g0 = (i / gvec) * per;
+        const int g0 = grp[k] * per;
         for (int j = 0; j < per; ++j) s += part[g0 + j];
       }
-      inv[k] = 1.0f / sqrtf(s * inv_n + eps);
+      inv[k] = root(s);
     }
   } else {
 #pragma unroll
@@ -136,7 +161,7 @@ __device__ __forceinline__ void group_inv(const float (&v)[KV][V], float (&inv)[
 #pragma unroll
     for (int k = 0; k < KV; ++k) {
       const int i = tid + k * nt;
-      inv[k] = i < nvec ? 1.0f / sqrtf(gsum[i / gvec] * inv_n + eps) : 0.f;
+      inv[k] = i < nvec ? root(gsum[grp[k]]) : 0.f;
     }
   }
 }
@@ -154,6 +179,10 @@ __global__ void __launch_bounds__(kMaxThreads, kMinBlocks) norm_conv_kernel(cons
   const int r1 = min(a.T, r0 + a.run);
   if (r0 >= a.T) return;
   const int halo = a.conv ? a.taps - 1 : 0;
+  const float inv_n = 1.0f / static_cast<float>(gvec * V);
+  int grp[KV];
+#pragma unroll
+  for (int k = 0; k < KV; ++k) grp[k] = (tid + k * nt) / gvec;
 
   float win[MAXT > 1 ? MAXT - 1 : 1][KV][V];   // the last taps - 1 convolution inputs, oldest first, at the array's end
 #pragma unroll
@@ -283,7 +312,7 @@ __global__ void __launch_bounds__(kMaxThreads, kMinBlocks) norm_conv_kernel(cons
     if (t + 1 < r1) fetch(t + 1);
     if (a.y) {
       float inv[KV];
-      group_inv<V, KV>(y, inv, sm + flip * stride, sm + flip * stride + nvec, nvec, gvec, fast, a.eps);
+      group_inv<V, KV, sizeof(E) == 4>(y, inv, sm + flip * stride, sm + flip * stride + nvec, nvec, gvec, grp, inv_n, fast, a.eps);
       flip ^= 1;
 #pragma unroll
       for (int k = 0; k < KV; ++k) {
@@ -304,7 +333,7 @@ __global__ void __launch_bounds__(kMaxThreads, kMinBlocks) norm_conv_kernel(cons
       }
     }
     float inv[KV];
-    group_inv<V, KV>(x, inv, sm + flip * stride, sm + flip * stride + nvec, nvec, gvec, fast, a.eps);
+    group_inv<V, KV, sizeof(E) == 4>(x, inv, sm + flip * stride, sm + flip * stride + nvec, nvec, gvec, grp, inv_n, fast, a.eps);
     flip ^= 1;
 #pragma unroll
     for (int k = 0; k < KV; ++k) {                                           // x now holds h
@@ -394,14 +423,20 @@ static int launch_norm(const NormArgs& a, int threads, cudaStream_t st) {
 
 template <typename E>
 static int dispatch_norm(NormArgs a, cudaStream_t st) {
-  if ((a.H / a.groups) % 4 == 0) {
+  const int per_group = a.H / a.groups;
+  auto threads = [](int n) { return (n + 31) / 32 * 32; };
+  if (per_group % 8 == 0) {
+    // eight channels per thread: a thread's channels share their group, so one reduction serves them all
+    const int nvec = a.H / 8;
+    if (nvec <= 256) return launch_norm<E, 8, 1, 256, 3>(a, threads(nvec), st);
+    if (nvec <= 512) return launch_norm<E, 8, 1, 512, 1>(a, threads(nvec), st);
+    if (nvec <= 1024) return launch_norm<E, 8, 2, 512, 1>(a, threads((nvec + 1) / 2), st);
+    return -13;
+  }
+  if (per_group % 4 == 0) {
     const int nvec = a.H / 4;
-    auto threads = [&](int kv) { return ((nvec + kv - 1) / kv + 31) / 32 * 32; };
-    // prompts: small blocks (several per SM, each at its own token) hide the loads and barriers better than wide ones
-    if (a.T >= 512 && nvec >= 256 && nvec <= kNormThreads) return launch_norm<E, 4, 2, 256, 3>(a, threads(2), st);
-    if (nvec <= kNormThreads) return launch_norm<E, 4, 1>(a, threads(1), st);
-    if (nvec <= 2 * kNormThreads) return launch_norm<E, 4, 2>(a, threads(2), st);
-    if (nvec <= 4 * kNormThreads) return launch_norm<E, 4, 4>(a, threads(4), st);
+    if (nvec <= kNormThreads) return launch_norm<E, 4, 1>(a, threads(nvec), st);
+    if (nvec <= 4 * kNormThreads) return launch_norm<E, 4, 4>(a, threads((nvec + 3) / 4), st);
     return -13;
   }
   if (a.H <= kNormThreads) return launch_norm<E, 1, 1>(a, (a.H + 31) / 32 * 32, st);

@@ -230,7 +230,7 @@ def _delta_oracle(m, w, x, st, eps):
     return (R.rms(o, eps) * w.out_norm) * R.silu(x["g"].view(n, m.heads, m.vdim))
 
 
-DELTAS = [delta(), delta(2, 2, 40, 136, 5), delta(1, 1, 16, 16, 1), delta(3, 1, 33, 7, 2), delta(4, 2, 128, 128, 4), delta(2, 1, 256, 64, 4),
+DELTAS = [delta(), delta(4, 4, 64, 128, 3), delta(2, 2, 40, 136, 5), delta(1, 1, 16, 16, 1), delta(3, 1, 33, 7, 2), delta(4, 2, 128, 128, 4), delta(2, 1, 256, 64, 4),
           delta(2, 2, 64, 300, 16)]
 
 
