@@ -603,6 +603,11 @@ static int launch_chunks(const DeltaArgs& p, void* scratch, long long scratch_by
   int slab = static_cast<int>(scratch_bytes / per_chunk);
   if (slab < 1) return -14;
   const int total = p.T / kChunk + p.S;                     // no portion has more than one chunk that is not full
+  const int wave = 2 * 148 / p.heads;                       // chunks whose blocks fill the GPU once (two per SM)
+  if (wave > 0 && slab > wave) {                            // whole waves of delta_prepare per slab
+    int waves = slab * p.heads / (2 * 148);
+    slab = waves * 2 * 148 / p.heads;
+  }
   if (slab > total) slab = total;
   const size_t units = static_cast<size_t>(slab) * p.heads;
   ChunkBufs b;

@@ -109,7 +109,7 @@ __device__ __forceinline__ void unpack(const Packed<float, 1>& a, float (&v)[1])
 __device__ __forceinline__ void unpack(const Packed<__nv_bfloat16, 1>& a, float (&v)[1]) { v[0] = __bfloat162float(a.q); }
 
 constexpr int kNormThreads = 512;
-constexpr int kSlotBatch = 8;       // routed rows of a token whose loads are in flight together
+constexpr int kSlotBatch = 4;       // routed rows of a token whose loads are in flight together
 
 // 1 / sqrt(mean of squares + eps) of the group each of this thread's vectors lies in.  `part` holds one number per 32
 // vectors when groups are whole multiples of that (fast), else one per vector; `gsum` one per group (slow form only).
@@ -405,11 +405,16 @@ __global__ void __launch_bounds__(kMaxThreads, kMinBlocks) norm_conv_kernel(cons
 }
 
 template <typename E, int V, int KV, int kMaxThreads = kNormThreads, int kMinBlocks = 1>
-static int launch_norm(const NormArgs& a, int threads, cudaStream_t st) {
+static int launch_norm(NormArgs a, int threads, cudaStream_t st) {
   const int nvec = a.H / V, gvec = nvec / a.groups;
   const int stride = (gvec % 32 == 0) ? nvec / 32 : nvec + a.groups;
   const size_t smem = static_cast<size_t>(2 * stride) * 4;
   if (smem > 48 * 1024) return -12;
+  if (a.run <= 0) {
+    // decode: one token per block; prompts: one wave of blocks, each with a run of tokens
+    const int run = (a.T + kMinBlocks * 148 - 1) / (kMinBlocks * 148);
+    a.run = run <= 2 ? 1 : run > 64 ? 64 : run;
+  }
   const dim3 grid((a.T + a.run - 1) / a.run);
   if (!a.conv || a.taps <= 4) {
     if (a.slot_w) launch_pdl(norm_conv_kernel<E, V, KV, 4, true, kMaxThreads, kMinBlocks>, grid, dim3(threads), smem, st, a);
@@ -468,11 +473,6 @@ extern "C" int cafd_norm_conv(const NormArgs* args, int is_f32, cafd_stream_t s)
   if (a.conv && (a.row_idx || !a.q_start || a.S < 1 || (a.taps > 1 && (!a.state || !a.state_in || !a.state_out)))) return -10;
   if (!a.embed && !a.x_in) return -10;
   if (a.x_out && a.x_out == a.x_in) return -11;
-  if (a.run <= 0) {
-    // decode: one token per block; prompts: runs long enough that the recomputed inputs stay a small share
-    int run = (a.T + 4 * 148 - 1) / (4 * 148);
-    a.run = run <= 2 ? 1 : run > 32 ? 32 : run;
-  }
   cudaStream_t st = static_cast<cudaStream_t>(s);
   return is_f32 ? dispatch_norm<float>(a, st) : dispatch_norm<__nv_bfloat16>(a, st);
 }
