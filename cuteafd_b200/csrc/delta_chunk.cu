@@ -60,6 +60,8 @@ __device__ __forceinline__ void split2(float a, float b, uint32_t& hi, uint32_t&
   hi = pack_bf16(a, b);
   lo = pack_bf16(a - bf16_lo(hi), b - bf16_hi(hi));
 }
+// silu on the special-function unit; the clamp keeps the denominator finite (below -80 the result rounds to zero anyway)
+__device__ __forceinline__ float silu_fast(float x) { return __fdividef(x, 1.0f + __expf(fminf(-x, 80.f))); }
 __device__ __forceinline__ uint4 as4(const uint32_t (&r)[4]) { return make_uint4(r[0], r[1], r[2], r[3]); }
 
 // Chunk `c` of the step -> its sequence and place.  False past the last chunk.
@@ -139,8 +141,8 @@ __global__ void __launch_bounds__(kChunkThreads, 2) delta_prepare_kernel(const D
 #pragma unroll
       for (int j = 0; j < 4; ++j) { y0 = fmaf(w0[j], x0[j], y0); y1 = fmaf(w1[j], x1[j], y1); }
       const bool live = i0 + r < len;
-      y0 = live ? y0 / (1.0f + __expf(-y0)) : 0.f;
-      y1 = live ? y1 / (1.0f + __expf(-y1)) : 0.f;
+      y0 = live ? silu_fast(y0) : 0.f;
+      y1 = live ? silu_fast(y1) : 0.f;
       uint32_t hi, lo;
       split2(y0, y1, hi, lo);
       const int at = (grp * kPer + r) * kP + 2 * pr;
@@ -431,7 +433,12 @@ __global__ void __launch_bounds__(kChunkThreads, 2) delta_prepare_kernel(const D
 template <int D>
 __global__ void __launch_bounds__(kChunkThreads, 1) delta_scan_kernel(const DeltaArgs p, const ChunkBufs b) {
   constexpr int kKS = D / 16, kSP = kSlice + 8;
-  __shared__ __align__(16) __nv_bfloat16 sh[D * kSP], sl[D * kSP], vh[kChunk * kSP], vl[kChunk * kSP];
+  extern __shared__ __align__(16) uint8_t smem_raw[];
+  __nv_bfloat16* sh = reinterpret_cast<__nv_bfloat16*>(smem_raw);   // the state's halves [D][kSP] each, then u's [64][kSP]
+  __nv_bfloat16* sl = sh + D * kSP;
+  __nv_bfloat16* vh = sl + D * kSP;
+  __nv_bfloat16* vl = vh + kChunk * kSP;
+  uint4* ring = reinterpret_cast<uint4*>(vl + kChunk * kSP);        // per warp and parity: K fragments, then P fragments or U
   pdl_wait();
   pdl_trigger();
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
@@ -480,28 +487,39 @@ __global__ void __launch_bounds__(kChunkThreads, 1) delta_scan_kernel(const Delt
 #pragma unroll
     for (int ks = 0; ks < kKS; ++ks) { fa[ks][0] = __ldcg(src + ks * 64); fa[ks][1] = __ldcg(src + ks * 64 + 32); }
   };
-  load_a(c_lo);
-  __syncthreads();
-  for (int c = c_lo; c < c_hi; ++c) {
+  // operands of the second half travel through shared memory, also one chunk ahead; a warp reads only what its own lanes
+  // copied, so waiting for the copies is all the ordering they need
+  constexpr int kRing = 512;                                // uint4 per warp and parity: 256 K, 256 P (or 128 U)
+  auto copy_b = [&](int c) {
     const size_t unit = static_cast<size_t>(c - b.chunk0) * p.heads + h;
-    // operands of the second half of this chunk
-    uint4 fp[4][2], fk[4][2];
-    float4 u[4];
-    const float g_end = __ldcg(b.g + unit);
-    if (first) {
-      const float4* src = b.u + ((unit * 4 + mt) * (p.vdim >> 3) + (v0 >> 3)) * 32 + lane;
-#pragma unroll
-      for (int nt = 0; nt < 4; ++nt) u[nt] = __ldcg(src + nt * 32);
-    } else {
-      const uint4* src = b.p + (unit * 4 + mt) * 4 * 64 + lane;
-#pragma unroll
-      for (int ks = 0; ks < 4; ++ks) { fp[ks][0] = __ldcg(src + ks * 64); fp[ks][1] = __ldcg(src + ks * 64 + 32); }
-    }
+    uint4* dst = ring + ((c & 1) * 8 + warp) * kRing + lane;
+    auto cp = [&](uint4* d, const void* s) {
+      asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(smem_u32(d)), "l"(s) : "memory");
+    };
     if (holds) {
       const uint4* src = b.k + (unit * kKS + warp) * 4 * 64 + lane;
 #pragma unroll
-      for (int ks = 0; ks < 4; ++ks) { fk[ks][0] = __ldcg(src + ks * 64); fk[ks][1] = __ldcg(src + ks * 64 + 32); }
+      for (int i = 0; i < 8; ++i) cp(dst + i * 32, src + i * 32);
     }
+    if (first) {
+      const float4* src = b.u + ((unit * 4 + mt) * (p.vdim >> 3) + (v0 >> 3)) * 32 + lane;
+#pragma unroll
+      for (int nt = 0; nt < 4; ++nt) cp(dst + 256 + nt * 32, src + nt * 32);
+    } else {
+      const uint4* src = b.p + (unit * 4 + mt) * 4 * 64 + lane;
+#pragma unroll
+      for (int i = 0; i < 8; ++i)
+        if ((i >> 1) <= mt) cp(dst + 256 + i * 32, src + i * 32);
+    }
+    asm volatile("cp.async.commit_group;" ::: "memory");
+  };
+  load_a(c_lo);
+  copy_b(c_lo);
+  __syncthreads();
+  for (int c = c_lo; c < c_hi; ++c) {
+    const size_t unit = static_cast<size_t>(c - b.chunk0) * p.heads + h;
+    const float g_end = __ldcg(b.g + unit);
+    const uint4* mine = ring + ((c & 1) * 8 + warp) * kRing + lane;
     float acc[4][4] = {};
 #pragma unroll
     for (int ks = 0; ks < kKS; ++ks) {
@@ -519,16 +537,22 @@ __global__ void __launch_bounds__(kChunkThreads, 1) delta_scan_kernel(const Delt
         }
       }
     }
-    if (c + 1 < c_hi) load_a(c + 1);
+    asm volatile("cp.async.wait_group 0;" ::: "memory");
+    __syncwarp();
+    if (c + 1 < c_hi) {
+      load_a(c + 1);
+      copy_b(c + 1);
+    }
     if (first) {
 #pragma unroll
       for (int nt = 0; nt < 4; ++nt) {
         uint32_t hi, lo;
         const int at = (16 * mt + gr) * kSP + nt * 8 + tc;
-        split2(u[nt].x - acc[nt][0], u[nt].y - acc[nt][1], hi, lo);
+        const float4 u = *reinterpret_cast<const float4*>(mine + 256 + nt * 32);
+        split2(u.x - acc[nt][0], u.y - acc[nt][1], hi, lo);
         *reinterpret_cast<uint32_t*>(vh + at) = hi;
         *reinterpret_cast<uint32_t*>(vl + at) = lo;
-        split2(u[nt].z - acc[nt][2], u[nt].w - acc[nt][3], hi, lo);
+        split2(u.z - acc[nt][2], u.w - acc[nt][3], hi, lo);
         *reinterpret_cast<uint32_t*>(vh + at + 8 * kSP) = hi;
         *reinterpret_cast<uint32_t*>(vl + at + 8 * kSP) = lo;
       }
@@ -560,8 +584,8 @@ __global__ void __launch_bounds__(kChunkThreads, 1) delta_scan_kernel(const Delt
             mma16816(d[nt], al, bh[nn][e], bh[nn][e + 1]);
           }
         };
-        if (holds) mul(S, fk[ks][0], fk[ks][1]);
-        if (want_o) mul(acc, fp[ks][0], fp[ks][1]);
+        if (holds) mul(S, mine[ks * 64], mine[ks * 64 + 32]);
+        if (want_o) mul(acc, mine[256 + ks * 64], mine[256 + ks * 64 + 32]);
       }
     }
     put_state();
@@ -594,15 +618,17 @@ constexpr size_t unit_bytes(int D, int vdim) {
 template <int D>
 static int launch_chunks(const DeltaArgs& p, void* scratch, long long scratch_bytes, cudaStream_t st) {
   constexpr size_t smem = static_cast<size_t>(4) * kChunk * (D + 8) * 2 + 2 * kChunk * kTPitch * 4;
+  constexpr size_t scan_smem = static_cast<size_t>(2 * D + 2 * kChunk) * (kSlice + 8) * 2 + 2 * 8 * 512 * 16;
   static bool attr = false;
   if (!attr) {
+    CAFD_CHECK_CUDA(cudaFuncSetAttribute(delta_scan_kernel<D>, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(scan_smem)));
     CAFD_CHECK_CUDA(cudaFuncSetAttribute(delta_prepare_kernel<D>, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem)));
     attr = true;
   }
   const size_t per_chunk = unit_bytes(D, p.vdim) * p.heads;
   int slab = static_cast<int>(scratch_bytes / per_chunk);
   if (slab < 1) return -14;
-  const int total = p.T / kChunk + p.S;                     // no portion has more than one chunk that is not full
+  const int total = (p.T + (kChunk - 1) * p.S) / kChunk;    // every portion ends in at most one chunk that is not full
   const int wave = 2 * 148 / p.heads;                       // chunks whose blocks fill the GPU once (two per SM)
   if (wave > 0 && slab > wave) {                            // whole waves of delta_prepare per slab
     int waves = slab * p.heads / (2 * 148);
@@ -622,7 +648,7 @@ static int launch_chunks(const DeltaArgs& p, void* scratch, long long scratch_by
   for (b.chunk0 = 0; b.chunk0 < total; b.chunk0 += slab) {
     const int n = total - b.chunk0 < slab ? total - b.chunk0 : slab;
     launch_pdl(delta_prepare_kernel<D>, dim3(n, p.heads), dim3(kChunkThreads), smem, st, p, b);
-    launch_pdl(delta_scan_kernel<D>, dim3(p.heads, p.vdim / kSlice, p.S), dim3(kChunkThreads), 0, st, p, b);
+    launch_pdl(delta_scan_kernel<D>, dim3(p.heads, p.vdim / kSlice, p.S), dim3(kChunkThreads), scan_smem, st, p, b);
   }
   const long long rows = static_cast<long long>(p.T) * p.heads;
   const int blocks = static_cast<int>(rows < 8 * 148 * 8 ? (rows + 7) / 8 : 148 * 8);

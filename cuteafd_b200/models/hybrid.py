@@ -423,7 +423,7 @@ class HybridEngine:
         args = (a, L.offs, m, L, self.kv.state, off["S"], off["conv"], b.state_in, b.state_out, b.q_start, out, ws.raw, self.cfg.rms_eps)
         if b.prefill and b.max_q_len >= self.CHUNKED_DELTA_TOKENS and K.delta_chunk_ok(m, self.dtype):
             K.delta_chunked(ws.chunk, *args)
-            slabs = -(-(T // 64 + b.q_start.shape[0] - 1) * K.delta_chunk_bytes(m) // ws.chunk.numel())
+            slabs = -(-((T + 63 * (b.q_start.shape[0] - 1)) // 64) * K.delta_chunk_bytes(m) // ws.chunk.numel())
             self.launches += 2 * slabs + 1
         else:
             K.delta_step(*args)
