@@ -81,7 +81,7 @@ class NormArgs(C.Structure):
     _fields_ = [(n, C.c_void_p) for n in ("tokens", "embed", "x_in", "y", "slot_w", "slot_idx", "ident", "w_b", "w", "conv", "x_out",
                                           "h_out", "row_idx", "state", "state_in", "state_out", "q_start")]
     _fields_ += [("slot_stride", C.c_longlong), ("state_off", C.c_longlong)]
-    _fields_ += [(n, C.c_int) for n in ("T", "H", "S", "ldy", "groups", "taps", "top_k", "n_experts", "vocab", "run")] + [("eps", C.c_float)]
+    _fields_ += [(n, C.c_int) for n in ("T", "H", "S", "ldy", "ldh", "groups", "taps", "top_k", "n_experts", "vocab", "run")] + [("eps", C.c_float)]
 
 
 class LatentPrep(C.Structure):

@@ -58,6 +58,7 @@ class HybridWeights:
     def build(cfg: ModelConfig, get, device: torch.device) -> "HybridWeights":
         """``get(name) -> tensor`` under the checkpoint's names (any float dtype, any device)."""
         dt = engine_dtype(cfg)
+        H, Hp = cfg.hidden, pad8(cfg.hidden)
 
         def t(name: str, shape: tuple | None = None) -> torch.Tensor:
             x = get(name).to(device=device, dtype=dt)
@@ -65,29 +66,32 @@ class HybridWeights:
                 raise ValueError(f"{name}: shape {tuple(x.shape)}, the configuration says {shape}")
             return x.contiguous()
 
+        def reads(x: torch.Tensor) -> torch.Tensor:
+            """A matrix that reads the layer input: columns up to whole 16-byte rows."""
+            return x if Hp == H else torch.nn.functional.pad(x, (0, Hp - H)).contiguous()
+
         def f(name: str) -> torch.Tensor:
             return get(name).to(device=device, dtype=torch.float32).contiguous()
 
         def fuse(parts: list[tuple[str, torch.Tensor]]) -> tuple[torch.Tensor, dict]:
             rows = sum(pad8(x.shape[0]) for _, x in parts)
-            out = torch.zeros(rows, cfg.hidden, dtype=dt, device=device)
+            out = torch.zeros(rows, Hp, dtype=dt, device=device)
             offs, o = {}, 0
             for n, x in parts:
-                out[o:o + x.shape[0]] = x
+                out[o:o + x.shape[0], :H] = x
                 offs[n] = o
                 o += pad8(x.shape[0])
             return out, offs
 
         def heads_o(name: str, heads: int, vdim: int) -> torch.Tensor:
             """o projection with every head's columns padded to the row layout the mixers write."""
-            w = t(name, (cfg.hidden, heads * vdim)).view(cfg.hidden, heads, vdim)
-            out = torch.zeros(cfg.hidden, heads, pad8(vdim), dtype=dt, device=device)
-            out[..., :vdim] = w
-            return out.view(cfg.hidden, heads * pad8(vdim))
+            w = t(name, (H, heads * vdim)).view(H, heads, vdim)
+            out = torch.zeros(Hp, heads, pad8(vdim), dtype=dt, device=device)
+            out[:H, :, :vdim] = w
+            return out.view(Hp, heads * pad8(vdim))
 
-        H = cfg.hidden
         W = HybridWeights(cfg)
-        W.embed, W.final_norm, W.lm_head = t("embed", (cfg.vocab_size, H)), f("final.norm"), t("head", (cfg.vocab_size, H))
+        W.embed, W.final_norm, W.lm_head = t("embed", (cfg.vocab_size, H)), f("final.norm"), reads(t("head", (cfg.vocab_size, H)))
         for i, spec in enumerate(cfg.layer_specs):
             pre, m, r, L = f"l{i}.", spec.mixer, spec.router, HybridLayer()
             x = pre + "mix."
@@ -117,14 +121,14 @@ class HybridWeights:
                 y = pre + "mlp."
                 L.norm2, L.norm2b = f(pre + "norm2"), f(pre + "norm2b")
                 L.canon2 = f(pre + "canon2").T.contiguous()
-                L.router, L.correction = t(y + "router", (r.outputs, H)), f(y + "correction")
+                L.router, L.correction = reads(t(y + "router", (r.outputs, H))), f(y + "correction")
                 F = pad8(r.ffn)
-                L.w_gate, L.w_up = (torch.zeros(r.experts, F, H, dtype=dt, device=device) for _ in range(2))
-                L.w_down = torch.zeros(r.experts, H, F, dtype=dt, device=device)
+                L.w_gate, L.w_up = (torch.zeros(r.experts, F, Hp, dtype=dt, device=device) for _ in range(2))
+                L.w_down = torch.zeros(r.experts, Hp, F, dtype=dt, device=device)
                 for e in range(r.experts):
-                    L.w_gate[e, :r.ffn] = t(f"{y}e{e}.gate", (r.ffn, H))
-                    L.w_up[e, :r.ffn] = t(f"{y}e{e}.up", (r.ffn, H))
-                    L.w_down[e, :, :r.ffn] = t(f"{y}e{e}.down", (H, r.ffn))
+                    L.w_gate[e, :r.ffn, :H] = t(f"{y}e{e}.gate", (r.ffn, H))
+                    L.w_up[e, :r.ffn, :H] = t(f"{y}e{e}.up", (r.ffn, H))
+                    L.w_down[e, :H, :r.ffn] = t(f"{y}e{e}.down", (H, r.ffn))
             W.layers.append(L)
         return W
 
@@ -246,8 +250,6 @@ class HybridEngine:
 
     def __init__(self, cfg: ModelConfig, weights: HybridWeights, kv: HybridCache, max_tokens: int, max_seqs: int = 64):
         assert cfg.is_hybrid
-        if cfg.hidden % 8:
-            raise ValueError(f"width {cfg.hidden} is not a multiple of 8")
         self.cfg, self.W, self.kv = cfg, weights, kv
         self.device = dev = weights.embed.device
         self.dtype = dt = engine_dtype(cfg)
@@ -260,8 +262,9 @@ class HybridEngine:
             pass
         ws = self.ws = _Ws()
         ws.x = [torch.empty(max_tokens, H, dtype=torch.float32, device=dev) for _ in range(2)]
-        ws.h = [torch.empty(max_tokens, H, dtype=dt, device=dev) for _ in range(2)]
-        ws.y = torch.empty(max_tokens, H, dtype=dt, device=dev)
+        Hp = pad8(H)                     # rows the matrix products read are whole 16-byte pieces; the padding stays zero
+        ws.h = [torch.zeros(max_tokens, Hp, dtype=dt, device=dev) for _ in range(2)]
+        ws.y = torch.zeros(max_tokens, Hp, dtype=dt, device=dev)
         ws.proj = torch.empty(max_tokens * max(L.w_in.shape[0] for L in weights.layers), dtype=dt, device=dev)
         outs = max((s.router.outputs for s in cfg.layer_specs if s.router), default=1)
         ws.router = torch.empty(max_tokens * outs, dtype=torch.float32, device=dev)
@@ -285,7 +288,7 @@ class HybridEngine:
                     chunks = max(max(1, self.CHUNK_SCRATCH_BYTES // per), 1)
                     scratch = max(scratch, per * min(chunks, max_tokens // 64 + max_seqs))
             if r is not None and r not in self._moe:
-                self._moe[r] = LocalExchange(ExchangeGeometry(H, pad8(r.ffn), r.experts, r.top, max_tokens, 1), dev, dtype=dt)
+                self._moe[r] = LocalExchange(ExchangeGeometry(Hp, pad8(r.ffn), r.experts, r.top, max_tokens, 1), dev, dtype=dt)
         ws.raw = torch.empty(max_tokens * raw, dtype=torch.float32, device=dev) if raw else None
         ws.chunk = torch.empty(scratch, dtype=torch.uint8, device=dev) if scratch else None
         self.moe = None
@@ -320,10 +323,11 @@ class HybridEngine:
         x = self._x.clone()
         p = self._pending
         if p:
-            y, G = p["y"].float(), self.cfg.norm_groups
+            H = self.cfg.hidden
+            y, G = p["y"][:, :H].float(), self.cfg.norm_groups
             if "slots" in p:
                 w, idx, n, ident = p["slots"]
-                rows = torch.where((idx >= n)[..., None], ident.float()[:, None], y[:T * w.shape[1]].view(T, w.shape[1], -1))
+                rows = torch.where((idx >= n)[..., None], ident[:, :H].float()[:, None], y[:T * w.shape[1]].view(T, w.shape[1], -1))
                 y = (w[..., None] * rows).sum(1)
             g = y.view(T, G, -1)
             x = x + (g / torch.sqrt((g * g).mean(-1, keepdim=True) + self.cfg.rms_eps)).view(T, -1) * p["w_b"]
@@ -438,7 +442,7 @@ class HybridEngine:
                   group_score="max")
         logits = None
         idx, w = moe.att.idx[:T], moe.att.w[:T]
-        if self.dtype == torch.bfloat16 and T <= self.FUSED_ROUTE_TOKENS and self.cfg.hidden <= 8192:
+        if self.dtype == torch.bfloat16 and T <= self.FUSED_ROUTE_TOKENS and h.shape[1] <= 8192:
             K.norm_route(h, None, 0.0, L.router, None, idx, w, r.top, **kw)
             self.launches += 1
         else:

@@ -677,8 +677,9 @@ def norm_conv(h_out: torch.Tensor, w: torch.Tensor, groups: int, eps: float, *, 
               run: int = 0) -> None:
     """x = embed[tokens] or ``x_in`` (fp32); x += groupnorm(y) * w_b; h = groupnorm(x) * w; h_out = h + causal_conv(h).
 
-    ``slots`` = (weights [T, k], ids [T, k], number of experts, identity rows [T, H]): ``y`` then holds the routed experts'
-    rows [T * k, H] and is their weighted sum.  ``conv`` [taps, H] fp32 (last row = current token) with the sequences'
+    Rows of ``h_out``, ``y`` and the identity rows may be longer than H (whole 16-byte pieces); the rest is left alone.
+    ``slots`` = (weights [T, k], ids [T, k], number of experts, identity rows): ``y`` then holds the routed experts' rows
+    [T * k, ...] and is their weighted sum.  ``conv`` [taps, H] fp32 (last row = current token) with the sequences'
     earlier inputs in ``state`` [slots, floats] at ``state_off``.  ``rows``: compute only these rows (no convolution)."""
     a = _n.NormArgs()
     H = w.shape[0]
@@ -686,12 +687,12 @@ def norm_conv(h_out: torch.Tensor, w: torch.Tensor, groups: int, eps: float, *, 
     a.w_b, a.w, a.conv, a.x_out, a.h_out, a.row_idx = _ptr(w_b), w.data_ptr(), _ptr(conv), _ptr(x_out), h_out.data_ptr(), _ptr(rows)
     a.vocab = embed.shape[0] if embed is not None else 0
     a.T, a.H, a.groups, a.eps, a.run = h_out.shape[0], H, groups, eps, run
-    a.ldy = y.stride(0) if y is not None else 0
-    assert h_out.is_contiguous() and h_out.shape[1] == H and w.dtype == torch.float32
+    a.ldy, a.ldh = y.stride(0) if y is not None else 0, h_out.stride(0)
+    assert h_out.shape[1] >= H and h_out.stride(1) == 1 and w.dtype == torch.float32
     if slots is not None:
         sw, si, n, ident = slots
         a.slot_w, a.slot_idx, a.n_experts, a.ident, a.top_k = sw.data_ptr(), si.data_ptr(), n, ident.data_ptr(), sw.shape[1]
-        assert y.stride(0) == H and ident.stride(0) == H and sw.is_contiguous() and si.is_contiguous()
+        assert ident.stride(0) == a.ldh and sw.is_contiguous() and si.is_contiguous()
     if conv is not None:
         a.taps, a.S = conv.shape[0], q_start.shape[0] - 1
         a.state, a.state_in, a.state_out, a.q_start = state.data_ptr(), state_in.data_ptr(), state_out.data_ptr(), q_start.data_ptr()

@@ -274,7 +274,7 @@ def kernel_geometry(cfg: ModelConfig) -> str:
     """Why the CUDA engines cannot run this geometry ("" = they can): their attention kernels are written for one head
     shape per family."""
     if cfg.is_hybrid:
-        return "the hybrid engine takes a width that is a multiple of 8" if cfg.hidden % 8 else ""
+        return ""
     if cfg.is_mla:
         if (cfg.kv_lora_rank, cfg.qk_rope_dim, cfg.qk_nope_dim, cfg.v_head_dim) != (512, 64, 128, 128):
             return "the MLA kernels take the DeepSeek shape (latent 512, rope 64, nope 128, value 128)"

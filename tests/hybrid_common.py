@@ -32,6 +32,13 @@ def plain_config():
         LayerSpec(delta(4, 1, 64, 24, 4))], canon_taps=1, norm_groups=1, eps=1e-3)
 
 
+def narrow_config():
+    """A width that is no multiple of 8, so that rows are padded between the kernels, and longer convolutions."""
+    return hybrid_config("narrow", 77, 90, [
+        LayerSpec(latent(2, 12, 4, 10, 18, 21), RouterSpec(3, 10, 2, 1, 2, 1)),
+        LayerSpec(delta(3, 3, 10, 6, 6), RouterSpec(4, 9, 2, 0, 2, 2))], canon_taps=6, norm_groups=3, eps=1e-4)
+
+
 def wide_config(window=100):
     """The sizes the tensor-core kernels take."""
     return hybrid_config("wide", 500, 256, [

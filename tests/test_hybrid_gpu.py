@@ -10,7 +10,7 @@ import torch
 from cuteafd_b200.config import RouterSpec
 from cuteafd_b200.ref import hybrid as R
 
-from tests.hybrid_common import delta, err, latent, odd_config, oracle_logits, params, plain_config, tokens, wide_config
+from tests.hybrid_common import delta, err, latent, narrow_config, odd_config, oracle_logits, params, plain_config, tokens, wide_config
 
 pytestmark = pytest.mark.gpu
 DTYPES = [torch.float32, torch.bfloat16]
@@ -60,7 +60,9 @@ def test_norm_conv(dtype, H, groups, taps):
         qs, n = [0], T[step]
         for x in lens[step]:
             qs.append(qs[-1] + x)
-        h, x0 = torch.empty(n, H, dtype=dtype, device=dev()), torch.empty(n, H, device=dev())
+        hp = torch.full((n, -(-H // 8) * 8), 9.0, dtype=dtype, device=dev())
+        h, x0 = hp[:, :H], torch.empty(n, H, device=dev())
+        ypad = torch.nn.functional.pad(ys[step], (0, hp.shape[1] - H)).to(dev(), dtype)
         kw = dict(state=state, state_in=i32(ins), state_out=i32(outs), q_start=i32(qs), conv=cd)
         K.norm_conv(h, w.to(dev()), groups, eps, tokens=i32(toks[step]), embed=emb.to(dev(), dtype), x_out=x0, state_off=32, **kw)
         x = emb[torch.tensor(toks[step])]
@@ -72,7 +74,7 @@ def test_norm_conv(dtype, H, groups, taps):
             if taps > 1:
                 assert torch.allclose(state[outs[s], 32:32 + (taps - 1) * H].view(taps - 1, H).cpu(), past[s], atol=2e-5)
         x1 = torch.empty_like(x0)
-        K.norm_conv(h, w.to(dev()), groups, eps, x_in=x0, y=ys[step].to(dev(), dtype), w_b=wb.to(dev()), x_out=x1, state_off=second, run=7, **kw)
+        K.norm_conv(h, w.to(dev()), groups, eps, x_in=x0, y=ypad, w_b=wb.to(dev()), x_out=x1, state_off=second, run=7, **kw)
         x = x + R.group_rms(ys[step], wb, groups, eps)
         close(x1, x, torch.float32)
         for s in range(4):
@@ -80,8 +82,9 @@ def test_norm_conv(dtype, H, groups, taps):
             y, past_y[s] = R.causal_conv(g, c, past_y[s])
             close(h[qs[s]:qs[s + 1]], g + y, dtype)
         rows = [n - 1, 0, n // 2]
-        hf = torch.empty(3, H, dtype=dtype, device=dev())
-        K.norm_conv(hf, w.to(dev()), groups, eps, x_in=x0, y=ys[step].to(dev(), dtype), w_b=wb.to(dev()), rows=i32(rows))
+        assert (hp[:, H:] == 9.0).all()
+        hf = torch.empty(3, hp.shape[1], dtype=dtype, device=dev())[:, :H]
+        K.norm_conv(hf, w.to(dev()), groups, eps, x_in=x0, y=ypad, w_b=wb.to(dev()), rows=i32(rows))
         close(hf, R.group_rms(x[rows], w, groups, eps), dtype)
         ins, outs = outs, [1, 6, 7, 10] if step == 0 else outs
 
@@ -380,7 +383,7 @@ def check(got, want, dtype):
 
 
 SPREAD = {"f32": 0.4, "bf16": 2.0}
-CASES = [(odd_config(), "f32"), (odd_config(), "bf16"), (plain_config(), "f32"), (plain_config(), "bf16"), (wide_config(), "f32"),
+CASES = [(narrow_config(), "f32"), (narrow_config(), "bf16"), (odd_config(), "f32"), (odd_config(), "bf16"), (plain_config(), "f32"), (plain_config(), "bf16"), (wide_config(), "f32"),
          (wide_config(), "bf16")]
 IDS = [f"{c.name}-{d}" for c, d in CASES]
 
