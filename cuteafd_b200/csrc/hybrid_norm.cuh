@@ -171,10 +171,25 @@ __device__ __forceinline__ void group_inv(const float (&v)[KV][V], float (&inv)[
 template <typename E, int V, int KV, int MAXT, bool kSlots, int kMaxThreads, int kMinBlocks>
 __global__ void __launch_bounds__(kMaxThreads, kMinBlocks) norm_conv_kernel(const NormArgs a) {
   extern __shared__ float sm[];
-  pdl_wait();
-  pdl_trigger();
   const int tid = threadIdx.x, nt = blockDim.x;
   const int nvec = a.H / V, gvec = nvec / a.groups;
+  if (a.run == 1) {
+    // decode: the weights (and, when a block is a sequence, its state) are on their way into L2 while the previous
+    // kernel drains; nothing is read here
+    auto pull = [](const float* q) { asm volatile("prefetch.global.L2 [%0];" ::"l"(q)); };
+    const bool own_seq = a.conv && a.S == a.T && a.state;
+    const float* st = own_seq ? a.state + static_cast<size_t>(a.state_in[blockIdx.x]) * a.slot_stride + a.state_off : nullptr;
+    for (int i = tid * 32; i < a.H; i += nt * 32) {         // one 128-byte line per step
+      pull(a.w + i);
+      if (a.w_b) pull(a.w_b + i);
+      if (a.conv)
+        for (int j = 0; j < a.taps; ++j) pull(a.conv + static_cast<size_t>(j) * a.H + i);
+      if (st)
+        for (int j = 0; j + 1 < a.taps; ++j) pull(st + static_cast<size_t>(j) * a.H + i);
+    }
+  }
+  pdl_wait();
+  pdl_trigger();
   const bool fast = (gvec & 31) == 0;
   const int stride = fast ? (nvec >> 5) : nvec + a.groups;   // two alternating reduction buffers
   const int r0 = blockIdx.x * a.run;
