@@ -54,7 +54,7 @@ def main() -> None:
     ap.add_argument("--no-graphs", action="store_true")
     ap.add_argument("--config", default="qwen3", choices=["qwen3", "dsv3", "karusun"],
                     help="karusun = the per-layer hybrid (latent attention + delta-rule layers) at the sizes of a real model's layers, and the "
-                         "MLA engine at equal size beside it (one GPU); qwen3 = the headline Qwen3-30B-A3B bf16 card (with 8 GPUs the DeepSeek-V3 card follows it); dsv3 = only "
+                         "MLA engine at equal size beside it, three sizes (one GPU); qwen3 = the headline Qwen3-30B-A3B bf16 card (with 8 GPUs the DeepSeek-V3 card follows it); dsv3 = only "
                          "the DeepSeek-V3 shape: MLA attention replicas, E4M3 block-scaled experts on the other GPUs (needs 8 GPUs)")
     ap.add_argument("--attention-ranks", type=int, default=0,
                     help="data-parallel attention replicas of the disaggregated layout (0 = 1 on two GPUs, 2 on four or more)")
@@ -99,10 +99,11 @@ def main() -> None:
         """Build the deployment of one model configuration, run the card on it, tear it down.  Returns (cfg, card result
         or None on ranks that do not drive a card, parallelism string, clocks summary)."""
         cfg = qwen3_30b_a3b()
-        if name in ("karusun", "karusun-mla"):
+        if name.startswith("karusun"):            # karusun[-mla][:size]
             from cuteafd_b200.config import karusun_bench, karusun_bench_mla
             assert world == 1, "per-layer hybrids run on one GPU"
-            cfg = karusun_bench() if name == "karusun" else karusun_bench_mla()
+            kind, _, size = name.partition(":")
+            cfg = (karusun_bench if kind == "karusun" else karusun_bench_mla)(size or "base")
         if name == "dsv3":
             from cuteafd_b200 import deepseek_v3
             cfg = deepseek_v3().replace(mtp_layers=0)
@@ -232,10 +233,11 @@ def main() -> None:
             if rank == 0 and out is not None:
                 out["extra"]["dsv3_error"] = f"{type(e).__name__}: {e}"
     if args.config == "karusun" and out is not None:
-        mcfg, mres, _, mclk = run_config("karusun-mla")
-        out["extra"].update(card_extra(mres, "mla_equal_size_"))
-        out["extra"]["mla_equal_size_config"] = {"model": mcfg.name, "clocks": mclk, "parameters": mcfg.total_params(),
-                                                 "hybrid_parameters": cfg.total_params()}
+        # the MLA engine at equal size, then both at the other sizes
+        for name in ("karusun-mla:base", "karusun:small", "karusun-mla:small", "karusun:large", "karusun-mla:large"):
+            c, r2, _, k2 = run_config(name)
+            out["extra"].update(card_extra(r2, c.name.replace("-", "_") + "_"))
+            out["extra"][c.name.replace("-", "_") + "_config"] = {"parameters": c.total_params(), "clocks": k2}
     if world > 1:
         dist.barrier()
         dist.destroy_process_group()

@@ -353,26 +353,32 @@ def hybrid_config(name: str, vocab: int, hidden: int, specs, canon_taps: int, no
         norm_topk_prob=False, router_bias=bool(routers))
 
 
-def karusun_bench() -> ModelConfig:
-    """A Karusun-shaped stack at the sizes of a real model's layers (latent 512 + 64, heads of 128, 64 experts top-6 of which
-    the last eight hand their input through): three delta-rule layers to one latent attention layer."""
-    r = RouterSpec(experts=56, ffn=1024, top=6, identity=8, groups=8, groups_kept=4)
-    lat = LatentSpec(heads=32, dim=128, rot_dim=64, vdim=128, kv_rank=512, window=2048, scale=192 ** -0.5, rope_base=1.0e6)
-    delta = DeltaSpec(heads=32, kv_heads=16, dim=128, vdim=128, conv=4)
-    specs = [LayerSpec(lat if i % 4 == 3 else delta, r) for i in range(24)]
-    return hybrid_config("karusun-bench", 65536, 2048, specs, canon_taps=4, norm_groups=4, eps=1e-5)
+# Benchmark sizes: width, layers, heads, expert width (latent 512 + 64 and heads of 128 throughout, as real models have them)
+KARUSUN_SIZES = {"small": (1024, 24, 16, 512), "base": (2048, 24, 32, 1024), "large": (4096, 12, 64, 1536)}
 
 
-def karusun_bench_mla() -> ModelConfig:
+def karusun_bench(size: str = "base") -> ModelConfig:
+    """A Karusun-shaped stack at the sizes of a real model's layers (latent 512 + 64, heads of 128, 64 router outputs top-6 of
+    which the last eight hand their input through): three delta-rule layers to one latent attention layer."""
+    width, layers, heads, ffn = KARUSUN_SIZES[size]
+    r = RouterSpec(experts=56, ffn=ffn, top=6, identity=8, groups=8, groups_kept=4)
+    lat = LatentSpec(heads=heads, dim=128, rot_dim=64, vdim=128, kv_rank=512, window=2048, scale=192 ** -0.5, rope_base=1.0e6)
+    delta = DeltaSpec(heads=heads, kv_heads=heads // 2, dim=128, vdim=128, conv=4)
+    specs = [LayerSpec(lat if i % 4 == 3 else delta, r) for i in range(layers)]
+    return hybrid_config(f"karusun-{size}", 65536, width, specs, canon_taps=4, norm_groups=4, eps=1e-5)
+
+
+def karusun_bench_mla(size: str = "base") -> ModelConfig:
     """The MLA decoder at the size of ``karusun_bench``: same width, depth, heads, latent, experts and vocabulary."""
-    return ModelConfig(name="karusun-bench-mla", family="deepseek_v3", vocab_size=65536, num_layers=24, hidden=2048, attention="mla",
-                       num_heads=32, q_lora_rank=0, kv_lora_rank=512, qk_nope_dim=128, qk_rope_dim=64, v_head_dim=128, rope_theta=1.0e6,
-                       rope_interleaved=False, rms_eps=1e-5, dense_ffn=0, first_dense_layers=0, num_experts=56, expert_ffn=1024, top_k=6,
+    width, layers, heads, ffn = KARUSUN_SIZES[size]
+    return ModelConfig(name=f"mla-{size}", family="deepseek_v3", vocab_size=65536, num_layers=layers, hidden=width, attention="mla",
+                       num_heads=heads, q_lora_rank=0, kv_lora_rank=512, qk_nope_dim=128, qk_rope_dim=64, v_head_dim=128, rope_theta=1.0e6,
+                       rope_interleaved=False, rms_eps=1e-5, dense_ffn=0, first_dense_layers=0, num_experts=56, expert_ffn=ffn, top_k=6,
                        scoring="softmax", num_groups=8, topk_groups=4, num_shared_experts=0, norm_topk_prob=False, router_bias=True)
 
 
 PRESETS = {
-    "karusun-bench": karusun_bench,
+    "karusun-base": karusun_bench,
     "tiny-moe": tiny_moe,
     "mixtral-8x7b": mixtral_8x7b,
     "mistral-7b": mistral_7b,

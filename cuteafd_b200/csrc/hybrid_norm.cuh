@@ -111,7 +111,6 @@ __device__ __forceinline__ void unpack(const Packed<float, 1>& a, float (&v)[1])
 __device__ __forceinline__ void unpack(const Packed<__nv_bfloat16, 1>& a, float (&v)[1]) { v[0] = __bfloat162float(a.q); }
 
 constexpr int kNormThreads = 512;
-constexpr int kSlotBatch = 4;       // routed rows of a token whose loads are in flight together
 
 // 1 / sqrt(mean of squares + eps) of the group each of this thread's vectors lies in.  `part` holds one number per 32
 // vectors when groups are whole multiples of that (fast), else one per vector; `gsum` one per group (slow form only).
@@ -171,9 +170,11 @@ __device__ __forceinline__ void group_inv(const float (&v)[KV][V], float (&inv)[
 template <typename E, int V, int KV, int MAXT, bool kSlots, int kMaxThreads, int kMinBlocks>
 __global__ void __launch_bounds__(kMaxThreads, kMinBlocks) norm_conv_kernel(const NormArgs a) {
   extern __shared__ float sm[];
+  // routed rows of a token whose loads are in flight together (prompts: several blocks per SM share the registers)
+  constexpr int kSlotBatch = kMinBlocks == 1 ? 8 : 4;
   const int tid = threadIdx.x, nt = blockDim.x;
   const int nvec = a.H / V, gvec = nvec / a.groups;
-  if (a.run == 1) {
+  if (kMinBlocks == 1 && a.run == 1) {
     // decode: the weights (and, when a block is a sequence, its state) are on their way into L2 while the previous
     // kernel drains; nothing is read here
     auto pull = [](const float* q) { asm volatile("prefetch.global.L2 [%0];" ::"l"(q)); };
@@ -445,7 +446,9 @@ static int dispatch_norm(const NormArgs& a, cudaStream_t st) {
   const bool few = !a.conv || a.taps <= 4;
   if (few && per_group % 8 == 0) {
     // eight channels per thread: a thread's channels share their group, so one reduction serves them all
-    if (a.H <= 2048) return launch_norm<E, 8, 1, 4, 256, 3>(a, st);
+    // prompts: several blocks per SM, each at its own token, hide the loads and barriers; decode: one block per token
+    if (a.T > 256 && a.H <= 2048) return launch_norm<E, 8, 1, 4, 256, 3>(a, st);
+    if (a.T > 256 && a.H <= 4096) return launch_norm<E, 8, 2, 4, 256, 2>(a, st);
     if (a.H <= 4096) return launch_norm<E, 8, 1, 4, 512, 1>(a, st);
     if (a.H <= 8192) return launch_norm<E, 8, 2, 4, 512, 1>(a, st);
     return -13;
