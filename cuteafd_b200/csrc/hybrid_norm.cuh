@@ -26,9 +26,9 @@ struct NormArgs {
   const float* slot_w;        // [T, top_k]
   const int* slot_idx;        // [T, top_k]; an index >= n_experts is an identity slot
   const void* ident;          // [T, ldh] E: what identity slots hand through
-  const float* w_b;           // [H]
-  const float* w;             // [H]
-  const float* conv;          // [taps, H], null = no convolution
+  const void* w_b;            // [H] E
+  const void* w;              // [H] E
+  const void* conv;           // [taps, H] E, null = no convolution
   float* x_out;               // [T, H] or null
   void* h_out;                // [rows, ldh] E
   const int* row_idx;         // rows to compute (null = all, in order); only without a convolution
@@ -177,14 +177,14 @@ __global__ void __launch_bounds__(kMaxThreads, kMinBlocks) norm_conv_kernel(cons
   if (kMinBlocks == 1 && a.run == 1) {
     // decode: the weights (and, when a block is a sequence, its state) are on their way into L2 while the previous
     // kernel drains; nothing is read here
-    auto pull = [](const float* q) { asm volatile("prefetch.global.L2 [%0];" ::"l"(q)); };
+    auto pull = [](const void* q) { asm volatile("prefetch.global.L2 [%0];" ::"l"(q)); };
     const bool own_seq = a.conv && a.S == a.T && a.state;
     const float* st = own_seq ? a.state + static_cast<size_t>(a.state_in[blockIdx.x]) * a.slot_stride + a.state_off : nullptr;
     for (int i = tid * 32; i < a.H; i += nt * 32) {         // one 128-byte line per step
-      pull(a.w + i);
-      if (a.w_b) pull(a.w_b + i);
+      pull(static_cast<const E*>(a.w) + i);
+      if (a.w_b) pull(static_cast<const E*>(a.w_b) + i);
       if (a.conv)
-        for (int j = 0; j < a.taps; ++j) pull(a.conv + static_cast<size_t>(j) * a.H + i);
+        for (int j = 0; j < a.taps; ++j) pull(static_cast<const E*>(a.conv) + static_cast<size_t>(j) * a.H + i);
       if (st)
         for (int j = 0; j + 1 < a.taps; ++j) pull(st + static_cast<size_t>(j) * a.H + i);
     }
@@ -197,6 +197,7 @@ __global__ void __launch_bounds__(kMaxThreads, kMinBlocks) norm_conv_kernel(cons
   const int r1 = min(a.T, r0 + a.run);
   if (r0 >= a.T) return;
   const int halo = a.conv ? a.taps - 1 : 0;
+  const E* conv_w = static_cast<const E*>(a.conv);
   const float inv_n = 1.0f / static_cast<float>(gvec * V);
   int grp[KV];
 #pragma unroll
@@ -327,7 +328,17 @@ __global__ void __launch_bounds__(kMaxThreads, kMinBlocks) norm_conv_kernel(cons
         }
       }
     }
-    if (t + 1 < r1) fetch(t + 1);
+    if (t + 1 < r1) {
+      fetch(t + 1);
+      if constexpr (kSlots && kMinBlocks > 1) {               // the next token's routed rows on their way into L2
+        const int lines = (a.H * static_cast<int>(sizeof(E)) + 127) / 128;
+        for (int l = tid; l < a.top_k * lines; l += nt) {
+          const int s = l / lines, nrow = (t + 1) * a.top_k + s;
+          if (a.slot_idx[nrow] < a.n_experts)
+            asm volatile("prefetch.global.L2 [%0];" ::"l"(reinterpret_cast<const uint8_t*>(static_cast<const E*>(a.y) + static_cast<size_t>(nrow) * a.ldy) + (l - s * lines) * 128));
+        }
+      }
+    }
     if (a.y) {
       float inv[KV];
       group_inv<V, KV, sizeof(E) == 4>(y, inv, sm + flip * stride, sm + flip * stride + nvec, nvec, gvec, grp, inv_n, fast, a.eps);
@@ -337,7 +348,7 @@ __global__ void __launch_bounds__(kMaxThreads, kMinBlocks) norm_conv_kernel(cons
         const int i = tid + k * nt;
         if (i < nvec) {
           float wb[V];
-          load_vec<float, V>(a.w_b + i * V, wb);
+          load_vec<E, V>(static_cast<const E*>(a.w_b) + i * V, wb);
 #pragma unroll
           for (int e = 0; e < V; ++e) x[k][e] += y[k][e] * inv[k] * wb[e];
         }
@@ -358,7 +369,7 @@ __global__ void __launch_bounds__(kMaxThreads, kMinBlocks) norm_conv_kernel(cons
       const int i = tid + k * nt;
       if (i < nvec) {
         float wn[V];
-        load_vec<float, V>(a.w + i * V, wn);
+        load_vec<E, V>(static_cast<const E*>(a.w) + i * V, wn);
 #pragma unroll
         for (int e = 0; e < V; ++e) x[k][e] = x[k][e] * inv[k] * wn[e];
       }
@@ -373,7 +384,7 @@ __global__ void __launch_bounds__(kMaxThreads, kMinBlocks) norm_conv_kernel(cons
           for (int e = 0; e < V; ++e) o[e] = x[k][e];
           if (a.conv) {
             float c[V];
-            load_vec<float, V>(a.conv + static_cast<size_t>(a.taps - 1) * a.H + i * V, c);
+            load_vec<E, V>(conv_w + static_cast<size_t>(a.taps - 1) * a.H + i * V, c);
             float acc[V];
 #pragma unroll
             for (int e = 0; e < V; ++e) acc[e] = c[e] * x[k][e];
@@ -381,7 +392,7 @@ __global__ void __launch_bounds__(kMaxThreads, kMinBlocks) norm_conv_kernel(cons
             for (int j = 0; j < MAXT - 1; ++j) {
               const int tap = j - (MAXT - 1 - halo);
               if (tap >= 0) {
-                load_vec<float, V>(a.conv + static_cast<size_t>(tap) * a.H + i * V, c);
+                load_vec<E, V>(conv_w + static_cast<size_t>(tap) * a.H + i * V, c);
 #pragma unroll
                 for (int e = 0; e < V; ++e) acc[e] += c[e] * win[j][k][e];
               }

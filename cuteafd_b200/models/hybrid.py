@@ -91,12 +91,12 @@ class HybridWeights:
             return out.view(Hp, heads * pad8(vdim))
 
         W = HybridWeights(cfg)
-        W.embed, W.final_norm, W.lm_head = t("embed", (cfg.vocab_size, H)), f("final.norm"), reads(t("head", (cfg.vocab_size, H)))
+        W.embed, W.final_norm, W.lm_head = t("embed", (cfg.vocab_size, H)), t("final.norm", (H,)), reads(t("head", (cfg.vocab_size, H)))
         for i, spec in enumerate(cfg.layer_specs):
             pre, m, r, L = f"l{i}.", spec.mixer, spec.router, HybridLayer()
             x = pre + "mix."
-            L.norm1, L.norm1b = f(pre + "norm1"), f(pre + "norm1b")
-            L.canon1 = f(pre + "canon1").T.contiguous()
+            L.norm1, L.norm1b = t(pre + "norm1", (H,)), t(pre + "norm1b", (H,))
+            L.canon1 = t(pre + "canon1", (H, cfg.canon_taps)).T.contiguous()
             if isinstance(m, LatentSpec):
                 L.w_in, L.offs = fuse([("q", t(x + "q", (m.heads * (m.dim + m.rot_dim), H))), ("kv", t(x + "dkv", (m.record, H))),
                                        ("g", t(x + "g", (m.heads * m.vdim, H)))])
@@ -119,8 +119,8 @@ class HybridWeights:
             L.w_o = heads_o(x + "o", m.heads, m.vdim)
             if r is not None:
                 y = pre + "mlp."
-                L.norm2, L.norm2b = f(pre + "norm2"), f(pre + "norm2b")
-                L.canon2 = f(pre + "canon2").T.contiguous()
+                L.norm2, L.norm2b = t(pre + "norm2", (H,)), t(pre + "norm2b", (H,))
+                L.canon2 = t(pre + "canon2", (H, cfg.canon_taps)).T.contiguous()
                 L.router, L.correction = reads(t(y + "router", (r.outputs, H))), f(y + "correction")
                 F = pad8(r.ffn)
                 L.w_gate, L.w_up = (torch.zeros(r.experts, F, Hp, dtype=dt, device=device) for _ in range(2))

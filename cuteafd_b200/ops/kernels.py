@@ -675,11 +675,11 @@ def norm_conv(h_out: torch.Tensor, w: torch.Tensor, groups: int, eps: float, *, 
               x_out: torch.Tensor | None = None, rows: torch.Tensor | None = None, state: torch.Tensor | None = None, state_off: int = 0,
               state_in: torch.Tensor | None = None, state_out: torch.Tensor | None = None, q_start: torch.Tensor | None = None,
               run: int = 0) -> None:
-    """x = embed[tokens] or ``x_in`` (fp32); x += groupnorm(y) * w_b; h = groupnorm(x) * w; h_out = h + causal_conv(h).
+    """Weights are in the activations' type.  x = embed[tokens] or ``x_in`` (fp32); x += groupnorm(y) * w_b; h = groupnorm(x) * w; h_out = h + causal_conv(h).
 
     Rows of ``h_out``, ``y`` and the identity rows may be longer than H (whole 16-byte pieces); the rest is left alone.
     ``slots`` = (weights [T, k], ids [T, k], number of experts, identity rows): ``y`` then holds the routed experts' rows
-    [T * k, ...] and is their weighted sum.  ``conv`` [taps, H] fp32 (last row = current token) with the sequences'
+    [T * k, ...] and is their weighted sum.  ``conv`` [taps, H] (last row = current token) with the sequences'
     earlier inputs in ``state`` [slots, floats] at ``state_off``.  ``rows``: compute only these rows (no convolution)."""
     a = _n.NormArgs()
     H = w.shape[0]
@@ -688,7 +688,7 @@ def norm_conv(h_out: torch.Tensor, w: torch.Tensor, groups: int, eps: float, *, 
     a.vocab = embed.shape[0] if embed is not None else 0
     a.T, a.H, a.groups, a.eps, a.run = h_out.shape[0], H, groups, eps, run
     a.ldy, a.ldh = y.stride(0) if y is not None else 0, h_out.stride(0)
-    assert h_out.shape[1] >= H and h_out.stride(1) == 1 and w.dtype == torch.float32
+    assert h_out.shape[1] >= H and h_out.stride(1) == 1 and w.dtype == h_out.dtype and (w_b is None or w_b.dtype == h_out.dtype)
     if slots is not None:
         sw, si, n, ident = slots
         a.slot_w, a.slot_idx, a.n_experts, a.ident, a.top_k = sw.data_ptr(), si.data_ptr(), n, ident.data_ptr(), sw.shape[1]
@@ -697,7 +697,7 @@ def norm_conv(h_out: torch.Tensor, w: torch.Tensor, groups: int, eps: float, *, 
         a.taps, a.S = conv.shape[0], q_start.shape[0] - 1
         a.state, a.state_in, a.state_out, a.q_start = state.data_ptr(), state_in.data_ptr(), state_out.data_ptr(), q_start.data_ptr()
         a.slot_stride, a.state_off = state.stride(0), state_off
-        assert conv.is_contiguous() and conv.dtype == torch.float32 and state.dtype == torch.float32
+        assert conv.is_contiguous() and conv.dtype == h_out.dtype and state.dtype == torch.float32
     _n.check(_n.cuda_lib().cafd_norm_conv(C.byref(a), int(h_out.dtype == torch.float32), _stream()), "norm_conv")
 
 

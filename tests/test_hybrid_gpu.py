@@ -46,7 +46,7 @@ def test_norm_conv(dtype, H, groups, taps):
     lens = [[40, 1, 2, 19], [1, 33, 2, 1]]                    # two steps of four sequences
     T = [sum(x) for x in lens]
     emb = rnd(V, H, seed=1, dtype=dtype)
-    w, wb, c = 1 + rnd(H, seed=2, scale=0.2), 1 + rnd(H, seed=3, scale=0.2), rnd(H, taps, seed=4, scale=0.4)
+    w, wb, c = (x.to(dtype).float() for x in (1 + rnd(H, seed=2, scale=0.2), 1 + rnd(H, seed=3, scale=0.2), rnd(H, taps, seed=4, scale=0.4)))
     toks = [tokens(n, V, 5 + i) for i, n in enumerate(T)]
     ys = [rnd(n, H, seed=7 + i, dtype=dtype) for i, n in enumerate(T)]
     second = 32 + -(-(taps - 1) * H // 32) * 32
@@ -55,7 +55,8 @@ def test_norm_conv(dtype, H, groups, taps):
     ins, outs = [0, 0, 0, 0], [3, 5, 2, 9]
     past = [torch.zeros(taps - 1, H) for _ in range(4)]
     past_y = [torch.zeros(taps - 1, H) for _ in range(4)]
-    cd = c.T.contiguous().to(dev())
+    cd = c.T.contiguous().to(dev(), dtype)
+    wd, wbd = w.to(dev(), dtype), wb.to(dev(), dtype)
     for step in range(2):
         qs, n = [0], T[step]
         for x in lens[step]:
@@ -64,7 +65,7 @@ def test_norm_conv(dtype, H, groups, taps):
         h, x0 = hp[:, :H], torch.empty(n, H, device=dev())
         ypad = torch.nn.functional.pad(ys[step], (0, hp.shape[1] - H)).to(dev(), dtype)
         kw = dict(state=state, state_in=i32(ins), state_out=i32(outs), q_start=i32(qs), conv=cd)
-        K.norm_conv(h, w.to(dev()), groups, eps, tokens=i32(toks[step]), embed=emb.to(dev(), dtype), x_out=x0, state_off=32, **kw)
+        K.norm_conv(h, wd, groups, eps, tokens=i32(toks[step]), embed=emb.to(dev(), dtype), x_out=x0, state_off=32, **kw)
         x = emb[torch.tensor(toks[step])]
         assert torch.equal(x0.cpu(), x)
         for s in range(4):
@@ -74,7 +75,7 @@ def test_norm_conv(dtype, H, groups, taps):
             if taps > 1:
                 assert torch.allclose(state[outs[s], 32:32 + (taps - 1) * H].view(taps - 1, H).cpu(), past[s], atol=2e-5)
         x1 = torch.empty_like(x0)
-        K.norm_conv(h, w.to(dev()), groups, eps, x_in=x0, y=ypad, w_b=wb.to(dev()), x_out=x1, state_off=second, run=7, **kw)
+        K.norm_conv(h, wd, groups, eps, x_in=x0, y=ypad, w_b=wbd, x_out=x1, state_off=second, run=7, **kw)
         x = x + R.group_rms(ys[step], wb, groups, eps)
         close(x1, x, torch.float32)
         for s in range(4):
@@ -84,20 +85,21 @@ def test_norm_conv(dtype, H, groups, taps):
         rows = [n - 1, 0, n // 2]
         assert (hp[:, H:] == 9.0).all()
         hf = torch.empty(3, hp.shape[1], dtype=dtype, device=dev())[:, :H]
-        K.norm_conv(hf, w.to(dev()), groups, eps, x_in=x0, y=ypad, w_b=wb.to(dev()), rows=i32(rows))
+        K.norm_conv(hf, wd, groups, eps, x_in=x0, y=ypad, w_b=wbd, rows=i32(rows))
         close(hf, R.group_rms(x[rows], w, groups, eps), dtype)
         ins, outs = outs, [1, 6, 7, 10] if step == 0 else outs
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
-def test_norm_conv_sums_routed_rows_and_identity_slots(dtype):
+@pytest.mark.parametrize("T,k,H", [(37, 3, 72), (600, 6, 256), (300, 9, 2560), (5, 12, 4096)])
+def test_norm_conv_sums_routed_rows_and_identity_slots(dtype, T, k, H):
     from cuteafd_b200.ops import kernels as K
-    T, k, H, E = 37, 3, 72, 4
+    E = 4
     y, ident, x = rnd(T * k, H, seed=1, dtype=dtype), rnd(T, H, seed=2, dtype=dtype), rnd(T, H, seed=3)
     idx = torch.randint(0, E + 2, (T, k), generator=torch.Generator().manual_seed(4))
-    wts, wb, w = rnd(T, k, seed=5).abs(), 1 + rnd(H, seed=6, scale=0.2), 1 + rnd(H, seed=7, scale=0.2)
+    wts, wb, w = rnd(T, k, seed=5).abs(), (1 + rnd(H, seed=6, scale=0.2)).to(dtype).float(), (1 + rnd(H, seed=7, scale=0.2)).to(dtype).float()
     h, xo = torch.empty(T, H, dtype=dtype, device=dev()), torch.empty(T, H, device=dev())
-    K.norm_conv(h, w.to(dev()), 2, 1e-5, x_in=x.to(dev()), y=y.to(dev(), dtype), w_b=wb.to(dev()), x_out=xo,
+    K.norm_conv(h, w.to(dev(), dtype), 2, 1e-5, x_in=x.to(dev()), y=y.to(dev(), dtype), w_b=wb.to(dev(), dtype), x_out=xo,
                 slots=(wts.to(dev()), i32(idx.tolist()), E, ident.to(dev(), dtype)))
     rows = torch.where((idx >= E)[..., None], ident[:, None], y.view(T, k, H))
     want = x + R.group_rms((wts[..., None] * rows).sum(1), wb, 2, 1e-5)
