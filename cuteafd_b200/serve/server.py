@@ -509,6 +509,9 @@ def build_state(args) -> ServerState:
         rows = args.concurrency * 8
         world = int(os.environ.get("WORLD_SIZE", "1"))
         if world > 1:
+            from ..loader.snapshot import read_config
+            if (read_config(snapshot)[0] if snapshot else PRESETS[args.preset or "qwen3-30b-a3b"]()).is_hybrid:
+                raise SystemExit("per-layer hybrids are not split over GPUs: serve them from one process")
             # Disaggregated deployment (launched with one process per GPU): rank 0 runs attention, the dense backbone
             # and this HTTP server; the other ranks hold the routed experts and serve announced steps until rank 0
             # stops them.  The attention engine plugs into the same backend as the single-GPU engine.

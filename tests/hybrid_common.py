@@ -75,3 +75,17 @@ def err(got, want):
     d = got.float() - want.float()
     d, w = d - d.mean(-1, keepdim=True), want - want.mean(-1, keepdim=True)
     return d.pow(2).mean(-1).sqrt() / w.pow(2).mean().sqrt()
+
+
+def write_model(cfg, p, directory):
+    """config.json and model.safetensors (bfloat16) of ``cfg`` with parameters ``p``; returns the path."""
+    import json
+    import os
+
+    from cuteafd_b200.loader.safetensors_io import write_file
+    from cuteafd_b200.loader.snapshot import to_hf_config
+    os.makedirs(directory, exist_ok=True)
+    with open(os.path.join(directory, "config.json"), "w") as f:
+        json.dump(to_hf_config(cfg), f)
+    write_file(os.path.join(directory, "model.safetensors"), {k: v.to(torch.bfloat16) for k, v in p.items()})
+    return str(directory)

@@ -212,5 +212,19 @@ def test_scheduler_generates_like_the_oracle(draft):
     assert got["tokens"] == _greedy(cfg, p, again, 6) and got["usage"]["cached_tokens"] in (70, 81)
 
 
+def test_serve_builds_over_a_snapshot(tmp_path):
+    from cuteafd_b200.cli import build_parser
+    from cuteafd_b200.runtime.scheduler import Request, collect
+    from cuteafd_b200.serve.server import build_state
+    cfg = odd_config().replace(vocab_size=271)            # the byte tokenizer takes 260
+    path = write_random_snapshot(cfg, str(tmp_path / "m"), seed=3)
+    st = build_state(build_parser().parse_args(["serve", "--fake-engine", "--snapshot", path, "--speculator", "off"]))
+    r = st.sched.submit(Request([5, 6, 7], max_tokens=4))
+    for _ in range(20):
+        st.sched.step()
+    _, p = load_params(path)
+    assert collect(r, 1.0)["tokens"] == _greedy(cfg, p, [5, 6, 7], 4)
+
+
 def test_delta_channels():
     assert DeltaSpec(6, 2, 20, 36, 3).conv_channels == 2 * 40 + 216

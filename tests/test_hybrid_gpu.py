@@ -10,7 +10,7 @@ import torch
 from cuteafd_b200.config import RouterSpec
 from cuteafd_b200.ref import hybrid as R
 
-from tests.hybrid_common import delta, err, latent, narrow_config, odd_config, oracle_logits, params, plain_config, tokens, wide_config
+from tests.hybrid_common import delta, err, latent, narrow_config, odd_config, oracle_logits, params, plain_config, tokens, wide_config, write_model
 
 pytestmark = pytest.mark.gpu
 DTYPES = [torch.float32, torch.bfloat16]
@@ -181,6 +181,36 @@ def test_latent_attention_windows(dtype, m, edge):
             K.mla_attention(qp, cache, table, i32(lens), i32(q_start), i32(bs), i32(bt), out, m.scale, splits, sc, out_tpad=t_pad, window=m.window)
             close(out[:, :T].transpose(0, 1), want, dtype)
         assert K.read_status() == 0
+
+
+@pytest.mark.parametrize("edge", [0, 1, 2])
+@pytest.mark.parametrize("window", [1, 64, 100, 129, 1000])
+def test_expanded_prompt_attention_windows(window, edge):
+    """The expanded form (per-head keys and values of the whole prompt, shared rotated part from the cache) under a
+    sliding window, one key outscoring the rest just inside, just outside or in the page before."""
+    from cuteafd_b200.ops import kernels as K
+    n, heads, scale = 330, 4, 192 ** -0.5 * 1.5
+    q, k, v = rnd(n, heads, 192, seed=1, scale=0.2), rnd(n, heads, 192, seed=2), rnd(n, heads, 128, seed=3)
+    k[..., 128:] = k[:, :1, 128:]                                    # all heads share the rotated part
+    for t in range(n):
+        at = t // 64 * 64 - 1 if edge == 2 else t - window + (1 if edge == 0 else 0)
+        if at >= 0:
+            q[t] += 0.7 * k[at]
+    q, k, v = (x.to(torch.bfloat16).float() for x in (q, k, v))
+    lat = torch.zeros(n, 576)
+    lat[:, 512:] = k[:, 0, 128:]
+    cache, table = _paged([lat], [n], 576, torch.bfloat16)
+    rows = -(-n // 64) * 64
+    kx, vx = (torch.zeros(rows, heads * 128, dtype=torch.bfloat16, device=dev()) for _ in range(2))
+    kx[:n], vx[:n] = k[..., :128].reshape(n, -1), v.reshape(n, -1)
+    qa = torch.zeros(n, heads, 576, dtype=torch.bfloat16, device=dev())
+    qa[..., 512:] = q[..., 128:]
+    wide = torch.zeros(n, heads * 192 + 40, dtype=torch.bfloat16, device=dev())      # query columns inside longer rows
+    wide[:, 8:8 + heads * 192] = q.reshape(n, -1)
+    out = torch.zeros(n, heads, 128, dtype=torch.bfloat16, device=dev())
+    K.attn_prefill_mla(wide[:, 8:8 + heads * 192], qa, kx, vx, i32([0]), cache, table, i32([n]), i32([0, n]), out, n, heads, scale, window=window)
+    close(out, R.window_attention(q, k, v, 0, window, scale), torch.bfloat16)
+    assert K.read_status() == 0
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
@@ -544,17 +574,39 @@ def test_generator_matches_the_backend_under_graphs():
     assert out == truth
 
 
+def test_serve_builds_over_a_snapshot(tmp_path):
+    """``serve --snapshot``: loading, page and slot pools, scheduler with the n-gram drafter, decode graphs, sampling."""
+    from cuteafd_b200.cli import build_parser
+    from cuteafd_b200.runtime.sampling import SamplingParams
+    from cuteafd_b200.runtime.scheduler import Request, collect
+    from cuteafd_b200.serve.server import build_state
+    cfg = odd_config().replace(vocab_size=271)            # the byte tokenizer takes 260
+    p = params(cfg, 3, spread=2.0)
+    path = write_model(cfg, p, str(tmp_path / "m"))
+    st = build_state(build_parser().parse_args(["serve", "--snapshot", path, "--max-context-tokens", "512", "--concurrency", "3",
+                                                "--speculator", "ngram"]))
+    st.sched.eos_ids = ()
+    assert type(st.sched.be.engine).__name__ == "HybridEngine" and st.sched.be.tier is None
+    prompt = (tokens(9, cfg.vocab_size, 3) * 12)[:100]
+    greedy = [st.sched.submit(Request(list(prompt[i:]), max_tokens=24)) for i in range(3)]
+    drawn = [st.sched.submit(Request(list(prompt), max_tokens=24, params=SamplingParams(temperature=1.0, seed=7))) for _ in range(2)]
+    while st.sched.step():
+        pass
+    for i, r in enumerate(greedy):
+        got = collect(r, 1.0)["tokens"]
+        want = oracle_logits(cfg, p, prompt[i:] + got)[len(prompt) - i - 1:-1]
+        best = want.max(-1).values
+        assert len(got) == 24 and (best - want[torch.arange(24), got] < 0.05 * best.abs()).all()    # bf16: a near tie may go either way
+    a, b = (collect(r, 1.0)["tokens"] for r in drawn)
+    assert len(a) == 24 and a[0] == b[0]
+
+
 @pytest.mark.parametrize("dtype", ["bfloat16", "float32"])
 def test_trace_replay_program(dtype, tmp_path):
     import os
-    from cuteafd_b200.loader.snapshot import to_hf_config
-    from cuteafd_b200.loader.safetensors_io import write_file
     cfg = odd_config()
     p = params(cfg, spread=2.0)
-    d = tmp_path / "m"
-    d.mkdir()
-    (d / "config.json").write_text(json.dumps(to_hf_config(cfg)))
-    write_file(str(d / "model.safetensors"), {k: v.to(torch.bfloat16) for k, v in p.items()})
+    d = write_model(cfg, p, str(tmp_path / "m"))
     a, b = tokens(120, cfg.vocab_size, 1), tokens(30, cfg.vocab_size, 2)
     steps = [{"entries": [{"id": "a", "tokens": a[:50], "want": [49, 0]}, {"id": "b", "tokens": b[:2], "want": []}], "end": []},
              {"entries": [{"id": "a", "tokens": a[50:51], "want": []}], "end": []},
@@ -562,7 +614,7 @@ def test_trace_replay_program(dtype, tmp_path):
              {"entries": [{"id": "c", "tokens": a, "want": [119]}], "end": ["c"]}]
     text = "".join(json.dumps(dict(s, step=i)) + "\n" for i, s in enumerate(steps))
     root = os.path.dirname(os.path.dirname(os.path.abspath(__file__)))
-    r = subprocess.run([os.path.join(root, "bin", "trace_run"), "--model", str(d), "--dtype", dtype, "--out", str(tmp_path), "--max-tokens", "192"],
+    r = subprocess.run([os.path.join(root, "bin", "trace_run"), "--model", d, "--dtype", dtype, "--out", str(tmp_path), "--max-tokens", "192"],
                        input=text, capture_output=True, text=True, timeout=200)
     assert r.returncode == 0, r.stderr[-2000:]
     assert [x for x in r.stdout.splitlines() if x.startswith("done")] == [f"done {i}" for i in range(4)]
