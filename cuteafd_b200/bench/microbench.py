@@ -5,6 +5,7 @@
     python -m cuteafd_b200.bench.microbench attn-decode --seqs 32 --len 8192
     python -m cuteafd_b200.bench.microbench mla --seqs 8 --len 8192 --qlen 1 --heads 128 [--topk 2048]
     python -m cuteafd_b200.bench.microbench w4 --tokens 8 --features 7168 --k 2048 --fmt nvfp4
+    python -m cuteafd_b200.bench.microbench hybrid --size base
     python -m cuteafd_b200.bench.microbench sampler --rows 32 --vocab 151936
     python -m cuteafd_b200.bench.microbench moe --tokens 1,16,128,1024,8192 --hidden 7168 --ffn 2048 \
         --experts 256 --top-k 8 --scoring sigmoid
@@ -331,6 +332,49 @@ def bench_sampler(a, dev, pk):
     report(f"sample_rows rows={n} V={V} top_k={a.top_k} top_p={a.top_p}", ms, 0.0, n * V * 4.0, pk)
 
 
+def bench_hybrid(a, dev, pk) -> None:
+    """The per-layer hybrids' own kernels beside the like kernels of the MLA decoder, at one of the benchmark sizes."""
+    from ..config import KARUSUN_SIZES, DeltaSpec, LayerSpec, hybrid_config
+    from ..models.hybrid import HybridCache, HybridWeights
+    H, _, heads, _ = KARUSUN_SIZES[a.size]
+    bf, T, k = torch.bfloat16, a.tokens, 6
+
+    def i32(v):
+        return torch.tensor(list(v), dtype=torch.int32, device=dev)
+
+    def run(name, fn, nbytes, flops=0.0):
+        report(name, time_eager(fn, dev, a.iters), flops, nbytes, pk)
+    for n in (8, T):
+        S = n if n == 8 else 1
+        x, xo, y, h = torch.randn(n, H, device=dev), torch.empty(n, H, device=dev), torch.randn(n, H, device=dev, dtype=bf), torch.empty(n, H, device=dev, dtype=bf)
+        w, c, st = torch.ones(H, device=dev, dtype=bf), (torch.randn(4, H, device=dev) * 0.1).to(bf), torch.zeros(2 + 2 * S, 3 * H, device=dev)
+        kw = dict(x_in=x, w_b=w, x_out=xo, conv=c, state=st, state_in=i32(range(2, 2 + S)), state_out=i32(range(2 + S, 2 + 2 * S)),
+                  q_start=i32(range(S + 1) if S > 1 else (0, n)))
+        ys, idx = torch.randn(n * k, H, device=dev, dtype=bf), torch.randint(0, 64, (n, k), device=dev, dtype=torch.int32)
+        sw = torch.rand(n, k, device=dev)
+        own = S * 6 * H * 4 if S > 1 else 0
+        run(f"norm_conv {n} rows", lambda: K.norm_conv(h, w, 4, 1e-5, y=y, **kw), n * H * 12 + own)
+        run(f"norm_conv {n} rows, top-{k} routed sum", lambda: K.norm_conv(h, w, 4, 1e-5, y=ys, slots=(sw, idx, 56, y), **kw), n * H * (10 + 2 * k) + own)
+        run(f"(MLA) rmsnorm {n} rows", lambda: K.rmsnorm(y, w, 1e-5, out=h), n * H * 4)
+        run(f"(MLA) combine + norm {n} rows", lambda: K.moe_combine(ys, sw, h, residual=y, norm_w=w, eps=1e-5, x_out=ys[:n]), n * H * (6 + 2 * k))
+    m = DeltaSpec(heads, heads // 2, 128, 128, 4)
+    cfg = hybrid_config("bench", 128, H, [LayerSpec(m)], 4, 4, 1e-5)
+    L = HybridWeights.random_init(cfg, dev).layers[0]
+    n_in = L.w_in.shape[0]
+    for B in (1, 8, 32):
+        kv = HybridCache(cfg, 4, dev, 2 + 2 * B)
+        p, out = torch.randn(B, n_in, device=dev, dtype=bf), torch.empty(B, heads, 128, device=dev, dtype=bf)
+        args = (p, L.offs, m, L, kv.state, kv.offsets[0]["S"], kv.offsets[0]["conv"], i32(range(2, 2 + B)), i32(range(2 + B, 2 + 2 * B)), i32(range(B + 1)))
+        run(f"delta_step {B} sequences x {heads} heads", lambda: K.delta_step(*args, out, None, 1e-5), B * heads * 128 * 128 * 8)
+    kv = HybridCache(cfg, 4, dev, 4)
+    p, out, raw = torch.randn(T, n_in, device=dev, dtype=bf), torch.empty(T, heads, 128, device=dev, dtype=bf), torch.empty(T * heads * 128, device=dev)
+    scratch = torch.empty(128 << 20, dtype=torch.uint8, device=dev)
+    args = (p, L.offs, m, L, kv.state, kv.offsets[0]["S"], kv.offsets[0]["conv"], i32([0]), i32([2]), i32([0, T]))
+    macs = T / 64 * heads * 64 * (64 * 128 * 5 + 128 * 128 * 3)
+    run(f"delta_chunked {T} tokens x {heads} heads", lambda: K.delta_chunked(scratch, *args, out, raw, 1e-5), T * n_in * 2 + T * heads * 256, 2 * macs)
+    run(f"latent_gate {T} rows", lambda: K.latent_gate(out, p, 0, heads, 128), T * heads * 128 * 6)
+
+
 def main() -> None:
     ap = argparse.ArgumentParser()
     sub = ap.add_subparsers(dest="cmd", required=True)
@@ -370,14 +414,16 @@ def main() -> None:
     sm = sub.add_parser("sampler")
     sm.add_argument("--rows", type=int, default=32); sm.add_argument("--vocab", type=int, default=151936)
     sm.add_argument("--top-k", type=int, default=50); sm.add_argument("--top-p", type=float, default=0.9)
-    for s in (g, p, d, m, ml, mp_, w4, sm):
+    hy = sub.add_parser("hybrid")
+    hy.add_argument("--size", default="base", choices=["small", "base", "large"]); hy.add_argument("--tokens", type=int, default=8192)
+    for s in (g, p, d, m, ml, mp_, w4, sm, hy):
         s.add_argument("--iters", type=int, default=10)
     a = ap.parse_args()
     dev = torch.device("cuda", int(os.environ.get("LOCAL_RANK", "0")))
     torch.cuda.set_device(dev)
     pk = peaks()
     {"exl3": bench_exl3, "gemm-fp8": bench_gemm_fp8, "indexer": bench_indexer, "gemm": bench_gemm, "attn-prefill": bench_attn_prefill, "attn-decode": bench_attn_decode, "moe": bench_moe,
-     "mla": bench_mla, "mla-prefill": bench_mla_prefill_expanded, "w4": bench_w4, "sampler": bench_sampler}[a.cmd](a, dev, pk)
+     "mla": bench_mla, "mla-prefill": bench_mla_prefill_expanded, "w4": bench_w4, "sampler": bench_sampler, "hybrid": bench_hybrid}[a.cmd](a, dev, pk)
 
 
 if __name__ == "__main__":

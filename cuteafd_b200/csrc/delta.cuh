@@ -46,8 +46,9 @@ __device__ __forceinline__ void de_store4(__nv_bfloat16* p, const float (&v)[4])
   *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16(v[0], v[1]), pack_bf16(v[2], v[3]));
 }
 
-// out[t, h] = raw[t, h] / rms(raw[t, h]) * norm_w * silu(gate): one warp per (token, head), two in flight where a head
-// is at most 128 columns of whole 16-byte pieces
+// out[t, h] = raw[t, h] / rms(raw[t, h]) * norm_w * silu(gate): one warp per (token, head), several in flight where a head
+// is at most 128 columns of whole pieces of four
+constexpr int kOutRows = 4;
 template <typename E>
 __global__ void __launch_bounds__(256) delta_out_kernel(const DeltaArgs p) {
   pdl_wait();
@@ -55,32 +56,32 @@ __global__ void __launch_bounds__(256) delta_out_kernel(const DeltaArgs p) {
   const long long n = static_cast<long long>(p.T) * p.heads, stride = static_cast<long long>(gridDim.x) * 8;
   const int lane = threadIdx.x & 31;
   long long i = static_cast<long long>(blockIdx.x) * 8 + (threadIdx.x >> 5);
-  if (p.vdim <= 128 && p.vdim % 4 == 0 && p.out_vd % 4 == 0 && p.ld % 4 == 0 && p.g_off % 4 == 0) {
+  if (n < (1ll << 30) && p.vdim <= 128 && p.vdim % 4 == 0 && p.out_vd % 4 == 0 && p.ld % 4 == 0 && p.g_off % 4 == 0) {
     const bool on = 4 * lane < p.vdim;
     float nw[4] = {};
     if (on) de_load4(p.norm_w + 4 * lane, nw);
-    for (; i < n; i += 2 * stride) {
-      float o[2][4] = {}, g[2][4] = {};
+    const uint32_t rows = static_cast<uint32_t>(n), step = static_cast<uint32_t>(stride), heads = static_cast<uint32_t>(p.heads);
+    for (uint32_t r0 = static_cast<uint32_t>(i); r0 < rows; r0 += kOutRows * step) {
+      float o[kOutRows][4] = {}, g[kOutRows][4] = {};
 #pragma unroll
-      for (int j = 0; j < 2; ++j) {
-        const long long r = i + j * stride;
-        if (r < n && on) {
-          const long long t = r / p.heads;
-          const int h = static_cast<int>(r - t * p.heads);
-          de_load4(p.raw + r * p.vdim + 4 * lane, o[j]);
-          de_load4(static_cast<const E*>(p.proj) + t * p.ld + p.g_off + h * p.vdim + 4 * lane, g[j]);
+      for (int j = 0; j < kOutRows; ++j) {
+        const uint32_t r = r0 + j * step;
+        if (r < rows && on) {
+          const uint32_t t = r / heads, h = r - t * heads;
+          de_load4(p.raw + static_cast<size_t>(r) * p.vdim + 4 * lane, o[j]);
+          de_load4(static_cast<const E*>(p.proj) + static_cast<size_t>(t) * p.ld + p.g_off + h * p.vdim + 4 * lane, g[j]);
         }
       }
 #pragma unroll
-      for (int j = 0; j < 2; ++j) {
-        const long long r = i + j * stride;
+      for (int j = 0; j < kOutRows; ++j) {
+        const uint32_t r = r0 + j * step;
         const float ss = warp_sum(o[j][0] * o[j][0] + o[j][1] * o[j][1] + o[j][2] * o[j][2] + o[j][3] * o[j][3]);
         const float inv = 1.0f / sqrtf(ss / static_cast<float>(p.vdim) + p.eps);
-        if (r < n && on) {
+        if (r < rows && on) {
           float v[4];
 #pragma unroll
-          for (int e = 0; e < 4; ++e) v[e] = o[j][e] * inv * nw[e] * g[j][e] * sigmoid_f(g[j][e]);
-          de_store4(static_cast<E*>(p.out) + r * p.out_vd + 4 * lane, v);
+          for (int e = 0; e < 4; ++e) v[e] = o[j][e] * inv * nw[e] * g[j][e] / (1.0f + __expf(fminf(-g[j][e], 80.f)));
+          de_store4(static_cast<E*>(p.out) + static_cast<size_t>(r) * p.out_vd + 4 * lane, v);
         }
       }
     }
