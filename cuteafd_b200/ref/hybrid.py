@@ -49,8 +49,8 @@ def rotate_half(x: torch.Tensor, positions: torch.Tensor, base: float) -> torch.
 
 
 def window_attention(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, start: int, window: int, scale: float) -> torch.Tensor:
-    """Softmax attention; q [T, H, Dk] at positions start.., k [L, H, Dk], v [L, H, Dv] at positions 0..; a query at
-    position i sees j with 0 <= i - j < window."""
+    """Softmax attention of q [T, H, Dk] (positions start, start + 1, ...) over k [L, H, Dk], v [L, H, Dv] (positions 0, 1, ...);
+    the query at position i reads keys i - window + 1 .. i."""
     out = []
     for t in range(q.shape[0]):
         i = start + t
