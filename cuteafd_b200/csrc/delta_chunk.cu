@@ -55,6 +55,17 @@ __device__ __forceinline__ void mma16816(float (&c)[4], const uint32_t (&a)[4], 
                : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
                : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
 }
+// Four neighbouring n tiles of a split product: hi hi, hi lo and lo hi over all four in turn, so that no product waits for
+// the one before it.
+__device__ __forceinline__ void mma_split4(float (*c)[4], const uint32_t (&ah)[4], const uint32_t (&al)[4], const uint32_t (&bh)[2][4],
+                                           const uint32_t (&bl)[2][4]) {
+#pragma unroll
+  for (int nt = 0; nt < 4; ++nt) mma16816(c[nt], ah, bh[nt >> 1][(nt & 1) * 2], bh[nt >> 1][(nt & 1) * 2 + 1]);
+#pragma unroll
+  for (int nt = 0; nt < 4; ++nt) mma16816(c[nt], ah, bl[nt >> 1][(nt & 1) * 2], bl[nt >> 1][(nt & 1) * 2 + 1]);
+#pragma unroll
+  for (int nt = 0; nt < 4; ++nt) mma16816(c[nt], al, bh[nt >> 1][(nt & 1) * 2], bh[nt >> 1][(nt & 1) * 2 + 1]);
+}
 // two values -> packed high halves and packed low halves
 __device__ __forceinline__ void split2(float a, float b, uint32_t& hi, uint32_t& lo) {
   hi = pack_bf16(a, b);
@@ -219,16 +230,15 @@ __global__ void __launch_bounds__(kChunkThreads, 2) delta_prepare_kernel(const D
         uint32_t bh[4], bl[4];
         const int bo = (nh * 32 + nn * 16 + (lane >> 4) * 8 + (lane & 7)) * kP + ks * 16 + ((lane >> 3) & 1) * 8;
         ldsm4(bh, kh + bo); ldsm4(bl, kl + bo);
+        // (neighbouring products go to different accumulators: one that waits for the previous would stall the warp)
 #pragma unroll
-        for (int e = 0; e < 2; ++e) {
-          float (&c)[4] = ck[2 * nn + e];
-          mma16816(c, ah, bh[2 * e], bh[2 * e + 1]);
-          mma16816(c, ah, bl[2 * e], bl[2 * e + 1]);
-          mma16816(c, al, bh[2 * e], bh[2 * e + 1]);
-          float (&d)[4] = cq[2 * nn + e];
-          mma16816(d, qh, bh[2 * e], bh[2 * e + 1]);
-          mma16816(d, qh, bl[2 * e], bl[2 * e + 1]);
-          mma16816(d, ql, bh[2 * e], bh[2 * e + 1]);
+        for (int term = 0; term < 3; ++term) {
+          const uint32_t (&bb)[4] = term == 1 ? bl : bh;
+#pragma unroll
+          for (int e = 0; e < 2; ++e) {
+            mma16816(ck[2 * nn + e], term == 2 ? al : ah, bb[2 * e], bb[2 * e + 1]);
+            mma16816(cq[2 * nn + e], term == 2 ? ql : qh, bb[2 * e], bb[2 * e + 1]);
+          }
         }
       }
     }
@@ -353,16 +363,14 @@ __global__ void __launch_bounds__(kChunkThreads, 2) delta_prepare_kernel(const D
       uint32_t ah[4], al[4];
       t_frag(ks, true, ah, al);
 #pragma unroll
-      for (int nn = 0; nn < NT / 2; ++nn) {
-        uint32_t bh[4], bl[4];
-        const int bo = (ks * 16 + (lane & 15)) * kP + nh * (D / 2) + nn * 16 + (lane >> 4) * 8;
-        ldsm4t(bh, kh + bo); ldsm4t(bl, kl + bo);
+      for (int n0 = 0; n0 < NT / 2; n0 += 2) {
+        uint32_t bh[2][4], bl[2][4];
 #pragma unroll
-        for (int e = 0; e < 2; ++e) {
-          mma16816(c[2 * nn + e], ah, bh[2 * e], bh[2 * e + 1]);
-          mma16816(c[2 * nn + e], ah, bl[2 * e], bl[2 * e + 1]);
-          mma16816(c[2 * nn + e], al, bh[2 * e], bh[2 * e + 1]);
+        for (int nn = 0; nn < 2; ++nn) {
+          const int bo = (ks * 16 + (lane & 15)) * kP + nh * (D / 2) + (n0 + nn) * 16 + (lane >> 4) * 8;
+          ldsm4t(bh[nn], kh + bo); ldsm4t(bl[nn], kl + bo);
         }
+        mma_split4(&c[2 * n0], ah, al, bh, bl);
       }
     }
 #pragma unroll
@@ -389,18 +397,13 @@ __global__ void __launch_bounds__(kChunkThreads, 2) delta_prepare_kernel(const D
       for (int ks = 0; ks <= mt; ++ks) {
         uint32_t ah[4], al[4];
         t_frag(ks, false, ah, al);
+        uint32_t bh[2][4], bl[2][4];
 #pragma unroll
         for (int nn = 0; nn < 2; ++nn) {
-          uint32_t bh[4], bl[4];
           const int bo = (ks * 16 + (lane & 15)) * kP + nh * 32 + nn * 16 + (lane >> 4) * 8;
-          ldsm4t(bh, yh + bo); ldsm4t(bl, yl + bo);
-#pragma unroll
-          for (int e = 0; e < 2; ++e) {
-            mma16816(c[2 * nn + e], ah, bh[2 * e], bh[2 * e + 1]);
-            mma16816(c[2 * nn + e], ah, bl[2 * e], bl[2 * e + 1]);
-            mma16816(c[2 * nn + e], al, bh[2 * e], bh[2 * e + 1]);
-          }
+          ldsm4t(bh[nn], yh + bo); ldsm4t(bl[nn], yl + bo);
         }
+        mma_split4(c, ah, al, bh, bl);
       }
 #pragma unroll
       for (int nt = 0; nt < 4; ++nt)
@@ -524,18 +527,13 @@ __global__ void __launch_bounds__(kChunkThreads, 1) delta_scan_kernel(const Delt
 #pragma unroll
     for (int ks = 0; ks < kKS; ++ks) {
       const uint32_t ah[4] = {fa[ks][0].x, fa[ks][0].y, fa[ks][0].z, fa[ks][0].w}, al[4] = {fa[ks][1].x, fa[ks][1].y, fa[ks][1].z, fa[ks][1].w};
+      uint32_t bh[2][4], bl[2][4];
 #pragma unroll
       for (int nn = 0; nn < 2; ++nn) {
-        uint32_t bh[4], bl[4];
         const int bo = (ks * 16 + (lane & 15)) * kSP + nn * 16 + (lane >> 4) * 8;
-        ldsm4t(bh, sh + bo); ldsm4t(bl, sl + bo);
-#pragma unroll
-        for (int e = 0; e < 2; ++e) {
-          mma16816(acc[2 * nn + e], ah, bh[2 * e], bh[2 * e + 1]);
-          mma16816(acc[2 * nn + e], ah, bl[2 * e], bl[2 * e + 1]);
-          mma16816(acc[2 * nn + e], al, bh[2 * e], bh[2 * e + 1]);
-        }
+        ldsm4t(bh[nn], sh + bo); ldsm4t(bl[nn], sl + bo);
       }
+      mma_split4(acc, ah, al, bh, bl);
     }
     asm volatile("cp.async.wait_group 0;" ::: "memory");
     __syncwarp();
@@ -576,13 +574,7 @@ __global__ void __launch_bounds__(kChunkThreads, 1) delta_scan_kernel(const Delt
         }
         auto mul = [&](float (&d)[4][4], const uint4& fh, const uint4& fl) {
           const uint32_t ah[4] = {fh.x, fh.y, fh.z, fh.w}, al[4] = {fl.x, fl.y, fl.z, fl.w};
-#pragma unroll
-          for (int nt = 0; nt < 4; ++nt) {
-            const int nn = nt >> 1, e = (nt & 1) * 2;
-            mma16816(d[nt], ah, bh[nn][e], bh[nn][e + 1]);
-            mma16816(d[nt], ah, bl[nn][e], bl[nn][e + 1]);
-            mma16816(d[nt], al, bh[nn][e], bh[nn][e + 1]);
-          }
+          mma_split4(d, ah, al, bh, bl);
         };
         if (holds) mul(S, mine[ks * 64], mine[ks * 64 + 32]);
         if (want_o) mul(acc, mine[256 + ks * 64], mine[256 + ks * 64 + 32]);
