@@ -48,6 +48,60 @@ class DeltaSpec:
 
 
 @dataclass(frozen=True)
+class RopeSpec:
+    """Rotary positions on the first ``dims`` dimensions of a head, pairs (2i, 2i + 1).  ``factor`` other than 1: frequencies
+    whose wavelength is above ``original / low`` are divided by it, those below ``original / high`` are kept, the band between
+    is blended linearly in the number of turns over ``original`` positions."""
+    dims: int
+    base: float
+    factor: float = 1.0
+    low: float = 1.0
+    high: float = 4.0
+    original: int = 0
+
+
+@dataclass(frozen=True)
+class AttentionSpec:
+    """Softmax attention of one layer over paged keys and values, with a causal convolution of ``conv`` taps on the channels of
+    q, k and v (0 = none).  A query at position i sees the last ``window`` positions (0 = all of them) and the first
+    ``keep_first`` ones.  ``maps`` 2 is differential attention: two score maps per head over the same values, combined as
+    map 1 - lambda * map 2, the difference normed per head and scaled by 1 - ``diff`` (lambda's constant part)."""
+    heads: int
+    kv_heads: int
+    dim: int                             # query / key dims per map and head
+    vdim: int
+    window: int
+    keep_first: int
+    scale: float
+    rope: RopeSpec
+    conv: int = 0
+    maps: int = 1
+    diff: float = 0.0
+
+    @property
+    def q_channels(self) -> int:
+        return self.heads * self.maps * self.dim
+
+    @property
+    def k_channels(self) -> int:
+        return self.kv_heads * self.maps * self.dim
+
+    @property
+    def v_channels(self) -> int:
+        return self.kv_heads * self.vdim
+
+    @property
+    def conv_channels(self) -> int:
+        return self.q_channels + self.k_channels + self.v_channels
+
+
+@dataclass(frozen=True)
+class DenseSpec:
+    """SwiGLU feed-forward of width ``ffn``."""
+    ffn: int
+
+
+@dataclass(frozen=True)
 class RouterSpec:
     """Routed feed-forward of one layer: ``experts`` SwiGLU experts of width ``ffn`` and ``identity`` outputs that hand the
     input through; ``top`` of them per token out of the best ``groups_kept`` of ``groups``."""
@@ -65,14 +119,29 @@ class RouterSpec:
 
 @dataclass(frozen=True)
 class LayerSpec:
-    mixer: Any                           # LatentSpec | DeltaSpec
-    router: RouterSpec | None = None     # None = the layer has no feed-forward
+    mixer: Any                           # LatentSpec | DeltaSpec | AttentionSpec
+    router: RouterSpec | None = None     # None = the layer has no routed feed-forward
+    dense: DenseSpec | None = None       # dense feed-forward (parallel layers)
+    # parallel: mixer and feed-forward read one norm and are added together, nothing is normed after them; otherwise the
+    # sublayers follow one another, each with a norm before and after it and a convolution on its input
+    parallel: bool = False
 
     @staticmethod
     def from_dict(d: dict[str, Any]) -> "LayerSpec":
         m = d["mixer"]
-        mixer = LatentSpec(**m) if "kv_rank" in m else DeltaSpec(**m)
-        return LayerSpec(mixer, RouterSpec(**d["router"]) if d.get("router") else None)
+        if "rope" in m:
+            mixer = AttentionSpec(**{**m, "rope": RopeSpec(**m["rope"])})
+        else:
+            mixer = LatentSpec(**m) if "kv_rank" in m else DeltaSpec(**m)
+        return LayerSpec(mixer, RouterSpec(**d["router"]) if d.get("router") else None,
+                         DenseSpec(**d["dense"]) if d.get("dense") else None, bool(d.get("parallel", False)))
+
+
+@dataclass(frozen=True)
+class LayerRun:
+    """One run of a layer: looped layers run several times with the same weights, each run with its own cache and state."""
+    layer: int
+    add_embedding: bool = False          # the embedding row is added to the residual right before this run
 
 
 @dataclass(frozen=True)
@@ -136,6 +205,9 @@ class ModelConfig:
     layer_specs: tuple = ()
     canon_taps: int = 0                  # taps of the convolution every sublayer's input passes (0 = none)
     norm_groups: int = 1                 # channel groups of the RMS norms
+    norm_offset: float = 0.0             # added to the stored norm weights (1: they are stored around zero)
+    loop: tuple = ()                     # (start, stop, times): layers [start, stop) run ``times`` times in a row
+    logit_softcap: float = 0.0           # logits = cap * tanh(logits / cap); 0 = none
     compute_dtype: str = "bf16"          # bf16 | f32 (every product and activation in 32-bit; hybrid engine only)
 
     # ---- derived -----------------------------------------------------------------
@@ -152,27 +224,42 @@ class ModelConfig:
         return self.attention == "hybrid"
 
     @property
+    def layer_runs(self) -> tuple:
+        """The layers in the order they run (``LayerRun``), loops unrolled."""
+        start, stop, times = self.loop or (0, 0, 1)
+        once = [LayerRun(i) for i in range(start, stop)]
+        again = [LayerRun(i, i == start) for i in range(start, stop)]
+        return tuple([LayerRun(i) for i in range(start)] + once + again * (times - 1)
+                     + [LayerRun(i) for i in range(stop, self.num_layers)])
+
+    @property
     def state_bytes(self) -> int:
         """Recurrent state of one sequence (fp32): delta-rule states and the last inputs of every causal convolution."""
         n = 0
-        for s in self.layer_specs:
-            n += (self.canon_taps - 1) * self.hidden * (2 if s.router is not None else 1)
-            if isinstance(s.mixer, DeltaSpec):
-                n += s.mixer.heads * s.mixer.dim * s.mixer.vdim + (s.mixer.conv - 1) * s.mixer.conv_channels
+        for s in (self.layer_specs[r.layer] for r in self.layer_runs):
+            m = s.mixer
+            if not s.parallel:
+                n += (self.canon_taps - 1) * self.hidden * (2 if s.router is not None else 1)
+            if isinstance(m, DeltaSpec):
+                n += m.heads * m.dim * m.vdim
+            if not isinstance(m, LatentSpec):
+                n += max(0, m.conv - 1) * m.conv_channels
         return 4 * n
 
     def kv_elems_of(self, layer: int) -> int:
-        """Elements ``layer`` caches per token."""
+        """Elements one run of ``layer`` caches per token."""
         if self.is_hybrid:
             m = self.layer_specs[layer].mixer
+            if isinstance(m, AttentionSpec):
+                return m.k_channels + m.v_channels
             return m.record if isinstance(m, LatentSpec) else 0
         return self.kv_record_elems
 
     @property
     def kv_record_elems(self) -> int:
-        """Elements cached per token per layer (latent+rope for MLA, K and V for GQA; the average over a hybrid's layers)."""
+        """Elements cached per token per layer (latent+rope for MLA, K and V for GQA; a hybrid's layer runs averaged over its layers)."""
         if self.is_hybrid:
-            return -(-sum(self.kv_elems_of(i) for i in range(self.num_layers)) // max(1, self.num_layers))
+            return -(-sum(self.kv_elems_of(r.layer) for r in self.layer_runs) // max(1, self.num_layers))
         if self.is_mla:
             return self.kv_lora_rank + self.qk_rope_dim
         return 2 * self.num_kv_heads * self.head_dim
@@ -201,6 +288,9 @@ class ModelConfig:
 
     def mixer_params(self, layer: int) -> int:
         h, m = self.hidden, self.layer_specs[layer].mixer
+        if isinstance(m, AttentionSpec):
+            return (h * (m.conv_channels + m.heads * m.vdim) + m.conv * m.conv_channels
+                    + (4 * m.dim if m.maps == 2 else 0))
         if isinstance(m, LatentSpec):
             return (h * (m.heads * (m.dim + m.rot_dim) + m.record + 2 * m.heads * m.vdim)
                     + m.kv_rank * (1 + m.heads * (m.dim + m.vdim)))
@@ -224,7 +314,9 @@ class ModelConfig:
 
     def layer_params(self, layer: int) -> int:
         if self.is_hybrid:
-            r = self.layer_specs[layer].router
+            r, d = self.layer_specs[layer].router, self.layer_specs[layer].dense
+            if self.layer_specs[layer].parallel:
+                return self.mixer_params(layer) + self.hidden + (3 * self.hidden * d.ffn if d is not None else 0)
             p = self.mixer_params(layer) + (2 + self.canon_taps) * self.hidden
             if r is not None:
                 p += (2 + self.canon_taps) * self.hidden + r.outputs * (self.hidden + 1) + 3 * r.experts * self.hidden * r.ffn
@@ -250,6 +342,8 @@ class ModelConfig:
         d = {k: v for k, v in d.items() if k in names}
         if "window_layers" in d:
             d["window_layers"] = tuple(d["window_layers"])
+        if "loop" in d:
+            d["loop"] = tuple(d["loop"])
         if d.get("layer_specs"):
             d["layer_specs"] = tuple(v if isinstance(v, LayerSpec) else LayerSpec.from_dict(v) for v in d["layer_specs"])
         return ModelConfig(**d)
@@ -333,24 +427,35 @@ def kimi_k2() -> ModelConfig:
 
 
 def hybrid_config(name: str, vocab: int, hidden: int, specs, canon_taps: int, norm_groups: int, eps: float,
-                  family: str = "karusun") -> ModelConfig:
+                  family: str = "karusun", **kw: Any) -> ModelConfig:
     """ModelConfig of a per-layer design.  The flat fields carry the widest layer's values for code that only sizes
-    things (planner, reports); the engine reads the specs."""
+    things (planner, reports); the engine reads the specs.  ``kw``: further fields (norm_offset, loop, logit_softcap)."""
     specs = tuple(specs)
     lat = [s.mixer for s in specs if isinstance(s.mixer, LatentSpec)]
+    att = [s.mixer for s in specs if isinstance(s.mixer, AttentionSpec)]
     routers = [s.router for s in specs if s.router is not None]
     big = max(lat, key=lambda m: m.heads * (m.dim + m.rot_dim), default=None)
     wide = max(routers, key=lambda r: r.experts * r.ffn, default=None)
+    top = max(att, key=lambda m: m.conv_channels, default=None)
+    rope = big.rope_base if big else top.rope.base if top else 10000.0
+    head_dim = (big.dim + big.rot_dim) if big else (top.maps * top.dim) if top else specs[0].mixer.dim
     return ModelConfig(
         name=name, family=family, vocab_size=vocab, num_layers=len(specs), hidden=hidden, attention="hybrid", layer_specs=specs,
-        canon_taps=canon_taps, norm_groups=norm_groups, rms_eps=eps, rope_interleaved=False,
-        num_heads=max(s.mixer.heads for s in specs), num_kv_heads=1, head_dim=(big.dim + big.rot_dim) if big else specs[0].mixer.dim,
+        canon_taps=canon_taps, norm_groups=norm_groups, rms_eps=eps, rope_interleaved=not lat and bool(att),
+        num_heads=max(s.mixer.heads for s in specs), num_kv_heads=top.kv_heads if top else 1, head_dim=head_dim,
         q_lora_rank=0, kv_lora_rank=big.kv_rank if big else 0, qk_nope_dim=big.dim if big else 0, qk_rope_dim=big.rot_dim if big else 0,
-        v_head_dim=big.vdim if big else specs[0].mixer.vdim, rope_theta=big.rope_base if big else 10000.0,
-        sliding_window=max((m.window for m in lat), default=0), dense_ffn=0, first_dense_layers=0,
-        num_experts=wide.experts if wide else 0, expert_ffn=wide.ffn if wide else 0, top_k=wide.top if wide else 0,
+        v_head_dim=big.vdim if big else specs[0].mixer.vdim, rope_theta=rope,
+        sliding_window=max((m.window for m in lat + att), default=0), dense_ffn=max((s.dense.ffn for s in specs if s.dense), default=0),
+        first_dense_layers=0, num_experts=wide.experts if wide else 0, expert_ffn=wide.ffn if wide else 0, top_k=wide.top if wide else 0,
         num_groups=wide.groups if wide else 1, topk_groups=wide.groups_kept if wide else 1, num_shared_experts=0,
-        norm_topk_prob=False, router_bias=bool(routers))
+        norm_topk_prob=False, router_bias=bool(routers), **kw)
+
+
+def parallel_config(name: str, vocab: int, hidden: int, specs, eps: float, loop: tuple = (), logit_softcap: float = 0.0,
+                    family: str = "guberax") -> ModelConfig:
+    """ModelConfig of a stack of parallel layers: norm weights stored around zero, an optional loop, capped logits."""
+    return hybrid_config(name, vocab, hidden, specs, canon_taps=1, norm_groups=1, eps=eps, family=family, norm_offset=1.0,
+                         loop=tuple(loop), logit_softcap=logit_softcap)
 
 
 # Benchmark sizes: width, layers, heads, expert width (latent 512 + 64 and heads of 128 throughout, as real models have them)
@@ -377,8 +482,35 @@ def karusun_bench_mla(size: str = "base") -> ModelConfig:
                        scoring="softmax", num_groups=8, topk_groups=4, num_shared_experts=0, norm_topk_prob=False, router_bias=True)
 
 
+# Benchmark sizes: width, layers, heads, key / value heads, feed-forward width (two 64-wide maps and 128-wide values per head)
+GUBERAX_SIZES = {"small": (1024, 24, 8, 4, 2816), "base": (2048, 24, 16, 8, 5632), "large": (4096, 16, 32, 8, 11008)}
+
+
+def guberax_bench(size: str = "base") -> ModelConfig:
+    """A Guberax-shaped stack at the sizes of a real model's layers: differential attention with a 2048-token window and 128
+    kept tokens, four-tap convolutions, the middle third of the layers run twice."""
+    width, layers, heads, kv_heads, ffn = GUBERAX_SIZES[size]
+    m = AttentionSpec(heads=heads, kv_heads=kv_heads, dim=64, vdim=128, window=2048, keep_first=128, scale=64 ** -0.5,
+                      rope=RopeSpec(64, 5.0e5, 8.0, 1.0, 4.0, 8192), conv=4, maps=2, diff=0.5)
+    once = layers - layers // 4
+    start = (once - layers // 4) // 2
+    return parallel_config(f"guberax-{size}", 65536, width, [LayerSpec(m, dense=DenseSpec(ffn), parallel=True)] * once, eps=1e-6,
+                           loop=(start, start + layers // 4, 2), logit_softcap=30.0)
+
+
+def guberax_bench_gqa(size: str = "base") -> ModelConfig:
+    """The dense GQA decoder at the size of ``guberax_bench``: as many layer runs of the same width, heads, window and
+    feed-forward."""
+    width, layers, heads, kv_heads, ffn = GUBERAX_SIZES[size]
+    return ModelConfig(name=f"gqa-{size}", family="llama", vocab_size=65536, num_layers=layers, hidden=width, attention="gqa",
+                       num_heads=heads, num_kv_heads=kv_heads, head_dim=128, qk_norm=False, sliding_window=2048, rope_theta=5.0e5,
+                       rope_interleaved=False, rms_eps=1e-6, dense_ffn=ffn, first_dense_layers=layers, num_experts=0, expert_ffn=0,
+                       top_k=0, num_shared_experts=0)
+
+
 PRESETS = {
     "karusun-base": karusun_bench,
+    "guberax-base": guberax_bench,
     "tiny-moe": tiny_moe,
     "mixtral-8x7b": mixtral_8x7b,
     "mistral-7b": mistral_7b,
@@ -393,8 +525,10 @@ PRESETS = {
 def scaled_down(cfg: ModelConfig, layers: int = 2, vocab: int = 2048) -> ModelConfig:
     """Same per-layer geometry with fewer layers and a small vocabulary (tests, smoke)."""
     if cfg.is_hybrid:
+        start, stop, times = cfg.loop or (0, 0, 1)
         return hybrid_config(cfg.name + "-mini", vocab, cfg.hidden, cfg.layer_specs[:layers], cfg.canon_taps, cfg.norm_groups,
-                             cfg.rms_eps, cfg.family)
+                             cfg.rms_eps, cfg.family, norm_offset=cfg.norm_offset, logit_softcap=cfg.logit_softcap,
+                             loop=(start, min(stop, layers), times) if start < layers and cfg.loop else ())
     first_dense = min(cfg.first_dense_layers, max(layers - 1, 0)) if cfg.first_dense_layers else 0
     return cfg.replace(name=cfg.name + "-mini", num_layers=layers, vocab_size=vocab,
                        first_dense_layers=first_dense)

@@ -161,7 +161,7 @@ class KarusunModel(FamilyModel):
         if e:
             return "routed_expert", layer, int(e.group(1))
         if rest.startswith("mlp."):
-            return "router", layer, None
+            return ("router" if rest in ("mlp.router", "mlp.correction") else "dense_ffn"), layer, None
         return ("norm" if rest.startswith(("norm", "canon")) else "other"), layer, None
 
 
@@ -174,6 +174,15 @@ class Karusun(Family):
 
     def open(self, cfg: ModelConfig, hf_config: dict) -> FamilyModel:
         return KarusunModel(self, cfg, ExpertContract(formats=("bf16",)))
+
+
+class Guberax(Karusun):
+    """Stacks of parallel layers (differential attention beside a dense feed-forward), some of them looped: served by the
+    hybrid engine."""
+    id, model_types, attention = "guberax", ("guberax",), "hybrid"
+
+    def detect(self, hf_config: dict) -> bool:
+        return hf_config.get("architecture") == "Guberax"
 
 
 class TinyMoe(Family):
@@ -195,7 +204,7 @@ def canonical_name(name: str) -> str:
     return _MIXTRAL_RE.sub(lambda m: m.group(1) + _MIXTRAL_PROJ[m.group(2)] + m.group(3), name)
 
 
-REGISTRY: tuple[Family, ...] = (DeepseekV32(), DeepseekV3(), Qwen3Moe(), Glm4Moe(), Qwen2(), Llama(), TinyMoe(), Karusun())
+REGISTRY: tuple[Family, ...] = (DeepseekV32(), DeepseekV3(), Qwen3Moe(), Glm4Moe(), Qwen2(), Llama(), TinyMoe(), Karusun(), Guberax())
 
 
 def detect(hf_config: dict) -> Family | None:

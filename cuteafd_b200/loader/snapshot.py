@@ -12,7 +12,8 @@ import os
 
 import torch
 
-from ..config import DeltaSpec, LatentSpec, LayerSpec, ModelConfig, RouterSpec, hybrid_config
+from ..config import (AttentionSpec, DeltaSpec, DenseSpec, LatentSpec, LayerSpec, ModelConfig, RopeSpec, RouterSpec, hybrid_config,
+                      parallel_config)
 from ..ref.model import init_weights
 from . import formats
 from .safetensors_io import write_sharded
@@ -24,6 +25,8 @@ ARCH = {"llama": "LlamaForCausalLM", "qwen3_moe": "Qwen3MoeForCausalLM", "deepse
 
 def _layer_list_to_json(cfg: ModelConfig) -> dict:
     """config.json of a per-layer design (the ``layers`` list form)."""
+    if cfg.family == "guberax":
+        return _parallel_layers_to_json(cfg)
     layers = []
     for s in cfg.layer_specs:
         m, r = s.mixer, s.router
@@ -40,9 +43,63 @@ def _layer_list_to_json(cfg: ModelConfig) -> dict:
             "canon": {"taps": cfg.canon_taps}, "norm": {"eps": cfg.rms_eps, "groups": cfg.norm_groups}}
 
 
+def _parallel_layers_to_json(cfg: ModelConfig) -> dict:
+    layers = []
+    for s in cfg.layer_specs:
+        m, r = s.mixer, s.mixer.rope
+        rot = {"base": r.base, "dims": r.dims}
+        if r.factor != 1.0:
+            rot["scaling"] = {"factor": r.factor, "low": r.low, "high": r.high, "original": r.original}
+        e = {"heads": m.heads, "kv_heads": m.kv_heads, "dim": m.dim, "vdim": m.vdim, "conv": m.conv, "diff": m.diff, "scale": m.scale, "rot": rot}
+        if m.window:
+            e["mask"] = {"size": m.window, "keep_first": m.keep_first}
+        layers.append({"type": "attention", "mixer": e, "mlp": None if s.dense is None else {"kind": "dense", "ff": s.dense.ffn}})
+    d = {"architecture": "Guberax", "name": cfg.name, "vocab": cfg.vocab_size, "width": cfg.hidden, "layers": layers, "norm": {"eps": cfg.rms_eps}}
+    if cfg.loop:
+        d["loop"] = dict(zip(("start", "stop", "times"), cfg.loop))
+    if cfg.logit_softcap:
+        d["logit_softcap"] = cfg.logit_softcap
+    return d
+
+
+def _parallel_layers_from_json(d: dict) -> ModelConfig:
+    """Parallel layers of differential attention and a dense feed-forward (``architecture`` Guberax)."""
+    specs = []
+    for i, e in enumerate(d["layers"]):
+        m, mlp = e["mixer"], e.get("mlp")
+        if e["type"] != "attention":
+            raise ValueError(f"layer {i}: unsupported mixer {e['type']!r}")
+        rot, mask = m["rot"], m.get("mask") or {}
+        sc = rot.get("scaling") or {}
+        rope = RopeSpec(dims=rot.get("dims", m["dim"]), base=float(rot["base"]))
+        if float(sc.get("factor", 1.0)) != 1.0:
+            rope = RopeSpec(rope.dims, rope.base, float(sc["factor"]), float(sc["low"]), float(sc["high"]), int(sc["original"]))
+        mixer = AttentionSpec(heads=m["heads"], kv_heads=m.get("kv_heads") or m["heads"], dim=m["dim"], vdim=m.get("vdim") or m["dim"],
+                              window=mask.get("size") or 0, keep_first=(mask.get("keep_first") or 0) if mask.get("size") else 0,
+                              scale=float(m["scale"]), rope=rope, conv=m.get("conv") or 0, maps=2, diff=float(m["diff"]))
+        if mixer.heads % mixer.kv_heads:
+            raise ValueError(f"layer {i}: {mixer.heads} heads over {mixer.kv_heads} key heads")
+        if rope.dims % 2 or rope.dims > mixer.dim:
+            raise ValueError(f"layer {i}: {rope.dims} rotated dims of {mixer.dim}")
+        dense = None
+        if mlp is not None:
+            if mlp.get("kind") != "dense":
+                raise ValueError(f"layer {i}: unsupported feed-forward {mlp.get('kind')!r}")
+            dense = DenseSpec(mlp["ff"])
+        specs.append(LayerSpec(mixer, dense=dense, parallel=True))
+    lp = d.get("loop")
+    loop = (lp["start"], lp["stop"], lp["times"]) if lp else ()
+    if loop and not (0 <= loop[0] < loop[1] <= len(specs) and loop[2] >= 1):
+        raise ValueError(f"loop {loop} over {len(specs)} layers")
+    return parallel_config(d.get("name", d["architecture"].lower()), d["vocab"], d["width"], specs, float(d["norm"]["eps"]), loop,
+                           float(d.get("logit_softcap") or 0.0))
+
+
 def _layer_list_from_json(d: dict) -> ModelConfig:
     """The ``layers`` list form of config.json.  Every layer carries its own sizes; a type or kind that is not built is
     refused by name."""
+    if d["architecture"] == "Guberax":
+        return _parallel_layers_from_json(d)
     specs = []
     for i, e in enumerate(d["layers"]):
         m, mlp = e["mixer"], e.get("mlp")
@@ -169,7 +226,7 @@ def _rope_scaling(d: dict) -> dict:
 
 def from_hf_config(d: dict) -> ModelConfig:
     """Map a config.json onto the engine's geometry.  Unknown architectures raise ValueError."""
-    if d.get("architecture") == "Karusun":
+    if d.get("architecture") in ("Karusun", "Guberax"):
         return _layer_list_from_json(d)
     mt = d.get("model_type", "")
     extra = d.get("cuteafd", {})

@@ -1,5 +1,6 @@
 """CPU oracle of the per-layer hybrid decoders (``ModelConfig.layer_specs``): windowed latent attention layers and gated
-delta-rule layers in any order, each behind grouped RMS norms, input convolutions and a routed feed-forward.
+delta-rule layers in any order, each behind grouped RMS norms, input convolutions and a routed feed-forward; parallel
+layers of differential attention beside a dense feed-forward, some of them looped.
 
 One function per mechanism, written as the equations read: no chunking, no absorbed products, one token at a time where a
 recurrence runs.  ``HybridRefDecoder`` strings them together over a parameter dictionary in the checkpoint's own tensor
@@ -8,9 +9,11 @@ names and plugs into the same places as ``RefDecoder``.  All arithmetic is in th
 """
 from __future__ import annotations
 
+import math
+
 import torch
 
-from ..config import DeltaSpec, LatentSpec, ModelConfig, RouterSpec
+from ..config import AttentionSpec, DeltaSpec, LatentSpec, ModelConfig, RopeSpec, RouterSpec
 
 Params = dict[str, torch.Tensor]
 
@@ -46,6 +49,56 @@ def rotate_half(x: torch.Tensor, positions: torch.Tensor, base: float) -> torch.
     a = a.reshape(a.shape[0], *([1] * (x.dim() - 2)), d // 2)
     u, v = x[..., :d // 2], x[..., d // 2:]
     return torch.cat([u * a.cos() - v * a.sin(), v * a.cos() + u * a.sin()], -1)
+
+
+def scaled_frequencies(r: RopeSpec) -> list[float]:
+    """Turns per position of every rotated pair: short wavelengths as they are, long ones stretched by the factor, a linear
+    blend (in turns over the original length) between."""
+    out = []
+    for i in range(r.dims // 2):
+        f = r.base ** (-2.0 * i / r.dims)
+        if r.factor != 1.0:
+            turns = r.original * f / (2.0 * math.pi)              # original length over wavelength
+            if turns < r.low:
+                f = f / r.factor
+            elif turns <= r.high:
+                s = (turns - r.low) / (r.high - r.low)
+                f = (1.0 - s) * f / r.factor + s * f
+        out.append(f)
+    return out
+
+
+def rotate_pairs(x: torch.Tensor, positions: torch.Tensor, r: RopeSpec) -> torch.Tensor:
+    """x [T, ..., d]: dimensions 2i and 2i + 1 of the first ``r.dims`` are a pair turned by position * frequency."""
+    a = positions.to(x.dtype)[:, None] * torch.tensor(scaled_frequencies(r), dtype=x.dtype)
+    a = a.reshape(a.shape[0], *([1] * (x.dim() - 2)), r.dims // 2)
+    out = x.clone()
+    u, v = x[..., 0:r.dims:2], x[..., 1:r.dims:2]
+    out[..., 0:r.dims:2] = u * a.cos() - v * a.sin()
+    out[..., 1:r.dims:2] = v * a.cos() + u * a.sin()
+    return out
+
+
+def sink_attention(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, start: int, window: int, keep: int, scale: float) -> torch.Tensor:
+    """Softmax attention of q [T, H, Dk] (positions start, start + 1, ...) over k [L, H, Dk], v [L, H, Dv] (positions 0, 1, ...):
+    the query at position i reads the keys j <= i that lie among the last ``window`` positions (0: anywhere) or the first
+    ``keep``."""
+    out = []
+    for t in range(q.shape[0]):
+        i = start + t
+        seen = [j for j in range(i + 1) if window == 0 or i - j < window or j < keep]
+        s = torch.einsum("hd,jhd->hj", q[t], k[seen]) * scale
+        out.append(torch.einsum("hj,jhd->hd", torch.softmax(s, -1), v[seen]))
+    return torch.stack(out)
+
+
+def difference_weight(p: Params, pre: str, diff: float) -> torch.Tensor:
+    """lambda: the weight of the second map, one number per layer."""
+    return torch.exp((p[pre + "lq1"] * p[pre + "lk1"]).sum()) - torch.exp((p[pre + "lq2"] * p[pre + "lk2"]).sum()) + diff
+
+
+def softcap(x: torch.Tensor, cap: float) -> torch.Tensor:
+    return cap * torch.tanh(x / cap)
 
 
 def window_attention(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, start: int, window: int, scale: float) -> torch.Tensor:
@@ -149,6 +202,28 @@ def delta_mixer(h: torch.Tensor, p: Params, pre: str, m: DeltaSpec, eps: float, 
     return o @ p[pre + "o"].T
 
 
+def attention_mixer(h: torch.Tensor, p: Params, pre: str, m: AttentionSpec, eps: float, start: int, st: dict) -> torch.Tensor:
+    """Attention with convolved and rotated queries and keys; with two maps per head their difference, normed per head."""
+    T, rep = h.shape[0], m.heads // m.kv_heads
+    pos = torch.arange(start, start + T)
+    x = {}
+    for n in ("q", "k", "v"):
+        x[n] = h @ p[pre + n].T
+        if m.conv:
+            x[n], st["conv." + n] = causal_conv(x[n], p[pre + n + ".conv"], st["conv." + n])
+    q = rotate_pairs(x["q"].view(T, m.heads, m.maps, m.dim), pos, m.rope)
+    st["k"] = torch.cat([st["k"], rotate_pairs(x["k"].view(T, m.kv_heads, m.maps, m.dim), pos, m.rope)])
+    st["v"] = torch.cat([st["v"], x["v"].view(T, m.kv_heads, m.vdim)])
+    k, v = st["k"].repeat_interleave(rep, 1), st["v"].repeat_interleave(rep, 1)
+    a = [sink_attention(q[:, :, j], k[:, :, j], v, start, m.window, m.keep_first, m.scale) for j in range(m.maps)]
+    o = a[0] if m.maps == 1 else rms(a[0] - difference_weight(p, pre, m.diff) * a[1], eps) * (1 - m.diff)
+    return o.reshape(T, m.heads * m.vdim) @ p[pre + "o"].T
+
+
+def dense_ffn(h: torch.Tensor, p: Params, pre: str) -> torch.Tensor:
+    return (silu(h @ p[pre + "gate"].T) * (h @ p[pre + "up"].T)) @ p[pre + "down"].T
+
+
 # ---- state ----------------------------------------------------------------------------------------------------------
 class HybridState:
     """What one sequence carries: latent records per position, and the recurrent parts.  The recurrent parts cannot be
@@ -158,11 +233,16 @@ class HybridState:
         self.length_ = 0
         self.layers: list[dict] = []
         self.marks: dict[int, list[dict]] = {}
-        for spec in cfg.layer_specs:
+        for spec in (cfg.layer_specs[r.layer] for r in cfg.layer_runs):
             z = lambda *s: torch.zeros(*s, dtype=dtype)               # noqa: E731
-            st = {"canon1": z(cfg.canon_taps - 1, cfg.hidden), "canon2": z(cfg.canon_taps - 1, cfg.hidden)}
+            st = {} if spec.parallel else {"canon1": z(cfg.canon_taps - 1, cfg.hidden), "canon2": z(cfg.canon_taps - 1, cfg.hidden)}
             m = spec.mixer
-            if isinstance(m, LatentSpec):
+            if isinstance(m, AttentionSpec):
+                st.update(k=z(0, m.kv_heads, m.maps, m.dim), v=z(0, m.kv_heads, m.vdim))
+                for n, c in (("q", m.q_channels), ("k", m.k_channels), ("v", m.v_channels)):
+                    if m.conv:
+                        st["conv." + n] = z(m.conv - 1, c)
+            elif isinstance(m, LatentSpec):
                 st.update(c=z(0, m.kv_rank), kr=z(0, m.rot_dim))
             else:
                 st.update(S=z(m.heads, m.dim, m.vdim))
@@ -202,6 +282,11 @@ class HybridRefDecoder:
     def _layer(self, i: int, x: torch.Tensor, start: int, st: dict) -> torch.Tensor:
         cfg, p, spec, pre = self.cfg, self.p, self.cfg.layer_specs[i], f"l{i}."
 
+        if spec.parallel:
+            h = group_rms(x, p[pre + "norm1"] + cfg.norm_offset, cfg.norm_groups, cfg.rms_eps)
+            y = attention_mixer(h, p, pre + "mix.", spec.mixer, cfg.rms_eps, start, st)
+            return x + (y if spec.dense is None else y + dense_ffn(h, p, pre + "mlp."))
+
         def sublayer(x, n, fn):
             h = group_rms(x, p[f"{pre}norm{n}"], cfg.norm_groups, cfg.rms_eps)
             y, st[f"canon{n}"] = causal_conv(h, p[f"{pre}canon{n}"], st[f"canon{n}"])
@@ -217,9 +302,10 @@ class HybridRefDecoder:
         return x
 
     def _run(self, tokens: torch.Tensor, kv: HybridState) -> torch.Tensor:
-        x, start = self.p["embed"][tokens], kv.length_
-        for i in range(len(self.cfg.layer_specs)):
-            x = self._layer(i, x, start, kv.layers[i])
+        e, start = self.p["embed"][tokens], kv.length_
+        x = e
+        for n, r in enumerate(self.cfg.layer_runs):
+            x = self._layer(r.layer, x + e if r.add_embedding else x, start, kv.layers[n])
             if self.trace is not None:
                 self.trace.append(x)
         kv.length_ = start + tokens.shape[0]
@@ -238,7 +324,9 @@ class HybridRefDecoder:
         return torch.cat(out)
 
     def head(self, x: torch.Tensor) -> torch.Tensor:
-        return group_rms(x, self.p["final.norm"], self.cfg.norm_groups, self.cfg.rms_eps) @ self.p["head"].T
+        cfg = self.cfg
+        z = group_rms(x, self.p["final.norm"] + cfg.norm_offset, cfg.norm_groups, cfg.rms_eps) @ self.p["head"].T
+        return softcap(z, cfg.logit_softcap) if cfg.logit_softcap else z
 
     def forward(self, tokens: torch.Tensor, kv: HybridState, embeds: tuple | None = None) -> torch.Tensor:
         return self.head(self.hidden_states(tokens, kv, embeds))
@@ -252,12 +340,26 @@ def init_hybrid_weights(cfg: ModelConfig, seed: int = 0, dtype: torch.dtype = to
         return (torch.randn(*shape, generator=g) * (s if s is not None else std if std is not None else shape[-1] ** -0.5)).to(dtype)
 
     def near_one(n: int) -> torch.Tensor:
-        return (1 + 0.2 * torch.randn(n, generator=g)).to(dtype)
+        return (1 - cfg.norm_offset + 0.2 * torch.randn(n, generator=g)).to(dtype)
 
     H = cfg.hidden
     p: Params = {"embed": w(cfg.vocab_size, H, s=1.0), "final.norm": near_one(H), "head": w(cfg.vocab_size, H)}
     for i, spec in enumerate(cfg.layer_specs):
         pre, m, r = f"l{i}.", spec.mixer, spec.router
+        if spec.parallel:
+            x, d = pre + "mix.", spec.dense
+            p[pre + "norm1"] = near_one(H)
+            for n, c in (("q", m.q_channels), ("k", m.k_channels), ("v", m.v_channels)):
+                p[x + n] = w(c, H)
+                if m.conv:
+                    p[x + n + ".conv"] = w(c, m.conv)
+            if m.maps == 2:
+                p.update({x + n: w(m.dim, s=0.5 * m.dim ** -0.5) for n in ("lq1", "lk1", "lq2", "lk2")})
+            p[x + "o"] = w(H, m.heads * m.vdim)
+            if d is not None:
+                x = pre + "mlp."
+                p[x + "gate"], p[x + "up"], p[x + "down"] = w(d.ffn, H), w(d.ffn, H), w(H, d.ffn)
+            continue
         for n in ("norm1", "norm1b") + (("norm2", "norm2b") if r is not None else ()):
             p[pre + n] = near_one(H)
         for n in ("canon1",) + (("canon2",) if r is not None else ()):
@@ -288,4 +390,5 @@ def bf16_params(p: Params, dtype: torch.dtype = torch.float32) -> Params:
 
 
 __all__ = ["HybridRefDecoder", "HybridState", "init_hybrid_weights", "bf16_params", "group_rms", "causal_conv", "rotate_half",
+           "scaled_frequencies", "rotate_pairs", "sink_attention", "difference_weight", "softcap", "attention_mixer", "dense_ffn",
            "window_attention", "delta_recurrence", "route", "routed_ffn", "latent_mixer", "delta_mixer", "rms", "unit"]
