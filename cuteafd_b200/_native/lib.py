@@ -81,7 +81,25 @@ class NormArgs(C.Structure):
     _fields_ = [(n, C.c_void_p) for n in ("tokens", "embed", "x_in", "y", "slot_w", "slot_idx", "ident", "w_b", "w", "conv", "x_out",
                                           "h_out", "row_idx", "state", "state_in", "state_out", "q_start")]
     _fields_ += [("slot_stride", C.c_longlong), ("state_off", C.c_longlong)]
-    _fields_ += [(n, C.c_int) for n in ("T", "H", "S", "ldy", "ldh", "groups", "taps", "top_k", "n_experts", "vocab", "run")] + [("eps", C.c_float)]
+    _fields_ += [(n, C.c_int) for n in ("T", "H", "S", "ldy", "ldh", "groups", "taps", "top_k", "n_experts", "vocab", "run")]
+    _fields_ += [("eps", C.c_float), ("w_off", C.c_float)]
+
+
+class ConvRope(C.Structure):
+    """cafd_conv_rope_kv (csrc/conv_rope.cu)."""
+    _fields_ = [(n, C.c_void_p) for n in ("proj", "conv_w", "table", "slots", "q_start", "state_in", "state_out", "state", "q_out",
+                                          "k_cache", "v_cache")]
+    _fields_ += [("slot_stride", C.c_longlong), ("state_off", C.c_longlong)]
+    _fields_ += [(n, C.c_int) for n in ("T", "S", "ld", "q_off", "k_off", "v_off", "nq", "nk", "nv", "maps_dim", "dim", "vdim", "kv_heads",
+                                        "rot", "taps", "run")]
+
+
+class PagedAttn(C.Structure):
+    """cafd_paged_attn (csrc/attention_any.cu)."""
+    _fields_ = [(n, C.c_void_p) for n in ("q", "k_cache", "v_cache", "page_table", "positions", "q_start", "out")]
+    _fields_ += [(n, C.c_int) for n in ("T", "S", "heads", "kv_heads", "maps", "dim", "vdim", "window", "keep", "max_pages", "ldo",
+                                        "head_pitch", "heads_per_block")]
+    _fields_ += [(n, C.c_float) for n in ("scale", "lam", "out_scale", "eps")]
 
 
 class LatentPrep(C.Structure):
@@ -203,6 +221,10 @@ def cuda_lib():
         _sig(lib, "cafd_sample_rows", [P, I, I, P, P, I, P, P, P])
         _sig(lib, "cafd_accept_prefix", [P, P, P, I, P, P, P])
         _sig(lib, "cafd_norm_conv", [C.POINTER(NormArgs), I, P])
+        _sig(lib, "cafd_rope_table", [P, P, P, I, I, P])
+        _sig(lib, "cafd_conv_rope_kv", [C.POINTER(ConvRope), I, P])
+        _sig(lib, "cafd_softcap", [P, I, I, C.c_longlong, F, P])
+        _sig(lib, "cafd_paged_attn", [C.POINTER(PagedAttn), I, P])
         _sig(lib, "cafd_delta_chunked", [C.POINTER(DeltaArgs), P, C.c_longlong, P])
         _sig(lib, "cafd_delta_chunk_bytes", [I, I, I], C.c_longlong)
         _sig(lib, "cafd_swap_ids", [P, P, I, P])

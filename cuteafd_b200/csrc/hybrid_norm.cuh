@@ -1,10 +1,12 @@
 // Residual stream of the per-layer hybrid decoders: everything between two sublayers in one launch.
 //
-//   x   = embed[token]                      (first launch)       or the fp32 residual of the previous launch
+//   x   = embed[token]                      (first launch)       or the fp32 residual of the previous launch, or their sum
+//                                           (a loop's next pass)
 //   x  += groupnorm(y) * w_b                y = a mixer's output rows, or the routed experts' rows summed here:
-//                                           sum over slots of weight * (expert row, or the input row for an identity slot)
-//   h   = groupnorm(x) * w                  RMS norm in equal runs of channels, each with its own root mean square
-//   out = h + sum_j c[j] * h(t - taps + 1 + j)     causal convolution over time per channel
+//                                           sum over slots of weight * (expert row, or the input row for an identity slot);
+//                                           without w_b: x += y
+//   h   = groupnorm(x) * (w + w_off)        RMS norm in equal runs of channels, each with its own root mean square
+//   out = h + sum_j c[j] * h(t - taps + 1 + j)     causal convolution over time per channel (optional)
 //
 // A block walks a run of consecutive tokens with every channel in registers, so the convolution's earlier inputs are the
 // registers of the previous iterations; the few inputs before the run are recomputed from the residual, or come from the
@@ -21,12 +23,12 @@ namespace cafd {
 struct NormArgs {
   const int* tokens;          // with embed: token ids
   const void* embed;          // [vocab, H] E, or null
-  const float* x_in;          // [T, H]
+  const float* x_in;          // [T, H] or null (with embed: the embedding row is added to it)
   const void* y;              // [T, ldy] E, or the slot rows [T * top_k, ldy] E with slot_w; null = nothing to add
   const float* slot_w;        // [T, top_k]
   const int* slot_idx;        // [T, top_k]; an index >= n_experts is an identity slot
   const void* ident;          // [T, ldh] E: what identity slots hand through
-  const void* w_b;            // [H] E
+  const void* w_b;            // [H] E, null = y is added as it is
   const void* w;              // [H] E
   const void* conv;           // [taps, H] E, null = no convolution
   float* x_out;               // [T, H] or null
@@ -38,7 +40,7 @@ struct NormArgs {
   const int* q_start;         // [S + 1]
   long long slot_stride, state_off;
   int T, H, S, ldy, ldh, groups, taps, top_k, n_experts, vocab, run;   // ldy, ldh: elements from row to row of y, of h_out and ident
-  float eps;
+  float eps, w_off;
 };
 
 template <typename E> __device__ __forceinline__ float ld_e(const E* p);
@@ -244,7 +246,7 @@ __global__ void __launch_bounds__(kMaxThreads, kMinBlocks) norm_conv_kernel(cons
   Packed<E, V> ny[KV];
   auto fetch = [&](int tt) {
     const int row = a.row_idx ? a.row_idx[tt] : tt;
-    if (!a.embed) {
+    if (a.x_in) {
       const float* src = a.x_in + static_cast<size_t>(row) * a.H;
 #pragma unroll
       for (int k = 0; k < KV; ++k) {
@@ -274,6 +276,11 @@ __global__ void __launch_bounds__(kMaxThreads, kMinBlocks) norm_conv_kernel(cons
     for (int k = 0; k < KV; ++k)
 #pragma unroll
       for (int e = 0; e < V; ++e) { x[k][e] = 0.f; y[k][e] = 0.f; }
+    if (a.x_in) {
+#pragma unroll
+      for (int k = 0; k < KV; ++k)
+        if (tid + k * nt < nvec) unpack(nx[k], x[k]);
+    }
     if (a.embed) {
       int tok = a.tokens[row];
       tok = tok < 0 ? 0 : tok >= a.vocab ? a.vocab - 1 : tok;
@@ -281,12 +288,13 @@ __global__ void __launch_bounds__(kMaxThreads, kMinBlocks) norm_conv_kernel(cons
 #pragma unroll
       for (int k = 0; k < KV; ++k) {
         const int i = tid + k * nt;
-        if (i < nvec) load_vec<E, V>(src + i * V, x[k]);
-      }
-    } else {
+        if (i < nvec) {
+          float v[V];
+          load_vec<E, V>(src + i * V, v);
 #pragma unroll
-      for (int k = 0; k < KV; ++k)
-        if (tid + k * nt < nvec) unpack(nx[k], x[k]);
+          for (int e = 0; e < V; ++e) x[k][e] += v[e];
+        }
+      }
     }
     if (!kSlots && a.y) {
 #pragma unroll
@@ -339,7 +347,12 @@ __global__ void __launch_bounds__(kMaxThreads, kMinBlocks) norm_conv_kernel(cons
         }
       }
     }
-    if (a.y) {
+    if (a.y && !a.w_b) {
+#pragma unroll
+      for (int k = 0; k < KV; ++k)
+#pragma unroll
+        for (int e = 0; e < V; ++e) x[k][e] += y[k][e];
+    } else if (a.y) {
       float inv[KV];
       group_inv<V, KV, sizeof(E) == 4>(y, inv, sm + flip * stride, sm + flip * stride + nvec, nvec, gvec, grp, inv_n, fast, a.eps);
       flip ^= 1;
@@ -371,7 +384,7 @@ __global__ void __launch_bounds__(kMaxThreads, kMinBlocks) norm_conv_kernel(cons
         float wn[V];
         load_vec<E, V>(static_cast<const E*>(a.w) + i * V, wn);
 #pragma unroll
-        for (int e = 0; e < V; ++e) x[k][e] = x[k][e] * inv[k] * wn[e];
+        for (int e = 0; e < V; ++e) x[k][e] = x[k][e] * inv[k] * (wn[e] + a.w_off);
       }
     }
     if (own) {
@@ -455,6 +468,13 @@ template <typename E>
 static int dispatch_norm(const NormArgs& a, cudaStream_t st) {
   const int per_group = a.H / a.groups;
   const bool few = !a.conv || a.taps <= 4;
+  if (!a.conv && per_group % 8 == 0) {          // no convolution: no window of earlier rows in registers
+    if (a.T > 256 && a.H <= 2048) return launch_norm<E, 8, 1, 1, 256, 4>(a, st);
+    if (a.T > 256 && a.H <= 4096) return launch_norm<E, 8, 2, 1, 256, 3>(a, st);
+    if (a.H <= 4096) return launch_norm<E, 8, 1, 1, 512, 1>(a, st);
+    if (a.H <= 8192) return launch_norm<E, 8, 2, 1, 512, 1>(a, st);
+    return -13;
+  }
   if (few && per_group % 8 == 0) {
     // eight channels per thread: a thread's channels share their group, so one reduction serves them all
     // prompts: several blocks per SM, each at its own token, hide the loads and barriers; decode: one block per token

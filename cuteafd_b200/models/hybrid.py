@@ -1,22 +1,25 @@
 """Per-layer hybrid decoders (``ModelConfig.layer_specs``): windowed latent attention and gated delta-rule layers in any
 order, grouped RMS norms before and after every sublayer, a causal convolution on every sublayer's input, routed
-feed-forwards with identity outputs.
+feed-forwards with identity outputs; and stacks of parallel layers (differential attention beside a dense feed-forward under
+one norm), some of them looped.
 
 A layer is a fixed launch sequence over preallocated workspaces:
 
     norm_conv -> fused projection -> mixer kernels -> o projection -> norm_conv -> routes -> plan / dispatch -> fc1 -> fc2
+    parallel:  norm_conv -> fused q / k / v -> conv_rope_kv -> attention -> gate / up -> [o | down] as one product
 
 ``norm_conv`` is everything between two sublayers (the routed rows' weighted sum, the norm after the sublayer, the fp32
 residual, the norm before the next one, its convolution).  What a sequence carries besides latent records lives in slots
 of one fp32 pool; a step reads one slot per sequence and writes another (``Batch.state_in`` / ``state_out``), so a step
 can be repeated and a slot can be shared with a cached prefix.  ``compute_dtype`` "f32" runs the same sequence with every
-product and activation in 32-bit.
+product and activation in 32-bit.  A looped layer runs several times with the same weights; cache and state belong to the run
+(``ModelConfig.layer_runs``), not to the layer.
 """
 from __future__ import annotations
 
 import torch
 
-from ..config import DeltaSpec, LatentSpec, ModelConfig
+from ..config import AttentionSpec, DeltaSpec, LatentSpec, ModelConfig, RopeSpec
 from ..ops import kernels as K
 from ..parallel.moe_exchange import ExchangeGeometry, LocalExchange
 from .gqa_moe import PAGE, Batch
@@ -36,12 +39,22 @@ def record_pitch(m: LatentSpec) -> int:
     return pad8(m.record)
 
 
+def rope_frequencies(r: RopeSpec) -> torch.Tensor:
+    """fp32 [dims / 2] turns per position, worked out in fp64."""
+    f = r.base ** (-torch.arange(0, r.dims, 2, dtype=torch.float64) / max(1, r.dims))
+    if r.factor != 1.0:
+        wave = 2 * torch.pi / f
+        s = (r.original / wave - r.low) / (r.high - r.low) if r.high != r.low else torch.zeros_like(f)
+        f = torch.where(wave < r.original / r.high, f, torch.where(wave > r.original / r.low, f / r.factor, (1 - s) * f / r.factor + s * f))
+    return f.float()
+
+
 class HybridLayer:
     """One layer's weights in the layout the kernels stream: the projections that read the same input are one matrix
     (``offs`` names its sections, each padded to a multiple of 8 rows), experts are stacked."""
     __slots__ = ("norm1", "norm1b", "norm2", "norm2b", "canon1", "canon2", "w_in", "offs", "w_o",
                  "kv_norm", "w_uk", "w_uv", "w_kb", "conv_w", "A_log", "dt_bias", "out_norm",
-                 "router", "correction", "w_gate", "w_up", "w_down")
+                 "router", "correction", "w_gate", "w_up", "w_down", "w_out", "lam")
 
     def __init__(self) -> None:
         for s in self.__slots__:
@@ -91,10 +104,35 @@ class HybridWeights:
             return out.view(Hp, heads * pad8(vdim))
 
         W = HybridWeights(cfg)
+        def attention(m: AttentionSpec, x: str, L: HybridLayer) -> None:
+            L.w_in, L.offs = fuse([("q", t(x + "q", (m.q_channels, H))), ("k", t(x + "k", (m.k_channels, H))), ("v", t(x + "v", (m.v_channels, H)))])
+            if m.conv:
+                L.conv_w = torch.cat([f(x + n + ".conv") for n in ("q", "k", "v")])
+                if tuple(L.conv_w.shape) != (m.conv_channels, m.conv):
+                    raise ValueError(f"{x}*.conv: {tuple(L.conv_w.shape)}, the configuration says {(m.conv_channels, m.conv)}")
+                L.conv_w = L.conv_w.T.contiguous()
+            L.lam = 0.0
+            if m.maps == 2:
+                q1, k1, q2, k2 = (get(x + n).double() for n in ("lq1", "lk1", "lq2", "lk2"))
+                L.lam = float((q1 * k1).sum().exp() - (q2 * k2).sum().exp()) + m.diff
+
         W.embed, W.final_norm, W.lm_head = t("embed", (cfg.vocab_size, H)), t("final.norm", (H,)), reads(t("head", (cfg.vocab_size, H)))
         for i, spec in enumerate(cfg.layer_specs):
             pre, m, r, L = f"l{i}.", spec.mixer, spec.router, HybridLayer()
             x = pre + "mix."
+            if spec.parallel:
+                L.norm1 = t(pre + "norm1", (H,))
+                attention(m, x, L)
+                L.w_out, d = heads_o(x + "o", m.heads, m.vdim), spec.dense
+                if d is not None:
+                    y, F = pre + "mlp.", pad8(d.ffn)
+                    L.w_gate, L.w_up = (torch.zeros(F, Hp, dtype=dt, device=device) for _ in range(2))
+                    L.w_gate[:d.ffn, :H], L.w_up[:d.ffn, :H] = t(y + "gate", (d.ffn, H)), t(y + "up", (d.ffn, H))
+                    down = torch.zeros(Hp, F, dtype=dt, device=device)
+                    down[:H, :d.ffn] = t(y + "down", (H, d.ffn))
+                    L.w_out = torch.cat([L.w_out, down], 1).contiguous()
+                W.layers.append(L)
+                continue
             L.norm1, L.norm1b = t(pre + "norm1", (H,)), t(pre + "norm1b", (H,))
             L.canon1 = t(pre + "canon1", (H, cfg.canon_taps)).T.contiguous()
             if isinstance(m, LatentSpec):
@@ -145,7 +183,7 @@ class HybridWeights:
         def get(name: str) -> torch.Tensor:
             shape = shapes[name]
             if name.rsplit(".", 1)[-1].startswith("norm"):
-                return torch.ones(shape, device=device)
+                return torch.full(shape, 1.0 - cfg.norm_offset, device=device)
             s = 0.3 if "conv" in name or "canon" in name else std
             x = torch.empty(shape, dtype=torch.float32, device=device).normal_(0.0, s, generator=g)
             return x - 3.0 if name.endswith("dt_bias") else x
@@ -159,6 +197,18 @@ def tensor_shapes(cfg: ModelConfig) -> dict[str, tuple]:
     for i, spec in enumerate(cfg.layer_specs):
         pre, m, r = f"l{i}.", spec.mixer, spec.router
         x = pre + "mix."
+        if spec.parallel:
+            out[pre + "norm1"], out[x + "o"] = (H,), (H, m.heads * m.vdim)
+            for n, c in (("q", m.q_channels), ("k", m.k_channels), ("v", m.v_channels)):
+                out[x + n] = (c, H)
+                if m.conv:
+                    out[x + n + ".conv"] = (c, m.conv)
+            if m.maps == 2:
+                out.update({x + n: (m.dim,) for n in ("lq1", "lk1", "lq2", "lk2")})
+            if spec.dense is not None:
+                d = spec.dense.ffn
+                out.update({pre + "mlp.gate": (d, H), pre + "mlp.up": (d, H), pre + "mlp.down": (H, d)})
+            continue
         out.update({pre + "norm1": (H,), pre + "norm1b": (H,), pre + "canon1": (H, cfg.canon_taps), x + "o": (H, m.heads * m.vdim),
                     x + "g": (m.heads * m.vdim, H)})
         if isinstance(m, LatentSpec):
@@ -185,28 +235,38 @@ def tensor_core_latent(cfg: ModelConfig, m: LatentSpec) -> bool:
 
 
 class HybridCache:
-    """Paged latent records of the latent attention layers and the slot pool of everything recurrent.
+    """Paged records of the attention layers and the slot pool of everything recurrent, per layer run.
 
-    ``c``: one pool [pages, 64, record] per latent layer (page 0 stays zero).  ``state`` [slots, floats] fp32: slot 0 is
-    the zero state every sequence starts from, slot 1 takes the writes of dummy steps."""
+    ``c``: one pool [pages, 64, record] per run of a latent layer; ``k`` / ``v``: [pages, kv heads, 64, width] per run of an
+    attention layer (page 0 stays zero).  ``of_run``: a run's pool or (K, V) pools.  ``state`` [slots, floats] fp32: slot 0 is
+    the zero state every sequence starts from, slot 1 takes the writes of dummy steps; ``offsets`` names a run's parts."""
 
     def __init__(self, cfg: ModelConfig, num_pages: int, device: torch.device, state_slots: int = 34):
         dt = engine_dtype(cfg)
         self.num_pages = num_pages
         self.c: list[torch.Tensor] = []
-        self.of_layer: dict[int, torch.Tensor] = {}
+        self.k: list[torch.Tensor] = []
+        self.v: list[torch.Tensor] = []
+        self.of_run: dict = {}
         self.offsets: list[dict[str, int]] = []
         n = 0
-        for i, spec in enumerate(cfg.layer_specs):
+        for i, run in enumerate(cfg.layer_runs):
+            spec = cfg.layer_specs[run.layer]
             m, off = spec.mixer, {}
-            parts = [("canon1", (cfg.canon_taps - 1) * cfg.hidden)]
+            parts = [] if spec.parallel else [("canon1", (cfg.canon_taps - 1) * cfg.hidden)]
             if spec.router is not None:
                 parts.append(("canon2", (cfg.canon_taps - 1) * cfg.hidden))
             if isinstance(m, DeltaSpec):
                 parts += [("S", m.heads * m.dim * m.vdim), ("conv", (m.conv - 1) * m.conv_channels)]
+            elif isinstance(m, AttentionSpec):
+                parts.append(("conv", max(0, m.conv - 1) * m.conv_channels))
+                kv = [torch.zeros(num_pages, m.kv_heads, PAGE, w, dtype=dt, device=device) for w in (m.maps * m.dim, m.vdim)]
+                self.of_run[i] = tuple(kv)
+                self.k.append(kv[0])
+                self.v.append(kv[1])
             else:
-                self.of_layer[i] = torch.zeros(num_pages, PAGE, record_pitch(m), dtype=dt, device=device)
-                self.c.append(self.of_layer[i])
+                self.of_run[i] = torch.zeros(num_pages, PAGE, record_pitch(m), dtype=dt, device=device)
+                self.c.append(self.of_run[i])
             for name, size in parts:
                 off[name] = n
                 n += -(-size // 32) * 32
@@ -218,10 +278,10 @@ class HybridCache:
         return self.state.shape[0]
 
     def bytes_per_page(self) -> int:
-        return sum(t[0].numel() * t.element_size() for t in self.c)
+        return sum(t[0].numel() * t.element_size() for t in self.c + self.k + self.v)
 
     def copy_page(self, src: int, dst: int) -> None:
-        for c in self.c:
+        for c in self.c + self.k + self.v:
             c[dst].copy_(c[src])
 
 
@@ -238,6 +298,16 @@ class _LatentWs:
         i = torch.arange(0, m.rot_dim, 2, dtype=torch.float64)
         self.inv_freq = (m.rope_base ** (-i / max(1, m.rot_dim))).float().to(device)
         self.lat = self.k_exp = self.v_exp = None      # expanded-form prompts: made on first use
+
+
+class _AttnWs:
+    """Workspaces of the attention layers of one shape; ``table`` is shared by all that rotate alike."""
+
+    def __init__(self, cfg: ModelConfig, m: AttentionSpec, max_tokens: int, device: torch.device, tables: dict):
+        self.q = torch.zeros(max_tokens, m.q_channels, dtype=engine_dtype(cfg), device=device)
+        if m.rope not in tables:
+            tables[m.rope] = (rope_frequencies(m.rope).to(device), torch.zeros(max_tokens, max(1, m.rope.dims // 2), 2, device=device))
+        self.table = tables[m.rope][1]
 
 
 class HybridEngine:
@@ -269,6 +339,8 @@ class HybridEngine:
         outs = max((s.router.outputs for s in cfg.layer_specs if s.router), default=1)
         ws.router = torch.empty(max_tokens * outs, dtype=torch.float32, device=dev)
         self._lat: dict[LatentSpec, _LatentWs] = {}
+        self._attn: dict[AttentionSpec, _AttnWs] = {}
+        self._rope: dict[RopeSpec, tuple] = {}       # frequencies, the step's table
         self._delta: dict[DeltaSpec, torch.Tensor] = {}
         self._moe: dict = {}
         raw = scratch = 0
@@ -277,6 +349,9 @@ class HybridEngine:
             if isinstance(m, LatentSpec):
                 if m not in self._lat:
                     self._lat[m] = _LatentWs(cfg, m, max_tokens, dev)
+            elif isinstance(m, AttentionSpec):
+                if m not in self._attn:
+                    self._attn[m] = _AttnWs(cfg, m, max_tokens, dev, self._rope)
             else:
                 if m not in self._delta:
                     self._delta[m] = torch.zeros(max_tokens, m.heads, pad8(m.vdim), dtype=dt, device=dev)
@@ -289,6 +364,9 @@ class HybridEngine:
                     scratch = max(scratch, per * min(chunks, max_tokens // 64 + max_seqs))
             if r is not None and r not in self._moe:
                 self._moe[r] = LocalExchange(ExchangeGeometry(Hp, pad8(r.ffn), r.experts, r.top, max_tokens, 1), dev, dtype=dt)
+        # rows of a parallel layer's second product: the heads' values, then the feed-forward's activations
+        act = max((L.w_out.shape[1] for L in weights.layers if L.w_out is not None), default=0)
+        ws.act = torch.zeros(max_tokens * act, dtype=dt, device=dev) if act else None
         ws.raw = torch.empty(max_tokens * raw, dtype=torch.float32, device=dev) if raw else None
         ws.chunk = torch.empty(scratch, dtype=torch.uint8, device=dev) if scratch else None
         self.moe = None
@@ -306,14 +384,16 @@ class HybridEngine:
         self._pending: dict = {}
 
     # ---- between sublayers ------------------------------------------------------------------------------------------
-    def _between(self, b: Batch, T: int, w: torch.Tensor, conv: torch.Tensor, off: int) -> torch.Tensor:
+    def _between(self, b: Batch, T: int, w: torch.Tensor, conv: torch.Tensor | None, off: int = 0, add_embedding: bool = False) -> torch.Tensor:
         """Residual, norms and input convolution up to the next sublayer; returns its input rows."""
         ws, p = self.ws, self._pending
         h = ws.h[self._hi][:T]
-        src = dict(tokens=b.tokens, embed=self.W.embed) if self._x is None else dict(x_in=self._x)
+        src = {} if self._x is None else dict(x_in=self._x)
+        if self._x is None or add_embedding:
+            src.update(tokens=b.tokens, embed=self.W.embed)
         xo = ws.x[0 if self._x is None or self._x.data_ptr() != ws.x[0].data_ptr() else 1][:T]
         K.norm_conv(h, w, self.cfg.norm_groups, self.cfg.rms_eps, conv=conv, x_out=xo, state=self.kv.state, state_off=off,
-                    state_in=b.state_in, state_out=b.state_out, q_start=b.q_start, **src, **p)
+                    state_in=b.state_in, state_out=b.state_out, q_start=b.q_start, w_offset=self.cfg.norm_offset, **src, **p)
         self._x, self._hi = xo, self._hi ^ 1
         self.launches += 1
         return h
@@ -329,6 +409,8 @@ class HybridEngine:
                 w, idx, n, ident = p["slots"]
                 rows = torch.where((idx >= n)[..., None], ident[:, :H].float()[:, None], y[:T * w.shape[1]].view(T, w.shape[1], -1))
                 y = (w[..., None] * rows).sum(1)
+            if p.get("w_b") is None:
+                return x + y
             g = y.view(T, G, -1)
             x = x + (g / torch.sqrt((g * g).mean(-1, keepdim=True) + self.cfg.rms_eps)).view(T, -1) * p["w_b"]
         return x
@@ -348,10 +430,10 @@ class HybridEngine:
             self._blocks[key] = (torch.arange(S, **i32).repeat_interleave(nb).contiguous(), (torch.arange(nb, **i32) * per).repeat(S).contiguous())
         return self._blocks[key]
 
-    def _latent(self, i: int, m: LatentSpec, h: torch.Tensor, T: int, b: Batch) -> None:
+    def _latent(self, n: int, i: int, m: LatentSpec, h: torch.Tensor, T: int, b: Batch) -> None:
         L, ws, lw = self.W.layers[i], self.ws, self._lat[m]
         a = self._project(i, h, T)
-        cache = self.kv.of_layer[i]
+        cache = self.kv.of_run[n]
         key = (T, m.heads)
         if key not in self._tiles:
             self._tiles[key] = _HeadTiles(T, m.heads, self.device)
@@ -420,10 +502,31 @@ class HybridEngine:
                         self._scratch if splits > 1 else None, out_tpad=t_pad, window=m.window)
         self.launches += 1 if splits > 1 else 0
 
-    def _delta_mixer(self, i: int, m: DeltaSpec, h: torch.Tensor, T: int, b: Batch) -> None:
+    def _attention(self, n: int, i: int, m: AttentionSpec, h: torch.Tensor, T: int, b: Batch, out: torch.Tensor) -> None:
+        """Attention of layer run n; head h's values go to columns [h * pad8(vdim), + vdim) of ``out``."""
+        L, aw = self.W.layers[i], self._attn[m]
+        a = self._project(i, h, T)
+        (k, v), q = self.kv.of_run[n], aw.q[:T]
+        K.conv_rope_kv(a, L.offs, m, L.conv_w, aw.table, b.slots, q, k, v, state=self.kv.state, state_off=self.kv.offsets[n]["conv"],
+                       state_in=b.state_in, state_out=b.state_out, q_start=b.q_start)
+        K.paged_attn(q, k, v, m, b.page_table, b.positions, b.q_start, out, pad8(m.vdim), L.lam, self.cfg.rms_eps)
+        self.launches += 2
+
+    def _parallel(self, n: int, i: int, spec, h: torch.Tensor, T: int, b: Batch) -> None:
+        """Mixer and feed-forward on the same rows; one product over both reads their outputs side by side."""
+        L, m = self.W.layers[i], spec.mixer
+        act = self.ws.act[:T * L.w_out.shape[1]].view(T, L.w_out.shape[1])
+        self._attention(n, i, m, h, T, b, act)
+        if spec.dense is not None:
+            K.linear(h, L.w_gate, out=act[:, m.heads * pad8(m.vdim):], w_up=L.w_up)
+            self.launches += 1
+        K.linear(act, L.w_out, out=self.ws.y[:T])
+        self.launches += 1
+
+    def _delta_mixer(self, n: int, i: int, m: DeltaSpec, h: torch.Tensor, T: int, b: Batch) -> None:
         L, ws = self.W.layers[i], self.ws
         a = self._project(i, h, T)
-        off, out = self.kv.offsets[i], self._delta[m][:T]
+        off, out = self.kv.offsets[n], self._delta[m][:T]
         args = (a, L.offs, m, L, self.kv.state, off["S"], off["conv"], b.state_in, b.state_out, b.q_start, out, ws.raw, self.cfg.rms_eps)
         if b.prefill and b.max_q_len >= self.CHUNKED_DELTA_TOKENS and K.delta_chunk_ok(m, self.dtype):
             K.delta_chunked(ws.chunk, *args)
@@ -460,20 +563,31 @@ class HybridEngine:
         if b.embeds is not None:
             raise ValueError("media rows are not part of this family")
         self._x, self._hi, self._pending = None, 0, {}
-        for i, spec in enumerate(self.cfg.layer_specs):
-            L, off, m, r = self.W.layers[i], self.kv.offsets[i], spec.mixer, spec.router
+        for r, (freq, table) in self._rope.items():
+            if r.dims:
+                K.rope_table(b.positions, freq, table.view(-1)[:T * r.dims])
+                self.launches += 1
+        for n, run in enumerate(self.cfg.layer_runs):
+            i, spec = run.layer, self.cfg.layer_specs[run.layer]
+            L, off, m, r = self.W.layers[i], self.kv.offsets[n], spec.mixer, spec.router
+            if spec.parallel:
+                self._parallel(n, i, spec, self._between(b, T, L.norm1, None, add_embedding=run.add_embedding), T, b)
+                self._pending = dict(y=self.ws.y[:T])
+                if self.layer_hook is not None:
+                    self.layer_hook(n, self.residual(T))
+                continue
             h = self._between(b, T, L.norm1, L.canon1, off["canon1"])
             if isinstance(m, LatentSpec):
-                self._latent(i, m, h, T, b)
+                self._latent(n, i, m, h, T, b)
             else:
-                self._delta_mixer(i, m, h, T, b)
+                self._delta_mixer(n, i, m, h, T, b)
             self._pending = dict(y=self.ws.y[:T], w_b=L.norm1b)
             if r is not None:
                 h = self._between(b, T, L.norm2, L.canon2, off["canon2"])
                 slots = self._experts(i, r, h, T)
                 self._pending = dict(y=self._moe[r].att.combine, w_b=L.norm2b, slots=slots)
             if self.layer_hook is not None:
-                self.layer_hook(i, self.residual(T))
+                self.layer_hook(n, self.residual(T))
         return T
 
     def head(self, T: int, rows: torch.Tensor | None = None) -> torch.Tensor:
@@ -482,9 +596,14 @@ class HybridEngine:
         xn = self.ws.h[self._hi][:n]
         if rows is not None and rows.dtype != torch.int32:
             rows = rows.to(torch.int32)
-        K.norm_conv(xn, self.W.final_norm, self.cfg.norm_groups, self.cfg.rms_eps, x_in=self._x, rows=rows, **self._pending)
+        K.norm_conv(xn, self.W.final_norm, self.cfg.norm_groups, self.cfg.rms_eps, x_in=self._x, rows=rows, w_offset=self.cfg.norm_offset,
+                    **self._pending)
         self.launches += 2
-        return K.linear(xn, self.W.lm_head, out=self.logits[:n], out_f32=True)
+        out = K.linear(xn, self.W.lm_head, out=self.logits[:n], out_f32=True)
+        if self.cfg.logit_softcap:
+            K.softcap(out, self.cfg.logit_softcap)
+            self.launches += 1
+        return out
 
     def forward(self, b: Batch) -> torch.Tensor:
         return self.head(self.layers(b), b.last_rows)

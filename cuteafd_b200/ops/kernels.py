@@ -668,14 +668,15 @@ def mla_unabsorb_small(o_lat: torch.Tensor, w_uv: torch.Tensor, attn: torch.Tens
              "mla_unabsorb_small")
 
 
-# ---- per-layer hybrids (csrc/hybrid_norm.cu, latent.cu, delta.cu) --------------------------------------------
+# ---- per-layer hybrids (csrc/hybrid_norm.cu, latent.cu, delta.cu, conv_rope.cu, attention_any.cu) --------------------------------------------
 def norm_conv(h_out: torch.Tensor, w: torch.Tensor, groups: int, eps: float, *, tokens: torch.Tensor | None = None,
               embed: torch.Tensor | None = None, x_in: torch.Tensor | None = None, y: torch.Tensor | None = None,
               w_b: torch.Tensor | None = None, slots: tuple | None = None, conv: torch.Tensor | None = None,
               x_out: torch.Tensor | None = None, rows: torch.Tensor | None = None, state: torch.Tensor | None = None, state_off: int = 0,
               state_in: torch.Tensor | None = None, state_out: torch.Tensor | None = None, q_start: torch.Tensor | None = None,
-              run: int = 0) -> None:
-    """Weights are in the activations' type.  x = embed[tokens] or ``x_in`` (fp32); x += groupnorm(y) * w_b; h = groupnorm(x) * w; h_out = h + causal_conv(h).
+              run: int = 0, w_offset: float = 0.0) -> None:
+    """Weights are in the activations' type.  x = embed[tokens], ``x_in`` (fp32) or, given both, their sum; x += groupnorm(y) * w_b
+    (without ``w_b``: x += y); h = groupnorm(x) * (w + ``w_offset``); h_out = h + causal_conv(h).
 
     Rows of ``h_out``, ``y`` and the identity rows may be longer than H (whole 16-byte pieces); the rest is left alone.
     ``slots`` = (weights [T, k], ids [T, k], number of experts, identity rows): ``y`` then holds the routed experts' rows
@@ -686,7 +687,7 @@ def norm_conv(h_out: torch.Tensor, w: torch.Tensor, groups: int, eps: float, *, 
     a.tokens, a.embed, a.x_in, a.y = _ptr(tokens), _ptr(embed), _ptr(x_in), _ptr(y)
     a.w_b, a.w, a.conv, a.x_out, a.h_out, a.row_idx = _ptr(w_b), w.data_ptr(), _ptr(conv), _ptr(x_out), h_out.data_ptr(), _ptr(rows)
     a.vocab = embed.shape[0] if embed is not None else 0
-    a.T, a.H, a.groups, a.eps, a.run = h_out.shape[0], H, groups, eps, run
+    a.T, a.H, a.groups, a.eps, a.run, a.w_off = h_out.shape[0], H, groups, eps, run, w_offset
     a.ldy, a.ldh = y.stride(0) if y is not None else 0, h_out.stride(0)
     assert h_out.shape[1] >= H and h_out.stride(1) == 1 and w.dtype == h_out.dtype and (w_b is None or w_b.dtype == h_out.dtype)
     if slots is not None:
@@ -703,6 +704,57 @@ def norm_conv(h_out: torch.Tensor, w: torch.Tensor, groups: int, eps: float, *, 
 
 def swap_ids(a: torch.Tensor, b: torch.Tensor) -> None:
     _n.check(_n.cuda_lib().cafd_swap_ids(a.data_ptr(), b.data_ptr(), a.numel(), _stream()), "swap_ids")
+
+
+def rope_table(positions: torch.Tensor, freq: torch.Tensor, out: torch.Tensor) -> None:
+    """out [T, half, 2] fp32 = cos, sin of positions [T] * freq [half]."""
+    T, half = positions.shape[0], freq.shape[0]
+    assert out.is_contiguous() and out.numel() == 2 * T * half
+    _n.check(_n.cuda_lib().cafd_rope_table(positions.data_ptr(), freq.data_ptr(), out.data_ptr(), T, half, _stream()), "rope_table")
+
+
+def conv_rope_kv(proj: torch.Tensor, offs: dict, m, conv_w: torch.Tensor | None, table: torch.Tensor, slots: torch.Tensor, q_out: torch.Tensor,
+                 k_cache: torch.Tensor, v_cache: torch.Tensor, *, state: torch.Tensor | None = None, state_off: int = 0,
+                 state_in: torch.Tensor | None = None, state_out: torch.Tensor | None = None, q_start: torch.Tensor | None = None) -> None:
+    """Convolution over time, rotation and the paged K / V write of one step.  ``m`` carries heads / kv_heads / maps / dim / vdim and
+    rope.dims, ``conv_w`` [taps, channels] fp32 (last row = the current token), ``table`` the step's ``rope_table``."""
+    p = _n.ConvRope()
+    p.proj, p.conv_w, p.table, p.slots, p.q_start = proj.data_ptr(), _ptr(conv_w), table.data_ptr(), slots.data_ptr(), _ptr(q_start)
+    p.q_out, p.k_cache, p.v_cache = q_out.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr()
+    p.T, p.ld, p.q_off, p.k_off, p.v_off = proj.shape[0], proj.stride(0), offs["q"], offs["k"], offs["v"]
+    p.nq, p.nk, p.nv = m.heads * m.maps * m.dim, m.kv_heads * m.maps * m.dim, m.kv_heads * m.vdim
+    p.maps_dim, p.dim, p.vdim, p.kv_heads, p.rot = m.maps * m.dim, m.dim, m.vdim, m.kv_heads, m.rope.dims
+    assert q_out.is_contiguous() and k_cache.is_contiguous() and v_cache.is_contiguous() and q_out.dtype == proj.dtype == k_cache.dtype == v_cache.dtype
+    assert q_out.numel() >= p.T * p.nq and k_cache.shape[1:] == (m.kv_heads, 64, p.maps_dim) and v_cache.shape[1:] == (m.kv_heads, 64, m.vdim)
+    if conv_w is not None:
+        p.taps, p.S = conv_w.shape[0], q_start.shape[0] - 1
+        assert conv_w.is_contiguous() and conv_w.dtype == torch.float32 and conv_w.shape[1] == p.nq + p.nk + p.nv
+        p.state, p.state_in, p.state_out = state.data_ptr(), state_in.data_ptr(), state_out.data_ptr()
+        p.slot_stride, p.state_off = state.stride(0), state_off
+    _n.check(_n.cuda_lib().cafd_conv_rope_kv(C.byref(p), int(proj.dtype == torch.float32), _stream()), "conv_rope_kv")
+
+
+def paged_attn(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, m, page_table: torch.Tensor, positions: torch.Tensor,
+               q_start: torch.Tensor, out: torch.Tensor, head_pitch: int, lam: float = 0.0, eps: float = 0.0) -> None:
+    """Attention at any head sizes: q [T, heads * maps * dim]; head h's values go to columns [h * head_pitch, + vdim) of ``out``
+    (rows of any length).  ``m``: an ``AttentionSpec``; ``lam`` / ``eps``: second map's weight and the head norm's epsilon."""
+    p = _n.PagedAttn()
+    p.q, p.k_cache, p.v_cache, p.page_table = q.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(), page_table.data_ptr()
+    p.positions, p.q_start, p.out = positions.data_ptr(), q_start.data_ptr(), out.data_ptr()
+    p.T, p.heads, p.kv_heads, p.maps, p.dim, p.vdim = q.shape[0], m.heads, m.kv_heads, m.maps, m.dim, m.vdim
+    p.S, p.max_pages = page_table.shape
+    p.window, p.keep, p.ldo, p.head_pitch = m.window, m.keep_first, out.stride(0), head_pitch
+    p.scale, p.lam, p.out_scale, p.eps = m.scale, lam, 1.0 - m.diff, eps
+    assert q.is_contiguous() and q.dtype == out.dtype == k_cache.dtype and page_table.is_contiguous() and q_start.shape[0] == p.S + 1
+    assert k_cache.is_contiguous() and v_cache.is_contiguous() and k_cache.shape[1:] == (m.kv_heads, 64, m.maps * m.dim)
+    _n.check(_n.cuda_lib().cafd_paged_attn(C.byref(p), int(q.dtype == torch.float32), _stream()), "paged_attn")
+
+
+def softcap(x: torch.Tensor, cap: float) -> torch.Tensor:
+    """x = cap * tanh(x / cap) in place; x [rows, n] fp32 (rows of any pitch)."""
+    assert x.dtype == torch.float32 and x.stride(1) == 1
+    _n.check(_n.cuda_lib().cafd_softcap(x.data_ptr(), x.shape[0], x.shape[1], x.stride(0), cap, _stream()), "softcap")
+    return x
 
 
 def latent_prep(a: torch.Tensor, q_off: int, kv_off: int, heads: int, dim: int, rot: int, norm_w: torch.Tensor, inv_freq: torch.Tensor,
