@@ -8,6 +8,12 @@
 //   each warp owns 16 of the 64 tokens of a page; per-warp online softmax; warps merged in
 //   shared memory; splits merged by a second kernel in split order (deterministic).
 //
+// With kMaps = 2 (differential attention: two 64-wide score maps per head over the same 128-wide values; query and key rows
+// hold [map 1 | map 2]) a tile's rows are (query token, head, map) and a row's query fragment is zero in the other map's half,
+// so the same products serve.  Map 1 - lambda * map 2, its norm over the head's values and a constant factor follow when the
+// row is complete: here without splits, in the merge with them.
+// A sliding window may come with kept first tokens; their pages are walked before the window's.
+//
 // Reference counterparts: split-KV partial + merge drafter attention
 // (native/shared/cuda/draft_attention.cu:42-295) and the LSE state merge
 // (native/shared/cuda/attention.cu:925).
@@ -65,16 +71,34 @@ struct AttnPeers {
   int n, split_offset, total_splits;
 };
 
+// Kept first tokens, output row pitch and, with two maps, how they are combined.
+struct AttnExtras {
+  int keep, ldo;
+  float lambda, out_scale, eps;
+};
+
+// The combined value of one head's 128 values, one per thread: a - lambda * b over its root mean square, times out_scale.
+__device__ __forceinline__ float combine_maps(float a, float b, const AttnExtras& x, float* red) {
+  const float o = a - x.lambda * b;
+  const float ss = warp_sum(o * o);
+  if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = ss;
+  __syncthreads();
+  const float tot = (red[0] + red[1]) + (red[2] + red[3]);
+  __syncthreads();
+  return o * (x.out_scale / sqrtf(tot * (1.0f / kD) + x.eps));
+}
+
+template <int kMaps>
 __global__ void __launch_bounds__(128) attn_decode_kernel(
     const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __restrict__ k_cache,
     const __nv_bfloat16* __restrict__ v_cache, const int* __restrict__ page_table, const int* __restrict__ seq_lens,
     const int* __restrict__ q_start, __nv_bfloat16* __restrict__ out, float* __restrict__ partial, int max_pages,
     int Hq, int Hkv, int tiles_per_seq, int splits, float scale_log2, const int* __restrict__ kv_base, int window, int split_pages,
-    const AttnPeers peers) {
+    const AttnPeers peers, const AttnExtras ex) {
   pdl_wait();
   pdl_trigger();
   extern __shared__ __align__(128) uint8_t smem[];
-  const int group = Hq / Hkv;
+  const int group = kMaps * (Hq / Hkv);          // rows per query token
   const int q_per_tile = 16 / group;
   const int seq = blockIdx.x / tiles_per_seq;
   const int qt = blockIdx.x % tiles_per_seq;
@@ -106,11 +130,12 @@ __global__ void __launch_bounds__(128) attn_decode_kernel(
     const bool valid = qi < q_len;
     limit[half] = valid ? min(seq_len, base_vis + qi + 1) : 0;
     lo[half] = !valid ? 0x7fffffff : (window > 0 ? max(0, limit[half] - window) : 0);
-    const __nv_bfloat16* qrow = q + (static_cast<size_t>(q0 + (valid ? qi : 0)) * Hq + kvh * group + r % group) * kD;
+    const __nv_bfloat16* qrow = q + (static_cast<size_t>(q0 + (valid ? qi : 0)) * Hq + kvh * (group / kMaps) + (r % group) / kMaps) * kD;
 #pragma unroll
     for (int ks = 0; ks < 8; ++ks) {
-      qa[ks][half] = valid ? *reinterpret_cast<const uint32_t*>(qrow + 16 * ks + 2 * t4) : 0u;
-      qa[ks][half + 2] = valid ? *reinterpret_cast<const uint32_t*>(qrow + 16 * ks + 8 + 2 * t4) : 0u;
+      const bool on = valid && (kMaps == 1 || (ks >> 2) == (r & 1));
+      qa[ks][half] = on ? *reinterpret_cast<const uint32_t*>(qrow + 16 * ks + 2 * t4) : 0u;
+      qa[ks][half + 2] = on ? *reinterpret_cast<const uint32_t*>(qrow + 16 * ks + 8 + 2 * t4) : 0u;
     }
   }
   int max_limit = limit[0] > limit[1] ? limit[0] : limit[1];
@@ -120,13 +145,17 @@ __global__ void __launch_bounds__(128) attn_decode_kernel(
 #pragma unroll
   for (int o = 16; o > 0; o >>= 1) min_lo = min(min_lo, __shfl_xor_sync(0xffffffffu, min_lo, o));
 
-  // pages [first_page, total_pages) hold every position some row of the tile sees; the splits share them
+  // pages [0, kept) and [first_page, total_pages) hold every position some row of the tile sees; the splits share them
   const int total_pages = (max_limit + kPage - 1) / kPage;
   const int first_page = min(min_lo / kPage, total_pages);
+  const int kept = min((ex.keep + kPage - 1) / kPage, first_page);
+  const int gap = first_page - kept;             // page of ordinal i: i + (i < kept ? 0 : gap)
+  const int n_pages = total_pages - gap;
   // split_pages > 0: split s owns pages [s * split_pages, (s + 1) * split_pages) of every sequence, whatever the step holds
-  const int per_split = split_pages > 0 ? split_pages : (total_pages - first_page + splits - 1) / splits;
-  const int p0 = split_pages > 0 ? max(first_page, split * split_pages) : first_page + split * per_split;
-  const int p1 = min(total_pages, (split_pages > 0 ? split * split_pages : p0) + per_split);
+  auto ordinal = [&](int page) { return page <= kept ? page : max(kept, page - gap); };   // visible pages before `page`
+  const int per_split = (n_pages + splits - 1) / splits;
+  const int p0 = split_pages > 0 ? min(n_pages, ordinal(split * split_pages)) : split * per_split;
+  const int p1 = min(n_pages, split_pages > 0 ? ordinal((split + 1) * split_pages) : p0 + per_split);
 
   float m_run[2] = {-INFINITY, -INFINITY};
   float l_run[2] = {0.f, 0.f};
@@ -137,17 +166,20 @@ __global__ void __launch_bounds__(128) attn_decode_kernel(
     for (int j = 0; j < 4; ++j) o_acc[i][j] = 0.f;
 
   const int* pt = page_table + static_cast<size_t>(seq) * max_pages;
+  auto page_at = [&](int i) { return i + (i < kept ? 0 : gap); };
   if (p0 < p1) {
-    load_page(smem, k_cache, pt[p0], kvh, Hkv);
-    load_page(smem + kTileBytes, v_cache, pt[p0], kvh, Hkv);
+    const int first = pt[page_at(p0)];
+    load_page(smem, k_cache, first, kvh, Hkv);
+    load_page(smem + kTileBytes, v_cache, first, kvh, Hkv);
   }
   cp_async_commit();
   for (int p = p0; p < p1; ++p) {
     const int stage = (p - p0) & 1;
     if (p + 1 < p1) {
       uint8_t* nxt = smem + (stage ^ 1) * 2 * kTileBytes;
-      load_page(nxt, k_cache, pt[p + 1], kvh, Hkv);
-      load_page(nxt + kTileBytes, v_cache, pt[p + 1], kvh, Hkv);
+      const int page = pt[page_at(p + 1)];
+      load_page(nxt, k_cache, page, kvh, Hkv);
+      load_page(nxt + kTileBytes, v_cache, page, kvh, Hkv);
     }
     cp_async_commit();
     cp_async_wait<1>();
@@ -170,7 +202,7 @@ __global__ void __launch_bounds__(128) attn_decode_kernel(
       }
     }
     // ---- mask + online softmax (rows g and g + 8) ---------------------------------------------
-    const int tok_base = p * kPage + warp * 16;
+    const int tok_base = page_at(p) * kPage + warp * 16;
     float mx[2] = {-INFINITY, -INFINITY};
 #pragma unroll
     for (int nt = 0; nt < 2; ++nt)
@@ -178,7 +210,7 @@ __global__ void __launch_bounds__(128) attn_decode_kernel(
       for (int j = 0; j < 4; ++j) {
         const int half = j >> 1;
         const int tok = tok_base + nt * 8 + 2 * t4 + (j & 1);
-        const float v = (tok < limit[half] && tok >= lo[half]) ? s[nt][j] * scale_log2 : -INFINITY;
+        const float v = (tok < limit[half] && (tok >= lo[half] || tok < ex.keep)) ? s[nt][j] * scale_log2 : -INFINITY;
         s[nt][j] = v;
         mx[half] = fmaxf(mx[half], v);
       }
@@ -243,7 +275,8 @@ __global__ void __launch_bounds__(128) attn_decode_kernel(
     sm_l[warp * 16 + g] = l_run[0]; sm_l[warp * 16 + g + 8] = l_run[1];
   }
   __syncthreads();
-  for (int i = threadIdx.x; i < 16 * kD; i += blockDim.x) {
+  float o_map1 = 0.f;                            // kMaps == 2, no splits: the head's first map, one value per thread
+  for (int i = threadIdx.x; i < 16 * kD; i += blockDim.x) {   // every iteration: row i / 128, value threadIdx.x
     const int r = i / kD, d = i % kD;
     float M = -INFINITY;
 #pragma unroll
@@ -264,8 +297,12 @@ __global__ void __launch_bounds__(128) attn_decode_kernel(
     } else if (splits == 1) {
       const int qi = first_q + r / group;
       if (qi < q_len) {
-        __nv_bfloat16* orow = out + (static_cast<size_t>(q0 + qi) * Hq + kvh * group + r % group) * kD;
-        orow[d] = __float2bfloat16(L > 0.f ? O / L : 0.f);
+        float v = L > 0.f ? O / L : 0.f;
+        if (kMaps == 2) {
+          if ((r & 1) == 0) { o_map1 = v; continue; }
+          v = combine_maps(o_map1, v, ex, sm_l + 64);
+        }
+        out[static_cast<size_t>(q0 + qi) * ex.ldo + (kvh * (group / kMaps) + (r % group) / kMaps) * kD + d] = __float2bfloat16(v);
       }
     } else {
       part[r * kD + d] = O;
@@ -274,31 +311,40 @@ __global__ void __launch_bounds__(128) attn_decode_kernel(
   }
 }
 
-// One block per (tile, kv head, row): thread d walks the splits in order for its output element.
+// One block per (tile, kv head, row; with two maps row pair): thread d walks the splits in order for its output element.
+template <int kMaps>
 __global__ void __launch_bounds__(128) attn_merge_kernel(const float* __restrict__ partial,
                                                          const int* __restrict__ q_start,
                                                          __nv_bfloat16* __restrict__ out, int Hq, int Hkv,
-                                                         int tiles_per_seq, int splits) {
+                                                         int tiles_per_seq, int splits, const AttnExtras ex) {
+  __shared__ float red[4];
   pdl_wait();
   pdl_trigger();
   const int group = Hq / Hkv;
-  const int q_per_tile = 16 / group;
+  const int q_per_tile = 16 / (group * kMaps);
   const int seq = blockIdx.x / tiles_per_seq, qt = blockIdx.x % tiles_per_seq, kvh = blockIdx.y, r = blockIdx.z;
   const int q0 = q_start[seq], q_len = q_start[seq + 1] - q0;
   const int qi = qt * q_per_tile + r / group;
   if (qi >= q_len) return;
   const int d = threadIdx.x;
   const float* base = partial + (static_cast<size_t>(blockIdx.x) * Hkv + kvh) * splits * kPartialFloats;
-  float M = -INFINITY;
-  for (int s = 0; s < splits; ++s) M = fmaxf(M, __ldg(base + s * kPartialFloats + 16 * kD + r));
-  float L = 0.f, O = 0.f;
-  for (int s = 0; s < splits; ++s) {
-    const float m = __ldg(base + s * kPartialFloats + 16 * kD + r);
-    const float f = (m == -INFINITY) ? 0.f : exp2f(m - M);
-    L += __ldg(base + s * kPartialFloats + 16 * kD + 16 + r) * f;
-    O += __ldg(base + s * kPartialFloats + r * kD + d) * f;
+  float v[kMaps];
+#pragma unroll
+  for (int m = 0; m < kMaps; ++m) {
+    const int row = r * kMaps + m;
+    float M = -INFINITY;
+    for (int s = 0; s < splits; ++s) M = fmaxf(M, __ldg(base + s * kPartialFloats + 16 * kD + row));
+    float L = 0.f, O = 0.f;
+    for (int s = 0; s < splits; ++s) {
+      const float mx = __ldg(base + s * kPartialFloats + 16 * kD + row);
+      const float f = (mx == -INFINITY) ? 0.f : exp2f(mx - M);
+      L += __ldg(base + s * kPartialFloats + 16 * kD + 16 + row) * f;
+      O += __ldg(base + s * kPartialFloats + row * kD + d) * f;
+    }
+    v[m] = L > 0.f ? O / L : 0.f;
   }
-  out[(static_cast<size_t>(q0 + qi) * Hq + kvh * group + r % group) * kD + d] = __float2bfloat16(L > 0.f ? O / L : 0.f);
+  const float o = kMaps == 2 ? combine_maps(v[0], v[kMaps - 1], ex, red) : v[0];
+  out[static_cast<size_t>(q0 + qi) * ex.ldo + (kvh * group + r % group) * kD + d] = __float2bfloat16(o);
 }
 
 }  // namespace cafd
@@ -318,16 +364,17 @@ extern "C" long long cafd_attn_decode_scratch_floats(int num_seqs, int tiles_per
   return static_cast<long long>(num_seqs) * tiles_per_seq * Hkv * splits * kPartialFloats;
 }
 
-// q [total_q, Hq, 128]; caches [pages, 64, Hkv, 128]; page_table [num_seqs, max_pages];
-// seq_lens [num_seqs] (kv length including the new tokens); q_start [num_seqs + 1].
-// max_q_len bounds the query tokens of any sequence; scratch holds the split partials.
+// q [total_q, Hq, 128] (two maps: [total_q, Hq, 2, 64]); caches [pages, Hkv, 64, 128]; page_table [num_seqs, max_pages];
+// seq_lens [num_seqs] (kv length including the new tokens); q_start [num_seqs + 1]; out rows of ldo elements, head h's values at
+// column 128 h.  max_q_len bounds the query tokens of any sequence; scratch holds the split partials.  keep: kept first tokens
+// beside a window; lambda, out_scale and eps: two maps only.
 extern "C" int cafd_attn_decode(const void* q, const void* k_cache, const void* v_cache, const int* page_table,
                                 const int* seq_lens, const int* q_start, void* out, float* scratch, int num_seqs,
                                 int max_q_len, int max_pages, int Hq, int Hkv, int D, int splits, float scale,
-                                int window, cafd_stream_t s) {
+                                int window, int keep, int ldo, int maps, float lambda, float out_scale, float eps, cafd_stream_t s) {
   if (num_seqs <= 0) return 0;
-  if (D != kD || Hq % Hkv || window < 0) return -10;
-  const int group = Hq / Hkv;
+  if (D != kD || Hq % Hkv || window < 0 || keep < 0 || maps < 1 || maps > 2 || ldo < Hq * kD) return -10;
+  const int group = maps * (Hq / Hkv);
   if (group > 16 || 16 % group) return -11;
   if (splits < 1) splits = 1;
   if (splits > 1 && !scratch) return -12;
@@ -339,19 +386,22 @@ extern "C" int cafd_attn_decode(const void* q, const void* k_cache, const void* 
   const int smem = 4 * kTileBytes;   // two stages of K+V; reused for the warp merge (needs 33 KiB)
   static bool attr = false;
   if (!attr) {
-    CAFD_CHECK_CUDA(cudaFuncSetAttribute(attn_decode_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
+    CAFD_CHECK_CUDA(cudaFuncSetAttribute(attn_decode_kernel<1>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
+    CAFD_CHECK_CUDA(cudaFuncSetAttribute(attn_decode_kernel<2>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
     attr = true;
   }
   dim3 grid(num_seqs * tiles_per_seq, Hkv, splits);
-  launch_pdl(attn_decode_kernel, grid, dim3(128), smem, st, 
+  const AttnExtras ex{window > 0 ? keep : 0, ldo, lambda, out_scale, eps};
+  auto kern = maps == 2 ? attn_decode_kernel<2> : attn_decode_kernel<1>;
+  launch_pdl(kern, grid, dim3(128), smem, st,
       static_cast<const __nv_bfloat16*>(q), static_cast<const __nv_bfloat16*>(k_cache),
       static_cast<const __nv_bfloat16*>(v_cache), page_table, seq_lens, q_start, static_cast<__nv_bfloat16*>(out),
       scratch, max_pages, Hq, Hkv, tiles_per_seq, splits, scale * 1.4426950408889634f, static_cast<const int*>(nullptr),
-      window, fixed_kv_split_tokens() / kPage, AttnPeers{});
+      window, fixed_kv_split_tokens() / kPage, AttnPeers{}, ex);
   if (splits > 1) {
-    dim3 g2(num_seqs * tiles_per_seq, Hkv, 16);
-    launch_pdl(attn_merge_kernel, g2, dim3(128), 0, st, scratch, q_start, static_cast<__nv_bfloat16*>(out), Hq, Hkv, tiles_per_seq,
-                                          splits);
+    dim3 g2(num_seqs * tiles_per_seq, Hkv, 16 / maps);
+    auto merge = maps == 2 ? attn_merge_kernel<2> : attn_merge_kernel<1>;
+    launch_pdl(merge, g2, dim3(128), 0, st, scratch, q_start, static_cast<__nv_bfloat16*>(out), Hq, Hkv, tiles_per_seq, splits, ex);
   }
   return static_cast<int>(cudaGetLastError());
 }
@@ -375,7 +425,7 @@ extern "C" int cafd_attn_decode_partial(const void* q, const void* k_cache, cons
   const int smem = 4 * kTileBytes;
   static bool attr = false;
   if (!attr) {
-    CAFD_CHECK_CUDA(cudaFuncSetAttribute(attn_decode_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
+    CAFD_CHECK_CUDA(cudaFuncSetAttribute(attn_decode_kernel<1>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
     attr = true;
   }
   AttnPeers peers{};
@@ -385,10 +435,10 @@ extern "C" int cafd_attn_decode_partial(const void* q, const void* k_cache, cons
   }
   peers.n = n_peers; peers.split_offset = my_rank * splits; peers.total_splits = n_peers * splits;
   dim3 grid(num_seqs * tiles_per_seq, Hkv, splits);
-  launch_pdl(attn_decode_kernel, grid, dim3(128), smem, st, static_cast<const __nv_bfloat16*>(q),
+  launch_pdl(attn_decode_kernel<1>, grid, dim3(128), smem, st, static_cast<const __nv_bfloat16*>(q),
              static_cast<const __nv_bfloat16*>(k_cache), static_cast<const __nv_bfloat16*>(v_cache), page_table, seq_lens, q_start,
              static_cast<__nv_bfloat16*>(nullptr), peers.scratch[my_rank], max_pages, Hq, Hkv, tiles_per_seq, splits,
-             scale * 1.4426950408889634f, kv_base, 0, 0, peers);
+             scale * 1.4426950408889634f, kv_base, 0, 0, peers, AttnExtras{0, Hq * kD});
   return static_cast<int>(cudaGetLastError());
 }
 
@@ -402,7 +452,7 @@ extern "C" int cafd_attn_merge(const float* scratch, const int* q_start, void* o
   const int q_per_tile = 16 / group;
   const int tiles_per_seq = (max_q_len + q_per_tile - 1) / q_per_tile;
   dim3 g2(num_seqs * tiles_per_seq, Hkv, 16);
-  launch_pdl(attn_merge_kernel, g2, dim3(128), 0, static_cast<cudaStream_t>(s), scratch, q_start, static_cast<__nv_bfloat16*>(out),
-             Hq, Hkv, tiles_per_seq, total_splits);
+  launch_pdl(attn_merge_kernel<1>, g2, dim3(128), 0, static_cast<cudaStream_t>(s), scratch, q_start, static_cast<__nv_bfloat16*>(out),
+             Hq, Hkv, tiles_per_seq, total_splits, AttnExtras{0, Hq * kD});
   return static_cast<int>(cudaGetLastError());
 }

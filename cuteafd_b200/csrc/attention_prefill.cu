@@ -20,6 +20,15 @@
 // is added to the scores with four more MMAs per tile, its keys read straight from the paged latent cache
 // (columns 512..575 of every record).  Query dims are then 128 + 64, value dims 128.
 //
+// With kMaps = 2 a head has two 64-wide score maps over the same 128-wide values (differential attention): query and key
+// rows hold [map 1 | map 2], exactly the two 64-wide halves of the Q and K tiles.  The pipeline then runs over units
+// (tile, map), maps alternating: S and P buffer = map, one O accumulator per map (TMEM: 2 x 128 + 2 x 128 columns), K and V
+// stages released by the tile's second unit.  The epilogue combines the maps: O1 / l1 - lambda O2 / l2, divided by its root
+// mean square over the head's values, times a constant.
+//
+// A sliding window may come with kept first tokens, which every later row sees too: the tiles that hold them are walked
+// before the window's.
+//
 // Replaces the reference's mma.sync prefill kernels (native/families/glm5/cuda/glm_mla_prefill.cu:78-135)
 // and its exported attention programs for the GQA families.
 #include "cafd_api.h"
@@ -48,6 +57,10 @@ struct PrefillDev {
   int Hq, Hkv;
   float scale_log2;
   int window;              // sliding window: a query at position t sees keys (t - window, t]; 0 = all earlier keys
+  int keep;                // with a window: and the keys [0, keep)
+  int ldo;                 // elements from row to row of out
+  // kMaps == 2 only
+  float lambda, out_scale, eps;
   // kRope only
   const int* kv_tmp_start; // [seqs] first row of the sequence in the expansion buffers (multiple of 64)
   int q_head_stride;       // elements between heads in the nope query matrix (192 for [T, heads * 192])
@@ -55,7 +68,7 @@ struct PrefillDev {
   int qr_col0;             // first rope column inside a head of that matrix (512)
 };
 
-template <bool kRope>
+template <bool kRope, int kMaps>
 __global__ void __launch_bounds__(kPrefillThreads, 1)
 attn_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ CUtensorMap tm_k,
                     const __grid_constant__ CUtensorMap tm_v, const __grid_constant__ CUtensorMap tm_qr,
@@ -94,9 +107,13 @@ attn_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_const
   const int row0 = qt * kBQ;                       // first query row of this tile (within the chunk)
   const int pos0 = kv_len - q_len + row0;          // its absolute position
   const int last_pos = min(pos0 + kBQ - 1, kv_len - 1);
-  // kv tiles [tile0, last_pos / kBKV]: with a sliding window the tiles wholly before the first row's window are skipped
-  const int tile0 = p.window > 0 ? max(0, pos0 - p.window + 1) / kBKV : 0;
+  // kv tiles: with a sliding window those wholly before the first row's window are skipped, except the first ones if they hold
+  // kept tokens
+  const int win_tile = p.window > 0 ? max(0, pos0 - p.window + 1) / kBKV : 0;
+  const int kept_tiles = p.window > 0 ? min((p.keep + kBKV - 1) / kBKV, win_tile) : 0;
+  const int tile0 = win_tile - kept_tiles;         // tile of ordinal j: j + (j < kept_tiles ? 0 : tile0)
   const int n_tiles = last_pos / kBKV + 1 - tile0;
+  const int n_units = n_tiles * kMaps;             // (tile, map) pairs
   const int seq_pages = (kv_len + kPageTok - 1) / kPageTok;
 
   if (threadIdx.x == 0) {
@@ -132,7 +149,7 @@ attn_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_const
       const int* pt = p.page_table + static_cast<size_t>(seq) * p.max_pages;
       const int tmp_page0 = kRope ? p.kv_tmp_start[seq] / kPageTok : 0;
       auto pages_of = [&](int jj, int& pa, int& pb, int& ka, int& kb) {
-        const int j = jj + tile0;
+        const int j = jj + (jj < kept_tiles ? 0 : tile0);
         pa = 2 * j < seq_pages ? pt[2 * j] : 0;                      // page 0 is the all-zero page
         pb = 2 * j + 1 < seq_pages ? pt[2 * j + 1] : 0;
         // expanded K / V (kRope) sit in order in their buffer: "page" = row block of 64; past the end TMA fills zeros
@@ -189,13 +206,21 @@ attn_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_const
       constexpr uint32_t idesc_pv = make_idesc(128, 128, 1, 1, 0, 1);   // B = V is MN-major
       const uint32_t aQ = smem_u32(sQ), aP = smem_u32(sP);
       bool ok = mbar_wait(&q_full, 0, p.status, kTimeoutFullBarrier);
-      auto issue_qk = [&](int j) -> bool {
-        const int st = j & 1;
-        const uint32_t ph = (j >> 1) & 1;
-        if (!mbar_wait(&k_full[st], ph, p.status, kTimeoutFullBarrier)) return false;
-        if (!mbar_wait(&s_empty[st], ph ^ 1, p.status, kTimeoutTmemEmpty)) return false;
+      auto issue_qk = [&](int u) -> bool {
+        const int j = u / kMaps, st = j & 1, sb = u & 1;
+        if ((kMaps == 1 || sb == 0) && !mbar_wait(&k_full[st], (j >> 1) & 1, p.status, kTimeoutFullBarrier)) return false;
+        if (!mbar_wait(&s_empty[sb], ((u >> 1) & 1) ^ 1, p.status, kTimeoutTmemEmpty)) return false;
         tc_fence_after();
         const uint32_t aK = smem_u32(sK + st * kTileB);
+        if (kMaps == 2) {
+#pragma unroll
+          for (int k4 = 0; k4 < 4; ++k4)
+            umma_f16(tS + sb * 128, smem_desc_k_sw128(aQ + sb * kHalfBytes + k4 * 32),
+                     smem_desc_k_sw128(aK + sb * kHalfBytes + k4 * 32), idesc_qk, k4 ? 1u : 0u);
+          if (sb == 1) umma_commit(&k_empty[st]);
+          umma_commit(&s_full[sb]);
+          return true;
+        }
 #pragma unroll
         for (int h = 0; h < 2; ++h)
 #pragma unroll
@@ -218,26 +243,25 @@ attn_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_const
       // the scores stay one tile ahead.)
       constexpr int kAhead = kVS == 2 ? 2 : 1;
       if (ok) ok = issue_qk(0);
-      if (ok && kAhead == 2 && n_tiles > 1) ok = issue_qk(1);
-      for (int j = 0; ok && j < n_tiles; ++j) {
-        if (j + kAhead < n_tiles) { if (!issue_qk(j + kAhead)) { ok = false; break; } }
-        const int st = j & 1;
-        const uint32_t ph = (j >> 1) & 1;
-        const int pb = j % kPB;
-        if (!mbar_wait(&p_ready[pb], (j / kPB) & 1, p.status, kTimeoutSoftmax)) { ok = false; break; }
-        const int vs = kVS == 2 ? st : 0;
-        const uint32_t vph = kVS == 2 ? ph : (j & 1);
-        if (!mbar_wait(&v_full[vs], vph, p.status, kTimeoutFullBarrier)) { ok = false; break; }
+      if (ok && kAhead == 2 && n_units > 1) ok = issue_qk(1);
+      for (int u = 0; ok && u < n_units; ++u) {
+        if (u + kAhead < n_units) { if (!issue_qk(u + kAhead)) { ok = false; break; } }
+        const int j = u / kMaps, pb = u % kPB;
+        if (!mbar_wait(&p_ready[pb], (u / kPB) & 1, p.status, kTimeoutSoftmax)) { ok = false; break; }
+        const int vs = kVS == 2 ? (j & 1) : 0;
+        const uint32_t vph = kVS == 2 ? ((j >> 1) & 1) : (j & 1);
+        if ((kMaps == 1 || pb == 0) && !mbar_wait(&v_full[vs], vph, p.status, kTimeoutFullBarrier)) { ok = false; break; }
         tc_fence_after();
+        const uint32_t tOm = kMaps == 2 ? tO + pb * 128 : tO;
         const uint32_t aV = smem_u32(sV + vs * kTileB);
 #pragma unroll
         for (int k8 = 0; k8 < 8; ++k8) {
           // A = P: atom (k8 / 4) of 64 kv columns, 32 bytes per K step inside it
           // B = V: 16 kv rows per step (2 KiB), two 64-wide d halves 16 KiB apart
-          umma_f16(tO, smem_desc_k_sw128(aP + pb * kTileB + (k8 >> 2) * kHalfBytes + (k8 & 3) * 32),
+          umma_f16(tOm, smem_desc_k_sw128(aP + pb * kTileB + (k8 >> 2) * kHalfBytes + (k8 & 3) * 32),
                    smem_desc_mn_sw128(aV + k8 * 2048, kHalfBytes), idesc_pv, (j | k8) ? 1u : 0u);
         }
-        umma_commit(&v_empty[vs]);
+        if (kMaps == 1 || pb == 1) umma_commit(&v_empty[vs]);
         umma_commit(&pv_done[pb]);
       }
     }
@@ -250,18 +274,22 @@ attn_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_const
     const int rowpos = pos0 + row;
     const uint32_t lane_off = static_cast<uint32_t>(quad * 32) << 16;
     float m_run = -INFINITY, l_run = 0.f;           // l_run: this half's share of the row sum
+    float m_alt = -INFINITY, l_alt = 0.f;           // kMaps == 2: the other map's (the pairs change places after every unit)
     bool ok = true;
-    for (int j = 0; ok && j < n_tiles; ++j) {
-      const int st = j & 1;
-      const uint32_t ph = (j >> 1) & 1;
+    for (int u = 0; ok && u < n_units; ++u) {
+      const int j = u / kMaps, st = u & 1;
+      const uint32_t ph = (u >> 1) & 1;
+      const uint32_t tOm = kMaps == 2 ? tO + st * 128 : tO;
       if (!mbar_wait(&s_full[st], ph, p.status, kTimeoutTmemFull)) { ok = false; break; }
       tc_fence_after();
       const uint32_t tSj = tS + st * 128 + lane_off + half * 64;
-      const int col0 = (j + tile0) * kBKV;                      // first kv position of this tile
-      // uniform over the CTA: the tile reaches past the first row's diagonal, or starts before the last row's window
-      const bool need_mask = (col0 + kBKV - 1) > pos0 || (p.window > 0 && col0 < pos0 + kBQ - p.window);
+      const int col0 = (j + (j < kept_tiles ? 0 : tile0)) * kBKV;   // first kv position of this tile
+      // uniform over the CTA: the tile reaches past the first row's diagonal, or starts before the last row's window and is not
+      // wholly kept
+      const bool need_mask = (col0 + kBKV - 1) > pos0 || (p.window > 0 && col0 < pos0 + kBQ - p.window && col0 + kBKV > p.keep);
       const int col_limit = rowpos - col0 - half * 64;          // local columns <= col_limit are visible
       const int col_lo = p.window > 0 ? col_limit - p.window + 1 : -(1 << 30);   // and local columns >= col_lo
+      const int col_keep = p.keep - col0 - half * 64;           // or < col_keep
       // This half of the score row goes to registers with one wait; the TMEM buffer is handed back at once, so
       // the MMA warp can start the scores of tile j + 2 while this tile's exponentials run.
       uint32_t r[64];
@@ -273,7 +301,7 @@ attn_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_const
       if (need_mask) {
 #pragma unroll
         for (int i = 0; i < 64; ++i)
-          if (i > col_limit || i < col_lo) r[i] = 0xff800000u;    // -inf
+          if (i > col_limit || (i < col_lo && i >= col_keep)) r[i] = 0xff800000u;    // -inf
       }
       float mx4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};   // four chains: the maximum is latency-bound
 #pragma unroll
@@ -297,20 +325,21 @@ attn_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_const
       const float corr = (m_run == -INFINITY) ? 0.f : fast_exp2(m_run - base);
       // O may be rescaled once P V of the previous tile has completed; P buffer pb is free once the P V that read
       // it (tile j - kPB) has
-      const int pb = j % kPB;
+      const int pb = u % kPB;
       const bool rescale = j > 0 && __any_sync(0xffffffffu, corr != 1.0f);
-      if (j >= kPB && !mbar_wait(&pv_done[pb], (j / kPB - 1) & 1, p.status, kTimeoutTmemFull)) { ok = false; break; }
+      if (u >= kPB && !mbar_wait(&pv_done[pb], (u / kPB - 1) & 1, p.status, kTimeoutTmemFull)) { ok = false; break; }
       if (rescale) {
-        if (!mbar_wait(&pv_done[(j - 1) % kPB], ((j - 1) / kPB) & 1, p.status, kTimeoutTmemFull)) { ok = false; break; }
+        // (with two maps the P V that last touched this map's O is the one just waited for)
+        if (kMaps == 1 && !mbar_wait(&pv_done[(u - 1) % kPB], ((u - 1) / kPB) & 1, p.status, kTimeoutTmemFull)) { ok = false; break; }
         tc_fence_after();
 #pragma unroll 1
         for (int c = 0; c < 2; ++c) {             // this half's 64 columns of O
           uint32_t o[32];
-          tmem_ld_32x32(tO + lane_off + half * 64 + c * 32, o);
+          tmem_ld_32x32(tOm + lane_off + half * 64 + c * 32, o);
           tmem_ld_wait();
 #pragma unroll
           for (int i = 0; i < 32; ++i) o[i] = __float_as_uint(__uint_as_float(o[i]) * corr);
-          tmem_st_32x32(tO + lane_off + half * 64 + c * 32, o);
+          tmem_st_32x32(tOm + lane_off + half * 64 + c * 32, o);
         }
       }
       // P = exp2(S * scale - m) as bf16 into swizzled shared memory; running sum in fp32
@@ -342,9 +371,55 @@ attn_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_const
       fence_async_smem();
       tc_fence_before();
       mbar_arrive(&p_ready[pb]);
+      if (kMaps == 2) {
+        float x = m_run; m_run = m_alt; m_alt = x;
+        x = l_run; l_run = l_alt; l_alt = x;
+      }
     }
     // ---- epilogue: O / l ---------------------------------------------------------------------------
-    if (ok && mbar_wait(&pv_done[(n_tiles - 1) % kPB], ((n_tiles - 1) / kPB) & 1, p.status, kTimeoutTmemFull)) {
+    if (kMaps == 2) {
+      // Both maps end with the last tile (n_units is even).  Once their last P V have run the P buffers are free: the row sums
+      // and then the squares of the two column halves meet there.
+      const uint32_t last = (n_tiles - 1) & 1, fph = n_tiles & 1;      // fph: the barriers' next phase
+      float* xl = reinterpret_cast<float*>(sP);
+      ok = ok && mbar_wait(&pv_done[0], last, p.status, kTimeoutTmemFull) && mbar_wait(&pv_done[1], last, p.status, kTimeoutTmemFull);
+      if (ok) {
+        tc_fence_after();
+        xl[half * 128 + row] = l_run;
+        xl[256 + half * 128 + row] = l_alt;
+        mbar_arrive(&mx_bar[0]);
+        ok = mbar_wait(&mx_bar[0], fph, p.status, kTimeoutSoftmax);
+      }
+      float o[64], ss = 0.f;
+      if (ok) {
+        const float l1 = l_run + xl[(half ^ 1) * 128 + row], l2 = l_alt + xl[256 + (half ^ 1) * 128 + row];
+        const float w1 = l1 > 0.f ? 1.0f / l1 : 0.f, w2 = l2 > 0.f ? p.lambda / l2 : 0.f;
+#pragma unroll
+        for (int c = 0; c < 2; ++c) {
+          uint32_t a[32], b[32];
+          tmem_ld_32x32(tO + lane_off + half * 64 + c * 32, a);
+          tmem_ld_32x32(tO + 128 + lane_off + half * 64 + c * 32, b);
+          tmem_ld_wait();
+#pragma unroll
+          for (int i = 0; i < 32; ++i) {
+            const float v = __uint_as_float(a[i]) * w1 - __uint_as_float(b[i]) * w2;
+            o[c * 32 + i] = v;
+            ss += v * v;
+          }
+        }
+        xl[512 + half * 128 + row] = ss;
+        mbar_arrive(&mx_bar[1]);
+        ok = mbar_wait(&mx_bar[1], fph, p.status, kTimeoutSoftmax);
+      }
+      if (ok && row0 + row < q_len) {
+        const float k = p.out_scale / sqrtf((ss + xl[512 + (half ^ 1) * 128 + row]) * (1.0f / kHD) + p.eps);
+        __nv_bfloat16* orow = p.out + static_cast<size_t>(q0 + row0 + row) * p.ldo + head * kHD + half * 64;
+#pragma unroll
+        for (int i = 0; i < 64; i += 8)
+          *reinterpret_cast<uint4*>(orow + i) = make_uint4(pack_bf16(o[i] * k, o[i + 1] * k), pack_bf16(o[i + 2] * k, o[i + 3] * k),
+                                                           pack_bf16(o[i + 4] * k, o[i + 5] * k), pack_bf16(o[i + 6] * k, o[i + 7] * k));
+      }
+    } else if (ok && mbar_wait(&pv_done[(n_tiles - 1) % kPB], ((n_tiles - 1) / kPB) & 1, p.status, kTimeoutTmemFull)) {
       // The last P V has run, so every softmax thread is past its last read of the exchange buffer: the two halves
       // now add their row sums through it.
       float* xl = reinterpret_cast<float*>(s_xch);
@@ -356,7 +431,7 @@ attn_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_const
       tc_fence_after();
       const float inv = l_run > 0.f ? 1.0f / l_run : 0.f;
       const bool row_ok = (row0 + row) < q_len;
-      __nv_bfloat16* orow = p.out + (static_cast<size_t>(q0 + row0 + row) * p.Hq + head) * kHD + half * 64;
+      __nv_bfloat16* orow = p.out + static_cast<size_t>(q0 + row0 + row) * p.ldo + head * kHD + half * 64;
 #pragma unroll 1
       for (int c = 0; c < 2; ++c) {
         uint32_t r[32];
@@ -388,15 +463,16 @@ attn_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_const
 
 using namespace cafd;
 
-// q/out [total_q, Hq, 128] bf16; caches [num_pages, 64, Hkv, 128] bf16 (page 0 all zero);
-// page_table [num_seqs, max_pages]; seq_lens [num_seqs]; q_start [num_seqs + 1];
-// max_q_len = longest chunk (grid sizing).
+// q [total_q, Hq, 128] bf16 (two maps: [total_q, Hq, 2, 64]); out rows of ldo elements, head h's 128 values at column 128 h;
+// caches [num_pages, Hkv, 64, 128] bf16 (page 0 all zero); page_table [num_seqs, max_pages]; seq_lens [num_seqs];
+// q_start [num_seqs + 1]; max_q_len = longest chunk (grid sizing).  maps 1: lambda, out_scale and eps are unused.
 extern "C" int cafd_attn_prefill(const void* q, const void* k_cache, const void* v_cache, const int* page_table,
                                  const int* seq_lens, const int* q_start, void* out, uint32_t* status, int total_q,
                                  int num_seqs, int max_q_len, int num_pages, int max_pages, int Hq, int Hkv, int D,
-                                 float scale, int window, cafd_stream_t s) {
+                                 float scale, int window, int keep, int ldo, int maps, float lambda, float out_scale, float eps,
+                                 cafd_stream_t s) {
   if (num_seqs <= 0 || total_q <= 0) return 0;
-  if (D != kHD || Hq % Hkv || window < 0) return -10;
+  if (D != kHD || Hq % Hkv || window < 0 || keep < 0 || maps < 1 || maps > 2 || ldo < Hq * kHD || ldo % 8) return -10;
   CUtensorMap tq, tk, tv;
   int rc = cached_tmap_2d(&tq, q, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, total_q, static_cast<uint64_t>(Hq) * kHD,
                           static_cast<uint64_t>(Hq) * kHD * 2, kBQ, 64);
@@ -412,7 +488,7 @@ extern "C" int cafd_attn_prefill(const void* q, const void* k_cache, const void*
   if (rc) return rc;
   rc = make_tmap_nd(&tv, v_cache, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 4, dims, strides, box, true);
   if (rc) return rc;
-  PrefillDev p;
+  PrefillDev p{};
   p.page_table = page_table;
   p.seq_lens = seq_lens;
   p.q_start = q_start;
@@ -423,14 +499,20 @@ extern "C" int cafd_attn_prefill(const void* q, const void* k_cache, const void*
   p.Hkv = Hkv;
   p.scale_log2 = scale * 1.4426950408889634f;
   p.window = window;
-  p.kv_tmp_start = nullptr; p.q_head_stride = kHD; p.qr_head_stride = 0; p.qr_col0 = 0;
+  p.keep = window > 0 ? keep : 0;
+  p.ldo = ldo;
+  p.lambda = lambda; p.out_scale = out_scale; p.eps = eps;
+  p.q_head_stride = kHD;
   static bool attr = false;
   if (!attr) {
-    CAFD_CHECK_CUDA(cudaFuncSetAttribute(attn_prefill_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, kPrefillSmem));
+    CAFD_CHECK_CUDA(cudaFuncSetAttribute(attn_prefill_kernel<false, 1>, cudaFuncAttributeMaxDynamicSharedMemorySize, kPrefillSmem));
+    CAFD_CHECK_CUDA(cudaFuncSetAttribute(attn_prefill_kernel<false, 2>, cudaFuncAttributeMaxDynamicSharedMemorySize, kPrefillSmem));
     attr = true;
   }
   dim3 grid((max_q_len + kBQ - 1) / kBQ, Hq, num_seqs);
-  launch_pdl(attn_prefill_kernel<false>, grid, dim3(kPrefillThreads), kPrefillSmem, static_cast<cudaStream_t>(s), tq, tk, tv, tq, tq, p);
+  cudaStream_t st = static_cast<cudaStream_t>(s);
+  if (maps == 2) launch_pdl(attn_prefill_kernel<false, 2>, grid, dim3(kPrefillThreads), kPrefillSmem, st, tq, tk, tv, tq, tq, p);
+  else launch_pdl(attn_prefill_kernel<false, 1>, grid, dim3(kPrefillThreads), kPrefillSmem, st, tq, tk, tv, tq, tq, p);
   return static_cast<int>(cudaGetLastError());
 }
 
@@ -469,21 +551,22 @@ extern "C" int cafd_attn_prefill_mla(const void* q_nope, int q_pitch, int q_head
   const uint32_t lbox[3] = {64, kPageTok, 1};
   rc = make_tmap_nd(&tkr, latent_cache, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 3, ldims, lstrides, lbox, true);
   if (rc) return rc;
-  PrefillDev p;
+  PrefillDev p{};
   p.page_table = page_table; p.seq_lens = seq_lens; p.q_start = q_start;
   p.out = static_cast<__nv_bfloat16*>(out);
   p.status = status;
   p.max_pages = max_pages; p.Hq = heads; p.Hkv = heads;
   p.scale_log2 = scale * 1.4426950408889634f;
   p.window = window;
+  p.ldo = heads * kHD;
   p.kv_tmp_start = kv_tmp_start; p.q_head_stride = q_head_stride; p.qr_head_stride = qr_head_stride; p.qr_col0 = qr_col0;
   static bool attr = false;
   if (!attr) {
-    CAFD_CHECK_CUDA(cudaFuncSetAttribute(attn_prefill_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, kPrefillSmemRope));
+    CAFD_CHECK_CUDA(cudaFuncSetAttribute(attn_prefill_kernel<true, 1>, cudaFuncAttributeMaxDynamicSharedMemorySize, kPrefillSmemRope));
     attr = true;
   }
   dim3 grid((max_q_len + kBQ - 1) / kBQ, heads, num_seqs);
-  launch_pdl(attn_prefill_kernel<true>, grid, dim3(kPrefillThreads), kPrefillSmemRope, static_cast<cudaStream_t>(s), tq, tk, tv, tqr, tkr, p);
+  launch_pdl(attn_prefill_kernel<true, 1>, grid, dim3(kPrefillThreads), kPrefillSmemRope, static_cast<cudaStream_t>(s), tq, tk, tv, tqr, tkr, p);
   return static_cast<int>(cudaGetLastError());
 }
 

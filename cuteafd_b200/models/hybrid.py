@@ -234,6 +234,12 @@ def tensor_core_latent(cfg: ModelConfig, m: LatentSpec) -> bool:
             and 128 % m.heads == 0)
 
 
+def tensor_core_attention(cfg: ModelConfig, m: AttentionSpec) -> bool:
+    """Whether the tensor-core attention kernels take this layer: key rows (all maps) and values of 128."""
+    rows = m.maps * (m.heads // m.kv_heads)
+    return engine_dtype(cfg) == torch.bfloat16 and m.maps * m.dim == 128 and m.vdim == 128 and rows <= 16 and 16 % rows == 0
+
+
 class HybridCache:
     """Paged records of the attention layers and the slot pool of everything recurrent, per layer run.
 
@@ -308,6 +314,7 @@ class _AttnWs:
         if m.rope not in tables:
             tables[m.rope] = (rope_frequencies(m.rope).to(device), torch.zeros(max_tokens, max(1, m.rope.dims // 2), 2, device=device))
         self.table = tables[m.rope][1]
+        self.tensor_core = tensor_core_attention(cfg, m)
 
 
 class HybridEngine:
@@ -378,6 +385,7 @@ class HybridEngine:
         self._blocks: dict = {}
         self._zero1 = torch.zeros(1, dtype=torch.int32, device=dev)
         self._scratch: torch.Tensor | None = None
+        self._outgrown: list = []
         self.fixed_kv_split = K.batch_invariant_from_env()
         self.layer_hook = None           # callable(layer, residual [T, H]) for tests and traces (eager mode only)
         self.launches = 0
@@ -421,6 +429,13 @@ class HybridEngine:
         a = self.ws.proj[:T * w.shape[0]].view(T, w.shape[0])
         self.launches += 1
         return K.linear(h, w, out=a)
+
+    def _partials(self, floats: int) -> torch.Tensor:
+        """Scratch for the partial sums of split attention.  An outgrown buffer is kept: a captured graph may still write it."""
+        if self._scratch is None or self._scratch.numel() < floats:
+            self._outgrown.append(self._scratch)
+            self._scratch = torch.empty(floats, dtype=torch.float32, device=self.device)
+        return self._scratch
 
     def _block_table(self, S: int, max_q_len: int, per: int):
         key = (S, max_q_len, per)
@@ -496,8 +511,7 @@ class HybridEngine:
             splits = K.kv_splits_fixed(max_pages, cap=64)
         if splits > 1:
             need = K.mla_scratch_floats(nb, splits)
-            if self._scratch is None or self._scratch.numel() < need:
-                self._scratch = torch.empty(need, dtype=torch.float32, device=self.device)
+            self._partials(need)
         K.mla_attention(lw.q_abs[:T], cache, b.page_table, b.seq_lens, b.q_start, bseq, btok, o_slab, m.scale, splits,
                         self._scratch if splits > 1 else None, out_tpad=t_pad, window=m.window)
         self.launches += 1 if splits > 1 else 0
@@ -509,8 +523,23 @@ class HybridEngine:
         (k, v), q = self.kv.of_run[n], aw.q[:T]
         K.conv_rope_kv(a, L.offs, m, L.conv_w, aw.table, b.slots, q, k, v, state=self.kv.state, state_off=self.kv.offsets[n]["conv"],
                        state_in=b.state_in, state_out=b.state_out, q_start=b.q_start)
-        K.paged_attn(q, k, v, m, b.page_table, b.positions, b.q_start, out, pad8(m.vdim), L.lam, self.cfg.rms_eps)
         self.launches += 2
+        if not aw.tensor_core:
+            K.paged_attn(q, k, v, m, b.page_table, b.positions, b.q_start, out, pad8(m.vdim), L.lam, self.cfg.rms_eps)
+            return
+        kw = dict(scale=m.scale, window=m.window, keep=m.keep_first, maps=m.maps, lam=L.lam, out_scale=1.0 - m.diff, eps=self.cfg.rms_eps)
+        q = q.view(T, m.heads, 128)
+        if b.prefill:
+            K.attn_prefill(q, k, v, b.page_table, b.seq_lens, b.q_start, out, b.max_q_len, **kw)
+            return
+        S, max_pages = b.page_table.shape
+        q_per_tile = 16 // (m.maps * (m.heads // m.kv_heads))
+        tiles = (b.max_q_len + q_per_tile - 1) // q_per_tile
+        splits = (K.kv_splits_fixed(max_pages) if self.fixed_kv_split else
+                  K.attn_decode_splits(S, tiles, m.kv_heads, max_pages, m.window, m.keep_first))
+        need = K.attn_decode_scratch_floats(S, b.max_q_len, m.maps * m.heads, m.kv_heads, splits)
+        K.attn_decode(q, k, v, b.page_table, b.seq_lens, b.q_start, out, self._partials(need) if splits > 1 else None, b.max_q_len, splits, **kw)
+        self.launches += 1 if splits > 1 else 0
 
     def _parallel(self, n: int, i: int, spec, h: torch.Tensor, T: int, b: Batch) -> None:
         """Mixer and feed-forward on the same rows; one product over both reads their outputs side by side."""

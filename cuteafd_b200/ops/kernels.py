@@ -364,14 +364,14 @@ def moe_combine(buf: torch.Tensor, w: torch.Tensor, out: torch.Tensor, *, shared
 
 
 # ---- attention -------------------------------------------------------------------------------------
-def attn_decode_splits(num_seqs: int, tiles_per_seq: int, Hkv: int, max_pages: int, window: int = 0) -> int:
-    """KV splits for the decode attention kernel (``window`` > 0: a row reads at most the pages its window touches, so
+def attn_decode_splits(num_seqs: int, tiles_per_seq: int, Hkv: int, max_pages: int, window: int = 0, keep: int = 0) -> int:
+    """KV splits for the decode attention kernel (``window`` > 0: a row reads at most the pages its window and the kept tokens touch, so
     the splits are sized for those, not for the whole table).  The kernel keeps one 64-token page pair in flight per CTA, so
     HBM is only saturated with about three CTAs per SM (64 KB of shared memory each): aim for one full wave of
     3 x SMs CTAs, and never let a split grow past ~1K tokens (measured: 8 x 8K context 46 -> 33 us, 32 x 8K
     131 -> 99 us against the old one-CTA-per-SM rule)."""
     if window > 0:
-        max_pages = min(max_pages, (window + 63) // 64 + 1)
+        max_pages = min(max_pages, (window + 63) // 64 + 1 + (keep + 63) // 64)
     ctas = max(1, num_seqs * tiles_per_seq * Hkv)
     want = max((3 * num_sms()) // ctas, (max_pages + 15) // 16, 1)
     return max(1, min(want, max(1, max_pages // 4), 32))
@@ -411,19 +411,28 @@ def kv_splits_fixed(max_pages: int, cap: int = 0) -> int:
     return n
 
 
+def _attn_out(q: torch.Tensor, out: torch.Tensor, maps: int) -> int:
+    """Row pitch of an attention output [T, heads, D] or [T, columns]."""
+    assert q.is_contiguous() and out.stride(-1) == 1 and (out.dim() == 2 or out.is_contiguous()) and maps in (1, 2)
+    return out.stride(0)
+
+
 def attn_decode(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, page_table: torch.Tensor,
                 seq_lens: torch.Tensor, q_start: torch.Tensor, out: torch.Tensor, scratch: torch.Tensor | None,
-                max_q_len: int, splits: int, scale: float | None = None, window: int = 0) -> torch.Tensor:
-    """``window`` > 0: a query at position t sees keys (t - window, t] only (sliding-window layers); the pages
-    before the window are not read."""
+                max_q_len: int, splits: int, scale: float | None = None, window: int = 0, keep: int = 0, maps: int = 1,
+                lam: float = 0.0, out_scale: float = 1.0, eps: float = 0.0) -> torch.Tensor:
+    """``window`` > 0: a query at position t sees keys (t - window, t] (sliding-window layers) and the first ``keep``; the pages
+    between are not read.  ``maps`` 2: q [T, heads, 2 x 64] and keys hold two score maps per head; the output is map 1 - ``lam`` *
+    map 2 over its root mean square (``eps`` inside), times ``out_scale``.  ``out``: [T, heads, D], or rows [T, columns] whose first
+    heads * D columns are written."""
     _, Hq, D = q.shape
     Hkv = k_cache.shape[1]                 # pools are [pages, kv heads, 64, D]
     num_seqs, max_pages = page_table.shape
     scale = scale if scale is not None else 1.0 / math.sqrt(D)
     _n.check(_n.cuda_lib().cafd_attn_decode(q.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(), page_table.data_ptr(),
                                             seq_lens.data_ptr(), q_start.data_ptr(), out.data_ptr(), _ptr(scratch),
-                                            num_seqs, max_q_len, max_pages, Hq, Hkv, D, splits, scale, int(window), _stream()),
-             "attn_decode")
+                                            num_seqs, max_q_len, max_pages, Hq, Hkv, D, splits, scale, int(window), int(keep),
+                                            _attn_out(q, out, maps), maps, lam, out_scale, eps, _stream()), "attn_decode")
     return out
 
 
@@ -460,15 +469,18 @@ def attn_decode_scratch_floats(num_seqs: int, max_q_len: int, Hq: int, Hkv: int,
 
 def attn_prefill(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, page_table: torch.Tensor,
                  seq_lens: torch.Tensor, q_start: torch.Tensor, out: torch.Tensor, max_q_len: int,
-                 scale: float | None = None, window: int = 0) -> torch.Tensor:
-    total_q, Hq, D = q.shape
-    num_pages, Hkv, _, _ = k_cache.shape   # pools are [pages, kv heads, 64, D]
+                 scale: float | None = None, window: int = 0, keep: int = 0, maps: int = 1, lam: float = 0.0, out_scale: float = 1.0,
+                 eps: float = 0.0) -> torch.Tensor:
+    """Prompt attention; the arguments mean what they mean for ``attn_decode``."""
+    T, Hq, D = q.shape
+    num_pages, Hkv = k_cache.shape[0], k_cache.shape[1]
     num_seqs, max_pages = page_table.shape
     scale = scale if scale is not None else 1.0 / math.sqrt(D)
     _n.check(_n.cuda_lib().cafd_attn_prefill(q.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(), page_table.data_ptr(),
                                              seq_lens.data_ptr(), q_start.data_ptr(), out.data_ptr(),
-                                             status_word(q.device).data_ptr(), total_q, num_seqs, max_q_len, num_pages,
-                                             max_pages, Hq, Hkv, D, scale, int(window), _stream()), "attn_prefill")
+                                             status_word(q.device).data_ptr(), T, num_seqs, max_q_len, num_pages,
+                                             max_pages, Hq, Hkv, D, scale, int(window), int(keep), _attn_out(q, out, maps), maps, lam,
+                                             out_scale, eps, _stream()), "attn_prefill")
     return out
 
 

@@ -94,7 +94,10 @@ def render(rep: PlanReport) -> str:
          + (f"MLA {c.num_heads} heads (q_lora {c.q_lora_rank}, kv_lora {c.kv_lora_rank}, nope {c.qk_nope_dim}, rope {c.qk_rope_dim}, v {c.v_head_dim})"
             if c.is_mla else ", ".join(f"{n} {k}" for k, n in sorted(Counter(
                 f"latent (rank {m.kv_rank} + {m.rot_dim}, {m.heads} heads, window {m.window})" if hasattr(m, "kv_rank")
+                else (f"{'differential ' if m.maps == 2 else ''}attention ({m.heads}/{m.kv_heads} heads x {m.dim} + {m.vdim}, window {m.window}"
+                      f", keeps {m.keep_first})") if hasattr(m, "rope")
                 else f"delta ({m.heads} heads x {m.dim} x {m.vdim})" for m in (s.mixer for s in c.layer_specs)).items()))
+            + (f", layers {c.loop[0]} to {c.loop[1] - 1} looped {c.loop[2]} times" if c.loop else "")
             if c.is_hybrid else f"GQA {c.num_heads}/{c.num_kv_heads} heads x {c.head_dim}"),
          f"ffn        dense {c.dense_ffn} x {c.first_dense_layers} layers; {c.num_experts} routed experts x {c.expert_ffn} "
          f"({c.scoring} top-{c.top_k}" + (f", {c.num_groups} groups keep {c.topk_groups}" if c.num_groups > 1 else "") + ")"

@@ -83,13 +83,11 @@ def sink_attention(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, start: int
     """Softmax attention of q [T, H, Dk] (positions start, start + 1, ...) over k [L, H, Dk], v [L, H, Dv] (positions 0, 1, ...):
     the query at position i reads the keys j <= i that lie among the last ``window`` positions (0: anywhere) or the first
     ``keep``."""
-    out = []
-    for t in range(q.shape[0]):
-        i = start + t
-        seen = [j for j in range(i + 1) if window == 0 or i - j < window or j < keep]
-        s = torch.einsum("hd,jhd->hj", q[t], k[seen]) * scale
-        out.append(torch.einsum("hj,jhd->hd", torch.softmax(s, -1), v[seen]))
-    return torch.stack(out)
+    i = torch.arange(start, start + q.shape[0])[:, None]
+    j = torch.arange(k.shape[0])[None]
+    seen = (j <= i) & ((i - j < window) | (j < keep)) if window else j <= i
+    s = torch.einsum("thd,jhd->htj", q, k) * scale
+    return torch.einsum("htj,jhd->thd", torch.softmax(s.masked_fill(~seen, -math.inf), -1), v)
 
 
 def difference_weight(p: Params, pre: str, diff: float) -> torch.Tensor:

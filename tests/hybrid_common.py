@@ -1,7 +1,8 @@
 """Small per-layer hybrid configurations and helpers shared by the hybrid tests."""
 import torch
 
-from cuteafd_b200.config import DeltaSpec, LatentSpec, LayerSpec, RouterSpec, hybrid_config
+from cuteafd_b200.config import (AttentionSpec, DeltaSpec, DenseSpec, LatentSpec, LayerSpec, RopeSpec, RouterSpec, hybrid_config,
+                                 parallel_config)
 from cuteafd_b200.ref import hybrid as R
 
 
@@ -45,6 +46,39 @@ def wide_config(window=100):
         LayerSpec(latent(8, 128, 64, 128, 512, window, base=1e5), RouterSpec(8, 128, 2, 2, 5, 3)),
         LayerSpec(delta(4, 2, 128, 128, 4), RouterSpec(6, 64, 3, 3, 3, 2)),
         LayerSpec(latent(16, 128, 64, 128, 512, 2 * window + 3, base=1e4))], canon_taps=4, norm_groups=4, eps=1e-5)
+
+
+def attention(heads=6, kv_heads=2, dim=12, vdim=20, window=37, keep=5, rope=RopeSpec(8, 5000.0, 3.0, 1.0, 4.0, 100), conv=3, diff=0.3, scale=None):
+    return AttentionSpec(heads, kv_heads, dim, vdim, window, keep, scale if scale is not None else 1.6 * dim ** -0.5, rope, conv, 2, diff)
+
+
+def parallel(m, ffn=None):
+    return LayerSpec(m, dense=DenseSpec(ffn) if ffn else None, parallel=True)
+
+
+def looped_config():
+    """Every layer differs: head sizes that are no multiples of 8, odd ones among them, layers without a feed-forward, a window
+    of one token, one that starts inside the kept tokens, none at all; the middle runs three times."""
+    return parallel_config("looped", 203, 104, [
+        parallel(attention(), 72),
+        parallel(attention(3, 3, 8, 8, 1, 2, RopeSpec(8, 300.0), 1, 0.0)),
+        parallel(attention(5, 1, 15, 7, 130, 70, RopeSpec(10, 1e4, 8.0, 0.5, 2.0, 64), 5, 0.8), 33),
+        parallel(attention(4, 4, 16, 24, 0, 0, RopeSpec(16, 700.0), 4, 0.45), 40)], 2e-5, loop=(1, 3, 3), logit_softcap=9.0)
+
+
+def bare_config():
+    """Values that make a mechanism vanish: one head, no kept tokens, no loop, no cap, no rotation, a width that is no multiple
+    of 8."""
+    return parallel_config("bare", 77, 90, [
+        parallel(attention(1, 1, 10, 6, 21, 0, RopeSpec(10, 1e3), 2), 11),
+        parallel(attention(8, 2, 8, 16, 64, 64, RopeSpec(0, 1e3), 3, 0.2), 24)], 1e-3)
+
+
+def paired_config(window=100, keep=70):
+    """The sizes the tensor-core attention kernels take; everything runs twice."""
+    return parallel_config("paired", 500, 256, [
+        parallel(attention(4, 2, 64, 128, window, keep, RopeSpec(64, 1e5, 4.0, 1.0, 4.0, 256), 4, 0.6), 192),
+        parallel(attention(8, 1, 64, 128, 2 * window + 3, 3, RopeSpec(32, 1e4), 3, 0.2), 136)], 1e-5, loop=(0, 2, 2), logit_softcap=30.0)
 
 
 def params(cfg, seed=0, spread=0.4):
