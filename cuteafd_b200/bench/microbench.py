@@ -6,6 +6,7 @@
     python -m cuteafd_b200.bench.microbench mla --seqs 8 --len 8192 --qlen 1 --heads 128 [--topk 2048]
     python -m cuteafd_b200.bench.microbench w4 --tokens 8 --features 7168 --k 2048 --fmt nvfp4
     python -m cuteafd_b200.bench.microbench hybrid --size base
+    python -m cuteafd_b200.bench.microbench parallel --size base
     python -m cuteafd_b200.bench.microbench sampler --rows 32 --vocab 151936
     python -m cuteafd_b200.bench.microbench moe --tokens 1,16,128,1024,8192 --hidden 7168 --ffn 2048 \
         --experts 256 --top-k 8 --scoring sigmoid
@@ -375,6 +376,75 @@ def bench_hybrid(a, dev, pk) -> None:
     run(f"latent_gate {T} rows", lambda: K.latent_gate(out, p, 0, heads, 128), T * heads * 128 * 6)
 
 
+def bench_parallel(a, dev, pk) -> None:
+    """The kernels of parallel layers with differential attention beside the like kernels of the dense GQA decoder, at one of the
+    benchmark sizes."""
+    from ..config import GUBERAX_SIZES, guberax_bench
+    from ..models.hybrid import rope_frequencies
+    H, _, heads, kvh, ffn = GUBERAX_SIZES[a.size]
+    cfg, bf, T = guberax_bench(a.size), torch.bfloat16, a.tokens
+    m = cfg.layer_specs[0].mixer
+    w = m.window
+    freq = rope_frequencies(m.rope).to(dev)
+
+    def i32(v):
+        return torch.tensor(list(v), dtype=torch.int32, device=dev)
+
+    def run(name, fn, nbytes, flops=0.0):
+        report(name, time_eager(fn, dev, a.iters), flops, nbytes, pk)
+    diff = dict(scale=m.scale, window=w, keep=m.keep_first, maps=2, lam=0.5, out_scale=0.5, eps=1e-6)
+    for n in (1, 8, 32, T):
+        S = n if n < T else 1
+        x, xo, y, h = torch.randn(n, H, device=dev), torch.empty(n, H, device=dev), torch.randn(n, H, device=dev, dtype=bf), torch.empty(n, H, device=dev, dtype=bf)
+        wt = torch.zeros(H, device=dev, dtype=bf)
+        run(f"norm_conv, plain add, {n} rows", lambda: K.norm_conv(h, wt, 1, 1e-6, x_in=x, y=y, x_out=xo, w_offset=1.0), n * H * 12)
+        run(f"(GQA) rmsnorm {n} rows", lambda: K.rmsnorm(y, wt, 1e-6, out=h), n * H * 4)
+        C = m.conv_channels
+        ctx = T
+        pps = (ctx + 63) // 64
+        kc, vc = (torch.randn(S * pps + 1, kvh, 64, 128, device=dev, dtype=bf) for _ in range(2))
+        table = (torch.arange(S * pps, dtype=torch.int32, device=dev) + 1).view(S, pps).contiguous()
+        a_ = torch.randn(n, C, device=dev, dtype=bf)
+        offs = dict(q=0, k=m.q_channels, v=m.q_channels + m.k_channels)
+        pos = i32([ctx - 1] * S) if n < T else i32(range(T))
+        slots = (table[:, -1] * 64 + 63).int() if n < T else i32(range(64, 64 + T))
+        cw, st = torch.randn(m.conv, C, device=dev), torch.zeros(2 + 2 * S, 3 * C, device=dev)
+        tab, q = torch.empty(n, 32, 2, device=dev), torch.randn(n, heads, 128, device=dev, dtype=bf)
+        K.rope_table(pos, freq, tab)
+        qs, sl = (i32(range(S + 1)), i32([ctx] * S)) if n < T else (i32([0, T]), i32([T]))
+        si, so = i32(range(2, 2 + S)), i32(range(2 + S, 2 + 2 * S))
+        run(f"conv_rope_kv {n} rows", lambda: K.conv_rope_kv(a_, offs, m, cw, tab, slots, q, kc, vc, state=st, state_in=si, state_out=so, q_start=qs),
+            n * C * 4 + S * C * 24)
+        f64 = torch.ones(64, device=dev)
+        run(f"(GQA) qk_rope_kv {n} rows", lambda: K.qk_rope_kv(a_, None, None, f64, pos, slots, q, kc, vc, heads, kvh, 128, 1e-6, False), n * C * 4)
+        out, wide = torch.empty(n, heads, 128, device=dev, dtype=bf), torch.empty(n, heads * 128 + ffn, device=dev, dtype=bf)
+        if n == T:
+            pairs = T * w - w * w / 2 + max(0, T - w - m.keep_first) * m.keep_first
+            run(f"attn_prefill, two maps, {T} tokens, window {w} + {m.keep_first}", lambda: K.attn_prefill(q, kc, vc, table, sl, qs, wide, T, **diff),
+                T * C * 4, pairs * heads * 2 * (2 * 64 + 2 * 128))
+            pairs = T * w - w * w / 2
+            run(f"(GQA) attn_prefill {T} tokens, window {w}", lambda: K.attn_prefill(q, kc, vc, table, sl, qs, out, T, window=w), T * C * 4, pairs * heads * 4 * 128)
+            logits = torch.randn(32, cfg.vocab_size, device=dev)
+            run("softcap 32 rows", lambda: K.softcap(logits, 30.0), logits.numel() * 8)
+            run(f"rope_table {T} rows", lambda: K.rope_table(pos, freq, tab), T * 32 * 8)
+        else:
+            for tag, kw, keep, hm in ((", two maps", diff, m.keep_first, 2), ("(GQA) ", dict(window=w), 0, 1)):
+                sp = K.attn_decode_splits(S, 1, kvh, pps, w, keep)
+                sc = torch.empty(K.attn_decode_scratch_floats(S, 1, hm * heads, kvh, sp), device=dev)
+                o = wide if hm == 2 else out
+                run((tag + "attn_decode" if hm == 1 else "attn_decode" + tag) + f", {S} x {ctx}, window {w} + {keep}, {sp} splits",
+                    lambda: K.attn_decode(q, kc, vc, table, sl, qs, o, sc, 1, sp, **kw), S * (w + keep) * kvh * 512)
+        g, u, wo = (torch.randn(r, c, device=dev, dtype=bf) * 0.02 for r, c in ((ffn, H), (ffn, H), (H, heads * 128 + ffn)))
+        flop = 2.0 * n * H
+        run(f"gate / up product {n} rows", lambda: K.linear(h, g, out=wide[:, heads * 128:], w_up=u), 4 * ffn * H + n * (H + ffn) * 2, flop * 2 * ffn)
+        run(f"[o | down] product {n} rows", lambda: K.linear(wide, wo, out=y), 2 * wo.numel() + n * (H + wo.shape[1]) * 2, flop * wo.shape[1])
+        o1, d1 = wo[:, :heads * 128].contiguous(), wo[:, heads * 128:].contiguous()
+        on, dn = out.view(n, -1), torch.randn(n, ffn, device=dev, dtype=bf)
+        run(f"(GQA) o product + residual {n} rows", lambda: K.linear(on, o1, out=y, residual=y), 2 * o1.numel() + n * (2 * H + heads * 128) * 2, flop * heads * 128)
+        run(f"(GQA) down product + residual {n} rows", lambda: K.linear(dn, d1, out=y, residual=y), 2 * d1.numel() + n * (2 * H + ffn) * 2, flop * ffn)
+    assert K.read_status() == 0
+
+
 def main() -> None:
     ap = argparse.ArgumentParser()
     sub = ap.add_subparsers(dest="cmd", required=True)
@@ -416,14 +486,17 @@ def main() -> None:
     sm.add_argument("--top-k", type=int, default=50); sm.add_argument("--top-p", type=float, default=0.9)
     hy = sub.add_parser("hybrid")
     hy.add_argument("--size", default="base", choices=["small", "base", "large"]); hy.add_argument("--tokens", type=int, default=8192)
-    for s in (g, p, d, m, ml, mp_, w4, sm, hy):
+    pa = sub.add_parser("parallel")
+    pa.add_argument("--size", default="base", choices=["small", "base", "large"]); pa.add_argument("--tokens", type=int, default=8192)
+    for s in (g, p, d, m, ml, mp_, w4, sm, hy, pa):
         s.add_argument("--iters", type=int, default=10)
     a = ap.parse_args()
     dev = torch.device("cuda", int(os.environ.get("LOCAL_RANK", "0")))
     torch.cuda.set_device(dev)
     pk = peaks()
     {"exl3": bench_exl3, "gemm-fp8": bench_gemm_fp8, "indexer": bench_indexer, "gemm": bench_gemm, "attn-prefill": bench_attn_prefill, "attn-decode": bench_attn_decode, "moe": bench_moe,
-     "mla": bench_mla, "mla-prefill": bench_mla_prefill_expanded, "w4": bench_w4, "sampler": bench_sampler, "hybrid": bench_hybrid}[a.cmd](a, dev, pk)
+     "mla": bench_mla, "mla-prefill": bench_mla_prefill_expanded, "w4": bench_w4, "sampler": bench_sampler, "hybrid": bench_hybrid,
+     "parallel": bench_parallel}[a.cmd](a, dev, pk)
 
 
 if __name__ == "__main__":
