@@ -4,7 +4,7 @@
 //
 //   rope_table       cos / sin of position * frequency for every token of the step, once per step and kind of rotation:
 //                    every layer that rotates alike reads it
-//   conv_rope_kv     eight channels per thread walking a run of tokens, the convolution's earlier inputs in registers
+//   conv_rope_kv     four channels per thread walking a run of tokens, the convolution's earlier inputs in registers
 //   conv_rope_kv_any any head sizes and any number of taps: one channel per thread and token
 //
 // A sequence's last taps - 1 projected rows are fp32 in its state slot (oldest first, [taps - 1, channels]); a step reads one
@@ -45,11 +45,10 @@ __global__ void __launch_bounds__(256) rope_table_kernel(const int* __restrict__
   }
 }
 
-// Where channel c of the concatenated [q | k | v] channels goes for one token; null = nowhere.
+// Where channel c of the concatenated [q | k | v] channels goes for token t, whose K / V slot is `slot`; null = nowhere.
 template <typename E>
-__device__ __forceinline__ E* conv_rope_dest(const ConvRope& p, int t, int c) {
+__device__ __forceinline__ E* conv_rope_dest(const ConvRope& p, int t, int slot, int c) {
   if (c < p.nq) return static_cast<E*>(p.q_out) + static_cast<size_t>(t) * p.nq + c;
-  const int slot = p.slots[t];
   if (slot < 0) return nullptr;
   const bool is_k = c < p.nq + p.nk;
   const int per = is_k ? p.maps_dim : p.vdim;
@@ -71,103 +70,110 @@ __device__ __forceinline__ int seq_of(const int* q_start, int S, int t) {
 }
 
 template <typename E, int MAXT>
-__global__ void __launch_bounds__(128) conv_rope_kv_kernel(const ConvRope p) {
-  constexpr int V = 8, W = MAXT > 1 ? MAXT - 1 : 1;
+__global__ void __launch_bounds__(128, MAXT <= 4 && sizeof(E) == 2 ? 7 : 2) conv_rope_kv_kernel(const ConvRope p) {
+  constexpr int V = 4, W = MAXT - 1, kBatch = 4;
+  extern __shared__ float4 sm4[];               // the run's angles [run][rot / 2] cos, sin, then its slots [run]
+  float2* s_cs = reinterpret_cast<float2*>(sm4);
+  int* s_slot = reinterpret_cast<int*>(s_cs + p.run * (p.rot >> 1));
   const int C = p.nq + p.nk + p.nv;
   const int c = (blockIdx.y * blockDim.x + threadIdx.x) * V;
   const int halo = p.conv_w ? p.taps - 1 : 0;
-  float w[MAXT][V];                             // taps, oldest first, at the array's end (weights: not written by any kernel)
+  float w[MAXT][V];                             // w[k]: weight of the input k tokens back (no kernel writes the weights)
 #pragma unroll
-  for (int j = 0; j < MAXT; ++j) {
-    const int tap = j - (MAXT - 1 - halo);
+  for (int k = 0; k < MAXT; ++k) {
 #pragma unroll
-    for (int e = 0; e < V; ++e) w[j][e] = 0.f;
-    if (p.conv_w && tap >= 0 && c < C) load_vec<float, V>(p.conv_w + static_cast<size_t>(tap) * C + c, w[j]);
+    for (int e = 0; e < V; ++e) w[k][e] = !p.conv_w && k == 0 ? 1.f : 0.f;
+    if (p.conv_w && k <= halo && c < C) load_vec<float, V>(p.conv_w + static_cast<size_t>(halo - k) * C + c, w[k]);
   }
   pdl_wait();
   pdl_trigger();
-  if (c >= C) return;
   const int r0 = blockIdx.x * p.run, r1 = min(p.T, r0 + p.run);
-  if (r0 >= r1) return;
-  const int col = conv_rope_col(p, c);
-  const E* src = static_cast<const E*>(p.proj) + col;
-  const int d0 = c < p.nq + p.nk ? (c < p.nq ? c : c - p.nq) % p.dim : p.rot;   // first dimension inside its map; v: past the rotated ones
+  for (int i = threadIdx.x; i < (r1 - r0) * (p.rot >> 1); i += blockDim.x) s_cs[i] = p.table[static_cast<size_t>(r0) * (p.rot >> 1) + i];
+  for (int i = threadIdx.x; i < r1 - r0; i += blockDim.x) s_slot[i] = p.slots[r0 + i];
+  __syncthreads();
+  if (c >= C) return;
+  const E* src = static_cast<const E*>(p.proj) + conv_rope_col(p, c);
+  const bool is_q = c < p.nq, is_v = c >= p.nq + p.nk;
+  const int d0 = is_v ? p.rot : (is_q ? c : c - p.nq) % p.dim;   // first dimension inside its map; v: past the rotated ones
   const bool turns = d0 < p.rot;
-  float win[W][V];                              // the last taps - 1 inputs, oldest first, at the array's end
-#pragma unroll
-  for (int j = 0; j < W; ++j)
-#pragma unroll
-    for (int e = 0; e < V; ++e) win[j][e] = 0.f;
+  // K / V: where token (page 0, offset 0) would put these channels, elements per token of a head and per page
+  E* const dst0 = is_q ? static_cast<E*>(p.q_out) + c : conv_rope_dest<E>(p, 0, 0, c);
+  const int per = is_v ? p.vdim : p.maps_dim;
+  const size_t page = static_cast<size_t>(p.kv_heads) * 64 * per;
   int seq = 0, s_lo = 0, s_hi = p.T;
   if (halo > 0) {
     seq = seq_of(p.q_start, p.S, r0);
     s_lo = p.q_start[seq];
     s_hi = p.q_start[seq + 1];
   }
-  // inputs before token t0 of sequence seq: rows of this step, or the sequence's state where they lie before it
-  auto fill = [&](int t0) {
-    const float* st = p.state + static_cast<size_t>(p.state_in[seq]) * p.slot_stride + p.state_off + c;
+  float x[W + kBatch][V];                       // a batch of kBatch tokens' inputs behind the W before it
 #pragma unroll
-    for (int j = 0; j < W; ++j) {
-      const int back = W - j;                   // input of token t0 - back
-      if (back <= halo) {
-        const int row = t0 - back;
-        if (row >= s_lo) load_vec<E, V>(src + static_cast<size_t>(row) * p.ld, win[j]);
-        else load_vec<float, V>(st + static_cast<size_t>(halo + row - s_lo) * C, win[j]);
-      }
+  for (int i = 0; i < W; ++i)
+#pragma unroll
+    for (int e = 0; e < V; ++e) x[i][e] = 0.f;
+  Packed<E, V> nx[kBatch];                      // the next batch's rows, on their way while one is worked on
+#pragma unroll
+  for (int j = 0; j < kBatch; ++j) nx[j] = load_packed<E, V>(src + static_cast<size_t>(min(r0 + j, p.T - 1)) * p.ld);
+  for (int t = r0; t < r1; t += kBatch) {
+#pragma unroll
+    for (int j = 0; j < kBatch; ++j) unpack(nx[j], x[W + j]);
+    if (t + kBatch < r1) {
+#pragma unroll
+      for (int j = 0; j < kBatch; ++j) nx[j] = load_packed<E, V>(src + static_cast<size_t>(min(t + kBatch + j, p.T - 1)) * p.ld);
     }
-  };
-  if (halo > 0) fill(r0);
-  Packed<E, V> nx = load_packed<E, V>(src + static_cast<size_t>(r0) * p.ld);
-  for (int t = r0; t < r1; ++t) {
-    if (halo > 0 && t == s_hi) {                // next sequence (empty ones are skipped)
-      do { ++seq; s_lo = s_hi; s_hi = p.q_start[seq + 1]; } while (s_hi == s_lo && seq + 1 < p.S);
-      fill(t);
-    }
-    float x[V], y[V];
-    unpack(nx, x);
-    if (t + 1 < r1) nx = load_packed<E, V>(src + static_cast<size_t>(t + 1) * p.ld);
-    if (p.conv_w) {
 #pragma unroll
-      for (int e = 0; e < V; ++e) y[e] = w[MAXT - 1][e] * x[e];
+    for (int j = 0; j < kBatch; ++j) {
+      const int row = t + j;
+      if (row >= r1) break;
+      if (halo > 0 && (row == r0 || row == s_hi)) {
+        // The inputs before a run's or a sequence's first token: rows of this step, or the state where they lie before it.
+        // (The slots held another sequence's last inputs, which are done with.)
+        while (row == s_hi && seq + 1 < p.S) { ++seq; s_lo = s_hi; s_hi = p.q_start[seq + 1]; }      // empty sequences are skipped
+        const float* st = p.state + static_cast<size_t>(p.state_in[seq]) * p.slot_stride + p.state_off + c;
 #pragma unroll
-      for (int j = 0; j < MAXT - 1; ++j)
-#pragma unroll
-        for (int e = 0; e < V; ++e) y[e] = fmaf(w[j][e], win[j][e], y[e]);
-    } else {
-#pragma unroll
-      for (int e = 0; e < V; ++e) y[e] = x[e];
-    }
-    if (turns) {
-      const float2* cs = p.table + static_cast<size_t>(t) * (p.rot >> 1) + (d0 >> 1);
-#pragma unroll
-      for (int i = 0; i < V / 2; ++i) {
-        if (d0 + 2 * i < p.rot) {
-          const float2 k = cs[i];
-          const float u = y[2 * i], v = y[2 * i + 1];
-          y[2 * i] = u * k.x - v * k.y;
-          y[2 * i + 1] = v * k.x + u * k.y;
+        for (int k = 1; k < MAXT; ++k) {
+          if (k <= halo) {
+            if (row - k >= s_lo) load_vec<E, V>(src + static_cast<size_t>(row - k) * p.ld, x[W + j - k]);
+            else load_vec<float, V>(st + static_cast<size_t>(halo + row - k - s_lo) * C, x[W + j - k]);
+          }
         }
       }
-    }
-    E* dst = conv_rope_dest<E>(p, t, c);
-    if (dst) store_vec<E, V>(dst, y);
-    if (halo > 0) {
+      float y[V];
 #pragma unroll
-      for (int j = 0; j + 1 < W; ++j)
+      for (int e = 0; e < V; ++e) y[e] = w[0][e] * x[W + j][e];
 #pragma unroll
-        for (int e = 0; e < V; ++e) win[j][e] = win[j + 1][e];
+      for (int k = W; k > 0; --k) {
+        if (k <= halo) {                        // (past the taps there may be another sequence's inputs)
 #pragma unroll
-      for (int e = 0; e < V; ++e) win[W - 1][e] = x[e];
-      if (t == s_hi - 1) {
+          for (int e = 0; e < V; ++e) y[e] = fmaf(w[k][e], x[W + j - k][e], y[e]);
+        }
+      }
+      if (turns) {
+        const float2* cs = s_cs + (row - r0) * (p.rot >> 1) + (d0 >> 1);
+#pragma unroll
+        for (int i = 0; i < V / 2; ++i) {
+          if (d0 + 2 * i < p.rot) {
+            const float2 a = cs[i];
+            const float u = y[2 * i], v = y[2 * i + 1];
+            y[2 * i] = u * a.x - v * a.y;
+            y[2 * i + 1] = v * a.x + u * a.y;
+          }
+        }
+      }
+      const int slot = is_q ? 0 : s_slot[row - r0];
+      const size_t off = is_q ? static_cast<size_t>(row) * p.nq : (slot >> 6) * page + (slot & 63) * per;
+      if (slot >= 0) store_vec<E, V>(dst0 + off, y);
+      if (halo > 0 && row == s_hi - 1) {        // the sequence's last halo inputs, oldest first
         float* st = p.state + static_cast<size_t>(p.state_out[seq]) * p.slot_stride + p.state_off + c;
 #pragma unroll
-        for (int j = 0; j < W; ++j) {
-          const int dst_row = j - (W - halo);
-          if (dst_row >= 0) store_vec<float, V>(st + static_cast<size_t>(dst_row) * C, win[j]);
-        }
+        for (int k = 0; k < W; ++k)
+          if (k < halo) store_vec<float, V>(st + static_cast<size_t>(halo - 1 - k) * C, x[W + j - k]);
       }
     }
+#pragma unroll
+    for (int i = 0; i < W; ++i)
+#pragma unroll
+      for (int e = 0; e < V; ++e) x[i][e] = x[kBatch + i][e];
   }
 }
 
@@ -206,7 +212,7 @@ __global__ void __launch_bounds__(256) conv_rope_kv_any_kernel(const ConvRope p)
       y = d & 1 ? y * k.x + o * k.y : y * k.x - o * k.y;
     }
   }
-  E* dst = conv_rope_dest<E>(p, t, c);
+  E* dst = conv_rope_dest<E>(p, t, c < p.nq ? 0 : p.slots[t], c);
   if (dst) {
     float v[1] = {y};
     store_vec<E, 1>(dst, v);
@@ -237,21 +243,24 @@ __global__ void __launch_bounds__(256) softcap_kernel(float* __restrict__ x, int
 template <typename E>
 static int launch_conv_rope(ConvRope p, cudaStream_t st) {
   const int C = p.nq + p.nk + p.nv;
-  const bool vec = p.dim % 8 == 0 && p.vdim % 8 == 0 && p.ld % 8 == 0 && p.q_off % 8 == 0 && p.k_off % 8 == 0 && p.v_off % 8 == 0 &&
+  const bool vec = p.dim % 4 == 0 && p.vdim % 4 == 0 && p.ld % 4 == 0 && p.q_off % 4 == 0 && p.k_off % 4 == 0 && p.v_off % 4 == 0 &&
                    p.state_off % 4 == 0 && p.slot_stride % 4 == 0 && (!p.conv_w || p.taps <= 8);
   if (!vec) {
     launch_pdl(conv_rope_kv_any_kernel<E>, dim3(p.T, (C + 255) / 256), dim3(256), 0, st, p);
     return static_cast<int>(cudaGetLastError());
   }
-  const int cols = (C / 8 + 127) / 128;
-  // decode: one token per block; prompts: runs long enough that re-reading their halo is cheap, blocks enough for every SM
-  const int want = 148 * 12;
+  const int cols = (C / 4 + 127) / 128;
+  // decode: one token per block; prompts: one wave of blocks, each with a run of tokens whose angles fit in shared memory
+  const int want = 148 * 7;
   int run = (p.T * cols + want - 1) / want;
   run = p.T <= 64 ? 1 : run < 4 ? 4 : run > 64 ? 64 : run;
-  p.run = run;
-  const dim3 grid((p.T + run - 1) / run, cols);
-  if (!p.conv_w || p.taps <= 4) launch_pdl(conv_rope_kv_kernel<E, 4>, grid, dim3(128), 0, st, p);
-  else launch_pdl(conv_rope_kv_kernel<E, 8>, grid, dim3(128), 0, st, p);
+  const int row_bytes = p.rot * 4 + 4, fit = 40 * 1024 / row_bytes;
+  if (fit < 1) return -12;
+  p.run = run < fit ? run : fit;
+  const dim3 grid((p.T + p.run - 1) / p.run, cols);
+  const size_t smem = static_cast<size_t>(p.run) * row_bytes;
+  if (!p.conv_w || p.taps <= 4) launch_pdl(conv_rope_kv_kernel<E, 4>, grid, dim3(128), smem, st, p);
+  else launch_pdl(conv_rope_kv_kernel<E, 8>, grid, dim3(128), smem, st, p);
   return static_cast<int>(cudaGetLastError());
 }
 
