@@ -60,7 +60,8 @@ __device__ __forceinline__ E* conv_rope_dest(const ConvRope& p, int t, int slot,
 __device__ __forceinline__ int conv_rope_col(const ConvRope& p, int c) {
   return c < p.nq ? p.q_off + c : c < p.nq + p.nk ? p.k_off + c - p.nq : p.v_off + c - p.nq - p.nk;
 }
-__device__ __forceinline__ int seq_of(const int* q_start, int S, int t) {
+__device__ __forceinline__ int seq_of(const int* q_start, int S, int T, int t) {
+  if (S == T && q_start[t] == t && q_start[t + 1] == t + 1) return t;     // decode: a token per sequence
   int s = 0, hi = S;
   while (hi - s > 1) {
     const int mid = (s + hi) >> 1;
@@ -88,11 +89,21 @@ __global__ void __launch_bounds__(128, MAXT <= 4 && sizeof(E) == 2 ? 7 : 2) conv
   pdl_wait();
   pdl_trigger();
   const int r0 = blockIdx.x * p.run, r1 = min(p.T, r0 + p.run);
+  const E* src = static_cast<const E*>(p.proj) + conv_rope_col(p, min(c, C - V));
+  Packed<E, V> nx[kBatch];                      // the next batch's rows, on their way while one is worked on
+#pragma unroll
+  for (int j = 0; j < kBatch; ++j) nx[j] = load_packed<E, V>(src + static_cast<size_t>(min(r0 + j, p.T - 1)) * p.ld);
+  int seq = 0, s_lo = 0, s_hi = p.T, s_in = 0;
+  if (halo > 0) {
+    seq = seq_of(p.q_start, p.S, p.T, r0);
+    s_lo = p.q_start[seq];
+    s_hi = p.q_start[seq + 1];
+    s_in = p.state_in[seq];
+  }
   for (int i = threadIdx.x; i < (r1 - r0) * (p.rot >> 1); i += blockDim.x) s_cs[i] = p.table[static_cast<size_t>(r0) * (p.rot >> 1) + i];
   for (int i = threadIdx.x; i < r1 - r0; i += blockDim.x) s_slot[i] = p.slots[r0 + i];
   __syncthreads();
   if (c >= C) return;
-  const E* src = static_cast<const E*>(p.proj) + conv_rope_col(p, c);
   const bool is_q = c < p.nq, is_v = c >= p.nq + p.nk;
   const int d0 = is_v ? p.rot : (is_q ? c : c - p.nq) % p.dim;   // first dimension inside its map; v: past the rotated ones
   const bool turns = d0 < p.rot;
@@ -100,20 +111,11 @@ __global__ void __launch_bounds__(128, MAXT <= 4 && sizeof(E) == 2 ? 7 : 2) conv
   E* const dst0 = is_q ? static_cast<E*>(p.q_out) + c : conv_rope_dest<E>(p, 0, 0, c);
   const int per = is_v ? p.vdim : p.maps_dim;
   const size_t page = static_cast<size_t>(p.kv_heads) * 64 * per;
-  int seq = 0, s_lo = 0, s_hi = p.T;
-  if (halo > 0) {
-    seq = seq_of(p.q_start, p.S, r0);
-    s_lo = p.q_start[seq];
-    s_hi = p.q_start[seq + 1];
-  }
   float x[W + kBatch][V];                       // a batch of kBatch tokens' inputs behind the W before it
 #pragma unroll
   for (int i = 0; i < W; ++i)
 #pragma unroll
     for (int e = 0; e < V; ++e) x[i][e] = 0.f;
-  Packed<E, V> nx[kBatch];                      // the next batch's rows, on their way while one is worked on
-#pragma unroll
-  for (int j = 0; j < kBatch; ++j) nx[j] = load_packed<E, V>(src + static_cast<size_t>(min(r0 + j, p.T - 1)) * p.ld);
   for (int t = r0; t < r1; t += kBatch) {
 #pragma unroll
     for (int j = 0; j < kBatch; ++j) unpack(nx[j], x[W + j]);
@@ -128,8 +130,13 @@ __global__ void __launch_bounds__(128, MAXT <= 4 && sizeof(E) == 2 ? 7 : 2) conv
       if (halo > 0 && (row == r0 || row == s_hi)) {
         // The inputs before a run's or a sequence's first token: rows of this step, or the state where they lie before it.
         // (The slots held another sequence's last inputs, which are done with.)
-        while (row == s_hi && seq + 1 < p.S) { ++seq; s_lo = s_hi; s_hi = p.q_start[seq + 1]; }      // empty sequences are skipped
-        const float* st = p.state + static_cast<size_t>(p.state_in[seq]) * p.slot_stride + p.state_off + c;
+        while (row == s_hi && seq + 1 < p.S) {  // (empty sequences are skipped)
+          ++seq;
+          s_lo = s_hi;
+          s_hi = p.q_start[seq + 1];
+          s_in = p.state_in[seq];
+        }
+        const float* st = p.state + static_cast<size_t>(s_in) * p.slot_stride + p.state_off + c;
 #pragma unroll
         for (int k = 1; k < MAXT; ++k) {
           if (k <= halo) {
@@ -188,7 +195,7 @@ __global__ void __launch_bounds__(256) conv_rope_kv_any_kernel(const ConvRope p)
   int seq = 0, s_lo = 0, s_hi = p.T;
   const float* st = nullptr;
   if (halo > 0) {
-    seq = seq_of(p.q_start, p.S, t);
+    seq = seq_of(p.q_start, p.S, p.T, t);
     s_lo = p.q_start[seq];
     s_hi = p.q_start[seq + 1];
     st = p.state + static_cast<size_t>(p.state_in[seq]) * p.slot_stride + p.state_off;

@@ -83,12 +83,12 @@ def _parallel_layers_from_json(d: dict) -> ModelConfig:
             raise ValueError(f"layer {i}: {rope.dims} rotated dims of {mixer.dim}")
         dense = None
         if mlp is not None:
-            if mlp.get("kind") != "dense":
-                raise ValueError(f"layer {i}: unsupported feed-forward {mlp.get('kind')!r}")
+            if mlp.get("kind") != "dense" or (mlp.get("act") or "silu") != "silu":
+                raise ValueError(f"layer {i}: unsupported feed-forward {mlp.get('kind')!r} {mlp.get('act') or ''}")
             dense = DenseSpec(mlp["ff"])
         specs.append(LayerSpec(mixer, dense=dense, parallel=True))
     lp = d.get("loop")
-    loop = (lp["start"], lp["stop"], lp["times"]) if lp else ()
+    loop = (lp["start"], lp["stop"], lp["times"]) if lp and lp["stop"] != lp["start"] else ()
     if loop and not (0 <= loop[0] < loop[1] <= len(specs) and loop[2] >= 1):
         raise ValueError(f"loop {loop} over {len(specs)} layers")
     return parallel_config(d.get("name", d["architecture"].lower()), d["vocab"], d["width"], specs, float(d["norm"]["eps"]), loop,

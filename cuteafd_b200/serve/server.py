@@ -534,7 +534,8 @@ def build_state(args) -> ServerState:
         else:
             cfg = PRESETS[args.preset or "qwen3-30b-a3b"]()
             if args.layers:
-                cfg = cfg.replace(num_layers=args.layers)
+                from ..config import scaled_down
+                cfg = scaled_down(cfg, args.layers, cfg.vocab_size) if cfg.is_hybrid else cfg.replace(num_layers=args.layers)
             kvf = getattr(args, "kv_format", "auto")
             if cfg.is_mla and (kvf == "fp8_ds_mla" or (kvf == "auto" and cfg.indexer_heads)):
                 cfg = cfg.replace(kv_format="fp8_ds_mla")

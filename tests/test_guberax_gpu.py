@@ -1,5 +1,6 @@
 """Stacks of parallel layers (differential attention beside a dense feed-forward, looped layers) on the GPU against the plain
-oracle: every kernel alone, then the engine through its serving backend."""
+oracle: every kernel alone, then the engine through its serving backend (greedy generation through the scheduler is with the
+other per-layer designs' in test_hybrid_gpu.py)."""
 import dataclasses
 import json
 import os
@@ -13,7 +14,7 @@ from cuteafd_b200.config import RopeSpec
 from cuteafd_b200.ref import hybrid as R
 
 from tests.hybrid_common import attention, bare_config, err, looped_config, oracle_logits, paired_config, params, tokens, write_model
-from tests.test_hybrid_gpu import DTYPES, _greedy, backend, check, close, dev, i32, rnd, run_cut
+from tests.test_hybrid_gpu import DTYPES, backend, check, close, dev, i32, rnd, run_cut
 
 pytestmark = pytest.mark.gpu
 
@@ -353,36 +354,6 @@ def test_far_keys_and_kept_tokens_in_the_engine(name):
         other = err(oracle_logits(cfg.replace(layer_specs=specs), p, toks), want)
         if dtype == "f32":
             assert other[150:].median() > 20 * e[150:].median()
-
-
-@pytest.mark.parametrize("draft,graphs", [(False, False), (False, True), (True, True)])
-def test_scheduler_generates_like_the_oracle(draft, graphs):
-    from cuteafd_b200.runtime.scheduler import Request, Scheduler, collect
-    from cuteafd_b200.runtime.speculation import NgramDrafter
-    cfg = looped_config()
-    p = params(cfg)
-    prompts = [tokens(70, cfg.vocab_size, 1), (tokens(5, cfg.vocab_size, 2) * 8)[:37], tokens(140, cfg.vocab_size, 3)]
-    n = 40
-    truth = [_greedy(cfg, p, q, n) for q in prompts]
-    again = prompts[0] + truth[0][:n - 1] + [3, 4]
-    be = backend(cfg, p, pages=60, chunk=96, slots=2 + 24, graphs=graphs)
-    sched = Scheduler(be, drafter=NgramDrafter(block=3) if draft else None)
-    reqs = [sched.submit(Request(list(q), max_tokens=n)) for q in prompts]
-    for _ in range(400):
-        if not sched.step() and not sched.pending and sched.waiting.empty():
-            break
-    for t, r in zip(truth, reqs):
-        got = collect(r, 1.0)
-        assert got["error"] is None and got["tokens"] == t
-    r = sched.submit(Request(list(again), max_tokens=6))           # resumes from a snapshot: pages and a state slot are shared
-    while sched.step():
-        pass
-    got = collect(r, 1.0)
-    assert got["tokens"] == _greedy(cfg, p, again, 6) and got["usage"]["cached_tokens"] >= 70
-    if graphs and not draft:
-        assert be.graph_stats["replays"] > 10
-    be.prefix.clear()
-    assert be.pool.free_pages == be.pool.usable_pages and be.states.free_slots == 24
 
 
 @pytest.mark.parametrize("cfg,dtype", [(looped_config(), "f32"), (paired_config(), "bf16")], ids=["looped", "paired"])

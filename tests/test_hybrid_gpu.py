@@ -10,7 +10,7 @@ import torch
 from cuteafd_b200.config import RouterSpec
 from cuteafd_b200.ref import hybrid as R
 
-from tests.hybrid_common import delta, err, latent, narrow_config, odd_config, oracle_logits, params, plain_config, tokens, wide_config, write_model
+from tests.hybrid_common import delta, err, latent, looped_config, narrow_config, odd_config, oracle_logits, params, plain_config, tokens, wide_config, write_model
 
 pytestmark = pytest.mark.gpu
 DTYPES = [torch.float32, torch.bfloat16]
@@ -501,8 +501,9 @@ def _greedy(cfg, p, prompt, n):
     return out
 
 
+@pytest.mark.parametrize("cfg", [odd_config(), looped_config()], ids=lambda c: c.name)
 @pytest.mark.parametrize("draft,graphs", [(False, False), (False, True), (True, True)])
-def test_scheduler_generates_like_the_oracle(draft, graphs):
+def test_scheduler_generates_like_the_oracle(draft, graphs, cfg):
     from cuteafd_b200.runtime.scheduler import Request, Scheduler, collect
     from cuteafd_b200.runtime.speculation import DrafterSpec
 
@@ -526,7 +527,6 @@ def test_scheduler_generates_like_the_oracle(draft, graphs):
 
         def forget(self, rid):
             pass
-    cfg = odd_config()
     p = params(cfg)
     prompts = [tokens(70, cfg.vocab_size, 1), tokens(5, cfg.vocab_size, 2), tokens(140, cfg.vocab_size, 3)]
     n = 40
