@@ -1,4 +1,6 @@
 """Small per-layer hybrid configurations and helpers shared by the hybrid tests."""
+import dataclasses
+
 import torch
 
 from cuteafd_b200.config import (AttentionSpec, DeltaSpec, DenseSpec, LatentSpec, LayerSpec, RopeSpec, RouterSpec, hybrid_config,
@@ -79,6 +81,14 @@ def paired_config(window=100, keep=70):
     return parallel_config("paired", 500, 256, [
         parallel(attention(4, 2, 64, 128, window, keep, RopeSpec(64, 1e5, 4.0, 1.0, 4.0, 256), 4, 0.6), 192),
         parallel(attention(8, 1, 64, 128, 2 * window + 3, 3, RopeSpec(32, 1e4), 3, 0.2), 136)], 1e-5, loop=(0, 2, 2), logit_softcap=30.0)
+
+
+def single_map_config():
+    """Plain attention (one map per head) in the same layers, at sizes of both kinds of kernels."""
+    one = lambda m: dataclasses.replace(m, maps=1, diff=0.0)                    # noqa: E731
+    return parallel_config("single", 300, 192, [
+        parallel(one(attention(4, 2, 128, 128, 90, 10, RopeSpec(64, 1e5), 3)), 88),
+        parallel(one(attention(3, 1, 20, 12, 50, 66, RopeSpec(20, 1e3), 2)), 40)], 1e-5, loop=(1, 2, 2))
 
 
 def params(cfg, seed=0, spread=0.4):

@@ -13,7 +13,7 @@ import torch
 from cuteafd_b200.config import RopeSpec
 from cuteafd_b200.ref import hybrid as R
 
-from tests.hybrid_common import attention, bare_config, err, looped_config, oracle_logits, paired_config, params, tokens, write_model
+from tests.hybrid_common import attention, bare_config, err, looped_config, oracle_logits, paired_config, params, single_map_config, tokens, write_model
 from tests.test_hybrid_gpu import DTYPES, backend, check, close, dev, i32, rnd, run_cut
 
 pytestmark = pytest.mark.gpu
@@ -175,13 +175,17 @@ def test_attention_windows_and_kept_tokens(dtype, m, edge):
         return
     kw = dict(scale=m.scale, window=m.window, keep=m.keep_first, maps=2, lam=lam, out_scale=1 - m.diff, eps=eps)
     q = q.view(T, m.heads, 128)
-    for splits in (0, 1, 2, 5):
+    for splits, fixed in ((0, 0), (1, 0), (2, 0), (5, 0), (9, 64), (5, 128)):
         out = torch.full((T, m.heads * 128 + 16), 5.0, dtype=dtype, device=dev())
         if splits == 0:
             K.attn_prefill(q, kc, vc, table, i32(lens), i32(q_start), out, max(q_lens), **kw)
         else:
             sc = torch.empty(K.attn_decode_scratch_floats(len(lens), max(q_lens), 2 * m.heads, m.kv_heads, splits), device=dev())
-            K.attn_decode(q, kc, vc, table, i32(lens), i32(q_start), out, sc, max(q_lens), splits, **kw)
+            K.set_fixed_kv_split(fixed)
+            try:
+                K.attn_decode(q, kc, vc, table, i32(lens), i32(q_start), out, sc, max(q_lens), splits, **kw)
+            finally:
+                K.set_fixed_kv_split(0)
         close(out[:, :m.heads * 128].view(T, m.heads, 128), want, dtype, k)
         assert (out[:, m.heads * 128:] == 5.0).all()
     assert K.read_status() == 0
@@ -222,7 +226,7 @@ def test_softcap():
 
 
 # ---- engine ------------------------------------------------------------------------------------------------------------
-CASES = [(c, d) for c in (looped_config(), bare_config(), paired_config()) for d in ("f32", "bf16")]
+CASES = [(c, d) for c in (looped_config(), bare_config(), paired_config(), single_map_config()) for d in ("f32", "bf16")]
 IDS = [f"{c.name}-{d}" for c, d in CASES]
 
 
