@@ -78,35 +78,36 @@ class MoeLayout(C.Structure):
 
 class NormArgs(C.Structure):
     """cafd_norm_conv (csrc/hybrid_norm.cu)."""
-    _fields_ = [(n, C.c_void_p) for n in ("tokens", "embed", "x_in", "y", "slot_w", "slot_idx", "ident", "w_b", "w", "conv", "x_out",
-                                          "h_out", "row_idx", "state", "state_in", "state_out", "q_start")]
+    _fields_ = [(n, C.c_void_p) for n in ("tokens", "embed", "x_in", "y", "slot_w", "slot_idx", "ident", "w_b", "w", "base", "step",
+                                          "w2", "h2_out", "conv", "x_out", "h_out", "row_idx", "state", "state_in", "state_out", "q_start")]
     _fields_ += [("slot_stride", C.c_longlong), ("state_off", C.c_longlong)]
-    _fields_ += [(n, C.c_int) for n in ("T", "H", "S", "ldy", "ldh", "groups", "taps", "top_k", "n_experts", "vocab", "run")]
-    _fields_ += [("eps", C.c_float), ("w_off", C.c_float)]
+    _fields_ += [(n, C.c_int) for n in ("T", "H", "S", "ldy", "ldh", "ldb", "groups", "taps", "top_k", "n_experts", "vocab", "run")]
+    _fields_ += [(n, C.c_float) for n in ("eps", "w_off", "e_scale")]
 
 
 class ConvRope(C.Structure):
     """cafd_conv_rope_kv (csrc/conv_rope.cu)."""
     _fields_ = [(n, C.c_void_p) for n in ("proj", "conv_w", "table", "slots", "q_start", "state_in", "state_out", "state", "q_out",
-                                          "k_cache", "v_cache")]
+                                          "k_cache", "v_cache", "q_norm", "k_norm")]
     _fields_ += [("slot_stride", C.c_longlong), ("state_off", C.c_longlong)]
     _fields_ += [(n, C.c_int) for n in ("T", "S", "ld", "q_off", "k_off", "v_off", "nq", "nk", "nv", "maps_dim", "dim", "vdim", "kv_heads",
-                                        "rot", "taps", "run")]
+                                        "rot", "taps", "run", "norm", "halves", "v_from_k", "units")]
+    _fields_ += [("eps", C.c_float)]
 
 
 class PagedAttn(C.Structure):
     """cafd_paged_attn (csrc/attention_any.cu)."""
-    _fields_ = [(n, C.c_void_p) for n in ("q", "k_cache", "v_cache", "page_table", "positions", "q_start", "out")]
+    _fields_ = [(n, C.c_void_p) for n in ("q", "k_cache", "v_cache", "page_table", "positions", "q_start", "out", "sink", "gate")]
     _fields_ += [(n, C.c_int) for n in ("T", "S", "heads", "kv_heads", "maps", "dim", "vdim", "window", "keep", "max_pages", "ldo",
-                                        "head_pitch", "heads_per_block")]
+                                        "head_pitch", "heads_per_block", "gate_ld")]
     _fields_ += [(n, C.c_float) for n in ("scale", "lam", "out_scale", "eps")]
 
 
 class LatentPrep(C.Structure):
     """cafd_latent_prep (csrc/latent.cu)."""
     _fields_ = [(n, C.c_void_p) for n in ("a", "norm_w", "inv_freq", "positions", "slots", "cache", "slab", "q_abs", "lat_out")]
-    _fields_ += [(n, C.c_int) for n in ("lda", "q_off", "kv_off", "heads", "dim", "rot", "rank", "rec", "dim_pad", "t_pad", "T")]
-    _fields_ += [("eps", C.c_float)]
+    _fields_ += [(n, C.c_int) for n in ("lda", "q_off", "kv_off", "heads", "dim", "rot", "rank", "rec", "dim_pad", "t_pad", "T", "halves")]
+    _fields_ += [("eps", C.c_float), ("mag", C.c_float)]
 
 
 class LatentAttn(C.Structure):
@@ -196,12 +197,12 @@ def cuda_lib():
         _sig(lib, "cafd_moe_dispatch", [P, P, P, I, I, I, C.POINTER(MoeLayout), P, P, P])
         _sig(lib, "cafd_moe_combine", [P, P, P, P, P, I, I, I, P, I, P, P, P])
         _sig(lib, "cafd_attn_decode_scratch_floats", [I, I, I, I], C.c_longlong)
-        _sig(lib, "cafd_attn_decode", [P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, F, I, I, I, I, F, F, F, P])
+        _sig(lib, "cafd_attn_decode", [P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, F, I, I, I, I, F, F, F, P, P, I, P])
         _sig(lib, "cafd_attn_decode_partial", [P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, F, P])
         _sig(lib, "cafd_attn_merge", [P, P, P, I, I, I, I, I, P])
         _sig(lib, "cafd_set_fixed_kv_split", [I])
         _sig(lib, "cafd_fixed_kv_split", [])
-        _sig(lib, "cafd_attn_prefill", [P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, F, I, I, I, I, F, F, F, P])
+        _sig(lib, "cafd_attn_prefill", [P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, F, I, I, I, I, F, F, F, P, P, I, P])
         _sig(lib, "cafd_mla_scratch_floats", [I, I], C.c_longlong)
         _sig(lib, "cafd_mla_attention", [P, P, P, P, P, P, P, P, P, P, C.c_longlong, I, I, I, I, I, I, F, P, I, I, P])
         _sig(lib, "cafd_indexer_scores", [P, P, P, I, F, P, P, P, P, P, P, P, C.c_longlong, I, I, I, I, I, I, P])
@@ -213,7 +214,7 @@ def cuda_lib():
         _sig(lib, "cafd_mla_attention_partial", [P, P, P, P, P, P, P, P, P, I, I, P, C.c_longlong, I, I, I, I, I, F, P])
         _sig(lib, "cafd_mla_merge", [P, P, P, P, P, I, I, I, I, P])
         _sig(lib, "cafd_mla_attention_gathered", [P, P, P, P, P, P, P, P, P, P, C.c_longlong, I, I, I, I, I, F, P, I, P])
-        _sig(lib, "cafd_attn_prefill_mla", [P, I, I, P, I, I, P, P, C.c_longlong, P, P, P, P, P, P, P, I, I, I, I, I, I, F, I, P])
+        _sig(lib, "cafd_attn_prefill_mla", [P, I, I, P, I, I, P, P, C.c_longlong, P, P, P, P, P, P, P, I, I, I, I, I, I, F, I, I, P])
         _sig(lib, "cafd_gemm_w4", [C.POINTER(GemmArgs), I, P, P, P])
         _sig(lib, "cafd_w4_dequant", [P, P, P, P, C.c_longlong, I, I, I, P])
         _sig(lib, "cafd_fp8_dequant_block128", [P, P, P, C.c_longlong, I, P])
@@ -221,7 +222,7 @@ def cuda_lib():
         _sig(lib, "cafd_sample_rows", [P, I, I, P, P, I, P, P, P])
         _sig(lib, "cafd_accept_prefix", [P, P, P, I, P, P, P])
         _sig(lib, "cafd_norm_conv", [C.POINTER(NormArgs), I, P])
-        _sig(lib, "cafd_rope_table", [P, P, P, I, I, P])
+        _sig(lib, "cafd_rope_table", [P, P, P, I, I, F, P])
         _sig(lib, "cafd_conv_rope_kv", [C.POINTER(ConvRope), I, P])
         _sig(lib, "cafd_softcap", [P, I, I, C.c_longlong, F, P])
         _sig(lib, "cafd_paged_attn", [C.POINTER(PagedAttn), I, P])
@@ -235,8 +236,8 @@ def cuda_lib():
         _sig(lib, "cafd_delta_step", [C.POINTER(DeltaArgs), I, P])
         _sig(lib, "cafd_mla_q_split", [P, I, P, P, P, P, I, I, I, I, P])
         _sig(lib, "cafd_mla_small_rows", [])
-        _sig(lib, "cafd_mla_absorb_small", [P, I, P, P, P, P, I, I, I, P])
-        _sig(lib, "cafd_mla_unabsorb_small", [P, I, P, P, I, I, P, I, P])
+        _sig(lib, "cafd_mla_absorb_small", [P, I, P, P, P, P, I, I, I, F, P])
+        _sig(lib, "cafd_mla_unabsorb_small", [P, I, P, P, I, I, P, I, I, P])
         _cuda = lib
         return lib
 

@@ -10,14 +10,40 @@ from __future__ import annotations
 
 import dataclasses
 import json
+import math
 from dataclasses import dataclass, field
 from typing import Any
 
 
 @dataclass(frozen=True)
+class RopeSpec:
+    """Rotary positions on the first ``dims`` dimensions of a head: pairs (2i, 2i + 1), or (i, i + dims / 2) with ``halves``.
+    ``factor`` other than 1 stretches the frequencies as ``kind`` says:
+
+    bands    wavelengths above ``original / low`` are divided by it, those below ``original / high`` are kept, the band between is
+             blended linearly in the number of turns over ``original`` positions
+    linear   every frequency is divided by it
+    yarn     between the pairs that make ``high`` and ``low`` turns over ``original`` positions the blend is linear in the pair's
+             index, and cosines and sines carry a ``magnitude``"""
+    dims: int
+    base: float
+    factor: float = 1.0
+    low: float = 1.0
+    high: float = 4.0
+    original: int = 0
+    kind: str = "bands"
+    halves: bool = False
+
+    @property
+    def magnitude(self) -> float:
+        return 0.1 * math.log(self.factor) + 1.0 if self.kind == "yarn" else 1.0
+
+
+@dataclass(frozen=True)
 class LatentSpec:
     """Latent attention of one layer: all heads' keys and values come out of a normed latent of ``kv_rank`` values plus one
-    shared rotated key part of ``rot_dim``; a query at position i sees the last ``window`` positions (0 = all of them)."""
+    shared rotated key part of ``rot_dim``; a query at position i sees the last ``window`` positions (0 = all of them).  ``gate``:
+    every output value is multiplied by the sigmoid of a projected one."""
     heads: int
     dim: int                             # unrotated query / key dims per head
     rot_dim: int
@@ -25,7 +51,8 @@ class LatentSpec:
     kv_rank: int
     window: int
     scale: float
-    rope_base: float
+    rope: RopeSpec
+    gate: bool = True
 
     @property
     def record(self) -> int:
@@ -48,24 +75,16 @@ class DeltaSpec:
 
 
 @dataclass(frozen=True)
-class RopeSpec:
-    """Rotary positions on the first ``dims`` dimensions of a head, pairs (2i, 2i + 1).  ``factor`` other than 1: frequencies
-    whose wavelength is above ``original / low`` are divided by it, those below ``original / high`` are kept, the band between
-    is blended linearly in the number of turns over ``original`` positions."""
-    dims: int
-    base: float
-    factor: float = 1.0
-    low: float = 1.0
-    high: float = 4.0
-    original: int = 0
-
-
-@dataclass(frozen=True)
 class AttentionSpec:
     """Softmax attention of one layer over paged keys and values, with a causal convolution of ``conv`` taps on the channels of
     q, k and v (0 = none).  A query at position i sees the last ``window`` positions (0 = all of them) and the first
     ``keep_first`` ones.  ``maps`` 2 is differential attention: two score maps per head over the same values, combined as
-    map 1 - lambda * map 2, the difference normed per head and scaled by 1 - ``diff`` (lambda's constant part)."""
+    map 1 - lambda * map 2, the difference normed per head and scaled by 1 - ``diff`` (lambda's constant part).
+
+    ``qk_norm``: RMS norm of queries and keys before their rotation, per head ("head", one weight vector for all heads) or over the
+    whole projection ("all").  ``v_from_k``: the values are the convolved keys before norm and rotation.  ``sink``: a learned
+    number per head whose exponential joins the softmax's denominator.  ``gate``: a head's output is multiplied by the sigmoid of
+    one projected number."""
     heads: int
     kv_heads: int
     dim: int                             # query / key dims per map and head
@@ -77,6 +96,10 @@ class AttentionSpec:
     conv: int = 0
     maps: int = 1
     diff: float = 0.0
+    qk_norm: str = ""                    # "" | "head" | "all"
+    v_from_k: bool = False
+    sink: bool = False
+    gate: bool = False
 
     @property
     def q_channels(self) -> int:
@@ -92,7 +115,8 @@ class AttentionSpec:
 
     @property
     def conv_channels(self) -> int:
-        return self.q_channels + self.k_channels + self.v_channels
+        """Projected channels of q, k and v (those the convolution runs over)."""
+        return self.q_channels + self.k_channels + (0 if self.v_from_k else self.v_channels)
 
 
 @dataclass(frozen=True)
@@ -104,13 +128,17 @@ class DenseSpec:
 @dataclass(frozen=True)
 class RouterSpec:
     """Routed feed-forward of one layer: ``experts`` SwiGLU experts of width ``ffn`` and ``identity`` outputs that hand the
-    input through; ``top`` of them per token out of the best ``groups_kept`` of ``groups``."""
+    input through; ``top`` of them per token out of the best ``groups_kept`` of ``groups``.  The router's bias takes part in the
+    selection alone, or with ``logit_bias`` is part of the logits; the weights are the chosen scores, with ``normalize`` divided by
+    their sum."""
     experts: int
     ffn: int
     top: int
     identity: int = 0
     groups: int = 1
     groups_kept: int = 1
+    logit_bias: bool = False
+    normalize: bool = False
 
     @property
     def outputs(self) -> int:
@@ -121,20 +149,20 @@ class RouterSpec:
 class LayerSpec:
     mixer: Any                           # LatentSpec | DeltaSpec | AttentionSpec
     router: RouterSpec | None = None     # None = the layer has no routed feed-forward
-    dense: DenseSpec | None = None       # dense feed-forward (parallel layers)
+    dense: DenseSpec | None = None       # dense feed-forward (parallel layers); beside a router: the shared expert
     # parallel: mixer and feed-forward read one norm and are added together, nothing is normed after them; otherwise the
     # sublayers follow one another, each with a norm before and after it and a convolution on its input
     parallel: bool = False
+    two_norms: bool = False              # parallel: the feed-forward reads a norm of its own
 
     @staticmethod
     def from_dict(d: dict[str, Any]) -> "LayerSpec":
-        m = d["mixer"]
+        m = dict(d["mixer"])
         if "rope" in m:
-            mixer = AttentionSpec(**{**m, "rope": RopeSpec(**m["rope"])})
-        else:
-            mixer = LatentSpec(**m) if "kv_rank" in m else DeltaSpec(**m)
-        return LayerSpec(mixer, RouterSpec(**d["router"]) if d.get("router") else None,
-                         DenseSpec(**d["dense"]) if d.get("dense") else None, bool(d.get("parallel", False)))
+            m["rope"] = RopeSpec(**m["rope"])
+        mixer = (LatentSpec if "kv_rank" in m else AttentionSpec if "rope" in m else DeltaSpec)(**m)
+        return LayerSpec(mixer, RouterSpec(**d["router"]) if d.get("router") else None, DenseSpec(**d["dense"]) if d.get("dense") else None,
+                         bool(d.get("parallel", False)), bool(d.get("two_norms", False)))
 
 
 @dataclass(frozen=True)
@@ -142,6 +170,7 @@ class LayerRun:
     """One run of a layer: looped layers run several times with the same weights, each run with its own cache and state."""
     layer: int
     add_embedding: bool = False          # the embedding row is added to the residual right before this run
+    join: int = -1                       # pass t >= 0 starts here: x = W [x; embedding row] + step vector t
 
 
 @dataclass(frozen=True)
@@ -207,6 +236,8 @@ class ModelConfig:
     norm_groups: int = 1                 # channel groups of the RMS norms
     norm_offset: float = 0.0             # added to the stored norm weights (1: they are stored around zero)
     loop: tuple = ()                     # (start, stop, times): layers [start, stop) run ``times`` times in a row
+    loop_join: bool = False              # every pass starts with a product of [x; embedding row] and adds a vector of its own
+    embed_scale: float = 1.0             # the embedding's rows are multiplied by it
     logit_softcap: float = 0.0           # logits = cap * tanh(logits / cap); 0 = none
     compute_dtype: str = "bf16"          # bf16 | f32 (every product and activation in 32-bit; hybrid engine only)
 
@@ -227,10 +258,9 @@ class ModelConfig:
     def layer_runs(self) -> tuple:
         """The layers in the order they run (``LayerRun``), loops unrolled."""
         start, stop, times = self.loop or (0, 0, 1)
-        once = [LayerRun(i) for i in range(start, stop)]
-        again = [LayerRun(i, i == start) for i in range(start, stop)]
-        return tuple([LayerRun(i) for i in range(start)] + once + again * (times - 1)
-                     + [LayerRun(i) for i in range(stop, self.num_layers)])
+        passes = [LayerRun(i, not self.loop_join and t > 0 and i == start, t if self.loop_join and i == start else -1)
+                  for t in range(times) for i in range(start, stop)]
+        return tuple([LayerRun(i) for i in range(start)] + passes + [LayerRun(i) for i in range(stop, self.num_layers)])
 
     @property
     def state_bytes(self) -> int:
@@ -289,10 +319,11 @@ class ModelConfig:
     def mixer_params(self, layer: int) -> int:
         h, m = self.hidden, self.layer_specs[layer].mixer
         if isinstance(m, AttentionSpec):
-            return (h * (m.conv_channels + m.heads * m.vdim) + m.conv * m.conv_channels
+            norms = {"": 0, "head": 2 * m.dim, "all": m.q_channels + m.k_channels}[m.qk_norm]
+            return (h * (m.conv_channels + m.heads * m.vdim + m.heads * m.gate) + m.conv * m.conv_channels + norms + m.heads * m.sink
                     + (4 * m.dim if m.maps == 2 else 0))
         if isinstance(m, LatentSpec):
-            return (h * (m.heads * (m.dim + m.rot_dim) + m.record + 2 * m.heads * m.vdim)
+            return (h * (m.heads * (m.dim + m.rot_dim) + m.record + (1 + m.gate) * m.heads * m.vdim)
                     + m.kv_rank * (1 + m.heads * (m.dim + m.vdim)))
         return h * (m.conv_channels + 2 * m.heads + 2 * m.heads * m.vdim) + m.conv * m.conv_channels + 2 * m.heads + m.vdim
 
@@ -314,12 +345,15 @@ class ModelConfig:
 
     def layer_params(self, layer: int) -> int:
         if self.is_hybrid:
-            r, d = self.layer_specs[layer].router, self.layer_specs[layer].dense
-            if self.layer_specs[layer].parallel:
-                return self.mixer_params(layer) + self.hidden + (3 * self.hidden * d.ffn if d is not None else 0)
-            p = self.mixer_params(layer) + (2 + self.canon_taps) * self.hidden
+            spec = self.layer_specs[layer]
+            r, d = spec.router, spec.dense
+            routed = r.outputs * (self.hidden + 1) + 3 * r.experts * self.hidden * r.ffn if r is not None else 0
+            if spec.parallel:
+                norms = 2 if spec.two_norms and (r is not None or d is not None) else 1
+                return self.mixer_params(layer) + norms * self.hidden + routed + (3 * self.hidden * d.ffn if d is not None else 0)
+            p = self.mixer_params(layer) + (2 + self.canon_taps) * self.hidden + routed
             if r is not None:
-                p += (2 + self.canon_taps) * self.hidden + r.outputs * (self.hidden + 1) + 3 * r.experts * self.hidden * r.ffn
+                p += (2 + self.canon_taps) * self.hidden
             return p
         p = self.attention_params() + 2 * self.hidden
         if self.is_moe_layer(layer):
@@ -331,6 +365,8 @@ class ModelConfig:
 
     def total_params(self) -> int:
         p = self.vocab_size * self.hidden * (1 if self.tie_embeddings else 2) + self.hidden
+        if self.loop and self.loop_join:
+            p += (2 * self.hidden + self.loop[2]) * self.hidden
         return p + sum(self.layer_params(i) for i in range(self.num_layers))
 
     def to_json(self) -> str:
@@ -437,25 +473,26 @@ def hybrid_config(name: str, vocab: int, hidden: int, specs, canon_taps: int, no
     big = max(lat, key=lambda m: m.heads * (m.dim + m.rot_dim), default=None)
     wide = max(routers, key=lambda r: r.experts * r.ffn, default=None)
     top = max(att, key=lambda m: m.conv_channels, default=None)
-    rope = big.rope_base if big else top.rope.base if top else 10000.0
+    rope = big.rope if big else top.rope if top else RopeSpec(0, 10000.0, halves=True)
     head_dim = (big.dim + big.rot_dim) if big else (top.maps * top.dim) if top else specs[0].mixer.dim
     return ModelConfig(
         name=name, family=family, vocab_size=vocab, num_layers=len(specs), hidden=hidden, attention="hybrid", layer_specs=specs,
-        canon_taps=canon_taps, norm_groups=norm_groups, rms_eps=eps, rope_interleaved=not lat and bool(att),
+        canon_taps=canon_taps, norm_groups=norm_groups, rms_eps=eps, rope_interleaved=not rope.halves,
         num_heads=max(s.mixer.heads for s in specs), num_kv_heads=top.kv_heads if top else 1, head_dim=head_dim,
         q_lora_rank=0, kv_lora_rank=big.kv_rank if big else 0, qk_nope_dim=big.dim if big else 0, qk_rope_dim=big.rot_dim if big else 0,
-        v_head_dim=big.vdim if big else specs[0].mixer.vdim, rope_theta=rope,
-        sliding_window=max((m.window for m in lat + att), default=0), dense_ffn=max((s.dense.ffn for s in specs if s.dense), default=0),
+        v_head_dim=big.vdim if big else specs[0].mixer.vdim, rope_theta=rope.base,
+        sliding_window=max((m.window for m in lat + att), default=0), dense_ffn=max((s.dense.ffn for s in specs if s.dense and not s.router), default=0),
         first_dense_layers=0, num_experts=wide.experts if wide else 0, expert_ffn=wide.ffn if wide else 0, top_k=wide.top if wide else 0,
-        num_groups=wide.groups if wide else 1, topk_groups=wide.groups_kept if wide else 1, num_shared_experts=0,
-        norm_topk_prob=False, router_bias=bool(routers), **kw)
+        num_groups=wide.groups if wide else 1, topk_groups=wide.groups_kept if wide else 1, num_shared_experts=int(any(s.router and s.dense for s in specs)),
+        norm_topk_prob=bool(wide and wide.normalize), router_bias=bool(routers), **kw)
 
 
 def parallel_config(name: str, vocab: int, hidden: int, specs, eps: float, loop: tuple = (), logit_softcap: float = 0.0,
-                    family: str = "guberax") -> ModelConfig:
-    """ModelConfig of a stack of parallel layers: norm weights stored around zero, an optional loop, capped logits."""
+                    family: str = "guberax", **kw: Any) -> ModelConfig:
+    """ModelConfig of a stack of parallel layers: norm weights stored around zero, an optional loop, capped logits.  ``kw``: further
+    fields (loop_join, embed_scale)."""
     return hybrid_config(name, vocab, hidden, specs, canon_taps=1, norm_groups=1, eps=eps, family=family, norm_offset=1.0,
-                         loop=tuple(loop), logit_softcap=logit_softcap)
+                         loop=tuple(loop), logit_softcap=logit_softcap, **kw)
 
 
 # Benchmark sizes: width, layers, heads, expert width (latent 512 + 64 and heads of 128 throughout, as real models have them)
@@ -467,7 +504,8 @@ def karusun_bench(size: str = "base") -> ModelConfig:
     which the last eight hand their input through): three delta-rule layers to one latent attention layer."""
     width, layers, heads, ffn = KARUSUN_SIZES[size]
     r = RouterSpec(experts=56, ffn=ffn, top=6, identity=8, groups=8, groups_kept=4)
-    lat = LatentSpec(heads=heads, dim=128, rot_dim=64, vdim=128, kv_rank=512, window=2048, scale=192 ** -0.5, rope_base=1.0e6)
+    lat = LatentSpec(heads=heads, dim=128, rot_dim=64, vdim=128, kv_rank=512, window=2048, scale=192 ** -0.5,
+                     rope=RopeSpec(64, 1.0e6, halves=True))
     delta = DeltaSpec(heads=heads, kv_heads=heads // 2, dim=128, vdim=128, conv=4)
     specs = [LayerSpec(lat if i % 4 == 3 else delta, r) for i in range(layers)]
     return hybrid_config(f"karusun-{size}", 65536, width, specs, canon_taps=4, norm_groups=4, eps=1e-5)
@@ -528,6 +566,7 @@ def scaled_down(cfg: ModelConfig, layers: int = 2, vocab: int = 2048) -> ModelCo
         start, stop, times = cfg.loop or (0, 0, 1)
         return hybrid_config(cfg.name + "-mini", vocab, cfg.hidden, cfg.layer_specs[:layers], cfg.canon_taps, cfg.norm_groups,
                              cfg.rms_eps, cfg.family, norm_offset=cfg.norm_offset, logit_softcap=cfg.logit_softcap,
+                             loop_join=cfg.loop_join, embed_scale=cfg.embed_scale,
                              loop=(start, min(stop, layers), times) if start < layers and cfg.loop else ())
     first_dense = min(cfg.first_dense_layers, max(layers - 1, 0)) if cfg.first_dense_layers else 0
     return cfg.replace(name=cfg.name + "-mini", num_layers=layers, vocab_size=vocab,

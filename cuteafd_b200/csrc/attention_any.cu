@@ -1,5 +1,5 @@
 // Softmax attention over paged keys and values at any head sizes, with a sliding window and kept first tokens, and with one or
-// two score maps per head (the tensor-core kernels of attention_prefill.cu and attention_decode.cu serve 128-wide key and value
+// two score maps per head; a head may have a sink and an output gate (the tensor-core kernels of attention_prefill.cu and attention_decode.cu serve 128-wide key and value
 // rows; this file serves every other size and the fp32 engines).
 //
 // One block per (token, kv head, run of its query heads).  Keys are walked in tiles that start at multiples of 32, first those
@@ -20,7 +20,9 @@ struct PagedAttn {
   const int* positions;       // [T]
   const int* q_start;         // [S + 1]
   void* out;                  // [T, ldo] E: head h's values at h * head_pitch
-  int T, S, heads, kv_heads, maps, dim, vdim, window, keep, max_pages, ldo, head_pitch, heads_per_block;
+  const float* sink;          // [heads] or null: exp(sink) joins the denominator; one map only
+  const void* gate;           // row t, head h: E gate[t * gate_ld + h], the head's values are multiplied by its sigmoid; or null; one map only
+  int T, S, heads, kv_heads, maps, dim, vdim, window, keep, max_pages, ldo, head_pitch, heads_per_block, gate_ld;
   float scale, lambda, out_scale, eps;
 };
 
@@ -124,7 +126,9 @@ __global__ void __launch_bounds__(kAnyThreads) paged_attn_kernel(const PagedAttn
     const int e = tid + k * kAnyThreads;
     if (e < n_acc) {
       const int r = e / p.vdim, d = e - r * p.vdim;
-      float v[1] = {acc[k] / sm_l[r]};
+      const float l = p.sink ? sm_l[r] + expf(p.sink[h0 + r] - sm_m[r]) : sm_l[r];
+      float v[1] = {acc[k] / l};
+      if (p.gate) v[0] /= 1.0f + expf(-ld_e<E>(static_cast<const E*>(p.gate) + static_cast<size_t>(t) * p.gate_ld + h0 + r));
       if (p.maps == 1) store_vec<E, 1>(out + (h0 + r) * p.head_pitch + d, v);
       else so[e] = v[0];
     }
@@ -156,7 +160,8 @@ extern "C" int cafd_paged_attn(const PagedAttn* args, int is_f32, cafd_stream_t 
   PagedAttn p = *args;
   if (p.T <= 0) return 0;
   if (p.S < 1 || p.kv_heads < 1 || p.heads % p.kv_heads || p.maps < 1 || p.maps > 2 || p.dim < 1 || p.vdim < 1 || p.window < 0 || p.keep < 0 ||
-      p.maps * p.vdim > kAnyAcc * kAnyThreads || p.head_pitch < p.vdim || p.ldo < (p.heads - 1) * p.head_pitch + p.vdim)
+      p.maps * p.vdim > kAnyAcc * kAnyThreads || p.head_pitch < p.vdim || p.ldo < (p.heads - 1) * p.head_pitch + p.vdim ||
+      (p.maps == 2 && (p.sink || p.gate)) || (p.gate && p.gate_ld < p.heads))
     return -10;
   if (p.window == 0) p.keep = 0;
   const int group = p.heads / p.kv_heads;

@@ -12,7 +12,9 @@
 // hold [map 1 | map 2]) a tile's rows are (query token, head, map) and a row's query fragment is zero in the other map's half,
 // so the same products serve.  Map 1 - lambda * map 2, its norm over the head's values and a constant factor follow when the
 // row is complete: here without splits, in the merge with them.
-// A sliding window may come with kept first tokens; their pages are walked before the window's.
+// A sliding window may come with kept first tokens; their pages are walked before the window's.  A head may have a sink, a number
+// whose exponential joins the softmax's denominator, and an output gate (the sigmoid of one number per token and head); both are
+// applied where a row is complete.
 //
 // Reference counterparts: split-KV partial + merge drafter attention
 // (native/shared/cuda/draft_attention.cu:42-295) and the LSE state merge
@@ -71,11 +73,22 @@ struct AttnPeers {
   int n, split_offset, total_splits;
 };
 
-// Kept first tokens, output row pitch and, with two maps, how they are combined.
+// Kept first tokens, output row pitch, with two maps how they are combined, with one sinks and gates.
 struct AttnExtras {
   int keep, ldo;
   float lambda, out_scale, eps;
+  const float* sink;             // [Hq] or null
+  const __nv_bfloat16* gate;     // row t, head h: gate[t * gate_ld + h]; or null
+  int gate_ld;
 };
+
+// A complete row of one head: M is the maximum its sums L and O refer to, in log2 units.
+__device__ __forceinline__ float finish_row(float O, float L, float M, const AttnExtras& x, int row, int head) {
+  if (x.sink) L += exp2f(x.sink[head] * 1.4426950408889634f - M);
+  float v = L > 0.f ? O / L : 0.f;
+  if (x.gate) v /= 1.0f + expf(-__bfloat162float(x.gate[static_cast<size_t>(row) * x.gate_ld + head]));
+  return v;
+}
 
 // The combined value of one head's 128 values, one per thread: a - lambda * b over its root mean square, times out_scale.
 __device__ __forceinline__ float combine_maps(float a, float b, const AttnExtras& x, float* red) {
@@ -297,12 +310,16 @@ __global__ void __launch_bounds__(128) attn_decode_kernel(
     } else if (splits == 1) {
       const int qi = first_q + r / group;
       if (qi < q_len) {
-        float v = L > 0.f ? O / L : 0.f;
+        const int head = kvh * (group / kMaps) + (r % group) / kMaps;
+        float v;
         if (kMaps == 2) {
+          v = L > 0.f ? O / L : 0.f;
           if ((r & 1) == 0) { o_map1 = v; continue; }
           v = combine_maps(o_map1, v, ex, sm_l + 64);
+        } else {
+          v = finish_row(O, L, M, ex, q0 + qi, head);
         }
-        out[static_cast<size_t>(q0 + qi) * ex.ldo + (kvh * (group / kMaps) + (r % group) / kMaps) * kD + d] = __float2bfloat16(v);
+        out[static_cast<size_t>(q0 + qi) * ex.ldo + head * kD + d] = __float2bfloat16(v);
       }
     } else {
       part[r * kD + d] = O;
@@ -341,7 +358,7 @@ __global__ void __launch_bounds__(128) attn_merge_kernel(const float* __restrict
       L += __ldg(base + s * kPartialFloats + 16 * kD + 16 + row) * f;
       O += __ldg(base + s * kPartialFloats + row * kD + d) * f;
     }
-    v[m] = L > 0.f ? O / L : 0.f;
+    v[m] = kMaps == 1 ? finish_row(O, L, M, ex, q0 + qi, kvh * group + r % group) : L > 0.f ? O / L : 0.f;
   }
   const float o = kMaps == 2 ? combine_maps(v[0], v[kMaps - 1], ex, red) : v[0];
   out[static_cast<size_t>(q0 + qi) * ex.ldo + (kvh * group + r % group) * kD + d] = __float2bfloat16(o);
@@ -367,13 +384,15 @@ extern "C" long long cafd_attn_decode_scratch_floats(int num_seqs, int tiles_per
 // q [total_q, Hq, 128] (two maps: [total_q, Hq, 2, 64]); caches [pages, Hkv, 64, 128]; page_table [num_seqs, max_pages];
 // seq_lens [num_seqs] (kv length including the new tokens); q_start [num_seqs + 1]; out rows of ldo elements, head h's values at
 // column 128 h.  max_q_len bounds the query tokens of any sequence; scratch holds the split partials.  keep: kept first tokens
-// beside a window; lambda, out_scale and eps: two maps only.
+// beside a window; lambda, out_scale and eps: two maps only; sink [Hq] and gate rows (gate_ld elements apart): one map only.
 extern "C" int cafd_attn_decode(const void* q, const void* k_cache, const void* v_cache, const int* page_table,
                                 const int* seq_lens, const int* q_start, void* out, float* scratch, int num_seqs,
                                 int max_q_len, int max_pages, int Hq, int Hkv, int D, int splits, float scale,
-                                int window, int keep, int ldo, int maps, float lambda, float out_scale, float eps, cafd_stream_t s) {
+                                int window, int keep, int ldo, int maps, float lambda, float out_scale, float eps, const float* sink,
+                                const void* gate, int gate_ld, cafd_stream_t s) {
   if (num_seqs <= 0) return 0;
   if (D != kD || Hq % Hkv || window < 0 || keep < 0 || maps < 1 || maps > 2 || ldo < Hq * kD) return -10;
+  if ((maps == 2 && (sink || gate)) || (gate && gate_ld < Hq)) return -10;
   const int group = maps * (Hq / Hkv);
   if (group > 16 || 16 % group) return -11;
   if (splits < 1) splits = 1;
@@ -391,7 +410,7 @@ extern "C" int cafd_attn_decode(const void* q, const void* k_cache, const void* 
     attr = true;
   }
   dim3 grid(num_seqs * tiles_per_seq, Hkv, splits);
-  const AttnExtras ex{window > 0 ? keep : 0, ldo, lambda, out_scale, eps};
+  const AttnExtras ex{window > 0 ? keep : 0, ldo, lambda, out_scale, eps, sink, static_cast<const __nv_bfloat16*>(gate), gate_ld};
   auto kern = maps == 2 ? attn_decode_kernel<2> : attn_decode_kernel<1>;
   launch_pdl(kern, grid, dim3(128), smem, st,
       static_cast<const __nv_bfloat16*>(q), static_cast<const __nv_bfloat16*>(k_cache),

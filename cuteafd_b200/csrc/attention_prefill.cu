@@ -27,7 +27,8 @@
 // mean square over the head's values, times a constant.
 //
 // A sliding window may come with kept first tokens, which every later row sees too: the tiles that hold them are walked
-// before the window's.
+// before the window's.  A head may have a sink (a number whose exponential joins the softmax's denominator) and an output gate
+// (the sigmoid of one number per token and head): both enter the epilogue's quotient.
 //
 // Replaces the reference's mma.sync prefill kernels (native/families/glm5/cuda/glm_mla_prefill.cu:78-135)
 // and its exported attention programs for the GQA families.
@@ -61,6 +62,10 @@ struct PrefillDev {
   int ldo;                 // elements from row to row of out
   // kMaps == 2 only
   float lambda, out_scale, eps;
+  // kMaps == 1 only
+  const float* sink;              // [Hq] or null
+  const __nv_bfloat16* gate;      // row t, head h: gate[t * gate_ld + h]; or null
+  int gate_ld;
   // kRope only
   const int* kv_tmp_start; // [seqs] first row of the sequence in the expansion buffers (multiple of 64)
   int q_head_stride;       // elements between heads in the nope query matrix (192 for [T, heads * 192])
@@ -429,8 +434,10 @@ attn_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_const
       if (mbar_wait(&mx_bar[fb], (n_tiles >> 1) & 1, p.status, kTimeoutSoftmax)) l_run += xl[(half ^ 1) * 128 + row];
       else l_run = 0.f;
       tc_fence_after();
-      const float inv = l_run > 0.f ? 1.0f / l_run : 0.f;
       const bool row_ok = (row0 + row) < q_len;
+      if (p.sink) l_run += exp2f(p.sink[head] * 1.4426950408889634f - (m_run == -INFINITY ? 0.f : m_run));   // both halves hold the same maximum
+      float inv = l_run > 0.f ? 1.0f / l_run : 0.f;
+      if (p.gate && row_ok) inv /= 1.0f + expf(-__bfloat162float(p.gate[static_cast<size_t>(q0 + row0 + row) * p.gate_ld + head]));
       __nv_bfloat16* orow = p.out + static_cast<size_t>(q0 + row0 + row) * p.ldo + head * kHD + half * 64;
 #pragma unroll 1
       for (int c = 0; c < 2; ++c) {
@@ -466,13 +473,15 @@ using namespace cafd;
 // q [total_q, Hq, 128] bf16 (two maps: [total_q, Hq, 2, 64]); out rows of ldo elements, head h's 128 values at column 128 h;
 // caches [num_pages, Hkv, 64, 128] bf16 (page 0 all zero); page_table [num_seqs, max_pages]; seq_lens [num_seqs];
 // q_start [num_seqs + 1]; max_q_len = longest chunk (grid sizing).  maps 1: lambda, out_scale and eps are unused.
+// sink [Hq] and gate rows (gate_ld elements apart): one map only, null = none.
 extern "C" int cafd_attn_prefill(const void* q, const void* k_cache, const void* v_cache, const int* page_table,
                                  const int* seq_lens, const int* q_start, void* out, uint32_t* status, int total_q,
                                  int num_seqs, int max_q_len, int num_pages, int max_pages, int Hq, int Hkv, int D,
                                  float scale, int window, int keep, int ldo, int maps, float lambda, float out_scale, float eps,
-                                 cafd_stream_t s) {
+                                 const float* sink, const void* gate, int gate_ld, cafd_stream_t s) {
   if (num_seqs <= 0 || total_q <= 0) return 0;
   if (D != kHD || Hq % Hkv || window < 0 || keep < 0 || maps < 1 || maps > 2 || ldo < Hq * kHD || ldo % 8) return -10;
+  if ((maps == 2 && (sink || gate)) || (gate && gate_ld < Hq)) return -10;
   CUtensorMap tq, tk, tv;
   int rc = cached_tmap_2d(&tq, q, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, total_q, static_cast<uint64_t>(Hq) * kHD,
                           static_cast<uint64_t>(Hq) * kHD * 2, kBQ, 64);
@@ -502,6 +511,7 @@ extern "C" int cafd_attn_prefill(const void* q, const void* k_cache, const void*
   p.keep = window > 0 ? keep : 0;
   p.ldo = ldo;
   p.lambda = lambda; p.out_scale = out_scale; p.eps = eps;
+  p.sink = sink; p.gate = static_cast<const __nv_bfloat16*>(gate); p.gate_ld = gate_ld;
   p.q_head_stride = kHD;
   static bool attr = false;
   if (!attr) {
@@ -522,14 +532,14 @@ extern "C" int cafd_attn_prefill(const void* q, const void* k_cache, const void*
 // h * qr_head_stride + qr_col0; k_exp / v_exp [tmp_rows, heads * 128] bf16 = per-head K_nope / V of every cached
 // token of the sequences, sequence s starting at row kv_tmp_start[s] (a multiple of 64); latent cache
 // [num_pages, 64, 576] supplies the shared rope keys (columns 512..575) through the page table.
-// out [total_q, heads, 128].
+// out rows of ldo elements, head h's 128 values at column 128 h.
 extern "C" int cafd_attn_prefill_mla(const void* q_nope, int q_pitch, int q_head_stride, const void* q_rope, int qr_head_stride, int qr_col0,
                                      const void* k_exp, const void* v_exp, long long tmp_rows, const int* kv_tmp_start,
                                      const void* latent_cache, const int* page_table, const int* seq_lens, const int* q_start,
                                      void* out, uint32_t* status, int total_q, int num_seqs, int max_q_len, int num_pages,
-                                     int max_pages, int heads, float scale, int window, cafd_stream_t s) {
+                                     int max_pages, int heads, float scale, int window, int ldo, cafd_stream_t s) {
   if (num_seqs <= 0 || total_q <= 0) return 0;
-  if (window < 0 || q_pitch < heads * q_head_stride || (q_pitch % 8)) return -10;
+  if (ldo < heads * kHD || ldo % 8 || window < 0 || q_pitch < heads * q_head_stride || (q_pitch % 8)) return -10;
   if (tmp_rows % kPageTok || (q_head_stride % 8) || (qr_head_stride % 8) || (qr_col0 % 8)) return -10;
   CUtensorMap tq, tqr, tk, tv, tkr;
   int rc = cached_tmap_2d(&tq, q_nope, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, total_q, static_cast<uint64_t>(heads) * q_head_stride,
@@ -558,7 +568,7 @@ extern "C" int cafd_attn_prefill_mla(const void* q_nope, int q_pitch, int q_head
   p.max_pages = max_pages; p.Hq = heads; p.Hkv = heads;
   p.scale_log2 = scale * 1.4426950408889634f;
   p.window = window;
-  p.ldo = heads * kHD;
+  p.ldo = ldo;
   p.kv_tmp_start = kv_tmp_start; p.q_head_stride = q_head_stride; p.qr_head_stride = qr_head_stride; p.qr_col0 = qr_col0;
   static bool attr = false;
   if (!attr) {

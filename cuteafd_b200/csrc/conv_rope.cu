@@ -1,11 +1,14 @@
 // From a step's fused projection rows to queries and cached keys and values, in one launch: a causal convolution over time
-// on every channel of q, k and v, rotary positions on the leading dimensions of q and k (pairs 2i, 2i + 1), the paged K / V
+// on every channel of q, k and v, an RMS norm of q and k, rotary positions on the leading dimensions of q and k, the paged K / V
 // write and the convolution state of every sequence.
 //
-//   rope_table       cos / sin of position * frequency for every token of the step, once per step and kind of rotation:
-//                    every layer that rotates alike reads it
-//   conv_rope_kv     four channels per thread walking a run of tokens, the convolution's earlier inputs in registers
-//   conv_rope_kv_any any head sizes and any number of taps: one channel per thread and token
+//   rope_table       cos / sin of position * frequency (times a constant) for every token of the step, once per step and kind of
+//                    rotation: every layer that rotates alike reads it
+//   conv_rope_kv     pairs (2i, 2i + 1), no norm: four channels per thread walking a run of tokens, the convolution's earlier
+//                    inputs in registers
+//   conv_rope_kv_any the same for any head sizes and any number of taps: one channel per thread and token
+//   conv_norm_rope_kv  with norms (per head or over the whole projection), pairs of either kind, values of their own or the
+//                    convolved keys: a block walks a run of tokens, the projected rows in a ring in shared memory
 //
 // A sequence's last taps - 1 projected rows are fp32 in its state slot (oldest first, [taps - 1, channels]); a step reads one
 // slot and writes another.  An output is a function of its own taps inputs in a fixed order, so it does not depend on where a
@@ -28,12 +31,19 @@ struct ConvRope {
   void* q_out;                // [T, q channels] E
   void* k_cache;              // [pages, kv heads, 64, maps * dim] E
   void* v_cache;              // [pages, kv heads, 64, vdim] E
+  const float* q_norm;        // [dim] (norm 1) or [nq] (norm 2)
+  const float* k_norm;        // [dim] or [nk]
   long long slot_stride, state_off;
   int T, S, ld, q_off, k_off, v_off, nq, nk, nv, maps_dim, dim, vdim, kv_heads, rot, taps, run;
+  int norm;                   // 0 none, 1 per head (and map), 2 over all of q and all of k
+  int halves;                 // rotated pairs are (i, i + rot / 2), else (2i, 2i + 1)
+  int v_from_k;               // nv = 0: the values are the convolved keys before norm and rotation
+  int units;                  // heads of q, k and v one block works on
+  float eps;
 };
 
 __global__ void __launch_bounds__(256) rope_table_kernel(const int* __restrict__ positions, const float* __restrict__ freq, float2* __restrict__ out,
-                                                         int T, int half) {
+                                                         int T, int half, float mag) {
   pdl_wait();
   pdl_trigger();
   const int n = T * half;
@@ -41,7 +51,7 @@ __global__ void __launch_bounds__(256) rope_table_kernel(const int* __restrict__
     const int t = i / half;
     float s, c;
     sincosf(static_cast<float>(positions[t]) * freq[i - t * half], &s, &c);
-    out[i] = make_float2(c, s);
+    out[i] = make_float2(c * mag, s * mag);
   }
 }
 
@@ -230,6 +240,209 @@ __global__ void __launch_bounds__(256) conv_rope_kv_any_kernel(const ConvRope p)
   }
 }
 
+__device__ __forceinline__ void cp_async_bytes(void* dst, const void* src, int bytes) {
+  const uint32_t d = smem_u32(dst);
+  if (bytes == 16) asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(d), "l"(src) : "memory");
+  else if (bytes == 8) asm volatile("cp.async.ca.shared.global [%0], [%1], 8;" ::"r"(d), "l"(src) : "memory");
+  else asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"(d), "l"(src) : "memory");
+}
+
+// Convolution, norm, rotation and the K / V write.  A block owns `units` consecutive heads of [q | k | v] and walks a run of
+// tokens.  Per token: the thread that owns V channels convolves them (inputs from the ring, or from the state where they lie
+// before the step) into shared memory, the heads' square sums are taken (by the lanes of a head where a head is a power of two
+// of at most 32 vectors, else by a warp per head), then the channels are normed and rotated with their partners.
+constexpr int kCnrThreads = 256, kCnrAhead = 2;
+
+template <typename E, int V>
+__global__ void __launch_bounds__(kCnrThreads) conv_norm_rope_kv_kernel(const ConvRope p) {
+  extern __shared__ float4 sm4[];
+  __shared__ float part[2][kCnrThreads / 32];
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  const int uq = p.nq / p.dim, uk = p.nk / p.dim, uv = p.nv / p.vdim, kmaps = p.maps_dim / p.dim;
+  const int u0 = blockIdx.y * p.units, u1 = min(uq + uk + uv, u0 + p.units);
+  auto chan = [&](int u) { return u <= uq + uk ? u * p.dim : p.nq + p.nk + (u - uq - uk) * p.vdim; };
+  const int c0 = chan(u0), c1 = chan(u1), n = c1 - c0, nvec = n / V, C = p.nq + p.nk + p.nv;
+  const int halo = p.conv_w ? p.taps - 1 : 0, ring = halo + 1 + kCnrAhead;
+  const int nqk = min(c1, p.nq + p.nk) - c0;    // channels of q and k among this block's (they come first); may be <= 0
+  const int max_n = p.units * (p.dim > p.vdim ? p.dim : p.vdim);
+  float* const y = reinterpret_cast<float*>(sm4);                        // [max_n] convolved channels of q and k
+  float* const ss = y + ((max_n + 3) & ~3);                              // [units] square sums of the heads
+  E* const rows = reinterpret_cast<E*>(ss + ((p.units + 3) & ~3));       // [ring][row_pitch]
+  const int row_pitch = (max_n + 15) & ~15;
+  const int vpu = p.dim / V;                                             // vectors of a head of q or k
+  const bool lanes = p.norm && vpu <= 32 && (vpu & (vpu - 1)) == 0;
+  const int half = p.rot >> 1;
+  pdl_wait();
+  pdl_trigger();
+  const int r0 = blockIdx.x * p.run, r1 = min(p.T, r0 + p.run);
+  auto fetch = [&](int row) {
+    if (row < r1) {
+      const E* src = static_cast<const E*>(p.proj) + static_cast<size_t>(row) * p.ld;
+      E* dst = rows + (row % ring) * row_pitch;
+      for (int i = tid; i < nvec; i += kCnrThreads) {
+        const E* a = src + conv_rope_col(p, c0 + i * V);
+        if constexpr (V * sizeof(E) >= 16) {
+#pragma unroll
+          for (int b = 0; b < V; b += 16 / static_cast<int>(sizeof(E))) cp_async_bytes(dst + i * V + b, a + b, 16);
+        } else if constexpr (V * sizeof(E) >= 4) {
+          cp_async_bytes(dst + i * V, a, V * sizeof(E));
+        } else {
+          dst[i] = *a;
+        }
+      }
+    }
+    asm volatile("cp.async.commit_group;" ::: "memory");
+  };
+  for (int row = max(0, r0 - halo); row < r0; ++row) fetch(row);
+#pragma unroll
+  for (int a = 0; a < kCnrAhead; ++a) fetch(r0 + a);
+  int seq = 0, s_lo = 0, s_hi = p.T, s_in = 0;
+  if (halo > 0) {
+    seq = seq_of(p.q_start, p.S, p.T, r0);
+    s_lo = p.q_start[seq];
+    s_hi = p.q_start[seq + 1];
+    s_in = p.state_in[seq];
+  }
+  for (int t = r0; t < r1; ++t) {
+    fetch(t + kCnrAhead);
+    asm volatile("cp.async.wait_group %0;" ::"n"(kCnrAhead) : "memory");
+    __syncthreads();                            // row t is here; the last token's y and ss are done with
+    while (halo > 0 && t == s_hi && seq + 1 < p.S) {                     // next sequence (empty ones are skipped)
+      ++seq;
+      s_lo = s_hi;
+      s_hi = p.q_start[seq + 1];
+      s_in = p.state_in[seq];
+    }
+    const float* st = halo > 0 ? p.state + static_cast<size_t>(s_in) * p.slot_stride + p.state_off : nullptr;
+    const int slot = p.slots[t];
+    for (int i = tid; i < (nvec + 31) / 32 * 32; i += kCnrThreads) {     // whole warps: the lanes of a head sum up together
+      const int c = c0 + i * V;
+      float v[V];
+#pragma unroll
+      for (int e = 0; e < V; ++e) v[e] = 0.f;
+      if (i < nvec) {
+        load_vec<E, V>(rows + (t % ring) * row_pitch + i * V, v);
+        if (p.conv_w) {
+          float w[V], x[V];
+          load_vec<float, V>(p.conv_w + static_cast<size_t>(halo) * C + c, w);
+#pragma unroll
+          for (int e = 0; e < V; ++e) v[e] *= w[e];
+          for (int j = 0; j < halo; ++j) {
+            const int row = t - halo + j;
+            load_vec<float, V>(p.conv_w + static_cast<size_t>(j) * C + c, w);
+            if (row >= s_lo) load_vec<E, V>(rows + (row % ring) * row_pitch + i * V, x);
+            else load_vec<float, V>(st + static_cast<size_t>(halo + row - s_lo) * C + c, x);
+#pragma unroll
+            for (int e = 0; e < V; ++e) v[e] = fmaf(w[e], x[e], v[e]);
+          }
+        }
+        if (i * V < nqk) {
+          store_vec<float, V>(y + i * V, v);
+          if (p.v_from_k && c >= p.nq && slot >= 0) {
+            const int cc = c - p.nq, g = cc / p.vdim;
+            store_vec<E, V>(static_cast<E*>(p.v_cache) + ((static_cast<size_t>(slot >> 6) * p.kv_heads + g) * 64 + (slot & 63)) * p.vdim + (cc - g * p.vdim), v);
+          }
+        } else if (E* dst = conv_rope_dest<E>(p, t, slot, c)) {
+          store_vec<E, V>(dst, v);
+        }
+        if (halo > 0 && t == s_hi - 1) {        // the sequence's last halo inputs, oldest first
+          float* so = p.state + static_cast<size_t>(p.state_out[seq]) * p.slot_stride + p.state_off + c;
+          for (int j = 0; j < halo; ++j) {
+            const int row = t - halo + 1 + j;
+            float x[V];
+            if (row >= s_lo) load_vec<E, V>(rows + (row % ring) * row_pitch + i * V, x);
+            else load_vec<float, V>(st + static_cast<size_t>(halo + row - s_lo) * C + c, x);
+            store_vec<float, V>(so + static_cast<size_t>(j) * C, x);
+          }
+        }
+      }
+      if (lanes) {
+        float s = 0.f;
+#pragma unroll
+        for (int e = 0; e < V; ++e) s += v[e] * v[e];
+        for (int o = 1; o < vpu; o <<= 1) s += __shfl_xor_sync(0xffffffffu, s, o);
+        if (i * V < nqk && i % vpu == 0) ss[i / vpu] = s;
+      }
+    }
+    __syncthreads();
+    if (nqk <= 0) continue;
+    const int nu = nqk / p.dim, nuq = max(0, min(u1, uq) - u0);          // heads of q and k here, of q among them
+    if (p.norm && !lanes) {
+      for (int u = warp; u < nu; u += kCnrThreads / 32) {
+        float s = 0.f;
+        for (int d = lane; d < p.dim; d += 32) s = fmaf(y[u * p.dim + d], y[u * p.dim + d], s);
+        s = warp_sum(s);
+        if (lane == 0) ss[u] = s;
+      }
+      __syncthreads();
+    }
+    float inv_q = 1.f, inv_k = 1.f;
+    if (p.norm == 2) {                          // (a block then owns all heads)
+      float a = 0.f, b = 0.f;
+      for (int u = tid; u < nu; u += kCnrThreads) (u < nuq ? a : b) += ss[u];
+      a = warp_sum(a);
+      b = warp_sum(b);
+      if (lane == 0) { part[0][warp] = a; part[1][warp] = b; }
+      __syncthreads();
+      a = b = 0.f;
+#pragma unroll
+      for (int w = 0; w < kCnrThreads / 32; ++w) { a += part[0][w]; b += part[1][w]; }
+      inv_q = 1.0f / sqrtf(a / static_cast<float>(p.nq) + p.eps);
+      inv_k = 1.0f / sqrtf(b / static_cast<float>(p.nk) + p.eps);
+    }
+    const float2* cs = p.table + static_cast<size_t>(t) * half;
+    for (int i = tid; i * V < nqk; i += kCnrThreads) {
+      const int c = c0 + i * V, u = i * V / p.dim, d = i * V - u * p.dim;
+      const bool is_q = c < p.nq;
+      const float* wn = !p.norm ? nullptr : p.norm == 1 ? (is_q ? p.q_norm : p.k_norm) + d : is_q ? p.q_norm + c : p.k_norm + c - p.nq;
+      const float inv = p.norm == 1 ? 1.0f / sqrtf(ss[u] / static_cast<float>(p.dim) + p.eps) : is_q ? inv_q : inv_k;
+      auto normed = [&](int at, float (&v)[V]) {                         // the normed channels `at` places from this thread's
+        load_vec<float, V>(y + i * V + at, v);
+        if (wn) {
+          float w[V];
+          load_vec<float, V>(wn + at, w);
+#pragma unroll
+          for (int e = 0; e < V; ++e) v[e] = v[e] * inv * w[e];
+        }
+      };
+      float v[V];
+      normed(0, v);
+      if (d < p.rot) {
+        if (p.halves) {                         // (V divides rot / 2)
+          const bool first = d < half;
+          float o[V];
+          normed(first ? half : -half, o);
+          const float2* a = cs + (first ? d : d - half);
+#pragma unroll
+          for (int e = 0; e < V; ++e) v[e] = first ? v[e] * a[e].x - o[e] * a[e].y : v[e] * a[e].x + o[e] * a[e].y;
+        } else if constexpr (V == 1) {
+          float o[1];
+          normed(d & 1 ? -1 : 1, o);
+          const float2 a = cs[d >> 1];
+          v[0] = d & 1 ? v[0] * a.x + o[0] * a.y : v[0] * a.x - o[0] * a.y;
+        } else {                                // (V divides rot)
+#pragma unroll
+          for (int e = 0; e < V; e += 2) {
+            const float2 a = cs[(d + e) >> 1];
+            const float x0 = v[e], x1 = v[e + 1];
+            v[e] = x0 * a.x - x1 * a.y;
+            v[e + 1] = x1 * a.x + x0 * a.y;
+          }
+        }
+      }
+      E* dst;
+      if (is_q) {
+        dst = static_cast<E*>(p.q_out) + static_cast<size_t>(t) * p.nq + c;
+      } else {
+        const int uu = u0 + u - uq, g = uu / kmaps;                         // key head (with two maps: of map uu % kmaps)
+        dst = slot < 0 ? nullptr : static_cast<E*>(p.k_cache) + ((static_cast<size_t>(slot >> 6) * p.kv_heads + g) * 64 + (slot & 63)) * p.maps_dim + (uu - g * kmaps) * p.dim + d;
+      }
+      if (dst) store_vec<E, V>(dst, v);
+    }
+  }
+  asm volatile("cp.async.wait_group 0;" ::: "memory");
+}
+
 // logits = cap * tanh(logits / cap), rows of n values `ld` apart
 __global__ void __launch_bounds__(256) softcap_kernel(float* __restrict__ x, int n, long long ld, float cap) {
   pdl_wait();
@@ -271,25 +484,71 @@ static int launch_conv_rope(ConvRope p, cudaStream_t st) {
   return static_cast<int>(cudaGetLastError());
 }
 
+template <typename E, int V>
+static int launch_conv_norm_rope(ConvRope p, cudaStream_t st) {
+  const int units = p.nq / p.dim + p.nk / p.dim + p.nv / p.vdim, wide = p.dim > p.vdim ? p.dim : p.vdim;
+  const int ring = (p.conv_w ? p.taps : 1) + kCnrAhead;
+  auto bytes = [&](int u) {
+    return static_cast<size_t>((u * wide + 3) / 4 * 4 + (u + 3) / 4 * 4) * 4 + static_cast<size_t>(ring) * ((u * wide + 15) / 16 * 16) * sizeof(E);
+  };
+  // a norm over the whole projection needs all heads in one block; else few tokens are spread over more blocks by heads
+  p.units = units;
+  if (p.norm != 2) {
+    const int want = (2 * 148 + p.T - 1) / p.T, room = 64 * 1024;
+    int per = (units + want - 1) / want;
+    const int least = (512 + wide - 1) / wide;                           // at least 512 channels a block
+    if (per < least) per = least;
+    if (per > units) per = units;
+    while (per > 1 && bytes(per) > static_cast<size_t>(room)) --per;
+    p.units = per;
+  }
+  const size_t smem = bytes(p.units);
+  if (smem > 200 * 1024) return -12;
+  static bool attr = false;
+  if (!attr) {
+    CAFD_CHECK_CUDA(cudaFuncSetAttribute(conv_norm_rope_kv_kernel<E, V>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
+    attr = true;
+  }
+  const int cols = (units + p.units - 1) / p.units;
+  const int resident = smem > 100 * 1024 ? 1 : smem > 50 * 1024 ? 3 : smem > 32 * 1024 ? 4 : 6;
+  int run = (p.T * cols + 148 * resident - 1) / (148 * resident);        // one wave of blocks
+  p.run = p.T <= 64 ? 1 : run < 1 ? 1 : run > 64 ? 64 : run;
+  const dim3 grid((p.T + p.run - 1) / p.run, cols);
+  launch_pdl(conv_norm_rope_kv_kernel<E, V>, grid, dim3(kCnrThreads), smem, st, p);
+  return static_cast<int>(cudaGetLastError());
+}
+
+template <typename E>
+static int dispatch_conv_norm_rope(const ConvRope& p, cudaStream_t st) {
+  auto fits = [&](int v) {
+    const int pair = p.halves ? p.rot / 2 : p.rot;
+    return p.dim % v == 0 && p.vdim % v == 0 && p.ld % v == 0 && p.q_off % v == 0 && p.k_off % v == 0 && p.v_off % v == 0 && pair % v == 0 &&
+           p.state_off % 4 == 0 && p.slot_stride % 4 == 0;
+  };
+  return fits(8) ? launch_conv_norm_rope<E, 8>(p, st) : fits(4) ? launch_conv_norm_rope<E, 4>(p, st) : launch_conv_norm_rope<E, 1>(p, st);
+}
+
 }  // namespace cafd
 
 using namespace cafd;
 
-extern "C" int cafd_rope_table(const int* positions, const float* freq, void* out, int T, int half, cafd_stream_t s) {
+extern "C" int cafd_rope_table(const int* positions, const float* freq, void* out, int T, int half, float mag, cafd_stream_t s) {
   if (T <= 0 || half <= 0) return 0;
   const int blocks = (T * half + 255) / 256;
   launch_pdl(rope_table_kernel, dim3(blocks < 1184 ? blocks : 1184), dim3(256), 0, static_cast<cudaStream_t>(s), positions, freq,
-             static_cast<float2*>(out), T, half);
+             static_cast<float2*>(out), T, half, mag);
   return static_cast<int>(cudaGetLastError());
 }
 
 extern "C" int cafd_conv_rope_kv(const ConvRope* p, int is_f32, cafd_stream_t s) {
   if (p->T <= 0) return 0;
-  if (p->dim <= 0 || p->rot < 0 || p->rot % 2 || p->rot > p->dim || p->maps_dim % p->dim || p->nk != p->kv_heads * p->maps_dim ||
-      p->nv != p->kv_heads * p->vdim || p->nq % p->dim)
+  if (p->dim <= 0 || p->vdim <= 0 || p->rot < 0 || p->rot % 2 || p->rot > p->dim || p->maps_dim % p->dim || p->nk != p->kv_heads * p->maps_dim ||
+      p->nv != (p->v_from_k ? 0 : p->kv_heads * p->vdim) || p->nq % p->dim || p->norm < 0 || p->norm > 2)
     return -10;
+  if ((p->norm && (!p->q_norm || !p->k_norm)) || (p->v_from_k && (p->vdim != p->dim || p->maps_dim != p->dim))) return -10;
   if (p->conv_w && (p->taps < 1 || !p->q_start || p->S < 1 || (p->taps > 1 && (!p->state || !p->state_in || !p->state_out)))) return -10;
   cudaStream_t st = static_cast<cudaStream_t>(s);
+  if (p->norm || p->halves || p->v_from_k) return is_f32 ? dispatch_conv_norm_rope<float>(*p, st) : dispatch_conv_norm_rope<__nv_bfloat16>(*p, st);
   return is_f32 ? launch_conv_rope<float>(*p, st) : launch_conv_rope<__nv_bfloat16>(*p, st);
 }
 

@@ -1,11 +1,13 @@
 // Residual stream of the per-layer hybrid decoders: everything between two sublayers in one launch.
 //
-//   x   = embed[token]                      (first launch)       or the fp32 residual of the previous launch, or their sum
+//   x   = embed[token] * e_scale            (first launch)       or the fp32 residual of the previous launch, or their sum
 //                                           (a loop's next pass)
+//   x  += step                              one vector for all tokens (optional)
 //   x  += groupnorm(y) * w_b                y = a mixer's output rows, or the routed experts' rows summed here:
 //                                           sum over slots of weight * (expert row, or the input row for an identity slot);
-//                                           without w_b: x += y
+//                                           without w_b: x += y; `base` rows are added to the routed sum as they are
 //   h   = groupnorm(x) * (w + w_off)        RMS norm in equal runs of channels, each with its own root mean square
+//                                           (without w: h = x); a second weight vector gives a second output of the same norm
 //   out = h + sum_j c[j] * h(t - taps + 1 + j)     causal convolution over time per channel (optional)
 //
 // A block walks a run of consecutive tokens with every channel in registers, so the convolution's earlier inputs are the
@@ -29,7 +31,11 @@ struct NormArgs {
   const int* slot_idx;        // [T, top_k]; an index >= n_experts is an identity slot
   const void* ident;          // [T, ldh] E: what identity slots hand through
   const void* w_b;            // [H] E, null = y is added as it is
-  const void* w;              // [H] E
+  const void* w;              // [H] E, null = the rows leave as they are, without a norm
+  const void* base;           // [T, ldb] E, null = none; only with slot_w
+  const void* step;           // [H] E, null = none
+  const void* w2;             // [H] E, null = none: weights of the second output; only without a convolution
+  void* h2_out;               // [rows, ldh] E
   const void* conv;           // [taps, H] E, null = no convolution
   float* x_out;               // [T, H] or null
   void* h_out;                // [rows, ldh] E
@@ -39,8 +45,8 @@ struct NormArgs {
   const int* state_out;       // [S] slot written
   const int* q_start;         // [S + 1]
   long long slot_stride, state_off;
-  int T, H, S, ldy, ldh, groups, taps, top_k, n_experts, vocab, run;   // ldy, ldh: elements from row to row of y, of h_out and ident
-  float eps, w_off;
+  int T, H, S, ldy, ldh, ldb, groups, taps, top_k, n_experts, vocab, run;   // ldy, ldh, ldb: elements from row to row of y, of h_out and ident, of base
+  float eps, w_off, e_scale;
 };
 
 template <typename E> __device__ __forceinline__ float ld_e(const E* p);
@@ -183,7 +189,8 @@ __global__ void __launch_bounds__(kMaxThreads, kMinBlocks) norm_conv_kernel(cons
     const bool own_seq = a.conv && a.S == a.T && a.state;
     const float* st = own_seq ? a.state + static_cast<size_t>(a.state_in[blockIdx.x]) * a.slot_stride + a.state_off : nullptr;
     for (int i = tid * 32; i < a.H; i += nt * 32) {         // one 128-byte line per step
-      pull(static_cast<const E*>(a.w) + i);
+      if (a.w) pull(static_cast<const E*>(a.w) + i);
+      if (a.w2) pull(static_cast<const E*>(a.w2) + i);
       if (a.w_b) pull(static_cast<const E*>(a.w_b) + i);
       if (a.conv)
         for (int j = 0; j < a.taps; ++j) pull(static_cast<const E*>(a.conv) + static_cast<size_t>(j) * a.H + i);
@@ -242,6 +249,8 @@ __global__ void __launch_bounds__(kMaxThreads, kMinBlocks) norm_conv_kernel(cons
   if (a.conv && t == s_lo && halo > 0) load_state();
   int flip = 0;
   // The residual and the sublayer's output of the next token are loaded while this one is normalised.
+  const E* const plain = static_cast<const E*>(kSlots ? a.base : a.y);
+  const int ld_plain = kSlots ? a.ldb : a.ldy;
   Packed<float, V> nx[KV];
   Packed<E, V> ny[KV];
   auto fetch = [&](int tt) {
@@ -254,8 +263,8 @@ __global__ void __launch_bounds__(kMaxThreads, kMinBlocks) norm_conv_kernel(cons
         if (i < nvec) nx[k] = load_packed<float, V>(src + i * V);
       }
     }
-    if (!kSlots && a.y) {
-      const E* src = static_cast<const E*>(a.y) + static_cast<size_t>(row) * a.ldy;
+    if (plain) {
+      const E* src = plain + static_cast<size_t>(row) * ld_plain;
 #pragma unroll
       for (int k = 0; k < KV; ++k) {
         const int i = tid + k * nt;
@@ -292,11 +301,23 @@ __global__ void __launch_bounds__(kMaxThreads, kMinBlocks) norm_conv_kernel(cons
           float v[V];
           load_vec<E, V>(src + i * V, v);
 #pragma unroll
+          for (int e = 0; e < V; ++e) x[k][e] = fmaf(v[e], a.e_scale, x[k][e]);
+        }
+      }
+    }
+    if (a.step) {
+#pragma unroll
+      for (int k = 0; k < KV; ++k) {
+        const int i = tid + k * nt;
+        if (i < nvec) {
+          float v[V];
+          load_vec<E, V>(static_cast<const E*>(a.step) + i * V, v);
+#pragma unroll
           for (int e = 0; e < V; ++e) x[k][e] += v[e];
         }
       }
     }
-    if (!kSlots && a.y) {
+    if (plain) {
 #pragma unroll
       for (int k = 0; k < KV; ++k)
         if (tid + k * nt < nvec) unpack(ny[k], y[k]);
@@ -374,6 +395,7 @@ __global__ void __launch_bounds__(kMaxThreads, kMinBlocks) norm_conv_kernel(cons
         if (i < nvec) store_vec<float, V>(a.x_out + static_cast<size_t>(row) * a.H + i * V, x[k]);
       }
     }
+    if (a.w) {
     float inv[KV];
     group_inv<V, KV, sizeof(E) == 4>(x, inv, sm + flip * stride, sm + flip * stride + nvec, nvec, gvec, grp, inv_n, fast, a.eps);
     flip ^= 1;
@@ -382,10 +404,18 @@ __global__ void __launch_bounds__(kMaxThreads, kMinBlocks) norm_conv_kernel(cons
       const int i = tid + k * nt;
       if (i < nvec) {
         float wn[V];
+        if (a.w2 && own) {
+          float o[V];
+          load_vec<E, V>(static_cast<const E*>(a.w2) + i * V, wn);
+#pragma unroll
+          for (int e = 0; e < V; ++e) o[e] = x[k][e] * inv[k] * (wn[e] + a.w_off);
+          store_vec<E, V>(static_cast<E*>(a.h2_out) + static_cast<size_t>(t) * a.ldh + i * V, o);
+        }
         load_vec<E, V>(static_cast<const E*>(a.w) + i * V, wn);
 #pragma unroll
         for (int e = 0; e < V; ++e) x[k][e] = x[k][e] * inv[k] * (wn[e] + a.w_off);
       }
+    }
     }
     if (own) {
 #pragma unroll

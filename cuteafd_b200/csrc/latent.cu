@@ -2,7 +2,7 @@
 // mla_attention.cu serves the 512 + 64 record; this file serves every other record and the fp32 engines).
 //
 //   latent_prep   one block per token: RMS norm of the latent, rotation of the shared key part and of every head's
-//                 rotated query part, the cache record, and the unrotated query parts moved head-major for the absorb
+//                 rotated query part (pairs of halves or of neighbours; cosines and sines times a constant), the cache record, and the unrotated query parts moved head-major for the absorb
 //                 product q W_uk
 //   latent_attn   absorbed attention: scores q_abs . record over the window, softmax in fp32, the weighted sum of latents
 //   latent_gate   attn *= sigmoid(gate row)
@@ -30,8 +30,8 @@ struct LatentPrep {
   void* slab;                 // [heads, t_pad, dim_pad] E
   void* q_abs;                // [T, heads, rec] E: the rotated part goes to [rank, rank + rot)
   void* lat_out;              // [T, rank] E or null: a contiguous copy of the normed latents
-  int lda, q_off, kv_off, heads, dim, rot, rank, rec, dim_pad, t_pad, T;
-  float eps;
+  int lda, q_off, kv_off, heads, dim, rot, rank, rec, dim_pad, t_pad, T, halves;
+  float eps, mag;
 };
 
 template <typename E>
@@ -47,8 +47,8 @@ __global__ void __launch_bounds__(256) latent_prep_kernel(const LatentPrep p) {
   for (int i = tid; i < half; i += blockDim.x) {
     float s, c;
     sincosf(pos * p.inv_freq[i], &s, &c);
-    cs[i] = c;
-    cs[half + i] = s;
+    cs[i] = c * p.mag;
+    cs[half + i] = s * p.mag;
   }
   float ss = 0.f;
   for (int i = tid; i < p.rank; i += blockDim.x) { const float v = to_f<E>(kv[i]); ss += v * v; }
@@ -67,10 +67,11 @@ __global__ void __launch_bounds__(256) latent_prep_kernel(const LatentPrep p) {
     if (p.lat_out) static_cast<E*>(p.lat_out)[static_cast<size_t>(t) * p.rank + i] = v;
   }
   for (int i = tid; i < half; i += blockDim.x) {
-    const float u = to_f<E>(kv[p.rank + i]), v = to_f<E>(kv[p.rank + half + i]);
+    const int e0 = p.rank + (p.halves ? i : 2 * i), e1 = p.halves ? e0 + half : e0 + 1;
+    const float u = to_f<E>(kv[e0]), v = to_f<E>(kv[e1]);
     if (slot >= 0) {
-      rec[p.rank + i] = from_f<E>(u * cs[i] - v * cs[half + i]);
-      rec[p.rank + half + i] = from_f<E>(v * cs[i] + u * cs[half + i]);
+      rec[e0] = from_f<E>(u * cs[i] - v * cs[half + i]);
+      rec[e1] = from_f<E>(v * cs[i] + u * cs[half + i]);
     }
   }
   const E* q = row + p.q_off;
@@ -83,10 +84,11 @@ __global__ void __launch_bounds__(256) latent_prep_kernel(const LatentPrep p) {
   }
   for (int i = tid; i < p.heads * half; i += blockDim.x) {
     const int h = i / half, d = i - h * half;
-    const float u = to_f<E>(q[h * qd + p.dim + d]), v = to_f<E>(q[h * qd + p.dim + half + d]);
+    const int e0 = p.halves ? d : 2 * d, e1 = p.halves ? e0 + half : e0 + 1;
+    const float u = to_f<E>(q[h * qd + p.dim + e0]), v = to_f<E>(q[h * qd + p.dim + e1]);
     E* o = static_cast<E*>(p.q_abs) + (static_cast<size_t>(t) * p.heads + h) * p.rec + p.rank;
-    o[d] = from_f<E>(u * cs[d] - v * cs[half + d]);
-    o[half + d] = from_f<E>(v * cs[d] + u * cs[half + d]);
+    o[e0] = from_f<E>(u * cs[d] - v * cs[half + d]);
+    o[e1] = from_f<E>(v * cs[d] + u * cs[half + d]);
   }
 }
 

@@ -196,7 +196,8 @@ constexpr int kSmallT = 16;
 __global__ void __launch_bounds__(128) mla_absorb_small_kernel(const __nv_bfloat16* __restrict__ q, int ldq,
                                                                const __nv_bfloat16* __restrict__ w_uk,
                                                                const float* __restrict__ inv_freq, const int* __restrict__ positions,
-                                                               __nv_bfloat16* __restrict__ q_abs, int T, int heads, int interleaved) {
+                                                               __nv_bfloat16* __restrict__ q_abs, int T, int heads, int interleaved,
+                                                               float mag) {
   pdl_wait();
   pdl_trigger();
   __shared__ float sq[kSmallT][kNope];
@@ -213,6 +214,8 @@ __global__ void __launch_bounds__(128) mla_absorb_small_kernel(const __nv_bfloat
       __nv_bfloat16* dst = q_abs + (static_cast<size_t>(t) * heads + h) * kRecord + kLatent;
       float sn, cs;
       sincosf(static_cast<float>(positions[t]) * inv_freq[lane], &sn, &cs);
+      sn *= mag;
+      cs *= mag;
       if (interleaved) {
         const uint32_t v = *reinterpret_cast<const uint32_t*>(r + 2 * lane);
         const float x0 = bf16_lo(v), x1 = bf16_hi(v);
@@ -251,12 +254,12 @@ __global__ void __launch_bounds__(128) mla_absorb_small_kernel(const __nv_bfloat
 }
 
 // o_lat [heads, t_pad, 512] (head-major attention output) -> attn [T, heads * 128]: attn[t, h] = o_lat[h, t] @ W_uv[h]^T
-// (W_uv [heads, 128, 512]), times sigmoid(gate[t, h * 128 ..]) where a gate is given.  grid (heads, 2): CTA (h, s) computes output rows [64 s, 64 s + 64); each of its eight
+// (W_uv [heads, 128, 512]; rows of ldo elements), times sigmoid(gate[t, h * 128 ..]) where a gate is given.  grid (heads, 2): CTA (h, s) computes output rows [64 s, 64 s + 64); each of its eight
 // warps takes eight weight rows, lanes along K (a warp load is 512 contiguous bytes), all sixteen loads in flight.
 __global__ void __launch_bounds__(256) mla_unabsorb_small_kernel(const __nv_bfloat16* __restrict__ o_lat, int t_pad,
                                                                  const __nv_bfloat16* __restrict__ w_uv,
                                                                  __nv_bfloat16* __restrict__ attn, int T, int heads,
-                                                                 const __nv_bfloat16* __restrict__ gate, int ldg) {
+                                                                 const __nv_bfloat16* __restrict__ gate, int ldg, int ldo) {
   pdl_wait();
   pdl_trigger();
   __shared__ __align__(16) __nv_bfloat16 sx[kSmallT][kLatent];
@@ -291,7 +294,7 @@ __global__ void __launch_bounds__(256) mla_unabsorb_small_kernel(const __nv_bflo
 #pragma unroll
       for (int r = 1; r < 8; ++r) v = lane == r ? acc[r] : v;
       if (gate) v /= 1.0f + expf(-__bfloat162float(gate[static_cast<size_t>(t) * ldg + h * 128 + row0 + lane]));
-      attn[static_cast<size_t>(t) * heads * 128 + h * 128 + row0 + lane] = __float2bfloat16(v);
+      attn[static_cast<size_t>(t) * ldo + h * 128 + row0 + lane] = __float2bfloat16(v);
     }
   }
 }
@@ -356,22 +359,23 @@ extern "C" int cafd_mla_q_split(const void* q, int ldq, const float* inv_freq, c
 
 extern "C" int cafd_mla_small_rows(void) { return cafd::kSmallT; }
 
-// Decode-sized steps (T <= cafd_mla_small_rows()): q split + RoPE + absorb in one launch, and the un-absorb.
+// Decode-sized steps (T <= cafd_mla_small_rows()): q split + RoPE (cosines and sines times mag) + absorb in one launch, and the
+// un-absorb.
 extern "C" int cafd_mla_absorb_small(const void* q, int ldq, const void* w_uk, const float* inv_freq, const int* positions,
-                                     void* q_abs, int T, int heads, int interleaved, cafd_stream_t s) {
+                                     void* q_abs, int T, int heads, int interleaved, float mag, cafd_stream_t s) {
   if (T <= 0) return 0;
   if (T > cafd::kSmallT || (ldq & 1)) return -10;
   launch_pdl(mla_absorb_small_kernel, dim3(heads, 4), dim3(128), 0, static_cast<cudaStream_t>(s),
              static_cast<const __nv_bfloat16*>(q), ldq, static_cast<const __nv_bfloat16*>(w_uk), inv_freq, positions,
-             static_cast<__nv_bfloat16*>(q_abs), T, heads, interleaved);
+             static_cast<__nv_bfloat16*>(q_abs), T, heads, interleaved, mag);
   return static_cast<int>(cudaGetLastError());
 }
 extern "C" int cafd_mla_unabsorb_small(const void* o_lat, int t_pad, const void* w_uv, void* attn, int T, int heads, const void* gate, int ldg,
-                                       cafd_stream_t s) {
+                                       int ldo, cafd_stream_t s) {
   if (T <= 0) return 0;
-  if (T > cafd::kSmallT) return -10;
+  if (T > cafd::kSmallT || ldo < heads * 128) return -10;
   launch_pdl(mla_unabsorb_small_kernel, dim3(heads, 2), dim3(256), 0, static_cast<cudaStream_t>(s),
              static_cast<const __nv_bfloat16*>(o_lat), t_pad, static_cast<const __nv_bfloat16*>(w_uv),
-             static_cast<__nv_bfloat16*>(attn), T, heads, static_cast<const __nv_bfloat16*>(gate), ldg);
+             static_cast<__nv_bfloat16*>(attn), T, heads, static_cast<const __nv_bfloat16*>(gate), ldg, ldo);
   return static_cast<int>(cudaGetLastError());
 }

@@ -2,7 +2,8 @@
 // token's E router scores into top-k expert ids and gate weights (softmax or sigmoid scoring, selection bias,
 // group-limited routing, ties to the lowest id).  Contract of the reference router
 // (native/shared/cuda/expert_router.cu:12-55,108-158): bias is used for selection only, weights come from the
-// unbiased scores, normalised over the top-k with +1e-20, times the routed scale.
+// unbiased scores, normalised over the top-k with +1e-20, times the routed scale.  Scoring 2 is softmax over logits the bias is
+// part of: it then shapes the weights too.
 #pragma once
 
 #include "common.cuh"
@@ -13,7 +14,7 @@ namespace cafd {
 // One warp routes one token: `row` points at its E router logits in global memory.
 template <int kPerLane>
 __device__ __forceinline__ void route_row(const float* row, const float* __restrict__ bias, int* __restrict__ out_idx,
-                                          float* __restrict__ out_w, int t, int E, int top_k, int sigmoid, int num_groups,
+                                          float* __restrict__ out_w, int t, int E, int top_k, int scoring, int num_groups,
                                           int topk_groups, int normalize, float routed_scale, int group_max = 0) {
   const int lane = threadIdx.x & 31;
   float score[kPerLane], sel[kPerLane];
@@ -22,9 +23,10 @@ __device__ __forceinline__ void route_row(const float* row, const float* __restr
   for (int j = 0; j < kPerLane; ++j) {
     const int e = j * 32 + lane;
     score[j] = e < E ? __ldcg(row + e) : -INFINITY;     // written by other blocks (or an earlier kernel): skip L1
+    if (scoring == 2 && bias && e < E) score[j] += bias[e];
     mx = fmaxf(mx, score[j]);
   }
-  if (sigmoid) {
+  if (scoring == 1) {
 #pragma unroll
     for (int j = 0; j < kPerLane; ++j) {
       const int e = j * 32 + lane;
@@ -49,7 +51,7 @@ __device__ __forceinline__ void route_row(const float* row, const float* __restr
 #pragma unroll
   for (int j = 0; j < kPerLane; ++j) {
     const int e = j * 32 + lane;
-    sel[j] = e < E ? score[j] + (bias ? bias[e] : 0.f) : -INFINITY;
+    sel[j] = e < E ? score[j] + (bias && scoring != 2 ? bias[e] : 0.f) : -INFINITY;
   }
   if (num_groups > 1) {
     const int per_group = E / num_groups;

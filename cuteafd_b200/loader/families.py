@@ -161,7 +161,9 @@ class KarusunModel(FamilyModel):
         if e:
             return "routed_expert", layer, int(e.group(1))
         if rest.startswith("mlp."):
-            return ("router" if rest in ("mlp.router", "mlp.correction") else "dense_ffn"), layer, None
+            role = ("router" if rest in ("mlp.router", "mlp.router.b", "mlp.correction") else
+                    "shared_expert" if rest.startswith("mlp.shared.") else "dense_ffn")
+            return role, layer, None
         return ("norm" if rest.startswith(("norm", "canon")) else "other"), layer, None
 
 
@@ -185,6 +187,25 @@ class Guberax(Karusun):
         return hf_config.get("architecture") == "Guberax"
 
 
+class RofapelModel(KarusunModel):
+    """The loop's joining product and step vectors beside the tensors of the layers."""
+
+    def classify(self, name: str) -> tuple[str, int | None, int | None]:
+        return ("dense_ffn", None, None) if name in ("loop.in", "loop.step") else super().classify(name)
+
+
+class Rofapel(Karusun):
+    """Parallel layers with a norm for each half (latent, windowed or plain attention beside a dense or routed feed-forward), some
+    of them looped: served by the hybrid engine."""
+    id, model_types, attention = "rofapel", ("rofapel",), "hybrid"
+
+    def detect(self, hf_config: dict) -> bool:
+        return hf_config.get("architecture") == "Rofapel"
+
+    def open(self, cfg: ModelConfig, hf_config: dict) -> FamilyModel:
+        return RofapelModel(self, cfg, ExpertContract(formats=("bf16",)))
+
+
 class TinyMoe(Family):
     id, model_types = "tiny_moe", ("tiny_moe",)
 
@@ -204,7 +225,7 @@ def canonical_name(name: str) -> str:
     return _MIXTRAL_RE.sub(lambda m: m.group(1) + _MIXTRAL_PROJ[m.group(2)] + m.group(3), name)
 
 
-REGISTRY: tuple[Family, ...] = (DeepseekV32(), DeepseekV3(), Qwen3Moe(), Glm4Moe(), Qwen2(), Llama(), TinyMoe(), Karusun(), Guberax())
+REGISTRY: tuple[Family, ...] = (DeepseekV32(), DeepseekV3(), Qwen3Moe(), Glm4Moe(), Qwen2(), Llama(), TinyMoe(), Karusun(), Guberax(), Rofapel())
 
 
 def detect(hf_config: dict) -> Family | None:

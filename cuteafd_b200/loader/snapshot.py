@@ -27,13 +27,15 @@ def _layer_list_to_json(cfg: ModelConfig) -> dict:
     """config.json of a per-layer design (the ``layers`` list form)."""
     if cfg.family == "guberax":
         return _parallel_layers_to_json(cfg)
+    if cfg.family == "rofapel":
+        return _two_norm_layers_to_json(cfg)
     layers = []
     for s in cfg.layer_specs:
         m, r = s.mixer, s.router
         if isinstance(m, LatentSpec):
             e = {"type": "latent_attention", "mixer": {
                 "heads": m.heads, "dim": m.dim, "rot_dim": m.rot_dim, "vdim": m.vdim, "kv_rank": m.kv_rank, "scale": m.scale,
-                "mask": {"size": m.window}, "rot": {"base": m.rope_base, "dims": m.rot_dim}}}
+                "mask": {"size": m.window}, "rot": {"base": m.rope.base, "dims": m.rot_dim}}}
         else:
             e = {"type": "delta", "mixer": {"heads": m.heads, "kv_heads": m.kv_heads, "dim": m.dim, "vdim": m.vdim, "conv": m.conv}}
         e["mlp"] = None if r is None else {"kind": "moe", "expert": {"ff": r.ffn}, "router": {
@@ -62,6 +64,120 @@ def _parallel_layers_to_json(cfg: ModelConfig) -> dict:
     return d
 
 
+def _loop_of(d: dict, layers: int) -> tuple:
+    lp = d.get("loop")
+    loop = (lp["start"], lp["stop"], lp["times"]) if lp and lp["stop"] != lp["start"] else ()
+    if loop and not (0 <= loop[0] < loop[1] <= layers and loop[2] >= 1):
+        raise ValueError(f"loop {loop} over {layers} layers")
+    return loop
+
+
+def _silu_only(i: int, *parts: dict) -> None:
+    for e in parts:
+        if (e.get("act") or "silu") != "silu":
+            raise ValueError(f"layer {i}: unsupported feed-forward activation {e['act']!r}")
+
+
+# How the two attention mixers of Rofapel treat queries, keys and values; everything else about them is in the configuration.
+_TWO_NORM_ATTENTION = {"attention": dict(qk_norm="all", gate=True),
+                       "attention_2": dict(qk_norm="head", v_from_k=True, sink=True, gate=True)}
+
+
+def _rope_from_json(i: int, rot: dict, dims: int, halves: bool) -> RopeSpec:
+    """``rot`` of a mixer whose rotated vectors are ``dims`` wide."""
+    sc, n = rot.get("scaling") or {}, rot.get("dims", dims)
+    if n % 2 or n > dims:
+        raise ValueError(f"layer {i}: {n} rotated dims of {dims}")
+    if not sc:
+        return RopeSpec(n, float(rot["base"]), halves=halves)
+    if set(sc) == {"factor"}:
+        return RopeSpec(n, float(rot["base"]), float(sc["factor"]), kind="linear", halves=halves)
+    if set(sc) == {"factor", "original", "fast", "slow"}:
+        return RopeSpec(n, float(rot["base"]), float(sc["factor"]), float(sc["slow"]), float(sc["fast"]), sc["original"], "yarn", halves)
+    raise ValueError(f"layer {i}: unsupported rotary scaling {sorted(sc)}")
+
+
+def _rope_to_json(r: RopeSpec) -> dict:
+    rot = {"base": r.base, "dims": r.dims}
+    if r.kind == "linear":
+        rot["scaling"] = {"factor": r.factor}
+    elif r.kind == "yarn":
+        rot["scaling"] = {"factor": r.factor, "original": r.original, "fast": r.high, "slow": r.low}
+    return rot
+
+
+def _two_norm_layers_to_json(cfg: ModelConfig) -> dict:
+    layers = []
+    for s in cfg.layer_specs:
+        m, r = s.mixer, s.router
+        e = {"heads": m.heads, "dim": m.dim, "vdim": m.vdim, "scale": m.scale, "rot": _rope_to_json(m.rope)}
+        if isinstance(m, LatentSpec):
+            kind = "latent_attention"
+            e.update(rot_dim=m.rot_dim, kv_rank=m.kv_rank)
+        else:
+            kind = "attention_2" if m.v_from_k else "attention"
+            e["kv_heads"] = m.kv_heads
+            if m.conv:
+                e["conv"] = m.conv
+        if m.window:
+            e["mask"] = {"size": m.window}
+        mlp = None
+        if r is not None:
+            mlp = {"kind": "moe", "expert": {"ff": r.ffn}, "router": {"experts": r.experts, "top": r.top}}
+            if s.dense is not None:
+                mlp["shared"] = {"ff": s.dense.ffn}
+        elif s.dense is not None:
+            mlp = {"kind": "dense", "ff": s.dense.ffn}
+        layers.append({"type": kind, "mixer": e, "mlp": mlp})
+    d = {"architecture": "Rofapel", "name": cfg.name, "vocab": cfg.vocab_size, "width": cfg.hidden, "layers": layers,
+         "norm": {"eps": cfg.rms_eps}, "embedding": {"scale": cfg.embed_scale}}
+    if cfg.loop:
+        d["loop"] = dict(zip(("start", "stop", "times"), cfg.loop))
+    return d
+
+
+def _two_norm_layers_from_json(d: dict) -> ModelConfig:
+    """Parallel layers with a norm for each half: latent attention or one of two attention mixers beside a dense or routed
+    feed-forward (``architecture`` Rofapel)."""
+    specs = []
+    for i, e in enumerate(d["layers"]):
+        m, mlp, kind = e["mixer"], e.get("mlp"), e["type"]
+        window = (m.get("mask") or {}).get("size") or 0
+        if kind == "latent_attention":
+            rope = _rope_from_json(i, m["rot"], m["rot_dim"], halves=False)
+            if rope.dims != m["rot_dim"]:
+                raise ValueError(f"layer {i}: {rope.dims} rotated dims of a rotated part of {m['rot_dim']} are not supported")
+            mixer = LatentSpec(heads=m["heads"], dim=m["dim"], rot_dim=m["rot_dim"], vdim=m["vdim"], kv_rank=m["kv_rank"], window=window,
+                               scale=float(m["scale"]), rope=rope, gate=False)
+        elif kind in _TWO_NORM_ATTENTION:
+            mixer = AttentionSpec(heads=m["heads"], kv_heads=m.get("kv_heads") or m["heads"], dim=m["dim"], vdim=m.get("vdim") or m["dim"],
+                                  window=window, keep_first=0, scale=float(m["scale"]), rope=_rope_from_json(i, m["rot"], m["dim"], halves=True),
+                                  conv=m.get("conv") or 0, **_TWO_NORM_ATTENTION[kind])
+            if mixer.heads % mixer.kv_heads:
+                raise ValueError(f"layer {i}: {mixer.heads} heads over {mixer.kv_heads} key heads")
+            if mixer.v_from_k and mixer.vdim != mixer.dim:
+                raise ValueError(f"layer {i}: values of {mixer.vdim} out of keys of {mixer.dim}")
+        else:
+            raise ValueError(f"layer {i}: unsupported mixer {kind!r}")
+        router = dense = None
+        if mlp is not None and mlp.get("kind") == "dense":
+            _silu_only(i, mlp)
+            dense = DenseSpec(mlp["ff"])
+        elif mlp is not None and mlp.get("kind") == "moe":
+            r, shared = mlp["router"], mlp.get("shared")
+            _silu_only(i, mlp["expert"], shared or {})
+            router = RouterSpec(experts=r["experts"], ffn=mlp["expert"]["ff"], top=r["top"], logit_bias=True, normalize=True)
+            if not 1 <= router.top <= router.experts:
+                raise ValueError(f"layer {i}: {router.top} of {router.experts} experts")
+            dense = DenseSpec(shared["ff"]) if shared else None
+        elif mlp is not None:
+            raise ValueError(f"layer {i}: unsupported feed-forward {mlp.get('kind')!r}")
+        specs.append(LayerSpec(mixer, router, dense, parallel=True, two_norms=True))
+    return parallel_config(d.get("name", d["architecture"].lower()), d["vocab"], d["width"], specs, float(d["norm"]["eps"]),
+                           _loop_of(d, len(specs)), family="rofapel", loop_join=True,
+                           embed_scale=float((d.get("embedding") or {}).get("scale", 1.0)))
+
+
 def _parallel_layers_from_json(d: dict) -> ModelConfig:
     """Parallel layers of differential attention and a dense feed-forward (``architecture`` Guberax)."""
     specs = []
@@ -87,10 +203,7 @@ def _parallel_layers_from_json(d: dict) -> ModelConfig:
                 raise ValueError(f"layer {i}: unsupported feed-forward {mlp.get('kind')!r} {mlp.get('act') or ''}")
             dense = DenseSpec(mlp["ff"])
         specs.append(LayerSpec(mixer, dense=dense, parallel=True))
-    lp = d.get("loop")
-    loop = (lp["start"], lp["stop"], lp["times"]) if lp and lp["stop"] != lp["start"] else ()
-    if loop and not (0 <= loop[0] < loop[1] <= len(specs) and loop[2] >= 1):
-        raise ValueError(f"loop {loop} over {len(specs)} layers")
+    loop = _loop_of(d, len(specs))
     return parallel_config(d.get("name", d["architecture"].lower()), d["vocab"], d["width"], specs, float(d["norm"]["eps"]), loop,
                            float(d.get("logit_softcap") or 0.0))
 
@@ -100,6 +213,8 @@ def _layer_list_from_json(d: dict) -> ModelConfig:
     refused by name."""
     if d["architecture"] == "Guberax":
         return _parallel_layers_from_json(d)
+    if d["architecture"] == "Rofapel":
+        return _two_norm_layers_from_json(d)
     specs = []
     for i, e in enumerate(d["layers"]):
         m, mlp = e["mixer"], e.get("mlp")
@@ -108,7 +223,8 @@ def _layer_list_from_json(d: dict) -> ModelConfig:
             if rot.get("dims", m["rot_dim"]) != m["rot_dim"]:
                 raise ValueError(f"layer {i}: {rot['dims']} rotated dims of a rotated part of {m['rot_dim']} are not supported")
             mixer = LatentSpec(heads=m["heads"], dim=m["dim"], rot_dim=m["rot_dim"], vdim=m["vdim"], kv_rank=m["kv_rank"],
-                               window=m["mask"]["size"], scale=float(m["scale"]), rope_base=float(rot["base"]))
+                               window=m["mask"]["size"], scale=float(m["scale"]),
+                               rope=RopeSpec(m["rot_dim"], float(rot["base"]), halves=True))
         elif e["type"] == "delta":
             mixer = DeltaSpec(heads=m["heads"], kv_heads=m.get("kv_heads", m["heads"]), dim=m["dim"], vdim=m["vdim"], conv=m["conv"])
             if mixer.heads % mixer.kv_heads:
@@ -226,7 +342,7 @@ def _rope_scaling(d: dict) -> dict:
 
 def from_hf_config(d: dict) -> ModelConfig:
     """Map a config.json onto the engine's geometry.  Unknown architectures raise ValueError."""
-    if d.get("architecture") in ("Karusun", "Guberax"):
+    if d.get("architecture") in ("Karusun", "Guberax", "Rofapel"):
         return _layer_list_from_json(d)
     mt = d.get("model_type", "")
     extra = d.get("cuteafd", {})

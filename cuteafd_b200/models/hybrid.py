@@ -1,25 +1,29 @@
 """Per-layer hybrid decoders (``ModelConfig.layer_specs``): windowed latent attention and gated delta-rule layers in any
 order, grouped RMS norms before and after every sublayer, a causal convolution on every sublayer's input, routed
-feed-forwards with identity outputs; and stacks of parallel layers (differential attention beside a dense feed-forward under
-one norm), some of them looped.
+feed-forwards with identity outputs; and stacks of parallel layers (plain, differential or latent attention beside a dense or routed
+feed-forward, under one norm or one each), some of them looped.
 
 A layer is a fixed launch sequence over preallocated workspaces:
 
     norm_conv -> fused projection -> mixer kernels -> o projection -> norm_conv -> routes -> plan / dispatch -> fc1 -> fc2
     parallel:  norm_conv -> fused q / k / v -> conv_rope_kv -> attention -> gate / up -> [o | down] as one product
+               (routed: the shared expert's gate / up and down there, routes -> plan / dispatch -> fc1 -> fc2 beside it)
 
 ``norm_conv`` is everything between two sublayers (the routed rows' weighted sum, the norm after the sublayer, the fp32
 residual, the norm before the next one, its convolution).  What a sequence carries besides latent records lives in slots
 of one fp32 pool; a step reads one slot per sequence and writes another (``Batch.state_in`` / ``state_out``), so a step
 can be repeated and a slot can be shared with a cached prefix.  ``compute_dtype`` "f32" runs the same sequence with every
 product and activation in 32-bit.  A looped layer runs several times with the same weights; cache and state belong to the run
-(``ModelConfig.layer_runs``), not to the layer.
+(``ModelConfig.layer_runs``), not to the layer.  Where a pass starts with a product of [x; embedding row], both halves lie in one
+buffer whose second half is written once per step.
 """
 from __future__ import annotations
 
+import math
+
 import torch
 
-from ..config import AttentionSpec, DeltaSpec, LatentSpec, ModelConfig, RopeSpec
+from ..config import AttentionSpec, DeltaSpec, LatentSpec, ModelConfig, RopeSpec, RouterSpec
 from ..ops import kernels as K
 from ..parallel.moe_exchange import ExchangeGeometry, LocalExchange
 from .gqa_moe import PAGE, Batch
@@ -40,13 +44,31 @@ def record_pitch(m: LatentSpec) -> int:
 
 
 def rope_frequencies(r: RopeSpec) -> torch.Tensor:
-    """fp32 [dims / 2] turns per position, worked out in fp64."""
+    """fp32 [dims / 2] radians per position, worked out in fp64."""
     f = r.base ** (-torch.arange(0, r.dims, 2, dtype=torch.float64) / max(1, r.dims))
-    if r.factor != 1.0:
+    if r.factor == 1.0 or not r.dims:
+        return f.float()
+    if r.kind == "linear":
+        f = f / r.factor
+    elif r.kind == "yarn":
+        log_base = math.log(r.base)
+        edge = [r.dims * math.log(r.original / (2 * math.pi * turns)) / (2 * log_base) for turns in (r.high, r.low)]
+        lo, hi = max(math.floor(edge[0]), 0), min(math.ceil(edge[1]), r.dims - 1)
+        ramp = ((torch.arange(r.dims // 2, dtype=torch.float64) - lo) / max(hi - lo, 0.001)).clamp(0.0, 1.0)
+        f = torch.lerp(f, f / r.factor, ramp)
+    else:
         wave = 2 * torch.pi / f
         s = (r.original / wave - r.low) / (r.high - r.low) if r.high != r.low else torch.zeros_like(f)
         f = torch.where(wave < r.original / r.high, f, torch.where(wave > r.original / r.low, f / r.factor, (1 - s) * f / r.factor + s * f))
     return f.float()
+
+
+def out_columns(m, d) -> tuple[int, int]:
+    """Columns of a parallel layer's second product: (the heads' values, the dense activations after them).  Latent heads are
+    written by a product whose rows are heads, so a row is then a whole number of heads long."""
+    vp = pad8(m.vdim)
+    f = pad8(d.ffn) if d is not None else 0
+    return m.heads * vp, -(-f // vp) * vp if isinstance(m, LatentSpec) else f
 
 
 class HybridLayer:
@@ -54,7 +76,7 @@ class HybridLayer:
     (``offs`` names its sections, each padded to a multiple of 8 rows), experts are stacked."""
     __slots__ = ("norm1", "norm1b", "norm2", "norm2b", "canon1", "canon2", "w_in", "offs", "w_o",
                  "kv_norm", "w_uk", "w_uv", "w_kb", "conv_w", "A_log", "dt_bias", "out_norm",
-                 "router", "correction", "w_gate", "w_up", "w_down", "w_out", "lam")
+                 "router", "correction", "w_gate", "w_up", "w_down", "d_gate", "d_up", "w_out", "lam", "q_norm", "k_norm", "sink")
 
     def __init__(self) -> None:
         for s in self.__slots__:
@@ -64,7 +86,7 @@ class HybridLayer:
 class HybridWeights:
     def __init__(self, cfg: ModelConfig):
         self.cfg = cfg
-        self.embed = self.final_norm = self.lm_head = None
+        self.embed = self.final_norm = self.lm_head = self.loop_in = self.loop_step = None
         self.layers: list[HybridLayer] = []
 
     @staticmethod
@@ -83,8 +105,11 @@ class HybridWeights:
             """A matrix that reads the layer input: columns up to whole 16-byte rows."""
             return x if Hp == H else torch.nn.functional.pad(x, (0, Hp - H)).contiguous()
 
-        def f(name: str) -> torch.Tensor:
-            return get(name).to(device=device, dtype=torch.float32).contiguous()
+        def f(name: str, shape: tuple | None = None) -> torch.Tensor:
+            x = get(name).to(device=device, dtype=torch.float32).contiguous()
+            if shape is not None and tuple(x.shape) != shape:
+                raise ValueError(f"{name}: shape {tuple(x.shape)}, the configuration says {shape}")
+            return x
 
         def fuse(parts: list[tuple[str, torch.Tensor]]) -> tuple[torch.Tensor, dict]:
             rows = sum(pad8(x.shape[0]) for _, x in parts)
@@ -105,29 +130,72 @@ class HybridWeights:
 
         W = HybridWeights(cfg)
         def attention(m: AttentionSpec, x: str, L: HybridLayer) -> None:
-            L.w_in, L.offs = fuse([("q", t(x + "q", (m.q_channels, H))), ("k", t(x + "k", (m.k_channels, H))), ("v", t(x + "v", (m.v_channels, H)))])
+            own = ("q", "k") if m.v_from_k else ("q", "k", "v")
+            rows = dict(q=m.q_channels, k=m.k_channels, v=m.v_channels)
+            L.w_in, L.offs = fuse([(n, t(x + n, (rows[n], H))) for n in own] + ([("g", t(x + "g", (m.heads, H)))] if m.gate else []))
             if m.conv:
-                L.conv_w = torch.cat([f(x + n + ".conv") for n in ("q", "k", "v")])
+                L.conv_w = torch.cat([f(x + n + ".conv") for n in own])
                 if tuple(L.conv_w.shape) != (m.conv_channels, m.conv):
                     raise ValueError(f"{x}*.conv: {tuple(L.conv_w.shape)}, the configuration says {(m.conv_channels, m.conv)}")
                 L.conv_w = L.conv_w.T.contiguous()
+            if m.qk_norm:
+                L.q_norm, L.k_norm = (f(x + n + ".norm", (m.dim if m.qk_norm == "head" else rows[n],)) for n in ("q", "k"))
+            if m.sink:
+                L.sink = f(x + "sink", (m.heads,))
             L.lam = 0.0
             if m.maps == 2:
                 q1, k1, q2, k2 = (get(x + n).double() for n in ("lq1", "lk1", "lq2", "lk2"))
                 L.lam = float((q1 * k1).sum().exp() - (q2 * k2).sum().exp()) + m.diff
 
+        def latent(m: LatentSpec, x: str, L: HybridLayer) -> None:
+            L.w_in, L.offs = fuse([("q", t(x + "q", (m.heads * (m.dim + m.rot_dim), H))), ("kv", t(x + "dkv", (m.record, H)))]
+                                  + ([("g", t(x + "g", (m.heads * m.vdim, H)))] if m.gate else []))
+            L.kv_norm = f(x + "dkv.norm", (m.kv_rank,))
+            uk = t(x + "uk", (m.heads * m.dim, m.kv_rank)).view(m.heads, m.dim, m.kv_rank)
+            L.w_uk = torch.zeros(m.heads, m.kv_rank, pad8(m.dim), dtype=dt, device=device)
+            L.w_uk[..., :m.dim] = uk.transpose(1, 2)
+            L.w_uv = torch.zeros(m.heads, m.vdim, pad8(m.kv_rank), dtype=dt, device=device)
+            L.w_uv[..., :m.kv_rank] = t(x + "uv", (m.heads * m.vdim, m.kv_rank)).view(m.heads, m.vdim, m.kv_rank)
+            if tensor_core_latent(cfg, m):
+                L.w_kb = uk.reshape(m.heads * m.dim, m.kv_rank).contiguous()
+
+        def routed(r: RouterSpec, y: str, L: HybridLayer) -> None:
+            L.router, L.correction = reads(t(y + "router", (r.outputs, H))), f(y + ("router.b" if r.logit_bias else "correction"), (r.outputs,))
+            F = pad8(r.ffn)
+            L.w_gate, L.w_up = (torch.zeros(r.experts, F, Hp, dtype=dt, device=device) for _ in range(2))
+            L.w_down = torch.zeros(r.experts, Hp, F, dtype=dt, device=device)
+            for e in range(r.experts):
+                L.w_gate[e, :r.ffn, :H] = t(f"{y}e{e}.gate", (r.ffn, H))
+                L.w_up[e, :r.ffn, :H] = t(f"{y}e{e}.up", (r.ffn, H))
+                L.w_down[e, :H, :r.ffn] = t(f"{y}e{e}.down", (H, r.ffn))
+
         W.embed, W.final_norm, W.lm_head = t("embed", (cfg.vocab_size, H)), t("final.norm", (H,)), reads(t("head", (cfg.vocab_size, H)))
+        if cfg.loop and cfg.loop_join:
+            w = t("loop.in", (H, 2 * H))
+            W.loop_in = torch.cat([reads(w[:, :H]), reads(w[:, H:])], 1).contiguous()
+            W.loop_step = t("loop.step", (cfg.loop[2], H))
         for i, spec in enumerate(cfg.layer_specs):
             pre, m, r, L = f"l{i}.", spec.mixer, spec.router, HybridLayer()
             x = pre + "mix."
             if spec.parallel:
+                d, y = spec.dense, pre + "mlp."
                 L.norm1 = t(pre + "norm1", (H,))
-                attention(m, x, L)
-                L.w_out, d = heads_o(x + "o", m.heads, m.vdim), spec.dense
+                if spec.two_norms and (d is not None or r is not None):
+                    L.norm2 = t(pre + "norm2", (H,))
+                if isinstance(m, LatentSpec):
+                    if m.gate:
+                        raise ValueError(f"layer {i}: gated latent attention beside a feed-forward is not supported")
+                    latent(m, x, L)
+                else:
+                    attention(m, x, L)
+                if r is not None:
+                    routed(r, y, L)
+                    y += "shared."
+                L.w_out = heads_o(x + "o", m.heads, m.vdim)
                 if d is not None:
-                    y, F = pre + "mlp.", pad8(d.ffn)
-                    L.w_gate, L.w_up = (torch.zeros(F, Hp, dtype=dt, device=device) for _ in range(2))
-                    L.w_gate[:d.ffn, :H], L.w_up[:d.ffn, :H] = t(y + "gate", (d.ffn, H)), t(y + "up", (d.ffn, H))
+                    F = out_columns(m, d)[1]
+                    L.d_gate, L.d_up = (torch.zeros(F, Hp, dtype=dt, device=device) for _ in range(2))
+                    L.d_gate[:d.ffn, :H], L.d_up[:d.ffn, :H] = t(y + "gate", (d.ffn, H)), t(y + "up", (d.ffn, H))
                     down = torch.zeros(Hp, F, dtype=dt, device=device)
                     down[:H, :d.ffn] = t(y + "down", (H, d.ffn))
                     L.w_out = torch.cat([L.w_out, down], 1).contiguous()
@@ -136,16 +204,7 @@ class HybridWeights:
             L.norm1, L.norm1b = t(pre + "norm1", (H,)), t(pre + "norm1b", (H,))
             L.canon1 = t(pre + "canon1", (H, cfg.canon_taps)).T.contiguous()
             if isinstance(m, LatentSpec):
-                L.w_in, L.offs = fuse([("q", t(x + "q", (m.heads * (m.dim + m.rot_dim), H))), ("kv", t(x + "dkv", (m.record, H))),
-                                       ("g", t(x + "g", (m.heads * m.vdim, H)))])
-                L.kv_norm = f(x + "dkv.norm")
-                uk = t(x + "uk", (m.heads * m.dim, m.kv_rank)).view(m.heads, m.dim, m.kv_rank)
-                L.w_uk = torch.zeros(m.heads, m.kv_rank, pad8(m.dim), dtype=dt, device=device)
-                L.w_uk[..., :m.dim] = uk.transpose(1, 2)
-                L.w_uv = torch.zeros(m.heads, m.vdim, pad8(m.kv_rank), dtype=dt, device=device)
-                L.w_uv[..., :m.kv_rank] = t(x + "uv", (m.heads * m.vdim, m.kv_rank)).view(m.heads, m.vdim, m.kv_rank)
-                if tensor_core_latent(cfg, m):
-                    L.w_kb = uk.reshape(m.heads * m.dim, m.kv_rank).contiguous()
+                latent(m, x, L)
             else:
                 kd, vd = m.kv_heads * m.dim, m.heads * m.vdim
                 L.w_in, L.offs = fuse([(n, t(x + n, (rows, H))) for n, rows in
@@ -159,14 +218,7 @@ class HybridWeights:
                 y = pre + "mlp."
                 L.norm2, L.norm2b = t(pre + "norm2", (H,)), t(pre + "norm2b", (H,))
                 L.canon2 = t(pre + "canon2", (H, cfg.canon_taps)).T.contiguous()
-                L.router, L.correction = reads(t(y + "router", (r.outputs, H))), f(y + "correction")
-                F = pad8(r.ffn)
-                L.w_gate, L.w_up = (torch.zeros(r.experts, F, Hp, dtype=dt, device=device) for _ in range(2))
-                L.w_down = torch.zeros(r.experts, Hp, F, dtype=dt, device=device)
-                for e in range(r.experts):
-                    L.w_gate[e, :r.ffn, :H] = t(f"{y}e{e}.gate", (r.ffn, H))
-                    L.w_up[e, :r.ffn, :H] = t(f"{y}e{e}.up", (r.ffn, H))
-                    L.w_down[e, :H, :r.ffn] = t(f"{y}e{e}.down", (H, r.ffn))
+                routed(r, y, L)
             W.layers.append(L)
         return W
 
@@ -183,7 +235,7 @@ class HybridWeights:
         def get(name: str) -> torch.Tensor:
             shape = shapes[name]
             if name.rsplit(".", 1)[-1].startswith("norm"):
-                return torch.full(shape, 1.0 - cfg.norm_offset, device=device)
+                return torch.full(shape, 1.0 if ".mix." in name else 1.0 - cfg.norm_offset, device=device)
             s = 0.3 if "conv" in name or "canon" in name else std
             x = torch.empty(shape, dtype=torch.float32, device=device).normal_(0.0, s, generator=g)
             return x - 3.0 if name.endswith("dt_bias") else x
@@ -194,37 +246,65 @@ def tensor_shapes(cfg: ModelConfig) -> dict[str, tuple]:
     """Every tensor of the checkpoint and its shape."""
     H = cfg.hidden
     out: dict[str, tuple] = {"embed": (cfg.vocab_size, H), "final.norm": (H,), "head": (cfg.vocab_size, H)}
+    if cfg.loop and cfg.loop_join:
+        out.update({"loop.in": (H, 2 * H), "loop.step": (cfg.loop[2], H)})
     for i, spec in enumerate(cfg.layer_specs):
         pre, m, r = f"l{i}.", spec.mixer, spec.router
         x = pre + "mix."
         if spec.parallel:
             out[pre + "norm1"], out[x + "o"] = (H,), (H, m.heads * m.vdim)
-            for n, c in (("q", m.q_channels), ("k", m.k_channels), ("v", m.v_channels)):
-                out[x + n] = (c, H)
-                if m.conv:
-                    out[x + n + ".conv"] = (c, m.conv)
-            if m.maps == 2:
-                out.update({x + n: (m.dim,) for n in ("lq1", "lk1", "lq2", "lk2")})
+            if spec.two_norms and (spec.dense is not None or r is not None):
+                out[pre + "norm2"] = (H,)
+            if isinstance(m, LatentSpec):
+                out.update(_latent_shapes(x, m, H))
+            else:
+                for n, c in (("q", m.q_channels), ("k", m.k_channels)) + (() if m.v_from_k else (("v", m.v_channels),)):
+                    out[x + n] = (c, H)
+                    if m.conv:
+                        out[x + n + ".conv"] = (c, m.conv)
+                    if m.qk_norm and n != "v":
+                        out[f"{x}{n}.norm"] = (m.dim if m.qk_norm == "head" else c,)
+                if m.sink:
+                    out[x + "sink"] = (m.heads,)
+                if m.gate:
+                    out[x + "g"] = (m.heads, H)
+                if m.maps == 2:
+                    out.update({x + n: (m.dim,) for n in ("lq1", "lk1", "lq2", "lk2")})
+            y = pre + "mlp."
+            if r is not None:
+                out.update(_routed_shapes(y, r, H))
+                y += "shared."
             if spec.dense is not None:
                 d = spec.dense.ffn
-                out.update({pre + "mlp.gate": (d, H), pre + "mlp.up": (d, H), pre + "mlp.down": (H, d)})
+                out.update({y + "gate": (d, H), y + "up": (d, H), y + "down": (H, d)})
             continue
-        out.update({pre + "norm1": (H,), pre + "norm1b": (H,), pre + "canon1": (H, cfg.canon_taps), x + "o": (H, m.heads * m.vdim),
-                    x + "g": (m.heads * m.vdim, H)})
+        out.update({pre + "norm1": (H,), pre + "norm1b": (H,), pre + "canon1": (H, cfg.canon_taps), x + "o": (H, m.heads * m.vdim)})
         if isinstance(m, LatentSpec):
-            out.update({x + "q": (m.heads * (m.dim + m.rot_dim), H), x + "dkv": (m.record, H), x + "dkv.norm": (m.kv_rank,),
-                        x + "uk": (m.heads * m.dim, m.kv_rank), x + "uv": (m.heads * m.vdim, m.kv_rank)})
+            out.update(_latent_shapes(x, m, H))
         else:
             kd, vd = m.kv_heads * m.dim, m.heads * m.vdim
             for n, c in (("q", kd), ("k", kd), ("v", vd)):
                 out[x + n], out[x + n + ".conv"] = (c, H), (c, m.conv)
-            out.update({x + "b": (m.heads, H), x + "a": (m.heads, H), x + "A_log": (m.heads,), x + "dt_bias": (m.heads,), x + "norm": (m.vdim,)})
+            out.update({x + "g": (vd, H), x + "b": (m.heads, H), x + "a": (m.heads, H), x + "A_log": (m.heads,), x + "dt_bias": (m.heads,),
+                        x + "norm": (m.vdim,)})
         if r is not None:
-            y = pre + "mlp."
-            out.update({pre + "norm2": (H,), pre + "norm2b": (H,), pre + "canon2": (H, cfg.canon_taps), y + "router": (r.outputs, H),
-                        y + "correction": (r.outputs,)})
-            for e in range(r.experts):
-                out.update({f"{y}e{e}.gate": (r.ffn, H), f"{y}e{e}.up": (r.ffn, H), f"{y}e{e}.down": (H, r.ffn)})
+            out.update({pre + "norm2": (H,), pre + "norm2b": (H,), pre + "canon2": (H, cfg.canon_taps)})
+            out.update(_routed_shapes(pre + "mlp.", r, H))
+    return out
+
+
+def _latent_shapes(x: str, m: LatentSpec, H: int) -> dict[str, tuple]:
+    out = {x + "q": (m.heads * (m.dim + m.rot_dim), H), x + "dkv": (m.record, H), x + "dkv.norm": (m.kv_rank,),
+           x + "uk": (m.heads * m.dim, m.kv_rank), x + "uv": (m.heads * m.vdim, m.kv_rank)}
+    if m.gate:
+        out[x + "g"] = (m.heads * m.vdim, H)
+    return out
+
+
+def _routed_shapes(y: str, r: RouterSpec, H: int) -> dict[str, tuple]:
+    out = {y + "router": (r.outputs, H), y + ("router.b" if r.logit_bias else "correction"): (r.outputs,)}
+    for e in range(r.experts):
+        out.update({f"{y}e{e}.gate": (r.ffn, H), f"{y}e{e}.up": (r.ffn, H), f"{y}e{e}.down": (H, r.ffn)})
     return out
 
 
@@ -301,8 +381,7 @@ class _LatentWs:
         self.o_slab = torch.zeros(m.heads * rows * pad8(m.kv_rank), **kw)
         self.q_abs = torch.zeros(max_tokens, m.heads, record_pitch(m), **kw)
         self.attn = torch.zeros(max_tokens, m.heads, pad8(m.vdim), **kw)
-        i = torch.arange(0, m.rot_dim, 2, dtype=torch.float64)
-        self.inv_freq = (m.rope_base ** (-i / max(1, m.rot_dim))).float().to(device)
+        self.inv_freq = rope_frequencies(m.rope).to(device)
         self.lat = self.k_exp = self.v_exp = None      # expanded-form prompts: made on first use
 
 
@@ -342,6 +421,10 @@ class HybridEngine:
         Hp = pad8(H)                     # rows the matrix products read are whole 16-byte pieces; the padding stays zero
         ws.h = [torch.zeros(max_tokens, Hp, dtype=dt, device=dev) for _ in range(2)]
         ws.y = torch.zeros(max_tokens, Hp, dtype=dt, device=dev)
+        ws.h2 = torch.zeros(max_tokens, Hp, dtype=dt, device=dev) if any(L.norm2 is not None and L.norm2b is None for L in weights.layers) else None
+        if weights.loop_in is not None:  # [x | embedding row] of a pass's joining product, and what comes out of it
+            ws.join = torch.zeros(max_tokens, 2 * Hp, dtype=dt, device=dev)
+            ws.joined = torch.empty(max_tokens, H, dtype=torch.float32, device=dev)
         ws.proj = torch.empty(max_tokens * max(L.w_in.shape[0] for L in weights.layers), dtype=dt, device=dev)
         outs = max((s.router.outputs for s in cfg.layer_specs if s.router), default=1)
         ws.router = torch.empty(max_tokens * outs, dtype=torch.float32, device=dev)
@@ -381,7 +464,7 @@ class HybridEngine:
         self._logits = torch.empty(rows, pad8(cfg.vocab_size), dtype=torch.float32, device=dev)
         self.logits = self._logits[:, :cfg.vocab_size]
         self.next_tokens = torch.empty(rows, dtype=torch.int32, device=dev)
-        self._tiles: dict[tuple[int, int], _HeadTiles] = {}
+        self._tiles: dict[tuple[int, int, int], _HeadTiles] = {}
         self._blocks: dict = {}
         self._zero1 = torch.zeros(1, dtype=torch.int32, device=dev)
         self._scratch: torch.Tensor | None = None
@@ -392,19 +475,34 @@ class HybridEngine:
         self._pending: dict = {}
 
     # ---- between sublayers ------------------------------------------------------------------------------------------
-    def _between(self, b: Batch, T: int, w: torch.Tensor, conv: torch.Tensor | None, off: int = 0, add_embedding: bool = False) -> torch.Tensor:
-        """Residual, norms and input convolution up to the next sublayer; returns its input rows."""
-        ws, p = self.ws, self._pending
-        h = ws.h[self._hi][:T]
+    def _source(self, b: Batch, add_embedding: bool = False) -> dict:
+        """Where a launch between sublayers takes the residual from."""
         src = {} if self._x is None else dict(x_in=self._x)
         if self._x is None or add_embedding:
-            src.update(tokens=b.tokens, embed=self.W.embed)
+            src.update(tokens=b.tokens, embed=self.W.embed, embed_scale=self.cfg.embed_scale)
+        return src
+
+    def _between(self, b: Batch, T: int, w: torch.Tensor, conv: torch.Tensor | None, off: int = 0, add_embedding: bool = False,
+                 step: torch.Tensor | None = None, w2: torch.Tensor | None = None) -> torch.Tensor:
+        """Residual, norms and input convolution up to the next sublayer; returns its input rows (``w2``: the same norm's rows under
+        other weights go to ``ws.h2``)."""
+        ws, p = self.ws, self._pending
+        h = ws.h[self._hi][:T]
         xo = ws.x[0 if self._x is None or self._x.data_ptr() != ws.x[0].data_ptr() else 1][:T]
         K.norm_conv(h, w, self.cfg.norm_groups, self.cfg.rms_eps, conv=conv, x_out=xo, state=self.kv.state, state_off=off,
-                    state_in=b.state_in, state_out=b.state_out, q_start=b.q_start, w_offset=self.cfg.norm_offset, **src, **p)
+                    state_in=b.state_in, state_out=b.state_out, q_start=b.q_start, w_offset=self.cfg.norm_offset, step=step,
+                    w2=w2, h2_out=ws.h2[:T] if w2 is not None else None, **self._source(b, add_embedding), **p)
         self._x, self._hi = xo, self._hi ^ 1
         self.launches += 1
         return h
+
+    def _join(self, b: Batch, T: int) -> None:
+        """Start of a pass: the residual becomes a product of [x; embedding row] (the embedding's half is there already)."""
+        ws, cfg = self.ws, self.cfg
+        K.norm_conv(ws.join[:T], None, cfg.norm_groups, cfg.rms_eps, **self._source(b), **self._pending)
+        K.linear(ws.join[:T], self.W.loop_in, out=ws.joined[:T], out_f32=True, swap=True if cfg.hidden % 4 else None)
+        self._x, self._pending = ws.joined[:T], {}
+        self.launches += 2
 
     def residual(self, T: int) -> torch.Tensor:
         """The residual stream [T, H] after everything launched so far (tests and traces)."""
@@ -417,6 +515,8 @@ class HybridEngine:
                 w, idx, n, ident = p["slots"]
                 rows = torch.where((idx >= n)[..., None], ident[:, :H].float()[:, None], y[:T * w.shape[1]].view(T, w.shape[1], -1))
                 y = (w[..., None] * rows).sum(1)
+                if p.get("base") is not None:
+                    y = y + p["base"][:, :H].float()
             if p.get("w_b") is None:
                 return x + y
             g = y.view(T, G, -1)
@@ -445,17 +545,19 @@ class HybridEngine:
             self._blocks[key] = (torch.arange(S, **i32).repeat_interleave(nb).contiguous(), (torch.arange(nb, **i32) * per).repeat(S).contiguous())
         return self._blocks[key]
 
-    def _latent(self, n: int, i: int, m: LatentSpec, h: torch.Tensor, T: int, b: Batch) -> None:
+    def _latent(self, n: int, i: int, m: LatentSpec, h: torch.Tensor, T: int, b: Batch, out: torch.Tensor | None = None) -> None:
+        """Latent attention of layer run n and its o projection into ``ws.y``; with ``out`` the heads' values go to that buffer's
+        first columns instead, without gate and projection."""
         L, ws, lw = self.W.layers[i], self.ws, self._lat[m]
         a = self._project(i, h, T)
         cache = self.kv.of_run[n]
-        key = (T, m.heads)
-        if key not in self._tiles:
-            self._tiles[key] = _HeadTiles(T, m.heads, self.device)
-        ht = self._tiles[key]
         dp, rp, vp, rec = pad8(m.dim), pad8(m.kv_rank), pad8(m.vdim), record_pitch(m)
+        attn = lw.attn[:T] if out is None else out
+        key = (T, m.heads, attn.stride(0) // vp)
+        if key not in self._tiles:
+            self._tiles[key] = _HeadTiles(T, m.heads, self.device, out_heads=key[2])
+        ht = self._tiles[key]
         fast = L.w_kb is not None
-        attn = lw.attn[:T]
         expanded = fast and b.prefill and b.fresh and T >= self.EXPANDED_PREFILL_TOKENS
         if expanded and lw.lat is None:
             rows, kw = -(-self.max_tokens // 64) * 64, dict(dtype=self.dtype, device=self.device)
@@ -463,26 +565,28 @@ class HybridEngine:
             lw.k_exp, lw.v_exp = torch.zeros(rows, m.heads * 128, **kw), torch.zeros(rows, m.heads * 128, **kw)
         slab = lw.q_slab[:m.heads * ht.t_pad * dp].view(m.heads, ht.t_pad, dp)
         o_slab = lw.o_slab[:m.heads * ht.t_pad * rp].view(m.heads, ht.t_pad, rp)
-        qg = (a[:, L.offs["q"]:L.offs["q"] + m.heads * (m.dim + m.rot_dim)], a[:, L.offs["g"]:L.offs["g"] + m.heads * m.vdim])
+        q = a[:, L.offs["q"]:L.offs["q"] + m.heads * (m.dim + m.rot_dim)]
         # (the batch-invariant form keeps one absorb / un-absorb route for every decode width: the grouped GEMMs)
         small = fast and T <= K.MLA_SMALL_ROWS and not self.fixed_kv_split
         K.latent_prep(a, L.offs["q"], L.offs["kv"], m.heads, m.dim, m.rot_dim, L.kv_norm, lw.inv_freq, b.positions, b.slots, cache,
                       None if expanded or small else slab, None if small else lw.q_abs[:T], self.cfg.rms_eps,
-                      lat_out=lw.lat[:T] if expanded else None)
+                      lat_out=lw.lat[:T] if expanded else None, halves=m.rope.halves, magnitude=m.rope.magnitude)
         self.launches += 1
         if small:
             # decode-sized step: rotation and absorb in one launch, un-absorb and output gate in another
-            K.mla_absorb_small(qg[0], L.w_uk, lw.inv_freq, b.positions, lw.q_abs[:T], m.heads, False)
+            K.mla_absorb_small(q, L.w_uk, lw.inv_freq, b.positions, lw.q_abs[:T], m.heads, not m.rope.halves, m.rope.magnitude)
             self._attend_tensor_core(m, lw, T, b, cache, o_slab, ht.t_pad)
-            K.mla_unabsorb_small(o_slab, L.w_uv, attn, T, gate=qg[1])
-            K.linear(attn.view(T, -1), L.w_o, out=ws.y[:T])
-            self.launches += 4
+            K.mla_unabsorb_small(o_slab, L.w_uv, attn, T, gate=a[:, L.offs["g"]:L.offs["g"] + m.heads * m.vdim] if m.gate else None)
+            self.launches += 3
+            if out is None:
+                K.linear(attn.view(T, -1), L.w_o, out=ws.y[:T])
+                self.launches += 1
             return
         if expanded:
             rows = -(-T // 64) * 64
             K.linear(lw.lat[:T], L.w_kb, out=lw.k_exp[:T])
             K.linear(lw.lat[:T], L.w_uv.view(m.heads * m.vdim, m.kv_rank), out=lw.v_exp[:T])
-            K.attn_prefill_mla(qg[0], lw.q_abs[:T], lw.k_exp[:rows], lw.v_exp[:rows], self._zero1, cache, b.page_table, b.seq_lens, b.q_start,
+            K.attn_prefill_mla(q, lw.q_abs[:T], lw.k_exp[:rows], lw.v_exp[:rows], self._zero1, cache, b.page_table, b.seq_lens, b.q_start,
                                attn, b.max_q_len, m.heads, m.scale, window=m.window)
             self.launches += 3
         else:
@@ -495,7 +599,10 @@ class HybridEngine:
             K.grouped_linear(o_slab.view(-1, rp), L.w_uv, attn, ht.tile_expert, ht.tile_row0, ht.num_tiles, ht.max_tiles, ht.tile_rows,
                              row_dst=ht.row_dst, ldo=vp, split_k=False)
             self.launches += 3
-        K.latent_gate(attn, a, L.offs["g"], m.heads, m.vdim)
+        if out is not None:
+            return
+        if m.gate:
+            K.latent_gate(attn, a, L.offs["g"], m.heads, m.vdim)
         K.linear(attn.view(T, -1), L.w_o, out=ws.y[:T])
         self.launches += 2
 
@@ -522,12 +629,14 @@ class HybridEngine:
         a = self._project(i, h, T)
         (k, v), q = self.kv.of_run[n], aw.q[:T]
         K.conv_rope_kv(a, L.offs, m, L.conv_w, aw.table, b.slots, q, k, v, state=self.kv.state, state_off=self.kv.offsets[n]["conv"],
-                       state_in=b.state_in, state_out=b.state_out, q_start=b.q_start)
+                       state_in=b.state_in, state_out=b.state_out, q_start=b.q_start, q_norm=L.q_norm, k_norm=L.k_norm, eps=self.cfg.rms_eps)
         self.launches += 2
+        gate = a[:, L.offs["g"]:L.offs["g"] + m.heads] if m.gate else None
         if not aw.tensor_core:
-            K.paged_attn(q, k, v, m, b.page_table, b.positions, b.q_start, out, pad8(m.vdim), L.lam, self.cfg.rms_eps)
+            K.paged_attn(q, k, v, m, b.page_table, b.positions, b.q_start, out, pad8(m.vdim), L.lam, self.cfg.rms_eps, sink=L.sink, gate=gate)
             return
-        kw = dict(scale=m.scale, window=m.window, keep=m.keep_first, maps=m.maps, lam=L.lam, out_scale=1.0 - m.diff, eps=self.cfg.rms_eps)
+        kw = dict(scale=m.scale, window=m.window, keep=m.keep_first, maps=m.maps, lam=L.lam, out_scale=1.0 - m.diff, eps=self.cfg.rms_eps,
+                  sink=L.sink, gate=gate)
         q = q.view(T, m.heads, 128)
         if b.prefill:
             K.attn_prefill(q, k, v, b.page_table, b.seq_lens, b.q_start, out, b.max_q_len, **kw)
@@ -542,15 +651,20 @@ class HybridEngine:
         self.launches += 1 if splits > 1 else 0
 
     def _parallel(self, n: int, i: int, spec, h: torch.Tensor, T: int, b: Batch) -> None:
-        """Mixer and feed-forward on the same rows; one product over both reads their outputs side by side."""
-        L, m = self.W.layers[i], spec.mixer
+        """Mixer and feed-forward on rows of the same residual; one product over both reads the mixer's values and the dense (or
+        shared expert's) activations side by side, the routed experts' rows are summed by the next launch between layers."""
+        L, m, r = self.W.layers[i], spec.mixer, spec.router
         act = self.ws.act[:T * L.w_out.shape[1]].view(T, L.w_out.shape[1])
-        self._attention(n, i, m, h, T, b, act)
+        (self._latent if isinstance(m, LatentSpec) else self._attention)(n, i, m, h, T, b, act)
+        f = self.ws.h2[:T] if L.norm2 is not None else h
         if spec.dense is not None:
-            K.linear(h, L.w_gate, out=act[:, m.heads * pad8(m.vdim):], w_up=L.w_up)
+            K.linear(f, L.d_gate, out=act[:, m.heads * pad8(m.vdim):], w_up=L.d_up)
             self.launches += 1
         K.linear(act, L.w_out, out=self.ws.y[:T])
         self.launches += 1
+        self._pending = dict(y=self.ws.y[:T])
+        if r is not None:
+            self._pending = dict(slots=self._experts(i, r, f, T), y=self._moe[r].att.combine, base=self.ws.y[:T])
 
     def _delta_mixer(self, n: int, i: int, m: DeltaSpec, h: torch.Tensor, T: int, b: Batch) -> None:
         L, ws = self.W.layers[i], self.ws
@@ -570,8 +684,8 @@ class HybridEngine:
     # ---- routed feed-forward ----------------------------------------------------------------------------------------
     def _experts(self, i: int, r, h: torch.Tensor, T: int) -> tuple:
         L, moe = self.W.layers[i], self._moe[r]
-        kw = dict(scoring="softmax", bias=L.correction, num_groups=r.groups, topk_groups=r.groups_kept, normalize=False, routed_scale=1.0,
-                  group_score="max")
+        kw = dict(scoring="softmax_bias" if r.logit_bias else "softmax", bias=L.correction, num_groups=r.groups, topk_groups=r.groups_kept,
+                  normalize=r.normalize, routed_scale=1.0, group_score="max")
         logits = None
         idx, w = moe.att.idx[:T], moe.att.w[:T]
         if self.dtype == torch.bfloat16 and T <= self.FUSED_ROUTE_TOKENS and h.shape[1] <= 8192:
@@ -594,14 +708,20 @@ class HybridEngine:
         self._x, self._hi, self._pending = None, 0, {}
         for r, (freq, table) in self._rope.items():
             if r.dims:
-                K.rope_table(b.positions, freq, table.view(-1)[:T * r.dims])
+                K.rope_table(b.positions, freq, table.view(-1)[:T * r.dims], r.magnitude)
                 self.launches += 1
+        if self.W.loop_in is not None:
+            K.norm_conv(self.ws.join[:T, pad8(self.cfg.hidden):], None, self.cfg.norm_groups, self.cfg.rms_eps, **self._source(b))
+            self.launches += 1
         for n, run in enumerate(self.cfg.layer_runs):
             i, spec = run.layer, self.cfg.layer_specs[run.layer]
             L, off, m, r = self.W.layers[i], self.kv.offsets[n], spec.mixer, spec.router
             if spec.parallel:
-                self._parallel(n, i, spec, self._between(b, T, L.norm1, None, add_embedding=run.add_embedding), T, b)
-                self._pending = dict(y=self.ws.y[:T])
+                step = None
+                if run.join >= 0:
+                    self._join(b, T)
+                    step = self.W.loop_step[run.join]
+                self._parallel(n, i, spec, self._between(b, T, L.norm1, None, add_embedding=run.add_embedding, step=step, w2=L.norm2), T, b)
                 if self.layer_hook is not None:
                     self.layer_hook(n, self.residual(T))
                 continue

@@ -160,9 +160,10 @@ class LatentCache:
 
 
 class _HeadTiles:
-    """Tile table that lets the grouped GEMM treat heads as experts over a head-major slab [heads, t_pad, *]."""
+    """Tile table that lets the grouped GEMM treat heads as experts over a head-major slab [heads, t_pad, *].  ``out_heads``: a token's
+    output rows are that many heads apart (0 = ``heads``)."""
 
-    def __init__(self, T: int, heads: int, device: torch.device):
+    def __init__(self, T: int, heads: int, device: torch.device, out_heads: int = 0):
         self.tile_rows = 16 if T <= 16 else 32 if T <= 32 else 64 if T <= 64 else 128
         per_head = (T + self.tile_rows - 1) // self.tile_rows
         self.t_pad = per_head * self.tile_rows
@@ -173,7 +174,7 @@ class _HeadTiles:
         self.max_tiles = heads * per_head
         self.num_tiles = torch.tensor([self.max_tiles], **i32)
         t = torch.arange(self.t_pad, **i32)
-        dst = t[None, :] * heads + h[:, None]
+        dst = t[None, :] * (out_heads or heads) + h[:, None]
         self.row_dst = torch.where(t[None, :] < T, dst, torch.full_like(dst, -1)).reshape(-1).contiguous()
 
 

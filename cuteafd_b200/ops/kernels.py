@@ -254,10 +254,14 @@ def bump_epoch(epoch: torch.Tensor) -> None:
 
 
 # ---- MoE -------------------------------------------------------------------------------------------
+SCORING = {"softmax": 0, "sigmoid": 1, "softmax_bias": 2}
+
+
 def route_topk(logits: torch.Tensor, top_k: int, scoring: str = "softmax", bias: torch.Tensor | None = None,
                num_groups: int = 1, topk_groups: int = 1, normalize: bool = True, routed_scale: float = 1.0,
                out_idx: torch.Tensor | None = None, out_w: torch.Tensor | None = None, group_score: str = "top2"):
-    """``group_score``: what a group counts by in group-limited routing, the sum of its two best ("top2") or its best ("max")."""
+    """``group_score``: what a group counts by in group-limited routing, the sum of its two best ("top2") or its best ("max").
+    ``scoring`` "softmax_bias": softmax over logits the bias is part of (elsewhere it takes part in the selection alone)."""
     T, E = logits.shape
     assert logits.dtype == torch.float32 and logits.is_contiguous()
     if out_idx is None:
@@ -265,7 +269,7 @@ def route_topk(logits: torch.Tensor, top_k: int, scoring: str = "softmax", bias:
     if out_w is None:
         out_w = torch.empty(T, top_k, dtype=torch.float32, device=logits.device)
     _n.check(_n.cuda_lib().cafd_route_topk(logits.data_ptr(), _ptr(bias), out_idx.data_ptr(), out_w.data_ptr(), T, E,
-                                           top_k, int(scoring == "sigmoid"), num_groups, topk_groups, int(normalize),
+                                           top_k, SCORING[scoring], num_groups, topk_groups, int(normalize),
                                            routed_scale, int(group_score == "max"), _stream()), "route_topk")
     return out_idx, out_w
 
@@ -330,7 +334,7 @@ def norm_route(h: torch.Tensor, ln_w: torch.Tensor | None, eps: float, router_w:
     assert buf.is_contiguous()
     _n.check(_n.cuda_lib().cafd_norm_route(h.data_ptr(), _ptr(ln_w), eps, router_w.data_ptr(), _ptr(bias), _ptr(x_out),
                                            out_idx.data_ptr(), out_w.data_ptr(), buf.data_ptr(), sc[1].data_ptr(), T, H, E, top_k,
-                                           int(scoring == "sigmoid"), num_groups, topk_groups, int(normalize), routed_scale,
+                                           SCORING[scoring], num_groups, topk_groups, int(normalize), routed_scale,
                                            int(group_score == "max"), _stream()), "norm_route")
 
 
@@ -417,13 +421,23 @@ def _attn_out(q: torch.Tensor, out: torch.Tensor, maps: int) -> int:
     return out.stride(0)
 
 
+def _gate(gate: torch.Tensor | None, q: torch.Tensor, heads: int) -> tuple[int | None, int]:
+    """Address and row pitch of an attention's output gates."""
+    if gate is None:
+        return None, 0
+    assert gate.shape == (q.shape[0], heads) and gate.stride(1) == 1 and gate.dtype == q.dtype
+    return gate.data_ptr(), gate.stride(0)
+
+
 def attn_decode(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, page_table: torch.Tensor,
                 seq_lens: torch.Tensor, q_start: torch.Tensor, out: torch.Tensor, scratch: torch.Tensor | None,
                 max_q_len: int, splits: int, scale: float | None = None, window: int = 0, keep: int = 0, maps: int = 1,
-                lam: float = 0.0, out_scale: float = 1.0, eps: float = 0.0) -> torch.Tensor:
+                lam: float = 0.0, out_scale: float = 1.0, eps: float = 0.0, sink: torch.Tensor | None = None,
+                gate: torch.Tensor | None = None) -> torch.Tensor:
     """``window`` > 0: a query at position t sees keys (t - window, t] (sliding-window layers) and the first ``keep``; the pages
     between are not read.  ``maps`` 2: q [T, heads, 2 x 64] and keys hold two score maps per head; the output is map 1 - ``lam`` *
-    map 2 over its root mean square (``eps`` inside), times ``out_scale``.  ``out``: [T, heads, D], or rows [T, columns] whose first
+    map 2 over its root mean square (``eps`` inside), times ``out_scale``.  ``sink`` [heads] fp32: its exponential joins a head's
+    denominator; ``gate`` [T, heads] (rows of any pitch): a head's output is multiplied by its sigmoid (one map).  ``out``: [T, heads, D], or rows [T, columns] whose first
     heads * D columns are written."""
     _, Hq, D = q.shape
     Hkv = k_cache.shape[1]                 # pools are [pages, kv heads, 64, D]
@@ -432,7 +446,8 @@ def attn_decode(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, p
     _n.check(_n.cuda_lib().cafd_attn_decode(q.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(), page_table.data_ptr(),
                                             seq_lens.data_ptr(), q_start.data_ptr(), out.data_ptr(), _ptr(scratch),
                                             num_seqs, max_q_len, max_pages, Hq, Hkv, D, splits, scale, int(window), int(keep),
-                                            _attn_out(q, out, maps), maps, lam, out_scale, eps, _stream()), "attn_decode")
+                                            _attn_out(q, out, maps), maps, lam, out_scale, eps, _ptr(sink), *_gate(gate, q, Hq), _stream()),
+             "attn_decode")
     return out
 
 
@@ -470,7 +485,7 @@ def attn_decode_scratch_floats(num_seqs: int, max_q_len: int, Hq: int, Hkv: int,
 def attn_prefill(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, page_table: torch.Tensor,
                  seq_lens: torch.Tensor, q_start: torch.Tensor, out: torch.Tensor, max_q_len: int,
                  scale: float | None = None, window: int = 0, keep: int = 0, maps: int = 1, lam: float = 0.0, out_scale: float = 1.0,
-                 eps: float = 0.0) -> torch.Tensor:
+                 eps: float = 0.0, sink: torch.Tensor | None = None, gate: torch.Tensor | None = None) -> torch.Tensor:
     """Prompt attention; the arguments mean what they mean for ``attn_decode``."""
     T, Hq, D = q.shape
     num_pages, Hkv = k_cache.shape[0], k_cache.shape[1]
@@ -480,7 +495,7 @@ def attn_prefill(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, 
                                              seq_lens.data_ptr(), q_start.data_ptr(), out.data_ptr(),
                                              status_word(q.device).data_ptr(), T, num_seqs, max_q_len, num_pages,
                                              max_pages, Hq, Hkv, D, scale, int(window), int(keep), _attn_out(q, out, maps), maps, lam,
-                                             out_scale, eps, _stream()), "attn_prefill")
+                                             out_scale, eps, _ptr(sink), *_gate(gate, q, Hq), _stream()), "attn_prefill")
     return out
 
 
@@ -632,7 +647,7 @@ def attn_prefill_mla(q_nope: torch.Tensor, q_rope: torch.Tensor, k_exp: torch.Te
     """MLA prefill in expanded form.  q_nope [T, heads * 192] (first 128 columns of each head are used), q_rope
     [T, heads, 576]-like buffer holding the rotated rope dims at ``qr_col0`` of every head, k_exp / v_exp
     [rows, heads * 128] (kv_b applied to the cached latents in order; rows a multiple of 64), the latent cache for
-    the shared rope keys.  out [T, heads, 128]."""
+    the shared rope keys.  out [T, heads, 128], or rows [T, columns] whose first heads * 128 columns are written."""
     T = q_nope.shape[0]
     S, max_pages = page_table.shape
     assert q_nope.stride(1) == 1
@@ -642,7 +657,7 @@ def attn_prefill_mla(q_nope: torch.Tensor, q_rope: torch.Tensor, k_exp: torch.Te
                                                  v_exp.data_ptr(), k_exp.shape[0], kv_tmp_start.data_ptr(), latent_cache.data_ptr(),
                                                  page_table.data_ptr(), seq_lens.data_ptr(), q_start.data_ptr(), out.data_ptr(),
                                                  status_word(q_nope.device).data_ptr(), T, S, max_q_len, latent_cache.shape[0],
-                                                 max_pages, heads, scale, window, _stream()), "attn_prefill_mla")
+                                                 max_pages, heads, scale, window, out.stride(0), _stream()), "attn_prefill_mla")
     return out
 
 
@@ -660,48 +675,55 @@ MLA_SMALL_ROWS = 16      # steps of at most this many rows take the decode-sized
 
 
 def mla_absorb_small(q: torch.Tensor, w_uk: torch.Tensor, inv_freq: torch.Tensor, positions: torch.Tensor, q_abs: torch.Tensor,
-                     heads: int, interleaved: bool) -> None:
+                     heads: int, interleaved: bool, magnitude: float = 1.0) -> None:
     """Decode-sized steps (T <= 16): q [T, heads*192] -> q_abs [T, heads, 576] in one launch: the 128 nope dims of
-    every head multiplied by W_uk[h] [512, 128] into the latent part, the 64 rope dims rotated into the tail."""
+    every head multiplied by W_uk[h] [512, 128] into the latent part, the 64 rope dims rotated into the tail (cosines and sines
+    times ``magnitude``)."""
     T = q.shape[0]
     assert T <= MLA_SMALL_ROWS and q.shape[1] == heads * 192 and w_uk.shape == (heads, 512, 128) and w_uk.is_contiguous()
     _n.check(_n.cuda_lib().cafd_mla_absorb_small(q.data_ptr(), q.stride(0), w_uk.data_ptr(), inv_freq.data_ptr(),
-                                                 positions.data_ptr(), q_abs.data_ptr(), T, heads, int(interleaved), _stream()),
+                                                 positions.data_ptr(), q_abs.data_ptr(), T, heads, int(interleaved), magnitude, _stream()),
              "mla_absorb_small")
 
 
 def mla_unabsorb_small(o_lat: torch.Tensor, w_uv: torch.Tensor, attn: torch.Tensor, T: int, gate: torch.Tensor | None = None) -> None:
-    """Decode-sized steps: o_lat [heads, t_pad, 512] (head-major attention output) -> attn [T, heads*128] through
+    """Decode-sized steps: o_lat [heads, t_pad, 512] (head-major attention output) -> attn [T, heads*128] (or longer rows) through
     W_uv[h] [128, 512]; ``gate`` [T, heads*128] (any row stride): times sigmoid(gate)."""
     heads, t_pad, _ = o_lat.shape
-    assert T <= MLA_SMALL_ROWS and w_uv.shape == (heads, 128, 512) and w_uv.is_contiguous() and attn.is_contiguous()
+    assert T <= MLA_SMALL_ROWS and w_uv.shape == (heads, 128, 512) and w_uv.is_contiguous() and attn.stride(-1) == 1
     _n.check(_n.cuda_lib().cafd_mla_unabsorb_small(o_lat.data_ptr(), t_pad, w_uv.data_ptr(), attn.data_ptr(), T, heads, _ptr(gate),
-                                                   gate.stride(0) if gate is not None else 0, _stream()),
+                                                   gate.stride(0) if gate is not None else 0, attn.stride(0), _stream()),
              "mla_unabsorb_small")
 
 
 # ---- per-layer hybrids (csrc/hybrid_norm.cu, latent.cu, delta.cu, conv_rope.cu, attention_any.cu) --------------------------------------------
-def norm_conv(h_out: torch.Tensor, w: torch.Tensor, groups: int, eps: float, *, tokens: torch.Tensor | None = None,
+def norm_conv(h_out: torch.Tensor, w: torch.Tensor | None, groups: int, eps: float, *, tokens: torch.Tensor | None = None,
               embed: torch.Tensor | None = None, x_in: torch.Tensor | None = None, y: torch.Tensor | None = None,
               w_b: torch.Tensor | None = None, slots: tuple | None = None, conv: torch.Tensor | None = None,
               x_out: torch.Tensor | None = None, rows: torch.Tensor | None = None, state: torch.Tensor | None = None, state_off: int = 0,
               state_in: torch.Tensor | None = None, state_out: torch.Tensor | None = None, q_start: torch.Tensor | None = None,
-              run: int = 0, w_offset: float = 0.0) -> None:
-    """Weights are in the activations' type.  x = embed[tokens], ``x_in`` (fp32) or, given both, their sum; x += groupnorm(y) * w_b
-    (without ``w_b``: x += y); h = groupnorm(x) * (w + ``w_offset``); h_out = h + causal_conv(h).
+              run: int = 0, w_offset: float = 0.0, embed_scale: float = 1.0, step: torch.Tensor | None = None,
+              base: torch.Tensor | None = None, w2: torch.Tensor | None = None, h2_out: torch.Tensor | None = None) -> None:
+    """Weights are in the activations' type.  x = embed[tokens] * ``embed_scale``, ``x_in`` (fp32) or, given both, their sum; x +=
+    ``step`` [H]; x += groupnorm(y) * w_b (without ``w_b``: x += y); h = groupnorm(x) * (w + ``w_offset``), without ``w`` h = x; h_out =
+    h + causal_conv(h).  ``w2`` / ``h2_out``: a second output of the same norm under weights of its own (no convolution).
 
     Rows of ``h_out``, ``y`` and the identity rows may be longer than H (whole 16-byte pieces); the rest is left alone.
     ``slots`` = (weights [T, k], ids [T, k], number of experts, identity rows): ``y`` then holds the routed experts' rows
-    [T * k, ...] and is their weighted sum.  ``conv`` [taps, H] (last row = current token) with the sequences'
+    [T * k, ...] and is their weighted sum, plus the rows of ``base``.  ``conv`` [taps, H] (last row = current token) with the sequences'
     earlier inputs in ``state`` [slots, floats] at ``state_off``.  ``rows``: compute only these rows (no convolution)."""
     a = _n.NormArgs()
-    H = w.shape[0]
+    H = w.shape[0] if w is not None else embed.shape[1] if embed is not None else x_in.shape[1]
     a.tokens, a.embed, a.x_in, a.y = _ptr(tokens), _ptr(embed), _ptr(x_in), _ptr(y)
-    a.w_b, a.w, a.conv, a.x_out, a.h_out, a.row_idx = _ptr(w_b), w.data_ptr(), _ptr(conv), _ptr(x_out), h_out.data_ptr(), _ptr(rows)
+    a.w_b, a.w, a.conv, a.x_out, a.h_out, a.row_idx = _ptr(w_b), _ptr(w), _ptr(conv), _ptr(x_out), h_out.data_ptr(), _ptr(rows)
     a.vocab = embed.shape[0] if embed is not None else 0
     a.T, a.H, a.groups, a.eps, a.run, a.w_off = h_out.shape[0], H, groups, eps, run, w_offset
     a.ldy, a.ldh = y.stride(0) if y is not None else 0, h_out.stride(0)
-    assert h_out.shape[1] >= H and h_out.stride(1) == 1 and w.dtype == h_out.dtype and (w_b is None or w_b.dtype == h_out.dtype)
+    a.base, a.step, a.w2, a.h2_out, a.e_scale = _ptr(base), _ptr(step), _ptr(w2), _ptr(h2_out), embed_scale
+    a.ldb = base.stride(0) if base is not None else 0
+    assert h_out.shape[1] >= H and h_out.stride(1) == 1 and all(v is None or (v.dtype == h_out.dtype and v.shape[0] == H) for v in (w, w_b, w2, step))
+    assert (x_in is None or (x_in.dtype == torch.float32 and x_in.is_contiguous() and x_in.shape[1] == H)) and (base is None or base.dtype == h_out.dtype)
+    assert h2_out is None or (h2_out.stride(0) == a.ldh and h2_out.dtype == h_out.dtype)
     if slots is not None:
         sw, si, n, ident = slots
         a.slot_w, a.slot_idx, a.n_experts, a.ident, a.top_k = sw.data_ptr(), si.data_ptr(), n, ident.data_ptr(), sw.shape[1]
@@ -718,23 +740,30 @@ def swap_ids(a: torch.Tensor, b: torch.Tensor) -> None:
     _n.check(_n.cuda_lib().cafd_swap_ids(a.data_ptr(), b.data_ptr(), a.numel(), _stream()), "swap_ids")
 
 
-def rope_table(positions: torch.Tensor, freq: torch.Tensor, out: torch.Tensor) -> None:
-    """out [T, half, 2] fp32 = cos, sin of positions [T] * freq [half]."""
+def rope_table(positions: torch.Tensor, freq: torch.Tensor, out: torch.Tensor, magnitude: float = 1.0) -> None:
+    """out [T, half, 2] fp32 = cos, sin of positions [T] * freq [half], times ``magnitude``."""
     T, half = positions.shape[0], freq.shape[0]
     assert out.is_contiguous() and out.numel() == 2 * T * half
-    _n.check(_n.cuda_lib().cafd_rope_table(positions.data_ptr(), freq.data_ptr(), out.data_ptr(), T, half, _stream()), "rope_table")
+    _n.check(_n.cuda_lib().cafd_rope_table(positions.data_ptr(), freq.data_ptr(), out.data_ptr(), T, half, magnitude, _stream()), "rope_table")
 
 
 def conv_rope_kv(proj: torch.Tensor, offs: dict, m, conv_w: torch.Tensor | None, table: torch.Tensor, slots: torch.Tensor, q_out: torch.Tensor,
                  k_cache: torch.Tensor, v_cache: torch.Tensor, *, state: torch.Tensor | None = None, state_off: int = 0,
-                 state_in: torch.Tensor | None = None, state_out: torch.Tensor | None = None, q_start: torch.Tensor | None = None) -> None:
-    """Convolution over time, rotation and the paged K / V write of one step.  ``m`` carries heads / kv_heads / maps / dim / vdim and
-    rope.dims, ``conv_w`` [taps, channels] fp32 (last row = the current token), ``table`` the step's ``rope_table``."""
+                 state_in: torch.Tensor | None = None, state_out: torch.Tensor | None = None, q_start: torch.Tensor | None = None,
+                 q_norm: torch.Tensor | None = None, k_norm: torch.Tensor | None = None, eps: float = 0.0) -> None:
+    """Convolution over time, norm of queries and keys, rotation and the paged K / V write of one step.  ``m``: an ``AttentionSpec``,
+    ``conv_w`` [taps, channels] fp32 (last row = the current token), ``table`` the step's ``rope_table``, ``q_norm`` / ``k_norm`` fp32
+    weights of the norms (``m.qk_norm``)."""
     p = _n.ConvRope()
     p.proj, p.conv_w, p.table, p.slots, p.q_start = proj.data_ptr(), _ptr(conv_w), table.data_ptr(), slots.data_ptr(), _ptr(q_start)
     p.q_out, p.k_cache, p.v_cache = q_out.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr()
-    p.T, p.ld, p.q_off, p.k_off, p.v_off = proj.shape[0], proj.stride(0), offs["q"], offs["k"], offs["v"]
-    p.nq, p.nk, p.nv = m.heads * m.maps * m.dim, m.kv_heads * m.maps * m.dim, m.kv_heads * m.vdim
+    p.T, p.ld, p.q_off, p.k_off, p.v_off = proj.shape[0], proj.stride(0), offs["q"], offs["k"], offs.get("v", 0)
+    p.nq, p.nk, p.nv = m.q_channels, m.k_channels, 0 if m.v_from_k else m.v_channels
+    p.norm, p.halves, p.v_from_k, p.eps = {"": 0, "head": 1, "all": 2}[m.qk_norm], int(m.rope.halves), int(m.v_from_k), eps
+    if m.qk_norm:
+        p.q_norm, p.k_norm = q_norm.data_ptr(), k_norm.data_ptr()
+        assert q_norm.dtype == k_norm.dtype == torch.float32 and q_norm.is_contiguous() and k_norm.is_contiguous()
+        assert (q_norm.numel(), k_norm.numel()) == ((m.dim, m.dim) if m.qk_norm == "head" else (p.nq, p.nk))
     p.maps_dim, p.dim, p.vdim, p.kv_heads, p.rot = m.maps * m.dim, m.dim, m.vdim, m.kv_heads, m.rope.dims
     assert q_out.is_contiguous() and k_cache.is_contiguous() and v_cache.is_contiguous() and q_out.dtype == proj.dtype == k_cache.dtype == v_cache.dtype
     assert q_out.numel() >= p.T * p.nq and k_cache.shape[1:] == (m.kv_heads, 64, p.maps_dim) and v_cache.shape[1:] == (m.kv_heads, 64, m.vdim)
@@ -747,9 +776,11 @@ def conv_rope_kv(proj: torch.Tensor, offs: dict, m, conv_w: torch.Tensor | None,
 
 
 def paged_attn(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, m, page_table: torch.Tensor, positions: torch.Tensor,
-               q_start: torch.Tensor, out: torch.Tensor, head_pitch: int, lam: float = 0.0, eps: float = 0.0) -> None:
+               q_start: torch.Tensor, out: torch.Tensor, head_pitch: int, lam: float = 0.0, eps: float = 0.0,
+               sink: torch.Tensor | None = None, gate: torch.Tensor | None = None) -> None:
     """Attention at any head sizes: q [T, heads * maps * dim]; head h's values go to columns [h * head_pitch, + vdim) of ``out``
-    (rows of any length).  ``m``: an ``AttentionSpec``; ``lam`` / ``eps``: second map's weight and the head norm's epsilon."""
+    (rows of any length).  ``m``: an ``AttentionSpec``; ``lam`` / ``eps``: second map's weight and the head norm's epsilon; ``sink`` and
+    ``gate`` as in ``attn_decode``."""
     p = _n.PagedAttn()
     p.q, p.k_cache, p.v_cache, p.page_table = q.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(), page_table.data_ptr()
     p.positions, p.q_start, p.out = positions.data_ptr(), q_start.data_ptr(), out.data_ptr()
@@ -757,6 +788,8 @@ def paged_attn(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, m,
     p.S, p.max_pages = page_table.shape
     p.window, p.keep, p.ldo, p.head_pitch = m.window, m.keep_first, out.stride(0), head_pitch
     p.scale, p.lam, p.out_scale, p.eps = m.scale, lam, 1.0 - m.diff, eps
+    p.sink, (p.gate, p.gate_ld) = _ptr(sink), _gate(gate, q, m.heads)
+    assert sink is None or (sink.dtype == torch.float32 and sink.numel() == m.heads)
     assert q.is_contiguous() and q.dtype == out.dtype == k_cache.dtype and page_table.is_contiguous() and q_start.shape[0] == p.S + 1
     assert k_cache.is_contiguous() and v_cache.is_contiguous() and k_cache.shape[1:] == (m.kv_heads, 64, m.maps * m.dim)
     _n.check(_n.cuda_lib().cafd_paged_attn(C.byref(p), int(q.dtype == torch.float32), _stream()), "paged_attn")
@@ -771,16 +804,17 @@ def softcap(x: torch.Tensor, cap: float) -> torch.Tensor:
 
 def latent_prep(a: torch.Tensor, q_off: int, kv_off: int, heads: int, dim: int, rot: int, norm_w: torch.Tensor, inv_freq: torch.Tensor,
                 positions: torch.Tensor, slots: torch.Tensor, cache: torch.Tensor, slab: torch.Tensor | None, q_abs: torch.Tensor | None,
-                eps: float, lat_out: torch.Tensor | None = None) -> None:
-    """One launch per step and layer: latent norm, rotations, the cache record at ``slots`` and the query parts (unrotated
-    into ``slab`` [heads, t_pad, dim_pad], rotated into ``q_abs`` [T, heads, rec]); ``q_abs`` None: the record alone."""
+                eps: float, lat_out: torch.Tensor | None = None, halves: bool = True, magnitude: float = 1.0) -> None:
+    """One launch per step and layer: latent norm, rotations (pairs of ``halves`` or of neighbours; cosines and sines times
+    ``magnitude``), the cache record at ``slots`` and the query parts (unrotated into ``slab`` [heads, t_pad, dim_pad], rotated into
+    ``q_abs`` [T, heads, rec]); ``q_abs`` None: the record alone."""
     p = _n.LatentPrep()
     p.a, p.norm_w, p.inv_freq, p.positions, p.slots = a.data_ptr(), norm_w.data_ptr(), inv_freq.data_ptr(), positions.data_ptr(), slots.data_ptr()
     p.cache, p.slab, p.q_abs, p.lat_out = cache.data_ptr(), _ptr(slab), _ptr(q_abs), _ptr(lat_out)
     if q_abs is None:
         heads = 0
     p.lda, p.q_off, p.kv_off, p.heads, p.dim, p.rot, p.rank = a.stride(0), q_off, kv_off, heads, dim, rot, norm_w.shape[0]
-    p.rec, p.T, p.eps = cache.shape[-1], a.shape[0], eps
+    p.rec, p.T, p.eps, p.halves, p.mag = cache.shape[-1], a.shape[0], eps, int(halves), magnitude
     p.dim_pad, p.t_pad = (slab.shape[2], slab.shape[1]) if slab is not None else (0, 0)
     assert cache.is_contiguous() and a.dtype == cache.dtype
     assert q_abs is None or (q_abs.is_contiguous() and q_abs.shape[-1] == p.rec and q_abs.dtype == a.dtype)

@@ -1,6 +1,6 @@
 """CPU oracle of the per-layer hybrid decoders (``ModelConfig.layer_specs``): windowed latent attention layers and gated
 delta-rule layers in any order, each behind grouped RMS norms, input convolutions and a routed feed-forward; parallel
-layers of differential attention beside a dense feed-forward, some of them looped.
+layers of plain or differential or latent attention beside a dense or routed feed-forward, some of them looped.
 
 One function per mechanism, written as the equations read: no chunking, no absorbed products, one token at a time where a
 recurrence runs.  ``HybridRefDecoder`` strings them together over a parameter dictionary in the checkpoint's own tensor
@@ -41,53 +41,66 @@ def causal_conv(x: torch.Tensor, w: torch.Tensor, past: torch.Tensor) -> tuple[t
     return y, full[T:]
 
 
-def rotate_half(x: torch.Tensor, positions: torch.Tensor, base: float) -> torch.Tensor:
-    """x [T, ..., d]: dimension i is paired with i + d/2 and turned by position * base^(-2i/d)."""
-    d = x.shape[-1]
-    f = torch.tensor([base ** (-2.0 * i / d) for i in range(d // 2)], dtype=x.dtype)
-    a = positions.to(x.dtype)[:, None] * f
-    a = a.reshape(a.shape[0], *([1] * (x.dim() - 2)), d // 2)
-    u, v = x[..., :d // 2], x[..., d // 2:]
-    return torch.cat([u * a.cos() - v * a.sin(), v * a.cos() + u * a.sin()], -1)
-
-
 def scaled_frequencies(r: RopeSpec) -> list[float]:
-    """Turns per position of every rotated pair: short wavelengths as they are, long ones stretched by the factor, a linear
-    blend (in turns over the original length) between."""
+    """Turns per position (in radians) of every rotated pair.
+
+    bands: short wavelengths as they are, long ones stretched by the factor, a linear blend (in turns over the original length)
+    between.  linear: all stretched.  yarn: pair number x makes ``turns`` turns over the original length at
+    x = dims * ln(original / (2 pi turns)) / (2 ln base); from the x of ``high`` turns (rounded down) to that of ``low`` turns
+    (rounded up) the blend is linear in the pair's number."""
+    f = [r.base ** (-2.0 * i / r.dims) for i in range(r.dims // 2)]
+    if r.factor == 1.0:
+        return f
+    if r.kind == "linear":
+        return [x / r.factor for x in f]
     out = []
-    for i in range(r.dims // 2):
-        f = r.base ** (-2.0 * i / r.dims)
-        if r.factor != 1.0:
-            turns = r.original * f / (2.0 * math.pi)              # original length over wavelength
-            if turns < r.low:
-                f = f / r.factor
-            elif turns <= r.high:
-                s = (turns - r.low) / (r.high - r.low)
-                f = (1.0 - s) * f / r.factor + s * f
-        out.append(f)
+    if r.kind == "yarn":
+        number = lambda turns: r.dims * math.log(r.original / (2.0 * math.pi * turns)) / (2.0 * math.log(r.base))      # noqa: E731
+        lo, hi = max(math.floor(number(r.high)), 0), min(math.ceil(number(r.low)), r.dims - 1)
+        for i, x in enumerate(f):
+            ramp = min(1.0, max(0.0, (i - lo) / max(hi - lo, 0.001)))
+            out.append(x / r.factor * ramp + x * (1.0 - ramp))
+        return out
+    for x in f:
+        turns = r.original * x / (2.0 * math.pi)                  # original length over wavelength
+        if turns < r.low:
+            x = x / r.factor
+        elif turns <= r.high:
+            s = (turns - r.low) / (r.high - r.low)
+            x = (1.0 - s) * x / r.factor + s * x
+        out.append(x)
     return out
 
 
-def rotate_pairs(x: torch.Tensor, positions: torch.Tensor, r: RopeSpec) -> torch.Tensor:
-    """x [T, ..., d]: dimensions 2i and 2i + 1 of the first ``r.dims`` are a pair turned by position * frequency."""
+def rotate(x: torch.Tensor, positions: torch.Tensor, r: RopeSpec) -> torch.Tensor:
+    """x [T, ..., d]: the pairs of the first ``r.dims`` dimensions, neighbours (2i, 2i + 1) or halves (i, i + dims / 2), are turned by
+    position * frequency; cosines and sines carry the scaling's magnitude."""
+    h = r.dims // 2
+    mag = 0.1 * math.log(r.factor) + 1.0 if r.kind == "yarn" else 1.0
     a = positions.to(x.dtype)[:, None] * torch.tensor(scaled_frequencies(r), dtype=x.dtype)
-    a = a.reshape(a.shape[0], *([1] * (x.dim() - 2)), r.dims // 2)
+    a = a.reshape(a.shape[0], *([1] * (x.dim() - 2)), h)
+    c, s = mag * a.cos(), mag * a.sin()
+    first, second = (slice(0, h), slice(h, r.dims)) if r.halves else (slice(0, r.dims, 2), slice(1, r.dims, 2))
     out = x.clone()
-    u, v = x[..., 0:r.dims:2], x[..., 1:r.dims:2]
-    out[..., 0:r.dims:2] = u * a.cos() - v * a.sin()
-    out[..., 1:r.dims:2] = v * a.cos() + u * a.sin()
+    u, v = x[..., first], x[..., second]
+    out[..., first] = u * c - v * s
+    out[..., second] = v * c + u * s
     return out
 
 
-def sink_attention(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, start: int, window: int, keep: int, scale: float) -> torch.Tensor:
+def sink_attention(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, start: int, window: int, keep: int, scale: float,
+                   sink: torch.Tensor | None = None) -> torch.Tensor:
     """Softmax attention of q [T, H, Dk] (positions start, start + 1, ...) over k [L, H, Dk], v [L, H, Dv] (positions 0, 1, ...):
     the query at position i reads the keys j <= i that lie among the last ``window`` positions (0: anywhere) or the first
-    ``keep``."""
+    ``keep``.  ``sink`` [H]: exp(sink_h) joins head h's denominator, without a key or a value."""
     i = torch.arange(start, start + q.shape[0])[:, None]
     j = torch.arange(k.shape[0])[None]
     seen = (j <= i) & ((i - j < window) | (j < keep)) if window else j <= i
     s = torch.einsum("thd,jhd->htj", q, k) * scale
-    return torch.einsum("htj,jhd->thd", torch.softmax(s.masked_fill(~seen, -math.inf), -1), v)
+    s = s.masked_fill(~seen, -math.inf)
+    if sink is not None:
+        s = torch.cat([s, sink[:, None, None].expand(-1, q.shape[0], 1)], -1)
+    return torch.einsum("htj,jhd->thd", torch.softmax(s, -1)[..., :k.shape[0]], v)
 
 
 def difference_weight(p: Params, pre: str, diff: float) -> torch.Tensor:
@@ -101,11 +114,11 @@ def softcap(x: torch.Tensor, cap: float) -> torch.Tensor:
 
 def window_attention(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, start: int, window: int, scale: float) -> torch.Tensor:
     """Softmax attention of q [T, H, Dk] (positions start, start + 1, ...) over k [L, H, Dk], v [L, H, Dv] (positions 0, 1, ...);
-    the query at position i reads keys i - window + 1 .. i."""
+    the query at position i reads keys i - window + 1 .. i (window 0: 0 .. i)."""
     out = []
     for t in range(q.shape[0]):
         i = start + t
-        lo = max(0, i - window + 1)
+        lo = max(0, i - window + 1) if window else 0
         s = torch.einsum("hd,jhd->hj", q[t], k[lo:i + 1]) * scale
         out.append(torch.einsum("hj,jhd->hd", torch.softmax(s, -1), v[lo:i + 1]))
     return torch.stack(out)
@@ -149,8 +162,18 @@ def route(h: torch.Tensor, w: torch.Tensor, correction: torch.Tensor, r: RouterS
     return torch.tensor(ids), torch.stack(wts)
 
 
+def route_by_logits(h: torch.Tensor, w: torch.Tensor, bias: torch.Tensor, top: int) -> tuple[torch.Tensor, torch.Tensor]:
+    """The ``top`` largest of the biased logits; the weights are the softmax over those alone."""
+    z = h @ w.T + bias
+    ids = torch.tensor([sorted(range(z.shape[1]), key=lambda e: (-float(row[e]), e))[:top] for row in z])
+    return ids, torch.softmax(z.gather(1, ids), -1)
+
+
 def routed_ffn(h: torch.Tensor, p: Params, pre: str, r: RouterSpec) -> torch.Tensor:
-    ids, wts = route(h, p[pre + "router"], p[pre + "correction"], r)
+    if r.logit_bias:
+        ids, wts = route_by_logits(h, p[pre + "router"], p[pre + "router.b"], r.top)
+    else:
+        ids, wts = route(h, p[pre + "router"], p[pre + "correction"], r)
     y = torch.zeros_like(h)
     for e in ids.unique().tolist():
         t, slot = (ids == e).nonzero(as_tuple=True)
@@ -167,10 +190,10 @@ def latent_mixer(h: torch.Tensor, p: Params, pre: str, m: LatentSpec, eps: float
     T = h.shape[0]
     pos = torch.arange(start, start + T)
     q = (h @ p[pre + "q"].T).view(T, m.heads, m.dim + m.rot_dim)
-    q = torch.cat([q[..., :m.dim], rotate_half(q[..., m.dim:], pos, m.rope_base)], -1)
+    q = torch.cat([q[..., :m.dim], rotate(q[..., m.dim:], pos, m.rope)], -1)
     d = h @ p[pre + "dkv"].T
     c = rms(d[:, :m.kv_rank], eps) * p[pre + "dkv.norm"]
-    kr = rotate_half(d[:, m.kv_rank:], pos, m.rope_base)
+    kr = rotate(d[:, m.kv_rank:], pos, m.rope)
     st["c"] = torch.cat([st["c"], c])
     st["kr"] = torch.cat([st["kr"], kr])
     L = st["c"].shape[0]
@@ -178,7 +201,9 @@ def latent_mixer(h: torch.Tensor, p: Params, pre: str, m: LatentSpec, eps: float
     k = torch.cat([k, st["kr"][:, None].expand(L, m.heads, m.rot_dim)], -1)
     v = (st["c"] @ p[pre + "uv"].T).view(L, m.heads, m.vdim)
     o = window_attention(q, k, v, start, m.window, m.scale).reshape(T, m.heads * m.vdim)
-    return (o * torch.sigmoid(h @ p[pre + "g"].T)) @ p[pre + "o"].T
+    if m.gate:
+        o = o * torch.sigmoid(h @ p[pre + "g"].T)
+    return o @ p[pre + "o"].T
 
 
 def delta_mixer(h: torch.Tensor, p: Params, pre: str, m: DeltaSpec, eps: float, st: dict) -> torch.Tensor:
@@ -201,25 +226,46 @@ def delta_mixer(h: torch.Tensor, p: Params, pre: str, m: DeltaSpec, eps: float, 
 
 
 def attention_mixer(h: torch.Tensor, p: Params, pre: str, m: AttentionSpec, eps: float, start: int, st: dict) -> torch.Tensor:
-    """Attention with convolved and rotated queries and keys; with two maps per head their difference, normed per head."""
+    """Attention with convolved, normed and rotated queries and keys; with two maps per head their difference, normed per head."""
     T, rep = h.shape[0], m.heads // m.kv_heads
     pos = torch.arange(start, start + T)
     x = {}
-    for n in ("q", "k", "v"):
+    for n in ("q", "k") if m.v_from_k else ("q", "k", "v"):
         x[n] = h @ p[pre + n].T
         if m.conv:
             x[n], st["conv." + n] = causal_conv(x[n], p[pre + n + ".conv"], st["conv." + n])
-    q = rotate_pairs(x["q"].view(T, m.heads, m.maps, m.dim), pos, m.rope)
-    st["k"] = torch.cat([st["k"], rotate_pairs(x["k"].view(T, m.kv_heads, m.maps, m.dim), pos, m.rope)])
-    st["v"] = torch.cat([st["v"], x["v"].view(T, m.kv_heads, m.vdim)])
+    st["v"] = torch.cat([st["v"], x["k" if m.v_from_k else "v"].view(T, m.kv_heads, m.vdim)])
+    for n in ("q", "k"):
+        if m.qk_norm == "all":
+            x[n] = rms(x[n], eps) * p[f"{pre}{n}.norm"]
+        elif m.qk_norm == "head":
+            x[n] = (rms(x[n].view(T, -1, m.dim), eps) * p[f"{pre}{n}.norm"]).view(T, -1)
+    q = rotate(x["q"].view(T, m.heads, m.maps, m.dim), pos, m.rope)
+    st["k"] = torch.cat([st["k"], rotate(x["k"].view(T, m.kv_heads, m.maps, m.dim), pos, m.rope)])
     k, v = st["k"].repeat_interleave(rep, 1), st["v"].repeat_interleave(rep, 1)
-    a = [sink_attention(q[:, :, j], k[:, :, j], v, start, m.window, m.keep_first, m.scale) for j in range(m.maps)]
+    sink = p[pre + "sink"] if m.sink else None
+    a = [sink_attention(q[:, :, j], k[:, :, j], v, start, m.window, m.keep_first, m.scale, sink) for j in range(m.maps)]
     o = a[0] if m.maps == 1 else rms(a[0] - difference_weight(p, pre, m.diff) * a[1], eps) * (1 - m.diff)
+    if m.gate:
+        o = o * torch.sigmoid(h @ p[pre + "g"].T)[..., None]
     return o.reshape(T, m.heads * m.vdim) @ p[pre + "o"].T
 
 
 def dense_ffn(h: torch.Tensor, p: Params, pre: str) -> torch.Tensor:
     return (silu(h @ p[pre + "gate"].T) * (h @ p[pre + "up"].T)) @ p[pre + "down"].T
+
+
+def feed_forward(h: torch.Tensor, p: Params, pre: str, spec) -> torch.Tensor:
+    """A parallel layer's: dense, or the routed experts with the shared one beside them."""
+    if spec.router is None:
+        return dense_ffn(h, p, pre)
+    y = routed_ffn(h, p, pre, spec.router)
+    return y if spec.dense is None else y + dense_ffn(h, p, pre + "shared.")
+
+
+def join_embedding(x: torch.Tensor, x0: torch.Tensor, p: Params, t: int) -> torch.Tensor:
+    """Start of pass t of a loop: a product of [x; embedding row] and the pass's own vector."""
+    return torch.cat([x, x0], -1) @ p["loop.in"].T + p["loop.step"][t]
 
 
 # ---- state ----------------------------------------------------------------------------------------------------------
@@ -238,7 +284,7 @@ class HybridState:
             if isinstance(m, AttentionSpec):
                 st.update(k=z(0, m.kv_heads, m.maps, m.dim), v=z(0, m.kv_heads, m.vdim))
                 for n, c in (("q", m.q_channels), ("k", m.k_channels), ("v", m.v_channels)):
-                    if m.conv:
+                    if m.conv and not (n == "v" and m.v_from_k):
                         st["conv." + n] = z(m.conv - 1, c)
             elif isinstance(m, LatentSpec):
                 st.update(c=z(0, m.kv_rank), kr=z(0, m.rot_dim))
@@ -281,9 +327,13 @@ class HybridRefDecoder:
         cfg, p, spec, pre = self.cfg, self.p, self.cfg.layer_specs[i], f"l{i}."
 
         if spec.parallel:
-            h = group_rms(x, p[pre + "norm1"] + cfg.norm_offset, cfg.norm_groups, cfg.rms_eps)
-            y = attention_mixer(h, p, pre + "mix.", spec.mixer, cfg.rms_eps, start, st)
-            return x + (y if spec.dense is None else y + dense_ffn(h, p, pre + "mlp."))
+            norm = lambda n: group_rms(x, p[pre + n] + cfg.norm_offset, cfg.norm_groups, cfg.rms_eps)      # noqa: E731
+            mixer = latent_mixer if isinstance(spec.mixer, LatentSpec) else attention_mixer
+            h = norm("norm1")
+            y = mixer(h, p, pre + "mix.", spec.mixer, cfg.rms_eps, start, st)
+            if spec.dense is None and spec.router is None:
+                return x + y
+            return x + (y + feed_forward(norm("norm2") if spec.two_norms else h, p, pre + "mlp.", spec))
 
         def sublayer(x, n, fn):
             h = group_rms(x, p[f"{pre}norm{n}"], cfg.norm_groups, cfg.rms_eps)
@@ -300,9 +350,11 @@ class HybridRefDecoder:
         return x
 
     def _run(self, tokens: torch.Tensor, kv: HybridState) -> torch.Tensor:
-        e, start = self.p["embed"][tokens], kv.length_
+        e, start = self.p["embed"][tokens] * self.cfg.embed_scale, kv.length_
         x = e
         for n, r in enumerate(self.cfg.layer_runs):
+            if r.join >= 0:
+                x = join_embedding(x, e, self.p, r.join)
             x = self._layer(r.layer, x + e if r.add_embedding else x, start, kv.layers[n])
             if self.trace is not None:
                 self.trace.append(x)
@@ -340,22 +392,51 @@ def init_hybrid_weights(cfg: ModelConfig, seed: int = 0, dtype: torch.dtype = to
     def near_one(n: int) -> torch.Tensor:
         return (1 - cfg.norm_offset + 0.2 * torch.randn(n, generator=g)).to(dtype)
 
+    def latent_weights(x: str, m: LatentSpec) -> None:
+        p.update({x + "q": w(m.heads * (m.dim + m.rot_dim), H), x + "dkv": w(m.kv_rank + m.rot_dim, H),
+                  x + "dkv.norm": 1 + 0.2 * w(m.kv_rank, s=1.0), x + "uk": w(m.heads * m.dim, m.kv_rank), x + "uv": w(m.heads * m.vdim, m.kv_rank)})
+        if m.gate:
+            p[x + "g"] = w(m.heads * m.vdim, H)
+
+    def routed_weights(x: str, r: RouterSpec) -> None:
+        p[x + "router"] = w(r.outputs, H)
+        p[x + ("router.b" if r.logit_bias else "correction")] = w(r.outputs, s=0.7 if r.logit_bias else 0.1)
+        for e in range(r.experts):
+            p[f"{x}e{e}.gate"], p[f"{x}e{e}.up"], p[f"{x}e{e}.down"] = w(r.ffn, H), w(r.ffn, H), w(H, r.ffn)
+
     H = cfg.hidden
-    p: Params = {"embed": w(cfg.vocab_size, H, s=1.0), "final.norm": near_one(H), "head": w(cfg.vocab_size, H)}
+    p: Params = {"embed": w(cfg.vocab_size, H, s=1.0 / cfg.embed_scale), "final.norm": near_one(H), "head": w(cfg.vocab_size, H)}
+    if cfg.loop and cfg.loop_join:
+        p["loop.in"], p["loop.step"] = w(H, 2 * H), w(cfg.loop[2], H, s=0.3)
     for i, spec in enumerate(cfg.layer_specs):
         pre, m, r = f"l{i}.", spec.mixer, spec.router
         if spec.parallel:
             x, d = pre + "mix.", spec.dense
             p[pre + "norm1"] = near_one(H)
-            for n, c in (("q", m.q_channels), ("k", m.k_channels), ("v", m.v_channels)):
-                p[x + n] = w(c, H)
-                if m.conv:
-                    p[x + n + ".conv"] = w(c, m.conv)
-            if m.maps == 2:
-                p.update({x + n: w(m.dim, s=0.5 * m.dim ** -0.5) for n in ("lq1", "lk1", "lq2", "lk2")})
+            if isinstance(m, LatentSpec):
+                latent_weights(x, m)
+            else:
+                for n, c in (("q", m.q_channels), ("k", m.k_channels), ("v", m.v_channels)):
+                    if n == "v" and m.v_from_k:
+                        continue
+                    p[x + n] = w(c, H)
+                    if m.conv:
+                        p[x + n + ".conv"] = w(c, m.conv)
+                    if m.qk_norm and n != "v":
+                        p[f"{x}{n}.norm"] = 1 + 0.2 * w(m.dim if m.qk_norm == "head" else c, s=1.0)
+                if m.sink:
+                    p[x + "sink"] = w(m.heads, s=1.5)
+                if m.gate:
+                    p[x + "g"] = w(m.heads, H)
+                if m.maps == 2:
+                    p.update({x + n: w(m.dim, s=0.5 * m.dim ** -0.5) for n in ("lq1", "lk1", "lq2", "lk2")})
             p[x + "o"] = w(H, m.heads * m.vdim)
+            if spec.two_norms and (r is not None or d is not None):
+                p[pre + "norm2"] = near_one(H)
+            if r is not None:
+                routed_weights(pre + "mlp.", r)
             if d is not None:
-                x = pre + "mlp."
+                x = pre + ("mlp.shared." if r is not None else "mlp.")
                 p[x + "gate"], p[x + "up"], p[x + "down"] = w(d.ffn, H), w(d.ffn, H), w(H, d.ffn)
             continue
         for n in ("norm1", "norm1b") + (("norm2", "norm2b") if r is not None else ()):
@@ -364,9 +445,7 @@ def init_hybrid_weights(cfg: ModelConfig, seed: int = 0, dtype: torch.dtype = to
             p[pre + n] = w(H, cfg.canon_taps, s=0.3)
         x = pre + "mix."
         if isinstance(m, LatentSpec):
-            p.update({x + "q": w(m.heads * (m.dim + m.rot_dim), H), x + "dkv": w(m.kv_rank + m.rot_dim, H),
-                      x + "dkv.norm": near_one(m.kv_rank), x + "uk": w(m.heads * m.dim, m.kv_rank),
-                      x + "uv": w(m.heads * m.vdim, m.kv_rank), x + "g": w(m.heads * m.vdim, H)})
+            latent_weights(x, m)
         else:
             kd, vd = m.kv_heads * m.dim, m.heads * m.vdim
             p.update({x + "q": w(kd, H), x + "k": w(kd, H), x + "v": w(vd, H), x + "g": w(vd, H), x + "b": w(m.heads, H),
@@ -374,11 +453,7 @@ def init_hybrid_weights(cfg: ModelConfig, seed: int = 0, dtype: torch.dtype = to
                       x + "norm": near_one(m.vdim), x + "q.conv": w(kd, m.conv), x + "k.conv": w(kd, m.conv), x + "v.conv": w(vd, m.conv)})
         p[x + "o"] = w(H, m.heads * m.vdim)
         if r is not None:
-            x = pre + "mlp."
-            p[x + "router"] = w(r.experts + r.identity, H)
-            p[x + "correction"] = w(r.experts + r.identity, s=0.1)
-            for e in range(r.experts):
-                p[f"{x}e{e}.gate"], p[f"{x}e{e}.up"], p[f"{x}e{e}.down"] = w(r.ffn, H), w(r.ffn, H), w(H, r.ffn)
+            routed_weights(pre + "mlp.", r)
     return p
 
 
@@ -387,6 +462,7 @@ def bf16_params(p: Params, dtype: torch.dtype = torch.float32) -> Params:
     return {k: v.to(torch.bfloat16).to(dtype) for k, v in p.items()}
 
 
-__all__ = ["HybridRefDecoder", "HybridState", "init_hybrid_weights", "bf16_params", "group_rms", "causal_conv", "rotate_half",
-           "scaled_frequencies", "rotate_pairs", "sink_attention", "difference_weight", "softcap", "attention_mixer", "dense_ffn",
-           "window_attention", "delta_recurrence", "route", "routed_ffn", "latent_mixer", "delta_mixer", "rms", "unit"]
+__all__ = ["HybridRefDecoder", "HybridState", "init_hybrid_weights", "bf16_params", "group_rms", "causal_conv", "rotate",
+           "scaled_frequencies", "sink_attention", "difference_weight", "softcap", "attention_mixer", "dense_ffn", "feed_forward",
+           "join_embedding", "window_attention", "delta_recurrence", "route", "route_by_logits", "routed_ffn", "latent_mixer", "delta_mixer",
+           "rms", "unit"]

@@ -9,7 +9,8 @@ from cuteafd_b200.ref import hybrid as R
 
 
 def latent(heads=3, dim=24, rot_dim=8, vdim=20, kv_rank=40, window=37, scale=None, base=5000.0):
-    return LatentSpec(heads, dim, rot_dim, vdim, kv_rank, window, scale if scale is not None else 1.7 * (dim + rot_dim) ** -0.5, base)
+    return LatentSpec(heads, dim, rot_dim, vdim, kv_rank, window, scale if scale is not None else 1.7 * (dim + rot_dim) ** -0.5,
+                      RopeSpec(rot_dim, base, halves=True))
 
 
 def delta(heads=6, kv_heads=2, dim=20, vdim=36, conv=3):

@@ -116,7 +116,7 @@ def test_frequencies_are_kept_stretched_and_blended():
 
 def test_rotation_pairs_neighbours_and_leaves_the_rest():
     x = torch.tensor([[1.0, 0.0, 0.0, 1.0, 5.0]], dtype=torch.float64)
-    y = R.rotate_pairs(x, torch.tensor([3]), RopeSpec(4, 100.0))
+    y = R.rotate(x, torch.tensor([3]), RopeSpec(4, 100.0))
     assert y[0].tolist() == pytest.approx([math.cos(3), math.sin(3), -math.sin(0.3), math.cos(0.3), 5.0])
 
 

@@ -87,7 +87,7 @@ def test_convolution_rotation_and_pages(dtype, m):
             if m.conv:
                 y, past[s] = R.causal_conv(xs, w, past[s])
             n = ls[s]
-            rot = lambda z, h: R.rotate_pairs(z.reshape(n, h, 2, m.dim).double(), ps, m.rope).float()      # noqa: E731
+            rot = lambda z, h: R.rotate(z.reshape(n, h, 2, m.dim).double(), ps, m.rope).float()      # noqa: E731
             wq = rot(y[:, :m.q_channels], m.heads).reshape(n, -1)
             wk = rot(y[:, m.q_channels:m.q_channels + m.k_channels], m.kv_heads).reshape(n, m.kv_heads, -1)
             wv = y[:, -m.v_channels:].reshape(n, m.kv_heads, m.vdim)

@@ -222,14 +222,14 @@ def test_latent_prep(dtype):
     pos = [0, 1, 2, 63, 64, 1000, 5000] * 3
     slots = [64 + 3 * i for i in range(T)]
     slots[4] = -1
-    f = torch.tensor([m.rope_base ** (-2.0 * i / m.rot_dim) for i in range(m.rot_dim // 2)])
+    f = torch.tensor(R.scaled_frequencies(m.rope))
     cache = torch.zeros(4, 64, 48, dtype=dtype, device=dev())
     slab, qa = torch.zeros(3, 32, 24, dtype=dtype, device=dev()), torch.zeros(T, 3, 48, dtype=dtype, device=dev())
     lat = torch.zeros(T, m.kv_rank, dtype=dtype, device=dev())
     K.latent_prep(a.to(dev(), dtype), 8, 200, 3, 20, 12, w.to(dev()), f.to(dev()), i32(pos), i32(slots), cache, slab, qa, eps, lat_out=lat)
     q = a[:, 8:8 + 96].view(T, 3, 32)
     c = R.rms(a[:, 200:236], eps) * w
-    kr = R.rotate_half(a[:, 236:248], torch.tensor(pos), m.rope_base)
+    kr = R.rotate(a[:, 236:248], torch.tensor(pos), m.rope)
     got = cache.view(-1, 48).float().cpu()
     for t in range(T):
         if slots[t] >= 0:
@@ -237,7 +237,7 @@ def test_latent_prep(dtype):
     assert got[0].abs().max() == 0
     close(lat, c, dtype)
     close(slab[:, :T, :20].transpose(0, 1), q[..., :20], dtype)
-    close(qa[..., 36:], R.rotate_half(q[..., 20:], torch.tensor(pos), m.rope_base), dtype)
+    close(qa[..., 36:], R.rotate(q[..., 20:], torch.tensor(pos), m.rope), dtype)
 
 
 def _delta_layer(m, seed=0):
