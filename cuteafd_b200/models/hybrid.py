@@ -597,7 +597,7 @@ class HybridEngine:
             else:
                 K.latent_attn(lw.q_abs[:T], cache, m.kv_rank, m.rot_dim, b.page_table, b.positions, b.q_start, o_slab, m.scale, m.window)
             K.grouped_linear(o_slab.view(-1, rp), L.w_uv, attn, ht.tile_expert, ht.tile_row0, ht.num_tiles, ht.max_tiles, ht.tile_rows,
-                             row_dst=ht.row_dst, ldo=vp, split_k=False)
+                             row_dst=ht.row_out, ldo=vp, split_k=False)
             self.launches += 3
         if out is not None:
             return

@@ -160,8 +160,8 @@ class LatentCache:
 
 
 class _HeadTiles:
-    """Tile table that lets the grouped GEMM treat heads as experts over a head-major slab [heads, t_pad, *].  ``out_heads``: a token's
-    output rows are that many heads apart (0 = ``heads``)."""
+    """Tile table that lets the grouped GEMM treat heads as experts over a head-major slab [heads, t_pad, *].  ``row_out`` is
+    ``row_dst`` for outputs whose tokens are ``out_heads`` heads apart (0 = ``heads``)."""
 
     def __init__(self, T: int, heads: int, device: torch.device, out_heads: int = 0):
         self.tile_rows = 16 if T <= 16 else 32 if T <= 32 else 64 if T <= 64 else 128
@@ -174,8 +174,9 @@ class _HeadTiles:
         self.max_tiles = heads * per_head
         self.num_tiles = torch.tensor([self.max_tiles], **i32)
         t = torch.arange(self.t_pad, **i32)
-        dst = t[None, :] * (out_heads or heads) + h[:, None]
-        self.row_dst = torch.where(t[None, :] < T, dst, torch.full_like(dst, -1)).reshape(-1).contiguous()
+        rows = lambda n: torch.where(t[None, :] < T, t[None, :] * n + h[:, None], -1).to(torch.int32).reshape(-1).contiguous()      # noqa: E731
+        self.row_dst = rows(heads)
+        self.row_out = self.row_dst if out_heads in (0, heads) else rows(out_heads)
 
 
 class MlaMoeEngine(GqaMoeEngine):
