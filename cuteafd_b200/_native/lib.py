@@ -81,7 +81,7 @@ class NormArgs(C.Structure):
     _fields_ = [(n, C.c_void_p) for n in ("tokens", "embed", "x_in", "y", "slot_w", "slot_idx", "ident", "w_b", "w", "base", "step",
                                           "w2", "h2_out", "conv", "x_out", "h_out", "row_idx", "state", "state_in", "state_out", "q_start")]
     _fields_ += [("slot_stride", C.c_longlong), ("state_off", C.c_longlong)]
-    _fields_ += [(n, C.c_int) for n in ("T", "H", "S", "ldy", "ldh", "ldb", "groups", "taps", "top_k", "n_experts", "vocab", "run")]
+    _fields_ += [(n, C.c_int) for n in ("T", "H", "S", "ldy", "ldh", "ldb", "ldi", "groups", "taps", "top_k", "n_experts", "vocab", "run")]
     _fields_ += [(n, C.c_float) for n in ("eps", "w_off", "e_scale")]
 
 

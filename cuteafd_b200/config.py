@@ -546,9 +546,44 @@ def guberax_bench_gqa(size: str = "base") -> ModelConfig:
                        top_k=0, num_shared_experts=0)
 
 
+# Benchmark sizes: width, layer runs, heads, key / value heads, expert width (heads of 128, latent 512 + 64)
+ROFAPEL_SIZES = {"small": (1024, 24, 8, 4, 512), "base": (2048, 24, 16, 8, 1024), "large": (4096, 12, 32, 8, 1536)}
+
+
+def rofapel_bench(size: str = "base") -> ModelConfig:
+    """A Rofapel-shaped stack at the sizes of a real model's layers: latent, windowed (values out of keys) and plain attention in
+    turn, each beside 64 routed experts (top 6) and a shared one; a quarter of the layer runs are second passes."""
+    width, runs, heads, kv_heads, ffn = ROFAPEL_SIZES[size]
+    lat = LatentSpec(heads=heads, dim=128, rot_dim=64, vdim=128, kv_rank=512, window=0, scale=192 ** -0.5,
+                     rope=RopeSpec(64, 1.0e6, 8.0, 1.0, 32.0, 4096, "yarn"), gate=False)
+    att = AttentionSpec(heads=heads, kv_heads=kv_heads, dim=128, vdim=128, window=0, keep_first=0, scale=128 ** -0.5,
+                        rope=RopeSpec(128, 1.0e6, halves=True), qk_norm="all", gate=True)
+    win = AttentionSpec(heads=heads, kv_heads=kv_heads, dim=128, vdim=128, window=2048, keep_first=0, scale=128 ** -0.5,
+                        rope=RopeSpec(64, 1.0e4, 4.0, kind="linear", halves=True), conv=4, qk_norm="head", v_from_k=True, sink=True, gate=True)
+    r = RouterSpec(experts=64, ffn=ffn, top=6, logit_bias=True, normalize=True)
+    once = runs - runs // 4
+    start = (once - runs // 4) // 2
+    specs = [LayerSpec((lat, win, att)[i % 3], r, DenseSpec(ffn), parallel=True, two_norms=True) for i in range(once)]
+    return parallel_config(f"rofapel-{size}", 65536, width, specs, eps=1e-5, loop=(start, start + runs // 4, 2), family="rofapel",
+                           loop_join=True, embed_scale=width ** 0.5)
+
+
+def rofapel_bench_gqa(size: str = "base") -> ModelConfig:
+    """The GQA + MoE decoder at the size of ``rofapel_bench``: as many layer runs of the same width, heads, experts and shared
+    expert, per-head norms of queries and keys, the same window on the layers that have one there."""
+    width, runs, heads, kv_heads, ffn = ROFAPEL_SIZES[size]
+    a = rofapel_bench(size)
+    return ModelConfig(name=f"gqa-moe-{size}", family="qwen3_moe", vocab_size=65536, num_layers=runs, hidden=width, attention="gqa",
+                       num_heads=heads, num_kv_heads=kv_heads, head_dim=128, qk_norm=True, sliding_window=2048,
+                       window_layers=tuple(int(a.window_of(r.layer) > 0) for r in a.layer_runs), rope_theta=1.0e6, rope_interleaved=False,
+                       rms_eps=1e-5, dense_ffn=0, first_dense_layers=0, num_experts=64, expert_ffn=ffn, top_k=6, scoring="softmax",
+                       num_shared_experts=1, norm_topk_prob=True)
+
+
 PRESETS = {
     "karusun-base": karusun_bench,
     "guberax-base": guberax_bench,
+    "rofapel-base": rofapel_bench,
     "tiny-moe": tiny_moe,
     "mixtral-8x7b": mixtral_8x7b,
     "mistral-7b": mistral_7b,

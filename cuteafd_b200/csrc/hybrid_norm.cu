@@ -26,6 +26,7 @@ extern "C" int cafd_norm_conv(const NormArgs* args, int is_f32, cafd_stream_t s)
   NormArgs a = *args;
   if (a.T <= 0) return 0;
   if (a.H <= 0 || a.groups <= 0 || a.H % a.groups || (a.conv && (a.taps < 1 || a.taps > 16)) || !a.h_out || a.ldh < a.H || a.ldh % 8) return -10;
+  if (a.slot_w && (!a.ident || a.ldi < a.H || a.ldi % 8)) return -10;
   if ((!a.w && (a.conv || a.w2)) || (a.w2 && (!a.h2_out || a.conv)) || (a.base && (!a.slot_w || a.ldb < a.H || a.ldb % 8))) return -10;
   if (a.y && (a.ldy < a.H || a.ldy % 8)) return -10;
   if (a.conv && (a.row_idx || !a.q_start || a.S < 1 || (a.taps > 1 && (!a.state || !a.state_in || !a.state_out)))) return -10;

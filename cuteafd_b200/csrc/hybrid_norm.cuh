@@ -29,7 +29,7 @@ struct NormArgs {
   const void* y;              // [T, ldy] E, or the slot rows [T * top_k, ldy] E with slot_w; null = nothing to add
   const float* slot_w;        // [T, top_k]
   const int* slot_idx;        // [T, top_k]; an index >= n_experts is an identity slot
-  const void* ident;          // [T, ldh] E: what identity slots hand through
+  const void* ident;          // [T, ldi] E: what identity slots hand through
   const void* w_b;            // [H] E, null = y is added as it is
   const void* w;              // [H] E, null = the rows leave as they are, without a norm
   const void* base;           // [T, ldb] E, null = none; only with slot_w
@@ -45,7 +45,7 @@ struct NormArgs {
   const int* state_out;       // [S] slot written
   const int* q_start;         // [S + 1]
   long long slot_stride, state_off;
-  int T, H, S, ldy, ldh, ldb, groups, taps, top_k, n_experts, vocab, run;   // ldy, ldh, ldb: elements from row to row of y, of h_out and ident, of base
+  int T, H, S, ldy, ldh, ldb, ldi, groups, taps, top_k, n_experts, vocab, run;   // ldy, ldh, ldb, ldi: elements from row to row of y, of h_out, of base, of ident
   float eps, w_off, e_scale;
 };
 
@@ -342,7 +342,7 @@ __global__ void __launch_bounds__(kMaxThreads, kMinBlocks) norm_conv_kernel(cons
 #pragma unroll
             for (int j = 0; j < kSlotBatch; ++j)
               if (s0 + j < a.top_k)
-                raw[j] = load_packed<E, V>((src[j] < 0 ? static_cast<const E*>(a.ident) + static_cast<size_t>(row) * a.ldh
+                raw[j] = load_packed<E, V>((src[j] < 0 ? static_cast<const E*>(a.ident) + static_cast<size_t>(row) * a.ldi
                                                        : static_cast<const E*>(a.y) + static_cast<size_t>(src[j]) * a.ldy) + i * V);
 #pragma unroll
             for (int j = 0; j < kSlotBatch; ++j) {

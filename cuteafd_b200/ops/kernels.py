@@ -726,8 +726,8 @@ def norm_conv(h_out: torch.Tensor, w: torch.Tensor | None, groups: int, eps: flo
     assert h2_out is None or (h2_out.stride(0) == a.ldh and h2_out.dtype == h_out.dtype)
     if slots is not None:
         sw, si, n, ident = slots
-        a.slot_w, a.slot_idx, a.n_experts, a.ident, a.top_k = sw.data_ptr(), si.data_ptr(), n, ident.data_ptr(), sw.shape[1]
-        assert ident.stride(0) == a.ldh and sw.is_contiguous() and si.is_contiguous()
+        a.slot_w, a.slot_idx, a.n_experts, a.ident, a.top_k, a.ldi = sw.data_ptr(), si.data_ptr(), n, ident.data_ptr(), sw.shape[1], ident.stride(0)
+        assert ident.dtype == h_out.dtype and sw.is_contiguous() and si.is_contiguous()
     if conv is not None:
         a.taps, a.S = conv.shape[0], q_start.shape[0] - 1
         a.state, a.state_in, a.state_out, a.q_start = state.data_ptr(), state_in.data_ptr(), state_out.data_ptr(), q_start.data_ptr()

@@ -62,7 +62,7 @@ def workspace_bytes(cfg: ModelConfig, rows: int) -> int:
         attn = max((s.mixer.heads * (2 * s.mixer.record + s.mixer.dim + s.mixer.rot_dim + 3 * s.mixer.vdim) + s.mixer.record)
                    if hasattr(s.mixer, "kv_rank") else (s.mixer.conv_channels + s.mixer.q_channels + s.mixer.heads * s.mixer.vdim)
                    if hasattr(s.mixer, "rope") else (s.mixer.conv_channels + 2 * s.mixer.heads * s.mixer.vdim) for s in cfg.layer_specs)
-        h *= 2                                   # the residual is fp32 and alternates between two buffers
+        h *= 2 + 2 * bool(cfg.loop and cfg.loop_join)      # the residual is fp32 and alternates between two buffers; joining rows and what they give
     elif cfg.is_mla:
         attn = (cfg.q_lora_rank + cfg.kv_lora_rank + cfg.qk_rope_dim) + cfg.num_heads * (cfg.qk_head_dim + cfg.v_head_dim + cfg.kv_lora_rank + cfg.qk_rope_dim)
     else:

@@ -95,7 +95,7 @@ def render(rep: PlanReport) -> str:
             if c.is_mla else ", ".join(f"{n} {k}" for k, n in sorted(Counter(
                 f"latent (rank {m.kv_rank} + {m.rot_dim}, {m.heads} heads, window {m.window})" if hasattr(m, "kv_rank")
                 else (f"{'differential ' if m.maps == 2 else ''}attention ({m.heads}/{m.kv_heads} heads x {m.dim} + {m.vdim}, window {m.window}"
-                      f", keeps {m.keep_first})") if hasattr(m, "rope")
+                      f", keeps {m.keep_first}{', values out of keys' if m.v_from_k else ''})") if hasattr(m, "rope")
                 else f"delta ({m.heads} heads x {m.dim} x {m.vdim})" for m in (s.mixer for s in c.layer_specs)).items()))
             + (f", layers {c.loop[0]} to {c.loop[1] - 1} looped {c.loop[2]} times" if c.loop else "")
             if c.is_hybrid else f"GQA {c.num_heads}/{c.num_kv_heads} heads x {c.head_dim}"),

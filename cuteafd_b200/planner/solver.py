@@ -147,6 +147,11 @@ def component_bytes(cfg: ModelConfig, req: PlacementRequest) -> dict[str, int]:
         "mtp": cfg.mtp_layers * (weight_bytes(cfg.attention_params() + 2 * cfg.hidden * cfg.hidden, bfmt)
                                  + cfg.num_experts * weight_bytes(cfg.expert_params(), efmt)),
     }
+    if cfg.is_hybrid:                            # per-layer sizes
+        dense = [(s.router is not None, 3 * cfg.hidden * s.dense.ffn) for s in cfg.layer_specs if s.dense is not None]
+        join = (2 * cfg.hidden + cfg.loop[2]) * cfg.hidden if cfg.loop and cfg.loop_join else 0
+        out["dense_ffn"] = weight_bytes(sum(n for routed, n in dense if not routed) + join, bfmt)
+        out["shared_experts"] = weight_bytes(sum(n for routed, n in dense if routed), bfmt)
     return out
 
 

@@ -92,14 +92,69 @@ def single_map_config():
         parallel(one(attention(3, 1, 20, 12, 50, 66, RopeSpec(20, 1e3), 2)), 40)], 1e-5, loop=(1, 2, 2))
 
 
+def normed(heads=5, kv_heads=1, dim=14, vdim=7, rope=RopeSpec(10, 1e4, halves=True), window=0, scale=None):
+    """Attention with norms over the whole projections and a gate per head."""
+    return AttentionSpec(heads, kv_heads, dim, vdim, window, 0, scale if scale is not None else 1.6 * dim ** -0.5, rope, qk_norm="all", gate=True)
+
+
+def key_valued(heads=6, kv_heads=2, dim=20, window=37, rope=RopeSpec(12, 5000.0, 3.0, kind="linear", halves=True), conv=3, scale=None):
+    """Attention whose values are the convolved keys, norms per head, sinks and a gate per head."""
+    return AttentionSpec(heads, kv_heads, dim, dim, window, 0, scale if scale is not None else 1.3 * dim ** -0.5, rope, conv, qk_norm="head",
+                         v_from_k=True, sink=True, gate=True)
+
+
+def open_latent(heads=3, dim=24, rot_dim=12, vdim=20, kv_rank=40, rope=None, window=0, scale=None):
+    """Latent attention without a window or a gate, neighbouring pairs, YaRN scaling."""
+    return LatentSpec(heads, dim, rot_dim, vdim, kv_rank, window, scale if scale is not None else 1.7 * (dim + rot_dim) ** -0.5,
+                      rope or RopeSpec(rot_dim, 300.0, 5.0, 1.5, 24.0, 700, "yarn"), gate=False)
+
+
+def two_norms(m, ffn=None, experts=0, top=0, expert_ffn=0):
+    r = RouterSpec(experts, expert_ffn, top, logit_bias=True, normalize=True) if experts else None
+    return LayerSpec(m, r, DenseSpec(ffn) if ffn else None, parallel=True, two_norms=True)
+
+
+def joined_config():
+    """Every layer differs: routed with a shared expert and without, dense, none; odd head sizes, a window of one token; three
+    passes that each start with a product of [x; embedding row]."""
+    return parallel_config("joined", 203, 104, [
+        two_norms(key_valued(), 26, 6, 3, 28),
+        two_norms(open_latent(), 72),
+        two_norms(key_valued(3, 3, 8, 1, RopeSpec(8, 300.0, halves=True), 1), 0, 5, 1, 16),
+        two_norms(normed()),
+        two_norms(open_latent(5, 16, 8, 24, 64, RopeSpec(8, 1e4, 2.0, 0.5, 8.0, 100, "yarn")), 33, 9, 9, 8),
+        two_norms(normed(4, 4, 16, 24, RopeSpec(16, 700.0, halves=True)), 40)], 2e-5, loop=(1, 4, 3), family="rofapel", loop_join=True, embed_scale=5.0)
+
+
+def lone_config():
+    """Values that make a mechanism vanish: one head, one expert, one tap, one pass (over everything), no rotation, scales of one, a
+    width that is no multiple of 8."""
+    return parallel_config("lone", 77, 90, [
+        two_norms(key_valued(1, 1, 10, 64, RopeSpec(0, 1e3, kind="linear", halves=True), 1, 1.0), 11, 1, 1, 9),
+        two_norms(open_latent(1, 8, 4, 8, 12, RopeSpec(4, 1e3)), 24),
+        two_norms(normed(1, 1, 6, 5, RopeSpec(6, 1e2, halves=True), 65), 7, 3, 2, 10)], 1e-3, loop=(0, 3, 1), family="rofapel", loop_join=True)
+
+
+def joint_config(window=100):
+    """The sizes the tensor-core kernels take; the first two layers run twice."""
+    return parallel_config("joint", 500, 256, [
+        two_norms(open_latent(8, 128, 64, 128, 512, RopeSpec(64, 1e5, 4.0, 1.0, 32.0, 256, "yarn"), scale=0.1), 192, 8, 2, 128),
+        two_norms(key_valued(4, 2, 128, window, RopeSpec(64, 1e4, 2.0, kind="linear", halves=True), 4), 136),
+        two_norms(normed(8, 1, 128, 128, RopeSpec(128, 1e5, halves=True)), 128, 6, 3, 64)], 1e-5, loop=(0, 2, 2), family="rofapel", loop_join=True,
+        embed_scale=16.0)
+
+
 def params(cfg, seed=0, spread=0.4):
     """Random bf16-representable weights.  The selection correction is spread out by ``spread``: above 1 the choice is the
-    correction's alone, so that 16-bit rounding cannot flip a close one."""
+    correction's alone, so that 16-bit rounding cannot flip a close one; a bias that is part of the logits likewise."""
     p = R.init_hybrid_weights(cfg, seed)
     g = torch.Generator().manual_seed(seed + 99)
     for k in p:
         if k.endswith(".correction"):
             p[k] = (torch.randperm(p[k].numel(), generator=g).float() - p[k].numel() / 2) * spread
+        elif k.endswith(".router.b") and spread > 1:
+            p[k] = (torch.randperm(p[k].numel(), generator=g).float() - p[k].numel() / 2) * 0.3
+            p[k[:-2]] = p[k[:-2]] * 0.02
         elif k.endswith(".A_log"):
             p[k] = p[k] - 1.0
     return R.bf16_params(p)

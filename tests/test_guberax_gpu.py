@@ -1,6 +1,6 @@
-"""Stacks of parallel layers (differential attention beside a dense feed-forward, looped layers) on the GPU against the plain
-oracle: every kernel alone, then the engine through its serving backend (greedy generation through the scheduler is with the
-other per-layer designs' in test_hybrid_gpu.py)."""
+"""Stacks of parallel layers on the GPU against the plain oracle: the kernels of differential attention alone (those of the two-norm
+design are in test_rofapel_gpu.py), then the engine through its serving backend, both designs (greedy generation through the
+scheduler is with the other per-layer designs' in test_hybrid_gpu.py)."""
 import dataclasses
 import json
 import os
@@ -13,8 +13,9 @@ import torch
 from cuteafd_b200.config import RopeSpec
 from cuteafd_b200.ref import hybrid as R
 
-from tests.hybrid_common import attention, bare_config, err, looped_config, oracle_logits, paired_config, params, single_map_config, tokens, write_model
-from tests.test_hybrid_gpu import DTYPES, backend, check, close, dev, i32, rnd, run_cut
+from tests.hybrid_common import (attention, bare_config, err, joined_config, joint_config, lone_config, looped_config, oracle_logits, paired_config,
+                                 params, single_map_config, tokens, write_model)
+from tests.test_hybrid_gpu import DTYPES, SPREAD, backend, check, close, dev, i32, rnd, run_cut
 
 pytestmark = pytest.mark.gpu
 
@@ -226,13 +227,14 @@ def test_softcap():
 
 
 # ---- engine ------------------------------------------------------------------------------------------------------------
-CASES = [(c, d) for c in (looped_config(), bare_config(), paired_config(), single_map_config()) for d in ("f32", "bf16")]
+CASES = [(c, d) for c in (looped_config(), bare_config(), paired_config(), single_map_config(), joined_config(), lone_config(), joint_config())
+         for d in ("f32", "bf16")]
 IDS = [f"{c.name}-{d}" for c, d in CASES]
 
 
 @pytest.mark.parametrize("cfg,dtype", CASES, ids=IDS)
 def test_prompts_portions_and_decoding(cfg, dtype):
-    p, toks = params(cfg), tokens(333, cfg.vocab_size, 5)
+    p, toks = params(cfg, spread=SPREAD[dtype]), tokens(333, cfg.vocab_size, 5)
     want = oracle_logits(cfg, p, toks)
     be = backend(cfg, p, dtype)
     for cuts in ([333], [300] + [1] * 33, [2], [3, 61, 1, 64, 17], [63, 2], [128, 5]):
@@ -242,8 +244,8 @@ def test_prompts_portions_and_decoding(cfg, dtype):
 
 @pytest.mark.parametrize("cfg,dtype", CASES, ids=IDS)
 def test_residual_after_every_layer_run(cfg, dtype):
-    """Layer by layer, one short prompt; a run's residual is what the oracle has before the next pass adds the embedding."""
-    p, toks = params(cfg), tokens(41, cfg.vocab_size, 8)
+    """Layer by layer, one short prompt; a run's residual is what the oracle has before the next pass starts."""
+    p, toks = params(cfg, spread=SPREAD[dtype]), tokens(41, cfg.vocab_size, 8)
     m = R.HybridRefDecoder(cfg, p, mark_rows=0)
     m.trace = []
     with torch.no_grad():
@@ -256,11 +258,11 @@ def test_residual_after_every_layer_run(cfg, dtype):
         close(a, b, torch.float32 if dtype == "f32" else torch.bfloat16, 2.0)
 
 
-@pytest.mark.parametrize("cfg", [looped_config(), paired_config()], ids=lambda c: c.name)
+@pytest.mark.parametrize("cfg", [looped_config(), paired_config(), joined_config(), joint_config()], ids=lambda c: c.name)
 def test_decode_steps_match_prompt_steps(cfg):
     """The decode form (its own attention kernel, drafts as rows of one step) against prompt portions of the same tokens."""
-    dtype = "f32" if cfg.name == "looped" else "bf16"
-    p, seqs = params(cfg), [tokens(n, cfg.vocab_size, n) for n in (230, 66, 131)]
+    dtype = "f32" if cfg.name in ("looped", "joined") else "bf16"
+    p, seqs = params(cfg, spread=SPREAD[dtype]), [tokens(n, cfg.vocab_size, n) for n in (230, 66, 131)]
     want = [oracle_logits(cfg, p, t) for t in seqs]
     for rows in ([1, 1, 1], [4, 1, 3]):
         be = backend(cfg, p, dtype, pages=60, slots=20)
@@ -283,7 +285,7 @@ def test_decode_steps_match_prompt_steps(cfg):
 def test_mixed_batches_reuse_pages_and_slots(cfg, dtype):
     """Four live requests of unequal lengths, portions beside single tokens, in pools that only just hold them; every
     finished request's pages and slots serve the next."""
-    p = params(cfg)
+    p = params(cfg, spread=SPREAD[dtype])
     reqs = [tokens(n, cfg.vocab_size, 10 + i) for i, n in enumerate([150, 1, 90, 64, 65, 3, 128, 127, 2, 77])]
     want = [oracle_logits(cfg, p, t) for t in reqs]
     be = backend(cfg, p, dtype, pages=1 + 3 + 2 + 2 + 2, slots=2 + 8)
@@ -312,9 +314,9 @@ def test_mixed_batches_reuse_pages_and_slots(cfg, dtype):
     check(torch.cat([torch.cat(x) for x in got]), torch.cat(want), dtype)
 
 
-def test_a_row_does_not_depend_on_the_cut_or_the_batch():
+@pytest.mark.parametrize("cfg", [looped_config(), joined_config()], ids=lambda c: c.name)
+def test_a_row_does_not_depend_on_the_cut_or_the_batch(cfg):
     """32-bit: the same row computed in other portions and beside other requests differs by rounding alone."""
-    cfg = looped_config()
     p = params(cfg)
     be = backend(cfg, p)
     a, b = tokens(200, cfg.vocab_size, 1), tokens(130, cfg.vocab_size, 2)
@@ -327,8 +329,8 @@ def test_a_row_does_not_depend_on_the_cut_or_the_batch():
     assert err(torch.cat(got), alone).max() < 2e-6
 
 
-def test_long_decoding_and_large_steps():
-    cfg = bare_config()
+@pytest.mark.parametrize("cfg", [bare_config(), lone_config()], ids=lambda c: c.name)
+def test_long_decoding_and_large_steps(cfg):
     p, toks = params(cfg), tokens(900, cfg.vocab_size, 3)
     want = oracle_logits(cfg, p, toks)
     be = backend(cfg, p)
@@ -360,11 +362,12 @@ def test_far_keys_and_kept_tokens_in_the_engine(name):
             assert other[150:].median() > 20 * e[150:].median()
 
 
-@pytest.mark.parametrize("cfg,dtype", [(looped_config(), "f32"), (paired_config(), "bf16")], ids=["looped", "paired"])
+@pytest.mark.parametrize("cfg,dtype", [(looped_config(), "f32"), (paired_config(), "bf16"), (joined_config(), "f32"), (joint_config(), "bf16")],
+                         ids=["looped", "paired", "joined", "joint"])
 def test_generator_and_device_loop(cfg, dtype):
     """Greedy generation under decode graphs, and the device-resident decode loop that benchmarks time."""
     from cuteafd_b200.runtime.generate import Generator
-    p = params(cfg)
+    p = params(cfg, spread=SPREAD[dtype])
     be = backend(cfg, p, dtype, slots=20)
     gen = Generator(be.engine, be.pool, 20, 4, prefill_chunk=64, use_graphs=True)
     prompts = [tokens(100, cfg.vocab_size, 1), tokens(9, cfg.vocab_size, 2)]
@@ -383,14 +386,14 @@ def test_generator_and_device_loop(cfg, dtype):
         assert (best - want[torch.arange(12), o] < 0.06 * best.abs() + 1e-6).all()
 
 
-def test_serve_builds_over_a_snapshot(tmp_path):
+@pytest.mark.parametrize("cfg", [paired_config(), joint_config()], ids=lambda c: c.name)
+def test_serve_builds_over_a_snapshot(tmp_path, cfg):
     """``serve --snapshot``: loading, page and slot pools, scheduler with the n-gram drafter, decode graphs, sampling."""
     from cuteafd_b200.cli import build_parser
     from cuteafd_b200.runtime.sampling import SamplingParams
     from cuteafd_b200.runtime.scheduler import Request, collect
     from cuteafd_b200.serve.server import build_state
-    cfg = paired_config()
-    p = params(cfg, 3)
+    p = params(cfg, 3, spread=2.0)
     path = write_model(cfg, p, str(tmp_path / "m"))
     st = build_state(build_parser().parse_args(["serve", "--snapshot", path, "--max-context-tokens", "512", "--concurrency", "3",
                                                 "--speculator", "ngram"]))
@@ -410,11 +413,10 @@ def test_serve_builds_over_a_snapshot(tmp_path):
     assert len(a) == 24 and a[0] == b[0]
 
 
-@pytest.mark.parametrize("name", ["looped", "paired"])
+@pytest.mark.parametrize("cfg", [looped_config(), paired_config(), joined_config(), joint_config()], ids=lambda c: c.name)
 @pytest.mark.parametrize("dtype", ["bfloat16", "float32"])
-def test_trace_replay_program(dtype, name, tmp_path):
-    cfg = looped_config() if name == "looped" else paired_config()
-    p = params(cfg)
+def test_trace_replay_program(dtype, cfg, tmp_path):
+    p = params(cfg, spread=2.0)
     d = write_model(cfg, p, str(tmp_path / "m"))
     a, b = tokens(120, cfg.vocab_size, 1), tokens(30, cfg.vocab_size, 2)
     steps = [{"entries": [{"id": "a", "tokens": a[:50], "want": [49, 0]}, {"id": "b", "tokens": b[:2], "want": []}], "end": []},
