@@ -445,6 +445,91 @@ def bench_parallel(a, dev, pk) -> None:
     assert K.read_status() == 0
 
 
+def bench_two_norm(a, dev, pk) -> None:
+    """The kernels of two-norm parallel layers (norms over heads or projections, values out of keys, sinks, head gates, scaled latent
+    rotation, joined passes) beside the like kernels of the GQA + MoE and MLA decoders, at one of the benchmark sizes."""
+    from ..config import ROFAPEL_SIZES, rofapel_bench
+    from ..models.hybrid import rope_frequencies
+    H, _, heads, kvh, ffn = ROFAPEL_SIZES[a.size]
+    cfg, bf, T, top, E = rofapel_bench(a.size), torch.bfloat16, a.tokens, 6, 64
+    lat, win, att = (s.mixer for s in cfg.layer_specs[:3])
+
+    def i32(v):
+        return torch.tensor(list(v), dtype=torch.int32, device=dev)
+
+    def rand(*s):
+        return torch.randn(*s, device=dev, dtype=bf)
+
+    def run(name, fn, nbytes, flops=0.0):
+        report(name, time_eager(fn, dev, a.iters), flops, nbytes, pk)
+    w = torch.zeros(H, device=dev, dtype=bf)
+    for n in (1, 8, 32, T):
+        S = n if n < T else 1
+        x, xo, y, yo, h, h2, ys = torch.randn(n, H, device=dev), torch.empty(n, H, device=dev), *(rand(n, H) for _ in range(4)), rand(n * top, H)
+        idx, sw = torch.randint(0, E, (n, top), device=dev, dtype=torch.int32), torch.rand(n, top, device=dev)
+        run(f"norm_conv, two outputs, routed + plain rows, {n} rows",
+            lambda: K.norm_conv(h, w, 1, 1e-5, x_in=x, y=ys, base=y, slots=(sw, idx, E, h2), x_out=xo, w_offset=1.0, w2=w, h2_out=h2), n * H * (14 + 2 * top))
+        run(f"(GQA) combine + norm {n} rows", lambda: K.moe_combine(ys, sw, h, shared=y, residual=h2, norm_w=w, eps=1e-5, x_out=yo), n * H * (8 + 2 * top))
+        both, wj = rand(n, 2 * H), rand(H, 2 * H)
+        run(f"norm_conv, rows of a join, {n} rows", lambda: K.norm_conv(both, None, 1, 1e-5, x_in=x, y=ys, base=y, slots=(sw, idx, E, h2)), n * H * (8 + 2 * top))
+        run(f"join product, fp32 out, {n} rows", lambda: K.linear(both, wj, out=xo, out_f32=True), 4 * H * H + n * H * 8, 4.0 * n * H * H)
+        run(f"(GQA) a product of the same size {n} rows", lambda: K.linear(both, wj, out=h), 4 * H * H + n * H * 6, 4.0 * n * H * H)
+        rw, rb, z = rand(E, H), torch.zeros(E, device=dev), torch.empty(n, E, device=dev)
+        i_, w_ = torch.empty(n, top, dtype=torch.int32, device=dev), torch.empty(n, top, device=dev)
+        for tag, kw in (("", dict(scoring="softmax_bias", bias=rb)), ("(GQA) ", dict(scoring="softmax"))):
+            if n <= 64:
+                run(f"{tag}norm_route {n} rows", lambda: K.norm_route(h, None, 0.0, rw, None, i_, w_, top, **kw), E * H * 2 + n * H * 2)
+            else:
+                run(f"{tag}route_topk {n} rows", lambda: K.route_topk(z, top, out_idx=i_, out_w=w_, **kw), n * E * 4 + n * top * 8)
+        ctx, pps = T, (T + 63) // 64
+        kc, vc = rand(S * pps + 1, kvh, 64, 128), rand(S * pps + 1, kvh, 64, 128)
+        table = (torch.arange(S * pps, dtype=torch.int32, device=dev) + 1).view(S, pps).contiguous()
+        pos = i32([ctx - 1] * S) if n < T else i32(range(T))
+        slots = (table[:, -1] * 64 + 63).int() if n < T else i32(range(64, 64 + T))
+        qs, sl = (i32(range(S + 1)), i32([ctx] * S)) if n < T else (i32([0, T]), i32([T]))
+        q, gate = rand(n, heads, 128), rand(n, heads + 8)[:, :heads]
+        n1, f64, tab = torch.ones(heads * 128, device=dev), torch.ones(64, device=dev), torch.empty(n, 64, 2, device=dev)
+        nb = torch.ones(128, device=dev, dtype=bf)
+        si, so, st = i32(range(2, 2 + S)), i32(range(2 + S, 2 + 2 * S)), torch.zeros(2 + 2 * S, 3 * win.conv_channels, device=dev)
+        C = att.conv_channels
+        proj = rand(n, C + 8 * (1 + heads // 8))
+        for tag, m in (("norms per head, convolution, values out of keys", win), ("norms over the projection", att)):
+            offs = dict(q=0, k=m.q_channels, v=m.q_channels + m.k_channels)
+            K.rope_table(pos, rope_frequencies(m.rope).to(dev), tab.view(-1)[:n * m.rope.dims])
+            cw = torch.randn(m.conv, m.conv_channels, device=dev) if m.conv else None
+            nq, nk = (n1[:128], n1[:128]) if m.qk_norm == "head" else (n1, n1[:m.k_channels])
+            run(f"conv_norm_rope_kv, {tag}, {n} rows",
+                lambda: K.conv_rope_kv(proj, offs, m, cw, tab, slots, q, kc, vc, state=st, state_in=si, state_out=so, q_start=qs, q_norm=nq, k_norm=nk, eps=1e-5),
+                n * (m.conv_channels + C) * 2 + (S * m.conv_channels * 24 if m.conv else 0))
+        qkv = rand(n, C)
+        run(f"(GQA) qk_rope_kv with norms {n} rows", lambda: K.qk_rope_kv(qkv, nb, nb, f64, pos, slots, q, kc, vc, heads, kvh, 128, 1e-5, False), n * C * 4)
+        out, wide = rand(n, heads, 128), rand(n, heads * 128 + ffn)
+        sink = torch.zeros(heads, device=dev)
+        for tag, kw, o in (("sinks and gates, ", dict(sink=sink, gate=gate), wide), ("(GQA) ", {}, out)):
+            for wn in (win.window, 0):
+                if n == T:
+                    pairs = T * wn - wn * wn / 2 if wn else T * T / 2
+                    run(f"attn_prefill, {tag}{T} tokens, window {wn}", lambda: K.attn_prefill(q, kc, vc, table, sl, qs, o, T, window=wn, **kw), T * C * 4, pairs * heads * 512)
+                else:
+                    sp = K.attn_decode_splits(S, 1, kvh, pps, wn)
+                    sc = torch.empty(K.attn_decode_scratch_floats(S, 1, heads, kvh, sp), device=dev)
+                    run(f"attn_decode, {tag}{S} x {ctx}, window {wn}, {sp} splits", lambda: K.attn_decode(q, kc, vc, table, sl, qs, o, sc, 1, sp, window=wn, **kw),
+                        S * (wn or ctx) * kvh * 512)
+        if n < T:
+            continue
+        rec, kn, knb, fl = 576, torch.ones(512, device=dev), torch.ones(512, device=dev, dtype=bf), torch.ones(32, device=dev)
+        la, lq, lc, cache, qa = rand(n, heads * 192 + rec), rand(n, heads * 192), rand(n, rec), rand(S * pps + 1, 64, rec), rand(n, heads, rec)
+        lo, slab, kx, vx, z0 = rand(n, 512), rand(heads, n, 128), rand(n, heads * 128), rand(n, heads * 128), i32([0])
+        run(f"latent_prep {n} rows", lambda: K.latent_prep(la, 0, heads * 192, heads, 128, 64, kn, fl, pos, slots, cache, None, qa, 1e-5, lat_out=lo, halves=False,
+                                                           magnitude=1.2), n * (rec * 4 + 1024 + heads * 256))
+        run(f"(MLA) mla_prep_a {n} rows", lambda: K.mla_prep_a(lc, 0, None, knb, fl, pos, slots, None, cache, 1e-5, True, lat_out=lo), n * (rec * 4 + 1024))
+        run(f"(MLA) mla_q_split {n} rows", lambda: K.mla_q_split(lq, fl, pos, slab, qa, heads, True), n * heads * 192 * 4)
+        for tag, o in (("into longer rows, ", wide), ("(MLA) ", out)):
+            run(f"attn_prefill_mla, {tag}{n} tokens", lambda: K.attn_prefill_mla(lq, qa, kx, vx, z0, cache, table, sl, qs, o, n, heads, lat.scale),
+                n * heads * 192 * 4, n * n / 2 * heads * 2 * 320)
+    assert K.read_status() == 0
+
+
 def main() -> None:
     ap = argparse.ArgumentParser()
     sub = ap.add_subparsers(dest="cmd", required=True)
@@ -488,7 +573,9 @@ def main() -> None:
     hy.add_argument("--size", default="base", choices=["small", "base", "large"]); hy.add_argument("--tokens", type=int, default=8192)
     pa = sub.add_parser("parallel")
     pa.add_argument("--size", default="base", choices=["small", "base", "large"]); pa.add_argument("--tokens", type=int, default=8192)
-    for s in (g, p, d, m, ml, mp_, w4, sm, hy, pa):
+    tn = sub.add_parser("two-norm")
+    tn.add_argument("--size", default="base", choices=["small", "base", "large"]); tn.add_argument("--tokens", type=int, default=8192)
+    for s in (g, p, d, m, ml, mp_, w4, sm, hy, pa, tn):
         s.add_argument("--iters", type=int, default=10)
     a = ap.parse_args()
     dev = torch.device("cuda", int(os.environ.get("LOCAL_RANK", "0")))
@@ -496,7 +583,7 @@ def main() -> None:
     pk = peaks()
     {"exl3": bench_exl3, "gemm-fp8": bench_gemm_fp8, "indexer": bench_indexer, "gemm": bench_gemm, "attn-prefill": bench_attn_prefill, "attn-decode": bench_attn_decode, "moe": bench_moe,
      "mla": bench_mla, "mla-prefill": bench_mla_prefill_expanded, "w4": bench_w4, "sampler": bench_sampler, "hybrid": bench_hybrid,
-     "parallel": bench_parallel}[a.cmd](a, dev, pk)
+     "parallel": bench_parallel, "two-norm": bench_two_norm}[a.cmd](a, dev, pk)
 
 
 if __name__ == "__main__":

@@ -9,6 +9,8 @@
 //   conv_rope_kv_any the same for any head sizes and any number of taps: one channel per thread and token
 //   conv_norm_rope_kv  with norms (per head or over the whole projection), pairs of either kind, values of their own or the
 //                    convolved keys: a block walks a run of tokens, the projected rows in a ring in shared memory
+//   conv_norm_rope_128 the same for bf16 heads of 128: a warp owns whole heads, four channels per lane, and walks a run of tokens
+//                    with everything in registers; partners and square sums go by shuffles
 //
 // A sequence's last taps - 1 projected rows are fp32 in its state slot (oldest first, [taps - 1, channels]); a step reads one
 // slot and writes another.  An output is a function of its own taps inputs in a fixed order, so it does not depend on where a
@@ -257,6 +259,8 @@ template <typename E, int V>
 __global__ void __launch_bounds__(kCnrThreads) conv_norm_rope_kv_kernel(const ConvRope p) {
   extern __shared__ float4 sm4[];
   __shared__ float part[2][kCnrThreads / 32];
+  pdl_wait();
+  pdl_trigger();
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
   const int uq = p.nq / p.dim, uk = p.nk / p.dim, uv = p.nv / p.vdim, kmaps = p.maps_dim / p.dim;
   const int u0 = blockIdx.y * p.units, u1 = min(uq + uk + uv, u0 + p.units);
@@ -272,8 +276,6 @@ __global__ void __launch_bounds__(kCnrThreads) conv_norm_rope_kv_kernel(const Co
   const int vpu = p.dim / V;                                             // vectors of a head of q or k
   const bool lanes = p.norm && vpu <= 32 && (vpu & (vpu - 1)) == 0;
   const int half = p.rot >> 1;
-  pdl_wait();
-  pdl_trigger();
   const int r0 = blockIdx.x * p.run, r1 = min(p.T, r0 + p.run);
   auto fetch = [&](int row) {
     if (row < r1) {
@@ -443,6 +445,219 @@ __global__ void __launch_bounds__(kCnrThreads) conv_norm_rope_kv_kernel(const Co
   asm volatile("cp.async.wait_group 0;" ::: "memory");
 }
 
+// bf16, heads of 128 and up to four taps.  A warp owns NH heads of one kind (q, k or v), a lane the same four channels of each, so
+// weights, earlier inputs and the rows to come stay in registers.  kAll: norms over the projection (no convolution); a block
+// then holds all heads, and the square sums of a batch of tokens meet in shared memory behind one barrier.
+template <int NH, bool kConv, bool kAll>
+__global__ void __launch_bounds__(kAll ? 512 : 128, kAll ? 1 : 4) conv_norm_rope_128_kernel(const ConvRope p) {
+  constexpr int V = 4, W = 3, kBatch = kAll ? 2 : 4, kMaxWarps = kAll ? 16 : 1;
+  using Row = Packed<__nv_bfloat16, V>;
+  extern __shared__ float4 sm4[];               // the run's angles [run][rot / 2] cos, sin, then its slots [run]
+  __shared__ float part[2][kBatch][kMaxWarps];
+  const int half = p.rot >> 1, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  float2* s_cs = reinterpret_cast<float2*>(sm4);
+  int* s_slot = reinterpret_cast<int*>(s_cs + p.run * half);
+  const int uq = p.nq >> 7, uk = p.nk >> 7, C = p.nq + p.nk + p.nv;
+  const int u0 = (blockIdx.y * (blockDim.x >> 5) + warp) * NH;             // (the launch gives every warp its heads)
+  const bool is_q = u0 < uq, is_k = !is_q && u0 < uq + uk;
+  const int c = u0 * 128 + lane * V, d = lane * V;
+  const int halo = kConv ? p.taps - 1 : 0;
+  float w[kConv ? W + 1 : 1][NH][V];            // w[k]: weight of the input k tokens back
+  float wn[kAll ? NH : 1][V];
+  if constexpr (kConv) {
+#pragma unroll
+    for (int k = 0; k <= W; ++k)
+#pragma unroll
+      for (int h = 0; h < NH; ++h) {
+#pragma unroll
+        for (int e = 0; e < V; ++e) w[k][h][e] = 0.f;
+        if (k <= halo) load_vec<float, V>(p.conv_w + static_cast<size_t>(halo - k) * C + c + h * 128, w[k][h]);
+      }
+  }
+#pragma unroll
+  for (int h = 0; h < (kAll ? NH : 1); ++h) {
+#pragma unroll
+    for (int e = 0; e < V; ++e) wn[h][e] = 1.f;
+    if (p.norm && (is_q || is_k)) load_vec<float, V>((is_q ? p.q_norm + (kAll ? c : d) : p.k_norm + (kAll ? c - p.nq : d)) + h * 128, wn[h]);
+  }
+  pdl_wait();
+  pdl_trigger();
+  const int r0 = blockIdx.x * p.run, r1 = min(p.T, r0 + p.run);
+  const __nv_bfloat16* src = static_cast<const __nv_bfloat16*>(p.proj) + conv_rope_col(p, c);
+  auto row_at = [&](int row, int h) { return load_packed<__nv_bfloat16, V>(src + static_cast<size_t>(row) * p.ld + h * 128); };
+  Row nx[kBatch][NH];                           // the next batch's rows, on their way while one is worked on
+#pragma unroll
+  for (int j = 0; j < kBatch; ++j)
+#pragma unroll
+    for (int h = 0; h < NH; ++h) nx[j][h] = row_at(min(r0 + j, r1 - 1), h);
+  int seq = 0, s_lo = 0, s_hi = p.T, s_in = 0;
+  if (halo > 0) {
+    seq = seq_of(p.q_start, p.S, p.T, r0);
+    s_lo = p.q_start[seq];
+    s_hi = p.q_start[seq + 1];
+    s_in = p.state_in[seq];
+  }
+  for (int i = threadIdx.x; i < (r1 - r0) * half; i += blockDim.x) s_cs[i] = p.table[static_cast<size_t>(r0) * half + i];
+  for (int i = threadIdx.x; i < r1 - r0; i += blockDim.x) s_slot[i] = p.slots[r0 + i];
+  __syncthreads();
+  Row x[W + kBatch][NH];                        // a batch of rows behind the W before it
+#pragma unroll
+  for (int i = 0; i < W; ++i)
+#pragma unroll
+    for (int h = 0; h < NH; ++h) x[i][h].q = make_uint2(0u, 0u);
+  const bool turns = (is_q || is_k) && d < p.rot;
+  const bool first = d < half;
+  const int partner = !turns ? lane : first ? lane + half / V : lane - half / V;       // halves; neighbours lie in the same lane
+  int flip = 0;
+  for (int t = r0; t < r1; t += kBatch) {
+#pragma unroll
+    for (int j = 0; j < kBatch; ++j)
+#pragma unroll
+      for (int h = 0; h < NH; ++h) x[W + j][h] = nx[j][h];
+    if (t + kBatch < r1) {
+#pragma unroll
+      for (int j = 0; j < kBatch; ++j)
+#pragma unroll
+        for (int h = 0; h < NH; ++h) nx[j][h] = row_at(min(t + kBatch + j, r1 - 1), h);
+    }
+    float inv_all[kBatch];
+    if constexpr (kAll) {
+#pragma unroll
+      for (int j = 0; j < kBatch; ++j) {
+        float s = 0.f;
+#pragma unroll
+        for (int h = 0; h < NH; ++h) {
+          float v[V];
+          unpack(x[W + j][h], v);
+#pragma unroll
+          for (int e = 0; e < V; ++e) s = fmaf(v[e], v[e], s);
+        }
+        s = warp_sum(s);
+        if (lane == 0) part[flip][j][warp] = s;
+      }
+      __syncthreads();
+      const int w0 = is_q ? 0 : uq / NH, w1 = is_q ? uq / NH : (uq + uk) / NH;
+#pragma unroll
+      for (int j = 0; j < kBatch; ++j) {
+        const float s = warp_sum(lane >= w0 && lane < w1 ? part[flip][j][lane & (kMaxWarps - 1)] : 0.f);
+        inv_all[j] = 1.0f / sqrtf(s / static_cast<float>(is_q ? p.nq : p.nk) + p.eps);
+      }
+      flip ^= 1;
+    }
+#pragma unroll
+    for (int j = 0; j < kBatch; ++j) {
+      const int row = t + j;
+      if (row >= r1) break;
+      if (halo > 0 && (row == r0 || row == s_hi)) {
+        // The inputs before a run's or a sequence's first token: rows of this step, or the state where they lie before it.
+        // (The slots held another sequence's last inputs, which are done with.)
+        while (row == s_hi && seq + 1 < p.S) {  // (empty sequences are skipped)
+          ++seq;
+          s_lo = s_hi;
+          s_hi = p.q_start[seq + 1];
+          s_in = p.state_in[seq];
+        }
+        const float* st = p.state + static_cast<size_t>(s_in) * p.slot_stride + p.state_off + c;
+#pragma unroll
+        for (int k = 1; k <= W; ++k) {
+          if (k <= halo) {
+#pragma unroll
+            for (int h = 0; h < NH; ++h) {
+              if (row - k >= s_lo) {
+                x[W + j - k][h] = row_at(row - k, h);
+              } else {
+                float v[V];
+                load_vec<float, V>(st + static_cast<size_t>(halo + row - k - s_lo) * C + h * 128, v);
+                x[W + j - k][h].q = make_uint2(pack_bf16(v[0], v[1]), pack_bf16(v[2], v[3]));      // what was stored were bf16 rows
+              }
+            }
+          }
+        }
+      }
+      const int slot = s_slot[row - r0];
+      float2 cs[V];                             // neighbours use the first half of them
+      if (turns) {
+        const float2* a = s_cs + (row - r0) * half + (p.halves ? (first ? d : d - half) : d >> 1);
+#pragma unroll
+        for (int e = 0; e < V; ++e) cs[e] = p.halves || e < V / 2 ? a[e] : make_float2(1.f, 0.f);
+      }
+#pragma unroll
+      for (int h = 0; h < NH; ++h) {
+        float y[V];
+        unpack(x[W + j][h], y);
+        if constexpr (kConv) {
+#pragma unroll
+          for (int e = 0; e < V; ++e) y[e] *= w[0][h][e];
+#pragma unroll
+          for (int k = W; k > 0; --k) {
+            if (k <= halo) {                    // (past the taps there may be another sequence's inputs)
+              float v[V];
+              unpack(x[W + j - k][h], v);
+#pragma unroll
+              for (int e = 0; e < V; ++e) y[e] = fmaf(w[k][h][e], v[e], y[e]);
+            }
+          }
+        }
+        const size_t cell = slot < 0 ? 0 : (static_cast<size_t>(slot >> 6) * p.kv_heads) * 8192 + (slot & 63) * 128 + d;
+        const int g = u0 + h - uq - (is_k ? 0 : uk);                       // key or value head
+        if (!is_q && !is_k) {
+          if (slot >= 0) store_vec<__nv_bfloat16, V>(static_cast<__nv_bfloat16*>(p.v_cache) + cell + static_cast<size_t>(g) * 8192, y);
+          continue;
+        }
+        if (p.v_from_k && is_k && slot >= 0) store_vec<__nv_bfloat16, V>(static_cast<__nv_bfloat16*>(p.v_cache) + cell + static_cast<size_t>(g) * 8192, y);
+        if (p.norm) {
+          float inv;
+          if constexpr (kAll) {
+            inv = inv_all[j];
+          } else {
+            float s = 0.f;
+#pragma unroll
+            for (int e = 0; e < V; ++e) s = fmaf(y[e], y[e], s);
+            inv = 1.0f / sqrtf(warp_sum(s) * (1.0f / 128.0f) + p.eps);
+          }
+#pragma unroll
+          for (int e = 0; e < V; ++e) y[e] = y[e] * inv * wn[kAll ? h : 0][e];
+        }
+        if (p.halves) {
+#pragma unroll
+          for (int e = 0; e < V; ++e) {
+            const float o = __shfl_sync(0xffffffffu, y[e], partner);
+            if (turns) y[e] = first ? y[e] * cs[e].x - o * cs[e].y : y[e] * cs[e].x + o * cs[e].y;
+          }
+        } else if (turns) {
+#pragma unroll
+          for (int e = 0; e < V; e += 2) {
+            const float2 a = cs[e >> 1];
+            const float x0 = y[e], x1 = y[e + 1];
+            y[e] = x0 * a.x - x1 * a.y;
+            y[e + 1] = x1 * a.x + x0 * a.y;
+          }
+        }
+        if (is_q) store_vec<__nv_bfloat16, V>(static_cast<__nv_bfloat16*>(p.q_out) + static_cast<size_t>(row) * p.nq + c + h * 128, y);
+        else if (slot >= 0) store_vec<__nv_bfloat16, V>(static_cast<__nv_bfloat16*>(p.k_cache) + cell + static_cast<size_t>(g) * 8192, y);
+      }
+      if (halo > 0 && row == s_hi - 1) {        // the sequence's last halo inputs, oldest first
+        float* so = p.state + static_cast<size_t>(p.state_out[seq]) * p.slot_stride + p.state_off + c;
+#pragma unroll
+        for (int k = 0; k < W; ++k) {
+          if (k < halo) {
+#pragma unroll
+            for (int h = 0; h < NH; ++h) {
+              float v[V];
+              unpack(x[W + j - k][h], v);
+              store_vec<float, V>(so + static_cast<size_t>(halo - 1 - k) * C + h * 128, v);
+            }
+          }
+        }
+      }
+    }
+#pragma unroll
+    for (int i = 0; i < W; ++i)
+#pragma unroll
+      for (int h = 0; h < NH; ++h) x[i][h] = x[kBatch + i][h];
+  }
+}
+
 // logits = cap * tanh(logits / cap), rows of n values `ld` apart
 __global__ void __launch_bounds__(256) softcap_kernel(float* __restrict__ x, int n, long long ld, float cap) {
   pdl_wait();
@@ -518,8 +733,49 @@ static int launch_conv_norm_rope(ConvRope p, cudaStream_t st) {
   return static_cast<int>(cudaGetLastError());
 }
 
+template <int NH, bool kConv, bool kAll>
+static int launch_conv_norm_rope_128(ConvRope p, cudaStream_t st) {
+  const int groups = (p.nq + p.nk + p.nv) / 128 / NH;
+  int warps = groups;
+  if (!kAll) {
+    warps = 4;
+    while (groups % warps) --warps;
+  }
+  const int cols = groups / warps, row_bytes = p.rot * 4 + 4;
+  const int want = 148 * (warps < 16 ? 16 / warps : 1);                    // blocks of one wave: 16 warps of up to 128 registers a thread
+  int run = (p.T * cols + want - 1) / want;
+  run = p.T <= 64 ? 1 : run < 4 ? 4 : run > 128 ? 128 : run;
+  const int fit = 40 * 1024 / row_bytes;
+  p.run = run < fit ? run : fit;
+  launch_pdl(conv_norm_rope_128_kernel<NH, kConv, kAll>, dim3((p.T + p.run - 1) / p.run, cols), dim3(warps * 32),
+             static_cast<size_t>(p.run) * row_bytes, st, p);
+  return static_cast<int>(cudaGetLastError());
+}
+
+// Whether the kernel for heads of 128 takes this shape; -1 = it does not.
+static int dispatch_conv_norm_rope_128(const ConvRope& p, cudaStream_t st) {
+  const int pair = p.halves ? p.rot / 2 : p.rot;
+  if (p.dim != 128 || p.maps_dim != 128 || p.vdim != 128 || pair % 4 || p.ld % 4 || p.q_off % 4 || p.k_off % 4 || p.v_off % 4 || p.state_off % 4 ||
+      p.slot_stride % 4 || (p.conv_w && p.taps > 4))
+    return -1;
+  const int q = p.nq / 128, k = p.nk / 128, units = q + k + p.nv / 128;
+  if (p.norm == 2) {
+    if (p.conv_w) return -1;
+    if (q % 4 == 0 && k % 4 == 0 && units <= 64) return launch_conv_norm_rope_128<4, false, true>(p, st);
+    if (q % 2 == 0 && k % 2 == 0 && units <= 32) return launch_conv_norm_rope_128<2, false, true>(p, st);
+    return units <= 16 ? launch_conv_norm_rope_128<1, false, true>(p, st) : -1;
+  }
+  const bool two = q % 2 == 0 && k % 2 == 0;
+  if (p.conv_w) return two ? launch_conv_norm_rope_128<2, true, false>(p, st) : launch_conv_norm_rope_128<1, true, false>(p, st);
+  return two ? launch_conv_norm_rope_128<2, false, false>(p, st) : launch_conv_norm_rope_128<1, false, false>(p, st);
+}
+
 template <typename E>
 static int dispatch_conv_norm_rope(const ConvRope& p, cudaStream_t st) {
+  if (sizeof(E) == 2) {
+    const int rc = dispatch_conv_norm_rope_128(p, st);
+    if (rc != -1) return rc;
+  }
   auto fits = [&](int v) {
     const int pair = p.halves ? p.rot / 2 : p.rot;
     return p.dim % v == 0 && p.vdim % v == 0 && p.ld % v == 0 && p.q_off % v == 0 && p.k_off % v == 0 && p.v_off % v == 0 && pair % v == 0 &&
