@@ -1,4 +1,4 @@
-"""A few eager decode steps of a shortened Qwen3-30B-A3B-shape (or, with ``--config dsv3``, DeepSeek-V3-shape) model,
+"""A few eager decode steps of a shortened Qwen3-30B-A3B-shape (or, with ``--config``, DeepSeek-V3-shape or per-layer design) model,
 bracketed by cudaProfilerStart/Stop, as a target for per-kernel launch lists:
 
     python -m cuteafd_b200.bench.decode_profile --concurrency 8 --context 8192 --layers 2
@@ -26,7 +26,8 @@ def main() -> None:
     ap.add_argument("--context", type=int, default=8192)
     ap.add_argument("--layers", type=int, default=2)
     ap.add_argument("--steps", type=int, default=3)
-    ap.add_argument("--config", default="qwen3", choices=["qwen3", "dsv3"])
+    ap.add_argument("--config", default="qwen3", choices=["qwen3", "dsv3", "karusun", "guberax", "rofapel", "rofapel-gqa"])
+    ap.add_argument("--size", default="base", choices=["small", "base", "large"], help="benchmark size of a per-layer design")
     a = ap.parse_args()
     dev = torch.device("cuda:0")
     pps = a.context // 64 + 4
@@ -37,8 +38,19 @@ def main() -> None:
         cfg = deepseek_v3().replace(num_layers=a.layers, first_dense_layers=1, mtp_layers=0)
         W = MlaMoeWeights.random_init(cfg, dev)
         eng = MlaMoeEngine(cfg, W, LatentCache(cfg, pages, dev), max_tokens=a.context, max_seqs=a.concurrency)
+    elif a.config in ("karusun", "guberax", "rofapel"):
+        from .. import config as C
+        from ..models.hybrid import HybridCache, HybridEngine, HybridWeights
+        cfg = getattr(C, a.config + "_bench")(a.size)
+        cfg = C.scaled_down(cfg, a.layers, cfg.vocab_size)
+        W = HybridWeights.random_init(cfg, dev)
+        eng = HybridEngine(cfg, W, HybridCache(cfg, pages, dev, 2 + 4 * a.concurrency), max_tokens=a.context, max_seqs=a.concurrency)
     else:
-        cfg = qwen3_30b_a3b().replace(num_layers=a.layers)
+        cfg = qwen3_30b_a3b()
+        if a.config == "rofapel-gqa":
+            from ..config import rofapel_bench_gqa
+            cfg = rofapel_bench_gqa(a.size)
+        cfg = cfg.replace(num_layers=a.layers)
         W = GqaMoeWeights.random_init(cfg, dev)
         eng = GqaMoeEngine(cfg, W, KvCache(cfg, pages, dev), max_tokens=a.context, max_seqs=a.concurrency)
     gen = Generator(eng, make_pool(pages), pps, a.concurrency, prefill_chunk=a.context, use_graphs=False)
