@@ -82,8 +82,8 @@ class AttentionSpec:
     map 1 - lambda * map 2, the difference normed per head and scaled by 1 - ``diff`` (lambda's constant part).
 
     ``qk_norm``: RMS norm of queries and keys before their rotation, per head ("head", one weight vector for all heads) or over the
-    whole projection ("all").  ``v_from_k``: the values are the convolved keys before norm and rotation.  ``sink``: a learned
-    number per head whose exponential joins the softmax's denominator.  ``gate``: a head's output is multiplied by the sigmoid of
+    whole projection ("all").  ``v_from_k``: the values are the convolved keys before norm and rotation.  ``sink``: a
+    trained logit per head that takes a share of the softmax and hands nothing through.  ``gate``: a head's output is multiplied by the sigmoid of
     one projected number."""
     heads: int
     kv_heads: int

@@ -92,7 +92,7 @@ def sink_attention(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, start: int
                    sink: torch.Tensor | None = None) -> torch.Tensor:
     """Softmax attention of q [T, H, Dk] (positions start, start + 1, ...) over k [L, H, Dk], v [L, H, Dv] (positions 0, 1, ...):
     the query at position i reads the keys j <= i that lie among the last ``window`` positions (0: anywhere) or the first
-    ``keep``.  ``sink`` [H]: exp(sink_h) joins head h's denominator, without a key or a value."""
+    ``keep``.  ``sink`` [H]: a further logit per head that takes a share of the softmax and hands nothing through."""
     i = torch.arange(start, start + q.shape[0])[:, None]
     j = torch.arange(k.shape[0])[None]
     seen = (j <= i) & ((i - j < window) | (j < keep)) if window else j <= i

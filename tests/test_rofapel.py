@@ -185,7 +185,7 @@ def test_values_are_the_convolved_keys_before_norm_and_rotation():
     assert st["conv.k"].tolist() == [[1.0, 3.0]] and st["v"].shape == (2, 1, 2)
 
 
-def test_sink_counts_once_and_is_not_scaled():
+def test_sink_takes_its_share_whatever_the_scale():
     q, k, v = torch.zeros(1, 2, 1), torch.zeros(3, 2, 1), torch.ones(3, 2, 1)
     sink = torch.tensor([math.log(5.0), -40.0])
     y = R.sink_attention(q, k, v, 2, 0, 0, 100.0, sink)
