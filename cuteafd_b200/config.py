@@ -82,9 +82,11 @@ class AttentionSpec:
     map 1 - lambda * map 2, the difference normed per head and scaled by 1 - ``diff`` (lambda's constant part).
 
     ``qk_norm``: RMS norm of queries and keys before their rotation, per head ("head", one weight vector for all heads) or over the
-    whole projection ("all").  ``v_from_k``: the values are the convolved keys before norm and rotation.  ``sink``: a
-    trained logit per head that takes a share of the softmax and hands nothing through.  ``gate``: a head's output is multiplied by the sigmoid of
-    one projected number."""
+    whole projection ("all"), or after it, per head and without a weight ("rotated").  ``v_from_k``: the values are the convolved keys
+    before norm and rotation.  ``sink``: a trained logit per head that takes a share of the softmax and hands nothing through;
+    ``unit_sink``: the same with logit 0 for every head.  ``gate``: a head's output is multiplied by the sigmoid of one projected
+    number.  ``softcap``: scores pass cap * tanh(score / cap) (0 = they do not).  ``v_rope``: a value is rotated by its position
+    before it is cached, and a head's output is turned back by the query's."""
     heads: int
     kv_heads: int
     dim: int                             # query / key dims per map and head
@@ -96,10 +98,13 @@ class AttentionSpec:
     conv: int = 0
     maps: int = 1
     diff: float = 0.0
-    qk_norm: str = ""                    # "" | "head" | "all"
+    qk_norm: str = ""                    # "" | "head" | "all" | "rotated"
     v_from_k: bool = False
     sink: bool = False
     gate: bool = False
+    softcap: float = 0.0
+    unit_sink: bool = False
+    v_rope: RopeSpec | None = None
 
     @property
     def q_channels(self) -> int:
@@ -120,9 +125,62 @@ class AttentionSpec:
 
 
 @dataclass(frozen=True)
+class RglruSpec:
+    """Gated linear recurrence of ``width`` channels beside a gelu branch of the same width: a causal convolution of ``conv`` taps, then
+    per channel S <- a S + sqrt(1 - a^2) i u with a = exp(-``c`` r softplus(lam)); r and i are sigmoids of block-diagonal products
+    (``blocks`` square matrices each)."""
+    width: int
+    blocks: int
+    conv: int
+    c: float = 8.0
+
+    @property
+    def block(self) -> int:
+        return self.width // self.blocks
+
+
+@dataclass(frozen=True)
+class LightningSpec:
+    """Linear attention with one constant decay per head: S <- decay S + k v^T, o = S^T q on silu'd projections; all heads' outputs are
+    normed together under one weight vector and multiplied by the sigmoid of a projection as wide as they are."""
+    heads: int
+    dim: int
+    vdim: int
+    decay: tuple
+
+    @property
+    def channels(self) -> int:
+        """Projected channels of q, k, v and the gate."""
+        return 2 * self.heads * (self.dim + self.vdim)
+
+
+@dataclass(frozen=True)
+class PairSpec:
+    """Two mixers on the same rows: left_scale * left + right_scale * right."""
+    left: AttentionSpec
+    right: LightningSpec
+    left_scale: float = 1.0
+    right_scale: float = 1.0
+
+    @property
+    def heads(self) -> int:
+        return max(self.left.heads, self.right.heads)
+
+
+def attention_part(m: Any) -> AttentionSpec | None:
+    """The attention of a mixer that caches keys and values per position (one half of a pair, or the mixer itself)."""
+    m = m.left if isinstance(m, PairSpec) else m
+    return m if isinstance(m, AttentionSpec) else None
+
+
+@dataclass(frozen=True)
 class DenseSpec:
-    """SwiGLU feed-forward of width ``ffn``."""
+    """Gated feed-forward of width ``ffn``: with g and u the two projections, g sigmoid(``alpha`` g) (u + ``up_bias``).  ``limit`` other
+    than 0: g is cut off above it and u on both sides first."""
     ffn: int
+    limit: float = 0.0
+    alpha: float = 1.0
+    up_bias: float = 0.0
 
 
 @dataclass(frozen=True)
@@ -139,6 +197,7 @@ class RouterSpec:
     groups_kept: int = 1
     logit_bias: bool = False
     normalize: bool = False
+    scoring: str = "softmax"             # "softmax" | "sigmoid"
 
     @property
     def outputs(self) -> int:
@@ -147,22 +206,32 @@ class RouterSpec:
 
 @dataclass(frozen=True)
 class LayerSpec:
-    mixer: Any                           # LatentSpec | DeltaSpec | AttentionSpec
+    mixer: Any                           # LatentSpec | DeltaSpec | AttentionSpec | RglruSpec | PairSpec
     router: RouterSpec | None = None     # None = the layer has no routed feed-forward
     dense: DenseSpec | None = None       # dense feed-forward (parallel layers); beside a router: the shared expert
     # parallel: mixer and feed-forward read one norm and are added together, nothing is normed after them; otherwise the
     # sublayers follow one another, each with a norm before and after it and a convolution on its input
     parallel: bool = False
     two_norms: bool = False              # parallel: the feed-forward reads a norm of its own
+    # the sublayers follow one another and read the residual itself; what each gives is normed before it is added
+    post_norm: bool = False
 
     @staticmethod
     def from_dict(d: dict[str, Any]) -> "LayerSpec":
-        m = dict(d["mixer"])
-        if "rope" in m:
-            m["rope"] = RopeSpec(**m["rope"])
-        mixer = (LatentSpec if "kv_rank" in m else AttentionSpec if "rope" in m else DeltaSpec)(**m)
-        return LayerSpec(mixer, RouterSpec(**d["router"]) if d.get("router") else None, DenseSpec(**d["dense"]) if d.get("dense") else None,
-                         bool(d.get("parallel", False)), bool(d.get("two_norms", False)))
+        def mixer(m: dict[str, Any]) -> Any:
+            if "left" in m:
+                return PairSpec(**dict(m, left=mixer(m["left"]), right=mixer(m["right"])))
+            m = {k: RopeSpec(**v) if k in ("rope", "v_rope") and v else tuple(v) if k == "decay" else v for k, v in m.items()}
+            kind = (LatentSpec if "kv_rank" in m else AttentionSpec if "rope" in m else RglruSpec if "blocks" in m else
+                    LightningSpec if "decay" in m else DeltaSpec)
+            return kind(**m)
+        return LayerSpec(mixer(d["mixer"]), RouterSpec(**d["router"]) if d.get("router") else None,
+                         DenseSpec(**d["dense"]) if d.get("dense") else None, bool(d.get("parallel", False)), bool(d.get("two_norms", False)),
+                         bool(d.get("post_norm", False)))
+
+    @property
+    def has_ffn(self) -> bool:
+        return self.router is not None or self.dense is not None
 
 
 @dataclass(frozen=True)
@@ -235,9 +304,15 @@ class ModelConfig:
     canon_taps: int = 0                  # taps of the convolution every sublayer's input passes (0 = none)
     norm_groups: int = 1                 # channel groups of the RMS norms
     norm_offset: float = 0.0             # added to the stored norm weights (1: they are stored around zero)
+    norm_scalar: bool = False            # a norm's weight is one number for all channels
     loop: tuple = ()                     # (start, stop, times): layers [start, stop) run ``times`` times in a row
     loop_join: bool = False              # every pass starts with a product of [x; embedding row] and adds a vector of its own
     embed_scale: float = 1.0             # the embedding's rows are multiplied by it
+    # (buckets, mul_prev, mul_cur): row (previous token * mul_prev + token * mul_cur) mod buckets of a second table is added to the
+    # embedding row, for a sequence's first token the row after the last bucket
+    bigram: tuple = ()
+    # after every layer the residual becomes a weighted sum of the embedding rows and all layers' results so far
+    depth_average: bool = False
     logit_softcap: float = 0.0           # logits = cap * tanh(logits / cap); 0 = none
     compute_dtype: str = "bf16"          # bf16 | f32 (every product and activation in 32-bit; hybrid engine only)
 
@@ -262,26 +337,37 @@ class ModelConfig:
                   for t in range(times) for i in range(start, stop)]
         return tuple([LayerRun(i) for i in range(start)] + passes + [LayerRun(i) for i in range(stop, self.num_layers)])
 
+    def state_parts(self, layer: int) -> list[tuple[str, int]]:
+        """(name, floats) of everything recurrent one run of ``layer`` carries per sequence."""
+        spec = self.layer_specs[layer]
+        m, out = spec.mixer, []
+        if not spec.parallel and not spec.post_norm:
+            out.append(("canon1", (self.canon_taps - 1) * self.hidden))
+            if spec.router is not None:
+                out.append(("canon2", (self.canon_taps - 1) * self.hidden))
+        if isinstance(m, DeltaSpec):
+            out += [("S", m.heads * m.dim * m.vdim), ("conv", (m.conv - 1) * m.conv_channels)]
+        elif isinstance(m, RglruSpec):
+            out += [("S", m.width), ("conv", (m.conv - 1) * m.width)]
+        elif isinstance(m, PairSpec):
+            out.append(("S", m.right.heads * m.right.dim * m.right.vdim))
+        a = attention_part(m)
+        if a is not None:
+            out.append(("conv", max(0, a.conv - 1) * a.conv_channels))
+        return out
+
     @property
     def state_bytes(self) -> int:
-        """Recurrent state of one sequence (fp32): delta-rule states and the last inputs of every causal convolution."""
-        n = 0
-        for s in (self.layer_specs[r.layer] for r in self.layer_runs):
-            m = s.mixer
-            if not s.parallel:
-                n += (self.canon_taps - 1) * self.hidden * (2 if s.router is not None else 1)
-            if isinstance(m, DeltaSpec):
-                n += m.heads * m.dim * m.vdim
-            if not isinstance(m, LatentSpec):
-                n += max(0, m.conv - 1) * m.conv_channels
-        return 4 * n
+        """Recurrent state of one sequence (fp32): the mixers' states, the last inputs of every causal convolution, the last token."""
+        return 4 * (sum(n for r in self.layer_runs for _, n in self.state_parts(r.layer)) + bool(self.bigram))
 
     def kv_elems_of(self, layer: int) -> int:
         """Elements one run of ``layer`` caches per token."""
         if self.is_hybrid:
             m = self.layer_specs[layer].mixer
-            if isinstance(m, AttentionSpec):
-                return m.k_channels + m.v_channels
+            a = attention_part(m)
+            if a is not None:
+                return a.k_channels + a.v_channels
             return m.record if isinstance(m, LatentSpec) else 0
         return self.kv_record_elems
 
@@ -304,7 +390,8 @@ class ModelConfig:
     def window_of(self, layer: int) -> int:
         """Sliding window of ``layer`` in tokens; 0 = full causal attention."""
         if self.is_hybrid:
-            return getattr(self.layer_specs[layer].mixer, "window", 0)
+            m = self.layer_specs[layer].mixer
+            return getattr(attention_part(m) or m, "window", 0)
         if not self.sliding_window or self.is_mla:
             return 0
         if self.window_layers:
@@ -317,9 +404,18 @@ class ModelConfig:
         return self.num_experts > 0 and layer >= self.first_dense_layers
 
     def mixer_params(self, layer: int) -> int:
-        h, m = self.hidden, self.layer_specs[layer].mixer
+        return self._mixer_params(self.layer_specs[layer].mixer)
+
+    def _mixer_params(self, m: Any) -> int:
+        h = self.hidden
+        if isinstance(m, PairSpec):
+            return self._mixer_params(m.left) + self._mixer_params(m.right)
+        if isinstance(m, LightningSpec):
+            return h * (m.channels + m.heads * m.vdim) + m.heads * m.vdim
+        if isinstance(m, RglruSpec):
+            return m.width * (3 * h + m.conv + 2 * m.block + 6)
         if isinstance(m, AttentionSpec):
-            norms = {"": 0, "head": 2 * m.dim, "all": m.q_channels + m.k_channels}[m.qk_norm]
+            norms = {"": 0, "head": 2 * m.dim, "all": m.q_channels + m.k_channels, "rotated": 0}[m.qk_norm]
             return (h * (m.conv_channels + m.heads * m.vdim + m.heads * m.gate) + m.conv * m.conv_channels + norms + m.heads * m.sink
                     + (4 * m.dim if m.maps == 2 else 0))
         if isinstance(m, LatentSpec):
@@ -348,6 +444,10 @@ class ModelConfig:
             spec = self.layer_specs[layer]
             r, d = spec.router, spec.dense
             routed = r.outputs * (self.hidden + 1) + 3 * r.experts * self.hidden * r.ffn if r is not None else 0
+            if spec.post_norm:
+                norm = 1 if self.norm_scalar else self.hidden
+                return (self.mixer_params(layer) + routed + (3 * self.hidden * d.ffn if d is not None else 0) + norm * (1 + spec.has_ffn)
+                        + (layer + 2 if self.depth_average else 0))
             if spec.parallel:
                 norms = 2 if spec.two_norms and (r is not None or d is not None) else 1
                 return self.mixer_params(layer) + norms * self.hidden + routed + (3 * self.hidden * d.ffn if d is not None else 0)
@@ -364,7 +464,9 @@ class ModelConfig:
         return p
 
     def total_params(self) -> int:
-        p = self.vocab_size * self.hidden * (1 if self.tie_embeddings else 2) + self.hidden
+        p = self.vocab_size * self.hidden * (1 if self.tie_embeddings else 2) + (1 if self.norm_scalar else self.hidden)
+        if self.bigram:
+            p += (self.bigram[0] + 1) * self.hidden
         if self.loop and self.loop_join:
             p += (2 * self.hidden + self.loop[2]) * self.hidden
         return p + sum(self.layer_params(i) for i in range(self.num_layers))
@@ -378,8 +480,9 @@ class ModelConfig:
         d = {k: v for k, v in d.items() if k in names}
         if "window_layers" in d:
             d["window_layers"] = tuple(d["window_layers"])
-        if "loop" in d:
-            d["loop"] = tuple(d["loop"])
+        for k in ("loop", "bigram"):
+            if k in d:
+                d[k] = tuple(d[k])
         if d.get("layer_specs"):
             d["layer_specs"] = tuple(v if isinstance(v, LayerSpec) else LayerSpec.from_dict(v) for v in d["layer_specs"])
         return ModelConfig(**d)
@@ -468,23 +571,24 @@ def hybrid_config(name: str, vocab: int, hidden: int, specs, canon_taps: int, no
     things (planner, reports); the engine reads the specs.  ``kw``: further fields (norm_offset, loop, logit_softcap)."""
     specs = tuple(specs)
     lat = [s.mixer for s in specs if isinstance(s.mixer, LatentSpec)]
-    att = [s.mixer for s in specs if isinstance(s.mixer, AttentionSpec)]
+    att = [a for a in (attention_part(s.mixer) for s in specs) if a is not None]
     routers = [s.router for s in specs if s.router is not None]
     big = max(lat, key=lambda m: m.heads * (m.dim + m.rot_dim), default=None)
     wide = max(routers, key=lambda r: r.experts * r.ffn, default=None)
     top = max(att, key=lambda m: m.conv_channels, default=None)
     rope = big.rope if big else top.rope if top else RopeSpec(0, 10000.0, halves=True)
-    head_dim = (big.dim + big.rot_dim) if big else (top.maps * top.dim) if top else specs[0].mixer.dim
+    head_dim = (big.dim + big.rot_dim) if big else (top.maps * top.dim) if top else getattr(specs[0].mixer, "dim", 0)
+    vdim = big.vdim if big else top.vdim if top else getattr(specs[0].mixer, "vdim", 0)
     return ModelConfig(
         name=name, family=family, vocab_size=vocab, num_layers=len(specs), hidden=hidden, attention="hybrid", layer_specs=specs,
         canon_taps=canon_taps, norm_groups=norm_groups, rms_eps=eps, rope_interleaved=not rope.halves,
-        num_heads=max(s.mixer.heads for s in specs), num_kv_heads=top.kv_heads if top else 1, head_dim=head_dim,
+        num_heads=max(getattr(s.mixer, "heads", 1) for s in specs), num_kv_heads=top.kv_heads if top else 1, head_dim=head_dim,
         q_lora_rank=0, kv_lora_rank=big.kv_rank if big else 0, qk_nope_dim=big.dim if big else 0, qk_rope_dim=big.rot_dim if big else 0,
-        v_head_dim=big.vdim if big else specs[0].mixer.vdim, rope_theta=rope.base,
+        v_head_dim=vdim, rope_theta=rope.base,
         sliding_window=max((m.window for m in lat + att), default=0), dense_ffn=max((s.dense.ffn for s in specs if s.dense and not s.router), default=0),
         first_dense_layers=0, num_experts=wide.experts if wide else 0, expert_ffn=wide.ffn if wide else 0, top_k=wide.top if wide else 0,
         num_groups=wide.groups if wide else 1, topk_groups=wide.groups_kept if wide else 1, num_shared_experts=int(any(s.router and s.dense for s in specs)),
-        norm_topk_prob=bool(wide and wide.normalize), router_bias=bool(routers), **kw)
+        norm_topk_prob=bool(wide and wide.normalize), router_bias=bool(routers), scoring=wide.scoring if wide else "softmax", **kw)
 
 
 def parallel_config(name: str, vocab: int, hidden: int, specs, eps: float, loop: tuple = (), logit_softcap: float = 0.0,
@@ -493,6 +597,13 @@ def parallel_config(name: str, vocab: int, hidden: int, specs, eps: float, loop:
     fields (loop_join, embed_scale)."""
     return hybrid_config(name, vocab, hidden, specs, canon_taps=1, norm_groups=1, eps=eps, family=family, norm_offset=1.0,
                          loop=tuple(loop), logit_softcap=logit_softcap, **kw)
+
+
+def post_norm_config(name: str, vocab: int, hidden: int, specs, eps: float, bigram: tuple = (), logit_softcap: float = 0.0,
+                     family: str = "buzarax", **kw: Any) -> ModelConfig:
+    """ModelConfig of a stack whose sublayers are normed after they ran, under one number per norm, with averages over depth."""
+    return hybrid_config(name, vocab, hidden, specs, canon_taps=1, norm_groups=1, eps=eps, family=family, norm_scalar=True,
+                         bigram=tuple(bigram), depth_average=True, logit_softcap=logit_softcap, **kw)
 
 
 # Benchmark sizes: width, layers, heads, expert width (latent 512 + 64 and heads of 128 throughout, as real models have them)
@@ -601,7 +712,8 @@ def scaled_down(cfg: ModelConfig, layers: int = 2, vocab: int = 2048) -> ModelCo
         start, stop, times = cfg.loop or (0, 0, 1)
         return hybrid_config(cfg.name + "-mini", vocab, cfg.hidden, cfg.layer_specs[:layers], cfg.canon_taps, cfg.norm_groups,
                              cfg.rms_eps, cfg.family, norm_offset=cfg.norm_offset, logit_softcap=cfg.logit_softcap,
-                             loop_join=cfg.loop_join, embed_scale=cfg.embed_scale,
+                             loop_join=cfg.loop_join, embed_scale=cfg.embed_scale, norm_scalar=cfg.norm_scalar, bigram=cfg.bigram,
+                             depth_average=cfg.depth_average,
                              loop=(start, min(stop, layers), times) if start < layers and cfg.loop else ())
     first_dense = min(cfg.first_dense_layers, max(layers - 1, 0)) if cfg.first_dense_layers else 0
     return cfg.replace(name=cfg.name + "-mini", num_layers=layers, vocab_size=vocab,

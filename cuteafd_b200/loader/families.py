@@ -206,6 +206,28 @@ class Rofapel(Karusun):
         return RofapelModel(self, cfg, ExpertContract(formats=("bf16",)))
 
 
+class BuzaraxModel(KarusunModel):
+    """A second embedding table, and the weights of the averages over depth beside the norms."""
+
+    def classify(self, name: str) -> tuple[str, int | None, int | None]:
+        if name == "bigram":
+            return "embedding", None, None
+        m = re.fullmatch(r"l(\d+)\.dwa", name)
+        return ("norm", int(m.group(1)), None) if m else super().classify(name)
+
+
+class Buzarax(Karusun):
+    """Layers normed after their sublayers (a gated linear recurrence, or attention beside linear attention, then a dense or routed
+    feed-forward) with averages over depth: served by the hybrid engine."""
+    id, model_types, attention = "buzarax", ("buzarax",), "hybrid"
+
+    def detect(self, hf_config: dict) -> bool:
+        return hf_config.get("architecture") == "Buzarax"
+
+    def open(self, cfg: ModelConfig, hf_config: dict) -> FamilyModel:
+        return BuzaraxModel(self, cfg, ExpertContract(formats=("bf16",)))
+
+
 class TinyMoe(Family):
     id, model_types = "tiny_moe", ("tiny_moe",)
 
@@ -225,7 +247,8 @@ def canonical_name(name: str) -> str:
     return _MIXTRAL_RE.sub(lambda m: m.group(1) + _MIXTRAL_PROJ[m.group(2)] + m.group(3), name)
 
 
-REGISTRY: tuple[Family, ...] = (DeepseekV32(), DeepseekV3(), Qwen3Moe(), Glm4Moe(), Qwen2(), Llama(), TinyMoe(), Karusun(), Guberax(), Rofapel())
+REGISTRY: tuple[Family, ...] = (DeepseekV32(), DeepseekV3(), Qwen3Moe(), Glm4Moe(), Qwen2(), Llama(), TinyMoe(), Karusun(), Guberax(), Rofapel(),
+                                Buzarax())
 
 
 def detect(hf_config: dict) -> Family | None:

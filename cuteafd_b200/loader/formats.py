@@ -98,7 +98,7 @@ def detect_operands(cat: Catalog) -> dict[str, QuantOperand]:
 
 def plain_operands(cat: Catalog) -> dict[str, QuantOperand]:
     """Every tensor as an operand of its own, for checkpoints that store unquantised tensors under bare names."""
-    return {n: QuantOperand(n, _plain(e), (e.shape[0], e.shape[1] if len(e.shape) > 1 else 1), n, bits=8.0 * e.nbytes / max(e.numel, 1))
+    return {n: QuantOperand(n, _plain(e), (*e.shape, 1, 1)[:2], n, bits=8.0 * e.nbytes / max(e.numel, 1))
             for n, e in cat.entries.items()}
 
 

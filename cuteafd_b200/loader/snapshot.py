@@ -12,8 +12,8 @@ import os
 
 import torch
 
-from ..config import (AttentionSpec, DeltaSpec, DenseSpec, LatentSpec, LayerSpec, ModelConfig, RopeSpec, RouterSpec, hybrid_config,
-                      parallel_config)
+from ..config import (AttentionSpec, DeltaSpec, DenseSpec, LatentSpec, LayerSpec, LightningSpec, ModelConfig, PairSpec, RglruSpec, RopeSpec,
+                      RouterSpec, hybrid_config, parallel_config, post_norm_config)
 from ..ref.model import init_weights
 from . import formats
 from .safetensors_io import write_sharded
@@ -29,6 +29,8 @@ def _layer_list_to_json(cfg: ModelConfig) -> dict:
         return _parallel_layers_to_json(cfg)
     if cfg.family == "rofapel":
         return _two_norm_layers_to_json(cfg)
+    if cfg.family == "buzarax":
+        return _post_norm_layers_to_json(cfg)
     layers = []
     for s in cfg.layer_specs:
         m, r = s.mixer, s.router
@@ -178,6 +180,80 @@ def _two_norm_layers_from_json(d: dict) -> ModelConfig:
                            embed_scale=float((d.get("embedding") or {}).get("scale", 1.0)))
 
 
+# Constants of Buzarax's feed-forward that its configuration does not carry.
+_CLIPPED_ALPHA, _CLIPPED_UP_BIAS = 1.702, 1.0
+
+
+def _post_norm_layers_to_json(cfg: ModelConfig) -> dict:
+    layers = []
+    for s in cfg.layer_specs:
+        m, r, mlp = s.mixer, s.router, None
+        if isinstance(m, PairSpec):
+            a, b = m.left, m.right
+            e = {"type": "parallel", "mixer": {
+                "left": {"heads": a.heads, "kv_heads": a.kv_heads, "dim": a.dim, "vdim": a.vdim, "scale": a.scale, "softcap": a.softcap or None,
+                         "rot": _rope_to_json(a.rope)},
+                "right": {"heads": b.heads, "dim": b.dim, "vdim": b.vdim, "decay": list(b.decay)},
+                "left_scale": m.left_scale, "right_scale": m.right_scale}}
+        else:
+            e = {"type": "rglru", "mixer": {"width": m.width, "blocks": m.blocks, "conv": m.conv}}
+        if r is not None:
+            mlp = {"kind": "moe", "expert": {"ff": r.ffn}, "router": {"experts": r.experts, "top": r.top}}
+        elif s.dense is not None:
+            mlp = {"kind": "dense", "ff": s.dense.ffn, "limit": s.dense.limit}
+        layers.append(dict(e, mlp=mlp))
+    d = {"architecture": "Buzarax", "name": cfg.name, "vocab": cfg.vocab_size, "width": cfg.hidden, "layers": layers, "norm": {"eps": cfg.rms_eps},
+         "embedding": {}}
+    if cfg.bigram:
+        d["embedding"]["bigram"] = dict(zip(("buckets", "mul_prev", "mul_cur"), cfg.bigram))
+    if cfg.logit_softcap:
+        d["logit_softcap"] = cfg.logit_softcap
+    return d
+
+
+def _post_norm_layers_from_json(d: dict) -> ModelConfig:
+    """Layers whose sublayers are normed after they ran: a gated linear recurrence, or attention beside linear attention, then a dense
+    or routed feed-forward or none (``architecture`` Buzarax)."""
+    specs = []
+    for i, e in enumerate(d["layers"]):
+        m, mlp, kind = e["mixer"], e.get("mlp"), e["type"]
+        if kind == "rglru":
+            mixer = RglruSpec(width=m["width"], blocks=m["blocks"], conv=m["conv"])
+            if mixer.width % mixer.blocks:
+                raise ValueError(f"layer {i}: {mixer.width} channels in {mixer.blocks} blocks")
+        elif kind == "parallel":
+            a, b = m["left"], m["right"]
+            rope, vdim = _rope_from_json(i, a["rot"], a["dim"], halves=True), a.get("vdim") or a["dim"]
+            if vdim % 2:
+                raise ValueError(f"layer {i}: values of {vdim} are rotated in pairs")
+            left = AttentionSpec(heads=a["heads"], kv_heads=a.get("kv_heads") or a["heads"], dim=a["dim"], vdim=vdim, window=0, keep_first=0,
+                                 scale=float(a["scale"]), rope=rope, qk_norm="rotated", softcap=float(a.get("softcap") or 0.0), unit_sink=True,
+                                 v_rope=RopeSpec(vdim, rope.base, halves=True))
+            right = LightningSpec(heads=b["heads"], dim=b["dim"], vdim=b.get("vdim") or b["dim"], decay=tuple(float(x) for x in b["decay"]))
+            mixer = PairSpec(left, right, float(m.get("left_scale", 1.0)), float(m.get("right_scale", 1.0)))
+            if left.heads % left.kv_heads:
+                raise ValueError(f"layer {i}: {left.heads} heads over {left.kv_heads} key heads")
+            if len(right.decay) != right.heads:
+                raise ValueError(f"layer {i}: {len(right.decay)} decays for {right.heads} heads")
+        else:
+            raise ValueError(f"layer {i}: unsupported mixer {kind!r}")
+        router = dense = None
+        if mlp is not None and mlp.get("kind") == "dense":
+            dense = DenseSpec(mlp["ff"], limit=float(mlp.get("limit") or 0.0), alpha=_CLIPPED_ALPHA, up_bias=_CLIPPED_UP_BIAS)
+        elif mlp is not None and mlp.get("kind") == "moe":
+            _silu_only(i, mlp["expert"])
+            r = mlp["router"]
+            router = RouterSpec(experts=r["experts"], ffn=mlp["expert"]["ff"], top=r["top"], scoring="sigmoid")
+            if not 1 <= router.top <= router.experts:
+                raise ValueError(f"layer {i}: {router.top} of {router.experts} experts")
+        elif mlp is not None:
+            raise ValueError(f"layer {i}: unsupported feed-forward {mlp.get('kind')!r}")
+        specs.append(LayerSpec(mixer, router, dense, post_norm=True))
+    g = (d.get("embedding") or {}).get("bigram")
+    return post_norm_config(d.get("name", d["architecture"].lower()), d["vocab"], d["width"], specs, float(d["norm"]["eps"]),
+                            bigram=(g["buckets"], g["mul_prev"], g["mul_cur"]) if g else (), logit_softcap=float(d.get("logit_softcap") or 0.0))
+
+
 def _parallel_layers_from_json(d: dict) -> ModelConfig:
     """Parallel layers of differential attention and a dense feed-forward (``architecture`` Guberax)."""
     specs = []
@@ -215,6 +291,8 @@ def _layer_list_from_json(d: dict) -> ModelConfig:
         return _parallel_layers_from_json(d)
     if d["architecture"] == "Rofapel":
         return _two_norm_layers_from_json(d)
+    if d["architecture"] == "Buzarax":
+        return _post_norm_layers_from_json(d)
     specs = []
     for i, e in enumerate(d["layers"]):
         m, mlp = e["mixer"], e.get("mlp")
@@ -342,7 +420,7 @@ def _rope_scaling(d: dict) -> dict:
 
 def from_hf_config(d: dict) -> ModelConfig:
     """Map a config.json onto the engine's geometry.  Unknown architectures raise ValueError."""
-    if d.get("architecture") in ("Karusun", "Guberax", "Rofapel"):
+    if d.get("architecture") in ("Karusun", "Guberax", "Rofapel", "Buzarax"):
         return _layer_list_from_json(d)
     mt = d.get("model_type", "")
     extra = d.get("cuteafd", {})

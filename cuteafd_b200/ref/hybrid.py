@@ -1,6 +1,7 @@
 """CPU oracle of the per-layer hybrid decoders (``ModelConfig.layer_specs``): windowed latent attention layers and gated
 delta-rule layers in any order, each behind grouped RMS norms, input convolutions and a routed feed-forward; parallel
-layers of plain or differential or latent attention beside a dense or routed feed-forward, some of them looped.
+layers of plain or differential or latent attention beside a dense or routed feed-forward, some of them looped; layers normed
+after their sublayers (gated linear recurrences, attention beside linear attention) with averages over depth.
 
 One function per mechanism, written as the equations read: no chunking, no absorbed products, one token at a time where a
 recurrence runs.  ``HybridRefDecoder`` strings them together over a parameter dictionary in the checkpoint's own tensor
@@ -13,7 +14,7 @@ import math
 
 import torch
 
-from ..config import AttentionSpec, DeltaSpec, LatentSpec, ModelConfig, RopeSpec, RouterSpec
+from ..config import AttentionSpec, DeltaSpec, DenseSpec, LatentSpec, LightningSpec, ModelConfig, PairSpec, RglruSpec, RopeSpec, RouterSpec
 
 Params = dict[str, torch.Tensor]
 
@@ -89,14 +90,17 @@ def rotate(x: torch.Tensor, positions: torch.Tensor, r: RopeSpec) -> torch.Tenso
 
 
 def sink_attention(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, start: int, window: int, keep: int, scale: float,
-                   sink: torch.Tensor | None = None) -> torch.Tensor:
+                   sink: torch.Tensor | None = None, cap: float = 0.0) -> torch.Tensor:
     """Softmax attention of q [T, H, Dk] (positions start, start + 1, ...) over k [L, H, Dk], v [L, H, Dv] (positions 0, 1, ...):
     the query at position i reads the keys j <= i that lie among the last ``window`` positions (0: anywhere) or the first
-    ``keep``.  ``sink`` [H]: a further logit per head that takes a share of the softmax and hands nothing through."""
+    ``keep``.  ``sink`` [H]: a further logit per head that takes a share of the softmax and hands nothing through.  ``cap``: scores
+    are cap * tanh(score / cap)."""
     i = torch.arange(start, start + q.shape[0])[:, None]
     j = torch.arange(k.shape[0])[None]
     seen = (j <= i) & ((i - j < window) | (j < keep)) if window else j <= i
     s = torch.einsum("thd,jhd->htj", q, k) * scale
+    if cap:
+        s = softcap(s, cap)
     s = s.masked_fill(~seen, -math.inf)
     if sink is not None:
         s = torch.cat([s, sink[:, None, None].expand(-1, q.shape[0], 1)], -1)
@@ -137,6 +141,50 @@ def delta_recurrence(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, beta: to
     return torch.stack(out), S
 
 
+def decayed_products(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay, S: torch.Tensor) -> tuple[torch.Tensor, torch.Tensor]:
+    """Linear attention.  q, k [T, H, D], v [T, H, Dv], S [H, D, Dv]: per token the state of head h fades by decay[h], takes k v^T
+    and is read with q (the read sees this token's write)."""
+    d = torch.tensor(decay, dtype=S.dtype)[:, None, None]
+    out = []
+    for t in range(q.shape[0]):
+        S = d * S + k[t][:, :, None] * v[t][:, None, :]
+        out.append((S * q[t][:, :, None]).sum(1))
+    return torch.stack(out), S
+
+
+def block_products(u: torch.Tensor, w: torch.Tensor, b: torch.Tensor) -> torch.Tensor:
+    """u [T, C] in equal parts, part n through the square matrix w[n] [out, in] with the offsets b[n]."""
+    parts = u.view(u.shape[0], w.shape[0], -1)
+    return torch.stack([parts[:, n] @ w[n].T + b[n] for n in range(w.shape[0])], 1).reshape(u.shape)
+
+
+def softplus(x: torch.Tensor) -> torch.Tensor:
+    return torch.log1p(torch.exp(-x.abs())) + x.clamp_min(0)
+
+
+def gated_recurrence(u: torch.Tensor, r: torch.Tensor, i: torch.Tensor, lam: torch.Tensor, c: float, S: torch.Tensor):
+    """u, r, i [T, C] (r and i in (0, 1)), S [C]: log a = -c r softplus(lam), S <- a S + sqrt(1 - a^2) i u.  Returns (all S, the last)."""
+    out = []
+    for t in range(u.shape[0]):
+        log_a = -c * r[t] * softplus(lam)
+        S = torch.exp(log_a) * S + torch.sqrt(-torch.expm1(2 * log_a)) * i[t] * u[t]
+        out.append(S)
+    return torch.stack(out), S
+
+
+def gelu_tanh(z: torch.Tensor) -> torch.Tensor:
+    return 0.5 * z * (1 + torch.tanh(math.sqrt(2 / math.pi) * (z + 0.044715 * z ** 3)))
+
+
+def bigram_rows(tokens: list[int], previous: int, buckets: int, mul_prev: int, mul_cur: int) -> list[int]:
+    """Row of the second embedding table for each token; ``previous``: the token before them, -1 at a sequence's start."""
+    out = []
+    for t in tokens:
+        out.append(buckets if previous < 0 else (previous * mul_prev + t * mul_cur) % buckets)
+        previous = t
+    return out
+
+
 def unit(x: torch.Tensor) -> torch.Tensor:
     return x / torch.sqrt((x * x).sum(-1, keepdim=True) + 1e-6)
 
@@ -169,9 +217,18 @@ def route_by_logits(h: torch.Tensor, w: torch.Tensor, bias: torch.Tensor, top: i
     return ids, torch.softmax(z.gather(1, ids), -1)
 
 
+def route_by_sigmoid(h: torch.Tensor, w: torch.Tensor, correction: torch.Tensor, top: int) -> tuple[torch.Tensor, torch.Tensor]:
+    """Sigmoid scores; the ``top`` largest of score + correction are chosen and weigh in with their plain scores."""
+    s = torch.sigmoid(h @ w.T)
+    ids = torch.tensor([sorted(range(s.shape[1]), key=lambda e: (-float(row[e]), e))[:top] for row in s + correction])
+    return ids, s.gather(1, ids)
+
+
 def routed_ffn(h: torch.Tensor, p: Params, pre: str, r: RouterSpec) -> torch.Tensor:
     if r.logit_bias:
         ids, wts = route_by_logits(h, p[pre + "router"], p[pre + "router.b"], r.top)
+    elif r.scoring == "sigmoid":
+        ids, wts = route_by_sigmoid(h, p[pre + "router"], p[pre + "correction"], r.top)
     else:
         ids, wts = route(h, p[pre + "router"], p[pre + "correction"], r)
     y = torch.zeros_like(h)
@@ -234,33 +291,72 @@ def attention_mixer(h: torch.Tensor, p: Params, pre: str, m: AttentionSpec, eps:
         x[n] = h @ p[pre + n].T
         if m.conv:
             x[n], st["conv." + n] = causal_conv(x[n], p[pre + n + ".conv"], st["conv." + n])
-    st["v"] = torch.cat([st["v"], x["k" if m.v_from_k else "v"].view(T, m.kv_heads, m.vdim)])
+    v = x["k" if m.v_from_k else "v"].view(T, m.kv_heads, m.vdim)
+    st["v"] = torch.cat([st["v"], rotate(v, pos, m.v_rope) if m.v_rope else v])
     for n in ("q", "k"):
         if m.qk_norm == "all":
             x[n] = rms(x[n], eps) * p[f"{pre}{n}.norm"]
         elif m.qk_norm == "head":
             x[n] = (rms(x[n].view(T, -1, m.dim), eps) * p[f"{pre}{n}.norm"]).view(T, -1)
-    q = rotate(x["q"].view(T, m.heads, m.maps, m.dim), pos, m.rope)
-    st["k"] = torch.cat([st["k"], rotate(x["k"].view(T, m.kv_heads, m.maps, m.dim), pos, m.rope)])
+    q, k = rotate(x["q"].view(T, m.heads, m.maps, m.dim), pos, m.rope), rotate(x["k"].view(T, m.kv_heads, m.maps, m.dim), pos, m.rope)
+    if m.qk_norm == "rotated":
+        q, k = rms(q, eps), rms(k, eps)
+    st["k"] = torch.cat([st["k"], k])
     k, v = st["k"].repeat_interleave(rep, 1), st["v"].repeat_interleave(rep, 1)
-    sink = p[pre + "sink"] if m.sink else None
-    a = [sink_attention(q[:, :, j], k[:, :, j], v, start, m.window, m.keep_first, m.scale, sink) for j in range(m.maps)]
+    sink = p[pre + "sink"] if m.sink else torch.zeros(m.heads, dtype=h.dtype) if m.unit_sink else None
+    a = [sink_attention(q[:, :, j], k[:, :, j], v, start, m.window, m.keep_first, m.scale, sink, m.softcap) for j in range(m.maps)]
+    if m.v_rope:
+        a = [rotate(o, -pos, m.v_rope) for o in a]
     o = a[0] if m.maps == 1 else rms(a[0] - difference_weight(p, pre, m.diff) * a[1], eps) * (1 - m.diff)
     if m.gate:
         o = o * torch.sigmoid(h @ p[pre + "g"].T)[..., None]
     return o.reshape(T, m.heads * m.vdim) @ p[pre + "o"].T
 
 
-def dense_ffn(h: torch.Tensor, p: Params, pre: str) -> torch.Tensor:
-    return (silu(h @ p[pre + "gate"].T) * (h @ p[pre + "up"].T)) @ p[pre + "down"].T
+def lightning_mixer(h: torch.Tensor, p: Params, pre: str, m: LightningSpec, eps: float, st: dict) -> torch.Tensor:
+    T = h.shape[0]
+    q, k = (silu(h @ p[pre + n].T).view(T, m.heads, m.dim) for n in "qk")
+    o, st["S"] = decayed_products(q, k, silu(h @ p[pre + "v"].T).view(T, m.heads, m.vdim), m.decay, st["S"])
+    o = rms(o.reshape(T, m.heads * m.vdim), eps) * p[pre + "norm"] * torch.sigmoid(h @ p[pre + "g"].T)
+    return o @ p[pre + "o"].T
+
+
+def pair_mixer(h: torch.Tensor, p: Params, pre: str, m: PairSpec, eps: float, start: int, st: dict) -> torch.Tensor:
+    return (m.left_scale * attention_mixer(h, p, pre + "left.", m.left, eps, start, st)
+            + m.right_scale * lightning_mixer(h, p, pre + "right.", m.right, eps, st))
+
+
+def rglru_mixer(h: torch.Tensor, p: Params, pre: str, m: RglruSpec, st: dict) -> torch.Tensor:
+    """Gated linear recurrence on one branch, gelu on the other, multiplied."""
+    y = gelu_tanh(h @ p[pre + "y"].T + p[pre + "y.b"])
+    u, st["conv"] = causal_conv(h @ p[pre + "x"].T + p[pre + "x.b"], p[pre + "conv"], st["conv"])
+    u = u + p[pre + "conv.b"]
+    r, i = (torch.sigmoid(block_products(u, p[pre + n], p[pre + n + ".b"])) for n in ("ra", "ri"))
+    s, st["S"] = gated_recurrence(u, r, i, p[pre + "lam"], m.c, st["S"])
+    return (s * y) @ p[pre + "o"].T
+
+
+def dense_ffn(h: torch.Tensor, p: Params, pre: str, d: DenseSpec = DenseSpec(0)) -> torch.Tensor:
+    g, u = h @ p[pre + "gate"].T, h @ p[pre + "up"].T
+    if d.limit:
+        g, u = g.clamp_max(d.limit), u.clamp(-d.limit, d.limit)
+    return (g * torch.sigmoid(d.alpha * g) * (u + d.up_bias)) @ p[pre + "down"].T
 
 
 def feed_forward(h: torch.Tensor, p: Params, pre: str, spec) -> torch.Tensor:
-    """A parallel layer's: dense, or the routed experts with the shared one beside them."""
+    """Dense, or the routed experts with the shared one beside them."""
     if spec.router is None:
-        return dense_ffn(h, p, pre)
+        return dense_ffn(h, p, pre, spec.dense)
     y = routed_ffn(h, p, pre, spec.router)
-    return y if spec.dense is None else y + dense_ffn(h, p, pre + "shared.")
+    return y if spec.dense is None else y + dense_ffn(h, p, pre + "shared.", spec.dense)
+
+
+def depth_average(w: torch.Tensor, results: list[torch.Tensor]) -> torch.Tensor:
+    """The embedding rows and the layers' results so far, each times its weight."""
+    x = torch.zeros_like(results[0])
+    for a, y in zip(w, results, strict=True):
+        x = x + a * y
+    return x
 
 
 def join_embedding(x: torch.Tensor, x0: torch.Tensor, p: Params, t: int) -> torch.Tensor:
@@ -275,12 +371,20 @@ class HybridState:
 
     def __init__(self, cfg: ModelConfig, dtype: torch.dtype = torch.float32):
         self.length_ = 0
+        self.last_token = -1
         self.layers: list[dict] = []
-        self.marks: dict[int, list[dict]] = {}
+        self.marks: dict[int, tuple] = {}
         for spec in (cfg.layer_specs[r.layer] for r in cfg.layer_runs):
             z = lambda *s: torch.zeros(*s, dtype=dtype)               # noqa: E731
-            st = {} if spec.parallel else {"canon1": z(cfg.canon_taps - 1, cfg.hidden), "canon2": z(cfg.canon_taps - 1, cfg.hidden)}
+            st = {} if spec.parallel or spec.post_norm else {"canon1": z(cfg.canon_taps - 1, cfg.hidden), "canon2": z(cfg.canon_taps - 1, cfg.hidden)}
             m = spec.mixer
+            if isinstance(m, RglruSpec):
+                st.update(S=z(m.width), conv=z(m.conv - 1, m.width))
+                self.layers.append(st)
+                continue
+            if isinstance(m, PairSpec):
+                st.update(S=z(m.right.heads, m.right.dim, m.right.vdim))
+                m = m.left
             if isinstance(m, AttentionSpec):
                 st.update(k=z(0, m.kv_heads, m.maps, m.dim), v=z(0, m.kv_heads, m.vdim))
                 for n, c in (("q", m.q_channels), ("k", m.k_channels), ("v", m.v_channels)):
@@ -307,8 +411,12 @@ class HybridState:
             return
         if length not in self.marks:
             raise ValueError(f"recurrent state at {self.length_} tokens cannot return to {length}")
-        self.layers = [dict(st) for st in self.marks[length]]
+        layers, self.last_token = self.marks[length]
+        self.layers = [dict(st) for st in layers]
         self.length_ = length
+
+    def mark(self) -> None:
+        self.marks[self.length_] = ([dict(st) for st in self.layers], self.last_token)
 
 
 # ---- whole model ----------------------------------------------------------------------------------------------------
@@ -335,6 +443,12 @@ class HybridRefDecoder:
                 return x + y
             return x + (y + feed_forward(norm("norm2") if spec.two_norms else h, p, pre + "mlp.", spec))
 
+        if spec.post_norm:
+            m, norm = spec.mixer, lambda y, n: rms(y, cfg.rms_eps) * p[pre + n]                                   # noqa: E731
+            y = pair_mixer(x, p, pre + "mix.", m, cfg.rms_eps, start, st) if isinstance(m, PairSpec) else rglru_mixer(x, p, pre + "mix.", m, st)
+            x = x + norm(y, "norm1")
+            return x + norm(feed_forward(x, p, pre + "mlp.", spec), "norm2") if spec.has_ffn else x
+
         def sublayer(x, n, fn):
             h = group_rms(x, p[f"{pre}norm{n}"], cfg.norm_groups, cfg.rms_eps)
             y, st[f"canon{n}"] = causal_conv(h, p[f"{pre}canon{n}"], st[f"canon{n}"])
@@ -351,11 +465,18 @@ class HybridRefDecoder:
 
     def _run(self, tokens: torch.Tensor, kv: HybridState) -> torch.Tensor:
         e, start = self.p["embed"][tokens] * self.cfg.embed_scale, kv.length_
-        x = e
+        if self.cfg.bigram:
+            ids = tokens.tolist()
+            e = e + self.p["bigram"][bigram_rows(ids, kv.last_token, *self.cfg.bigram)]
+            kv.last_token = ids[-1] if ids else kv.last_token
+        x, results = e, [e]
         for n, r in enumerate(self.cfg.layer_runs):
             if r.join >= 0:
                 x = join_embedding(x, e, self.p, r.join)
             x = self._layer(r.layer, x + e if r.add_embedding else x, start, kv.layers[n])
+            if self.cfg.depth_average:
+                results.append(x)
+                x = depth_average(self.p[f"l{r.layer}.dwa"], results)
             if self.trace is not None:
                 self.trace.append(x)
         kv.length_ = start + tokens.shape[0]
@@ -364,13 +485,14 @@ class HybridRefDecoder:
     def hidden_states(self, tokens: torch.Tensor, kv: HybridState, embeds: tuple | None = None) -> torch.Tensor:
         if embeds is not None:
             raise ValueError("media rows are not part of this family")
-        kv.marks = {kv.length_: [dict(st) for st in kv.layers]}
+        kv.marks = {}
+        kv.mark()
         if tokens.shape[0] > self.mark_rows:
             return self._run(tokens, kv)
         out = []
         for t in range(tokens.shape[0]):
             out.append(self._run(tokens[t:t + 1], kv))
-            kv.marks[kv.length_] = [dict(st) for st in kv.layers]
+            kv.mark()
         return torch.cat(out)
 
     def head(self, x: torch.Tensor) -> torch.Tensor:
@@ -405,11 +527,41 @@ def init_hybrid_weights(cfg: ModelConfig, seed: int = 0, dtype: torch.dtype = to
             p[f"{x}e{e}.gate"], p[f"{x}e{e}.up"], p[f"{x}e{e}.down"] = w(r.ffn, H), w(r.ffn, H), w(H, r.ffn)
 
     H = cfg.hidden
-    p: Params = {"embed": w(cfg.vocab_size, H, s=1.0 / cfg.embed_scale), "final.norm": near_one(H), "head": w(cfg.vocab_size, H)}
+    p: Params = {"embed": w(cfg.vocab_size, H, s=1.0 / cfg.embed_scale), "final.norm": near_one(1)[0] if cfg.norm_scalar else near_one(H), "head": w(cfg.vocab_size, H)}
     if cfg.loop and cfg.loop_join:
         p["loop.in"], p["loop.step"] = w(H, 2 * H), w(cfg.loop[2], H, s=0.3)
+    if cfg.bigram:
+        p["bigram"] = w(cfg.bigram[0] + 1, H, s=0.7)
     for i, spec in enumerate(cfg.layer_specs):
         pre, m, r = f"l{i}.", spec.mixer, spec.router
+        if spec.post_norm:
+            x = pre + "mix."
+            for n in ("norm1", "norm2")[:1 + spec.has_ffn]:
+                p[pre + n] = 0.8 * near_one(1)[0] if cfg.norm_scalar else near_one(H)
+            if cfg.depth_average:
+                p[pre + "dwa"] = torch.cat([w(i + 1, s=0.3), near_one(1)])
+            if isinstance(m, PairSpec):
+                a, b = m.left, m.right
+                for n, c in (("q", a.q_channels), ("k", a.k_channels), ("v", a.v_channels)):
+                    p[f"{x}left.{n}"] = w(c, H)
+                p[x + "left.o"] = w(H, a.heads * a.vdim)
+                for n, c in (("q", b.heads * b.dim), ("k", b.heads * b.dim), ("v", b.heads * b.vdim), ("g", b.heads * b.vdim)):
+                    p[f"{x}right.{n}"] = w(c, H)
+                p[x + "right.o"], p[x + "right.norm"] = w(H, b.heads * b.vdim), near_one(b.heads * b.vdim)
+            else:
+                c = m.width
+                for n in "yx":
+                    p[x + n], p[f"{x}{n}.b"] = w(c, H), w(c, s=0.5)
+                p[x + "conv"], p[x + "conv.b"], p[x + "lam"] = w(c, m.conv), w(c, s=0.3), w(c, s=1.5) - 3
+                for n in ("ra", "ri"):
+                    p[x + n], p[f"{x}{n}.b"] = w(m.blocks, m.block, m.block), w(m.blocks, m.block, s=0.5)
+                p[x + "o"] = w(H, c)
+            if r is not None:
+                routed_weights(pre + "mlp.", r)
+            elif spec.dense is not None:
+                d, x = spec.dense, pre + "mlp."
+                p[x + "gate"], p[x + "up"], p[x + "down"] = w(d.ffn, H), w(d.ffn, H), w(H, d.ffn)
+            continue
         if spec.parallel:
             x, d = pre + "mix.", spec.dense
             p[pre + "norm1"] = near_one(H)
@@ -465,4 +617,5 @@ def bf16_params(p: Params, dtype: torch.dtype = torch.float32) -> Params:
 __all__ = ["HybridRefDecoder", "HybridState", "init_hybrid_weights", "bf16_params", "group_rms", "causal_conv", "rotate",
            "scaled_frequencies", "sink_attention", "difference_weight", "softcap", "attention_mixer", "dense_ffn", "feed_forward",
            "join_embedding", "window_attention", "delta_recurrence", "route", "route_by_logits", "routed_ffn", "latent_mixer", "delta_mixer",
-           "rms", "unit"]
+           "rms", "unit", "decayed_products", "block_products", "softplus", "gated_recurrence", "gelu_tanh", "bigram_rows", "route_by_sigmoid",
+           "lightning_mixer", "pair_mixer", "rglru_mixer", "depth_average"]
