@@ -32,6 +32,7 @@ class GemmArgs(C.Structure):
         ("rs_ranks", C.c_int), ("rs_rows_per_rank", C.c_int), ("rs_my_rank", C.c_int), ("n_signal_flags", C.c_int),
         ("n_wait_flags", C.c_int), ("reserved0", C.c_int),
         ("rs_out", C.c_void_p * 8), ("signal_flags", C.c_void_p * 8),
+        ("glu", C.c_int), ("glu_limit", C.c_float), ("glu_alpha", C.c_float), ("glu_bias", C.c_float),
     ]
 
 
@@ -79,28 +80,54 @@ class MoeLayout(C.Structure):
 class NormArgs(C.Structure):
     """cafd_norm_conv (csrc/hybrid_norm.cu)."""
     _fields_ = [(n, C.c_void_p) for n in ("tokens", "embed", "x_in", "y", "slot_w", "slot_idx", "ident", "w_b", "w", "base", "step",
-                                          "w2", "h2_out", "conv", "x_out", "h_out", "row_idx", "state", "state_in", "state_out", "q_start")]
-    _fields_ += [("slot_stride", C.c_longlong), ("state_off", C.c_longlong)]
-    _fields_ += [(n, C.c_int) for n in ("T", "H", "S", "ldy", "ldh", "ldb", "ldi", "groups", "taps", "top_k", "n_experts", "vocab", "run")]
+                                          "w2", "h2_out", "conv", "x_out", "h_out", "row_idx", "state", "state_in", "state_out", "q_start",
+                                          "rows2", "embed2", "past", "past_w", "past_out")]
+    _fields_ += [(n, C.c_longlong) for n in ("slot_stride", "state_off", "past_stride")]
+    _fields_ += [(n, C.c_int) for n in ("T", "H", "S", "ldy", "ldh", "ldb", "ldi", "groups", "taps", "top_k", "n_experts", "vocab", "run", "vocab2",
+                                        "n_past")]
     _fields_ += [(n, C.c_float) for n in ("eps", "w_off", "e_scale")]
+
+
+class BigramArgs(C.Structure):
+    """cafd_bigram_rows (csrc/hybrid_norm.cu)."""
+    _fields_ = [(n, C.c_void_p) for n in ("tokens", "q_start", "state_in", "state_out", "state", "rows")]
+    _fields_ += [(n, C.c_longlong) for n in ("slot_stride", "state_off", "mul_prev", "mul_cur", "buckets")]
+    _fields_ += [(n, C.c_int) for n in ("T", "S")]
+
+
+class RglruArgs(C.Structure):
+    """cafd_rglru_* (csrc/rglru.cu)."""
+    _fields_ = [(n, C.c_void_p) for n in ("proj", "y_bias", "x_bias", "conv_w", "conv_b", "lam", "w", "gate_bias", "u", "gates", "out", "carry",
+                                          "state", "state_in", "state_out", "q_start")]
+    _fields_ += [(n, C.c_longlong) for n in ("slot_stride", "s_off", "c_off")]
+    _fields_ += [(n, C.c_int) for n in ("T", "S", "ld", "x_off", "y_off", "width", "blocks", "taps", "u_pitch", "t_pad", "ldo", "max_q")]
+    _fields_ += [("c", C.c_float)]
+
+
+class LightningArgs(C.Structure):
+    """cafd_lightning_* (csrc/lightning.cuh)."""
+    _fields_ = [(n, C.c_void_p) for n in ("proj", "decay", "norm_w", "raw", "out", "scratch", "state", "state_in", "state_out", "q_start")]
+    _fields_ += [(n, C.c_longlong) for n in ("slot_stride", "s_off", "scratch_bytes")]
+    _fields_ += [(n, C.c_int) for n in ("T", "S", "ld", "q_off", "k_off", "v_off", "g_off", "heads", "dim", "vdim", "ldo", "out_vd", "max_q")]
+    _fields_ += [("eps", C.c_float)]
 
 
 class ConvRope(C.Structure):
     """cafd_conv_rope_kv (csrc/conv_rope.cu)."""
     _fields_ = [(n, C.c_void_p) for n in ("proj", "conv_w", "table", "slots", "q_start", "state_in", "state_out", "state", "q_out",
-                                          "k_cache", "v_cache", "q_norm", "k_norm")]
+                                          "k_cache", "v_cache", "q_norm", "k_norm", "v_table")]
     _fields_ += [("slot_stride", C.c_longlong), ("state_off", C.c_longlong)]
     _fields_ += [(n, C.c_int) for n in ("T", "S", "ld", "q_off", "k_off", "v_off", "nq", "nk", "nv", "maps_dim", "dim", "vdim", "kv_heads",
                                         "rot", "taps", "run", "norm", "halves", "v_from_k", "units")]
-    _fields_ += [("eps", C.c_float)]
+    _fields_ += [("eps", C.c_float), ("rot_sq", C.c_float)]
 
 
 class PagedAttn(C.Structure):
     """cafd_paged_attn (csrc/attention_any.cu)."""
-    _fields_ = [(n, C.c_void_p) for n in ("q", "k_cache", "v_cache", "page_table", "positions", "q_start", "out", "sink", "gate")]
+    _fields_ = [(n, C.c_void_p) for n in ("q", "k_cache", "v_cache", "page_table", "positions", "q_start", "out", "sink", "gate", "v_table")]
     _fields_ += [(n, C.c_int) for n in ("T", "S", "heads", "kv_heads", "maps", "dim", "vdim", "window", "keep", "max_pages", "ldo",
                                         "head_pitch", "heads_per_block", "gate_ld")]
-    _fields_ += [(n, C.c_float) for n in ("scale", "lam", "out_scale", "eps")]
+    _fields_ += [(n, C.c_float) for n in ("scale", "lam", "out_scale", "eps", "cap")]
 
 
 class LatentPrep(C.Structure):
@@ -222,6 +249,10 @@ def cuda_lib():
         _sig(lib, "cafd_sample_rows", [P, I, I, P, P, I, P, P, P])
         _sig(lib, "cafd_accept_prefix", [P, P, P, I, P, P, P])
         _sig(lib, "cafd_norm_conv", [C.POINTER(NormArgs), I, P])
+        _sig(lib, "cafd_bigram_rows", [C.POINTER(BigramArgs), P])
+        for n in ("cafd_rglru_conv", "cafd_rglru_scan"):
+            _sig(lib, n, [C.POINTER(RglruArgs), I, P])
+        _sig(lib, "cafd_lightning_step", [C.POINTER(LightningArgs), I, P])
         _sig(lib, "cafd_rope_table", [P, P, P, I, I, F, P])
         _sig(lib, "cafd_conv_rope_kv", [C.POINTER(ConvRope), I, P])
         _sig(lib, "cafd_softcap", [P, I, I, C.c_longlong, F, P])
@@ -229,7 +260,7 @@ def cuda_lib():
         _sig(lib, "cafd_delta_chunked", [C.POINTER(DeltaArgs), P, C.c_longlong, P])
         _sig(lib, "cafd_delta_chunk_bytes", [I, I, I], C.c_longlong)
         _sig(lib, "cafd_swap_ids", [P, P, I, P])
-        _sig(lib, "cafd_gemm_f32", [P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, P])
+        _sig(lib, "cafd_gemm_f32", [P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, F, F, F, P])
         _sig(lib, "cafd_latent_prep", [C.POINTER(LatentPrep), I, P])
         _sig(lib, "cafd_latent_attn", [C.POINTER(LatentAttn), I, P])
         _sig(lib, "cafd_latent_gate", [P, P, I, I, I, I, I, I, I, P])

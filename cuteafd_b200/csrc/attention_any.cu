@@ -1,6 +1,7 @@
 // Softmax attention over paged keys and values at any head sizes, with a sliding window and kept first tokens, and with one or
-// two score maps per head; a head may have a sink and an output gate (the tensor-core kernels of attention_prefill.cu and attention_decode.cu serve 128-wide key and value
-// rows; this file serves every other size and the fp32 engines).
+// two score maps per head; scores may be capped, a head may have a sink, an output gate and an output that is turned back by its
+// position (the tensor-core kernels of attention_prefill.cu and attention_decode.cu serve 128-wide key and value rows; this file
+// serves every other size and the fp32 engines).
 //
 // One block per (token, kv head, run of its query heads).  Keys are walked in tiles that start at multiples of 32, first those
 // of the kept tokens, then those of the window, so a row's arithmetic depends on its own position only.  Scores, softmax and
@@ -22,8 +23,10 @@ struct PagedAttn {
   void* out;                  // [T, ldo] E: head h's values at h * head_pitch
   const float* sink;          // [heads] or null: exp(sink) joins the denominator; one map only
   const void* gate;           // row t, head h: E gate[t * gate_ld + h], the head's values are multiplied by its sigmoid; or null; one map only
+  const float2* v_table;      // [T, vdim / 2] cos, sin: a head's output is turned back by them, pairs (i, i + vdim / 2); or null; one map only
   int T, S, heads, kv_heads, maps, dim, vdim, window, keep, max_pages, ldo, head_pitch, heads_per_block, gate_ld;
   float scale, lambda, out_scale, eps;
+  float cap;                  // scores are cap * tanh(score / cap); 0 = they are not
 };
 
 constexpr int kAnyKeys = 32;
@@ -47,7 +50,7 @@ __global__ void __launch_bounds__(kAnyThreads) paged_attn_kernel(const PagedAttn
   float* sm_m = sp + max_rows * kAnyKeys;       // running maximum, sum and correction per row
   float* sm_l = sm_m + max_rows;
   float* sm_c = sm_l + max_rows;
-  float* so = sm_c + max_rows;                  // [rows][vdim] (two maps)
+  float* so = sm_c + max_rows;                  // [rows][vdim] (two maps, or outputs to turn back)
   const int seq = [&] {
     int s = 0, hi = p.S;
     while (hi - s > 1) {
@@ -89,7 +92,9 @@ __global__ void __launch_bounds__(kAnyThreads) paged_attn_kernel(const PagedAttn
       const float* b = sk + j * kp + (r % p.maps) * p.dim;
       float s = 0.f;
       for (int d = 0; d < p.dim; ++d) s = fmaf(a[d], b[d], s);
-      sp[e] = (at <= pos && (at >= lo || at < keep)) ? s * p.scale : -INFINITY;
+      s *= p.scale;
+      if (p.cap > 0.f) s = p.cap * tanhf(s / p.cap);
+      sp[e] = (at <= pos && (at >= lo || at < keep)) ? s : -INFINITY;
     }
     __syncthreads();
     for (int r = warp; r < rows; r += kAnyThreads / 32) {
@@ -127,14 +132,26 @@ __global__ void __launch_bounds__(kAnyThreads) paged_attn_kernel(const PagedAttn
     if (e < n_acc) {
       const int r = e / p.vdim, d = e - r * p.vdim;
       const float l = p.sink ? sm_l[r] + expf(p.sink[h0 + r] - sm_m[r]) : sm_l[r];
-      float v[1] = {acc[k] / l};
+      float v[1] = {acc[k] / l * (p.maps == 1 ? p.out_scale : 1.f)};
       if (p.gate) v[0] /= 1.0f + expf(-ld_e<E>(static_cast<const E*>(p.gate) + static_cast<size_t>(t) * p.gate_ld + h0 + r));
-      if (p.maps == 1) store_vec<E, 1>(out + (h0 + r) * p.head_pitch + d, v);
+      if (p.maps == 1 && !p.v_table) store_vec<E, 1>(out + (h0 + r) * p.head_pitch + d, v);
       else so[e] = v[0];
     }
   }
-  if (p.maps == 1) return;
+  if (p.maps == 1 && !p.v_table) return;
   __syncthreads();
+  if (p.v_table) {
+    const int vh = p.vdim >> 1;
+    for (int e = tid; e < n_acc; e += kAnyThreads) {
+      const int r = e / p.vdim, d = e - r * p.vdim;
+      const bool first = d < vh;
+      const float2 a = p.v_table[static_cast<size_t>(t) * vh + (first ? d : d - vh)];
+      const float o = so[first ? e + vh : e - vh];
+      float v[1] = {first ? so[e] * a.x + o * a.y : so[e] * a.x - o * a.y};
+      store_vec<E, 1>(out + (h0 + r) * p.head_pitch + d, v);
+    }
+    return;
+  }
   for (int h = warp; h < nh; h += kAnyThreads / 32) {
     float* a = so + 2 * h * p.vdim;
     const float* b = a + p.vdim;
@@ -161,7 +178,7 @@ extern "C" int cafd_paged_attn(const PagedAttn* args, int is_f32, cafd_stream_t 
   if (p.T <= 0) return 0;
   if (p.S < 1 || p.kv_heads < 1 || p.heads % p.kv_heads || p.maps < 1 || p.maps > 2 || p.dim < 1 || p.vdim < 1 || p.window < 0 || p.keep < 0 ||
       p.maps * p.vdim > kAnyAcc * kAnyThreads || p.head_pitch < p.vdim || p.ldo < (p.heads - 1) * p.head_pitch + p.vdim ||
-      (p.maps == 2 && (p.sink || p.gate)) || (p.gate && p.gate_ld < p.heads))
+      (p.maps == 2 && (p.sink || p.gate || p.v_table)) || (p.v_table && p.vdim % 2) || (p.gate && p.gate_ld < p.heads))
     return -10;
   if (p.window == 0) p.keep = 0;
   const int group = p.heads / p.kv_heads;
@@ -170,7 +187,7 @@ extern "C" int cafd_paged_attn(const PagedAttn* args, int is_f32, cafd_stream_t 
   auto bytes = [&](int h) {
     const int rows = h * p.maps;
     return static_cast<size_t>(rows * p.dim + kAnyKeys * ((p.maps * p.dim) | 1) + kAnyKeys * p.vdim + rows * kAnyKeys + 3 * rows +
-                               (p.maps == 2 ? rows * p.vdim : 0)) * 4;
+                               (p.maps == 2 || p.v_table ? rows * p.vdim : 0)) * 4;
   };
   while (hpb > 1 && bytes(hpb) > 200 * 1024) --hpb;
   if (bytes(hpb) > 200 * 1024) return -12;

@@ -73,6 +73,10 @@ typedef struct {
   int reserved0;
   void* rs_out[8];
   uint32_t* signal_flags[8];
+  // dual mode, cafd_gemm only.  glu 0: silu(g) * u.  glu 1: g' sigmoid(glu_alpha g') (u' + glu_bias) with g' = min(g, glu_limit) and
+  // u' = min(max(u, -glu_limit), glu_limit).
+  int glu;
+  float glu_limit, glu_alpha, glu_bias;
 } cafd_gemm_args;
 
 int cafd_gemm(const cafd_gemm_args* a, cafd_stream_t stream);

@@ -297,6 +297,16 @@ __device__ __forceinline__ float fast_exp2(float x) {
   asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
   return y;
 }
+// Gated unit of a feed-forward: kind 0 silu(g) * u, kind 1 cut off at a limit, with a slope and an offset (uniform over a launch).
+struct Glu {
+  int kind;
+  float limit, alpha, bias;
+};
+__device__ __forceinline__ float clipped_glu(float g, float u, const Glu& a) {
+  g = fminf(g, a.limit);
+  u = fminf(fmaxf(u, -a.limit), a.limit);
+  return g / (1.0f + __expf(-a.alpha * g)) * (u + a.bias);
+}
 __device__ __forceinline__ float silu(float x) { return x / (1.0f + __expf(-x)); }
 
 __device__ __forceinline__ float warp_sum(float v) {

@@ -7,8 +7,8 @@
 //   conv_rope_kv     pairs (2i, 2i + 1), no norm: four channels per thread walking a run of tokens, the convolution's earlier
 //                    inputs in registers
 //   conv_rope_kv_any the same for any head sizes and any number of taps: one channel per thread and token
-//   conv_norm_rope_kv  with norms (per head or over the whole projection), pairs of either kind, values of their own or the
-//                    convolved keys: a block walks a run of tokens, the projected rows in a ring in shared memory
+//   conv_norm_rope_kv  with norms (per head or over the whole projection), pairs of either kind, values of their own (rotated or
+//                    not) or the convolved keys: a block walks a run of tokens, the projected rows in a ring in shared memory
 //   conv_norm_rope_128 the same for bf16 heads of 128: a warp owns whole heads, four channels per lane, and walks a run of tokens
 //                    with everything in registers; partners and square sums go by shuffles
 //
@@ -33,8 +33,9 @@ struct ConvRope {
   void* q_out;                // [T, q channels] E
   void* k_cache;              // [pages, kv heads, 64, maps * dim] E
   void* v_cache;              // [pages, kv heads, 64, vdim] E
-  const float* q_norm;        // [dim] (norm 1) or [nq] (norm 2)
+  const float* q_norm;        // [dim] (norm 1, null = no weights) or [nq] (norm 2)
   const float* k_norm;        // [dim] or [nk]
+  const float2* v_table;      // [T, vdim / 2] cos, sin: values are rotated over their whole width, pairs (i, i + vdim / 2); null = not
   long long slot_stride, state_off;
   int T, S, ld, q_off, k_off, v_off, nq, nk, nv, maps_dim, dim, vdim, kv_heads, rot, taps, run;
   int norm;                   // 0 none, 1 per head (and map), 2 over all of q and all of k
@@ -42,6 +43,7 @@ struct ConvRope {
   int v_from_k;               // nv = 0: the values are the convolved keys before norm and rotation
   int units;                  // heads of q, k and v one block works on
   float eps;
+  float rot_sq;               // norm 1: weight of the rotated dimensions' squares (a norm taken after a rotation that scales by its root)
 };
 
 __global__ void __launch_bounds__(256) rope_table_kernel(const int* __restrict__ positions, const float* __restrict__ freq, float2* __restrict__ out,
@@ -276,6 +278,7 @@ __global__ void __launch_bounds__(kCnrThreads) conv_norm_rope_kv_kernel(const Co
   const int vpu = p.dim / V;                                             // vectors of a head of q or k
   const bool lanes = p.norm && vpu <= 32 && (vpu & (vpu - 1)) == 0;
   const int half = p.rot >> 1;
+  const int nrot = p.v_table ? n : nqk;                                  // channels that pass the second half of a token's work
   const int r0 = blockIdx.x * p.run, r1 = min(p.T, r0 + p.run);
   auto fetch = [&](int row) {
     if (row < r1) {
@@ -338,7 +341,7 @@ __global__ void __launch_bounds__(kCnrThreads) conv_norm_rope_kv_kernel(const Co
             for (int e = 0; e < V; ++e) v[e] = fmaf(w[e], x[e], v[e]);
           }
         }
-        if (i * V < nqk) {
+        if (i * V < nrot) {
           store_vec<float, V>(y + i * V, v);
           if (p.v_from_k && c >= p.nq && slot >= 0) {
             const int cc = c - p.nq, g = cc / p.vdim;
@@ -362,17 +365,18 @@ __global__ void __launch_bounds__(kCnrThreads) conv_norm_rope_kv_kernel(const Co
         float s = 0.f;
 #pragma unroll
         for (int e = 0; e < V; ++e) s += v[e] * v[e];
+        if ((i % vpu) * V < p.rot) s *= p.rot_sq;                        // (a vector lies on one side of the rotated dimensions' end)
         for (int o = 1; o < vpu; o <<= 1) s += __shfl_xor_sync(0xffffffffu, s, o);
         if (i * V < nqk && i % vpu == 0) ss[i / vpu] = s;
       }
     }
     __syncthreads();
-    if (nqk <= 0) continue;
-    const int nu = nqk / p.dim, nuq = max(0, min(u1, uq) - u0);          // heads of q and k here, of q among them
+    if (nrot <= 0) continue;
+    const int nu = max(0, nqk) / p.dim, nuq = max(0, min(u1, uq) - u0);          // heads of q and k here, of q among them
     if (p.norm && !lanes) {
       for (int u = warp; u < nu; u += kCnrThreads / 32) {
         float s = 0.f;
-        for (int d = lane; d < p.dim; d += 32) s = fmaf(y[u * p.dim + d], y[u * p.dim + d], s);
+        for (int d = lane; d < p.dim; d += 32) s = fmaf(y[u * p.dim + d] * (d < p.rot ? p.rot_sq : 1.f), y[u * p.dim + d], s);
         s = warp_sum(s);
         if (lane == 0) ss[u] = s;
       }
@@ -393,13 +397,29 @@ __global__ void __launch_bounds__(kCnrThreads) conv_norm_rope_kv_kernel(const Co
       inv_k = 1.0f / sqrtf(b / static_cast<float>(p.nk) + p.eps);
     }
     const float2* cs = p.table + static_cast<size_t>(t) * half;
-    for (int i = tid; i * V < nqk; i += kCnrThreads) {
+    for (int i = tid; i * V < nrot; i += kCnrThreads) {
+      if (i * V >= nqk) {                       // a value (V divides vdim / 2)
+        const int c = c0 + i * V, d = (c - p.nq - p.nk) % p.vdim, vh = p.vdim >> 1;
+        const bool first = d < vh;
+        const float2* a = p.v_table + static_cast<size_t>(t) * vh + (first ? d : d - vh);
+        float v[V], o[V];
+        load_vec<float, V>(y + i * V, v);
+        load_vec<float, V>(y + i * V + (first ? vh : -vh), o);
+#pragma unroll
+        for (int e = 0; e < V; ++e) v[e] = first ? v[e] * a[e].x - o[e] * a[e].y : v[e] * a[e].x + o[e] * a[e].y;
+        if (E* dst = conv_rope_dest<E>(p, t, slot, c)) store_vec<E, V>(dst, v);
+        continue;
+      }
       const int c = c0 + i * V, u = i * V / p.dim, d = i * V - u * p.dim;
       const bool is_q = c < p.nq;
-      const float* wn = !p.norm ? nullptr : p.norm == 1 ? (is_q ? p.q_norm : p.k_norm) + d : is_q ? p.q_norm + c : p.k_norm + c - p.nq;
+      const float* wn = !p.norm || !p.q_norm ? nullptr : p.norm == 1 ? (is_q ? p.q_norm : p.k_norm) + d : is_q ? p.q_norm + c : p.k_norm + c - p.nq;
       const float inv = p.norm == 1 ? 1.0f / sqrtf(ss[u] / static_cast<float>(p.dim) + p.eps) : is_q ? inv_q : inv_k;
       auto normed = [&](int at, float (&v)[V]) {                         // the normed channels `at` places from this thread's
         load_vec<float, V>(y + i * V + at, v);
+        if (p.norm && !wn) {
+#pragma unroll
+          for (int e = 0; e < V; ++e) v[e] *= inv;
+        }
         if (wn) {
           float w[V];
           load_vec<float, V>(wn + at, w);
@@ -478,7 +498,7 @@ __global__ void __launch_bounds__(kAll ? 512 : 128, kAll ? 1 : 4) conv_norm_rope
   for (int h = 0; h < (kAll ? NH : 1); ++h) {
 #pragma unroll
     for (int e = 0; e < V; ++e) wn[h][e] = 1.f;
-    if (p.norm && (is_q || is_k)) load_vec<float, V>((is_q ? p.q_norm + (kAll ? c : d) : p.k_norm + (kAll ? c - p.nq : d)) + h * 128, wn[h]);
+    if (p.norm && p.q_norm && (is_q || is_k)) load_vec<float, V>((is_q ? p.q_norm + (kAll ? c : d) : p.k_norm + (kAll ? c - p.nq : d)) + h * 128, wn[h]);
   }
   pdl_wait();
   pdl_trigger();
@@ -601,6 +621,14 @@ __global__ void __launch_bounds__(kAll ? 512 : 128, kAll ? 1 : 4) conv_norm_rope
         const size_t cell = slot < 0 ? 0 : (static_cast<size_t>(slot >> 6) * p.kv_heads) * 8192 + (slot & 63) * 128 + d;
         const int g = u0 + h - uq - (is_k ? 0 : uk);                       // key or value head
         if (!is_q && !is_k) {
+          if (p.v_table) {                      // pairs (i, i + 64): lanes 16 apart
+            const float2* a = p.v_table + static_cast<size_t>(row) * 64 + (lane & 15) * V;
+#pragma unroll
+            for (int e = 0; e < V; ++e) {
+              const float o = __shfl_xor_sync(0xffffffffu, y[e], 16);
+              y[e] = lane < 16 ? y[e] * a[e].x - o * a[e].y : y[e] * a[e].x + o * a[e].y;
+            }
+          }
           if (slot >= 0) store_vec<__nv_bfloat16, V>(static_cast<__nv_bfloat16*>(p.v_cache) + cell + static_cast<size_t>(g) * 8192, y);
           continue;
         }
@@ -613,6 +641,7 @@ __global__ void __launch_bounds__(kAll ? 512 : 128, kAll ? 1 : 4) conv_norm_rope
             float s = 0.f;
 #pragma unroll
             for (int e = 0; e < V; ++e) s = fmaf(y[e], y[e], s);
+            if (d < p.rot) s *= p.rot_sq;
             inv = 1.0f / sqrtf(warp_sum(s) * (1.0f / 128.0f) + p.eps);
           }
 #pragma unroll
@@ -779,7 +808,7 @@ static int dispatch_conv_norm_rope(const ConvRope& p, cudaStream_t st) {
   auto fits = [&](int v) {
     const int pair = p.halves ? p.rot / 2 : p.rot;
     return p.dim % v == 0 && p.vdim % v == 0 && p.ld % v == 0 && p.q_off % v == 0 && p.k_off % v == 0 && p.v_off % v == 0 && pair % v == 0 &&
-           p.state_off % 4 == 0 && p.slot_stride % 4 == 0;
+           p.state_off % 4 == 0 && p.slot_stride % 4 == 0 && (!p.v_table || (p.vdim / 2) % v == 0);
   };
   return fits(8) ? launch_conv_norm_rope<E, 8>(p, st) : fits(4) ? launch_conv_norm_rope<E, 4>(p, st) : launch_conv_norm_rope<E, 1>(p, st);
 }
@@ -801,10 +830,10 @@ extern "C" int cafd_conv_rope_kv(const ConvRope* p, int is_f32, cafd_stream_t s)
   if (p->dim <= 0 || p->vdim <= 0 || p->rot < 0 || p->rot % 2 || p->rot > p->dim || p->maps_dim % p->dim || p->nk != p->kv_heads * p->maps_dim ||
       p->nv != (p->v_from_k ? 0 : p->kv_heads * p->vdim) || p->nq % p->dim || p->norm < 0 || p->norm > 2)
     return -10;
-  if ((p->norm && (!p->q_norm || !p->k_norm)) || (p->v_from_k && (p->vdim != p->dim || p->maps_dim != p->dim))) return -10;
+  if ((p->norm && (!p->q_norm != !p->k_norm || (p->norm == 2 && !p->q_norm))) || (p->v_table && (p->vdim % 2 || p->v_from_k)) || (p->v_from_k && (p->vdim != p->dim || p->maps_dim != p->dim))) return -10;
   if (p->conv_w && (p->taps < 1 || !p->q_start || p->S < 1 || (p->taps > 1 && (!p->state || !p->state_in || !p->state_out)))) return -10;
   cudaStream_t st = static_cast<cudaStream_t>(s);
-  if (p->norm || p->halves || p->v_from_k) return is_f32 ? dispatch_conv_norm_rope<float>(*p, st) : dispatch_conv_norm_rope<__nv_bfloat16>(*p, st);
+  if (p->norm || p->halves || p->v_from_k || p->v_table) return is_f32 ? dispatch_conv_norm_rope<float>(*p, st) : dispatch_conv_norm_rope<__nv_bfloat16>(*p, st);
   return is_f32 ? launch_conv_rope<float>(*p, st) : launch_conv_rope<__nv_bfloat16>(*p, st);
 }
 

@@ -18,6 +18,7 @@ struct GemmF32 {
   const int* tile_row0;
   const int* num_x_tiles;
   int k, n, x_rows, ldx, ldo, rows_per_expert, tile_rows, sub_tiles;
+  Glu glu;
 };
 
 template <bool kDual>
@@ -73,7 +74,15 @@ __global__ void __launch_bounds__(kF32Threads) gemm_f32_kernel(const GemmF32 p) 
       const int col = col0 + tc + j;
       if (col >= p.n) continue;
       float v = acc[0][i][j];
-      if (kDual) v = v / (1.0f + expf(-v)) * acc[kDual ? 1 : 0][i][j];
+      if (kDual) {
+        float u = acc[kDual ? 1 : 0][i][j], alpha = 1.f;
+        if (p.glu.kind) {
+          v = fminf(v, p.glu.limit);
+          u = fminf(fmaxf(u, -p.glu.limit), p.glu.limit) + p.glu.bias;
+          alpha = p.glu.alpha;
+        }
+        v = v / (1.0f + expf(-alpha * v)) * u;
+      }
       p.out[static_cast<size_t>(dst) * p.ldo + col] = v;
     }
   }
@@ -83,14 +92,16 @@ __global__ void __launch_bounds__(kF32Threads) gemm_f32_kernel(const GemmF32 p) 
 
 using namespace cafd;
 
-// out[row_dst[r] or r] = x[r] @ w[expert of r's tile].T (with w1: silu(x @ w0.T) * (x @ w1.T)).  Dense: tile_expert,
+// out[row_dst[r] or r] = x[r] @ w[expert of r's tile].T (with w1: the gated unit of both products, cafd_gemm_args.glu).  Dense: tile_expert,
 // tile_row0, num_x_tiles and row_dst null, max_x_tiles = 0.  Grouped: tiles of tile_rows rows as the MoE plan writes them.
 extern "C" int cafd_gemm_f32(const float* w0, const float* w1, const float* x, float* out, const int* row_dst, const int* tile_expert,
                              const int* tile_row0, const int* num_x_tiles, int k, int n, int x_rows, int ldx, int ldo,
-                             int rows_per_expert, int max_x_tiles, int tile_rows, cafd_stream_t s) {
+                             int rows_per_expert, int max_x_tiles, int tile_rows, int glu, float glu_limit, float glu_alpha, float glu_bias,
+                             cafd_stream_t s) {
   if (x_rows <= 0 || n <= 0) return 0;
   if (!w0 || !x || !out || k <= 0) return -10;
-  GemmF32 p{w0, w1, x, out, row_dst, tile_expert, tile_row0, num_x_tiles, k, n, x_rows, ldx, ldo, rows_per_expert, tile_rows, 1};
+  GemmF32 p{w0, w1, x, out, row_dst, tile_expert, tile_row0, num_x_tiles, k, n, x_rows, ldx, ldo, rows_per_expert, tile_rows, 1,
+            Glu{glu, glu_limit, glu_alpha, glu_bias}};
   int tiles = max_x_tiles;
   if (!tile_row0) {
     p.tile_rows = kF32Tile;

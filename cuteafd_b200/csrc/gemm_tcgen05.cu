@@ -60,6 +60,7 @@ struct GemmDev {
   int x_tiles_static;
   int w_tiles;
   int out_f32;
+  Glu glu;
 };
 
 template <bool kSwap, bool kDual, int kBX, int kBW>
@@ -303,8 +304,13 @@ gemm_kernel(const __grid_constant__ CUtensorMap tm_w0, const __grid_constant__ C
               uint32_t u[32];
               tmem_ld_32x32(t0 + kBW + c0 + 32 * h, u);
               tmem_ld_wait();
+              if (p.glu.kind == 0) {
 #pragma unroll
-              for (int j = 0; j < 32; ++j) v[j] = silu(__uint_as_float(r[j])) * __uint_as_float(u[j]) * scale;
+                for (int j = 0; j < 32; ++j) v[j] = silu(__uint_as_float(r[j])) * __uint_as_float(u[j]) * scale;
+              } else {
+#pragma unroll
+                for (int j = 0; j < 32; ++j) v[j] = clipped_glu(__uint_as_float(r[j]), __uint_as_float(u[j]), p.glu) * scale;
+              }
             } else {
               tmem_ld_wait();
 #pragma unroll
@@ -401,7 +407,7 @@ gemm_kernel(const __grid_constant__ CUtensorMap tm_w0, const __grid_constant__ C
                 }
             }
 #pragma unroll
-            for (int j = 0; j < 16; ++j) v[j] = kDual ? silu(g[j]) * u[j] : g[j];
+            for (int j = 0; j < 16; ++j) v[j] = !kDual ? g[j] : p.glu.kind == 0 ? silu(g[j]) * u[j] : clipped_glu(g[j], u[j], p.glu);
           } else {
             uint32_t r[16];
             tmem_ld_32x16(t0 + c0, r);
@@ -410,7 +416,8 @@ gemm_kernel(const __grid_constant__ CUtensorMap tm_w0, const __grid_constant__ C
               tmem_ld_32x16(t0 + kBX + c0, u);
               tmem_ld_wait();
 #pragma unroll
-              for (int j = 0; j < 16; ++j) v[j] = silu(__uint_as_float(r[j])) * __uint_as_float(u[j]);
+              for (int j = 0; j < 16; ++j)
+                v[j] = p.glu.kind == 0 ? silu(__uint_as_float(r[j])) * __uint_as_float(u[j]) : clipped_glu(__uint_as_float(r[j]), __uint_as_float(u[j]), p.glu);
             } else {
               tmem_ld_wait();
 #pragma unroll
@@ -518,6 +525,7 @@ static int launch(const cafd_gemm_args* a, cudaStream_t stream) {
   p.w1_row_offset = a->w1_row_offset;
   p.w_tiles = (a->n_features + kBW - 1) / kBW;
   p.out_f32 = a->out_f32;
+  p.glu = Glu{a->glu, a->glu_limit, a->glu_alpha, a->glu_bias};
   p.splitk_scratch = nullptr;
   p.splitk_tickets = nullptr;
   p.splitk_max_units = 0;

@@ -1,11 +1,13 @@
 // Residual stream of the per-layer hybrid decoders: everything between two sublayers in one launch.
 //
-//   x   = embed[token] * e_scale            (first launch)       or the fp32 residual of the previous launch, or their sum
-//                                           (a loop's next pass)
+//   x   = embed[token] * e_scale            (first launch; a second table's row may be added)  or the fp32 residual of the previous
+//                                           launch, or their sum (a loop's next pass)
 //   x  += step                              one vector for all tokens (optional)
 //   x  += groupnorm(y) * w_b                y = a mixer's output rows, or the routed experts' rows summed here:
 //                                           sum over slots of weight * (expert row, or the input row for an identity slot);
 //                                           without w_b: x += y; `base` rows are added to the routed sum as they are
+//   x   = sum_j past_w[j] * past[j] + past_w[n] * x       average over depth (optional): earlier results of the same rows; x itself is
+//                                           kept for later ones first
 //   h   = groupnorm(x) * (w + w_off)        RMS norm in equal runs of channels, each with its own root mean square
 //                                           (without w: h = x); a second weight vector gives a second output of the same norm
 //   out = h + sum_j c[j] * h(t - taps + 1 + j)     causal convolution over time per channel (optional)
@@ -44,8 +46,13 @@ struct NormArgs {
   const int* state_in;        // [S] slot read
   const int* state_out;       // [S] slot written
   const int* q_start;         // [S + 1]
-  long long slot_stride, state_off;
-  int T, H, S, ldy, ldh, ldb, ldi, groups, taps, top_k, n_experts, vocab, run;   // ldy, ldh, ldb, ldi: elements from row to row of y, of h_out, of base, of ident
+  const int* rows2;           // [T] rows of the second table, with embed only; null = none
+  const void* embed2;         // [vocab2, H] E
+  const float* past;          // [n_past][T, H], past_stride floats from one to the next; only without a convolution
+  const float* past_w;        // [n_past + 1], null = no average
+  float* past_out;            // [T, H] or null: x before the average
+  long long slot_stride, state_off, past_stride;
+  int T, H, S, ldy, ldh, ldb, ldi, groups, taps, top_k, n_experts, vocab, run, vocab2, n_past;   // ldy, ldh, ldb, ldi: elements from row to row of y, of h_out, of base, of ident
   float eps, w_off, e_scale;
 };
 
@@ -175,7 +182,7 @@ __device__ __forceinline__ void group_inv(const float (&v)[KV][V], float (&inv)[
   }
 }
 
-template <typename E, int V, int KV, int MAXT, bool kSlots, int kMaxThreads, int kMinBlocks>
+template <typename E, int V, int KV, int MAXT, bool kSlots, bool kPast, int kMaxThreads, int kMinBlocks>
 __global__ void __launch_bounds__(kMaxThreads, kMinBlocks) norm_conv_kernel(const NormArgs a) {
   extern __shared__ float sm[];
   // routed rows of a token whose loads are in flight together (prompts: several blocks per SM share the registers)
@@ -304,6 +311,20 @@ __global__ void __launch_bounds__(kMaxThreads, kMinBlocks) norm_conv_kernel(cons
           for (int e = 0; e < V; ++e) x[k][e] = fmaf(v[e], a.e_scale, x[k][e]);
         }
       }
+      if (a.rows2) {
+        const int r2 = min(max(a.rows2[row], 0), a.vocab2 - 1);
+        src = static_cast<const E*>(a.embed2) + static_cast<size_t>(r2) * a.H;
+#pragma unroll
+        for (int k = 0; k < KV; ++k) {
+          const int i = tid + k * nt;
+          if (i < nvec) {
+            float v[V];
+            load_vec<E, V>(src + i * V, v);
+#pragma unroll
+            for (int e = 0; e < V; ++e) x[k][e] += v[e];
+          }
+        }
+      }
     }
     if (a.step) {
 #pragma unroll
@@ -385,6 +406,39 @@ __global__ void __launch_bounds__(kMaxThreads, kMinBlocks) norm_conv_kernel(cons
           load_vec<E, V>(static_cast<const E*>(a.w_b) + i * V, wb);
 #pragma unroll
           for (int e = 0; e < V; ++e) x[k][e] += y[k][e] * inv[k] * wb[e];
+        }
+      }
+    }
+    if constexpr (kPast) {
+      constexpr int kBatch = 4;                 // earlier results whose loads are in flight together
+      const float wx = a.past_w[a.n_past];
+#pragma unroll
+      for (int k = 0; k < KV; ++k) {
+        const int i = tid + k * nt;
+        if (i < nvec) {
+          const size_t at = static_cast<size_t>(row) * a.H + i * V;
+          if (a.past_out) store_vec<float, V>(a.past_out + at, x[k]);
+#pragma unroll
+          for (int e = 0; e < V; ++e) x[k][e] *= wx;
+          for (int j0 = 0; j0 < a.n_past; j0 += kBatch) {
+            Packed<float, V> raw[kBatch];
+            float g[kBatch];
+#pragma unroll
+            for (int j = 0; j < kBatch; ++j) {
+              const int jj = min(j0 + j, a.n_past - 1);
+              g[j] = a.past_w[jj];
+              if (j0 + j < a.n_past) raw[j] = load_packed<float, V>(a.past + jj * a.past_stride + at);
+            }
+#pragma unroll
+            for (int j = 0; j < kBatch; ++j) {
+              if (j0 + j < a.n_past) {
+                float v[V];
+                unpack(raw[j], v);
+#pragma unroll
+                for (int e = 0; e < V; ++e) x[k][e] = fmaf(g[j], v[e], x[k][e]);
+              }
+            }
+          }
         }
       }
     }
@@ -476,7 +530,7 @@ __global__ void __launch_bounds__(kMaxThreads, kMinBlocks) norm_conv_kernel(cons
   }
 }
 
-template <typename E, int V, int KV, int MAXT, int kMaxThreads, int kMinBlocks>
+template <typename E, int V, int KV, int MAXT, int kMaxThreads, int kMinBlocks, bool kPast = false>
 static int launch_norm(NormArgs a, cudaStream_t st) {
   const int nvec = a.H / V, gvec = nvec / a.groups;
   const int threads = ((nvec + KV - 1) / KV + 31) / 32 * 32;
@@ -489,8 +543,8 @@ static int launch_norm(NormArgs a, cudaStream_t st) {
     a.run = run <= 2 ? 1 : run > 64 ? 64 : run;
   }
   const dim3 grid((a.T + a.run - 1) / a.run);
-  if (a.slot_w) launch_pdl(norm_conv_kernel<E, V, KV, MAXT, true, kMaxThreads, kMinBlocks>, grid, dim3(threads), smem, st, a);
-  else launch_pdl(norm_conv_kernel<E, V, KV, MAXT, false, kMaxThreads, kMinBlocks>, grid, dim3(threads), smem, st, a);
+  if (a.slot_w) launch_pdl(norm_conv_kernel<E, V, KV, MAXT, true, kPast, kMaxThreads, kMinBlocks>, grid, dim3(threads), smem, st, a);
+  else launch_pdl(norm_conv_kernel<E, V, KV, MAXT, false, kPast, kMaxThreads, kMinBlocks>, grid, dim3(threads), smem, st, a);
   return static_cast<int>(cudaGetLastError());
 }
 
@@ -498,6 +552,16 @@ template <typename E>
 static int dispatch_norm(const NormArgs& a, cudaStream_t st) {
   const int per_group = a.H / a.groups;
   const bool few = !a.conv || a.taps <= 4;
+  if (a.past_w) {                               // (never with a convolution)
+    if (per_group % 8 == 0) {
+      if (a.T > 256 && a.H <= 2048) return launch_norm<E, 8, 1, 1, 256, 3, true>(a, st);
+      if (a.T > 256 && a.H <= 4096) return launch_norm<E, 8, 2, 1, 256, 2, true>(a, st);
+      if (a.H <= 4096) return launch_norm<E, 8, 1, 1, 512, 1, true>(a, st);
+      return a.H <= 8192 ? launch_norm<E, 8, 2, 1, 512, 1, true>(a, st) : -13;
+    }
+    if (per_group % 4 == 0) return a.H <= 8192 ? launch_norm<E, 4, 4, 1, 512, 1, true>(a, st) : -13;
+    return a.H <= 4096 ? launch_norm<E, 1, 8, 1, 512, 1, true>(a, st) : -13;
+  }
   if (!a.conv && per_group % 8 == 0) {          // no convolution: no window of earlier rows in registers
     if (a.T > 256 && a.H <= 2048) return launch_norm<E, 8, 1, 1, 256, 4>(a, st);
     if (a.T > 256 && a.H <= 4096) return launch_norm<E, 8, 2, 1, 256, 3>(a, st);

@@ -1,20 +1,24 @@
 """Per-layer hybrid decoders (``ModelConfig.layer_specs``): windowed latent attention and gated delta-rule layers in any
 order, grouped RMS norms before and after every sublayer, a causal convolution on every sublayer's input, routed
 feed-forwards with identity outputs; and stacks of parallel layers (plain, differential or latent attention beside a dense or routed
-feed-forward, under one norm or one each), some of them looped.
+feed-forward, under one norm or one each), some of them looped; and layers whose sublayers read the residual itself and are normed
+after they ran (a gated linear recurrence, or attention beside linear attention), with averages over depth.
 
 A layer is a fixed launch sequence over preallocated workspaces:
 
     norm_conv -> fused projection -> mixer kernels -> o projection -> norm_conv -> routes -> plan / dispatch -> fc1 -> fc2
     parallel:  norm_conv -> fused q / k / v -> conv_rope_kv -> attention -> gate / up -> [o | down] as one product
                (routed: the shared expert's gate / up and down there, routes -> plan / dispatch -> fc1 -> fc2 beside it)
+    normed after: norm_conv -> fused projection -> [conv_rope_kv -> attention, linear attention -> norm + gate] or [convolution ->
+               gates' product -> recurrence] -> o -> norm_conv -> feed-forward
 
 ``norm_conv`` is everything between two sublayers (the routed rows' weighted sum, the norm after the sublayer, the fp32
 residual, the norm before the next one, its convolution).  What a sequence carries besides latent records lives in slots
 of one fp32 pool; a step reads one slot per sequence and writes another (``Batch.state_in`` / ``state_out``), so a step
 can be repeated and a slot can be shared with a cached prefix.  ``compute_dtype`` "f32" runs the same sequence with every
 product and activation in 32-bit.  A looped layer runs several times with the same weights; cache and state belong to the run
-(``ModelConfig.layer_runs``), not to the layer.  Where a pass starts with a product of [x; embedding row], both halves lie in one
+(``ModelConfig.layer_runs``), not to the layer.  With averages over depth the layers' results of a step stay in fp32 buffers
+until its last layer has read them.  Where a pass starts with a product of [x; embedding row], both halves lie in one
 buffer whose second half is written once per step.
 """
 from __future__ import annotations
@@ -23,7 +27,7 @@ import math
 
 import torch
 
-from ..config import AttentionSpec, DeltaSpec, LatentSpec, ModelConfig, RopeSpec, RouterSpec
+from ..config import AttentionSpec, DeltaSpec, DenseSpec, LatentSpec, ModelConfig, PairSpec, RglruSpec, RopeSpec, RouterSpec, attention_part
 from ..ops import kernels as K
 from ..parallel.moe_exchange import ExchangeGeometry, LocalExchange
 from .gqa_moe import PAGE, Batch
@@ -76,7 +80,8 @@ class HybridLayer:
     (``offs`` names its sections, each padded to a multiple of 8 rows), experts are stacked."""
     __slots__ = ("norm1", "norm1b", "norm2", "norm2b", "canon1", "canon2", "w_in", "offs", "w_o",
                  "kv_norm", "w_uk", "w_uv", "w_kb", "conv_w", "A_log", "dt_bias", "out_norm",
-                 "router", "correction", "w_gate", "w_up", "w_down", "d_gate", "d_up", "w_out", "lam", "q_norm", "k_norm", "sink")
+                 "router", "correction", "w_gate", "w_up", "w_down", "d_gate", "d_up", "d_down", "w_out", "lam", "q_norm", "k_norm",
+                 "sink", "decay", "x_bias", "y_bias", "conv_b", "w_gates", "gate_bias", "dwa")
 
     def __init__(self) -> None:
         for s in self.__slots__:
@@ -86,7 +91,7 @@ class HybridLayer:
 class HybridWeights:
     def __init__(self, cfg: ModelConfig):
         self.cfg = cfg
-        self.embed = self.final_norm = self.lm_head = self.loop_in = self.loop_step = None
+        self.embed = self.bigram = self.final_norm = self.lm_head = self.loop_in = self.loop_step = None
         self.layers: list[HybridLayer] = []
 
     @staticmethod
@@ -121,6 +126,10 @@ class HybridWeights:
                 o += pad8(x.shape[0])
             return out, offs
 
+        def norm_weight(name: str) -> torch.Tensor:
+            """A weight per channel, also where the checkpoint has one number for all of them."""
+            return t(name, ()).expand(H).contiguous() if cfg.norm_scalar else t(name, (H,))
+
         def heads_o(name: str, heads: int, vdim: int) -> torch.Tensor:
             """o projection with every head's columns padded to the row layout the mixers write."""
             w = t(name, (H, heads * vdim)).view(H, heads, vdim)
@@ -138,10 +147,10 @@ class HybridWeights:
                 if tuple(L.conv_w.shape) != (m.conv_channels, m.conv):
                     raise ValueError(f"{x}*.conv: {tuple(L.conv_w.shape)}, the configuration says {(m.conv_channels, m.conv)}")
                 L.conv_w = L.conv_w.T.contiguous()
-            if m.qk_norm:
+            if m.qk_norm in ("head", "all"):
                 L.q_norm, L.k_norm = (f(x + n + ".norm", (m.dim if m.qk_norm == "head" else rows[n],)) for n in ("q", "k"))
-            if m.sink:
-                L.sink = f(x + "sink", (m.heads,))
+            if m.sink or m.unit_sink:
+                L.sink = f(x + "sink", (m.heads,)) if m.sink else torch.zeros(m.heads, dtype=torch.float32, device=device)
             L.lam = 0.0
             if m.maps == 2:
                 q1, k1, q2, k2 = (get(x + n).double() for n in ("lq1", "lk1", "lq2", "lk2"))
@@ -169,7 +178,45 @@ class HybridWeights:
                 L.w_up[e, :r.ffn, :H] = t(f"{y}e{e}.up", (r.ffn, H))
                 L.w_down[e, :H, :r.ffn] = t(f"{y}e{e}.down", (H, r.ffn))
 
-        W.embed, W.final_norm, W.lm_head = t("embed", (cfg.vocab_size, H)), t("final.norm", (H,)), reads(t("head", (cfg.vocab_size, H)))
+        def dense(d: DenseSpec, y: str, L: HybridLayer, F: int) -> torch.Tensor:
+            """Gate and up into the layer; returns down [H padded, F]."""
+            L.d_gate, L.d_up = (torch.zeros(F, Hp, dtype=dt, device=device) for _ in range(2))
+            L.d_gate[:d.ffn, :H], L.d_up[:d.ffn, :H] = t(y + "gate", (d.ffn, H)), t(y + "up", (d.ffn, H))
+            down = torch.zeros(Hp, F, dtype=dt, device=device)
+            down[:H, :d.ffn] = t(y + "down", (H, d.ffn))
+            return down
+
+        def pair(m: PairSpec, x: str, L: HybridLayer) -> None:
+            a, b = m.left, m.right
+            if a.conv or a.gate or a.sink or a.maps != 1 or a.qk_norm not in ("", "rotated"):
+                raise ValueError("attention with weights beyond its projections is not supported in a pair")
+            attention(a, x + "left.", L)
+            rows = dict(q=b.heads * b.dim, k=b.heads * b.dim, v=b.heads * b.vdim, g=b.heads * b.vdim)
+            w, offs = fuse([(n, t(f"{x}right.{n}", (rows[n], H))) for n in rows])
+            L.offs.update({"right." + n: o + L.w_in.shape[0] for n, o in offs.items()})
+            L.w_in = torch.cat([L.w_in, w])
+            L.w_out = torch.cat([heads_o(x + "left.o", a.heads, a.vdim), heads_o(x + "right.o", b.heads, b.vdim)], 1).contiguous()
+            # the right half's factor rides on its norm's weights; the left half's on what its attention hands out
+            L.out_norm = f(x + "right.norm", (b.heads * b.vdim,)) * m.right_scale
+            L.decay = torch.tensor(b.decay, dtype=torch.float32, device=device)
+
+        def rglru(m: RglruSpec, x: str, L: HybridLayer) -> None:
+            c, n, bs, bp = m.width, m.blocks, m.block, pad8(m.block)
+            L.w_in, L.offs = fuse([(k, t(x + k, (c, H))) for k in "xy"])
+            L.x_bias, L.y_bias, L.conv_b, L.lam = (f(x + k, (c,)) for k in ("x.b", "y.b", "conv.b", "lam"))
+            L.conv_w = f(x + "conv", (c, m.conv)).T.contiguous()
+            L.w_gates = torch.zeros(n, 2, bp, bp, dtype=dt, device=device)
+            L.gate_bias = torch.zeros(n, 2, bp, dtype=torch.float32, device=device)
+            for j, k in enumerate(("ra", "ri")):
+                L.w_gates[:, j, :bs, :bs] = t(x + k, (n, bs, bs))
+                L.gate_bias[:, j, :bs] = f(f"{x}{k}.b", (n, bs))
+            L.w_gates, L.gate_bias = L.w_gates.view(n, 2 * bp, bp), L.gate_bias.view(n, 2 * bp)
+            L.w_out = torch.zeros(Hp, pad8(c), dtype=dt, device=device)
+            L.w_out[:H, :c] = t(x + "o", (H, c))
+
+        W.embed, W.final_norm, W.lm_head = t("embed", (cfg.vocab_size, H)), norm_weight("final.norm"), reads(t("head", (cfg.vocab_size, H)))
+        if cfg.bigram:
+            W.bigram = t("bigram", (cfg.bigram[0] + 1, H))
         if cfg.loop and cfg.loop_join:
             w = t("loop.in", (H, 2 * H))
             W.loop_in = torch.cat([reads(w[:, :H]), reads(w[:, H:])], 1).contiguous()
@@ -177,6 +224,20 @@ class HybridWeights:
         for i, spec in enumerate(cfg.layer_specs):
             pre, m, r, L = f"l{i}.", spec.mixer, spec.router, HybridLayer()
             x = pre + "mix."
+            if spec.post_norm:
+                y = pre + "mlp."
+                L.norm1b = norm_weight(pre + "norm1")
+                (pair if isinstance(m, PairSpec) else rglru)(m, x, L)
+                if spec.has_ffn:
+                    L.norm2b = norm_weight(pre + "norm2")
+                if r is not None:
+                    routed(r, y, L)
+                elif spec.dense is not None:
+                    L.d_down = dense(spec.dense, y, L, pad8(spec.dense.ffn))
+                if cfg.depth_average:
+                    L.dwa = f(pre + "dwa", (i + 2,))
+                W.layers.append(L)
+                continue
             if spec.parallel:
                 d, y = spec.dense, pre + "mlp."
                 L.norm1 = t(pre + "norm1", (H,))
@@ -193,12 +254,7 @@ class HybridWeights:
                     y += "shared."
                 L.w_out = heads_o(x + "o", m.heads, m.vdim)
                 if d is not None:
-                    F = out_columns(m, d)[1]
-                    L.d_gate, L.d_up = (torch.zeros(F, Hp, dtype=dt, device=device) for _ in range(2))
-                    L.d_gate[:d.ffn, :H], L.d_up[:d.ffn, :H] = t(y + "gate", (d.ffn, H)), t(y + "up", (d.ffn, H))
-                    down = torch.zeros(Hp, F, dtype=dt, device=device)
-                    down[:H, :d.ffn] = t(y + "down", (H, d.ffn))
-                    L.w_out = torch.cat([L.w_out, down], 1).contiguous()
+                    L.w_out = torch.cat([L.w_out, dense(d, y, L, out_columns(m, d)[1])], 1).contiguous()
                 W.layers.append(L)
                 continue
             L.norm1, L.norm1b = t(pre + "norm1", (H,)), t(pre + "norm1b", (H,))
@@ -236,6 +292,8 @@ class HybridWeights:
             shape = shapes[name]
             if name.rsplit(".", 1)[-1].startswith("norm"):
                 return torch.full(shape, 1.0 if ".mix." in name else 1.0 - cfg.norm_offset, device=device)
+            if name.endswith(".dwa"):
+                return torch.full(shape, 1.0 / shape[0], device=device)
             s = 0.3 if "conv" in name or "canon" in name else std
             x = torch.empty(shape, dtype=torch.float32, device=device).normal_(0.0, s, generator=g)
             return x - 3.0 if name.endswith("dt_bias") else x
@@ -245,12 +303,28 @@ class HybridWeights:
 def tensor_shapes(cfg: ModelConfig) -> dict[str, tuple]:
     """Every tensor of the checkpoint and its shape."""
     H = cfg.hidden
-    out: dict[str, tuple] = {"embed": (cfg.vocab_size, H), "final.norm": (H,), "head": (cfg.vocab_size, H)}
+    one = () if cfg.norm_scalar else (H,)
+    out: dict[str, tuple] = {"embed": (cfg.vocab_size, H), "final.norm": one, "head": (cfg.vocab_size, H)}
+    if cfg.bigram:
+        out["bigram"] = (cfg.bigram[0] + 1, H)
     if cfg.loop and cfg.loop_join:
         out.update({"loop.in": (H, 2 * H), "loop.step": (cfg.loop[2], H)})
     for i, spec in enumerate(cfg.layer_specs):
         pre, m, r = f"l{i}.", spec.mixer, spec.router
         x = pre + "mix."
+        if spec.post_norm:
+            out[pre + "norm1"] = one
+            out.update(_pair_shapes(x, m, H) if isinstance(m, PairSpec) else _rglru_shapes(x, m, H))
+            if spec.has_ffn:
+                out[pre + "norm2"] = one
+            if r is not None:
+                out.update(_routed_shapes(pre + "mlp.", r, H))
+            elif spec.dense is not None:
+                d = spec.dense.ffn
+                out.update({pre + "mlp.gate": (d, H), pre + "mlp.up": (d, H), pre + "mlp.down": (H, d)})
+            if cfg.depth_average:
+                out[pre + "dwa"] = (i + 2,)
+            continue
         if spec.parallel:
             out[pre + "norm1"], out[x + "o"] = (H,), (H, m.heads * m.vdim)
             if spec.two_norms and (spec.dense is not None or r is not None):
@@ -301,6 +375,21 @@ def _latent_shapes(x: str, m: LatentSpec, H: int) -> dict[str, tuple]:
     return out
 
 
+def _pair_shapes(x: str, m: PairSpec, H: int) -> dict[str, tuple]:
+    a, b = m.left, m.right
+    out = {f"{x}left.{n}": (c, H) for n, c in (("q", a.q_channels), ("k", a.k_channels), ("v", a.v_channels))}
+    out.update({f"{x}right.{n}": (c, H) for n, c in (("q", b.heads * b.dim), ("k", b.heads * b.dim), ("v", b.heads * b.vdim), ("g", b.heads * b.vdim))})
+    return out | {x + "left.o": (H, a.heads * a.vdim), x + "right.o": (H, b.heads * b.vdim), x + "right.norm": (b.heads * b.vdim,)}
+
+
+def _rglru_shapes(x: str, m: RglruSpec, H: int) -> dict[str, tuple]:
+    c, out = m.width, {x + "o": (H, m.width), x + "conv": (m.width, m.conv)}
+    out.update({x + n: (c,) for n in ("x.b", "y.b", "conv.b", "lam")})
+    for n in ("ra", "ri"):
+        out.update({x + n: (m.blocks, m.block, m.block), f"{x}{n}.b": (m.blocks, m.block)})
+    return out | {x + "x": (c, H), x + "y": (c, H)}
+
+
 def _routed_shapes(y: str, r: RouterSpec, H: int) -> dict[str, tuple]:
     out = {y + "router": (r.outputs, H), y + ("router.b" if r.logit_bias else "correction"): (r.outputs,)}
     for e in range(r.experts):
@@ -317,7 +406,7 @@ def tensor_core_latent(cfg: ModelConfig, m: LatentSpec) -> bool:
 def tensor_core_attention(cfg: ModelConfig, m: AttentionSpec) -> bool:
     """Whether the tensor-core attention kernels take this layer: key rows (all maps) and values of 128."""
     rows = m.maps * (m.heads // m.kv_heads)
-    return engine_dtype(cfg) == torch.bfloat16 and m.maps * m.dim == 128 and m.vdim == 128 and rows <= 16 and 16 % rows == 0
+    return not m.softcap and engine_dtype(cfg) == torch.bfloat16 and m.maps * m.dim == 128 and m.vdim == 128 and rows <= 16 and 16 % rows == 0
 
 
 class HybridCache:
@@ -337,26 +426,22 @@ class HybridCache:
         self.offsets: list[dict[str, int]] = []
         n = 0
         for i, run in enumerate(cfg.layer_runs):
-            spec = cfg.layer_specs[run.layer]
-            m, off = spec.mixer, {}
-            parts = [] if spec.parallel else [("canon1", (cfg.canon_taps - 1) * cfg.hidden)]
-            if spec.router is not None:
-                parts.append(("canon2", (cfg.canon_taps - 1) * cfg.hidden))
-            if isinstance(m, DeltaSpec):
-                parts += [("S", m.heads * m.dim * m.vdim), ("conv", (m.conv - 1) * m.conv_channels)]
-            elif isinstance(m, AttentionSpec):
-                parts.append(("conv", max(0, m.conv - 1) * m.conv_channels))
-                kv = [torch.zeros(num_pages, m.kv_heads, PAGE, w, dtype=dt, device=device) for w in (m.maps * m.dim, m.vdim)]
+            m, off = cfg.layer_specs[run.layer].mixer, {}
+            att = attention_part(m)
+            if att is not None:
+                kv = [torch.zeros(num_pages, att.kv_heads, PAGE, w, dtype=dt, device=device) for w in (att.maps * att.dim, att.vdim)]
                 self.of_run[i] = tuple(kv)
                 self.k.append(kv[0])
                 self.v.append(kv[1])
-            else:
+            elif isinstance(m, LatentSpec):
                 self.of_run[i] = torch.zeros(num_pages, PAGE, record_pitch(m), dtype=dt, device=device)
                 self.c.append(self.of_run[i])
-            for name, size in parts:
+            for name, size in cfg.state_parts(run.layer):
                 off[name] = n
                 n += -(-size // 32) * 32
             self.offsets.append(off)
+        self.token_off = n               # a sequence's last token (models with a bigram table)
+        n += 32 * bool(cfg.bigram)
         self.state = torch.zeros(max(3, state_slots), max(n, 32), dtype=torch.float32, device=device)
 
     @property
@@ -392,8 +477,20 @@ class _AttnWs:
         self.q = torch.zeros(max_tokens, m.q_channels, dtype=engine_dtype(cfg), device=device)
         if m.rope not in tables:
             tables[m.rope] = (rope_frequencies(m.rope).to(device), torch.zeros(max_tokens, max(1, m.rope.dims // 2), 2, device=device))
-        self.table = tables[m.rope][1]
+        if m.v_rope is not None and m.v_rope not in tables:
+            tables[m.v_rope] = (rope_frequencies(m.v_rope).to(device), torch.zeros(max_tokens, max(1, m.v_rope.dims // 2), 2, device=device))
+        self.table, self.v_table = tables[m.rope][1], tables[m.v_rope][1] if m.v_rope is not None else None
         self.tensor_core = tensor_core_attention(cfg, m)
+
+
+class _RglruWs:
+    """Workspaces shared by the gated linear recurrences of one shape (rows of a block are whole 16-byte pieces; the padding stays zero)."""
+
+    def __init__(self, cfg: ModelConfig, m: RglruSpec, max_tokens: int, device: torch.device):
+        rows, bp, dt = -(-max_tokens // 128) * 128, pad8(m.block), engine_dtype(cfg)
+        self.u = torch.zeros(m.blocks * rows * bp, dtype=dt, device=device)
+        self.gates = torch.empty(m.blocks * rows * 2 * bp, dtype=torch.float32, device=device)
+        self.out = torch.zeros(max_tokens, pad8(m.width), dtype=dt, device=device)
 
 
 class HybridEngine:
@@ -418,6 +515,10 @@ class HybridEngine:
             pass
         ws = self.ws = _Ws()
         ws.x = [torch.empty(max_tokens, H, dtype=torch.float32, device=dev) for _ in range(2)]
+        # averages over depth: the embedding rows and every layer run's result but the last one's
+        runs = len(cfg.layer_runs)
+        ws.past = torch.empty(runs, max_tokens, H, dtype=torch.float32, device=dev) if cfg.depth_average else None
+        ws.rows2 = torch.zeros(max_tokens, dtype=torch.int32, device=dev) if cfg.bigram else None
         Hp = pad8(H)                     # rows the matrix products read are whole 16-byte pieces; the padding stays zero
         ws.h = [torch.zeros(max_tokens, Hp, dtype=dt, device=dev) for _ in range(2)]
         ws.y = torch.zeros(max_tokens, Hp, dtype=dt, device=dev)
@@ -432,6 +533,7 @@ class HybridEngine:
         self._attn: dict[AttentionSpec, _AttnWs] = {}
         self._rope: dict[RopeSpec, tuple] = {}       # frequencies, the step's table
         self._delta: dict[DeltaSpec, torch.Tensor] = {}
+        self._rglru: dict[RglruSpec, _RglruWs] = {}
         self._moe: dict = {}
         raw = scratch = 0
         for spec in cfg.layer_specs:
@@ -439,9 +541,14 @@ class HybridEngine:
             if isinstance(m, LatentSpec):
                 if m not in self._lat:
                     self._lat[m] = _LatentWs(cfg, m, max_tokens, dev)
-            elif isinstance(m, AttentionSpec):
-                if m not in self._attn:
-                    self._attn[m] = _AttnWs(cfg, m, max_tokens, dev, self._rope)
+            elif isinstance(m, RglruSpec):
+                if m not in self._rglru:
+                    self._rglru[m] = _RglruWs(cfg, m, max_tokens, dev)
+            elif (a := attention_part(m)) is not None:
+                if a not in self._attn:
+                    self._attn[a] = _AttnWs(cfg, a, max_tokens, dev, self._rope)
+                if isinstance(m, PairSpec):
+                    raw = max(raw, m.right.heads * m.right.vdim)
             else:
                 if m not in self._delta:
                     self._delta[m] = torch.zeros(max_tokens, m.heads, pad8(m.vdim), dtype=dt, device=dev)
@@ -455,7 +562,7 @@ class HybridEngine:
             if r is not None and r not in self._moe:
                 self._moe[r] = LocalExchange(ExchangeGeometry(Hp, pad8(r.ffn), r.experts, r.top, max_tokens, 1), dev, dtype=dt)
         # rows of a parallel layer's second product: the heads' values, then the feed-forward's activations
-        act = max((L.w_out.shape[1] for L in weights.layers if L.w_out is not None), default=0)
+        act = max((w.shape[1] for L in weights.layers for w in (L.w_out, L.d_down) if w is not None), default=0)
         ws.act = torch.zeros(max_tokens * act, dtype=dt, device=dev) if act else None
         ws.raw = torch.empty(max_tokens * raw, dtype=torch.float32, device=dev) if raw else None
         ws.chunk = torch.empty(scratch, dtype=torch.uint8, device=dev) if scratch else None
@@ -480,15 +587,20 @@ class HybridEngine:
         src = {} if self._x is None else dict(x_in=self._x)
         if self._x is None or add_embedding:
             src.update(tokens=b.tokens, embed=self.W.embed, embed_scale=self.cfg.embed_scale)
+            if self.W.bigram is not None:
+                src.update(second=(self.ws.rows2[:b.tokens.shape[0]], self.W.bigram))
         return src
 
-    def _between(self, b: Batch, T: int, w: torch.Tensor, conv: torch.Tensor | None, off: int = 0, add_embedding: bool = False,
+    def _between(self, b: Batch, T: int, w: torch.Tensor | None, conv: torch.Tensor | None, off: int = 0, add_embedding: bool = False,
                  step: torch.Tensor | None = None, w2: torch.Tensor | None = None) -> torch.Tensor:
         """Residual, norms and input convolution up to the next sublayer; returns its input rows (``w2``: the same norm's rows under
         other weights go to ``ws.h2``)."""
         ws, p = self.ws, self._pending
         h = ws.h[self._hi][:T]
-        xo = ws.x[0 if self._x is None or self._x.data_ptr() != ws.x[0].data_ptr() else 1][:T]
+        if self._x is None and ws.past is not None:
+            xo = ws.past[0, :T]
+        else:
+            xo = ws.x[0 if self._x is None or self._x.data_ptr() != ws.x[0].data_ptr() else 1][:T]
         K.norm_conv(h, w, self.cfg.norm_groups, self.cfg.rms_eps, conv=conv, x_out=xo, state=self.kv.state, state_off=off,
                     state_in=b.state_in, state_out=b.state_out, q_start=b.q_start, w_offset=self.cfg.norm_offset, step=step,
                     w2=w2, h2_out=ws.h2[:T] if w2 is not None else None, **self._source(b, add_embedding), **p)
@@ -521,6 +633,9 @@ class HybridEngine:
                 return x + y
             g = y.view(T, G, -1)
             x = x + (g / torch.sqrt((g * g).mean(-1, keepdim=True) + self.cfg.rms_eps)).view(T, -1) * p["w_b"]
+            if p.get("past") is not None:
+                results, w, _ = p["past"]
+                x = (w[:-1, None, None] * results[:, :T]).sum(0) + w[-1] * x
         return x
 
     # ---- mixers -----------------------------------------------------------------------------------------------------
@@ -623,17 +738,22 @@ class HybridEngine:
                         self._scratch if splits > 1 else None, out_tpad=t_pad, window=m.window)
         self.launches += 1 if splits > 1 else 0
 
-    def _attention(self, n: int, i: int, m: AttentionSpec, h: torch.Tensor, T: int, b: Batch, out: torch.Tensor) -> None:
-        """Attention of layer run n; head h's values go to columns [h * pad8(vdim), + vdim) of ``out``."""
+    def _attention(self, n: int, i: int, m: AttentionSpec, h: torch.Tensor, T: int, b: Batch, out: torch.Tensor,
+                   a: torch.Tensor | None = None, out_scale: float = 1.0) -> None:
+        """Attention of layer run n; head h's values, times ``out_scale``, go to columns [h * pad8(vdim), + vdim) of ``out``.  ``a``: the
+        projected rows, if they are there already."""
         L, aw = self.W.layers[i], self._attn[m]
-        a = self._project(i, h, T)
+        if a is None:
+            a = self._project(i, h, T)
         (k, v), q = self.kv.of_run[n], aw.q[:T]
         K.conv_rope_kv(a, L.offs, m, L.conv_w, aw.table, b.slots, q, k, v, state=self.kv.state, state_off=self.kv.offsets[n]["conv"],
-                       state_in=b.state_in, state_out=b.state_out, q_start=b.q_start, q_norm=L.q_norm, k_norm=L.k_norm, eps=self.cfg.rms_eps)
+                       state_in=b.state_in, state_out=b.state_out, q_start=b.q_start, q_norm=L.q_norm, k_norm=L.k_norm, eps=self.cfg.rms_eps,
+                       v_table=aw.v_table)
         self.launches += 2
         gate = a[:, L.offs["g"]:L.offs["g"] + m.heads] if m.gate else None
         if not aw.tensor_core:
-            K.paged_attn(q, k, v, m, b.page_table, b.positions, b.q_start, out, pad8(m.vdim), L.lam, self.cfg.rms_eps, sink=L.sink, gate=gate)
+            K.paged_attn(q, k, v, m, b.page_table, b.positions, b.q_start, out, pad8(m.vdim), L.lam, self.cfg.rms_eps, sink=L.sink, gate=gate,
+                         v_table=aw.v_table, out_scale=out_scale)
             return
         kw = dict(scale=m.scale, window=m.window, keep=m.keep_first, maps=m.maps, lam=L.lam, out_scale=1.0 - m.diff, eps=self.cfg.rms_eps,
                   sink=L.sink, gate=gate)
@@ -666,6 +786,67 @@ class HybridEngine:
         if r is not None:
             self._pending = dict(slots=self._experts(i, r, f, T), y=self._moe[r].att.combine, base=self.ws.y[:T])
 
+    def _pair(self, n: int, i: int, m: PairSpec, h: torch.Tensor, T: int, b: Batch) -> None:
+        """Attention and linear attention on the same rows; one product over both reads their values side by side."""
+        L, ws = self.W.layers[i], self.ws
+        a = self._project(i, h, T)
+        act = ws.act[:T * L.w_out.shape[1]].view(T, L.w_out.shape[1])
+        self._attention(n, i, m.left, h, T, b, act, a=a, out_scale=m.left_scale)
+        r = m.right
+        K.lightning_step(a, {k: L.offs["right." + k] for k in "qkvg"}, r, L, self.kv.state, self.kv.offsets[n]["S"], b.state_in, b.state_out,
+                         b.q_start, ws.raw, act[:, m.left.heads * pad8(m.left.vdim):], pad8(r.vdim), self.cfg.rms_eps)
+        K.linear(act, L.w_out, out=ws.y[:T])
+        self.launches += 3
+
+    def _rglru_mixer(self, n: int, i: int, m: RglruSpec, h: torch.Tensor, T: int, b: Batch) -> None:
+        L, rw, off = self.W.layers[i], self._rglru[m], self.kv.offsets[n]
+        a = self._project(i, h, T)
+        bp = pad8(m.block)
+        key = (T, m.blocks, 0)
+        if key not in self._tiles:
+            self._tiles[key] = _HeadTiles(T, m.blocks, self.device)
+        ht = self._tiles[key]
+        u = rw.u[:m.blocks * ht.t_pad * bp].view(m.blocks, ht.t_pad, bp)
+        gates = rw.gates[:m.blocks * ht.t_pad * 2 * bp].view(m.blocks, ht.t_pad, 2 * bp)
+        carry = None
+        if b.max_q_len > K.RGLRU_CHUNK:
+            need = 2 * m.width * (b.q_start.shape[0] - 1) * -(-b.max_q_len // K.RGLRU_CHUNK)
+            self._partials(need)
+            carry = self._scratch
+        out = rw.out[:T]
+        args = (a, L.offs, m, L, u, gates, self.kv.state, off["S"], off["conv"], b.state_in, b.state_out, b.q_start, out, carry, b.max_q_len)
+        K.rglru_conv(*args)
+        K.grouped_linear(u.view(-1, bp), L.w_gates, gates.view(-1, 2 * bp), ht.tile_expert, ht.tile_row0, ht.num_tiles, ht.max_tiles, ht.tile_rows,
+                         split_k=False)
+        K.rglru_scan(*args)
+        K.linear(out, L.w_out, out=self.ws.y[:T])
+        self.launches += 4 + (carry is not None)
+
+    def _dense(self, i: int, d: DenseSpec, h: torch.Tensor, T: int) -> None:
+        L, F = self.W.layers[i], pad8(d.ffn)
+        act = self.ws.act[:T * F].view(T, F)
+        K.linear(h, L.d_gate, out=act, w_up=L.d_up, glu=None if d == DenseSpec(d.ffn) else (d.limit or math.inf, d.alpha, d.up_bias))
+        K.linear(act, L.d_down, out=self.ws.y[:T])
+        self.launches += 2
+
+    def _post_norm(self, n: int, i: int, spec, T: int, b: Batch) -> None:
+        """Sublayers that read the residual and are normed after they ran; then the average over depth, in the launch that takes the
+        last sublayer's rows."""
+        L, m, r = self.W.layers[i], spec.mixer, spec.router
+        h = self._between(b, T, None, None)
+        (self._pair if isinstance(m, PairSpec) else self._rglru_mixer)(n, i, m, h, T, b)
+        self._pending = dict(y=self.ws.y[:T], w_b=L.norm1b)
+        if spec.has_ffn:
+            h = self._between(b, T, None, None)
+            self._pending = dict(y=self.ws.y[:T], w_b=L.norm2b)
+            if r is not None:
+                self._pending.update(slots=self._experts(i, r, h, T), y=self._moe[r].att.combine)
+            else:
+                self._dense(i, spec.dense, h, T)
+        if L.dwa is not None:
+            past = self.ws.past
+            self._pending["past"] = (past[:n + 1], L.dwa, past[n + 1, :T] if n + 1 < past.shape[0] else None)
+
     def _delta_mixer(self, n: int, i: int, m: DeltaSpec, h: torch.Tensor, T: int, b: Batch) -> None:
         L, ws = self.W.layers[i], self.ws
         a = self._project(i, h, T)
@@ -684,7 +865,7 @@ class HybridEngine:
     # ---- routed feed-forward ----------------------------------------------------------------------------------------
     def _experts(self, i: int, r, h: torch.Tensor, T: int) -> tuple:
         L, moe = self.W.layers[i], self._moe[r]
-        kw = dict(scoring="softmax_bias" if r.logit_bias else "softmax", bias=L.correction, num_groups=r.groups, topk_groups=r.groups_kept,
+        kw = dict(scoring="softmax_bias" if r.logit_bias else r.scoring, bias=L.correction, num_groups=r.groups, topk_groups=r.groups_kept,
                   normalize=r.normalize, routed_scale=1.0, group_score="max")
         logits = None
         idx, w = moe.att.idx[:T], moe.att.w[:T]
@@ -710,12 +891,20 @@ class HybridEngine:
             if r.dims:
                 K.rope_table(b.positions, freq, table.view(-1)[:T * r.dims], r.magnitude)
                 self.launches += 1
+        if self.W.bigram is not None:
+            K.bigram_rows(b.tokens, self.cfg.bigram, self.kv.state, self.kv.token_off, b.state_in, b.state_out, b.q_start, self.ws.rows2[:T])
+            self.launches += 1
         if self.W.loop_in is not None:
             K.norm_conv(self.ws.join[:T, pad8(self.cfg.hidden):], None, self.cfg.norm_groups, self.cfg.rms_eps, **self._source(b))
             self.launches += 1
         for n, run in enumerate(self.cfg.layer_runs):
             i, spec = run.layer, self.cfg.layer_specs[run.layer]
             L, off, m, r = self.W.layers[i], self.kv.offsets[n], spec.mixer, spec.router
+            if spec.post_norm:
+                self._post_norm(n, i, spec, T, b)
+                if self.layer_hook is not None:
+                    self.layer_hook(n, self.residual(T))
+                continue
             if spec.parallel:
                 step = None
                 if run.join >= 0:

@@ -92,8 +92,9 @@ def pick_token_tile(rows: int) -> int:
 
 def linear(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor | None = None, *, w_up: torch.Tensor | None = None,
            residual: torch.Tensor | None = None, out_f32: bool = False, swap: bool | None = None,
-           split_k: bool = True) -> torch.Tensor:
-    """y = x @ w.T (bf16 in, fp32 accumulate).  With ``w_up``: y = silu(x @ w.T) * (x @ w_up.T).
+           split_k: bool = True, glu: tuple | None = None) -> torch.Tensor:
+    """y = x @ w.T (bf16 in, fp32 accumulate).  With ``w_up``: y = silu(x @ w.T) * (x @ w_up.T), or with ``glu`` = (limit, alpha, bias)
+    and the products g and u: min(g, limit) sigmoid(alpha min(g, limit)) (min(max(u, -limit), limit) + bias).
 
     x [T, K], w [N, K].  ``swap`` picks the orientation (default: weights on M when T <= 128).
     """
@@ -101,7 +102,7 @@ def linear(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor | None = None, *,
     N = w.shape[0]
     if x.dtype == torch.float32:
         assert residual is None
-        return linear_f32(x, w, out, w_up=w_up)
+        return linear_f32(x, w, out, w_up=w_up, glu=glu)
     assert x.dtype == torch.bfloat16 and w.dtype == torch.bfloat16 and x.is_contiguous() and w.is_contiguous()
     assert w.shape[1] == K
     if out is None:
@@ -121,13 +122,16 @@ def linear(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor | None = None, *,
     if swap and T > 128:
         a.bx = 128
     a.out_f32, a.fp8, a.num_sms = int(out.dtype == torch.float32), 0, num_sms()
+    if glu is not None:
+        a.glu, (a.glu_limit, a.glu_alpha, a.glu_bias) = 1, glu
     if swap and split_k:
         _attach_splitk(a, x.device)
     _n.check(_n.cuda_lib().cafd_gemm(C.byref(a), _stream()), "cafd_gemm")
     return out
 
 
-def linear_f32(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor | None = None, *, w_up: torch.Tensor | None = None) -> torch.Tensor:
+def linear_f32(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor | None = None, *, w_up: torch.Tensor | None = None,
+               glu: tuple | None = None) -> torch.Tensor:
     """``linear`` with fp32 operands and fp32 products (no reduced-precision mode)."""
     T, K = x.shape
     N = w.shape[0]
@@ -136,7 +140,8 @@ def linear_f32(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor | None = None
         out = torch.empty(T, N, dtype=torch.float32, device=x.device)
     assert out.dtype == torch.float32
     _n.check(_n.cuda_lib().cafd_gemm_f32(w.data_ptr(), _ptr(w_up), x.data_ptr(), out.data_ptr(), None, None, None, None, K, N, T,
-                                         x.stride(0), out.stride(0), 0, 0, 0, _stream()), "gemm_f32")
+                                         x.stride(0), out.stride(0), 0, 0, 0, int(glu is not None), *(glu or (0.0, 0.0, 0.0)), _stream()),
+             "gemm_f32")
     return out
 
 
@@ -158,7 +163,7 @@ def grouped_linear(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, tile_exp
         _n.check(_n.cuda_lib().cafd_gemm_f32(w.data_ptr(), _ptr(w_up), x.data_ptr(), out_ptr if out_ptr is not None else out.data_ptr(),
                                              _ptr(row_dst), tile_expert.data_ptr(), tile_row0.data_ptr(), num_tiles.data_ptr(), K, N,
                                              x.shape[0], x.stride(0), ldo if ldo is not None else out.stride(0), N, max_tiles, tile_rows,
-                                             _stream()), "gemm_f32(grouped)")
+                                             0, 0.0, 0.0, 0.0, _stream()), "gemm_f32(grouped)")
         return
     a = _n.GemmArgs()
     a.w0, a.w1, a.x = w.data_ptr(), _ptr(w_up), x.data_ptr()
@@ -174,7 +179,7 @@ def grouped_linear(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, tile_exp
     a.w_rows_per_expert, a.w1_row_offset, a.max_x_tiles = N, 0, max_tiles
     swap = tile_rows < 128
     a.swap, a.dual, a.bx = int(swap), int(w_up is not None), tile_rows
-    a.out_f32, a.fp8, a.num_sms = 0, 0, num_sms()
+    a.out_f32, a.fp8, a.num_sms = int(out_ptr is None and out.dtype == torch.float32), 0, num_sms()
     if swap and split_k:
         _attach_splitk(a, x.device)
     _n.check(_n.cuda_lib().cafd_gemm(C.byref(a), _stream()), "cafd_gemm(grouped)")
@@ -696,14 +701,15 @@ def mla_unabsorb_small(o_lat: torch.Tensor, w_uv: torch.Tensor, attn: torch.Tens
              "mla_unabsorb_small")
 
 
-# ---- per-layer hybrids (csrc/hybrid_norm.cu, latent.cu, delta.cu, conv_rope.cu, attention_any.cu) --------------------------------------------
+# ---- per-layer hybrids (csrc/hybrid_norm.cu, latent.cu, delta.cu, conv_rope.cu, attention_any.cu, rglru.cu, lightning.cu) --------------------------------------------
 def norm_conv(h_out: torch.Tensor, w: torch.Tensor | None, groups: int, eps: float, *, tokens: torch.Tensor | None = None,
               embed: torch.Tensor | None = None, x_in: torch.Tensor | None = None, y: torch.Tensor | None = None,
               w_b: torch.Tensor | None = None, slots: tuple | None = None, conv: torch.Tensor | None = None,
               x_out: torch.Tensor | None = None, rows: torch.Tensor | None = None, state: torch.Tensor | None = None, state_off: int = 0,
               state_in: torch.Tensor | None = None, state_out: torch.Tensor | None = None, q_start: torch.Tensor | None = None,
               run: int = 0, w_offset: float = 0.0, embed_scale: float = 1.0, step: torch.Tensor | None = None,
-              base: torch.Tensor | None = None, w2: torch.Tensor | None = None, h2_out: torch.Tensor | None = None) -> None:
+              base: torch.Tensor | None = None, w2: torch.Tensor | None = None, h2_out: torch.Tensor | None = None,
+              second: tuple | None = None, past: tuple | None = None) -> None:
     """Weights are in the activations' type.  x = embed[tokens] * ``embed_scale``, ``x_in`` (fp32) or, given both, their sum; x +=
     ``step`` [H]; x += groupnorm(y) * w_b (without ``w_b``: x += y); h = groupnorm(x) * (w + ``w_offset``), without ``w`` h = x; h_out =
     h + causal_conv(h).  ``w2`` / ``h2_out``: a second output of the same norm under weights of its own (no convolution).
@@ -711,7 +717,10 @@ def norm_conv(h_out: torch.Tensor, w: torch.Tensor | None, groups: int, eps: flo
     Rows of ``h_out``, ``y`` and the identity rows may be longer than H (whole 16-byte pieces); the rest is left alone.
     ``slots`` = (weights [T, k], ids [T, k], number of experts, identity rows): ``y`` then holds the routed experts' rows
     [T * k, ...] and is their weighted sum, plus the rows of ``base``.  ``conv`` [taps, H] (last row = current token) with the sequences'
-    earlier inputs in ``state`` [slots, floats] at ``state_off``.  ``rows``: compute only these rows (no convolution)."""
+    earlier inputs in ``state`` [slots, floats] at ``state_off``.  ``rows``: compute only these rows (no convolution).
+
+    ``second`` = (row ids [T], table): rows of a second table are added to the embedding's.  ``past`` = (results [n, rows, H] fp32, weights
+    [n + 1] fp32, copy [rows, H] fp32 or None): x is kept in ``copy``, then becomes the weighted sum of the results and itself."""
     a = _n.NormArgs()
     H = w.shape[0] if w is not None else embed.shape[1] if embed is not None else x_in.shape[1]
     a.tokens, a.embed, a.x_in, a.y = _ptr(tokens), _ptr(embed), _ptr(x_in), _ptr(y)
@@ -733,7 +742,85 @@ def norm_conv(h_out: torch.Tensor, w: torch.Tensor | None, groups: int, eps: flo
         a.state, a.state_in, a.state_out, a.q_start = state.data_ptr(), state_in.data_ptr(), state_out.data_ptr(), q_start.data_ptr()
         a.slot_stride, a.state_off = state.stride(0), state_off
         assert conv.is_contiguous() and conv.dtype == h_out.dtype and state.dtype == torch.float32
+    if second is not None:
+        a.rows2, a.embed2, a.vocab2 = second[0].data_ptr(), second[1].data_ptr(), second[1].shape[0]
+        assert second[0].dtype == torch.int32 and second[1].dtype == h_out.dtype and second[1].is_contiguous() and second[1].shape[1] == H
+    if past is not None:
+        results, weights, copy = past
+        a.past, a.past_w, a.past_out = results.data_ptr(), weights.data_ptr(), _ptr(copy)
+        a.n_past, a.past_stride = results.shape[0], results.stride(0)
+        assert all(v is None or (v.dtype == torch.float32 and v.stride(-1) == 1) for v in past) and weights.numel() == a.n_past + 1
+        assert results.shape[2] == results.stride(1) == H and (copy is None or copy.stride(0) == H)
     _n.check(_n.cuda_lib().cafd_norm_conv(C.byref(a), int(h_out.dtype == torch.float32), _stream()), "norm_conv")
+
+
+def bigram_rows(tokens: torch.Tensor, bigram: tuple, state: torch.Tensor, off: int, state_in: torch.Tensor, state_out: torch.Tensor,
+                q_start: torch.Tensor, out: torch.Tensor) -> None:
+    """out [T] = (previous token * mul_prev + token * mul_cur) mod buckets, ``bigram`` = (buckets, mul_prev, mul_cur); a sequence's first
+    token gives ``buckets``.  The last token of every sequence is kept at ``off`` of its slot."""
+    a = _n.BigramArgs()
+    a.tokens, a.q_start, a.state_in, a.state_out, a.state, a.rows = (t.data_ptr() for t in (tokens, q_start, state_in, state_out, state, out))
+    a.slot_stride, a.state_off, (a.buckets, a.mul_prev, a.mul_cur) = state.stride(0), off, bigram
+    a.T, a.S = tokens.shape[0], q_start.shape[0] - 1
+    assert tokens.dtype == out.dtype == torch.int32 and state.dtype == torch.float32
+    _n.check(_n.cuda_lib().cafd_bigram_rows(C.byref(a), _stream()), "bigram_rows")
+
+
+RGLRU_CHUNK = 128                    # portions longer than this are cut into chunks of it
+
+
+def rglru_args(proj: torch.Tensor, offs: dict, m, w, u: torch.Tensor, gates: torch.Tensor | None, state: torch.Tensor, s_off: int, c_off: int,
+               state_in: torch.Tensor, state_out: torch.Tensor, q_start: torch.Tensor, out: torch.Tensor, carry: torch.Tensor | None = None,
+               max_q: int = 0) -> "_n.RglruArgs":
+    """Arguments of the gated linear recurrence's kernels.  ``m``: an ``RglruSpec``; ``w`` carries x_bias, y_bias, conv_b, lam [width], conv_w
+    [taps, width], w_gates [blocks, 2 * block (padded), block (padded)] and gate_bias [blocks, 2 * block (padded)] (fp32 but for w_gates);
+    ``u`` [blocks, t_pad, block (padded)] convolved rows, ``gates`` fp32 [blocks, t_pad, 2 * block (padded)]."""
+    p = _n.RglruArgs()
+    p.proj, p.y_bias, p.x_bias, p.conv_w, p.conv_b = proj.data_ptr(), w.y_bias.data_ptr(), w.x_bias.data_ptr(), w.conv_w.data_ptr(), w.conv_b.data_ptr()
+    p.lam, p.w, p.gate_bias, p.u, p.gates, p.out = w.lam.data_ptr(), w.w_gates.data_ptr(), w.gate_bias.data_ptr(), u.data_ptr(), _ptr(gates), out.data_ptr()
+    p.carry, p.state, p.state_in, p.state_out, p.q_start = _ptr(carry), state.data_ptr(), state_in.data_ptr(), state_out.data_ptr(), q_start.data_ptr()
+    p.slot_stride, p.s_off, p.c_off = state.stride(0), s_off, c_off
+    p.T, p.S, p.ld, p.x_off, p.y_off, p.width, p.blocks, p.taps = proj.shape[0], q_start.shape[0] - 1, proj.stride(0), offs["x"], offs["y"], m.width, m.blocks, m.conv
+    p.t_pad, p.u_pitch, p.ldo, p.max_q, p.c = u.shape[1], u.shape[2], out.stride(0), max_q, m.c
+    assert u.is_contiguous() and u.dtype == proj.dtype == out.dtype and out.stride(1) == 1 and state.dtype == torch.float32
+    assert gates is None or (gates.is_contiguous() and gates.dtype == torch.float32 and gates.shape == (m.blocks, p.t_pad, 2 * p.u_pitch))
+    assert carry is None or carry.numel() >= 2 * m.width * p.S * -(-max_q // RGLRU_CHUNK)
+    assert w.conv_w.shape == (m.conv, m.width) and w.gate_bias.shape == (m.blocks, 2 * p.u_pitch) and u.shape[0] == m.blocks
+    return p
+
+
+def rglru_conv(proj: torch.Tensor, *args, **kw) -> None:
+    """Bias and causal convolution of the recurrent branch into ``u``, and the sequences' last inputs (see ``rglru_args``)."""
+    _n.check(_n.cuda_lib().cafd_rglru_conv(C.byref(rglru_args(proj, *args, **kw)), int(proj.dtype == torch.float32), _stream()), "rglru_conv")
+
+
+def rglru_scan(proj: torch.Tensor, *args, **kw) -> None:
+    """Gates, decays, the recurrence and its product with the gelu branch (see ``rglru_args``)."""
+    _n.check(_n.cuda_lib().cafd_rglru_scan(C.byref(rglru_args(proj, *args, **kw)), int(proj.dtype == torch.float32), _stream()), "rglru_scan")
+
+
+def lightning_args(proj: torch.Tensor, offs: dict, m, w, state: torch.Tensor, s_off: int, state_in: torch.Tensor, state_out: torch.Tensor,
+                   q_start: torch.Tensor, raw: torch.Tensor, out: torch.Tensor, head_pitch: int, eps: float,
+                   scratch: torch.Tensor | None = None, max_q: int = 0) -> "_n.LightningArgs":
+    """Arguments of the linear attention kernels.  ``m``: a ``LightningSpec``, ``offs`` the sections q, k, v, g of ``proj``'s rows, ``w``
+    carries decay [heads] and out_norm [heads * vdim] (fp32); ``raw`` fp32 [T, heads * vdim]; head h's normed and gated values go to columns
+    [h * head_pitch, + vdim) of ``out``."""
+    p = _n.LightningArgs()
+    p.proj, p.decay, p.norm_w, p.raw, p.out = proj.data_ptr(), w.decay.data_ptr(), w.out_norm.data_ptr(), raw.data_ptr(), out.data_ptr()
+    p.scratch, p.scratch_bytes = _ptr(scratch), scratch.numel() * scratch.element_size() if scratch is not None else 0
+    p.state, p.state_in, p.state_out, p.q_start = state.data_ptr(), state_in.data_ptr(), state_out.data_ptr(), q_start.data_ptr()
+    p.slot_stride, p.s_off, p.ld = state.stride(0), s_off, proj.stride(0)
+    p.q_off, p.k_off, p.v_off, p.g_off = (offs[n] for n in "qkvg")
+    p.T, p.S, p.heads, p.dim, p.vdim = proj.shape[0], q_start.shape[0] - 1, m.heads, m.dim, m.vdim
+    p.ldo, p.out_vd, p.max_q, p.eps = out.stride(0), head_pitch, max_q, eps
+    assert out.stride(1) == 1 and out.dtype == proj.dtype and raw.dtype == state.dtype == torch.float32 and raw.numel() >= p.T * m.heads * m.vdim
+    return p
+
+
+def lightning_step(proj: torch.Tensor, *args, **kw) -> None:
+    """Linear attention over any mix of portions, token by token, then norm and gate (see ``lightning_args``)."""
+    _n.check(_n.cuda_lib().cafd_lightning_step(C.byref(lightning_args(proj, *args, **kw)), int(proj.dtype == torch.float32), _stream()),
+             "lightning_step")
 
 
 def swap_ids(a: torch.Tensor, b: torch.Tensor) -> None:
@@ -750,17 +837,22 @@ def rope_table(positions: torch.Tensor, freq: torch.Tensor, out: torch.Tensor, m
 def conv_rope_kv(proj: torch.Tensor, offs: dict, m, conv_w: torch.Tensor | None, table: torch.Tensor, slots: torch.Tensor, q_out: torch.Tensor,
                  k_cache: torch.Tensor, v_cache: torch.Tensor, *, state: torch.Tensor | None = None, state_off: int = 0,
                  state_in: torch.Tensor | None = None, state_out: torch.Tensor | None = None, q_start: torch.Tensor | None = None,
-                 q_norm: torch.Tensor | None = None, k_norm: torch.Tensor | None = None, eps: float = 0.0) -> None:
+                 q_norm: torch.Tensor | None = None, k_norm: torch.Tensor | None = None, eps: float = 0.0,
+                 v_table: torch.Tensor | None = None) -> None:
     """Convolution over time, norm of queries and keys, rotation and the paged K / V write of one step.  ``m``: an ``AttentionSpec``,
     ``conv_w`` [taps, channels] fp32 (last row = the current token), ``table`` the step's ``rope_table``, ``q_norm`` / ``k_norm`` fp32
-    weights of the norms (``m.qk_norm``)."""
+    weights of the norms (``m.qk_norm``), ``v_table`` the step's table of the values' rotation (``m.v_rope``)."""
     p = _n.ConvRope()
     p.proj, p.conv_w, p.table, p.slots, p.q_start = proj.data_ptr(), _ptr(conv_w), table.data_ptr(), slots.data_ptr(), _ptr(q_start)
     p.q_out, p.k_cache, p.v_cache = q_out.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr()
     p.T, p.ld, p.q_off, p.k_off, p.v_off = proj.shape[0], proj.stride(0), offs["q"], offs["k"], offs.get("v", 0)
     p.nq, p.nk, p.nv = m.q_channels, m.k_channels, 0 if m.v_from_k else m.v_channels
-    p.norm, p.halves, p.v_from_k, p.eps = {"": 0, "head": 1, "all": 2}[m.qk_norm], int(m.rope.halves), int(m.v_from_k), eps
-    if m.qk_norm:
+    p.norm, p.halves, p.v_from_k, p.eps = {"": 0, "head": 1, "all": 2, "rotated": 1}[m.qk_norm], int(m.rope.halves), int(m.v_from_k), eps
+    # a norm after the rotation is one before it whose squares are scaled as the rotation scales them
+    p.rot_sq = m.rope.magnitude ** 2 if m.qk_norm == "rotated" else 1.0
+    p.v_table = v_table.data_ptr() if m.v_rope is not None else None
+    assert m.v_rope is None or (m.v_rope.halves and m.v_rope.dims == m.vdim)
+    if m.qk_norm in ("head", "all"):
         p.q_norm, p.k_norm = q_norm.data_ptr(), k_norm.data_ptr()
         assert q_norm.dtype == k_norm.dtype == torch.float32 and q_norm.is_contiguous() and k_norm.is_contiguous()
         assert (q_norm.numel(), k_norm.numel()) == ((m.dim, m.dim) if m.qk_norm == "head" else (p.nq, p.nk))
@@ -777,17 +869,19 @@ def conv_rope_kv(proj: torch.Tensor, offs: dict, m, conv_w: torch.Tensor | None,
 
 def paged_attn(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, m, page_table: torch.Tensor, positions: torch.Tensor,
                q_start: torch.Tensor, out: torch.Tensor, head_pitch: int, lam: float = 0.0, eps: float = 0.0,
-               sink: torch.Tensor | None = None, gate: torch.Tensor | None = None) -> None:
+               sink: torch.Tensor | None = None, gate: torch.Tensor | None = None, v_table: torch.Tensor | None = None,
+               out_scale: float = 1.0) -> None:
     """Attention at any head sizes: q [T, heads * maps * dim]; head h's values go to columns [h * head_pitch, + vdim) of ``out``
-    (rows of any length).  ``m``: an ``AttentionSpec``; ``lam`` / ``eps``: second map's weight and the head norm's epsilon; ``sink`` and
-    ``gate`` as in ``attn_decode``."""
+    (rows of any length).  ``m``: an ``AttentionSpec``; ``lam`` / ``eps``: second map's weight and the head norm's epsilon; ``sink``,
+    ``gate`` and ``v_table`` as in ``attn_decode``; outputs are multiplied by ``out_scale``."""
     p = _n.PagedAttn()
     p.q, p.k_cache, p.v_cache, p.page_table = q.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(), page_table.data_ptr()
     p.positions, p.q_start, p.out = positions.data_ptr(), q_start.data_ptr(), out.data_ptr()
     p.T, p.heads, p.kv_heads, p.maps, p.dim, p.vdim = q.shape[0], m.heads, m.kv_heads, m.maps, m.dim, m.vdim
     p.S, p.max_pages = page_table.shape
     p.window, p.keep, p.ldo, p.head_pitch = m.window, m.keep_first, out.stride(0), head_pitch
-    p.scale, p.lam, p.out_scale, p.eps = m.scale, lam, 1.0 - m.diff, eps
+    p.scale, p.lam, p.out_scale, p.eps, p.cap = m.scale, lam, (1.0 - m.diff) * out_scale, eps, m.softcap
+    p.v_table = _ptr(v_table)
     p.sink, (p.gate, p.gate_ld) = _ptr(sink), _gate(gate, q, m.heads)
     assert sink is None or (sink.dtype == torch.float32 and sink.numel() == m.heads)
     assert q.is_contiguous() and q.dtype == out.dtype == k_cache.dtype and page_table.is_contiguous() and q_start.shape[0] == p.S + 1

@@ -59,10 +59,17 @@ def workspace_bytes(cfg: ModelConfig, rows: int) -> int:
     intermediates, and the MoE exchange rows (rows x top_k, in and out)."""
     h = cfg.hidden
     if cfg.is_hybrid:
-        attn = max((s.mixer.heads * (2 * s.mixer.record + s.mixer.dim + s.mixer.rot_dim + 3 * s.mixer.vdim) + s.mixer.record)
-                   if hasattr(s.mixer, "kv_rank") else (s.mixer.conv_channels + s.mixer.q_channels + s.mixer.heads * s.mixer.vdim)
-                   if hasattr(s.mixer, "rope") else (s.mixer.conv_channels + 2 * s.mixer.heads * s.mixer.vdim) for s in cfg.layer_specs)
+        def elements(m) -> int:
+            if hasattr(m, "right"):                        # the linear attention's outputs before their norm are fp32
+                return elements(m.left) + m.right.channels + 3 * m.right.heads * m.right.vdim
+            if hasattr(m, "blocks"):                       # so are the gates' products of a linear recurrence
+                return 8 * m.width
+            if hasattr(m, "kv_rank"):
+                return m.heads * (2 * m.record + m.dim + m.rot_dim + 3 * m.vdim) + m.record
+            return m.conv_channels + (m.q_channels + m.heads * m.vdim if hasattr(m, "rope") else 2 * m.heads * m.vdim)
+        attn = max(elements(s.mixer) for s in cfg.layer_specs)
         h *= 2 + 2 * bool(cfg.loop and cfg.loop_join)      # the residual is fp32 and alternates between two buffers; joining rows and what they give
+        attn += 2 * len(cfg.layer_runs) * cfg.hidden * cfg.depth_average      # every layer run's result, fp32
     elif cfg.is_mla:
         attn = (cfg.q_lora_rank + cfg.kv_lora_rank + cfg.qk_rope_dim) + cfg.num_heads * (cfg.qk_head_dim + cfg.v_head_dim + cfg.kv_lora_rank + cfg.qk_rope_dim)
     else:

@@ -93,7 +93,10 @@ def render(rep: PlanReport) -> str:
          f"geometry   {c.num_layers} layers, hidden {c.hidden}, vocab {c.vocab_size}, "
          + (f"MLA {c.num_heads} heads (q_lora {c.q_lora_rank}, kv_lora {c.kv_lora_rank}, nope {c.qk_nope_dim}, rope {c.qk_rope_dim}, v {c.v_head_dim})"
             if c.is_mla else ", ".join(f"{n} {k}" for k, n in sorted(Counter(
-                f"latent (rank {m.kv_rank} + {m.rot_dim}, {m.heads} heads, window {m.window})" if hasattr(m, "kv_rank")
+                f"rg-lru ({m.width} channels, {m.blocks} blocks)" if hasattr(m, "blocks")
+                else (f"attention ({m.left.heads}/{m.left.kv_heads} heads x {m.left.dim} + {m.left.vdim}) beside linear attention "
+                      f"({m.right.heads} heads x {m.right.dim} x {m.right.vdim})") if hasattr(m, "right")
+                else f"latent (rank {m.kv_rank} + {m.rot_dim}, {m.heads} heads, window {m.window})" if hasattr(m, "kv_rank")
                 else (f"{'differential ' if m.maps == 2 else ''}attention ({m.heads}/{m.kv_heads} heads x {m.dim} + {m.vdim}, window {m.window}"
                       f", keeps {m.keep_first}{', values out of keys' if m.v_from_k else ''})") if hasattr(m, "rope")
                 else f"delta ({m.heads} heads x {m.dim} x {m.vdim})" for m in (s.mixer for s in c.layer_specs)).items()))

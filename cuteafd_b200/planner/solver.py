@@ -150,6 +150,7 @@ def component_bytes(cfg: ModelConfig, req: PlacementRequest) -> dict[str, int]:
     if cfg.is_hybrid:                            # per-layer sizes
         dense = [(s.router is not None, 3 * cfg.hidden * s.dense.ffn) for s in cfg.layer_specs if s.dense is not None]
         join = (2 * cfg.hidden + cfg.loop[2]) * cfg.hidden if cfg.loop and cfg.loop_join else 0
+        out["embedding"] += (cfg.bigram[0] + 1) * cfg.hidden * 2 if cfg.bigram else 0
         out["dense_ffn"] = weight_bytes(sum(n for routed, n in dense if not routed) + join, bfmt)
         out["shared_experts"] = weight_bytes(sum(n for routed, n in dense if routed), bfmt)
     return out
