@@ -14,7 +14,7 @@
 // row is complete: here without splits, in the merge with them.
 // A sliding window may come with kept first tokens; their pages are walked before the window's.  A head may have a sink, a number
 // whose exponential joins the softmax's denominator, and an output gate (the sigmoid of one number per token and head); both are
-// applied where a row is complete.
+// applied where a row is complete, and so is a rotation of the output back by the query's position.  Scores may be capped.
 //
 // Reference counterparts: split-KV partial + merge drafter attention
 // (native/shared/cuda/draft_attention.cu:42-295) and the LSE state merge
@@ -76,10 +76,12 @@ struct AttnPeers {
 // Kept first tokens, output row pitch, with two maps how they are combined, with one sinks and gates.
 struct AttnExtras {
   int keep, ldo;
-  float lambda, out_scale, eps;
-  const float* sink;             // [Hq] or null
-  const __nv_bfloat16* gate;     // row t, head h: gate[t * gate_ld + h]; or null
-  int gate_ld;
+  float lambda = 0.f, out_scale = 1.f, eps = 0.f;
+  const float* sink = nullptr;             // [Hq] or null
+  const __nv_bfloat16* gate = nullptr;     // row t, head h: gate[t * gate_ld + h]; or null
+  int gate_ld = 0;
+  const float2* v_table = nullptr;         // [rows, 64] cos, sin; or null; one map only
+  float cap_log2 = 0.f;                    // cap * log2(e): scores are cap * tanh(score / cap), and the kernel's scale is 2 log2(e) * scale / cap; 0 = none
 };
 
 // A complete row of one head: M is the maximum its sums L and O refer to, in log2 units.
@@ -87,7 +89,18 @@ __device__ __forceinline__ float finish_row(float O, float L, float M, const Att
   if (x.sink) L += exp2f(x.sink[head] * 1.4426950408889634f - M);
   float v = L > 0.f ? O / L : 0.f;
   if (x.gate) v /= 1.0f + expf(-__bfloat162float(x.gate[static_cast<size_t>(row) * x.gate_ld + head]));
-  return v;
+  return v * x.out_scale;
+}
+
+// One head's 128 values, one per thread, turned back by the row's angles (pairs 64 apart); every thread of the block calls.
+__device__ __forceinline__ float turn_back(float v, const AttnExtras& x, int row, float* buf) {
+  const int d = threadIdx.x;
+  buf[d] = v;
+  __syncthreads();
+  const float o = buf[d ^ 64];
+  const float2 a = x.v_table[static_cast<size_t>(row) * 64 + (d & 63)];
+  __syncthreads();
+  return d < 64 ? v * a.x + o * a.y : v * a.x - o * a.y;
 }
 
 // The combined value of one head's 128 values, one per thread: a - lambda * b over its root mean square, times out_scale.
@@ -223,7 +236,8 @@ __global__ void __launch_bounds__(128) attn_decode_kernel(
       for (int j = 0; j < 4; ++j) {
         const int half = j >> 1;
         const int tok = tok_base + nt * 8 + 2 * t4 + (j & 1);
-        const float v = (tok < limit[half] && (tok >= lo[half] || tok < ex.keep)) ? s[nt][j] * scale_log2 : -INFINITY;
+        const float z = s[nt][j] * scale_log2;
+        const float v = (tok < limit[half] && (tok >= lo[half] || tok < ex.keep)) ? (ex.cap_log2 > 0.f ? ex.cap_log2 * tanh_exp2(z) : z) : -INFINITY;
         s[nt][j] = v;
         mx[half] = fmaxf(mx[half], v);
       }
@@ -318,6 +332,7 @@ __global__ void __launch_bounds__(128) attn_decode_kernel(
           v = combine_maps(o_map1, v, ex, sm_l + 64);
         } else {
           v = finish_row(O, L, M, ex, q0 + qi, head);
+          if (ex.v_table) v = turn_back(v, ex, q0 + qi, sm_l + 128);
         }
         out[static_cast<size_t>(q0 + qi) * ex.ldo + head * kD + d] = __float2bfloat16(v);
       }
@@ -334,7 +349,7 @@ __global__ void __launch_bounds__(128) attn_merge_kernel(const float* __restrict
                                                          const int* __restrict__ q_start,
                                                          __nv_bfloat16* __restrict__ out, int Hq, int Hkv,
                                                          int tiles_per_seq, int splits, const AttnExtras ex) {
-  __shared__ float red[4];
+  __shared__ float red[kMaps == 2 ? 4 : kD];
   pdl_wait();
   pdl_trigger();
   const int group = Hq / Hkv;
@@ -360,7 +375,7 @@ __global__ void __launch_bounds__(128) attn_merge_kernel(const float* __restrict
     }
     v[m] = kMaps == 1 ? finish_row(O, L, M, ex, q0 + qi, kvh * group + r % group) : L > 0.f ? O / L : 0.f;
   }
-  const float o = kMaps == 2 ? combine_maps(v[0], v[kMaps - 1], ex, red) : v[0];
+  const float o = kMaps == 2 ? combine_maps(v[0], v[kMaps - 1], ex, red) : ex.v_table ? turn_back(v[0], ex, q0 + qi, red) : v[0];
   out[static_cast<size_t>(q0 + qi) * ex.ldo + (kvh * group + r % group) * kD + d] = __float2bfloat16(o);
 }
 
@@ -384,15 +399,16 @@ extern "C" long long cafd_attn_decode_scratch_floats(int num_seqs, int tiles_per
 // q [total_q, Hq, 128] (two maps: [total_q, Hq, 2, 64]); caches [pages, Hkv, 64, 128]; page_table [num_seqs, max_pages];
 // seq_lens [num_seqs] (kv length including the new tokens); q_start [num_seqs + 1]; out rows of ldo elements, head h's values at
 // column 128 h.  max_q_len bounds the query tokens of any sequence; scratch holds the split partials.  keep: kept first tokens
-// beside a window; lambda, out_scale and eps: two maps only; sink [Hq] and gate rows (gate_ld elements apart): one map only.
+// beside a window; lambda and eps: two maps only; out_scale multiplies the output; sink [Hq], gate rows (gate_ld elements apart) and
+// v_table [rows, 64] (cos, sin of the output's rotation back): one map only; cap 0 = scores are not capped.
 extern "C" int cafd_attn_decode(const void* q, const void* k_cache, const void* v_cache, const int* page_table,
                                 const int* seq_lens, const int* q_start, void* out, float* scratch, int num_seqs,
                                 int max_q_len, int max_pages, int Hq, int Hkv, int D, int splits, float scale,
                                 int window, int keep, int ldo, int maps, float lambda, float out_scale, float eps, const float* sink,
-                                const void* gate, int gate_ld, cafd_stream_t s) {
+                                const void* gate, int gate_ld, float cap, const void* v_table, cafd_stream_t s) {
   if (num_seqs <= 0) return 0;
   if (D != kD || Hq % Hkv || window < 0 || keep < 0 || maps < 1 || maps > 2 || ldo < Hq * kD) return -10;
-  if ((maps == 2 && (sink || gate)) || (gate && gate_ld < Hq)) return -10;
+  if ((maps == 2 && (sink || gate || v_table || cap > 0.f)) || (gate && gate_ld < Hq)) return -10;
   const int group = maps * (Hq / Hkv);
   if (group > 16 || 16 % group) return -11;
   if (splits < 1) splits = 1;
@@ -410,12 +426,13 @@ extern "C" int cafd_attn_decode(const void* q, const void* k_cache, const void* 
     attr = true;
   }
   dim3 grid(num_seqs * tiles_per_seq, Hkv, splits);
-  const AttnExtras ex{window > 0 ? keep : 0, ldo, lambda, out_scale, eps, sink, static_cast<const __nv_bfloat16*>(gate), gate_ld};
+  const AttnExtras ex{window > 0 ? keep : 0, ldo, lambda, out_scale, eps, sink, static_cast<const __nv_bfloat16*>(gate), gate_ld,
+                      static_cast<const float2*>(v_table), cap * 1.4426950408889634f};
   auto kern = maps == 2 ? attn_decode_kernel<2> : attn_decode_kernel<1>;
   launch_pdl(kern, grid, dim3(128), smem, st,
       static_cast<const __nv_bfloat16*>(q), static_cast<const __nv_bfloat16*>(k_cache),
       static_cast<const __nv_bfloat16*>(v_cache), page_table, seq_lens, q_start, static_cast<__nv_bfloat16*>(out),
-      scratch, max_pages, Hq, Hkv, tiles_per_seq, splits, scale * 1.4426950408889634f, static_cast<const int*>(nullptr),
+      scratch, max_pages, Hq, Hkv, tiles_per_seq, splits, (cap > 0.f ? 2.f * scale / cap : scale) * 1.4426950408889634f, static_cast<const int*>(nullptr),
       window, fixed_kv_split_tokens() / kPage, AttnPeers{}, ex);
   if (splits > 1) {
     dim3 g2(num_seqs * tiles_per_seq, Hkv, 16 / maps);

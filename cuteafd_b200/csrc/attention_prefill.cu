@@ -28,7 +28,11 @@
 //
 // A sliding window may come with kept first tokens, which every later row sees too: the tiles that hold them are walked
 // before the window's.  A head may have a sink (a number whose exponential joins the softmax's denominator) and an output gate
-// (the sigmoid of one number per token and head): both enter the epilogue's quotient.
+// (the sigmoid of one number per token and head): both enter the epilogue's quotient; the output may be rotated back by the
+// query's position there.
+//
+// kCap: scores are cap * tanh(score / cap).  While every score of a warp's tile is small against the cap, tanh is an odd polynomial
+// (two scores per instruction); else it takes an exponential and a division.
 //
 // Replaces the reference's mma.sync prefill kernels (native/families/glm5/cuda/glm_mla_prefill.cu:78-135)
 // and its exported attention programs for the GQA families.
@@ -66,6 +70,8 @@ struct PrefillDev {
   const float* sink;              // [Hq] or null
   const __nv_bfloat16* gate;      // row t, head h: gate[t * gate_ld + h]; or null
   int gate_ld;
+  const float2* v_table;          // [rows, 64] cos, sin; or null
+  float cap_in, cap_log2;         // kCap: scale / cap, cap * log2(e); scale_log2 is then 1
   // kRope only
   const int* kv_tmp_start; // [seqs] first row of the sequence in the expansion buffers (multiple of 64)
   int q_head_stride;       // elements between heads in the nope query matrix (192 for [T, heads * 192])
@@ -73,7 +79,55 @@ struct PrefillDev {
   int qr_col0;             // first rope column inside a head of that matrix (512)
 };
 
-template <bool kRope, int kMaps>
+// tanh(x) / x as a polynomial in x^2, fitted over |x| <= kTanhRange by least squares at Chebyshev nodes: within 2e-8
+constexpr float kTanhRange = 0.75f;
+__device__ __forceinline__ uint64_t pack_f32x2(float a, float b) {
+  uint64_t r;
+  asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(a), "f"(b));
+  return r;
+}
+__device__ __forceinline__ uint64_t fma_f32x2(uint64_t a, uint64_t b, uint64_t c) {
+  uint64_t r;
+  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c));
+  return r;
+}
+__device__ __forceinline__ uint64_t mul_f32x2(uint64_t a, uint64_t b) {
+  uint64_t r;
+  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
+  return r;
+}
+// 64 scores in place: out * tanh(in * score)
+__device__ __forceinline__ void cap_scores(uint32_t (&r)[64], float in, float out) {
+  float m4[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+  for (int i = 0; i < 64; i += 4) {
+#pragma unroll
+    for (int k = 0; k < 4; ++k) m4[k] = fmaxf(m4[k], fabsf(__uint_as_float(r[i + k])));
+  }
+  const float top = fmaxf(fmaxf(m4[0], m4[1]), fmaxf(m4[2], m4[3])) * fabsf(in);
+  if (__any_sync(0xffffffffu, !(top <= kTanhRange))) {
+    const float arg = 2.f * 1.4426950408889634f * in;
+#pragma unroll
+    for (int i = 0; i < 64; ++i) r[i] = __float_as_uint(out * tanh_exp2(__uint_as_float(r[i]) * arg));
+    return;
+  }
+  constexpr float kC[6] = {0.999999972f, -0.333329667f, 0.133255153f, -0.0533498202f, 0.0195937858f, -0.00472395227f};
+  uint64_t c[6];
+#pragma unroll
+  for (int k = 0; k < 6; ++k) c[k] = pack_f32x2(kC[k] * out, kC[k] * out);
+  const uint64_t s = pack_f32x2(in, in);
+#pragma unroll
+  for (int i = 0; i < 64; i += 2) {
+    const uint64_t x = mul_f32x2(pack_f32x2(__uint_as_float(r[i]), __uint_as_float(r[i + 1])), s), y = mul_f32x2(x, x);
+    uint64_t q = c[5];
+#pragma unroll
+    for (int k = 4; k >= 0; --k) q = fma_f32x2(q, y, c[k]);
+    q = mul_f32x2(q, x);
+    asm("mov.b64 {%0, %1}, %2;" : "=r"(r[i]), "=r"(r[i + 1]) : "l"(q));
+  }
+}
+
+template <bool kRope, int kMaps, bool kCap = false>
 __global__ void __launch_bounds__(kPrefillThreads, 1)
 attn_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ CUtensorMap tm_k,
                     const __grid_constant__ CUtensorMap tm_v, const __grid_constant__ CUtensorMap tm_qr,
@@ -303,6 +357,7 @@ attn_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_const
       tmem_ld_wait();
       tc_fence_before();
       mbar_arrive(&s_empty[st]);
+      if constexpr (kCap) cap_scores(r, p.cap_in, p.cap_log2);
       if (need_mask) {
 #pragma unroll
         for (int i = 0; i < 64; ++i)
@@ -438,6 +493,32 @@ attn_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_const
       if (p.sink) l_run += exp2f(p.sink[head] * 1.4426950408889634f - (m_run == -INFINITY ? 0.f : m_run));   // both halves hold the same maximum
       float inv = l_run > 0.f ? 1.0f / l_run : 0.f;
       if (p.gate && row_ok) inv /= 1.0f + expf(-__bfloat162float(p.gate[static_cast<size_t>(q0 + row0 + row) * p.gate_ld + head]));
+      if constexpr (!kRope) inv *= p.out_scale;
+      if (!kRope && p.v_table) {
+        // values m and m + 64 turn together: this thread takes 32 of either half of the head
+        uint32_t a[32], b[32];
+        tmem_ld_32x32(tO + lane_off + half * 32, a);
+        tmem_ld_32x32(tO + lane_off + 64 + half * 32, b);
+        tmem_ld_wait();
+        if (row_ok) {
+          const float4* cs = reinterpret_cast<const float4*>(p.v_table + static_cast<size_t>(q0 + row0 + row) * 64 + half * 32);
+          __nv_bfloat16* dst = p.out + static_cast<size_t>(q0 + row0 + row) * p.ldo + head * kHD + half * 32;
+#pragma unroll
+          for (int i = 0; i < 32; i += 8) {
+            float u[8], v[8];
+#pragma unroll
+            for (int e = 0; e < 8; e += 2) {
+              const float4 t = cs[(i + e) >> 1];
+              const float a0 = __uint_as_float(a[i + e]) * inv, b0 = __uint_as_float(b[i + e]) * inv;
+              const float a1 = __uint_as_float(a[i + e + 1]) * inv, b1 = __uint_as_float(b[i + e + 1]) * inv;
+              u[e] = a0 * t.x + b0 * t.y; v[e] = b0 * t.x - a0 * t.y;
+              u[e + 1] = a1 * t.z + b1 * t.w; v[e + 1] = b1 * t.z - a1 * t.w;
+            }
+            *reinterpret_cast<uint4*>(dst + i) = make_uint4(pack_bf16(u[0], u[1]), pack_bf16(u[2], u[3]), pack_bf16(u[4], u[5]), pack_bf16(u[6], u[7]));
+            *reinterpret_cast<uint4*>(dst + 64 + i) = make_uint4(pack_bf16(v[0], v[1]), pack_bf16(v[2], v[3]), pack_bf16(v[4], v[5]), pack_bf16(v[6], v[7]));
+          }
+        }
+      } else {
       __nv_bfloat16* orow = p.out + static_cast<size_t>(q0 + row0 + row) * p.ldo + head * kHD + half * 64;
 #pragma unroll 1
       for (int c = 0; c < 2; ++c) {
@@ -456,6 +537,7 @@ attn_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_const
           }
         }
       }
+      }
     }
   }
   tc_fence_before();
@@ -472,16 +554,17 @@ using namespace cafd;
 
 // q [total_q, Hq, 128] bf16 (two maps: [total_q, Hq, 2, 64]); out rows of ldo elements, head h's 128 values at column 128 h;
 // caches [num_pages, Hkv, 64, 128] bf16 (page 0 all zero); page_table [num_seqs, max_pages]; seq_lens [num_seqs];
-// q_start [num_seqs + 1]; max_q_len = longest chunk (grid sizing).  maps 1: lambda, out_scale and eps are unused.
-// sink [Hq] and gate rows (gate_ld elements apart): one map only, null = none.
+// q_start [num_seqs + 1]; max_q_len = longest chunk (grid sizing).  maps 1: lambda and eps are unused.
+// sink [Hq], gate rows (gate_ld elements apart), v_table [total_q, 64] (cos, sin of the output's rotation back) and cap (0 = none): one
+// map only.
 extern "C" int cafd_attn_prefill(const void* q, const void* k_cache, const void* v_cache, const int* page_table,
                                  const int* seq_lens, const int* q_start, void* out, uint32_t* status, int total_q,
                                  int num_seqs, int max_q_len, int num_pages, int max_pages, int Hq, int Hkv, int D,
                                  float scale, int window, int keep, int ldo, int maps, float lambda, float out_scale, float eps,
-                                 const float* sink, const void* gate, int gate_ld, cafd_stream_t s) {
+                                 const float* sink, const void* gate, int gate_ld, float cap, const void* v_table, cafd_stream_t s) {
   if (num_seqs <= 0 || total_q <= 0) return 0;
   if (D != kHD || Hq % Hkv || window < 0 || keep < 0 || maps < 1 || maps > 2 || ldo < Hq * kHD || ldo % 8) return -10;
-  if ((maps == 2 && (sink || gate)) || (gate && gate_ld < Hq)) return -10;
+  if ((maps == 2 && (sink || gate || v_table || cap > 0.f)) || (gate && gate_ld < Hq)) return -10;
   CUtensorMap tq, tk, tv;
   int rc = cached_tmap_2d(&tq, q, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, total_q, static_cast<uint64_t>(Hq) * kHD,
                           static_cast<uint64_t>(Hq) * kHD * 2, kBQ, 64);
@@ -506,7 +589,10 @@ extern "C" int cafd_attn_prefill(const void* q, const void* k_cache, const void*
   p.max_pages = max_pages;
   p.Hq = Hq;
   p.Hkv = Hkv;
-  p.scale_log2 = scale * 1.4426950408889634f;
+  p.scale_log2 = cap > 0.f ? 1.f : scale * 1.4426950408889634f;
+  p.v_table = static_cast<const float2*>(v_table);
+  p.cap_in = cap > 0.f ? scale / cap : 0.f;
+  p.cap_log2 = cap * 1.4426950408889634f;
   p.window = window;
   p.keep = window > 0 ? keep : 0;
   p.ldo = ldo;
@@ -517,11 +603,13 @@ extern "C" int cafd_attn_prefill(const void* q, const void* k_cache, const void*
   if (!attr) {
     CAFD_CHECK_CUDA(cudaFuncSetAttribute(attn_prefill_kernel<false, 1>, cudaFuncAttributeMaxDynamicSharedMemorySize, kPrefillSmem));
     CAFD_CHECK_CUDA(cudaFuncSetAttribute(attn_prefill_kernel<false, 2>, cudaFuncAttributeMaxDynamicSharedMemorySize, kPrefillSmem));
+    CAFD_CHECK_CUDA(cudaFuncSetAttribute(attn_prefill_kernel<false, 1, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, kPrefillSmem));
     attr = true;
   }
   dim3 grid((max_q_len + kBQ - 1) / kBQ, Hq, num_seqs);
   cudaStream_t st = static_cast<cudaStream_t>(s);
   if (maps == 2) launch_pdl(attn_prefill_kernel<false, 2>, grid, dim3(kPrefillThreads), kPrefillSmem, st, tq, tk, tv, tq, tq, p);
+  else if (cap > 0.f) launch_pdl(attn_prefill_kernel<false, 1, true>, grid, dim3(kPrefillThreads), kPrefillSmem, st, tq, tk, tv, tq, tq, p);
   else launch_pdl(attn_prefill_kernel<false, 1>, grid, dim3(kPrefillThreads), kPrefillSmem, st, tq, tk, tv, tq, tq, p);
   return static_cast<int>(cudaGetLastError());
 }

@@ -297,6 +297,8 @@ __device__ __forceinline__ float fast_exp2(float x) {
   asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
   return y;
 }
+// tanh from one exponential: 1 - 2 / (1 + e^2x), to within a few units of fp32 rounding at 1; arg = 2 log2(e) x
+__device__ __forceinline__ float tanh_exp2(float arg) { return 1.0f - __fdividef(2.0f, 1.0f + fast_exp2(arg)); }
 // Gated unit of a feed-forward: kind 0 silu(g) * u, kind 1 cut off at a limit, with a slope and an offset (uniform over a launch).
 struct Glu {
   int kind;

@@ -406,7 +406,7 @@ def tensor_core_latent(cfg: ModelConfig, m: LatentSpec) -> bool:
 def tensor_core_attention(cfg: ModelConfig, m: AttentionSpec) -> bool:
     """Whether the tensor-core attention kernels take this layer: key rows (all maps) and values of 128."""
     rows = m.maps * (m.heads // m.kv_heads)
-    return not m.softcap and engine_dtype(cfg) == torch.bfloat16 and m.maps * m.dim == 128 and m.vdim == 128 and rows <= 16 and 16 % rows == 0
+    return engine_dtype(cfg) == torch.bfloat16 and m.maps * m.dim == 128 and m.vdim == 128 and rows <= 16 and 16 % rows == 0
 
 
 class HybridCache:
@@ -755,8 +755,8 @@ class HybridEngine:
             K.paged_attn(q, k, v, m, b.page_table, b.positions, b.q_start, out, pad8(m.vdim), L.lam, self.cfg.rms_eps, sink=L.sink, gate=gate,
                          v_table=aw.v_table, out_scale=out_scale)
             return
-        kw = dict(scale=m.scale, window=m.window, keep=m.keep_first, maps=m.maps, lam=L.lam, out_scale=1.0 - m.diff, eps=self.cfg.rms_eps,
-                  sink=L.sink, gate=gate)
+        kw = dict(scale=m.scale, window=m.window, keep=m.keep_first, maps=m.maps, lam=L.lam, out_scale=(1.0 - m.diff) * out_scale,
+                  eps=self.cfg.rms_eps, sink=L.sink, gate=gate, cap=m.softcap, v_table=aw.v_table)
         q = q.view(T, m.heads, 128)
         if b.prefill:
             K.attn_prefill(q, k, v, b.page_table, b.seq_lens, b.q_start, out, b.max_q_len, **kw)

@@ -438,12 +438,13 @@ def attn_decode(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, p
                 seq_lens: torch.Tensor, q_start: torch.Tensor, out: torch.Tensor, scratch: torch.Tensor | None,
                 max_q_len: int, splits: int, scale: float | None = None, window: int = 0, keep: int = 0, maps: int = 1,
                 lam: float = 0.0, out_scale: float = 1.0, eps: float = 0.0, sink: torch.Tensor | None = None,
-                gate: torch.Tensor | None = None) -> torch.Tensor:
+                gate: torch.Tensor | None = None, cap: float = 0.0, v_table: torch.Tensor | None = None) -> torch.Tensor:
     """``window`` > 0: a query at position t sees keys (t - window, t] (sliding-window layers) and the first ``keep``; the pages
     between are not read.  ``maps`` 2: q [T, heads, 2 x 64] and keys hold two score maps per head; the output is map 1 - ``lam`` *
     map 2 over its root mean square (``eps`` inside), times ``out_scale``.  ``sink`` [heads] fp32: its exponential joins a head's
-    denominator; ``gate`` [T, heads] (rows of any pitch): a head's output is multiplied by its sigmoid (one map).  ``out``: [T, heads, D], or rows [T, columns] whose first
-    heads * D columns are written."""
+    denominator; ``gate`` [T, heads] (rows of any pitch): a head's output is multiplied by its sigmoid; ``cap``: scores are
+    cap * tanh(score / cap); ``v_table`` [T, 64, 2]: cosines and sines of angles a head's output is turned back by, pairs (i, i + 64) (one
+    map).  ``out``: [T, heads, D], or rows [T, columns] whose first heads * D columns are written."""
     _, Hq, D = q.shape
     Hkv = k_cache.shape[1]                 # pools are [pages, kv heads, 64, D]
     num_seqs, max_pages = page_table.shape
@@ -451,8 +452,8 @@ def attn_decode(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, p
     _n.check(_n.cuda_lib().cafd_attn_decode(q.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(), page_table.data_ptr(),
                                             seq_lens.data_ptr(), q_start.data_ptr(), out.data_ptr(), _ptr(scratch),
                                             num_seqs, max_q_len, max_pages, Hq, Hkv, D, splits, scale, int(window), int(keep),
-                                            _attn_out(q, out, maps), maps, lam, out_scale, eps, _ptr(sink), *_gate(gate, q, Hq), _stream()),
-             "attn_decode")
+                                            _attn_out(q, out, maps), maps, lam, out_scale, eps, _ptr(sink), *_gate(gate, q, Hq), cap,
+                                            _ptr(v_table), _stream()), "attn_decode")
     return out
 
 
@@ -490,7 +491,8 @@ def attn_decode_scratch_floats(num_seqs: int, max_q_len: int, Hq: int, Hkv: int,
 def attn_prefill(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, page_table: torch.Tensor,
                  seq_lens: torch.Tensor, q_start: torch.Tensor, out: torch.Tensor, max_q_len: int,
                  scale: float | None = None, window: int = 0, keep: int = 0, maps: int = 1, lam: float = 0.0, out_scale: float = 1.0,
-                 eps: float = 0.0, sink: torch.Tensor | None = None, gate: torch.Tensor | None = None) -> torch.Tensor:
+                 eps: float = 0.0, sink: torch.Tensor | None = None, gate: torch.Tensor | None = None, cap: float = 0.0,
+                 v_table: torch.Tensor | None = None) -> torch.Tensor:
     """Prompt attention; the arguments mean what they mean for ``attn_decode``."""
     T, Hq, D = q.shape
     num_pages, Hkv = k_cache.shape[0], k_cache.shape[1]
@@ -500,7 +502,7 @@ def attn_prefill(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, 
                                              seq_lens.data_ptr(), q_start.data_ptr(), out.data_ptr(),
                                              status_word(q.device).data_ptr(), T, num_seqs, max_q_len, num_pages,
                                              max_pages, Hq, Hkv, D, scale, int(window), int(keep), _attn_out(q, out, maps), maps, lam,
-                                             out_scale, eps, _ptr(sink), *_gate(gate, q, Hq), _stream()), "attn_prefill")
+                                             out_scale, eps, _ptr(sink), *_gate(gate, q, Hq), cap, _ptr(v_table), _stream()), "attn_prefill")
     return out
 
 
