@@ -250,7 +250,9 @@ def cuda_lib():
         _sig(lib, "cafd_accept_prefix", [P, P, P, I, P, P, P])
         _sig(lib, "cafd_norm_conv", [C.POINTER(NormArgs), I, P])
         _sig(lib, "cafd_bigram_rows", [C.POINTER(BigramArgs), P])
-        for n in ("cafd_rglru_conv", "cafd_rglru_scan"):
+        _sig(lib, "cafd_rglru_step_ok", [I, I, I])
+        _sig(lib, "cafd_lightning_chunked", [C.POINTER(LightningArgs), P])
+        for n in ("cafd_rglru_conv", "cafd_rglru_scan", "cafd_rglru_step"):
             _sig(lib, n, [C.POINTER(RglruArgs), I, P])
         _sig(lib, "cafd_lightning_step", [C.POINTER(LightningArgs), I, P])
         _sig(lib, "cafd_rope_table", [P, P, P, I, I, F, P])

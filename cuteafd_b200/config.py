@@ -691,7 +691,36 @@ def rofapel_bench_gqa(size: str = "base") -> ModelConfig:
                        num_shared_experts=1, norm_topk_prob=True)
 
 
+# Benchmark sizes: width, layers, heads, key / value heads, expert width (heads of 128 in both halves of a pair, recurrences as wide as
+# the model in blocks of 128)
+BUZARAX_SIZES = {"small": (1024, 24, 8, 4, 512), "base": (2048, 24, 16, 8, 1024), "large": (4096, 12, 32, 8, 1536)}
+
+
+def buzarax_bench(size: str = "base") -> ModelConfig:
+    """A Buzarax-shaped stack at the sizes of a real model's layers: attention beside linear attention and gated linear recurrences in
+    turn, a dense feed-forward in the first layer, 64 routed experts (top 6) in the others."""
+    width, layers, heads, kv_heads, ffn = BUZARAX_SIZES[size]
+    att = AttentionSpec(heads=heads, kv_heads=kv_heads, dim=128, vdim=128, window=0, keep_first=0, scale=128 ** -0.5,
+                        rope=RopeSpec(64, 1.0e6, 4.0, 1.0, 32.0, 8192, "yarn", halves=True), qk_norm="rotated", softcap=30.0, unit_sink=True,
+                        v_rope=RopeSpec(128, 1.0e6, halves=True))
+    lin = LightningSpec(heads=heads, dim=128, vdim=128, decay=tuple(1.0 - 2.0 ** (-1 - 8.0 * h / heads) for h in range(heads)))
+    pair, rec = PairSpec(att, lin, 0.8, 0.5), RglruSpec(width=width, blocks=width // 128, conv=4)
+    r = RouterSpec(experts=64, ffn=ffn, top=6, scoring="sigmoid")
+    specs = [LayerSpec(rec if i % 2 else pair, r if i else None, None if i else DenseSpec(6 * ffn, 7.0, 1.702, 1.0), post_norm=True) for i in range(layers)]
+    return post_norm_config(f"buzarax-{size}", 65536, width, specs, eps=1e-5, bigram=(65521, 31, 7), logit_softcap=30.0)
+
+
+def buzarax_bench_gqa(size: str = "base") -> ModelConfig:
+    """The GQA + MoE decoder at the size of ``buzarax_bench``: same width, depth, heads, experts and vocabulary."""
+    width, layers, heads, kv_heads, ffn = BUZARAX_SIZES[size]
+    return ModelConfig(name=f"gqa-moe-{size}", family="qwen3_moe", vocab_size=65536, num_layers=layers, hidden=width, attention="gqa",
+                       num_heads=heads, num_kv_heads=kv_heads, head_dim=128, qk_norm=True, rope_theta=1.0e6, rope_interleaved=False, rms_eps=1e-5,
+                       dense_ffn=6 * ffn, first_dense_layers=1, num_experts=64, expert_ffn=ffn, top_k=6, scoring="softmax",
+                       num_shared_experts=0, norm_topk_prob=True)
+
+
 PRESETS = {
+    "buzarax-base": buzarax_bench,
     "karusun-base": karusun_bench,
     "guberax-base": guberax_bench,
     "rofapel-base": rofapel_bench,

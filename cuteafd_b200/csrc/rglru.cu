@@ -5,6 +5,8 @@
 //   rglru_scan   the gates' products to the output.  One thread per channel walks a sequence's tokens; long portions are cut into
 //                chunks: every chunk's decay and contribution first, then every chunk again from the state that the chunks before it
 //                give
+//   rglru_step   all of it in one launch for steps of up to 32 rows: a block convolves one block's channels, multiplies 32 of them
+//                through both gates and walks their recurrences
 //
 // From the gates' products on everything is fp32, so are the convolution's inputs in the state (the projected rows with their
 // bias).  A step reads one state slot and writes another.
@@ -169,6 +171,116 @@ __global__ void __launch_bounds__(kScanThreads) rglru_scan_kernel(const RglruArg
   }
 }
 
+constexpr int kStepRows = 32, kStepChans = 32, kStepThreads = 256;
+
+// Block (block of channels, 32 of its channels).  u of every row in shared memory; thread (gate row, every fourth token) for the products.
+template <typename E>
+__global__ void __launch_bounds__(kStepThreads) rglru_step_kernel(const RglruArgs p) {
+  extern __shared__ __align__(16) float sm[];
+  constexpr int kTok = kStepRows / 4;
+  const int tid = threadIdx.x, b = blockIdx.x, d0 = blockIdx.y * kStepChans, bs = p.width / p.blocks, kp = p.u_pitch, pitch = kp + 4;
+  const int nd = min(kStepChans, bs - d0), halo = p.taps - 1;
+  float* su = sm;                                // [T][pitch], as the products read it
+  float* sg = su + p.T * pitch;                  // [2][32][T + 1]
+  int* s_seq = reinterpret_cast<int*>(sg + 2 * kStepChans * (p.T + 1));   // [T] sequence, [T] its first row
+  E* sw = reinterpret_cast<E*>(s_seq + (2 * p.T + 3) / 4 * 4);            // [64][kp + 8]
+  constexpr int kV = 16 / static_cast<int>(sizeof(E));
+  // the weights do not depend on anything before this launch
+  const E* w = static_cast<const E*>(p.w) + static_cast<size_t>(b) * 2 * kp * kp;
+  for (int i = tid; i < 2 * kStepChans * (kp / kV); i += kStepThreads) {
+    const int r = i / (kp / kV), c = (i - r * (kp / kV)) * kV, g = r / kStepChans, d = r - g * kStepChans;
+    uint4 x = make_uint4(0, 0, 0, 0);
+    if (d < nd) x = *reinterpret_cast<const uint4*>(w + static_cast<size_t>(g * kp + d0 + d) * kp + c);
+    *reinterpret_cast<uint4*>(sw + r * (kp + 8) + c) = x;
+  }
+  pdl_wait();
+  pdl_trigger();
+  for (int t = tid; t < p.T; t += kStepThreads) {
+    const int s = rg_seq_of(p.q_start, p.S, t);
+    s_seq[t] = s;
+    s_seq[p.T + t] = p.q_start[s];
+  }
+  __syncthreads();
+  const E* proj = static_cast<const E*>(p.proj);
+  auto input = [&](int row, int s, int s_lo, int c) {   // the convolution's input at row, which may lie before this step
+    return row >= s_lo ? de_f<E>(proj[static_cast<size_t>(row) * p.ld + p.x_off + c]) + p.x_bias[c]
+                       : p.state[static_cast<size_t>(p.state_in[s]) * p.slot_stride + p.c_off + static_cast<size_t>(halo + row - s_lo) * p.width + c];
+  };
+  for (int i = tid; i < p.T * kp; i += kStepThreads) {
+    const int t = i / kp, d = i - t * kp;
+    float u = 0.f;
+    if (d < bs) {
+      const int c = b * bs + d, s = s_seq[t], s_lo = s_seq[p.T + t];
+      u = p.conv_b[c];
+#pragma unroll 4
+      for (int j = 0; j <= halo; ++j) u = fmaf(p.conv_w[static_cast<size_t>(j) * p.width + c], input(t - halo + j, s, s_lo, c), u);
+    }
+    su[t * pitch + d] = de_f<E>(de_e<E>(u));
+  }
+  __syncthreads();
+  {
+    const int r = tid >> 2, t0 = tid & 3;
+    float acc[kTok];
+#pragma unroll
+    for (int j = 0; j < kTok; ++j) acc[j] = 0.f;
+    const E* wr = sw + r * (kp + 8);
+    for (int k = 0; k < kp; k += 4) {
+      float wv[4];
+      de_load4(wr + k, wv);
+#pragma unroll
+      for (int j = 0; j < kTok; ++j) {
+        const int t = t0 + 4 * j;
+        if (t < p.T) {
+          const float4 x = *reinterpret_cast<const float4*>(su + t * pitch + k);
+          acc[j] = fmaf(wv[0], x.x, fmaf(wv[1], x.y, fmaf(wv[2], x.z, fmaf(wv[3], x.w, acc[j]))));
+        }
+      }
+    }
+    const int g = r / kStepChans, d = r - g * kStepChans;
+    const float bias = d < nd ? p.gate_bias[static_cast<size_t>(b) * 2 * kp + g * kp + d0 + d] : 0.f;
+#pragma unroll
+    for (int j = 0; j < kTok; ++j)
+      if (t0 + 4 * j < p.T) sg[r * (p.T + 1) + t0 + 4 * j] = sigmoid_f(acc[j] + bias);
+  }
+  __syncthreads();
+  const int d = tid & (kStepChans - 1);
+  if (d >= nd) return;
+  const int c = b * bs + d0 + d;
+  const float rate = -p.c * softplus(p.lam[c]), yb = p.y_bias[c];
+  for (int s = tid / kStepChans; s < p.S; s += kStepThreads / kStepChans) {
+    const int q0 = p.q_start[s], q1 = p.q_start[s + 1];
+    if (q0 >= q1) continue;
+    float* so = p.state + static_cast<size_t>(p.state_out[s]) * p.slot_stride;
+    float S = p.state[static_cast<size_t>(p.state_in[s]) * p.slot_stride + p.s_off + c];
+    for (int t = q0; t < q1; ++t) {
+      const float log_a = rate * sg[d * (p.T + 1) + t];
+      const float x = sqrtf(-expm1f(2.f * log_a)) * sg[(kStepChans + d) * (p.T + 1) + t] * su[t * pitch + d0 + d];
+      S = fmaf(expf(log_a), S, x);
+      static_cast<E*>(p.out)[static_cast<size_t>(t) * p.ldo + c] = de_e<E>(S * gelu_tanh(de_f<E>(proj[static_cast<size_t>(t) * p.ld + p.y_off + c]) + yb));
+    }
+    so[p.s_off + c] = S;
+    for (int j = 0; j < halo; ++j) so[p.c_off + static_cast<size_t>(j) * p.width + c] = input(q1 - halo + j, s, q0, c);
+  }
+}
+
+template <typename E>
+static size_t rglru_step_smem(int T, int u_pitch) {
+  return static_cast<size_t>(T * (u_pitch + 4) + 2 * kStepChans * (T + 1) + (2 * T + 3) / 4 * 4) * 4 + static_cast<size_t>(2 * kStepChans) * (u_pitch + 8) * sizeof(E);
+}
+
+template <typename E>
+static int launch_rglru_step(const RglruArgs& p, cudaStream_t st) {
+  const size_t smem = rglru_step_smem<E>(p.T, p.u_pitch);
+  if (p.T > kStepRows || p.u_pitch % 8 || smem > 200 * 1024) return -12;
+  static bool attr = false;
+  if (!attr) {
+    CAFD_CHECK_CUDA(cudaFuncSetAttribute(rglru_step_kernel<E>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
+    attr = true;
+  }
+  launch_pdl(rglru_step_kernel<E>, dim3(p.blocks, (p.width / p.blocks + kStepChans - 1) / kStepChans), dim3(kStepThreads), smem, st, p);
+  return static_cast<int>(cudaGetLastError());
+}
+
 template <typename E>
 static int launch_rglru_scan(const RglruArgs& p, cudaStream_t st) {
   const int cols = (p.width + kScanThreads - 1) / kScanThreads, chunks = (p.max_q + kScanChunk - 1) / kScanChunk;
@@ -215,4 +327,17 @@ extern "C" int cafd_rglru_scan(const RglruArgs* p, int is_f32, cafd_stream_t s) 
   if (!rglru_args_ok(*p) || !p->gates || !p->out || p->max_q < 1) return -10;
   cudaStream_t st = static_cast<cudaStream_t>(s);
   return is_f32 ? launch_rglru_scan<float>(*p, st) : launch_rglru_scan<__nv_bfloat16>(*p, st);
+}
+
+// Steps of up to 32 rows: convolution, gates and recurrence in one launch (u and gates are not used).
+extern "C" int cafd_rglru_step(const RglruArgs* p, int is_f32, cafd_stream_t s) {
+  if (p->T <= 0) return 0;
+  if (!rglru_args_ok(*p) || !p->w || !p->gate_bias || !p->out) return -10;
+  cudaStream_t st = static_cast<cudaStream_t>(s);
+  return is_f32 ? launch_rglru_step<float>(*p, st) : launch_rglru_step<__nv_bfloat16>(*p, st);
+}
+
+// Whether cafd_rglru_step takes a step of T rows in blocks of u_pitch (padded) channels.
+extern "C" int cafd_rglru_step_ok(int T, int u_pitch, int is_f32) {
+  return T <= kStepRows && u_pitch % 8 == 0 && (is_f32 ? rglru_step_smem<float>(T, u_pitch) : rglru_step_smem<__nv_bfloat16>(T, u_pitch)) <= 200 * 1024;
 }

@@ -152,7 +152,7 @@ def write_file(path: str, tensors: dict[str, torch.Tensor], metadata: dict[str, 
         t = tensors[name].detach().cpu().contiguous()
         if t.dtype not in NAMES:
             raise ValueError(f"{name}: dtype {t.dtype} has no safetensors name")
-        raw = t.view(torch.uint8).reshape(-1).numpy().tobytes() if t.numel() else b""
+        raw = t.reshape(-1).view(torch.uint8).numpy().tobytes() if t.numel() else b""
         header[name] = {"dtype": NAMES[t.dtype], "shape": list(t.shape), "data_offsets": [offset, offset + len(raw)]}
         offset += len(raw)
         blobs.append(raw)

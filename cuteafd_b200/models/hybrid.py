@@ -498,6 +498,7 @@ class HybridEngine:
     embed_rows = None
     EXPANDED_PREFILL_TOKENS = 64     # fresh prompt chunks of at least this many tokens use the expanded-form attention
     CHUNKED_DELTA_TOKENS = 32        # steps with a portion of at least this many tokens take the chunked delta rule
+    CHUNKED_LIGHTNING_TOKENS = 32    # likewise linear attention
     CHUNK_SCRATCH_BYTES = 128 << 20  # its operands of one slab of chunks (about an L2's worth)
     FUSED_ROUTE_TOKENS = 64          # steps up to this many tokens run router scores + selection as one launch
 
@@ -793,8 +794,13 @@ class HybridEngine:
         act = ws.act[:T * L.w_out.shape[1]].view(T, L.w_out.shape[1])
         self._attention(n, i, m.left, h, T, b, act, a=a, out_scale=m.left_scale)
         r = m.right
-        K.lightning_step(a, {k: L.offs["right." + k] for k in "qkvg"}, r, L, self.kv.state, self.kv.offsets[n]["S"], b.state_in, b.state_out,
-                         b.q_start, ws.raw, act[:, m.left.heads * pad8(m.left.vdim):], pad8(r.vdim), self.cfg.rms_eps)
+        args = (a, {k: L.offs["right." + k] for k in "qkvg"}, r, L, self.kv.state, self.kv.offsets[n]["S"], b.state_in, b.state_out,
+                b.q_start, ws.raw, act[:, m.left.heads * pad8(m.left.vdim):], pad8(r.vdim), self.cfg.rms_eps)
+        if b.prefill and b.max_q_len >= self.CHUNKED_LIGHTNING_TOKENS and K.lightning_chunk_ok(r, self.dtype):
+            K.lightning_chunked(*args, self._partials(K.lightning_scratch_bytes(r, T, b.q_start.shape[0] - 1) // 4))
+            self.launches += 2
+        else:
+            K.lightning_step(*args)
         K.linear(act, L.w_out, out=ws.y[:T])
         self.launches += 3
 
@@ -810,11 +816,14 @@ class HybridEngine:
         gates = rw.gates[:m.blocks * ht.t_pad * 2 * bp].view(m.blocks, ht.t_pad, 2 * bp)
         carry = None
         if b.max_q_len > K.RGLRU_CHUNK:
-            need = 2 * m.width * (b.q_start.shape[0] - 1) * -(-b.max_q_len // K.RGLRU_CHUNK)
-            self._partials(need)
-            carry = self._scratch
+            carry = self._partials(2 * m.width * (b.q_start.shape[0] - 1) * -(-b.max_q_len // K.RGLRU_CHUNK))
         out = rw.out[:T]
         args = (a, L.offs, m, L, u, gates, self.kv.state, off["S"], off["conv"], b.state_in, b.state_out, b.q_start, out, carry, b.max_q_len)
+        if K.rglru_step_ok(m, self.dtype, T):
+            K.rglru_step(*args)
+            K.linear(out, L.w_out, out=self.ws.y[:T])
+            self.launches += 2
+            return
         K.rglru_conv(*args)
         K.grouped_linear(u.view(-1, bp), L.w_gates, gates.view(-1, 2 * bp), ht.tile_expert, ht.tile_row0, ht.num_tiles, ht.max_tiles, ht.tile_rows,
                          split_k=False)

@@ -801,6 +801,16 @@ def rglru_scan(proj: torch.Tensor, *args, **kw) -> None:
     _n.check(_n.cuda_lib().cafd_rglru_scan(C.byref(rglru_args(proj, *args, **kw)), int(proj.dtype == torch.float32), _stream()), "rglru_scan")
 
 
+def rglru_step_ok(m, dtype: torch.dtype, T: int) -> bool:
+    """Whether a step of T rows runs as one launch."""
+    return bool(_n.cuda_lib().cafd_rglru_step_ok(T, -(-m.block // 8) * 8, int(dtype == torch.float32)))
+
+
+def rglru_step(proj: torch.Tensor, *args, **kw) -> None:
+    """``rglru_conv``, the gates' products and ``rglru_scan`` of a small step in one launch (see ``rglru_args``)."""
+    _n.check(_n.cuda_lib().cafd_rglru_step(C.byref(rglru_args(proj, *args, **kw)), int(proj.dtype == torch.float32), _stream()), "rglru_step")
+
+
 def lightning_args(proj: torch.Tensor, offs: dict, m, w, state: torch.Tensor, s_off: int, state_in: torch.Tensor, state_out: torch.Tensor,
                    q_start: torch.Tensor, raw: torch.Tensor, out: torch.Tensor, head_pitch: int, eps: float,
                    scratch: torch.Tensor | None = None, max_q: int = 0) -> "_n.LightningArgs":
@@ -823,6 +833,21 @@ def lightning_step(proj: torch.Tensor, *args, **kw) -> None:
     """Linear attention over any mix of portions, token by token, then norm and gate (see ``lightning_args``)."""
     _n.check(_n.cuda_lib().cafd_lightning_step(C.byref(lightning_args(proj, *args, **kw)), int(proj.dtype == torch.float32), _stream()),
              "lightning_step")
+
+
+def lightning_chunk_ok(m, dtype: torch.dtype) -> bool:
+    """Whether the chunked form takes linear attention of this shape."""
+    return dtype == torch.bfloat16 and m.dim in (32, 64, 96, 128) and m.vdim % 64 == 0
+
+
+def lightning_scratch_bytes(m, T: int, S: int) -> int:
+    """Scratch of the chunked form for a step of T rows in S portions."""
+    return (T // 128 + S) * m.heads * m.dim * m.vdim * 4
+
+
+def lightning_chunked(proj: torch.Tensor, *args, **kw) -> None:
+    """``lightning_step`` for prompt portions, 128 tokens at a time on the tensor cores; ``scratch`` of ``lightning_scratch_bytes``."""
+    _n.check(_n.cuda_lib().cafd_lightning_chunked(C.byref(lightning_args(proj, *args, **kw)), _stream()), "lightning_chunked")
 
 
 def swap_ids(a: torch.Tensor, b: torch.Tensor) -> None:

@@ -3,8 +3,8 @@ import dataclasses
 
 import torch
 
-from cuteafd_b200.config import (AttentionSpec, DeltaSpec, DenseSpec, LatentSpec, LayerSpec, RopeSpec, RouterSpec, hybrid_config,
-                                 parallel_config)
+from cuteafd_b200.config import (AttentionSpec, DeltaSpec, DenseSpec, LatentSpec, LayerSpec, LightningSpec, PairSpec, RglruSpec, RopeSpec,
+                                 RouterSpec, hybrid_config, parallel_config, post_norm_config)
 from cuteafd_b200.ref import hybrid as R
 
 
@@ -142,6 +142,51 @@ def joint_config(window=100):
         two_norms(key_valued(4, 2, 128, window, RopeSpec(64, 1e4, 2.0, kind="linear", halves=True), 4), 136),
         two_norms(normed(8, 1, 128, 128, RopeSpec(128, 1e5, halves=True)), 128, 6, 3, 64)], 1e-5, loop=(0, 2, 2), family="rofapel", loop_join=True,
         embed_scale=16.0)
+
+
+def turned(heads=6, kv_heads=2, dim=20, vdim=12, rope=RopeSpec(12, 300.0, 3.0, 1.5, 24.0, 200, "yarn", halves=True), scale=None, cap=4.0):
+    """Attention with queries and keys normed after their rotation, rotated values, capped scores and a sink of logit 0."""
+    return AttentionSpec(heads, kv_heads, dim, vdim, 0, 0, scale if scale is not None else 1.6 * dim ** -0.5, rope, qk_norm="rotated", softcap=cap,
+                         unit_sink=True, v_rope=RopeSpec(vdim, rope.base, halves=True))
+
+
+def fading(heads=5, dim=12, vdim=20, lo=0.55, hi=0.995):
+    """Linear attention whose heads forget at different rates."""
+    return LightningSpec(heads, dim, vdim, tuple(round(lo + (hi - lo) * h / max(1, heads - 1), 6) for h in range(heads)))
+
+
+def post(m, ffn=None, limit=1.1, experts=0, top=0, expert_ffn=0):
+    r = RouterSpec(experts, expert_ffn, top, scoring="sigmoid") if experts else None
+    return LayerSpec(m, r, DenseSpec(ffn, limit, 1.702, 1.0) if ffn else None, post_norm=True)
+
+
+def averaged_config():
+    """Every layer differs: pairs and recurrences of odd sizes, dense and routed feed-forwards and none, one expert of several, blocks of
+    five channels, one to five taps, values wider than one block's columns."""
+    return post_norm_config("averaged", 203, 104, [
+        post(PairSpec(turned(), fading(), 0.7, 0.4), 72),
+        post(RglruSpec(72, 3, 3), experts=6, top=3, expert_ffn=28),
+        post(RglruSpec(60, 5, 5)),
+        post(PairSpec(turned(3, 3, 8, 24, RopeSpec(8, 300.0, halves=True), cap=2.0), fading(2, 40, 136, 0.8), 0.9, 1.3), experts=5, top=1, expert_ffn=16),
+        post(RglruSpec(35, 7, 1), 33, 0.6)], 2e-5, bigram=(97, 31, 5), logit_softcap=9.0)
+
+
+def faint_config():
+    """Values that make a mechanism vanish: one head, one expert, one block, one tap, one bucket, no decay, scales of one, no caps, a
+    width that is no multiple of 8."""
+    return post_norm_config("faint", 77, 90, [
+        post(PairSpec(turned(1, 1, 6, 2, RopeSpec(6, 100.0, halves=True), cap=0.0), LightningSpec(1, 1, 1, (1.0,))), experts=1, top=1, expert_ffn=9),
+        post(RglruSpec(10, 1, 1), 24, 50.0),
+        post(PairSpec(turned(4, 1, 10, 6, RopeSpec(4, 50.0, halves=True)), fading(3, 7, 5, 0.0), 1.0, 0.3))], 1e-3, bigram=(1, 3, 1))
+
+
+def dual_config():
+    """The sizes the tensor-core kernels take, and recurrences in blocks of 128."""
+    return post_norm_config("dual", 500, 256, [
+        post(PairSpec(turned(4, 2, 128, 128, RopeSpec(64, 1e4, 4.0, 1.0, 32.0, 256, "yarn", halves=True), cap=6.0), fading(4, 128, 128, 0.7), 0.8, 0.5), 192),
+        post(RglruSpec(256, 2, 4), experts=8, top=2, expert_ffn=128),
+        post(PairSpec(turned(8, 1, 128, 128, RopeSpec(128, 1e5, halves=True), cap=30.0), fading(2, 64, 64, 0.9, 0.999), 1.2, 0.7), experts=6, top=3, expert_ffn=64),
+        post(RglruSpec(384, 3, 2), 136, 2.0)], 1e-5, bigram=(211, 127, 7), logit_softcap=20.0)
 
 
 def params(cfg, seed=0, spread=0.4):

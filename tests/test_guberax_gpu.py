@@ -1,6 +1,6 @@
 """Stacks of parallel layers on the GPU against the plain oracle: the kernels of differential attention alone (those of the two-norm
-design are in test_rofapel_gpu.py), then the engine through its serving backend, both designs (greedy generation through the
-scheduler is with the other per-layer designs' in test_hybrid_gpu.py)."""
+design are in test_rofapel_gpu.py, those of the design normed after its sublayers in test_buzarax_gpu.py), then the engine through its
+serving backend, all three designs (greedy generation through the scheduler is with the other per-layer designs' in test_hybrid_gpu.py)."""
 import dataclasses
 import json
 import os
@@ -13,8 +13,8 @@ import torch
 from cuteafd_b200.config import RopeSpec
 from cuteafd_b200.ref import hybrid as R
 
-from tests.hybrid_common import (attention, bare_config, err, joined_config, joint_config, lone_config, looped_config, oracle_logits, paired_config,
-                                 params, single_map_config, tokens, write_model)
+from tests.hybrid_common import (attention, averaged_config, bare_config, dual_config, err, faint_config, joined_config, joint_config, lone_config,
+                                 looped_config, oracle_logits, paired_config, params, single_map_config, tokens, write_model)
 from tests.test_hybrid_gpu import DTYPES, SPREAD, backend, check, close, dev, i32, rnd, run_cut
 
 pytestmark = pytest.mark.gpu
@@ -227,7 +227,8 @@ def test_softcap():
 
 
 # ---- engine ------------------------------------------------------------------------------------------------------------
-CASES = [(c, d) for c in (looped_config(), bare_config(), paired_config(), single_map_config(), joined_config(), lone_config(), joint_config())
+CASES = [(c, d) for c in (looped_config(), bare_config(), paired_config(), single_map_config(), joined_config(), lone_config(), joint_config(),
+                          averaged_config(), faint_config(), dual_config())
          for d in ("f32", "bf16")]
 IDS = [f"{c.name}-{d}" for c, d in CASES]
 
@@ -258,10 +259,11 @@ def test_residual_after_every_layer_run(cfg, dtype):
         close(a, b, torch.float32 if dtype == "f32" else torch.bfloat16, 2.0)
 
 
-@pytest.mark.parametrize("cfg", [looped_config(), paired_config(), joined_config(), joint_config()], ids=lambda c: c.name)
+@pytest.mark.parametrize("cfg", [looped_config(), paired_config(), joined_config(), joint_config(), averaged_config(), dual_config()],
+                         ids=lambda c: c.name)
 def test_decode_steps_match_prompt_steps(cfg):
     """The decode form (its own attention kernel, drafts as rows of one step) against prompt portions of the same tokens."""
-    dtype = "f32" if cfg.name in ("looped", "joined") else "bf16"
+    dtype = "f32" if cfg.name in ("looped", "joined", "averaged") else "bf16"
     p, seqs = params(cfg, spread=SPREAD[dtype]), [tokens(n, cfg.vocab_size, n) for n in (230, 66, 131)]
     want = [oracle_logits(cfg, p, t) for t in seqs]
     for rows in ([1, 1, 1], [4, 1, 3]):
@@ -314,7 +316,7 @@ def test_mixed_batches_reuse_pages_and_slots(cfg, dtype):
     check(torch.cat([torch.cat(x) for x in got]), torch.cat(want), dtype)
 
 
-@pytest.mark.parametrize("cfg", [looped_config(), joined_config()], ids=lambda c: c.name)
+@pytest.mark.parametrize("cfg", [looped_config(), joined_config(), averaged_config()], ids=lambda c: c.name)
 def test_a_row_does_not_depend_on_the_cut_or_the_batch(cfg):
     """32-bit: the same row computed in other portions and beside other requests differs by rounding alone."""
     p = params(cfg)
@@ -329,7 +331,7 @@ def test_a_row_does_not_depend_on_the_cut_or_the_batch(cfg):
     assert err(torch.cat(got), alone).max() < 2e-6
 
 
-@pytest.mark.parametrize("cfg", [bare_config(), lone_config()], ids=lambda c: c.name)
+@pytest.mark.parametrize("cfg", [bare_config(), lone_config(), faint_config()], ids=lambda c: c.name)
 def test_long_decoding_and_large_steps(cfg):
     p, toks = params(cfg), tokens(900, cfg.vocab_size, 3)
     want = oracle_logits(cfg, p, toks)
@@ -362,8 +364,9 @@ def test_far_keys_and_kept_tokens_in_the_engine(name):
             assert other[150:].median() > 20 * e[150:].median()
 
 
-@pytest.mark.parametrize("cfg,dtype", [(looped_config(), "f32"), (paired_config(), "bf16"), (joined_config(), "f32"), (joint_config(), "bf16")],
-                         ids=["looped", "paired", "joined", "joint"])
+@pytest.mark.parametrize("cfg,dtype", [(looped_config(), "f32"), (paired_config(), "bf16"), (joined_config(), "f32"), (joint_config(), "bf16"),
+                                       (averaged_config(), "f32"), (dual_config(), "bf16")],
+                         ids=["looped", "paired", "joined", "joint", "averaged", "dual"])
 def test_generator_and_device_loop(cfg, dtype):
     """Greedy generation under decode graphs, and the device-resident decode loop that benchmarks time."""
     from cuteafd_b200.runtime.generate import Generator
@@ -386,7 +389,7 @@ def test_generator_and_device_loop(cfg, dtype):
         assert (best - want[torch.arange(12), o] < 0.06 * best.abs() + 1e-6).all()
 
 
-@pytest.mark.parametrize("cfg", [paired_config(), joint_config()], ids=lambda c: c.name)
+@pytest.mark.parametrize("cfg", [paired_config(), joint_config(), dual_config()], ids=lambda c: c.name)
 def test_serve_builds_over_a_snapshot(tmp_path, cfg):
     """``serve --snapshot``: loading, page and slot pools, scheduler with the n-gram drafter, decode graphs, sampling."""
     from cuteafd_b200.cli import build_parser
@@ -413,7 +416,8 @@ def test_serve_builds_over_a_snapshot(tmp_path, cfg):
     assert len(a) == 24 and a[0] == b[0]
 
 
-@pytest.mark.parametrize("cfg", [looped_config(), paired_config(), joined_config(), joint_config()], ids=lambda c: c.name)
+@pytest.mark.parametrize("cfg", [looped_config(), paired_config(), joined_config(), joint_config(), averaged_config(), dual_config()],
+                         ids=lambda c: c.name)
 @pytest.mark.parametrize("dtype", ["bfloat16", "float32"])
 def test_trace_replay_program(dtype, cfg, tmp_path):
     p = params(cfg, spread=2.0)

@@ -10,7 +10,7 @@ import torch
 from cuteafd_b200.config import RouterSpec
 from cuteafd_b200.ref import hybrid as R
 
-from tests.hybrid_common import delta, err, latent, joined_config, looped_config, narrow_config, odd_config, oracle_logits, params, plain_config, tokens, wide_config, write_model
+from tests.hybrid_common import averaged_config, delta, err, latent, joined_config, looped_config, narrow_config, odd_config, oracle_logits, params, plain_config, tokens, wide_config, write_model
 
 pytestmark = pytest.mark.gpu
 DTYPES = [torch.float32, torch.bfloat16]
@@ -501,7 +501,7 @@ def _greedy(cfg, p, prompt, n):
     return out
 
 
-@pytest.mark.parametrize("cfg", [odd_config(), looped_config(), joined_config()], ids=lambda c: c.name)
+@pytest.mark.parametrize("cfg", [odd_config(), looped_config(), joined_config(), averaged_config()], ids=lambda c: c.name)
 @pytest.mark.parametrize("draft,graphs", [(False, False), (False, True), (True, True)])
 def test_scheduler_generates_like_the_oracle(draft, graphs, cfg):
     from cuteafd_b200.runtime.scheduler import Request, Scheduler, collect
