@@ -52,11 +52,13 @@ def main() -> None:
     ap.add_argument("--levels", default="1,8,32")
     ap.add_argument("--layers", type=int, default=0, help="debug only: fewer layers (marks the run invalid)")
     ap.add_argument("--no-graphs", action="store_true")
-    ap.add_argument("--config", default="qwen3", choices=["qwen3", "dsv3", "karusun", "guberax", "rofapel"],
+    ap.add_argument("--config", default="qwen3", choices=["qwen3", "dsv3", "karusun", "guberax", "rofapel", "buzarax"],
                     help="karusun = the per-layer hybrid (latent attention + delta-rule layers) at the sizes of a real model's layers, and the "
                          "MLA engine at equal size beside it, three sizes (one GPU); guberax = the looped parallel layers (differential attention) "
                          "beside the dense GQA engine at equal size, three sizes (one GPU); rofapel = parallel layers of latent, windowed and plain "
-                         "attention beside routed experts, some looped, beside the GQA + MoE engine at equal size, three sizes (one GPU); qwen3 = the headline Qwen3-30B-A3B bf16 card (with 8 GPUs the DeepSeek-V3 card follows it); dsv3 = only "
+                         "attention beside routed experts, some looped, beside the GQA + MoE engine at equal size, three sizes (one GPU); buzarax = attention "
+                         "beside linear attention and gated linear recurrences in turn, before routed experts, beside the GQA + MoE engine at equal size, "
+                         "three sizes (one GPU); qwen3 = the headline Qwen3-30B-A3B bf16 card (with 8 GPUs the DeepSeek-V3 card follows it); dsv3 = only "
                          "the DeepSeek-V3 shape: MLA attention replicas, E4M3 block-scaled experts on the other GPUs (needs 8 GPUs)")
     ap.add_argument("--attention-ranks", type=int, default=0,
                     help="data-parallel attention replicas of the disaggregated layout (0 = 1 on two GPUs, 2 on four or more)")
@@ -116,6 +118,11 @@ def main() -> None:
             assert world == 1, "per-layer designs run on one GPU"
             kind, _, size = name.partition(":")
             cfg = (rofapel_bench if kind == "rofapel" else rofapel_bench_gqa)(size or "base")
+        if name.startswith("buzarax"):            # buzarax[-gqa][:size]
+            from cuteafd_b200.config import buzarax_bench, buzarax_bench_gqa
+            assert world == 1, "per-layer designs run on one GPU"
+            kind, _, size = name.partition(":")
+            cfg = (buzarax_bench if kind == "buzarax" else buzarax_bench_gqa)(size or "base")
         if name == "dsv3":
             from cuteafd_b200 import deepseek_v3
             cfg = deepseek_v3().replace(mtp_layers=0)
@@ -244,9 +251,9 @@ def main() -> None:
         except Exception as e:                   # the headline line is still printed
             if rank == 0 and out is not None:
                 out["extra"]["dsv3_error"] = f"{type(e).__name__}: {e}"
-    if args.config in ("karusun", "guberax", "rofapel") and out is not None:
+    if args.config in ("karusun", "guberax", "rofapel", "buzarax") and out is not None:
         # the closest model's engine at equal size, then both at the other sizes
-        other = {"karusun": "karusun-mla", "guberax": "guberax-gqa", "rofapel": "rofapel-gqa"}[args.config]
+        other = {"karusun": "karusun-mla", "guberax": "guberax-gqa", "rofapel": "rofapel-gqa", "buzarax": "buzarax-gqa"}[args.config]
         for name in [f"{other}:base"] + [f"{k}:{s}" for s in ("small", "large") for k in (args.config, other)]:
             c, r2, _, k2 = run_config(name)
             out["extra"].update(card_extra(r2, c.name.replace("-", "_") + "_"))

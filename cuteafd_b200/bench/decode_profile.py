@@ -26,7 +26,7 @@ def main() -> None:
     ap.add_argument("--context", type=int, default=8192)
     ap.add_argument("--layers", type=int, default=2)
     ap.add_argument("--steps", type=int, default=3)
-    ap.add_argument("--config", default="qwen3", choices=["qwen3", "dsv3", "karusun", "guberax", "rofapel", "rofapel-gqa"])
+    ap.add_argument("--config", default="qwen3", choices=["qwen3", "dsv3", "karusun", "guberax", "rofapel", "rofapel-gqa", "buzarax", "buzarax-gqa"])
     ap.add_argument("--size", default="base", choices=["small", "base", "large"], help="benchmark size of a per-layer design")
     a = ap.parse_args()
     dev = torch.device("cuda:0")
@@ -38,7 +38,7 @@ def main() -> None:
         cfg = deepseek_v3().replace(num_layers=a.layers, first_dense_layers=1, mtp_layers=0)
         W = MlaMoeWeights.random_init(cfg, dev)
         eng = MlaMoeEngine(cfg, W, LatentCache(cfg, pages, dev), max_tokens=a.context, max_seqs=a.concurrency)
-    elif a.config in ("karusun", "guberax", "rofapel"):
+    elif a.config in ("karusun", "guberax", "rofapel", "buzarax"):
         from .. import config as C
         from ..models.hybrid import HybridCache, HybridEngine, HybridWeights
         cfg = getattr(C, a.config + "_bench")(a.size)
@@ -47,9 +47,9 @@ def main() -> None:
         eng = HybridEngine(cfg, W, HybridCache(cfg, pages, dev, 2 + 4 * a.concurrency), max_tokens=a.context, max_seqs=a.concurrency)
     else:
         cfg = qwen3_30b_a3b()
-        if a.config == "rofapel-gqa":
-            from ..config import rofapel_bench_gqa
-            cfg = rofapel_bench_gqa(a.size)
+        if a.config.endswith("-gqa"):
+            from .. import config as C
+            cfg = getattr(C, a.config.replace("-", "_bench_"))(a.size)
         cfg = cfg.replace(num_layers=a.layers)
         W = GqaMoeWeights.random_init(cfg, dev)
         eng = GqaMoeEngine(cfg, W, KvCache(cfg, pages, dev), max_tokens=a.context, max_seqs=a.concurrency)

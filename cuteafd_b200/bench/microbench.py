@@ -530,6 +530,117 @@ def bench_two_norm(a, dev, pk) -> None:
     assert K.read_status() == 0
 
 
+def bench_post_norm(a, dev, pk) -> None:
+    """The kernels of layers normed after their sublayers (averages over depth, gated linear recurrences, attention with capped scores and
+    turned values beside linear attention) beside the like kernels of the GQA + MoE decoder and of the delta-rule hybrid, at one of the
+    benchmark sizes."""
+    from ..config import BUZARAX_SIZES, DeltaSpec, LayerSpec, buzarax_bench, hybrid_config, scaled_down
+    from ..models.hybrid import HybridCache, HybridEngine, HybridWeights, pad8, rope_frequencies
+    H, layers, heads, kvh, ffn = BUZARAX_SIZES[a.size]
+    cfg, bf, T, top, E = buzarax_bench(a.size), torch.bfloat16, a.tokens, 6, 64
+    att, lin, rec = cfg.layer_specs[0].mixer.left, cfg.layer_specs[0].mixer.right, cfg.layer_specs[1].mixer
+
+    def i32(v):
+        return torch.tensor(list(v), dtype=torch.int32, device=dev)
+
+    def rand(*s):
+        return torch.randn(*s, device=dev, dtype=bf)
+
+    def run(name, fn, nbytes, flops=0.0):
+        report(name, time_eager(fn, dev, a.iters), flops, nbytes, pk)
+    small = scaled_down(cfg, 2, 128)
+    W = HybridWeights.random_init(small, dev)
+    L0, L1 = W.layers
+    delta = DeltaSpec(heads, heads // 2, 128, 128, 4)
+    dcfg = hybrid_config("bench", 128, H, [LayerSpec(delta)], 4, 4, 1e-5)
+    Ld = HybridWeights.random_init(dcfg, dev).layers[0]
+    w = torch.ones(H, device=dev, dtype=bf)
+    for n in (1, 8, 32, T):
+        S = n if n < T else 1
+        x, xo, y, yo, h, ys = torch.randn(n, H, device=dev), torch.empty(n, H, device=dev), *(rand(n, H) for _ in range(3)), rand(n * top, H)
+        idx, sw = torch.randint(0, E, (n, top), device=dev, dtype=torch.int32), torch.rand(n, top, device=dev)
+        half = layers // 2
+        past, pw = torch.randn(half + 1, n, H, device=dev), torch.rand(half + 1, device=dev)
+        run(f"norm_conv, norm of the sublayer, {n} rows", lambda: K.norm_conv(h, None, 1, 1e-5, x_in=x, y=y, w_b=w, x_out=xo), n * H * 12)
+        run(f"(GQA) rmsnorm {n} rows", lambda: K.rmsnorm(y, w, 1e-5, out=h), n * H * 4)
+        run(f"norm_conv, routed rows, average over {half} + 1 results, {n} rows",
+            lambda: K.norm_conv(h, None, 1, 1e-5, x_in=x, y=ys, slots=(sw, idx, E, y), w_b=w, x_out=xo, past=(past[:half], pw, past[half])),
+            n * H * (14 + 2 * top + 4 * half))
+        run(f"(GQA) combine + norm {n} rows", lambda: K.moe_combine(ys, sw, h, residual=y, norm_w=w, eps=1e-5, x_out=yo), n * H * (6 + 2 * top))
+        ctx, pps = T, (T + 63) // 64
+        kc, vc = rand(S * pps + 1, kvh, 64, 128), rand(S * pps + 1, kvh, 64, 128)
+        table = (torch.arange(S * pps, dtype=torch.int32, device=dev) + 1).view(S, pps).contiguous()
+        pos = i32([ctx - 1] * S) if n < T else i32(range(T))
+        slots = (table[:, -1] * 64 + 63).int() if n < T else i32(range(64, 64 + T))
+        qs, sl = (i32(range(S + 1)), i32([ctx] * S)) if n < T else (i32([0, T]), i32([T]))
+        si, so = i32(range(2, 2 + S)), i32(range(2 + S, 2 + 2 * S))
+        q, tab, vtab = rand(n, heads, 128), torch.empty(n, att.rope.dims // 2, 2, device=dev), torch.empty(n, 64, 2, device=dev)
+        K.rope_table(pos, rope_frequencies(att.rope).to(dev), tab, att.rope.magnitude)
+        K.rope_table(pos, rope_frequencies(att.v_rope).to(dev), vtab)
+        proj = rand(n, L0.w_in.shape[0])
+        C = att.conv_channels
+        run(f"conv_norm_rope_kv, norms after rotation, turned values, {n} rows",
+            lambda: K.conv_rope_kv(proj, L0.offs, att, None, tab, slots, q, kc, vc, eps=1e-5, v_table=vtab), n * C * 4)
+        nb, f64, qkv = torch.ones(128, device=dev, dtype=bf), torch.ones(64, device=dev), rand(n, C)
+        run(f"(GQA) qk_rope_kv with norms {n} rows", lambda: K.qk_rope_kv(qkv, nb, nb, f64, pos, slots, q, kc, vc, heads, kvh, 128, 1e-5, False), n * C * 4)
+        out, wide = rand(n, heads, 128), rand(n, L0.w_out.shape[1])
+        kw = dict(scale=att.scale, sink=torch.zeros(heads, device=dev), cap=att.softcap, v_table=vtab, out_scale=0.8)
+        qn = torch.nn.functional.rms_norm(q.float(), (128,)).to(bf)
+        for tag, k2, o in (("capped, turned, ", kw, wide), ("(GQA) ", {}, out)):
+            if n == T:
+                run(f"attn_prefill, {tag}{T} tokens", lambda: K.attn_prefill(qn, kc, vc, table, sl, qs, o, T, **k2), T * C * 4, T * T / 2 * heads * 512)
+            else:
+                sp = K.attn_decode_splits(S, 1, kvh, pps)
+                sc = torch.empty(K.attn_decode_scratch_floats(S, 1, heads, kvh, sp), device=dev)
+                run(f"attn_decode, {tag}{S} x {ctx}, {sp} splits", lambda: K.attn_decode(qn, kc, vc, table, sl, qs, o, sc, 1, sp, **k2), S * ctx * kvh * 512)
+        eng = HybridEngine(small, W, HybridCache(small, 4, dev, 2 + 2 * S), max_tokens=n, max_seqs=S)
+        off, act = eng.kv.offsets, wide[:, heads * pad8(128):]
+        args = (proj, {k: L0.offs["right." + k] for k in "qkvg"}, lin, L0, eng.kv.state, off[0]["S"], si, so, qs, eng.ws.raw, act, 128, 1e-5)
+        dproj, dout = rand(n, Ld.w_in.shape[0]), torch.empty(n, heads, 128, device=dev, dtype=bf)
+        dkv = HybridCache(dcfg, 4, dev, 2 + 2 * S)
+        dargs = (dproj, Ld.offs, delta, Ld, dkv.state, dkv.offsets[0]["S"], dkv.offsets[0]["conv"], si, so, qs)
+        rproj, rw = rand(n, L1.w_in.shape[0]), eng._rglru[rec]
+        state_bytes = heads * 128 * 128 * 8
+        if n < T:
+            run(f"linear attention + norm, {S} sequences x {heads} heads", lambda: K.lightning_step(*args), S * state_bytes + n * heads * 128 * 10)
+            run(f"(delta) delta_step {S} sequences x {heads} heads", lambda: K.delta_step(*dargs, dout, None, 1e-5), S * state_bytes + n * heads * 128 * 8)
+        else:
+            sc = torch.empty(K.lightning_scratch_bytes(lin, T, 1), dtype=torch.uint8, device=dev)
+            flops = 2.0 * T * heads * (2 * 128 * 128 + 2 * 64 * 128)
+            run(f"linear attention in chunks + norm, {T} tokens x {heads} heads", lambda: K.lightning_chunked(*args, sc), T * heads * 128 * 10, flops)
+            raw, scd = torch.empty(T * heads * 128, device=dev), torch.empty(128 << 20, dtype=torch.uint8, device=dev)
+            run(f"(delta) delta_chunked {T} tokens x {heads} heads", lambda: K.delta_chunked(scd, *dargs, dout, raw, 1e-5), T * heads * 128 * 8,
+                2.0 * T * heads * (64 * 128 * 5 + 128 * 128 * 3))
+            del raw, scd, sc
+        from ..models.mla_moe import _HeadTiles
+        ht = _HeadTiles(n, rec.blocks, dev)
+        u = rw.u[:rec.blocks * ht.t_pad * 128].view(rec.blocks, ht.t_pad, 128)
+        gates = rw.gates[:rec.blocks * ht.t_pad * 256].view(rec.blocks, ht.t_pad, 256)
+        carry = torch.empty(2 * rec.width * S * -(-T // K.RGLRU_CHUNK), device=dev) if n == T else None
+        rargs = (rproj, L1.offs, rec, L1, u, gates, eng.kv.state, off[1]["S"], off[1]["conv"], si, so, qs, rw.out[:n], carry, T if n == T else 1)
+        gate_w = rec.width * 128 * 4
+        if K.rglru_step_ok(rec, bf, n):
+            run(f"recurrence in one launch, {n} rows", lambda: K.rglru_step(*rargs), gate_w + S * rec.width * 32 + n * rec.width * 6)
+        run(f"recurrence: convolution {n} rows", lambda: K.rglru_conv(*rargs), n * rec.width * 4)
+        run(f"recurrence: products of the gates {n} rows", lambda: K.grouped_linear(u.view(-1, 128), L1.w_gates, gates.view(-1, 256), ht.tile_expert, ht.tile_row0,
+                                                                                    ht.num_tiles, ht.max_tiles, ht.tile_rows, split_k=False),
+            gate_w + n * rec.width * 10, 2.0 * n * rec.width * 256)
+        run(f"recurrence: scan {n} rows", lambda: K.rglru_scan(*rargs), n * rec.width * 14)
+        del eng
+        z, i_, w_ = torch.empty(n, E, device=dev), torch.empty(n, top, dtype=torch.int32, device=dev), torch.empty(n, top, device=dev)
+        rwt, rb = rand(E, H), torch.zeros(E, device=dev)
+        for tag, k2 in (("sigmoid ", dict(scoring="sigmoid", bias=rb, normalize=False)), ("(GQA) ", dict(scoring="softmax"))):
+            if n <= 64:
+                run(f"{tag}norm_route {n} rows", lambda: K.norm_route(h, None, 0.0, rwt, None, i_, w_, top, **k2), E * H * 2 + n * H * 2)
+            else:
+                run(f"{tag}route_topk {n} rows", lambda: K.route_topk(z, top, out_idx=i_, out_w=w_, **k2), n * E * 4 + n * top * 8)
+        F = 6 * ffn
+        o = rand(n, F)
+        for tag, k2 in (("clipped ", dict(glu=(7.0, 1.702, 1.0))), ("(GQA) ", {})):
+            run(f"{tag}gate / up product {n} rows", lambda: K.linear(h, L0.d_gate, out=o, w_up=L0.d_up, **k2), 4 * F * H + n * (H + F) * 2, 4.0 * n * H * F)
+    assert K.read_status() == 0
+
+
 def main() -> None:
     ap = argparse.ArgumentParser()
     sub = ap.add_subparsers(dest="cmd", required=True)
@@ -575,7 +686,9 @@ def main() -> None:
     pa.add_argument("--size", default="base", choices=["small", "base", "large"]); pa.add_argument("--tokens", type=int, default=8192)
     tn = sub.add_parser("two-norm")
     tn.add_argument("--size", default="base", choices=["small", "base", "large"]); tn.add_argument("--tokens", type=int, default=8192)
-    for s in (g, p, d, m, ml, mp_, w4, sm, hy, pa, tn):
+    pn = sub.add_parser("post-norm")
+    pn.add_argument("--size", default="base", choices=["small", "base", "large"]); pn.add_argument("--tokens", type=int, default=8192)
+    for s in (g, p, d, m, ml, mp_, w4, sm, hy, pa, tn, pn):
         s.add_argument("--iters", type=int, default=10)
     a = ap.parse_args()
     dev = torch.device("cuda", int(os.environ.get("LOCAL_RANK", "0")))
@@ -583,7 +696,7 @@ def main() -> None:
     pk = peaks()
     {"exl3": bench_exl3, "gemm-fp8": bench_gemm_fp8, "indexer": bench_indexer, "gemm": bench_gemm, "attn-prefill": bench_attn_prefill, "attn-decode": bench_attn_decode, "moe": bench_moe,
      "mla": bench_mla, "mla-prefill": bench_mla_prefill_expanded, "w4": bench_w4, "sampler": bench_sampler, "hybrid": bench_hybrid,
-     "parallel": bench_parallel, "two-norm": bench_two_norm}[a.cmd](a, dev, pk)
+     "parallel": bench_parallel, "two-norm": bench_two_norm, "post-norm": bench_post_norm}[a.cmd](a, dev, pk)
 
 
 if __name__ == "__main__":

@@ -175,7 +175,7 @@ def faint_config():
     """Values that make a mechanism vanish: one head, one expert, one block, one tap, one bucket, no decay, scales of one, no caps, a
     width that is no multiple of 8."""
     return post_norm_config("faint", 77, 90, [
-        post(PairSpec(turned(1, 1, 6, 2, RopeSpec(6, 100.0, halves=True), cap=0.0), LightningSpec(1, 1, 1, (1.0,))), experts=1, top=1, expert_ffn=9),
+        post(PairSpec(turned(1, 1, 6, 2, RopeSpec(6, 100.0, halves=True), cap=0.0), LightningSpec(1, 1, 4, (1.0,))), experts=1, top=1, expert_ffn=9),
         post(RglruSpec(10, 1, 1), 24, 50.0),
         post(PairSpec(turned(4, 1, 10, 6, RopeSpec(4, 50.0, halves=True)), fading(3, 7, 5, 0.0), 1.0, 0.3))], 1e-3, bigram=(1, 3, 1))
 
