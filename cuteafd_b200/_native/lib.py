@@ -97,7 +97,7 @@ class BigramArgs(C.Structure):
 
 class RglruArgs(C.Structure):
     """cafd_rglru_* (csrc/rglru.cu)."""
-    _fields_ = [(n, C.c_void_p) for n in ("proj", "y_bias", "x_bias", "conv_w", "conv_b", "lam", "w", "gate_bias", "u", "gates", "out", "carry",
+    _fields_ = [(n, C.c_void_p) for n in ("proj", "y_bias", "x_bias", "conv_w", "conv_b", "lam", "w", "gate_bias", "u", "gates", "out",
                                           "state", "state_in", "state_out", "q_start")]
     _fields_ += [(n, C.c_longlong) for n in ("slot_stride", "s_off", "c_off")]
     _fields_ += [(n, C.c_int) for n in ("T", "S", "ld", "x_off", "y_off", "width", "blocks", "taps", "u_pitch", "t_pad", "ldo", "max_q")]

@@ -616,8 +616,7 @@ def bench_post_norm(a, dev, pk) -> None:
         ht = _HeadTiles(n, rec.blocks, dev)
         u = rw.u[:rec.blocks * ht.t_pad * 128].view(rec.blocks, ht.t_pad, 128)
         gates = rw.gates[:rec.blocks * ht.t_pad * 256].view(rec.blocks, ht.t_pad, 256)
-        carry = torch.empty(2 * rec.width * S * -(-T // K.RGLRU_CHUNK), device=dev) if n == T else None
-        rargs = (rproj, L1.offs, rec, L1, u, gates, eng.kv.state, off[1]["S"], off[1]["conv"], si, so, qs, rw.out[:n], carry, T if n == T else 1)
+        rargs = (rproj, L1.offs, rec, L1, u, gates, eng.kv.state, off[1]["S"], off[1]["conv"], si, so, qs, rw.out[:n], T if n == T else 1)
         gate_w = rec.width * 128 * 4
         if K.rglru_step_ok(rec, bf, n):
             run(f"recurrence in one launch, {n} rows", lambda: K.rglru_step(*rargs), gate_w + S * rec.width * 32 + n * rec.width * 6)

@@ -814,12 +814,9 @@ class HybridEngine:
         ht = self._tiles[key]
         u = rw.u[:m.blocks * ht.t_pad * bp].view(m.blocks, ht.t_pad, bp)
         gates = rw.gates[:m.blocks * ht.t_pad * 2 * bp].view(m.blocks, ht.t_pad, 2 * bp)
-        carry = None
-        if b.max_q_len > K.RGLRU_CHUNK:
-            carry = self._partials(2 * m.width * (b.q_start.shape[0] - 1) * -(-b.max_q_len // K.RGLRU_CHUNK))
         out = rw.out[:T]
-        args = (a, L.offs, m, L, u, gates, self.kv.state, off["S"], off["conv"], b.state_in, b.state_out, b.q_start, out, carry, b.max_q_len)
-        if K.rglru_step_ok(m, self.dtype, T):
+        args = (a, L.offs, m, L, u, gates, self.kv.state, off["S"], off["conv"], b.state_in, b.state_out, b.q_start, out, b.max_q_len)
+        if K.rglru_step_ok(m, self.dtype, max(T, b.q_start.shape[0] - 1)):
             K.rglru_step(*args)
             K.linear(out, L.w_out, out=self.ws.y[:T])
             self.launches += 2
@@ -829,7 +826,7 @@ class HybridEngine:
                          split_k=False)
         K.rglru_scan(*args)
         K.linear(out, L.w_out, out=self.ws.y[:T])
-        self.launches += 4 + (carry is not None)
+        self.launches += 4
 
     def _dense(self, i: int, d: DenseSpec, h: torch.Tensor, T: int) -> None:
         L, F = self.W.layers[i], pad8(d.ffn)

@@ -768,25 +768,20 @@ def bigram_rows(tokens: torch.Tensor, bigram: tuple, state: torch.Tensor, off: i
     _n.check(_n.cuda_lib().cafd_bigram_rows(C.byref(a), _stream()), "bigram_rows")
 
 
-RGLRU_CHUNK = 128                    # portions longer than this are cut into chunks of it
-
-
 def rglru_args(proj: torch.Tensor, offs: dict, m, w, u: torch.Tensor, gates: torch.Tensor | None, state: torch.Tensor, s_off: int, c_off: int,
-               state_in: torch.Tensor, state_out: torch.Tensor, q_start: torch.Tensor, out: torch.Tensor, carry: torch.Tensor | None = None,
-               max_q: int = 0) -> "_n.RglruArgs":
+               state_in: torch.Tensor, state_out: torch.Tensor, q_start: torch.Tensor, out: torch.Tensor, max_q: int = 0) -> "_n.RglruArgs":
     """Arguments of the gated linear recurrence's kernels.  ``m``: an ``RglruSpec``; ``w`` carries x_bias, y_bias, conv_b, lam [width], conv_w
     [taps, width], w_gates [blocks, 2 * block (padded), block (padded)] and gate_bias [blocks, 2 * block (padded)] (fp32 but for w_gates);
     ``u`` [blocks, t_pad, block (padded)] convolved rows, ``gates`` fp32 [blocks, t_pad, 2 * block (padded)]."""
     p = _n.RglruArgs()
     p.proj, p.y_bias, p.x_bias, p.conv_w, p.conv_b = proj.data_ptr(), w.y_bias.data_ptr(), w.x_bias.data_ptr(), w.conv_w.data_ptr(), w.conv_b.data_ptr()
     p.lam, p.w, p.gate_bias, p.u, p.gates, p.out = w.lam.data_ptr(), w.w_gates.data_ptr(), w.gate_bias.data_ptr(), u.data_ptr(), _ptr(gates), out.data_ptr()
-    p.carry, p.state, p.state_in, p.state_out, p.q_start = _ptr(carry), state.data_ptr(), state_in.data_ptr(), state_out.data_ptr(), q_start.data_ptr()
+    p.state, p.state_in, p.state_out, p.q_start = state.data_ptr(), state_in.data_ptr(), state_out.data_ptr(), q_start.data_ptr()
     p.slot_stride, p.s_off, p.c_off = state.stride(0), s_off, c_off
     p.T, p.S, p.ld, p.x_off, p.y_off, p.width, p.blocks, p.taps = proj.shape[0], q_start.shape[0] - 1, proj.stride(0), offs["x"], offs["y"], m.width, m.blocks, m.conv
     p.t_pad, p.u_pitch, p.ldo, p.max_q, p.c = u.shape[1], u.shape[2], out.stride(0), max_q, m.c
     assert u.is_contiguous() and u.dtype == proj.dtype == out.dtype and out.stride(1) == 1 and state.dtype == torch.float32
     assert gates is None or (gates.is_contiguous() and gates.dtype == torch.float32 and gates.shape == (m.blocks, p.t_pad, 2 * p.u_pitch))
-    assert carry is None or carry.numel() >= 2 * m.width * p.S * -(-max_q // RGLRU_CHUNK)
     assert w.conv_w.shape == (m.conv, m.width) and w.gate_bias.shape == (m.blocks, 2 * p.u_pitch) and u.shape[0] == m.blocks
     return p
 
@@ -802,7 +797,7 @@ def rglru_scan(proj: torch.Tensor, *args, **kw) -> None:
 
 
 def rglru_step_ok(m, dtype: torch.dtype, T: int) -> bool:
-    """Whether a step of T rows runs as one launch."""
+    """Whether a step of up to T rows and sequences runs as one launch."""
     return bool(_n.cuda_lib().cafd_rglru_step_ok(T, -(-m.block // 8) * 8, int(dtype == torch.float32)))
 
 

@@ -302,8 +302,7 @@ def test_gated_linear_recurrence(dtype, m):
         ht = _HeadTiles(T, m.blocks, dev())
         u, gates = torch.zeros(m.blocks, ht.t_pad, bp, dtype=dtype, device=dev()), torch.empty(m.blocks, ht.t_pad, 2 * bp, device=dev())
         out = torch.full((T, pad8(m.width)), 5.0, dtype=dtype, device=dev())
-        carry = torch.empty(2 * m.width * 4 * -(-max(lens) // K.RGLRU_CHUNK), device=dev())
-        args = (a.to(dev(), dtype), offs, m, w, u, gates, state, 32, conv_at, i32(slots), i32(outs), i32(qs), out, carry, max(lens))
+        args = (a.to(dev(), dtype), offs, m, w, u, gates, state, 32, conv_at, i32(slots), i32(outs), i32(qs), out, max(lens))
 
         def three():
             K.rglru_conv(*args)
