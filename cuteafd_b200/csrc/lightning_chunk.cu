@@ -143,7 +143,7 @@ __global__ void __launch_bounds__(256) lightning_chunk_prefix_kernel(const Light
   float4 S = *reinterpret_cast<const float4*>(p.state + static_cast<size_t>(p.state_in[seq]) * p.slot_stride + at);
   float4* sums = static_cast<float4*>(p.scratch) + (static_cast<size_t>(first) * p.heads + h) * cells + i;
   const size_t step = static_cast<size_t>(p.heads) * cells;
-  constexpr int kAhead = 8;
+  constexpr int kAhead = 16;
   for (int c0 = 0; c0 < chunks; c0 += kAhead) {
     float4 x[kAhead];
 #pragma unroll

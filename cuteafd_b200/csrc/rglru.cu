@@ -3,7 +3,7 @@
 //
 //   rglru_conv   biases and convolution; rows leave block by block, as the grouped product of the gates reads them
 //   rglru_scan   the gates' products to the output.  Short portions: one thread per channel walks a sequence's tokens.  Longer ones: a
-//                block owns 16 channels and walks 128 tokens at a time, every thread 8 of them; the threads' decays and contributions
+//                block owns 16 channels and walks 256 tokens at a time, every thread 8 of them; the threads' decays and contributions
 //                meet in shared memory, and each goes over its tokens again, still in registers, from the state before them
 //   rglru_step   all of it in one launch for steps of up to 32 rows: a block convolves one block's channels, multiplies 16 of them
 //                through both gates and walks their recurrences
@@ -259,9 +259,9 @@ __global__ void __launch_bounds__(kScanThreads) rglru_scan_kernel(const RglruArg
   p.state[static_cast<size_t>(p.state_out[seq]) * p.slot_stride + p.s_off + c] = S;
 }
 
-constexpr int kWalkChans = 16, kWalkSubs = 16, kWalkTok = 8, kWalk = kWalkSubs * kWalkTok, kWalkThreads = kWalkChans * kWalkSubs;
+constexpr int kWalkChans = 16, kWalkSubs = 32, kWalkTok = 8, kWalk = kWalkSubs * kWalkTok, kWalkThreads = kWalkChans * kWalkSubs;
 
-// Long portions: thread (channel, run of 8 of the 128 tokens the block is at).
+// Long portions: thread (channel, run of 8 of the 256 tokens the block is at).
 template <typename E>
 __global__ void __launch_bounds__(kWalkThreads) rglru_walk_kernel(const RglruArgs p) {
   __shared__ float2 part[2][kWalkSubs][kWalkChans];
