@@ -704,7 +704,7 @@ def buzarax_bench(size: str = "base") -> ModelConfig:
                         rope=RopeSpec(64, 1.0e6, 4.0, 1.0, 32.0, 8192, "yarn", halves=True), qk_norm="rotated", softcap=30.0, unit_sink=True,
                         v_rope=RopeSpec(128, 1.0e6, halves=True))
     lin = LightningSpec(heads=heads, dim=128, vdim=128, decay=tuple(1.0 - 2.0 ** (-1 - 8.0 * h / heads) for h in range(heads)))
-    pair, rec = PairSpec(att, lin, 0.8, 0.5), RglruSpec(width=width, blocks=width // 128, conv=4)
+    pair, rec = PairSpec(att, lin, 0.75, 0.6), RglruSpec(width=width, blocks=width // 128, conv=4)
     r = RouterSpec(experts=64, ffn=ffn, top=6, scoring="sigmoid")
     specs = [LayerSpec(rec if i % 2 else pair, r if i else None, None if i else DenseSpec(6 * ffn, 7.0, 1.702, 1.0), post_norm=True) for i in range(layers)]
     return post_norm_config(f"buzarax-{size}", 65536, width, specs, eps=1e-5, bigram=(65521, 31, 7), logit_softcap=30.0)

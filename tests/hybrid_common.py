@@ -183,10 +183,10 @@ def faint_config():
 def dual_config():
     """The sizes the tensor-core kernels take, and recurrences in blocks of 128."""
     return post_norm_config("dual", 500, 256, [
-        post(PairSpec(turned(4, 2, 128, 128, RopeSpec(64, 1e4, 4.0, 1.0, 32.0, 256, "yarn", halves=True), cap=6.0), fading(4, 128, 128, 0.7), 0.8, 0.5), 192),
+        post(PairSpec(turned(4, 2, 128, 128, RopeSpec(64, 1e4, 4.0, 1.0, 32.0, 256, "yarn", halves=True), cap=6.0), fading(4, 128, 128, 0.7), 0.9, 0.6), 192),
         post(RglruSpec(256, 2, 4), experts=8, top=2, expert_ffn=128),
         post(PairSpec(turned(8, 1, 128, 128, RopeSpec(128, 1e5, halves=True), cap=30.0), fading(2, 64, 64, 0.9, 0.999), 1.2, 0.7), experts=6, top=3, expert_ffn=64),
-        post(RglruSpec(384, 3, 2), 136, 2.0)], 1e-5, bigram=(211, 127, 7), logit_softcap=20.0)
+        post(RglruSpec(384, 3, 2), 136, 2.0)], 1e-5, bigram=(211, 113, 9), logit_softcap=20.0)
 
 
 def params(cfg, seed=0, spread=0.4):
