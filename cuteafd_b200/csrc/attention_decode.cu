@@ -14,7 +14,8 @@
 // row is complete: here without splits, in the merge with them.
 // A sliding window may come with kept first tokens; their pages are walked before the window's.  A head may have a sink, a number
 // whose exponential joins the softmax's denominator, and an output gate (the sigmoid of one number per token and head); both are
-// applied where a row is complete, and so is a rotation of the output back by the query's position.  Scores may be capped.
+// applied where a row is complete, and so is (kTurn) a rotation of the output back by the query's position.  kTurn: scores may be
+// capped.
 //
 // Reference counterparts: split-KV partial + merge drafter attention
 // (native/shared/cuda/draft_attention.cu:42-295) and the LSE state merge
@@ -84,12 +85,13 @@ struct AttnExtras {
   float cap_log2 = 0.f;                    // cap * log2(e): scores are cap * tanh(score / cap), and the kernel's scale is 2 log2(e) * scale / cap; 0 = none
 };
 
-// A complete row of one head: M is the maximum its sums L and O refer to, in log2 units.
+// kTurn: with cap_log2, v_table and out_scale.  A complete row of one head: M is the maximum its sums L and O refer to, in log2 units.
+template <bool kTurn>
 __device__ __forceinline__ float finish_row(float O, float L, float M, const AttnExtras& x, int row, int head) {
   if (x.sink) L += exp2f(x.sink[head] * 1.4426950408889634f - M);
   float v = L > 0.f ? O / L : 0.f;
   if (x.gate) v /= 1.0f + expf(-__bfloat162float(x.gate[static_cast<size_t>(row) * x.gate_ld + head]));
-  return v * x.out_scale;
+  return kTurn ? v * x.out_scale : v;
 }
 
 // One head's 128 values, one per thread, turned back by the row's angles (pairs 64 apart); every thread of the block calls.
@@ -114,7 +116,7 @@ __device__ __forceinline__ float combine_maps(float a, float b, const AttnExtras
   return o * (x.out_scale / sqrtf(tot * (1.0f / kD) + x.eps));
 }
 
-template <int kMaps>
+template <int kMaps, bool kTurn = false>
 __global__ void __launch_bounds__(128) attn_decode_kernel(
     const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __restrict__ k_cache,
     const __nv_bfloat16* __restrict__ v_cache, const int* __restrict__ page_table, const int* __restrict__ seq_lens,
@@ -237,7 +239,7 @@ __global__ void __launch_bounds__(128) attn_decode_kernel(
         const int half = j >> 1;
         const int tok = tok_base + nt * 8 + 2 * t4 + (j & 1);
         const float z = s[nt][j] * scale_log2;
-        const float v = (tok < limit[half] && (tok >= lo[half] || tok < ex.keep)) ? (ex.cap_log2 > 0.f ? ex.cap_log2 * tanh_exp2(z) : z) : -INFINITY;
+        const float v = (tok < limit[half] && (tok >= lo[half] || tok < ex.keep)) ? (kTurn && ex.cap_log2 > 0.f ? ex.cap_log2 * tanh_exp2(z) : z) : -INFINITY;
         s[nt][j] = v;
         mx[half] = fmaxf(mx[half], v);
       }
@@ -331,8 +333,8 @@ __global__ void __launch_bounds__(128) attn_decode_kernel(
           if ((r & 1) == 0) { o_map1 = v; continue; }
           v = combine_maps(o_map1, v, ex, sm_l + 64);
         } else {
-          v = finish_row(O, L, M, ex, q0 + qi, head);
-          if (ex.v_table) v = turn_back(v, ex, q0 + qi, sm_l + 128);
+          v = finish_row<kTurn>(O, L, M, ex, q0 + qi, head);
+          if (kTurn && ex.v_table) v = turn_back(v, ex, q0 + qi, sm_l + 128);
         }
         out[static_cast<size_t>(q0 + qi) * ex.ldo + head * kD + d] = __float2bfloat16(v);
       }
@@ -344,12 +346,12 @@ __global__ void __launch_bounds__(128) attn_decode_kernel(
 }
 
 // One block per (tile, kv head, row; with two maps row pair): thread d walks the splits in order for its output element.
-template <int kMaps>
+template <int kMaps, bool kTurn = false>
 __global__ void __launch_bounds__(128) attn_merge_kernel(const float* __restrict__ partial,
                                                          const int* __restrict__ q_start,
                                                          __nv_bfloat16* __restrict__ out, int Hq, int Hkv,
                                                          int tiles_per_seq, int splits, const AttnExtras ex) {
-  __shared__ float red[kMaps == 2 ? 4 : kD];
+  __shared__ float red[kTurn ? kD : 4];
   pdl_wait();
   pdl_trigger();
   const int group = Hq / Hkv;
@@ -373,9 +375,9 @@ __global__ void __launch_bounds__(128) attn_merge_kernel(const float* __restrict
       L += __ldg(base + s * kPartialFloats + 16 * kD + 16 + row) * f;
       O += __ldg(base + s * kPartialFloats + row * kD + d) * f;
     }
-    v[m] = kMaps == 1 ? finish_row(O, L, M, ex, q0 + qi, kvh * group + r % group) : L > 0.f ? O / L : 0.f;
+    v[m] = kMaps == 1 ? finish_row<kTurn>(O, L, M, ex, q0 + qi, kvh * group + r % group) : L > 0.f ? O / L : 0.f;
   }
-  const float o = kMaps == 2 ? combine_maps(v[0], v[kMaps - 1], ex, red) : ex.v_table ? turn_back(v[0], ex, q0 + qi, red) : v[0];
+  const float o = kMaps == 2 ? combine_maps(v[0], v[kMaps - 1], ex, red) : kTurn && ex.v_table ? turn_back(v[0], ex, q0 + qi, red) : v[0];
   out[static_cast<size_t>(q0 + qi) * ex.ldo + (kvh * group + r % group) * kD + d] = __float2bfloat16(o);
 }
 
@@ -422,13 +424,15 @@ extern "C" int cafd_attn_decode(const void* q, const void* k_cache, const void* 
   static bool attr = false;
   if (!attr) {
     CAFD_CHECK_CUDA(cudaFuncSetAttribute(attn_decode_kernel<1>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
+    CAFD_CHECK_CUDA(cudaFuncSetAttribute(attn_decode_kernel<1, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
     CAFD_CHECK_CUDA(cudaFuncSetAttribute(attn_decode_kernel<2>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
     attr = true;
   }
   dim3 grid(num_seqs * tiles_per_seq, Hkv, splits);
   const AttnExtras ex{window > 0 ? keep : 0, ldo, lambda, out_scale, eps, sink, static_cast<const __nv_bfloat16*>(gate), gate_ld,
                       static_cast<const float2*>(v_table), cap * 1.4426950408889634f};
-  auto kern = maps == 2 ? attn_decode_kernel<2> : attn_decode_kernel<1>;
+  const bool turn = maps == 1 && (cap > 0.f || v_table || out_scale != 1.f);
+  auto kern = maps == 2 ? attn_decode_kernel<2> : turn ? attn_decode_kernel<1, true> : attn_decode_kernel<1>;
   launch_pdl(kern, grid, dim3(128), smem, st,
       static_cast<const __nv_bfloat16*>(q), static_cast<const __nv_bfloat16*>(k_cache),
       static_cast<const __nv_bfloat16*>(v_cache), page_table, seq_lens, q_start, static_cast<__nv_bfloat16*>(out),
@@ -436,7 +440,7 @@ extern "C" int cafd_attn_decode(const void* q, const void* k_cache, const void* 
       window, fixed_kv_split_tokens() / kPage, AttnPeers{}, ex);
   if (splits > 1) {
     dim3 g2(num_seqs * tiles_per_seq, Hkv, 16 / maps);
-    auto merge = maps == 2 ? attn_merge_kernel<2> : attn_merge_kernel<1>;
+    auto merge = maps == 2 ? attn_merge_kernel<2> : turn ? attn_merge_kernel<1, true> : attn_merge_kernel<1>;
     launch_pdl(merge, g2, dim3(128), 0, st, scratch, q_start, static_cast<__nv_bfloat16*>(out), Hq, Hkv, tiles_per_seq, splits, ex);
   }
   return static_cast<int>(cudaGetLastError());

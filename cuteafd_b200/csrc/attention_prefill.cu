@@ -28,10 +28,10 @@
 //
 // A sliding window may come with kept first tokens, which every later row sees too: the tiles that hold them are walked
 // before the window's.  A head may have a sink (a number whose exponential joins the softmax's denominator) and an output gate
-// (the sigmoid of one number per token and head): both enter the epilogue's quotient; the output may be rotated back by the
-// query's position there.
+// (the sigmoid of one number per token and head): both enter the epilogue's quotient; with kTurn the output may be rotated back by
+// the query's position there.
 //
-// kCap: scores are cap * tanh(score / cap).  While every score of a warp's tile is small against the cap, tanh is an odd polynomial
+// kTurn: scores may be cap * tanh(score / cap), the output may be turned back.  While every score of a warp's tile is small against the cap, tanh is an odd polynomial
 // (two scores per instruction); else it takes an exponential and a division.
 //
 // Replaces the reference's mma.sync prefill kernels (native/families/glm5/cuda/glm_mla_prefill.cu:78-135)
@@ -71,7 +71,7 @@ struct PrefillDev {
   const __nv_bfloat16* gate;      // row t, head h: gate[t * gate_ld + h]; or null
   int gate_ld;
   const float2* v_table;          // [rows, 64] cos, sin; or null
-  float cap_in, cap_log2;         // kCap: scale / cap, cap * log2(e); scale_log2 is then 1
+  float cap_in, cap_log2;         // scale / cap, cap * log2(e); scale_log2 is then 1.  These two and v_table: kTurn only
   // kRope only
   const int* kv_tmp_start; // [seqs] first row of the sequence in the expansion buffers (multiple of 64)
   int q_head_stride;       // elements between heads in the nope query matrix (192 for [T, heads * 192])
@@ -127,7 +127,7 @@ __device__ __forceinline__ void cap_scores(uint32_t (&r)[64], float in, float ou
   }
 }
 
-template <bool kRope, int kMaps, bool kCap = false>
+template <bool kRope, int kMaps, bool kTurn = false>
 __global__ void __launch_bounds__(kPrefillThreads, 1)
 attn_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ CUtensorMap tm_k,
                     const __grid_constant__ CUtensorMap tm_v, const __grid_constant__ CUtensorMap tm_qr,
@@ -357,7 +357,9 @@ attn_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_const
       tmem_ld_wait();
       tc_fence_before();
       mbar_arrive(&s_empty[st]);
-      if constexpr (kCap) cap_scores(r, p.cap_in, p.cap_log2);
+      if constexpr (kTurn) {
+        if (p.cap_log2 > 0.f) cap_scores(r, p.cap_in, p.cap_log2);
+      }
       if (need_mask) {
 #pragma unroll
         for (int i = 0; i < 64; ++i)
@@ -493,8 +495,8 @@ attn_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_const
       if (p.sink) l_run += exp2f(p.sink[head] * 1.4426950408889634f - (m_run == -INFINITY ? 0.f : m_run));   // both halves hold the same maximum
       float inv = l_run > 0.f ? 1.0f / l_run : 0.f;
       if (p.gate && row_ok) inv /= 1.0f + expf(-__bfloat162float(p.gate[static_cast<size_t>(q0 + row0 + row) * p.gate_ld + head]));
-      if constexpr (!kRope) inv *= p.out_scale;
-      if (!kRope && p.v_table) {
+      if constexpr (kTurn) inv *= p.out_scale;
+      if (kTurn && p.v_table) {
         // values m and m + 64 turn together: this thread takes 32 of either half of the head
         uint32_t a[32], b[32];
         tmem_ld_32x32(tO + lane_off + half * 32, a);
@@ -609,7 +611,7 @@ extern "C" int cafd_attn_prefill(const void* q, const void* k_cache, const void*
   dim3 grid((max_q_len + kBQ - 1) / kBQ, Hq, num_seqs);
   cudaStream_t st = static_cast<cudaStream_t>(s);
   if (maps == 2) launch_pdl(attn_prefill_kernel<false, 2>, grid, dim3(kPrefillThreads), kPrefillSmem, st, tq, tk, tv, tq, tq, p);
-  else if (cap > 0.f) launch_pdl(attn_prefill_kernel<false, 1, true>, grid, dim3(kPrefillThreads), kPrefillSmem, st, tq, tk, tv, tq, tq, p);
+  else if (cap > 0.f || v_table || out_scale != 1.f) launch_pdl(attn_prefill_kernel<false, 1, true>, grid, dim3(kPrefillThreads), kPrefillSmem, st, tq, tk, tv, tq, tq, p);
   else launch_pdl(attn_prefill_kernel<false, 1>, grid, dim3(kPrefillThreads), kPrefillSmem, st, tq, tk, tv, tq, tq, p);
   return static_cast<int>(cudaGetLastError());
 }

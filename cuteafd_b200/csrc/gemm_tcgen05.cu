@@ -84,7 +84,8 @@ struct GemmCfg {
   static_assert(kWBytes % 1024 == 0 && kXBytes % 1024 == 0, "tiles must keep 1024-byte alignment");
 };
 
-template <bool kSwap, bool kDual, int kBX, int kBW>
+// kClip: the gated unit of a dual product is the clipped one.
+template <bool kSwap, bool kDual, int kBX, int kBW, bool kClip>
 __global__ void __launch_bounds__(kGemmThreads, 1)
 gemm_kernel(const __grid_constant__ CUtensorMap tm_w0, const __grid_constant__ CUtensorMap tm_w1,
             const __grid_constant__ CUtensorMap tm_x, const GemmDev p) {
@@ -304,12 +305,10 @@ gemm_kernel(const __grid_constant__ CUtensorMap tm_w0, const __grid_constant__ C
               uint32_t u[32];
               tmem_ld_32x32(t0 + kBW + c0 + 32 * h, u);
               tmem_ld_wait();
-              if (p.glu.kind == 0) {
 #pragma unroll
-                for (int j = 0; j < 32; ++j) v[j] = silu(__uint_as_float(r[j])) * __uint_as_float(u[j]) * scale;
-              } else {
-#pragma unroll
-                for (int j = 0; j < 32; ++j) v[j] = clipped_glu(__uint_as_float(r[j]), __uint_as_float(u[j]), p.glu) * scale;
+              for (int j = 0; j < 32; ++j) {
+                const float g = __uint_as_float(r[j]), uj = __uint_as_float(u[j]);
+                v[j] = (kClip ? clipped_glu(g, uj, p.glu) : silu(g) * uj) * scale;
               }
             } else {
               tmem_ld_wait();
@@ -407,7 +406,7 @@ gemm_kernel(const __grid_constant__ CUtensorMap tm_w0, const __grid_constant__ C
                 }
             }
 #pragma unroll
-            for (int j = 0; j < 16; ++j) v[j] = !kDual ? g[j] : p.glu.kind == 0 ? silu(g[j]) * u[j] : clipped_glu(g[j], u[j], p.glu);
+            for (int j = 0; j < 16; ++j) v[j] = !kDual ? g[j] : kClip ? clipped_glu(g[j], u[j], p.glu) : silu(g[j]) * u[j];
           } else {
             uint32_t r[16];
             tmem_ld_32x16(t0 + c0, r);
@@ -417,7 +416,7 @@ gemm_kernel(const __grid_constant__ CUtensorMap tm_w0, const __grid_constant__ C
               tmem_ld_wait();
 #pragma unroll
               for (int j = 0; j < 16; ++j)
-                v[j] = p.glu.kind == 0 ? silu(__uint_as_float(r[j])) * __uint_as_float(u[j]) : clipped_glu(__uint_as_float(r[j]), __uint_as_float(u[j]), p.glu);
+                v[j] = kClip ? clipped_glu(__uint_as_float(r[j]), __uint_as_float(u[j]), p.glu) : silu(__uint_as_float(r[j])) * __uint_as_float(u[j]);
             } else {
               tmem_ld_wait();
 #pragma unroll
@@ -479,7 +478,7 @@ gemm_kernel(const __grid_constant__ CUtensorMap tm_w0, const __grid_constant__ C
   }
 }
 
-template <bool kSwap, bool kDual, int kBX, int kBW>
+template <bool kSwap, bool kDual, int kBX, int kBW, bool kClip = false>
 static int launch(const cafd_gemm_args* a, cudaStream_t stream) {
   using Cfg = GemmCfg<kSwap, kDual, kBX, kBW>;
   CUtensorMap tw0, tw1, tx;
@@ -554,7 +553,7 @@ static int launch(const cafd_gemm_args* a, cudaStream_t stream) {
       grid = sms;
     }
   }
-  auto kern = gemm_kernel<kSwap, kDual, kBX, kBW>;
+  auto kern = gemm_kernel<kSwap, kDual, kBX, kBW, kClip>;
   static bool attr_set = false;
   if (!attr_set) {
     CAFD_CHECK_CUDA(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, Cfg::kSmemBytes));
@@ -574,6 +573,16 @@ extern "C" int cafd_gemm(const cafd_gemm_args* a, cafd_stream_t stream_) {
   if ((a->signal_flag || a->n_signal_flags) && (!a->done_counter || !a->epoch)) return -12;
   if (a->rs_ranks < 0 || a->rs_ranks > 8 || a->n_signal_flags < 0 || a->n_signal_flags > 8 || (a->rs_ranks && a->rs_rows_per_rank <= 0)) return -16;
   if (a->wait_flag && !a->epoch) return -12;
+  if (a->dual && a->glu) {
+    if (!a->swap) return launch<false, true, 128, 128, true>(a, stream);
+    switch (a->bx) {
+      case 16: return launch<true, true, 16, 128, true>(a, stream);
+      case 32: return launch<true, true, 32, 128, true>(a, stream);
+      case 64: return launch<true, true, 64, 128, true>(a, stream);
+      case 128: return launch<true, true, 128, 128, true>(a, stream);
+    }
+    return -13;
+  }
   if (a->swap) {
     if (a->dual) {
       switch (a->bx) {
